@@ -91,6 +91,10 @@ int rewb200_sync(int slot, int timeout_ms);
  *                                            the peer heap when its bulk region holds the step (default), or NCCL always
  *   "record_routing" = "0" | "1"             test aid: sessions created afterwards keep every MoE layer's top-k expert ids
  *                                            of their last forward for rewb200_session_routing
+ *   "record_layers" = "0" | "1"              test aid: layered models keep the residual stream after every layer run
+ *   "latent_attention" = "auto" | "plain" | "absorbed"   latent attention: keys and values expanded per head for large prompt
+ *                                            portions and the cached latents themselves otherwise (default); always the
+ *                                            plain kernels; always on the latents
  *   "inject_alloc_fail" = "n"                test hook: the n-th activation-buffer allocation from now fails on the host
  *   "moe_overlap" = "on" | "off"             MoE layers on one rank, steps of at most 64 rows: the shared experts run on a
  *                                            second stream beside the routed experts (default on)
@@ -271,6 +275,34 @@ int rewb200_qlora_linear(const rewb200_buffer* x, const rewb200_nf4* h, const re
 int rewb200_linear_noalloc(int slot, const void* x_bf16, const void* w_bf16, const float* bias, void* y_bf16,
                            int64_t M, int64_t K, int64_t N);
 
+/* ---- layered models ---------------------------------------------------------
+ * Decoders whose layers are described one by one (rewb200_model_create_layers): which mixer a layer has and its
+ * sizes, its feed-forward, and a range of layers that runs several times.  A layer is the parallel block
+ * x += mixer(norm1(x)) + ff(norm2(x)).  `mixer` 1 is latent attention: queries through a latent of q_rank, keys and
+ * values from a cached latent of kv_rank, a rotated key part of rot_dim shared by all heads, an optional sigmoid
+ * gate per head on the output, a sliding window. */
+typedef struct rewb200_layer {
+  int32_t mixer;        /* 1: latent attention */
+  int32_t heads, dim, rot_dim, vdim, q_rank, kv_rank;
+  int32_t window;       /* keys a query sees, itself included; 0: all before it */
+  int32_t rope_dims;    /* rotated features of the rot_dim part, interleaved pairs */
+  int32_t out_gate;     /* 1: head h's output is multiplied by sigmoid(g . input)_h */
+  int32_t ff;           /* 0 none, 1 dense gated SiLU, 2 routed experts */
+  int32_t ffn;          /* hidden width of the dense feed-forward or of one expert */
+  int32_t experts, top_k;
+  int32_t renormalize;  /* 1: routing weights divided by the sum of the chosen ones */
+  int32_t expert_gated; /* 1: gated SiLU experts, 0: W_down relu(W_up x)^2 */
+  double rope_base;
+  float scale;          /* of the attention scores */
+  int32_t reserved;
+} rewb200_layer;
+typedef struct rewb200_stack {
+  int32_t loop_start, loop_stop, loop_times; /* layers loop_start .. loop_stop - 1 run loop_times times (0: no loop);
+                                              * every pass has its own cache.  Before pass t the vector step[t] is added
+                                              * to x, before every pass but the first also the embedding output. */
+  int32_t norm_zero_centred;                 /* block and final norm weights are stored as the distance from one */
+} rewb200_stack;
+
 /* ---- model + generate ------------------------------------------------------
  * LlamaForCausalLM / DeepSeekForCausalLM (src/rew/models/llama.nim:13-44,
  * src/rew/models/deepseek.nim:20-63) as one object with fused device layouts. */
@@ -290,6 +322,13 @@ typedef struct rewb200_config {
 } rewb200_config;
 
 int rewb200_model_create(int slot, const rewb200_config* cfg, rewb200_model** out);
+/* A layered model: `cfg` gives vocab, d_model, n_layers, max_seq, eps and dtype (its other fields are ignored),
+ * `layers` n_layers descriptions.  The output head is the embedding table.  Canonical tensors (Linear weights
+ * [in, out], see rew_b200/layered.py): embed, step [times, d] (with a loop); per layer norm1, dq, dq.norm, uq, dkv,
+ * dkv.norm, uk, uv, g (with out_gate), o, then with a feed-forward norm2 and gate, up, down (dense) or router and per
+ * expert [gate,] up, down; final norm. */
+int rewb200_model_create_layers(int slot, const rewb200_config* cfg, const rewb200_layer* layers, const rewb200_stack* stack,
+                                rewb200_model** out);
 void rewb200_model_free(rewb200_model* m);
 /* Number and canonical order of the logical tensors (see rew_b200/weights.py):
  * embed; per layer ln1.gamma ln1.beta q.w q.b k.w k.b v.w v.b o.w o.b ln2.gamma
@@ -360,6 +399,16 @@ int rewb200_lane_admit(rewb200_session* s, int lane, const int32_t* ids, int S, 
  * [lanes,n_steps], -1 for idle lanes.  Fails without side effects when the pool
  * cannot cover the growth of every active lane ("out of free blocks"). */
 int rewb200_lanes_step(rewb200_session* s, int n_steps, int32_t* out_ids);
+/* One step over unequal portions: entry e appends counts[e] tokens (ids: all entries' tokens one after the other) to
+ * lane lanes[e], which is admitted by its first portion.  Prompt portions and single decoded tokens mix freely; a
+ * layered model runs all entries as one batch, a grouped-query model one entry after the other.  want (optional,
+ * n_want places in the concatenated tokens, ascending) asks for those positions' logits, host f32 [n_want, vocab].
+ * next_ids (optional, host int32 [n_entries]) asks for the token after every entry with sample[e] != 0 (sample NULL:
+ * all), chosen as rewb200_lanes_step would; it becomes the lane's next input there.  seeds as rewb200_lane_admit,
+ * one per entry, or NULL.  Fails without side effects when the pool cannot hold the step. */
+int rewb200_lanes_feed(rewb200_session* s, int n_entries, const int32_t* lanes, const int32_t* counts, const int32_t* ids,
+                       int n_want, const int32_t* want, float* logits_out, const int32_t* sample, const uint64_t* seeds,
+                       int32_t* next_ids);
 /* Ends a lane's sequence and returns its blocks to the pool (idempotent). */
 int rewb200_lane_release(rewb200_session* s, int lane);
 
@@ -389,6 +438,9 @@ int rewb200_session_graph_kernels(const rewb200_session* s);
 /* Test aid (option record_routing): the expert ids MoE layer `moe_layer` (0-based among the MoE layers) chose for
  * the `rows` tokens of the session's last forward, host int32 [rows, top_k], in the router's order. */
 int rewb200_session_routing(rewb200_session* s, int moe_layer, int32_t* topi_out, int64_t rows);
+/* Layered models: the residual stream after every layer run of the session's last step that was not a captured
+ * decode, host f32 [layer_runs, rows, d_model] (test aid; option record_layers). */
+int rewb200_session_layers(rewb200_session* s, float* out, int64_t rows);
 /* Measurement aid: one decode step issued as plain launches with a CUDA event after every category of
  * launches; ms_by_category (host, n >= 11 floats) receives the device time per category, summed over the
  * layers: 0 embedding + first norm, 1 q|k|v Linear, 2 bias + RoPE + cache write, 3 attention, 4 o Linear,

@@ -30,6 +30,18 @@ class Config(C.Structure):
     ]
 
 
+class Layer(C.Structure):
+    """struct rewb200_layer"""
+    _fields_ = [(n, C.c_int32) for n in ("mixer", "heads", "dim", "rot_dim", "vdim", "q_rank", "kv_rank", "window", "rope_dims",
+                                         "out_gate", "ff", "ffn", "experts", "top_k", "renormalize", "expert_gated")] + [
+        ("rope_base", C.c_double), ("scale", C.c_float), ("reserved", C.c_int32)]
+
+
+class Stack(C.Structure):
+    """struct rewb200_stack"""
+    _fields_ = [(n, C.c_int32) for n in ("loop_start", "loop_stop", "loop_times", "norm_zero_centred")]
+
+
 _lib = None
 
 P = C.c_void_p
@@ -65,6 +77,7 @@ SIGNATURES = {
     "rewb200_moe_route": (C.c_int, [P, P, P, C.c_int, PP, PP]),
     "rewb200_linear_noalloc": (C.c_int, [C.c_int, P, P, P, P, C.c_int64, C.c_int64, C.c_int64]),
     "rewb200_model_create": (C.c_int, [C.c_int, C.POINTER(Config), PP]),
+    "rewb200_model_create_layers": (C.c_int, [C.c_int, C.POINTER(Config), C.POINTER(Layer), C.POINTER(Stack), PP]),
     "rewb200_model_free": (None, [P]),
     "rewb200_model_tensor_count": (C.c_int64, [P]),
     "rewb200_model_set_tensor": (C.c_int, [P, C.c_int64, F32P, C.c_int64]),
@@ -90,6 +103,7 @@ SIGNATURES = {
     "rewb200_lane_length": (C.c_int, [P, C.c_int]),
     "rewb200_lane_admit": (C.c_int, [P, C.c_int, I32P, C.c_int, C.c_uint64, I32P]),
     "rewb200_lanes_step": (C.c_int, [P, C.c_int, I32P]),
+    "rewb200_lanes_feed": (C.c_int, [P, C.c_int, I32P, I32P, I32P, C.c_int, I32P, F32P, I32P, C.POINTER(C.c_uint64), I32P]),
     "rewb200_lane_release": (C.c_int, [P, C.c_int]),
     "rewb200_session_set_sampling": (C.c_int, [P, C.c_float, C.c_int, C.c_float, C.c_float, C.c_float, C.c_int,
                                                C.POINTER(C.c_uint64)]),
@@ -98,6 +112,7 @@ SIGNATURES = {
     "rewb200_session_last_ms": (C.c_int, [P, F32P, F32P]),
     "rewb200_session_graph_kernels": (C.c_int, [P]),
     "rewb200_session_routing": (C.c_int, [P, C.c_int, I32P, C.c_int64]),
+    "rewb200_session_layers": (C.c_int, [P, F32P, C.c_int64]),
     "rewb200_session_trace_step": (C.c_int, [P, F32P, C.c_int]),
     "rewb200_session_profile_linears": (C.c_int, [P, C.c_int, F32P, I64P, I32P]),
     "rewb200_model_forward_all": (C.c_int, [P, I32P, C.c_int, C.c_int64, C.c_int, F32P]),

@@ -16,7 +16,8 @@ import numpy as np
 
 from . import _lib
 from ._lib import BF16, F32, I32, RewB200Error, check, lib
-from .weights import ModelConfig, from_bf16_bits, tensor_specs, to_bf16_bits
+from .layered import LayeredConfig
+from .weights import from_bf16_bits, tensor_specs, to_bf16_bits
 
 _NP = {F32: np.float32, I32: np.int32, _lib.I64: np.int64, _lib.F64: np.float64, _lib.U8: np.uint8,
        _lib.BOOL: np.bool_, _lib.I8: np.int8, _lib.I16: np.int16}
@@ -346,14 +347,17 @@ def dispatch(op, operands, attrs=()):
 
 
 class CausalLM:
-    """LlamaForCausalLM / DeepSeekForCausalLM on the device."""
+    """LlamaForCausalLM / DeepSeekForCausalLM (ModelConfig) or a layered model (LayeredConfig) on the device."""
 
-    def __init__(self, cfg: ModelConfig, slot=0):
+    def __init__(self, cfg, slot=0):
         _lib.init()
         self.cfg = cfg
-        self._c = cfg.to_c()
         h = C.c_void_p()
-        check(lib().rewb200_model_create(slot, C.byref(self._c), C.byref(h)))
+        if isinstance(cfg, LayeredConfig):
+            cfg.create(slot, C.byref(h))
+        else:
+            self._c = cfg.to_c()
+            check(lib().rewb200_model_create(slot, C.byref(self._c), C.byref(h)))
         self._h = h
         self._sessions = weakref.WeakSet()  # sessions point into the model: they are freed first
 
@@ -493,6 +497,13 @@ class Session:
         check(lib().rewb200_session_routing(self._h, moe_layer, out.ctypes.data_as(_lib.I32P), rows))
         return out
 
+    def layers(self, rows):
+        """The residual stream [layer runs, rows, d_model] of a layered model's last step (needs option record_layers=1)."""
+        cfg = self.model.cfg
+        out = np.empty((len(cfg.layer_runs), rows, cfg.d_model), np.float32)
+        check(lib().rewb200_session_layers(self._h, out.ctypes.data_as(_lib.F32P), rows))
+        return out
+
     TRACE_CATEGORIES = ("embed_norm", "qkv_linear", "qkv_post", "attention", "o_linear", "norm_after_attention",
                         "gate_up_linear", "down_linear", "routed_experts", "norm_after_ffn", "head_and_next_token")
 
@@ -580,6 +591,27 @@ class PagedSession(Session):
         out = np.empty((self.batch, n_steps), np.int32)
         check(lib().rewb200_lanes_step(self._h, n_steps, out.ctypes.data_as(_lib.I32P)))
         return out
+
+    def feed(self, portions, want=(), sample=None, seeds=None):
+        """One step over unequal portions.  portions: [(lane, ids)], prompt portions and single decoded tokens alike;
+        a lane is admitted by its first portion.  want: places in the concatenated tokens whose logits are returned.
+        sample: None (choose no token), True (after every portion), or one flag per portion.
+        Returns (logits [len(want), vocab], next ids [len(portions)], -1 where none was chosen)."""
+        n = len(portions)
+        arrs = [np.ascontiguousarray(t, dtype=np.int32).reshape(-1) for _, t in portions]
+        lanes = (C.c_int32 * n)(*[int(l) for l, _ in portions])
+        counts = (C.c_int32 * n)(*[a.size for a in arrs])
+        ids = np.ascontiguousarray(np.concatenate(arrs)) if n else np.empty(0, np.int32)
+        w = np.ascontiguousarray(list(want), dtype=np.int32)
+        logits = np.empty((w.size, self.model.cfg.vocab), np.float32)
+        nxt = np.full(n, -1, np.int32)
+        flags = None if sample is None or sample is True else (C.c_int32 * n)(*[int(bool(f)) for f in sample])
+        sd = None if seeds is None else (C.c_uint64 * n)(*[int(v) for v in seeds])
+        check(lib().rewb200_lanes_feed(self._h, n, lanes, counts, ids.ctypes.data_as(_lib.I32P), int(w.size),
+                                       w.ctypes.data_as(_lib.I32P) if w.size else None,
+                                       logits.ctypes.data_as(_lib.F32P) if w.size else None, flags, sd,
+                                       nxt.ctypes.data_as(_lib.I32P) if sample is not None else None))
+        return logits, nxt
 
     def release(self, lane):
         check(lib().rewb200_lane_release(self._h, lane))

@@ -74,6 +74,8 @@ struct Ctx {
   bool nf4_small = false;       // NF4 GEMV of up to four rows on the CUDA-core streamer instead of the tensor-core kernel (measured slower: off)
   bool tp_twoshot = true;       // tensor-parallel steps above 64 rows: sum over the peer heap (two-shot) instead of NCCL
   bool record_routing = false;  // sessions keep every MoE layer's top-k expert ids of their last forward (a test aid)
+  bool record_layers = false;   // layered models keep the residual stream after every layer run (a test aid)
+  int latent_impl = 0;          // latent attention: 0 by step size, 1 plain kernels, 2 always on the cached latents
   int inject_alloc_fail = 0;  // test hook: the n-th activation allocation from now fails on the host
   int option_epoch = 0;      // bumped by rewb200_set_option; captured graphs from older epochs are rebuilt
   void* pinned = nullptr;    // pinned host staging for H2D/D2H of buffers
@@ -188,6 +190,7 @@ enum Epilogue : int {
   EPI_BIAS_F32 = 1,     // out_f32[row][col] = acc + bias[col]
   EPI_BIAS_BF16 = 2,    // out_bf16[row][col] = acc + bias[col]
   EPI_SWIGLU_BF16 = 3,  // columns interleaved gate/up in groups of 8: out[row][col/2..] = silu(g+bg)*(u+bu)
+  EPI_RELU2_BF16 = 4,   // out_bf16[row][col] = max(acc + bias[col], 0)^2
 };
 
 struct LinearBf16Plan {
@@ -219,6 +222,9 @@ int linear_bf16_pick_ksplit(Ctx* c, int64_t M, int64_t K, int64_t N);
 // f32 path: C[M,N] = A[M,K] @ B[K,N] (+ bias[N]).
 int gemm_f32_launch(Ctx* c, const float* A, const float* B, const float* bias, float* C, int64_t M, int64_t K,
                     int64_t N);
+// The same with row strides (elements) for operands whose rows are padded.
+int gemm_f32_ld_launch(Ctx* c, const float* A, int64_t lda, const float* B, int64_t ldb, const float* bias, float* C, int64_t ldc,
+                       int64_t M, int64_t K, int64_t N);
 
 struct NormArgs {
   float* x_res;           // [rows,d] residual stream (in/out)
@@ -261,6 +267,14 @@ struct NormArgs {
   int64_t slot_lines;     // lines between two writers' slots
   const int* epoch;       // device counter, advanced once per forward on every rank alike
   int barrier_offset;
+  // Blocks whose branches read two norms of one x, and stacks that run a range of layers several times:
+  const float* partial2;  // a second set of f32 slabs added like `partial` (same split_stride), or nullptr
+  int nsplit2;
+  const float* gamma2;    // a second RMS norm of the same row: out2 = gamma2 * x / rms, or nullptr
+  void* out2;
+  int add_embed;          // 1: the embedding row of ids[row] is ADDED to the residual instead of replacing it
+  const float* add_vec;   // [d] f32 added to every row, or nullptr
+  int64_t d_mean;         // width the row statistics divide by when rows are padded (0: d); the padding is zero
 };
 int residual_norm_launch(Ctx* c, const NormArgs& a, int64_t rows);
 

@@ -80,26 +80,33 @@ __global__ void __launch_bounds__(NORM_THREADS) residual_norm_kernel(NormArgs a)
     erow = reinterpret_cast<const TE*>(a.embed) + id * d;
   }
   for (int64_t i = threadIdx.x; i < d; i += NORM_THREADS, ++cnt) {
-    float v = erow ? to_f<TE>(erow[i]) : xr[i];  // x_res is required when there is no table
+    float v = erow && !a.add_embed ? to_f<TE>(erow[i]) : xr[i];  // x_res is required when there is no table
     if (a.partial) {
       float p = 0.f;
       for (int s = 0; s < a.nsplit; ++s) p += a.partial[s * a.split_stride + row * d + i];
+      for (int s = 0; s < a.nsplit2; ++s) p += a.partial2[s * a.split_stride + row * d + i];
       if (a.bias) p += a.bias[i];
       v += p;
     }
+    if (erow && a.add_embed) v += to_f<TE>(erow[i]);
+    if (a.add_vec) v += a.add_vec[i];
     vals[cnt] = v;
-    if (a.x_res && (erow || a.partial)) xr[i] = v;
+    if (a.x_res && (erow || a.partial || a.add_vec)) xr[i] = v;
   }
   if (a.norm_kind < 0) return;
   TO* orow = reinterpret_cast<TO*>(a.out) + row * d;
+  const float dm = (float)(a.d_mean > 0 ? a.d_mean : d);
   if (a.norm_kind == 0) {
     float ss = 0.f;
     for (int k = 0; k < cnt; ++k) ss += vals[k] * vals[k];
     ss = block_sum(ss, red);
-    const float rms = sqrtf(ss / (float)d + a.eps);
+    const float rms = sqrtf(ss / dm + a.eps);
     cnt = 0;
-    for (int64_t i = threadIdx.x; i < d; i += NORM_THREADS, ++cnt)
-      orow[i] = from_f<TO>(a.gamma[i] * (vals[cnt] / rms));
+    for (int64_t i = threadIdx.x; i < d; i += NORM_THREADS, ++cnt) {
+      const float u = vals[cnt] / rms;
+      orow[i] = from_f<TO>(a.gamma[i] * u);
+      if (a.gamma2) reinterpret_cast<TO*>(a.out2)[row * d + i] = from_f<TO>(a.gamma2[i] * u);
+    }
   } else {
     float s1 = 0.f;
     for (int k = 0; k < cnt; ++k) s1 += vals[k];
@@ -172,6 +179,16 @@ __device__ __forceinline__ float4 partial_sum4(const NormArgs& a, int64_t idx) {
     const float4 p0 = *reinterpret_cast<const float4*>(pp + s * a.split_stride);
     p.x += p0.x; p.y += p0.y; p.z += p0.z; p.w += p0.w;
   }
+  return p;
+}
+
+// What a block with two branches, or a stack that runs layers several times, adds on top (NormArgs::partial2,
+// add_embed, add_vec) at column i of a row; idx = row * d + i.
+__device__ __forceinline__ void add4(float4& v, const float4 w) { v.x += w.x; v.y += w.y; v.z += w.z; v.w += w.w; }
+__device__ __forceinline__ float4 partial2_sum4(const NormArgs& a, int64_t idx) {
+  float4 p = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 4
+  for (int s = 0; s < a.nsplit2; ++s) add4(p, *reinterpret_cast<const float4*>(a.partial2 + s * a.split_stride + idx));
   return p;
 }
 
@@ -366,16 +383,19 @@ __global__ void __launch_bounds__(NORMV_THREADS) residual_norm_vec_kernel(NormAr
     const int64_t i = ((int64_t)c * NORMV_THREADS + threadIdx.x) * 4;
     float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
     if (i < d) {
-      v = erow ? Vec4<TE>::load(erow + i) : *reinterpret_cast<const float4*>(xr + i);
+      v = erow && !a.add_embed ? Vec4<TE>::load(erow + i) : *reinterpret_cast<const float4*>(xr + i);
       if (summed) {
         float4 p = vals[c];
+        if (a.nsplit2 > 0) add4(p, partial2_sum4(a, row * d + i));
         if (a.bias) {
           const float4 b = *reinterpret_cast<const float4*>(a.bias + i);
           p.x += b.x; p.y += b.y; p.z += b.z; p.w += b.w;
         }
         v.x += p.x; v.y += p.y; v.z += p.z; v.w += p.w;
       }
-      if (a.x_res && (erow || summed)) *reinterpret_cast<float4*>(xr + i) = v;
+      if (erow && a.add_embed) add4(v, Vec4<TE>::load(erow + i));
+      if (a.add_vec) add4(v, *reinterpret_cast<const float4*>(a.add_vec + i));
+      if (a.x_res && (erow || summed || a.add_vec)) *reinterpret_cast<float4*>(xr + i) = v;
     }
     vals[c] = v;
   }
@@ -387,7 +407,7 @@ __global__ void __launch_bounds__(NORMV_THREADS) residual_norm_vec_kernel(NormAr
 #pragma unroll
     for (int c = 0; c < NCH; ++c) ss += vals[c].x * vals[c].x + vals[c].y * vals[c].y + vals[c].z * vals[c].z + vals[c].w * vals[c].w;
     ss = block_sum(ss, red);
-    scale = sqrtf(ss / (float)d + a.eps);  // rmsNorm divides by this
+    scale = sqrtf(ss / (float)(a.d_mean > 0 ? a.d_mean : d) + a.eps);  // rmsNorm divides by this
   } else {
     float s1 = 0.f;
 #pragma unroll
@@ -412,8 +432,12 @@ __global__ void __launch_bounds__(NORMV_THREADS) residual_norm_vec_kernel(NormAr
     const float4 g = *reinterpret_cast<const float4*>(a.gamma + i);
     float4 o;
     if (a.norm_kind == 0) {
-      o.x = g.x * (vals[c].x / scale); o.y = g.y * (vals[c].y / scale);
-      o.z = g.z * (vals[c].z / scale); o.w = g.w * (vals[c].w / scale);
+      const float4 u = make_float4(vals[c].x / scale, vals[c].y / scale, vals[c].z / scale, vals[c].w / scale);
+      o.x = g.x * u.x; o.y = g.y * u.y; o.z = g.z * u.z; o.w = g.w * u.w;
+      if (a.gamma2) {
+        const float4 g2 = *reinterpret_cast<const float4*>(a.gamma2 + i);
+        Vec4<TO>::store(reinterpret_cast<TO*>(a.out2) + row * d + i, make_float4(g2.x * u.x, g2.y * u.y, g2.z * u.z, g2.w * u.w));
+      }
     } else {
       const float4 b = *reinterpret_cast<const float4*>(a.beta + i);
       o.x = g.x * ((vals[c].x - mean) * scale) + b.x; o.y = g.y * ((vals[c].y - mean) * scale) + b.y;
@@ -458,7 +482,7 @@ __global__ void __cluster_dims__(4, 1, 1) __launch_bounds__(256) residual_norm_c
   for (int c = 0; c < NCH; ++c) {
     const int64_t off = ((int64_t)c * 256 + threadIdx.x) * 4;
     xin[c] = make_float4(0.f, 0.f, 0.f, 0.f);
-    if (off < dq) xin[c] = erow ? Vec4<TE>::load(erow + col0 + off) : *reinterpret_cast<const float4*>(xr + col0 + off);
+    if (off < dq) xin[c] = erow && !a.add_embed ? Vec4<TE>::load(erow + col0 + off) : *reinterpret_cast<const float4*>(xr + col0 + off);
   }
   if (summed) {
     int64_t idx[NCH];
@@ -482,13 +506,16 @@ __global__ void __cluster_dims__(4, 1, 1) __launch_bounds__(256) residual_norm_c
       v = xin[c];
       if (summed) {
         float4 p = vals[c];
+        if (a.nsplit2 > 0) add4(p, partial2_sum4(a, row * d + i));
         if (a.bias) {
           const float4 b = *reinterpret_cast<const float4*>(a.bias + i);
           p.x += b.x; p.y += b.y; p.z += b.z; p.w += b.w;
         }
         v.x += p.x; v.y += p.y; v.z += p.z; v.w += p.w;
       }
-      if (a.x_res && (erow || summed)) *reinterpret_cast<float4*>(xr + i) = v;
+      if (erow && a.add_embed) add4(v, Vec4<TE>::load(erow + i));
+      if (a.add_vec) add4(v, *reinterpret_cast<const float4*>(a.add_vec + i));
+      if (a.x_res && (erow || summed || a.add_vec)) *reinterpret_cast<float4*>(xr + i) = v;
     }
     vals[c] = v;
   }
@@ -507,7 +534,7 @@ __global__ void __cluster_dims__(4, 1, 1) __launch_bounds__(256) residual_norm_c
     float ss = 0.f;
 #pragma unroll
     for (int c = 0; c < NCH; ++c) ss += vals[c].x * vals[c].x + vals[c].y * vals[c].y + vals[c].z * vals[c].z + vals[c].w * vals[c].w;
-    scale = sqrtf(row_sum(ss, 0) / (float)d + a.eps);  // rmsNorm divides by this
+    scale = sqrtf(row_sum(ss, 0) / (float)(a.d_mean > 0 ? a.d_mean : d) + a.eps);  // rmsNorm divides by this
   } else {
     float s1 = 0.f;
 #pragma unroll
@@ -532,8 +559,12 @@ __global__ void __cluster_dims__(4, 1, 1) __launch_bounds__(256) residual_norm_c
     const float4 g = *reinterpret_cast<const float4*>(a.gamma + i);
     float4 o;
     if (a.norm_kind == 0) {
-      o.x = g.x * (vals[c].x / scale); o.y = g.y * (vals[c].y / scale);
-      o.z = g.z * (vals[c].z / scale); o.w = g.w * (vals[c].w / scale);
+      const float4 u = make_float4(vals[c].x / scale, vals[c].y / scale, vals[c].z / scale, vals[c].w / scale);
+      o.x = g.x * u.x; o.y = g.y * u.y; o.z = g.z * u.z; o.w = g.w * u.w;
+      if (a.gamma2) {
+        const float4 g2 = *reinterpret_cast<const float4*>(a.gamma2 + i);
+        Vec4<bf16>::store(reinterpret_cast<bf16*>(a.out2) + row * d + i, make_float4(g2.x * u.x, g2.y * u.y, g2.z * u.z, g2.w * u.w));
+      }
     } else {
       const float4 b = *reinterpret_cast<const float4*>(a.beta + i);
       o.x = g.x * ((vals[c].x - mean) * scale) + b.x; o.y = g.y * ((vals[c].y - mean) * scale) + b.y;
@@ -1005,6 +1036,7 @@ int residual_norm_launch(Ctx* c, const NormArgs& a, int64_t rows) {
                                 rows * a.d / (a.payload_bf16 ? 4 : 2) <= a.slot_lines),
              "the fused all-reduce needs d_model % 4 == 0, local partials, at most 64 rows and a slot that holds the step");
   RB_REQUIRE(!a.partial_bf16 || a.d % 4 == 0, "bf16 partials need d_model % 4 == 0");
+  RB_REQUIRE(a.norm_kind <= 0 || (!a.gamma2 && a.d_mean == 0), "a second norm output and padded rows are for the RMS norm only");
   if (o16 && a.norm_kind >= 0 && rows <= 64 && a.d % 16 == 0 && a.d <= 16384 && c->norm_cluster) {
     const int nch = (int)((a.d / 16 + 255) / 256);  // float4 per thread over a quarter row
     dim3 g((unsigned)(rows * 4)), b(256);

@@ -17,86 +17,13 @@
 //     captured once into a CUDA graph and replayed; token ids, positions and
 //     the step counter live on the device, so a run of n steps needs no host
 //     round trip until the ids are copied back.
-#include <algorithm>
-#include <cstring>
-
-#include "common.cuh"
-#include "ptx.cuh"
+#include "engine.cuh"
 
 using namespace rewb;
 
 namespace rewb {
 
-int comm_world(int slot);
-int comm_rank(int slot);
-int comm_allreduce_sum(Ctx* c, int slot, void* ptr, int64_t n, int dtype);
-int comm_allgather_bytes(Ctx* c, int slot, const void* send, void* recv, size_t bytes_per_rank);
-int comm_check_async(int slot);
-int slab_sum_launch(Ctx* c, float* part, int nsplit, int64_t slab_elems);
-int epoch_bump_launch(Ctx* c, int* epoch, int by);
-int comm_alltoall_bytes(Ctx* c, int slot, const void* send, void* recv, size_t bytes_per_peer);
-int comm_alltoallv_rows(Ctx* c, int slot, const void* send, void* recv, size_t peer_stride_bytes, size_t row_bytes,
-                        const int* send_rows, const int* recv_rows);
-int moe_route_launch(Ctx* c, const float* logits, int64_t N, int E, int k, float* topw, int* topi);
-int moe_route_slabs_launch(Ctx* c, const float* logits, int nsplit, int64_t split_stride, const float* bias, int64_t N, int E,
-                           int k, float* topw, int* topi, int* zero, int n_zero);
-int moe_group_local_launch(Ctx* c, const void* x, int dtype, const int* topi, int64_t tokens, int k, int64_t d, int n_experts,
-                           int* offsets, void* xs, int* pair_pos);
-int moe_reset_launch(Ctx* c, int* cursor, int n_cursor, int* count, int n_count, int* meta, int n_meta);
-int moe_dispatch_launch(Ctx* c, const void* x, int dtype, const int* topi, int64_t tokens, int k, int64_t d,
-                        int experts_per_rank, int capacity, int* cursor, void* send_x, int* send_meta, int* pair_slot);
-int moe_group_launch(Ctx* c, const void* recv_x, int dtype, const int* recv_meta, int n_slots, int64_t d, int n_experts,
-                     int* count, int* offsets, int* cursor2, void* xs, int* slot_pos);
-int moe_return_launch(Ctx* c, const float* ys, const int* slot_pos, int n_slots, int64_t d, float* ret);
-int moe_combine_launch(Ctx* c, const float* back, const int* pair_slot, const float* topw, int64_t tokens, int k, int64_t d,
-                       float* out, int accumulate);
-int moe_dispatch_peer_launch(Ctx* c, const void* x, int dtype, const int* topi, int64_t tokens, int k, int64_t d,
-                             int experts_per_rank, int capacity, int* cursor, int* pair_slot, const A2aArgs& a);
-int moe_group_peer_launch(Ctx* c, int dtype, int n_slots, int capacity, int64_t d, int n_experts, int* count, int* offsets,
-                          int* cursor2, void* xs, int* slot_pos, const A2aArgs& a);
-int moe_return_peer_launch(Ctx* c, const float* ys, const int* slot_pos, int n_slots, int capacity, int64_t d, const A2aArgs& a);
-int moe_combine_peer_launch(Ctx* c, const int* pair_slot, const float* topw, int64_t tokens, int k, int64_t d, float* out,
-                            int accumulate, const A2aArgs& a);
-int sample_launch(Ctx* c, const float* logits, float* work, int64_t B, int64_t V, int* hist, int* hist_len, int hist_cap,
-                  uint32_t* keys, int* steps, int* next, float* logprob, int logprob_cap, float temperature, int top_k,
-                  float top_p, float min_p, float rep_penalty, int do_sample, const int* active);
-int argmax_partial_launch(Ctx* c, const float* logits, int64_t rows, int64_t V, int idx_offset, int nchunks, float* pv, int* pi);
-int argmax_gathered_launch(Ctx* c, const void* gathered, int world, int64_t rows, int nchunks, int* out);
-
 namespace {
-
-constexpr int PAGE = 64;
-
-struct LinW {
-  void* w = nullptr;   // [K,N] model dtype (for a quantised Linear: the shared dequantisation scratch)
-  float* b = nullptr;  // [N]
-  int64_t K = 0, N = 0;
-  LinearBf16Plan plan;
-  bool quant = false;  // weight held as NF4 codes
-  Nf4W nf4;
-  ColMap cm = {1, 1, 1, 0};  // logical column (the reference's [in,out]) -> device column of `w`
-};
-
-// Routed experts of one DeepSeekMoE layer held by this rank (src/rew/models/deepseek.nim:36-52).
-struct MoeDev {
-  LinW router;                 // gate: [d, n_routed]
-  void* gu = nullptr;          // [E_l][d][2f]  gate|up per expert (bf16: interleaved in groups of 8)
-  float* gu_b = nullptr;       // [E_l][2f]
-  void* down = nullptr;        // [E_l][f][d]
-  float* down_b = nullptr;     // [E_l][d]
-  LinearBf16Plan plan_gu, plan_down;
-  int E_l = 0;
-  int64_t f = 0;
-  std::vector<float> shared_down_bias;  // sum of the shared experts' down biases (uploaded at finalize)
-};
-
-struct LayerDev {
-  float *ln1g = nullptr, *ln1b = nullptr, *ln2g = nullptr, *ln2b = nullptr;
-  LinW qkv, o, gu, down;       // for a MoE layer gu/down are the fused SHARED experts (width n_shared * moe_ffn)
-  int64_t ffn_local = 0;
-  bool moe = false;
-  MoeDev x;
-};
 
 // f32 path: out[t] (+)= w_e(t) * y[t], w_e(t) = sum_j topw[t][j] * (topi[t][j] == e)
 // (routedWeightForExpert, src/rew/models/deepseek.nim:114-120,140-144)
@@ -131,6 +58,14 @@ __global__ void swiglu_rows_f32_kernel(const float* gu, float* out, int64_t rows
   const float x = gu[r * 2 * f + c];
   const float sig = 1.0f / (1.0f + expf(-x));
   out[i] = (x * sig) * gu[r * 2 * f + f + c];
+}
+
+// f32 path: out = max(x, 0)^2
+__global__ void relu2_f32_kernel(const float* x, float* out, int64_t n) {
+  const int64_t i = (int64_t)blockIdx.x * blockDim.x + threadIdx.x;
+  if (i >= n) return;
+  const float v = fmaxf(x[i], 0.f);
+  out[i] = v * v;
 }
 
 // Quantised gate|up: sums the split-K slabs of the LOGICAL [rows][gate(f) | up(f)] projection, adds the
@@ -216,88 +151,7 @@ __global__ void advance_kernel(const int* next, int* ids, int* pos, int* out_ids
 }  // namespace
 }  // namespace rewb
 
-struct rewb200_model {
-  Ctx* c = nullptr;
-  int slot = 0;
-  rewb200_config cfg;
-  int nh_l = 0, kvh_l = 0;      // local heads under tensor parallelism
-  int64_t vocab_l = 0;          // local slice of the vocabulary (lm_head is vocab-parallel)
-  int64_t nq = 0, nkv = 0, nqkv = 0;
-  void* embed = nullptr;
-  std::vector<LayerDev> layers;
-  float *ng = nullptr, *nb = nullptr;
-  LinW lm;
-  float *cosT = nullptr, *sinT = nullptr;
-  float* stage = nullptr;       // f32 upload staging
-  size_t stage_bytes = 0;
-  bool finalized = false;
-  int64_t weight_bytes = 0;
-  std::vector<void*> allocs;
-};
-
-struct rewb200_session {
-  rewb200_model* m = nullptr;
-  int B = 0, max_len = 0, max_pages = 0;
-  std::vector<void*> kc, vc;           // per layer
-  std::vector<CUtensorMap> tmK, tmV;   // per layer (bf16)
-  int* block_table = nullptr;
-  int *d_pos = nullptr, *d_ids = nullptr, *d_next = nullptr, *d_out = nullptr, *d_step = nullptr;
-  int out_capacity = 0;
-  int32_t* h_ids = nullptr;            // pinned
-  // activations, sized for `rows_cap` rows
-  int64_t rows_cap = 0;
-  float* x_res = nullptr;
-  void* xn = nullptr;
-  void* q = nullptr;
-  void* attn = nullptr;
-  void* h = nullptr;
-  float* part = nullptr;               // split-K partials (largest user)
-  size_t part_bytes = 0;
-  float* gu32 = nullptr;               // f32 path: gate|up GEMM output
-  float* logits = nullptr;             // [B or rows][V]
-  int64_t logits_rows = 0;
-  float* attn_scratch = nullptr;
-  size_t attn_scratch_bytes = 0;
-  void* argmax_scratch = nullptr;      // [B][64] (value, index) partials
-  void* gather_scratch = nullptr;      // tensor parallel: all-gathered argmax partials / logits
-  size_t gather_bytes = 0;
-  // MoE scratch, sized for rows_cap tokens (capacity = tokens * top_k slots per peer)
-  float* moe_logits = nullptr;
-  float* moe_topw = nullptr;
-  int* moe_topi = nullptr;
-  int* moe_ints = nullptr;             // cursor | count | offsets | cursor2 | send_meta | recv_meta | pair_slot | slot_pos | recv counts
-  size_t moe_ints_n = 0;
-  void *moe_send = nullptr, *moe_recv = nullptr, *moe_xs = nullptr, *moe_hs = nullptr;
-  float *moe_ys = nullptr, *moe_ret = nullptr, *moe_back = nullptr, *moe_tmp = nullptr;
-  int* route_rec = nullptr;            // option record_routing: every MoE layer's top-k expert ids of the last forward, [n_moe][rows_cap][k]
-  int64_t route_rows = 0;              // rows of the forward recorded last
-  cudaGraphExec_t graph = nullptr;
-  cudaEvent_t ev0 = nullptr, ev1 = nullptr;
-  float prefill_ms = 0.f, decode_ms = 0.f;
-  int host_pos = 0;                    // tokens so far (all sequences advance together)
-  int graph_kernels = 0;               // kernels in one captured decode step
-  int graph_epoch = -1;                // option epoch the graph was captured under
-  // GenerationConfig sampling (generate.nim:12-58); off = greedy argmax
-  bool samp_on = false;
-  float samp_temperature = 1.f, samp_top_p = 1.f, samp_min_p = 0.f, samp_rep = 1.f;
-  int samp_top_k = 0, samp_do_sample = 0;
-  std::vector<uint64_t> samp_seeds;    // one per sequence; keys restart from these on reset
-  int *samp_hist = nullptr, *samp_hist_len = nullptr, *samp_steps = nullptr;  // [B][max_len], [B], [B]
-  uint32_t* samp_keys = nullptr;       // [B][2]
-  float *samp_work = nullptr, *samp_logprob = nullptr;  // [B][V], [B][max_len]
-  // Paged lanes (continuous batching): a shared pool of KV pages handed out on demand
-  bool paged = false;
-  int num_blocks = 0;                  // pages in the pool; page 0 is the scratch page of idle lanes
-  std::vector<int> free_blocks;        // as PagedKvCache.freeBlocks (generate.nim:75,86-88)
-  std::vector<int> lane_len;           // tokens in the cache per lane
-  std::vector<char> lane_active;
-  std::vector<std::vector<int>> lane_pages;
-  int* d_active = nullptr;             // [B] or nullptr (every lane active)
-  int* d_ids_prefill = nullptr;        // ids of a single-lane prefill
-};
-
 namespace rewb {
-namespace {
 
 // Sampling restarts with every generate call: keys back to initKey(seed), step counters to zero.
 int samp_restart(rewb200_session* s) {
@@ -404,6 +258,14 @@ int acts_alloc(Ctx* c, T** p, size_t bytes) {
   return acts_alloc(c, (void**)p, bytes);
 }
 
+int swiglu_rows_f32_launch(Ctx* c, const float* gu, float* out, int64_t rows, int64_t f) {
+  const int64_t n = rows * f;
+  swiglu_rows_f32_kernel<<<(unsigned)((n + 255) / 256), 256, 0, c->stream>>>(gu, out, rows, f);
+  RB_CUDA(cudaGetLastError());
+  ++g_launch_total;
+  return REWB200_OK;
+}
+
 int ensure_acts(rewb200_session* s, int64_t rows, int64_t logits_rows) {
   rewb200_model* m = s->m;
   const rewb200_config& c = m->cfg;
@@ -413,7 +275,8 @@ int ensure_acts(rewb200_session* s, int64_t rows, int64_t logits_rows) {
     void** ptrs[] = {(void**)&s->x_res, &s->xn, &s->q, &s->attn, &s->h, (void**)&s->part, (void**)&s->gu32,
                      (void**)&s->moe_logits, (void**)&s->moe_topw, (void**)&s->moe_topi, (void**)&s->moe_ints, &s->moe_send,
                      &s->moe_recv, &s->moe_xs, &s->moe_hs, (void**)&s->moe_ys, (void**)&s->moe_ret, (void**)&s->moe_back,
-                     (void**)&s->moe_tmp, (void**)&s->route_rec};
+                     (void**)&s->moe_tmp, (void**)&s->route_rec, &s->xn2, &s->cq, (void**)&s->gate, (void**)&s->part2,
+                     (void**)&s->layer_rec};
     // From here until every allocation below has succeeded the session holds no activation buffers: a failed
     // growth must leave it in a state where the next call allocates again instead of launching on NULL.
     s->rows_cap = 0;
@@ -428,15 +291,13 @@ int ensure_acts(rewb200_session* s, int64_t rows, int64_t logits_rows) {
         *p = nullptr;
         RB_CUDA(cudaFree(q));
       }
-    int64_t fmax = 0;
-    for (const LayerDev& L : m->layers) fmax = std::max(fmax, L.ffn_local);
-    if (c.n_routed > 0) fmax = std::max<int64_t>(fmax, c.moe_ffn);
-    RB_TRY(acts_alloc(m->c, (void**)&s->x_res, (size_t)rows * c.d_model * sizeof(float)));
-    RB_TRY(acts_alloc(m->c, &s->xn, (size_t)rows * c.d_model * es));
+    const int64_t fmax = std::max(m->max_ffn, m->max_moe_ffn), dp = m->dp;
+    RB_TRY(acts_alloc(m->c, (void**)&s->x_res, (size_t)rows * dp * sizeof(float)));
+    RB_TRY(acts_alloc(m->c, &s->xn, (size_t)rows * dp * es));
     RB_TRY(acts_alloc(m->c, &s->q, (size_t)rows * std::max<int64_t>(m->nq, 1) * es));
     RB_TRY(acts_alloc(m->c, &s->attn, (size_t)rows * std::max<int64_t>(m->nq, 1) * es));
     RB_TRY(acts_alloc(m->c, &s->h, (size_t)rows * std::max<int64_t>(fmax, 1) * es));
-    const int64_t widest = std::max<int64_t>(m->nqkv, c.d_model);
+    const int64_t widest = std::max<int64_t>(m->nqkv, dp);
     // up to 16 split-K slabs of the widest residual-side Linear, or 4 of gate|up, at steps of at most 64 rows
     const size_t small_rows = (size_t)std::min<int64_t>(rows, 64);
     s->part_bytes = small_rows * std::max<size_t>(16 * widest, 4 * 2 * fmax) * sizeof(float);
@@ -446,29 +307,30 @@ int ensure_acts(rewb200_session* s, int64_t rows, int64_t logits_rows) {
       s->part_bytes = std::max(s->part_bytes, (size_t)32 * std::max<size_t>(16 * widest, 4 * 2 * fmax) * sizeof(float));
     RB_TRY(acts_alloc(m->c, (void**)&s->part, s->part_bytes));
     if (c.dtype == REWB200_F32) RB_TRY(acts_alloc(m->c, (void**)&s->gu32, (size_t)rows * 2 * std::max<int64_t>(fmax, 1) * sizeof(float)));
-    if (c.n_routed > 0) {
-      const int ep = c.ep_size, k = c.top_k, E_l = c.n_routed / ep;
+    if (m->n_moe > 0) {
+      const int ep = c.ep_size, k = m->max_topk, E_l = m->max_experts / ep;
       const int64_t cap = rows * k, slots = cap * ep;
-      RB_TRY(acts_alloc(m->c, (void**)&s->moe_logits, (size_t)std::max<int64_t>(rows, 8 * std::min<int64_t>(rows, 64)) * c.n_routed * sizeof(float)));  // or 8 split-K slabs of a small step
+      RB_TRY(acts_alloc(m->c, (void**)&s->moe_logits, (size_t)std::max<int64_t>(rows, 8 * std::min<int64_t>(rows, 64)) * m->max_experts * sizeof(float)));  // or 8 split-K slabs of a small step
       RB_TRY(acts_alloc(m->c, (void**)&s->moe_topw, (size_t)rows * k * sizeof(float)));
       RB_TRY(acts_alloc(m->c, (void**)&s->moe_topi, (size_t)rows * k * sizeof(int)));
       // the last 16 ints hold the per-peer counts this rank receives (prefix exchange of large steps)
       s->moe_ints_n = (size_t)(ep + 3 * (E_l + 1) + 3 * slots + rows * k) + 16;
       RB_TRY(acts_alloc(m->c, (void**)&s->moe_ints, s->moe_ints_n * sizeof(int)));
-      RB_TRY(acts_alloc(m->c, (void**)&s->moe_tmp, (size_t)rows * c.d_model * sizeof(float)));
-      if (m->c->record_routing) RB_TRY(acts_alloc(m->c, (void**)&s->route_rec, (size_t)c.n_layers * rows * k * sizeof(int)));
+      RB_TRY(acts_alloc(m->c, (void**)&s->moe_tmp, (size_t)rows * dp * sizeof(float)));
+      if (m->c->record_routing) RB_TRY(acts_alloc(m->c, (void**)&s->route_rec, (size_t)m->n_moe * rows * k * sizeof(int)));
       if (c.dtype == REWB200_BF16) {
-        RB_TRY(acts_alloc(m->c, &s->moe_send, (size_t)slots * c.d_model * es));
-        if (ep > 1) RB_TRY(acts_alloc(m->c, &s->moe_recv, (size_t)slots * c.d_model * es));
-        RB_TRY(acts_alloc(m->c, &s->moe_xs, (size_t)(slots + 128) * c.d_model * es));
-        RB_TRY(acts_alloc(m->c, &s->moe_hs, (size_t)(slots + 128) * c.moe_ffn * es));
-        RB_CUDA(cudaMemset(s->moe_xs, 0, (size_t)(slots + 128) * c.d_model * es));
-        RB_CUDA(cudaMemset(s->moe_hs, 0, (size_t)(slots + 128) * c.moe_ffn * es));
-        RB_TRY(acts_alloc(m->c, (void**)&s->moe_ys, (size_t)slots * c.d_model * sizeof(float)));
-        RB_TRY(acts_alloc(m->c, (void**)&s->moe_ret, (size_t)slots * c.d_model * sizeof(float)));
-        if (ep > 1) RB_TRY(acts_alloc(m->c, (void**)&s->moe_back, (size_t)slots * c.d_model * sizeof(float)));
+        RB_TRY(acts_alloc(m->c, &s->moe_send, (size_t)slots * dp * es));
+        if (ep > 1) RB_TRY(acts_alloc(m->c, &s->moe_recv, (size_t)slots * dp * es));
+        RB_TRY(acts_alloc(m->c, &s->moe_xs, (size_t)(slots + 128) * dp * es));
+        RB_TRY(acts_alloc(m->c, &s->moe_hs, (size_t)(slots + 128) * m->max_moe_ffn * es));
+        RB_CUDA(cudaMemset(s->moe_xs, 0, (size_t)(slots + 128) * dp * es));
+        RB_CUDA(cudaMemset(s->moe_hs, 0, (size_t)(slots + 128) * m->max_moe_ffn * es));
+        RB_TRY(acts_alloc(m->c, (void**)&s->moe_ys, (size_t)slots * dp * sizeof(float)));
+        RB_TRY(acts_alloc(m->c, (void**)&s->moe_ret, (size_t)slots * dp * sizeof(float)));
+        if (ep > 1) RB_TRY(acts_alloc(m->c, (void**)&s->moe_back, (size_t)slots * dp * sizeof(float)));
       }
     }
+    if (m->layered) RB_TRY(layered_acts(s, rows));
     s->rows_cap = rows;
   }
   if (logits_rows > s->logits_rows) {
@@ -492,7 +354,7 @@ int ensure_acts(rewb200_session* s, int64_t rows, int64_t logits_rows) {
 // y = x @ W for the model dtype.  `partial` selects the f32 split-K slab
 // output (bias deferred to the consumer) over a finished output with bias.
 int run_linear(rewb200_session* s, const LinW& w, const void* x, int64_t ldx, int64_t rows, bool partial, int epi,
-               void* out, int64_t ldo, int* ksplit_out, const QkvPostArgs* fuse_qkv = nullptr, bool* fused = nullptr) {
+               void* out, int64_t ldo, int* ksplit_out, const QkvPostArgs* fuse_qkv, bool* fused) {
   Ctx* c = s->m->c;
   if (fused) *fused = false;
   if (w.quant && rows <= 32) {
@@ -547,8 +409,8 @@ int run_linear(rewb200_session* s, const LinW& w, const void* x, int64_t ldx, in
                               partial ? nullptr : w.b, nullptr, 0);
   }
   if (ksplit_out) *ksplit_out = 1;
-  RB_REQUIRE(ldx == w.K && ldo == w.N, "f32 Linear expects dense rows");
-  return gemm_f32_launch(c, (const float*)x, (const float*)w.w, partial ? nullptr : w.b, (float*)out, rows, w.K, w.N);
+  RB_REQUIRE(ldx >= w.K && ldo >= w.N, "f32 Linear: rows shorter than the matrix is wide");
+  return gemm_f32_ld_launch(c, (const float*)x, ldx, (const float*)w.w, w.N, partial ? nullptr : w.b, (float*)out, ldo, rows, w.K, w.N);
 }
 
 // Routed experts of one MoE layer for the normalised rows in s->xn: router, top-k, dispatch to the
@@ -572,13 +434,13 @@ bool ep_uses_peer_heap(const rewb200_model* m, int64_t rows) {
          a2a_need(rows * cf.top_k * cf.ep_size, cf.d_model, dtype_size(cf.dtype), nullptr, nullptr) <= pi->a2a_bytes;
 }
 
-int moe_routed(rewb200_session* s, LayerDev& L, int64_t rows, bool accumulate, float* out = nullptr, int moe_index = 0) {
+int moe_routed(rewb200_session* s, MoeDev& X, const void* x, int64_t d, int64_t rows, bool accumulate, float* out, int moe_index) {
   rewb200_model* m = s->m;
   Ctx* c = m->c;
   const rewb200_config& cf = m->cfg;
-  MoeDev& X = L.x;
-  const int64_t d = cf.d_model, f = X.f;
-  const int k = cf.top_k, ep = cf.ep_size, E_l = X.E_l;
+  const int64_t f = X.f, ldr = X.router.N;
+  const int k = X.top_k, ep = cf.ep_size, E_l = X.E_l;
+  const int epi_up = X.gated ? EPI_SWIGLU_BF16 : EPI_RELU2_BF16;
   const int dt = cf.dtype;
   // expert parallel over the peer heap: the routing kernel also clears the dispatch kernel's per-peer cursors
   const bool peer = ep_uses_peer_heap(m, rows);
@@ -589,37 +451,41 @@ int moe_routed(rewb200_session* s, LayerDev& L, int64_t rows, bool accumulate, f
     const int nkb = (int)((d + 63) / 64);
     int ks = 1;
     while (ks < 8 && nkb / (ks * 2) >= 4) ks *= 2;
-    RB_TRY(linear_bf16_launch(c, X.router.plan, (const bf16*)s->xn, d, rows, EPI_PARTIAL_F32, ks, s->moe_logits, cf.n_routed,
+    RB_TRY(linear_bf16_launch(c, X.router.plan, (const bf16*)x, d, rows, EPI_PARTIAL_F32, ks, s->moe_logits, ldr,
                               nullptr, nullptr, 0));
-    RB_TRY(moe_route_slabs_launch(c, s->moe_logits, ks, rows * cf.n_routed, X.router.b, rows, cf.n_routed, k, s->moe_topw,
+    RB_TRY(moe_route_slabs_launch(c, s->moe_logits, ks, rows * ldr, X.router.b, rows, X.E, ldr, k, X.renorm, s->moe_topw,
                                   s->moe_topi, clear, peer ? ep : 0));
     cleared = peer;
   } else {
     if (dt == REWB200_BF16)
-      RB_TRY(linear_bf16_launch(c, X.router.plan, (const bf16*)s->xn, d, rows, EPI_BIAS_F32, 1, s->moe_logits, cf.n_routed,
+      RB_TRY(linear_bf16_launch(c, X.router.plan, (const bf16*)x, d, rows, EPI_BIAS_F32, 1, s->moe_logits, ldr,
                                 X.router.b, nullptr, 0));
     else
-      RB_TRY(gemm_f32_launch(c, (const float*)s->xn, (const float*)X.router.w, X.router.b, s->moe_logits, rows, d, cf.n_routed));
-    RB_TRY(moe_route_launch(c, s->moe_logits, rows, cf.n_routed, k, s->moe_topw, s->moe_topi));
+      RB_TRY(gemm_f32_launch(c, (const float*)x, (const float*)X.router.w, X.router.b, s->moe_logits, rows, d, ldr));
+    RB_TRY(moe_route_slabs_launch(c, s->moe_logits, 1, 0, nullptr, rows, X.E, ldr, k, X.renorm, s->moe_topw, s->moe_topi, nullptr, 0));
   }
   if (s->route_rec) {
-    RB_CUDA(cudaMemcpyAsync(s->route_rec + (size_t)moe_index * s->rows_cap * k, s->moe_topi, (size_t)rows * k * sizeof(int),
+    RB_CUDA(cudaMemcpyAsync(s->route_rec + (size_t)moe_index * s->rows_cap * m->max_topk, s->moe_topi, (size_t)rows * k * sizeof(int),
                             cudaMemcpyDeviceToDevice, c->stream));
     s->route_rows = rows;
   }
   if (dt == REWB200_F32) {
     // parity path: every local expert on every token, masked by its routing weight, as the reference does
     for (int e = 0; e < E_l; ++e) {
-      const float* gw = (const float*)X.gu + (size_t)e * d * 2 * f;
+      const int64_t fw = X.gated ? 2 * f : f;
+      const float* gw = (const float*)X.gu + (size_t)e * d * fw;
       const float* dw = (const float*)X.down + (size_t)e * f * d;
-      RB_TRY(gemm_f32_launch(c, (const float*)s->xn, gw, X.gu_b + (size_t)e * 2 * f, s->gu32, rows, d, 2 * f));
+      RB_TRY(gemm_f32_launch(c, (const float*)x, gw, X.gu_b + (size_t)e * fw, s->gu32, rows, d, fw));
       const int64_t n = rows * f;
-      swiglu_rows_f32_kernel<<<(unsigned)((n + 255) / 256), 256, 0, c->stream>>>(s->gu32, (float*)s->h, rows, f);
+      if (X.gated)
+        swiglu_rows_f32_kernel<<<(unsigned)((n + 255) / 256), 256, 0, c->stream>>>(s->gu32, (float*)s->h, rows, f);
+      else
+        relu2_f32_kernel<<<(unsigned)((n + 255) / 256), 256, 0, c->stream>>>(s->gu32, (float*)s->h, n);
       RB_CUDA(cudaGetLastError());
       RB_TRY(gemm_f32_launch(c, (const float*)s->h, dw, X.down_b + (size_t)e * d, s->moe_tmp, rows, f, d));
       const int64_t nd = rows * d;
       moe_dense_acc_kernel<<<(unsigned)((nd + 255) / 256), 256, 0, c->stream>>>(s->moe_tmp, s->moe_topw, s->moe_topi, k, e, rows,
-                                                                                d, s->part, (accumulate || e > 0) ? 1 : 0);
+                                                                                d, out ? out : s->part, (accumulate || e > 0) ? 1 : 0);
       RB_CUDA(cudaGetLastError());
       g_launch_total += 2;
     }
@@ -637,9 +503,9 @@ int moe_routed(rewb200_session* s, LayerDev& L, int64_t rows, bool accumulate, f
   if (ep == 1 && cap <= 2048) {
     // every expert is local and the step is small: one kernel sorts the pairs by expert and copies the
     // rows, the combine reads the expert outputs in place (no slot arrays, no atomics, no return copy)
-    RB_TRY(moe_group_local_launch(c, s->xn, dt, s->moe_topi, rows, k, d, E_l, offsets, s->moe_xs, pair_slot));
+    RB_TRY(moe_group_local_launch(c, x, dt, s->moe_topi, rows, k, d, E_l, offsets, s->moe_xs, pair_slot));
     const int max_rows_l = (int)std::min<int64_t>(rows, cap);
-    RB_TRY(linear_bf16_launch(c, X.plan_gu, (const bf16*)s->moe_xs, d, cap, EPI_SWIGLU_BF16, 1, s->moe_hs, f, X.gu_b, offsets,
+    RB_TRY(linear_bf16_launch(c, X.plan_gu, (const bf16*)s->moe_xs, d, cap, epi_up, 1, s->moe_hs, f, X.gu_b, offsets,
                               max_rows_l));
     RB_TRY(linear_bf16_launch(c, X.plan_down, (const bf16*)s->moe_hs, f, cap, EPI_BIAS_F32, 1, s->moe_ys, d, X.down_b, offsets,
                               max_rows_l));
@@ -663,10 +529,10 @@ int moe_routed(rewb200_session* s, LayerDev& L, int64_t rows, bool accumulate, f
     a.status = c->d_status;
     // large steps count with atomics: clear the counters; small ones need only the cursors, cleared by the routing kernel
     if (!cleared || slots > 4096) RB_TRY(moe_reset_launch(c, cursor, ep, count, E_l + 1, send_meta, 0));
-    RB_TRY(moe_dispatch_peer_launch(c, s->xn, dt, s->moe_topi, rows, k, d, E_l, (int)cap, cursor, pair_slot, a));
+    RB_TRY(moe_dispatch_peer_launch(c, x, dt, s->moe_topi, rows, k, d, E_l, (int)cap, cursor, pair_slot, a));
     RB_TRY(moe_group_peer_launch(c, dt, (int)slots, (int)cap, d, E_l, count, offsets, cursor2, s->moe_xs, slot_pos, a));
     const int max_rows_p = (int)std::min<int64_t>(rows * ep, slots);
-    RB_TRY(linear_bf16_launch(c, X.plan_gu, (const bf16*)s->moe_xs, d, slots, EPI_SWIGLU_BF16, 1, s->moe_hs, f, X.gu_b, offsets,
+    RB_TRY(linear_bf16_launch(c, X.plan_gu, (const bf16*)s->moe_xs, d, slots, epi_up, 1, s->moe_hs, f, X.gu_b, offsets,
                               max_rows_p));
     RB_TRY(linear_bf16_launch(c, X.plan_down, (const bf16*)s->moe_hs, f, slots, EPI_BIAS_F32, 1, s->moe_ys, d, X.down_b, offsets,
                               max_rows_p));
@@ -674,7 +540,7 @@ int moe_routed(rewb200_session* s, LayerDev& L, int64_t rows, bool accumulate, f
     return moe_combine_peer_launch(c, pair_slot, s->moe_topw, rows, k, d, out ? out : s->part, accumulate ? 1 : 0, a);
   }
   RB_TRY(moe_reset_launch(c, cursor, ep, count, E_l + 1, send_meta, (int)slots));
-  RB_TRY(moe_dispatch_launch(c, s->xn, dt, s->moe_topi, rows, k, d, E_l, (int)cap, cursor, s->moe_send, send_meta, pair_slot));
+  RB_TRY(moe_dispatch_launch(c, x, dt, s->moe_topi, rows, k, d, E_l, (int)cap, cursor, s->moe_send, send_meta, pair_slot));
   const void* rx = s->moe_send;
   const int* rmeta = send_meta;
   // Large steps outside a captured graph (prefill): exchange the per-peer pair counts first and move only the
@@ -710,7 +576,7 @@ int moe_routed(rewb200_session* s, LayerDev& L, int64_t rows, bool accumulate, f
   RB_TRY(moe_group_launch(c, rx, dt, rmeta, (int)slots, d, E_l, count, offsets, cursor2, s->moe_xs, slot_pos));
   // an expert receives each token at most once: at most rows * ep rows per group
   const int max_rows = (int)std::min<int64_t>(rows * ep, slots);
-  RB_TRY(linear_bf16_launch(c, X.plan_gu, (const bf16*)s->moe_xs, d, slots, EPI_SWIGLU_BF16, 1, s->moe_hs, f, X.gu_b, offsets,
+  RB_TRY(linear_bf16_launch(c, X.plan_gu, (const bf16*)s->moe_xs, d, slots, epi_up, 1, s->moe_hs, f, X.gu_b, offsets,
                             max_rows));
   RB_TRY(linear_bf16_launch(c, X.plan_down, (const bf16*)s->moe_hs, f, slots, EPI_BIAS_F32, 1, s->moe_ys, d, X.down_b, offsets,
                             max_rows));
@@ -726,6 +592,8 @@ int moe_routed(rewb200_session* s, LayerDev& L, int64_t rows, bool accumulate, f
   }
   return moe_combine_launch(c, back, pair_slot, s->moe_topw, rows, k, d, out ? out : s->part, accumulate ? 1 : 0);
 }
+
+namespace {
 
 // Copies the last-position logits [B, vocab] to the host; under tensor parallelism the
 // vocabulary slices are all-gathered first and re-interleaved on the host.
@@ -750,89 +618,17 @@ int fetch_logits(rewb200_session* s, int64_t rows, float* host) {
   return REWB200_OK;
 }
 
-// Per-category device times of one forward (REW_B200_TRACE-style measurement aid): an event after the
-// launches of each category, elapsed times summed per category after a synchronisation.  Events between
-// kernels switch programmatic dependent launch off at those points, so the sum exceeds the untraced step;
-// the split is what it is for.
-enum TraceCat : int { TC_EMBED = 0, TC_QKV, TC_QKV_POST, TC_ATTN, TC_O, TC_NORM_ATTN, TC_GATE_UP, TC_DOWN, TC_MOE, TC_NORM_FFN, TC_HEAD, TC_COUNT };
-struct Trace {
-  std::vector<cudaEvent_t> ev;
-  std::vector<int> cat;
-  cudaStream_t st = nullptr;
-  int begin(cudaStream_t s) {
-    st = s;
-    return mark(-1);
-  }
-  int mark(int c) {
-    cudaEvent_t e;
-    RB_CUDA(cudaEventCreate(&e));
-    RB_CUDA(cudaEventRecord(e, st));
-    ev.push_back(e);
-    cat.push_back(c);
-    return REWB200_OK;
-  }
-  int finish(float* ms) {  // ms[TC_COUNT]
-    for (int i = 0; i < TC_COUNT; ++i) ms[i] = 0.f;
-    RB_CUDA(cudaStreamSynchronize(st));
-    for (size_t i = 1; i < ev.size(); ++i) {
-      float t = 0.f;
-      RB_CUDA(cudaEventElapsedTime(&t, ev[i - 1], ev[i]));
-      if (cat[i] >= 0 && cat[i] < TC_COUNT) ms[cat[i]] += t;
-    }
-    return REWB200_OK;
-  }
-  ~Trace() {
-    for (cudaEvent_t e : ev) cudaEventDestroy(e);
-  }
-};
-
-struct FwdOpts {
-  Trace* trace = nullptr;     // when set, an event follows every category of launches
-  int S = 1;
-  int rope_shift = 0;
-  int causal = 1;
-  bool all_logits = false;  // lm_head on every row instead of the last position
-  bool from_device_ids = false;
-  // Lanes [b0, b0 + nb) of the session only (nb < 0: all).  The per-lane arrays (positions, block table,
-  // next ids, logits rows, sampling state) are indexed from b0; ids_src overrides where the nb*S input
-  // ids are read, so that a single-lane prefill does not disturb the other lanes' pending tokens.
-  int b0 = 0, nb = -1;
-  const int* ids_src = nullptr;
-  bool record_out = true;    // append the new ids to the session's [step][B] output buffer
-};
-
-// Enqueues one forward over rows = B*S tokens whose ids are in s->d_ids.
-int enqueue_forward(rewb200_session* s, const FwdOpts& o) {
+// The decoder blocks of a grouped-query model (llama.nim:106-129, deepseek.nim:198-220) over rows = nb*S tokens: embedding
+// and first norm, then every layer; leaves the final norm's output in s->xn.
+int gqa_blocks(rewb200_session* s, const FwdOpts& o, const NormArgs& na, int64_t rows, bool in_graph) {
   rewb200_model* m = s->m;
   Ctx* c = m->c;
   const rewb200_config& cf = m->cfg;
   const int b0 = o.b0, nb = o.nb < 0 ? s->B : o.nb;
-  const int64_t rows = (int64_t)nb * o.S;
   const int64_t d = cf.d_model;
   int* const pos = s->d_pos + b0;
   const int* const block_table = s->block_table + (size_t)b0 * s->max_pages;
-  float* const logits = o.all_logits ? s->logits : s->logits + (size_t)b0 * m->vocab_l;
-  int* const next = s->d_next + b0;
   const int dt = cf.dtype;
-
-  // A captured decode step is replayed as one graph launch: positions, block tables and all cache rows but
-  // the newest were written before that launch, which is what lets two kernels read them ahead of their
-  // stream dependency.  Plain launches (prefill, REW_B200_NO_GRAPH) chain across calls and get no such promise.
-  cudaStreamCaptureStatus cap_st = cudaStreamCaptureStatusNone;
-  RB_CUDA(cudaStreamIsCapturing(c->stream, &cap_st));
-  const bool in_graph = cap_st == cudaStreamCaptureStatusActive && o.S == 1;
-  NormArgs na;
-  memset(&na, 0, sizeof(na));
-  na.x_res = s->x_res;
-  na.d = d;
-  na.eps = cf.eps;
-  na.norm_kind = cf.norm_kind;
-  na.out = s->xn;
-  na.out_dtype = dt;
-  na.vocab = cf.vocab;
-  na.status = c->d_status;
-  na.embed_dtype = dt;
-
   // embedding gather + first norm
   {
     NormArgs a = na;
@@ -1033,7 +829,7 @@ int enqueue_forward(rewb200_session* s, const FwdOpts& o) {
       c->stream = main_stream;
       RB_TRY(st);
       RB_CUDA(cudaEventRecord(c->ev_join, c->side));
-      RB_TRY(moe_routed(s, L, rows, false, base + (size_t)ks * rows * d, moe_seen++));
+      RB_TRY(moe_routed(s, L.x, s->xn, d, rows, false, base + (size_t)ks * rows * d, moe_seen++));
       RB_CUDA(cudaStreamWaitEvent(c->stream, c->ev_join, 0));
       NormArgs a = na;
       a.partial = base;
@@ -1065,7 +861,7 @@ int enqueue_forward(rewb200_session* s, const FwdOpts& o) {
       if (o.trace) RB_TRY(o.trace->mark(TC_DOWN));
     }
     if (L.moe) {
-      RB_TRY(moe_routed(s, L, rows, ks > 0, nullptr, moe_seen++));
+      RB_TRY(moe_routed(s, L.x, s->xn, d, rows, ks > 0, nullptr, moe_seen++));
       if (ks == 0) ks = 1;
       if (o.trace) RB_TRY(o.trace->mark(TC_MOE));
     }
@@ -1086,25 +882,110 @@ int enqueue_forward(rewb200_session* s, const FwdOpts& o) {
   if (oneshot) RB_TRY(epoch_bump_launch(c, pi->epoch, 2 * cf.n_layers));  // same on every rank
   if (moe_seen > 0 && ep_uses_peer_heap(m, rows)) RB_TRY(epoch_bump_launch(c, comm_peer_info(m->slot)->epoch + 1, moe_seen));
   if (twoshot) RB_TRY(epoch_bump_launch(c, pi->epoch + 1, 2 * cf.n_layers));
-  // lm_head: last position of every sequence (generate.nim:172-190) or every row.
-  const int64_t lrows = o.all_logits ? rows : nb;
-  const char* xl = (const char*)s->xn + (o.all_logits ? 0 : (size_t)(o.S - 1) * d * dtype_size(dt));
-  const int64_t ldx = o.all_logits ? d : (int64_t)o.S * d;
-  if (dt == REWB200_BF16) {
-    RB_TRY(linear_bf16_launch(c, m->lm.plan, (const bf16*)xl, ldx, lrows, EPI_BIAS_F32, 1, logits, m->vocab_l, m->lm.b,
-                              nullptr, 0));
-  } else {
-    if (o.all_logits || o.S == 1) {
-      RB_TRY(gemm_f32_launch(c, (const float*)xl, (const float*)m->lm.w, m->lm.b, logits, lrows, d, m->vocab_l));
-    } else {
-      // gather the last rows into the head of q (free at this point), then GEMM
-      for (int b = 0; b < nb; ++b)
-        RB_CUDA(cudaMemcpyAsync((float*)s->q + (size_t)b * d, (const float*)s->xn + ((size_t)b * o.S + o.S - 1) * d,
-                                d * sizeof(float), cudaMemcpyDeviceToDevice, c->stream));
-      RB_TRY(gemm_f32_launch(c, (const float*)s->q, (const float*)m->lm.w, m->lm.b, logits, lrows, d, m->vocab_l));
-    }
+  return REWB200_OK;
+}
+
+// Room for the rows a step gathers for the lm_head, and for its output when the vocabulary is padded.
+int ensure_head_rows(rewb200_session* s, int64_t rows) {
+  rewb200_model* m = s->m;
+  const bool pad = m->vp != m->vocab_l;
+  if (rows <= s->xg_rows) return REWB200_OK;
+  RB_CUDA(cudaStreamSynchronize(m->c->stream));
+  s->xg_rows = 0;
+  if (s->graph) {
+    cudaGraphExecDestroy(s->graph);
+    s->graph = nullptr;
   }
-  if (!o.all_logits) {
+  for (void** p : {&s->xg, (void**)&s->logits_pad})
+    if (*p) {
+      void* q = *p;
+      *p = nullptr;
+      RB_CUDA(cudaFree(q));
+    }
+  RB_TRY(acts_alloc(m->c, &s->xg, (size_t)rows * m->dp * dtype_size(m->cfg.dtype)));
+  if (pad) RB_TRY(acts_alloc(m->c, (void**)&s->logits_pad, (size_t)rows * m->vp * sizeof(float)));
+  s->xg_rows = rows;
+  return REWB200_OK;
+}
+
+// The portions of a step that feeds S tokens to each of nb lanes, all at position pos0.
+std::vector<StepEntry> uniform_entries(const rewb200_session* s, int b0, int nb, int S, int pos0) {
+  (void)s;
+  std::vector<StepEntry> e;
+  for (int b = 0; b < nb; ++b) e.push_back({b0 + b, b * S, S, pos0});
+  return e;
+}
+
+// Enqueues one forward over rows = B*S tokens whose ids are in s->d_ids.
+int enqueue_forward(rewb200_session* s, const FwdOpts& o) {
+  rewb200_model* m = s->m;
+  Ctx* c = m->c;
+  const rewb200_config& cf = m->cfg;
+  const int b0 = o.b0, nb = o.nb < 0 ? s->B : o.nb;
+  int64_t rows = (int64_t)nb * o.S;
+  if (o.entries) {
+    rows = 0;
+    for (const StepEntry& e : *o.entries) rows += e.n;
+  }
+  const int64_t d = m->dp;
+  int* const pos = s->d_pos + b0;
+  const bool lists = o.out_rows != nullptr;
+  // where the logits of lanes [b0, b0 + nb) go: behind those of the wanted rows, or at their lane index
+  float* const logits = o.all_logits ? s->logits : s->logits + (size_t)(lists ? o.n_want : b0) * m->vocab_l;
+  int* const next = s->d_next + b0;
+  const int dt = cf.dtype;
+
+  // A captured decode step is replayed as one graph launch: positions, block tables and all cache rows but
+  // the newest were written before that launch, which is what lets two kernels read them ahead of their
+  // stream dependency.  Plain launches (prefill, REW_B200_NO_GRAPH) chain across calls and get no such promise.
+  cudaStreamCaptureStatus cap_st = cudaStreamCaptureStatusNone;
+  RB_CUDA(cudaStreamIsCapturing(c->stream, &cap_st));
+  const bool in_graph = cap_st == cudaStreamCaptureStatusActive && o.S == 1;
+  NormArgs na;
+  memset(&na, 0, sizeof(na));
+  na.x_res = s->x_res;
+  na.d = d;
+  na.eps = cf.eps;
+  na.norm_kind = cf.norm_kind;
+  na.out = s->xn;
+  na.out_dtype = dt;
+  na.vocab = cf.vocab;
+  na.status = c->d_status;
+  na.embed_dtype = dt;
+  if (m->layered) {
+    na.embed = m->embed;
+    na.ids = o.ids_src ? o.ids_src : s->d_ids;
+    if (d != cf.d_model) na.d_mean = cf.d_model;
+    RB_TRY(layered_blocks(s, o, na, rows));
+  } else {
+    RB_TRY(gqa_blocks(s, o, na, rows, in_graph));
+  }
+
+  // lm_head: last position of every sequence (generate.nim:172-190), every row, or the rows of a list.
+  const int64_t lrows = o.all_logits ? rows : lists ? o.n_want + (o.sample ? nb : 0) : nb;
+  const char* xl = (const char*)s->xn + (o.all_logits ? 0 : (size_t)(o.S - 1) * d * dtype_size(dt));
+  int64_t ldx = o.all_logits ? d : (int64_t)o.S * d;
+  float* lout = logits;
+  if (lists) {
+    RB_TRY(gather_rows_launch(c, s->xn, o.out_rows, s->xg, lrows, d, dt));
+    xl = (const char*)s->xg;
+    ldx = d;
+    lout = s->logits;
+  }
+  if (lrows > 0) {
+    const int64_t V = m->vocab_l, vp = m->vp;
+    float* const lm_out = vp == V ? lout : s->logits_pad;
+    if (dt == REWB200_BF16) {
+      RB_TRY(linear_bf16_launch(c, m->lm.plan, (const bf16*)xl, ldx, lrows, EPI_BIAS_F32, 1, lm_out, vp, m->lm.b, nullptr, 0));
+    } else {
+      RB_TRY(gemm_f32_ld_launch(c, (const float*)xl, ldx, (const float*)m->lm.w, vp, m->lm.b, lm_out, vp, lrows, m->lm.K, vp));
+    }
+    if (vp != V)
+      RB_CUDA(cudaMemcpy2DAsync(lout, V * sizeof(float), lm_out, vp * sizeof(float), V * sizeof(float), lrows, cudaMemcpyDeviceToDevice,
+                                c->stream));
+  }
+  if (!o.all_logits && o.sample) {
+    const int* act = o.sample_active ? o.sample_active : s->d_active ? s->d_active + b0 : nullptr;
     if (cf.tp_size > 1) {
       RB_REQUIRE(b0 == 0 && nb == s->B, "lane ranges are not available on a tensor-parallel model");
       // vocab-parallel: per-rank (value, index) partials, all-gathered, then the same first-max rule
@@ -1115,7 +996,6 @@ int enqueue_forward(rewb200_session* s, const FwdOpts& o) {
       RB_TRY(comm_allgather_bytes(c, m->slot, s->argmax_scratch, s->gather_scratch, (size_t)s->B * nch * 8));
       RB_TRY(argmax_gathered_launch(c, s->gather_scratch, cf.tp_size, s->B, nch, s->d_next));
     } else if (s->samp_on) {
-      const int* act = s->d_active ? s->d_active + b0 : nullptr;
       RB_TRY(sample_launch(c, logits, s->samp_work + (size_t)b0 * cf.vocab, nb, cf.vocab, s->samp_hist + (size_t)b0 * s->max_len,
                            s->samp_hist_len + b0, s->max_len, s->samp_keys + 2 * b0, s->samp_steps + b0, next,
                            s->samp_logprob + (size_t)b0 * s->max_len, s->max_len, s->samp_temperature, s->samp_top_k,
@@ -1124,8 +1004,7 @@ int enqueue_forward(rewb200_session* s, const FwdOpts& o) {
       RB_TRY(argmax_launch(c, logits, nb, cf.vocab, next, s->argmax_scratch, (size_t)s->B * 64 * 8));
     }
     RB_CUDA(launch_k(advance_kernel, dim3(1), dim3(256), 0, c->stream, c->use_pdl, (const int*)next, s->d_ids + b0, pos,
-                     o.record_out ? s->d_out : (int*)nullptr, s->d_step, (const int*)(s->d_active ? s->d_active + b0 : nullptr),
-                     nb, o.S, s->out_capacity));
+                     o.record_out ? s->d_out : (int*)nullptr, s->d_step, act, nb, o.advance >= 0 ? o.advance : o.S, s->out_capacity));
     ++g_launch_total;
   }
   if (o.trace) RB_TRY(o.trace->mark(TC_HEAD));
@@ -1180,7 +1059,8 @@ int rewb200_model_create(int slot, const rewb200_config* cfg, rewb200_model** ou
   m->cfg.tp_size = tp;
   m->cfg.ep_size = std::max(1, cfg->ep_size);
   RB_REQUIRE(cfg->vocab % tp == 0, "shardLayout: vocabulary must be divisible by the tensor-parallel size");
-  m->vocab_l = cfg->vocab / tp;
+  m->vocab_l = m->vp = cfg->vocab / tp;
+  m->dp = cfg->d_model;
   m->nh_l = cfg->n_heads / tp;
   m->kvh_l = cfg->n_kv_heads / tp;
   m->nq = (int64_t)m->nh_l * cfg->head_dim;
@@ -1217,6 +1097,8 @@ int rewb200_model_create(int slot, const rewb200_config* cfg, rewb200_model** ou
     if (L.moe) {
       MoeDev& X = L.x;
       X.E_l = cfg->n_routed / m->cfg.ep_size;
+      X.E = cfg->n_routed;
+      X.top_k = cfg->top_k;
       X.f = cfg->moe_ffn;
       X.shared_down_bias.assign(d, 0.f);
       RB_TRY(alloc_lin(m, &X.router, d, cfg->n_routed));
@@ -1227,6 +1109,15 @@ int rewb200_model_create(int slot, const rewb200_config* cfg, rewb200_model** ou
       RB_CUDA(cudaMemsetAsync(X.gu_b, 0, (size_t)X.E_l * 2 * X.f * sizeof(float), c->stream));
       RB_CUDA(cudaMemsetAsync(X.down_b, 0, (size_t)X.E_l * d * sizeof(float), c->stream));
     }
+  }
+  for (const LayerDev& L : m->layers) {
+    m->max_ffn = std::max(m->max_ffn, L.ffn_local);
+    if (L.moe) ++m->n_moe;
+  }
+  if (cfg->n_routed > 0) {
+    m->max_moe_ffn = cfg->moe_ffn;
+    m->max_experts = cfg->n_routed;
+    m->max_topk = cfg->top_k;
   }
   RB_TRY(alloc_vec(&m->ng, 1.f));
   RB_TRY(alloc_vec(&m->nb, 0.f));
@@ -1242,6 +1133,36 @@ int rewb200_model_create(int slot, const rewb200_config* cfg, rewb200_model** ou
   return REWB200_OK;
 }
 
+int rewb200_model_create_layers(int slot, const rewb200_config* cfg, const rewb200_layer* layers, const rewb200_stack* stack,
+                                rewb200_model** out) {
+  Ctx* c = ctx_get(slot);
+  if (!c) return REWB200_ERR;
+  RB_REQUIRE(cfg && layers && stack && out, "rewb200_model_create_layers: NULL argument");
+  RB_CUDA(cudaSetDevice(c->device));
+  RB_REQUIRE(cfg->dtype == REWB200_F32 || cfg->dtype == REWB200_BF16, "model dtype must be f32 or bf16");
+  RB_REQUIRE(cfg->vocab > 0 && cfg->d_model > 0 && cfg->n_layers > 0 && cfg->max_seq > 0, "model dimensions must be positive");
+  RB_REQUIRE(cfg->tp_size <= 1 && cfg->ep_size <= 1 && cfg->weight_quant == 0, "layered models run unsharded and unquantised");
+  rewb200_model* m = new rewb200_model();
+  m->c = c;
+  m->slot = slot;
+  m->cfg = *cfg;
+  m->cfg.tp_size = m->cfg.ep_size = 1;
+  m->cfg.tp_rank = m->cfg.ep_rank = 0;
+  m->cfg.n_routed = m->cfg.n_shared = m->cfg.first_dense = 0;
+  m->cfg.norm_kind = 0;
+  m->cfg.mask_kind = 1;
+  m->vocab_l = cfg->vocab;
+  const int st = layered_create(m, layers, stack);
+  if (st != REWB200_OK) {
+    const std::string why = rewb200_last_error();
+    rewb200_model_free(m);
+    set_error(why);
+    return st;
+  }
+  *out = m;
+  return REWB200_OK;
+}
+
 void rewb200_model_free(rewb200_model* m) {
   if (!m) return;
   cudaSetDevice(m->c->device);
@@ -1253,6 +1174,7 @@ void rewb200_model_free(rewb200_model* m) {
 
 int64_t rewb200_model_tensor_count(const rewb200_model* m) {
   if (!m) return 0;
+  if (m->layered) return layered_tensor_count(m);
   int64_t n = 1;
   for (int l = 0; l < m->cfg.n_layers; ++l)
     n += 12 + (layer_is_moe(m->cfg, l) ? 2 + 6 * (int64_t)(m->cfg.n_shared + m->cfg.n_routed) : 6);
@@ -1273,6 +1195,10 @@ namespace {
 // one expert-parallel rank: *owner_ep is that rank, -1 for everything else.
 int tensor_partition(const rewb200_model* m, int64_t index, int* dim, int* ndims, int64_t* shape, int* owner_ep) {
   const rewb200_config& c = m->cfg;
+  if (m->layered) {
+    *dim = *owner_ep = -1;
+    return layered_tensor_shape(m, index, ndims, shape);
+  }
   TensorRef r;
   RB_TRY(locate(m, index, &r));
   const int64_t d = c.d_model, hd = c.head_dim;
@@ -1383,6 +1309,7 @@ namespace {
 int set_tensor_impl(rewb200_model* m, int64_t index, const float* host, int64_t numel, bool shard) {
   RB_REQUIRE(!m->finalized, "model already finalized");
   RB_CUDA(cudaSetDevice(m->c->device));
+  if (m->layered) return layered_set_tensor(m, index, host, numel);
   const rewb200_config& c = m->cfg;
   TensorRef r;
   RB_TRY(locate(m, index, &r));
@@ -1495,6 +1422,7 @@ int rewb200_model_init_random(rewb200_model* m, uint64_t seed, float std) {
   RB_REQUIRE(m, "rewb200_model_init_random: NULL model");
   RB_REQUIRE(!m->finalized, "model already finalized");
   RB_CUDA(cudaSetDevice(m->c->device));
+  if (m->layered) return layered_init_random(m, seed, std);
   Ctx* c = m->c;
   const int dt = m->cfg.dtype;
   // replicated tensors (the embedding) use the seed alone; sharded ones also mix in the rank
@@ -1555,7 +1483,8 @@ int rewb200_model_finalize(rewb200_model* m) {
       }
     }
   }
-  if (m->cfg.dtype == REWB200_BF16) {
+  if (m->layered) RB_TRY(layered_plans(m));
+  if (m->cfg.dtype == REWB200_BF16 && !m->layered) {
     for (LayerDev& L : m->layers) {
       RB_TRY(linear_bf16_plan(&L.qkv.plan, (const bf16*)L.qkv.w, L.qkv.K, L.qkv.N, 0));
       RB_TRY(linear_bf16_plan(&L.o.plan, (const bf16*)L.o.w, L.o.K, L.o.N, 0));
@@ -1572,7 +1501,7 @@ int rewb200_model_finalize(rewb200_model* m) {
     RB_TRY(linear_bf16_plan(&m->lm.plan, (const bf16*)m->lm.w, m->lm.K, m->lm.N, 0));
   }
   for (LayerDev& L : m->layers)  // shared experts' down biases were summed on the host
-    if (L.moe && L.ffn_local > 0)
+    if (!m->layered && L.moe && L.ffn_local > 0)
       RB_CUDA(cudaMemcpyAsync(L.down.b, L.x.shared_down_bias.data(), m->cfg.d_model * sizeof(float), cudaMemcpyHostToDevice,
                               m->c->stream));
   if (m->stage) {
@@ -1619,21 +1548,25 @@ static int session_fill(rewb200_session* s, int batch, int max_len, int num_bloc
   s->paged = num_blocks > 0;
   s->num_blocks = num_blocks;
   const int64_t n_pages = s->paged ? (int64_t)num_blocks : (int64_t)batch * s->max_pages;
-  const size_t es = dtype_size(m->cfg.dtype);
-  const int64_t cache_rows = n_pages * m->kvh_l * PAGE;
-  const size_t cache_bytes = (size_t)cache_rows * m->cfg.head_dim * es;
-  s->kc.resize(m->cfg.n_layers);
-  s->vc.resize(m->cfg.n_layers);
-  s->tmK.resize(m->cfg.n_layers);
-  s->tmV.resize(m->cfg.n_layers);
-  for (int l = 0; l < m->cfg.n_layers; ++l) {
-    RB_CUDA(cudaMalloc(&s->kc[l], cache_bytes));
-    RB_CUDA(cudaMalloc(&s->vc[l], cache_bytes));
-    RB_CUDA(cudaMemsetAsync(s->kc[l], 0, cache_bytes, c->stream));
-    RB_CUDA(cudaMemsetAsync(s->vc[l], 0, cache_bytes, c->stream));
-    if (m->cfg.dtype == REWB200_BF16) {
-      RB_TRY(make_tmap_2d_bf16(&s->tmK[l], s->kc[l], m->cfg.head_dim, cache_rows, (uint64_t)m->cfg.head_dim * 2, 64, 64));
-      RB_TRY(make_tmap_2d_bf16(&s->tmV[l], s->vc[l], m->cfg.head_dim, cache_rows, (uint64_t)m->cfg.head_dim * 2, 64, 64));
+  if (m->layered) {
+    RB_TRY(layered_session(s, n_pages));
+  } else {
+    const size_t es = dtype_size(m->cfg.dtype);
+    const int64_t cache_rows = n_pages * m->kvh_l * PAGE;
+    const size_t cache_bytes = (size_t)cache_rows * m->cfg.head_dim * es;
+    s->kc.resize(m->cfg.n_layers);
+    s->vc.resize(m->cfg.n_layers);
+    s->tmK.resize(m->cfg.n_layers);
+    s->tmV.resize(m->cfg.n_layers);
+    for (int l = 0; l < m->cfg.n_layers; ++l) {
+      RB_CUDA(cudaMalloc(&s->kc[l], cache_bytes));
+      RB_CUDA(cudaMalloc(&s->vc[l], cache_bytes));
+      RB_CUDA(cudaMemsetAsync(s->kc[l], 0, cache_bytes, c->stream));
+      RB_CUDA(cudaMemsetAsync(s->vc[l], 0, cache_bytes, c->stream));
+      if (m->cfg.dtype == REWB200_BF16) {
+        RB_TRY(make_tmap_2d_bf16(&s->tmK[l], s->kc[l], m->cfg.head_dim, cache_rows, (uint64_t)m->cfg.head_dim * 2, 64, 64));
+        RB_TRY(make_tmap_2d_bf16(&s->tmV[l], s->vc[l], m->cfg.head_dim, cache_rows, (uint64_t)m->cfg.head_dim * 2, 64, 64));
+      }
     }
   }
   const int64_t n_bt = (int64_t)batch * s->max_pages;
@@ -1662,7 +1595,7 @@ static int session_fill(rewb200_session* s, int batch, int max_len, int num_bloc
   RB_CUDA(cudaMallocHost((void**)&s->h_ids, (size_t)batch * max_len * sizeof(int)));
   RB_CUDA(cudaMemsetAsync(s->d_pos, 0, batch * sizeof(int), c->stream));
   RB_CUDA(cudaMemsetAsync(s->d_step, 0, sizeof(int), c->stream));
-  s->attn_scratch_bytes = attn_scratch_bytes(batch, m->nh_l, m->cfg.head_dim, 16);
+  s->attn_scratch_bytes = m->layered ? 256 : attn_scratch_bytes(batch, m->nh_l, m->cfg.head_dim, 16);
   RB_CUDA(cudaMalloc((void**)&s->attn_scratch, s->attn_scratch_bytes));
   RB_CUDA(cudaMalloc(&s->argmax_scratch, (size_t)batch * 64 * 8));
   if (m->cfg.tp_size > 1) {
@@ -1699,7 +1632,8 @@ void rewb200_session_free(rewb200_session* s) {
   void* ptrs[] = {s->d_active, s->d_ids_prefill, s->block_table, s->d_pos, s->d_ids, s->d_next, s->d_out, s->d_step, s->x_res, s->xn, s->q,
                   s->attn, s->h, s->part, s->gu32, s->logits, s->attn_scratch, s->argmax_scratch, s->gather_scratch,
                   s->samp_hist, s->samp_hist_len, s->samp_steps, s->samp_keys, s->samp_work, s->samp_logprob, s->moe_logits, s->moe_topw, s->moe_topi, s->moe_ints,
-                  s->moe_send, s->moe_recv, s->moe_xs, s->moe_hs, s->moe_ys, s->moe_ret, s->moe_back, s->moe_tmp, s->route_rec};
+                  s->moe_send, s->moe_recv, s->moe_xs, s->moe_hs, s->moe_ys, s->moe_ret, s->moe_back, s->moe_tmp, s->route_rec,
+                  s->xn2, s->cq, s->gate, s->part2, s->qeff, s->olat, s->ml, s->kvx, s->latx, s->layer_rec, s->xg, s->logits_pad, s->plan_dev, s->feed_dev};
   for (void* p : ptrs)
     if (p) cudaFree(p);
   if (s->h_ids) cudaFreeHost(s->h_ids);
@@ -1734,6 +1668,15 @@ int rewb200_session_forward(rewb200_session* s, const int32_t* ids, int S, int32
   for (int64_t i = 0; i < rows; ++i)
     RB_REQUIRE(ids[i] >= 0 && ids[i] < m->cfg.vocab, "generate: token id out of range at index " + std::to_string(i));
   RB_TRY(ensure_acts(s, rows, s->B));
+  FwdOpts o;
+  o.S = S;
+  std::vector<StepEntry> entries;
+  if (m->layered) {
+    RB_TRY(ensure_head_rows(s, s->B));
+    entries = uniform_entries(s, 0, s->B, S, s->host_pos);
+    o.entries = &entries;
+    RB_TRY(layered_prepare(s, o, rows));
+  }
   memcpy(s->h_ids, ids, rows * sizeof(int32_t));
   RB_CUDA(cudaEventRecord(s->ev0, c->stream));
   RB_CUDA(cudaMemcpyAsync(s->d_ids, s->h_ids, rows * sizeof(int32_t), cudaMemcpyHostToDevice, c->stream));
@@ -1747,8 +1690,6 @@ int rewb200_session_forward(rewb200_session* s, const int32_t* ids, int S, int32
     RB_CUDA(cudaGetLastError());
     ++g_launch_total;
   }
-  FwdOpts o;
-  o.S = S;
   RB_TRY(enqueue_forward(s, o));
   RB_CUDA(cudaEventRecord(s->ev1, c->stream));
   if (next_ids)
@@ -1770,6 +1711,10 @@ static int decode_core(rewb200_session* s, int n_steps, int32_t* out_ids, float*
   RB_TRY(ensure_acts(s, std::max<int64_t>(s->B, s->rows_cap), s->B));
   FwdOpts o;
   o.S = 1;
+  if (m->layered) {
+    RB_TRY(ensure_head_rows(s, s->B));
+    RB_TRY(layered_prepare(s, o, s->B));
+  }
   const char* nograph = getenv("REW_B200_NO_GRAPH");
   const bool use_graph = !(nograph && nograph[0] == '1');
   if (s->graph && s->graph_epoch != c->option_epoch) {
@@ -1968,6 +1913,13 @@ int rewb200_lane_admit(rewb200_session* s, int lane, const int32_t* ids, int S, 
   o.nb = 1;
   o.ids_src = s->d_ids_prefill;
   o.record_out = false;
+  std::vector<StepEntry> entries;
+  if (m->layered) {
+    RB_TRY(ensure_head_rows(s, s->B));
+    entries = uniform_entries(s, lane, 1, S, 0);
+    o.entries = &entries;
+    RB_TRY(layered_prepare(s, o, S));
+  }
   RB_TRY(enqueue_forward(s, o));
   RB_CUDA(cudaEventRecord(s->ev1, c->stream));
   int32_t first = -1;
@@ -2001,6 +1953,145 @@ int rewb200_lanes_step(rewb200_session* s, int n_steps, int32_t* out_ids) {
   for (int b = 0; b < s->B; ++b)
     if (s->lane_active[b]) s->lane_len[b] += n_steps;
   return REWB200_OK;
+}
+
+int rewb200_lanes_feed(rewb200_session* s, int n_entries, const int32_t* lanes, const int32_t* counts, const int32_t* ids,
+                       int n_want, const int32_t* want, float* logits_out, const int32_t* sample, const uint64_t* seeds,
+                       int32_t* next_ids) {
+  RB_TRY(lane_check(s, 0, "rewb200_lanes_feed"));
+  RB_REQUIRE(n_entries > 0 && lanes && counts && ids, "rewb200_lanes_feed: a step needs at least one portion");
+  RB_REQUIRE(n_want >= 0 && (n_want == 0 || (want && logits_out)), "rewb200_lanes_feed: wanted places without a place for their logits");
+  rewb200_model* m = s->m;
+  Ctx* c = m->c;
+  RB_CUDA(cudaSetDevice(c->device));
+  // ---- checks first: nothing changes unless the whole step can run
+  std::vector<StepEntry> entries;
+  std::vector<char> seen(s->B, 0);
+  int64_t rows = 0;
+  int need = 0;
+  for (int e = 0; e < n_entries; ++e) {
+    const int l = lanes[e];
+    RB_TRY(lane_check(s, l, "rewb200_lanes_feed"));
+    RB_REQUIRE(!seen[l], "rewb200_lanes_feed: lane " + std::to_string(l) + " appears twice in one step");
+    seen[l] = 1;
+    RB_REQUIRE(counts[e] > 0, "rewb200_lanes_feed: a portion must not be empty");
+    const int pos0 = s->lane_active[l] ? s->lane_len[l] : 0;
+    RB_REQUIRE((int64_t)pos0 + counts[e] <= s->max_len, "KvCache.append: total length " + std::to_string((int64_t)pos0 + counts[e]) +
+                                                            " of lane " + std::to_string(l) + " exceeds maxLen " + std::to_string(s->max_len));
+    entries.push_back({l, (int)rows, counts[e], pos0});
+    rows += counts[e];
+    need += std::max(0, (pos0 + counts[e] + PAGE - 1) / PAGE - (int)s->lane_pages[l].size());
+  }
+  for (int64_t i = 0; i < rows; ++i)
+    RB_REQUIRE(ids[i] >= 0 && ids[i] < m->cfg.vocab, "generate: token id out of range at index " + std::to_string(i));
+  for (int i = 0; i < n_want; ++i)
+    RB_REQUIRE(want[i] >= 0 && want[i] < rows && (i == 0 || want[i] > want[i - 1]), "rewb200_lanes_feed: wanted places must ascend within the step");
+  RB_REQUIRE(need <= (int)s->free_blocks.size(), "PagedKvCache: out of free blocks (" + std::to_string(need) + " needed for the step, " +
+                                                     std::to_string(s->free_blocks.size()) + " free)");
+  // ---- activations, positions, pages
+  RB_TRY(ensure_acts(s, std::max<int64_t>(std::max<int64_t>(rows, s->B), s->rows_cap), (int64_t)n_want + s->B));
+  RB_TRY(ensure_head_rows(s, (int64_t)n_want + s->B));
+  bool any_sample = false;
+  std::vector<int> act(s->B, 0);
+  for (int e = 0; e < n_entries; ++e)
+    if (next_ids && (!sample || sample[e])) {
+      act[lanes[e]] = 1;
+      any_sample = true;
+    }
+  RB_CUDA(cudaStreamSynchronize(c->stream));  // the host-side tables below are read by no kernel in flight
+  for (const StepEntry& e : entries) {
+    RB_TRY(lane_reserve(s, e.lane, e.pos0 + e.n));
+    if (!s->lane_active[e.lane]) {
+      const int one = 1;
+      RB_CUDA(cudaMemcpy(s->d_active + e.lane, &one, sizeof(int), cudaMemcpyHostToDevice));
+      s->lane_active[e.lane] = 1;
+      s->lane_len[e.lane] = 0;
+      if (s->samp_on) {
+        const uint64_t seed = seeds ? seeds[&e - &entries[0]] : 0;
+        s->samp_seeds[e.lane] = seed;
+        const uint32_t k[2] = {(uint32_t)(seed & 0xFFFFFFFFull), (uint32_t)(seed >> 32)};
+        const int zero = 0;
+        RB_CUDA(cudaMemcpy(s->samp_keys + 2 * e.lane, k, sizeof(k), cudaMemcpyHostToDevice));
+        RB_CUDA(cudaMemcpy(s->samp_steps + e.lane, &zero, sizeof(int), cudaMemcpyHostToDevice));
+      }
+    }
+    if (s->samp_on) {  // tokens seen so far = everything fed to the model
+      const int n = e.pos0 + e.n;
+      RB_CUDA(cudaMemcpy(s->samp_hist + (size_t)e.lane * s->max_len + e.pos0, ids + e.row0, (size_t)e.n * sizeof(int), cudaMemcpyHostToDevice));
+      RB_CUDA(cudaMemcpy(s->samp_hist_len + e.lane, &n, sizeof(int), cudaMemcpyHostToDevice));
+    }
+    RB_CUDA(cudaMemcpy(s->d_pos + e.lane, &e.pos0, sizeof(int), cudaMemcpyHostToDevice));
+  }
+  // one upload: ids | rows of the lm_head (wanted places, then every lane's last row) | sampled lanes
+  std::vector<int> up((size_t)rows + n_want + s->B + s->B, 0);
+  memcpy(up.data(), ids, (size_t)rows * sizeof(int));
+  for (int i = 0; i < n_want; ++i) up[(size_t)rows + i] = want[i];
+  for (const StepEntry& e : entries) up[(size_t)rows + n_want + e.lane] = e.row0 + e.n - 1;
+  for (int b = 0; b < s->B; ++b) up[(size_t)rows + n_want + s->B + b] = act[b];
+  if (up.size() > s->feed_cap) {
+    if (s->feed_dev) RB_CUDA(cudaFree(s->feed_dev));
+    s->feed_dev = nullptr;
+    s->feed_cap = 0;
+    RB_CUDA(cudaMalloc((void**)&s->feed_dev, up.size() * sizeof(int)));
+    s->feed_cap = up.size();
+  }
+  RB_CUDA(cudaMemcpy(s->feed_dev, up.data(), up.size() * sizeof(int), cudaMemcpyHostToDevice));
+  const int* d_rows = s->feed_dev + rows;
+  const int* d_act = s->feed_dev + rows + n_want + s->B;
+  RB_CUDA(cudaEventRecord(s->ev0, c->stream));
+  if (m->layered) {
+    FwdOpts o;
+    o.entries = &entries;
+    o.ids_src = s->feed_dev;
+    o.record_out = false;
+    o.out_rows = d_rows;
+    o.n_want = n_want;
+    o.sample = any_sample;
+    o.sample_active = d_act;
+    o.advance = 0;
+    RB_TRY(layered_prepare(s, o, rows));
+    RB_TRY(enqueue_forward(s, o));
+    if (n_want > 0)
+      RB_CUDA(cudaMemcpyAsync(logits_out, s->logits, (size_t)n_want * m->cfg.vocab * sizeof(float), cudaMemcpyDeviceToHost, c->stream));
+  } else {
+    int w0 = 0;
+    for (const StepEntry& e : entries) {
+      // this portion's wanted places, relative to its first row, then its last row
+      int w1 = w0;
+      std::vector<int> list;
+      while (w1 < n_want && want[w1] < e.row0 + e.n) list.push_back(want[w1++] - e.row0);
+      list.push_back(e.n - 1);
+      RB_CUDA(cudaMemcpyAsync(s->feed_dev + rows, list.data(), list.size() * sizeof(int), cudaMemcpyHostToDevice, c->stream));
+      FwdOpts o;
+      o.S = e.n;
+      o.b0 = e.lane;
+      o.nb = 1;
+      o.ids_src = s->feed_dev + e.row0;
+      o.record_out = false;
+      o.out_rows = d_rows;
+      o.n_want = w1 - w0;
+      o.sample = act[e.lane] != 0;
+      o.advance = 0;
+      RB_TRY(enqueue_forward(s, o));
+      if (w1 > w0)
+        RB_CUDA(cudaMemcpyAsync(logits_out + (size_t)w0 * m->cfg.vocab, s->logits, (size_t)(w1 - w0) * m->cfg.vocab * sizeof(float),
+                                cudaMemcpyDeviceToHost, c->stream));
+      RB_CUDA(cudaStreamSynchronize(c->stream));  // `list` and the shared row list are reused by the next portion
+      w0 = w1;
+    }
+  }
+  RB_CUDA(cudaEventRecord(s->ev1, c->stream));
+  std::vector<int> next(s->B, -1);
+  if (any_sample) RB_CUDA(cudaMemcpyAsync(next.data(), s->d_next, s->B * sizeof(int), cudaMemcpyDeviceToHost, c->stream));
+  RB_CUDA(cudaStreamSynchronize(c->stream));
+  RB_CUDA(cudaEventElapsedTime(&s->prefill_ms, s->ev0, s->ev1));
+  for (const StepEntry& e : entries) {
+    s->lane_len[e.lane] = e.pos0 + e.n;
+    RB_CUDA(cudaMemcpy(s->d_pos + e.lane, &s->lane_len[e.lane], sizeof(int), cudaMemcpyHostToDevice));
+  }
+  if (next_ids)
+    for (int e = 0; e < n_entries; ++e) next_ids[e] = act[lanes[e]] ? next[lanes[e]] : -1;
+  return ctx_check_status(c);
 }
 
 int rewb200_lane_release(rewb200_session* s, int lane) {
@@ -2164,14 +2255,27 @@ int rewb200_session_graph_kernels(const rewb200_session* s) { return s ? s->grap
 int rewb200_session_routing(rewb200_session* s, int moe_layer, int32_t* topi_out, int64_t rows) {
   RB_REQUIRE(s && topi_out, "rewb200_session_routing: NULL argument");
   RB_REQUIRE(s->route_rec != nullptr, "rewb200_session_routing: set option record_routing=1 before the session's first forward");
-  int n_moe = 0;
-  for (const LayerDev& L : s->m->layers) n_moe += L.moe ? 1 : 0;
+  const int n_moe = s->m->n_moe;
   RB_REQUIRE(moe_layer >= 0 && moe_layer < n_moe && rows == s->route_rows, "rewb200_session_routing: layer or row count does not match the last forward");
   Ctx* c = s->m->c;
   RB_CUDA(cudaSetDevice(c->device));
   RB_CUDA(cudaStreamSynchronize(c->stream));
-  RB_CUDA(cudaMemcpy(topi_out, s->route_rec + (size_t)moe_layer * s->rows_cap * s->m->cfg.top_k,
-                     (size_t)rows * s->m->cfg.top_k * sizeof(int), cudaMemcpyDeviceToHost));
+  RB_CUDA(cudaMemcpy(topi_out, s->route_rec + (size_t)moe_layer * s->rows_cap * s->m->max_topk,
+                     (size_t)rows * s->m->max_topk * sizeof(int), cudaMemcpyDeviceToHost));
+  return REWB200_OK;
+}
+
+int rewb200_session_layers(rewb200_session* s, float* out, int64_t rows) {
+  RB_REQUIRE(s && out, "rewb200_session_layers: NULL argument");
+  RB_REQUIRE(s->layer_rec != nullptr && rows == s->layer_rows, "rewb200_session_layers: set option record_layers=1 before the session's first "
+                                                              "forward, and ask for the rows of the last step");
+  Ctx* c = s->m->c;
+  RB_CUDA(cudaSetDevice(c->device));
+  RB_CUDA(cudaStreamSynchronize(c->stream));
+  const int64_t d = s->m->cfg.d_model, dp = s->m->dp;
+  for (size_t r = 0; r < s->m->runs.size(); ++r)
+    RB_CUDA(cudaMemcpy2D(out + (size_t)r * rows * d, d * sizeof(float), s->layer_rec + r * s->rows_cap * dp, dp * sizeof(float),
+                         d * sizeof(float), rows, cudaMemcpyDeviceToHost));
   return REWB200_OK;
 }
 
@@ -2186,6 +2290,7 @@ int rewb200_session_trace_step(rewb200_session* s, float* ms_by_category, int n)
   FwdOpts o;
   o.S = 1;
   o.trace = &tr;
+  if (m->layered) RB_TRY(layered_prepare(s, o, s->B));
   RB_TRY(enqueue_forward(s, o));
   RB_TRY(tr.finish(ms_by_category));
   s->host_pos += 1;
@@ -2215,6 +2320,14 @@ int rewb200_model_forward_all(rewb200_session* s, const int32_t* ids, int S, int
   o.rope_shift = (int)offset;
   o.causal = causal;
   o.all_logits = true;
+  std::vector<StepEntry> entries;
+  if (m->layered) {
+    RB_REQUIRE(causal && offset == 0, "layered models: the cache-free forward is causal and starts at position 0");
+    RB_TRY(ensure_head_rows(s, rows));
+    entries = uniform_entries(s, 0, s->B, S, 0);
+    o.entries = &entries;
+    RB_TRY(layered_prepare(s, o, rows));
+  }
   RB_TRY(enqueue_forward(s, o));
   RB_TRY(fetch_logits(s, rows, logits_out));
   return ctx_check_status(c);

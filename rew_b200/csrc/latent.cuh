@@ -1,0 +1,98 @@
+// Latent attention (multi-head attention whose keys and values are linear in a cached low-rank latent): argument
+// structs and launchers of latent.cu.
+//
+// Per token the cache row holds [c (kv_rank) | k_rot (rot_dim)], shared by all heads.  A head's score against a key
+// is q_nope . (W_uk c) + q_rot . k_rot = [W_uk^T q_nope | q_rot] . [c | k_rot], and its output is
+// W_uv (sum_j p_j c_j), so attention can run on the cache rows themselves ("absorbed": small steps, decode) or on
+// keys and values expanded from them per head (large prompt portions).
+#pragma once
+#include "common.cuh"
+
+namespace rewb {
+
+// Which sequence (lane) and position a row of the step belongs to: explicit arrays (a step of unequal portions), or
+// S consecutive tokens for every lane from b0 on, starting at the lane's position pos0[lane].
+struct RowMap {
+  const int* row_lane;
+  const int* row_pos;
+  const int* pos0;
+  int b0, S;
+};
+
+// Runs of consecutive rows of one lane: an explicit list of (first row, rows), or (list == nullptr) the rows of
+// every lane of a uniform step in pieces of `per_tile`.
+struct RowTiles {
+  const int2* list;
+  int count;      // tiles
+  int S;          // rows per lane (list == nullptr)
+  int per_tile;   // rows per tile at most
+};
+
+struct LatentDims {
+  int heads, dim, rot_dim, vdim, q_rank, kv_rank;
+  int rope_dims;           // rotated features of the rot_dim part (interleaved pairs), the rest passes unchanged
+  int window;              // keys a query sees, itself included; 0: all
+  int gate;                // per-head output gate
+  float scale;
+  const float2* rope;      // [max_pos][rope_dims / 2] (cos, sin)
+  int max_pos;
+};
+
+// Finishes the fused input projection [q_rank | kv_rank | rot_dim | heads]: sums the split-K slabs, norms the query
+// latent and the key/value latent, rotates the shared key part, appends [c | k_rot] to the cache, applies the
+// sigmoid of the output gate.
+struct LatentPostArgs {
+  LatentDims m;
+  const float* partial;    // [nsplit][rows][ld]
+  int nsplit;
+  int64_t split_stride, ld;
+  const float *q_norm, *kv_norm;
+  float eps;
+  RowMap map;
+  void* cq;                // [rows][ldcq] act dtype
+  int64_t ldcq;
+  float* gate;             // [rows][heads]
+  void* cache;             // [pages][64][ldc]
+  const int* block_table;  // [lanes][max_pages]
+  int max_pages, capacity;
+  int64_t ldc;
+  int dtype;
+  int* status;
+};
+int latent_post_launch(Ctx* c, const LatentPostArgs& a, int64_t rows);
+
+// Absorbed attention of the rows in `tiles`.
+struct LatentAttnArgs {
+  LatentDims m;
+  RowMap map;
+  RowTiles tiles;
+  int max_tile_rows;       // rows of the longest tile
+  int64_t rows;            // rows of the whole step
+  // queries: either split-K slabs f32 [nsplit][rows][ldq] or (nsplit == 0) act dtype [rows][ldq]
+  const void* q;
+  int nsplit;
+  int64_t split_stride, ldq;
+  const void* ukv;         // [kv_rank][ld_ukv] act dtype: columns heads*dim of keys, then heads*vdim of values
+  int64_t ld_ukv;
+  void* qeff;              // scratch [rows][heads][ldc] act dtype
+  float* olat;             // scratch [rows][heads][kv splits][kv_rank] f32, not yet divided by the row sum
+  float2* ml;              // scratch [rows][heads][kv splits] running maximum and sum
+  int kv_splits;
+  const float* gate;       // [rows][heads]
+  void* out;               // [rows][ldo] act dtype, head-major columns
+  int64_t ldo;
+  const void* cache;
+  const CUtensorMap* tm_cache;  // bf16: [pages * 64][ldc], box 64 x 64
+  const int* block_table;
+  int max_pages;
+  int64_t ldc;
+  int dtype;
+  int* status;
+};
+int latent_attn_absorbed_launch(Ctx* c, const LatentAttnArgs& a);
+int latent_kv_splits(Ctx* c, const LatentDims& m, int64_t tiles, int64_t max_ctx);
+
+// Gathers rows of the step: dst[i] = src[index[i]] (width elements of `dtype`).
+int gather_rows_launch(Ctx* c, const void* src, const int* index, void* dst, int64_t n, int64_t width, int dtype);
+
+}  // namespace rewb

@@ -234,6 +234,10 @@ __global__ void __launch_bounds__(160) linear_bf16_kernel(const __grid_constant_
               float* o = reinterpret_cast<float*>(a.out) + grow * a.ldo + c;
               *reinterpret_cast<float2*>(o) = make_float2(v0, v1);
             } else {
+              if (a.epi == EPI_RELU2_BF16) {
+                v0 = fmaxf(v0, 0.f) * fmaxf(v0, 0.f);
+                v1 = fmaxf(v1, 0.f) * fmaxf(v1, 0.f);
+              }
               bf16* o = reinterpret_cast<bf16*>(a.out) + grow * a.ldo + c;
               *reinterpret_cast<uint32_t*>(o) = pack_bf16(v0, v1);
             }

@@ -81,6 +81,12 @@ __device__ __forceinline__ float ld_dsmem_f32(uint32_t cluster_addr) {
 }
 
 __device__ __forceinline__ float silu_f(float x) { return x * (1.0f / (1.0f + __expf(-x))); }
+// bf16 outputs: the square of relu (EPI_RELU2_BF16) or the value itself
+__device__ __forceinline__ float act_f(float v, bool relu2) {
+  if (!relu2) return v;
+  v = fmaxf(v, 0.f);
+  return v * v;
+}
 
 // Second half of the cluster split-K epilogue, run by the four epilogue warps of every CTA after the
 // cluster barrier: this CTA finishes tokens [rank * 32/KS, (rank+1) * 32/KS) of the tile.  All loads of
@@ -359,13 +365,14 @@ __global__ void __launch_bounds__(192) linear_tc_kernel(const __grid_constant__ 
             else if (a.epi == EPI_BIAS_F32)
               reinterpret_cast<float*>(a.out)[grow * a.ldo + feat] = v;
             else
-              reinterpret_cast<bf16*>(a.out)[grow * a.ldo + feat] = __float2bfloat16_rn(v);
+              reinterpret_cast<bf16*>(a.out)[grow * a.ldo + feat] = __float2bfloat16_rn(act_f(v, a.epi == EPI_RELU2_BF16));
           }
         }
       }
     } else {
       const bool swiglu = a.epi == EPI_SWIGLU_BF16;
       const bool out_f32 = a.epi == EPI_PARTIAL_F32 || a.epi == EPI_BIAS_F32;
+      const bool relu2 = a.epi == EPI_RELU2_BF16;
       const int tile_cols = swiglu ? 64 : 128;
       const int row_bytes = tile_cols * (out_f32 ? 4 : 2);
       uint8_t* stg = smem;
@@ -400,7 +407,7 @@ __global__ void __launch_bounds__(192) linear_tc_kernel(const __grid_constant__ 
           } else {
   #pragma unroll
             for (int j = 0; j < 32; ++j)
-              reinterpret_cast<bf16*>(stg + (c0 + j) * row_bytes)[q * 32 + lane] = __float2bfloat16_rn(__uint_as_float(r[j]) + bias_v);
+              reinterpret_cast<bf16*>(stg + (c0 + j) * row_bytes)[q * 32 + lane] = __float2bfloat16_rn(act_f(__uint_as_float(r[j]) + bias_v, relu2));
           }
         }
       }
@@ -631,6 +638,7 @@ __global__ void __launch_bounds__(192) linear_tc_persist_kernel(const __grid_con
     const int et = threadIdx.x - 64;
     const bool swiglu = a.epi == EPI_SWIGLU_BF16;
     const bool out_f32 = a.epi == EPI_PARTIAL_F32 || a.epi == EPI_BIAS_F32;
+    const bool relu2 = a.epi == EPI_RELU2_BF16;
     const int tile_cols = swiglu ? 64 : 128;
     const int row_bytes = tile_cols * (out_f32 ? 4 : 2);
     const int chunks_per_row = row_bytes / 16;
@@ -667,7 +675,7 @@ __global__ void __launch_bounds__(192) linear_tc_persist_kernel(const __grid_con
           } else {
 #pragma unroll
             for (int jj = 0; jj < 32; ++jj)
-              reinterpret_cast<bf16*>(stg + jj * C::STG_LD)[q * 32 + lane] = __float2bfloat16_rn(__uint_as_float(r[jj]) + bias_v);
+              reinterpret_cast<bf16*>(stg + jj * C::STG_LD)[q * 32 + lane] = __float2bfloat16_rn(act_f(__uint_as_float(r[jj]) + bias_v, relu2));
           }
         }
         asm volatile("bar.sync 1, 128;" ::: "memory");  // the four epilogue warps only
@@ -882,6 +890,7 @@ __global__ void __cluster_dims__(2, 1, 1) __launch_bounds__(192) linear_tc_pair_
     const int et = threadIdx.x - 64;
     const bool swiglu = a.epi == EPI_SWIGLU_BF16;
     const bool out_f32 = a.epi == EPI_PARTIAL_F32 || a.epi == EPI_BIAS_F32;
+    const bool relu2 = a.epi == EPI_RELU2_BF16;
     const int tile_cols = swiglu ? 64 : 128;
     const int row_bytes = tile_cols * (out_f32 ? 4 : 2);
     const int chunks_per_row = row_bytes / 16;
@@ -918,7 +927,7 @@ __global__ void __cluster_dims__(2, 1, 1) __launch_bounds__(192) linear_tc_pair_
           } else {
 #pragma unroll
             for (int jj = 0; jj < 32; ++jj)
-              reinterpret_cast<bf16*>(stg + jj * C::STG_LD)[q * 32 + lane] = __float2bfloat16_rn(__uint_as_float(r[jj]) + bias_v);
+              reinterpret_cast<bf16*>(stg + jj * C::STG_LD)[q * 32 + lane] = __float2bfloat16_rn(act_f(__uint_as_float(r[jj]) + bias_v, relu2));
           }
         }
         asm volatile("bar.sync 1, 128;" ::: "memory");  // the four epilogue warps only

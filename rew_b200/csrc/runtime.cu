@@ -290,6 +290,11 @@ int rewb200_set_option(int slot, const char* key, const char* value) {
     c->tp_twoshot = v == "heap";
   } else if (k == "record_routing") {
     c->record_routing = v != "0";
+  } else if (k == "record_layers") {
+    c->record_layers = v != "0";
+  } else if (k == "latent_attention") {
+    RB_REQUIRE(v == "auto" || v == "plain" || v == "absorbed", "option latent_attention: expected auto, plain or absorbed");
+    c->latent_impl = v == "plain" ? 1 : v == "absorbed" ? 2 : 0;
   } else if (k == "inject_alloc_fail") {
     const int n = atoi(v.c_str());
     RB_REQUIRE(n >= 0, "option inject_alloc_fail: a non-negative count");

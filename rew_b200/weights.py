@@ -66,7 +66,9 @@ def deepseek_v2_lite(**kw):
 
 
 def tensor_specs(cfg):
-    """[(name, shape)] in canonical order; every Linear is weight [in,out] then bias [out]."""
+    """[(name, shape)] in canonical order; every Linear is weight [in,out] then bias [out] (layered models: LayeredConfig)."""
+    if hasattr(cfg, "tensor_specs"):
+        return cfg.tensor_specs()
     d, hd = cfg.d_model, cfg.head_dim
     nq, nkv = cfg.n_heads * hd, cfg.n_kv_heads * hd
     specs = [("model.embedTokens.weight", (cfg.vocab, d))]
