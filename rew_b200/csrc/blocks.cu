@@ -120,8 +120,8 @@ int rope_table(rewb200_model* m, double base, int dims, float2** out) {
       t[(size_t)p * (dims / 2) + i] = make_float2((float)std::cos(p * f), (float)std::sin(p * f));
   }
   RB_TRY(dev_alloc(m, (void**)out, t.size() * sizeof(float2)));
+  if (!t.empty()) RB_CUDA(cudaMemcpyAsync(*out, t.data(), t.size() * sizeof(float2), cudaMemcpyHostToDevice, m->c->stream));
   RB_CUDA(cudaStreamSynchronize(m->c->stream));
-  if (!t.empty()) RB_CUDA(cudaMemcpy(*out, t.data(), t.size() * sizeof(float2), cudaMemcpyHostToDevice));
   return REWB200_OK;
 }
 
@@ -360,9 +360,9 @@ int layered_acts(rewb200_session* s, int64_t rows) {
   RB_TRY(acts_alloc(c, (void**)&s->part2, s->part_bytes));
   if (c->record_layers) RB_TRY(acts_alloc(c, (void**)&s->layer_rec, m->runs.size() * (size_t)rows * m->dp * sizeof(float)));
   // padding columns are multiplied by zero weights, so they must hold finite values from the start
-  RB_CUDA(cudaMemset(s->cq, 0, (size_t)rows * cq * es));
-  RB_CUDA(cudaMemset(s->attn, 0, (size_t)rows * m->nq * es));
-  RB_CUDA(cudaMemset(s->h, 0, (size_t)rows * std::max<int64_t>(std::max(m->max_ffn, m->max_moe_ffn), 1) * es));
+  RB_CUDA(cudaMemsetAsync(s->cq, 0, (size_t)rows * cq * es, c->stream));
+  RB_CUDA(cudaMemsetAsync(s->attn, 0, (size_t)rows * m->nq * es, c->stream));
+  RB_CUDA(cudaMemsetAsync(s->h, 0, (size_t)rows * std::max<int64_t>(std::max(m->max_ffn, m->max_moe_ffn), 1) * es, c->stream));
   return REWB200_OK;
 }
 
@@ -435,6 +435,10 @@ int layered_prepare(rewb200_session* s, const FwdOpts& o, int64_t rows) {
       for (int i = 0; i < e.n; i += ABS_TILE_ROWS) tiles.push_back(make_int2(e.row0 + i, std::min(ABS_TILE_ROWS, e.n - i)));
     }
     s->plan_abs_tiles = (int)tiles.size();
+    // the same rows in longer runs, whatever their lanes, for the per-head products around the attention
+    s->plan_chunks = 0;
+    for (int64_t i = 0; i < rows; i += kChunkRows, ++s->plan_chunks)
+      tiles.push_back(make_int2((int)i, (int)std::min<int64_t>(kChunkRows, rows - i)));
     const size_t at = h.size();
     h.resize(at + 2 * tiles.size());
     if (!tiles.empty()) memcpy(h.data() + at, tiles.data(), tiles.size() * sizeof(int2));
@@ -462,7 +466,7 @@ int layered_prepare(rewb200_session* s, const FwdOpts& o, int64_t rows) {
   if (abs_rows * qe > s->abs_rows) {
     s->abs_rows = 0;
     RB_TRY(regrow(s, &s->qeff, (size_t)abs_rows * qe * es));
-    RB_CUDA(cudaMemset(s->qeff, 0, (size_t)abs_rows * qe * es));
+    RB_CUDA(cudaMemsetAsync(s->qeff, 0, (size_t)abs_rows * qe * es, c->stream));
     s->abs_rows = abs_rows * qe;
   }
   return REWB200_OK;
@@ -477,12 +481,14 @@ int layered_blocks(rewb200_session* s, const FwdOpts& o, const NormArgs& na, int
   const int64_t dp = m->dp;
   const bool uniform = o.entries == nullptr;
   RowMap map = {nullptr, nullptr, s->d_pos, o.b0, o.S};
-  RowTiles abs = {nullptr, (int)rows, 1, 1};
+  RowTiles abs = {nullptr, (int)rows, 1, 1}, chunks = {nullptr, (int)((rows + kChunkRows - 1) / kChunkRows), 1, 1};
   if (!uniform) {
     map.row_lane = s->plan_dev;
     map.row_pos = s->plan_dev + rows;
     abs.list = reinterpret_cast<const int2*>(s->plan_dev + 2 * rows);
     abs.count = s->plan_abs_tiles;
+    chunks.list = abs.list + abs.count;
+    chunks.count = s->plan_chunks;
   }
   auto ahead_of = [&](size_t r, NormArgs& a) {  // what the norm launch in front of run r adds and writes
     if (r == m->runs.size()) {
@@ -585,6 +591,7 @@ int layered_blocks(rewb200_session* s, const FwdOpts& o, const NormArgs& na, int
     aa.m = A.m;
     aa.map = map;
     aa.tiles = abs;
+    aa.chunks = chunks;
     aa.max_tile_rows = uniform ? 1 : ABS_TILE_ROWS;
     aa.rows = rows;
     RB_TRY(run_linear(s, A.uq, s->cq, A.uq.K, rows, true, 0, s->part, A.uq.N, &ks));

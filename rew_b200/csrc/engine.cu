@@ -162,9 +162,9 @@ int samp_restart(rewb200_session* s) {
     k[2 * b + 1] = (uint32_t)(s->samp_seeds[b] >> 32);
   }
   RB_CUDA(cudaStreamSynchronize(c->stream));
-  RB_CUDA(cudaMemcpy(s->samp_keys, k.data(), k.size() * sizeof(uint32_t), cudaMemcpyHostToDevice));
-  RB_CUDA(cudaMemset(s->samp_steps, 0, s->B * sizeof(int)));
-  RB_CUDA(cudaMemset(s->samp_hist_len, 0, s->B * sizeof(int)));
+  RB_CUDA(cudaMemcpyAsync(s->samp_keys, k.data(), k.size() * sizeof(uint32_t), cudaMemcpyHostToDevice, c->stream));
+  RB_CUDA(cudaMemsetAsync(s->samp_steps, 0, s->B * sizeof(int), c->stream));
+  RB_CUDA(cudaMemsetAsync(s->samp_hist_len, 0, s->B * sizeof(int), c->stream));
   return REWB200_OK;
 }
 
@@ -323,8 +323,8 @@ int ensure_acts(rewb200_session* s, int64_t rows, int64_t logits_rows) {
         if (ep > 1) RB_TRY(acts_alloc(m->c, &s->moe_recv, (size_t)slots * dp * es));
         RB_TRY(acts_alloc(m->c, &s->moe_xs, (size_t)(slots + 128) * dp * es));
         RB_TRY(acts_alloc(m->c, &s->moe_hs, (size_t)(slots + 128) * m->max_moe_ffn * es));
-        RB_CUDA(cudaMemset(s->moe_xs, 0, (size_t)(slots + 128) * dp * es));
-        RB_CUDA(cudaMemset(s->moe_hs, 0, (size_t)(slots + 128) * m->max_moe_ffn * es));
+        RB_CUDA(cudaMemsetAsync(s->moe_xs, 0, (size_t)(slots + 128) * dp * es, m->c->stream));
+        RB_CUDA(cudaMemsetAsync(s->moe_hs, 0, (size_t)(slots + 128) * m->max_moe_ffn * es, m->c->stream));
         RB_TRY(acts_alloc(m->c, (void**)&s->moe_ys, (size_t)slots * dp * sizeof(float)));
         RB_TRY(acts_alloc(m->c, (void**)&s->moe_ret, (size_t)slots * dp * sizeof(float)));
         if (ep > 1) RB_TRY(acts_alloc(m->c, (void**)&s->moe_back, (size_t)slots * dp * sizeof(float)));
@@ -1859,7 +1859,7 @@ int lane_reserve(rewb200_session* s, int lane, int new_len) {
   std::vector<int> row((size_t)s->max_pages, 0);
   for (size_t i = 0; i < pages.size(); ++i) row[i] = pages[i];
   RB_CUDA(cudaStreamSynchronize(c->stream));
-  RB_CUDA(cudaMemcpy(s->block_table + (size_t)lane * s->max_pages, row.data(), row.size() * sizeof(int), cudaMemcpyHostToDevice));
+  RB_CUDA(cudaMemcpyAsync(s->block_table + (size_t)lane * s->max_pages, row.data(), row.size() * sizeof(int), cudaMemcpyHostToDevice, c->stream));
   return REWB200_OK;
 }
 
@@ -1894,17 +1894,17 @@ int rewb200_lane_admit(rewb200_session* s, int lane, const int32_t* ids, int S, 
   RB_TRY(ensure_acts(s, std::max<int64_t>(std::max<int64_t>(S, s->B), s->rows_cap), s->B));
   RB_CUDA(cudaStreamSynchronize(c->stream));
   const int one = 1, zero = 0;
-  RB_CUDA(cudaMemcpy(s->d_ids_prefill, ids, (size_t)S * sizeof(int), cudaMemcpyHostToDevice));
-  RB_CUDA(cudaMemcpy(s->d_pos + lane, &zero, sizeof(int), cudaMemcpyHostToDevice));
-  RB_CUDA(cudaMemcpy(s->d_active + lane, &one, sizeof(int), cudaMemcpyHostToDevice));
+  RB_CUDA(cudaMemcpyAsync(s->d_ids_prefill, ids, (size_t)S * sizeof(int), cudaMemcpyHostToDevice, c->stream));
+  RB_CUDA(cudaMemcpyAsync(s->d_pos + lane, &zero, sizeof(int), cudaMemcpyHostToDevice, c->stream));
+  RB_CUDA(cudaMemcpyAsync(s->d_active + lane, &one, sizeof(int), cudaMemcpyHostToDevice, c->stream));
   if (s->samp_on) {
     // this lane's generate() starts over: Key = initKey(seed), step 0, seen = the prompt
     s->samp_seeds[lane] = seed;
     const uint32_t k[2] = {(uint32_t)(seed & 0xFFFFFFFFull), (uint32_t)(seed >> 32)};
-    RB_CUDA(cudaMemcpy(s->samp_keys + 2 * lane, k, sizeof(k), cudaMemcpyHostToDevice));
-    RB_CUDA(cudaMemcpy(s->samp_steps + lane, &zero, sizeof(int), cudaMemcpyHostToDevice));
-    RB_CUDA(cudaMemcpy(s->samp_hist + (size_t)lane * s->max_len, ids, (size_t)S * sizeof(int), cudaMemcpyHostToDevice));
-    RB_CUDA(cudaMemcpy(s->samp_hist_len + lane, &S, sizeof(int), cudaMemcpyHostToDevice));
+    RB_CUDA(cudaMemcpyAsync(s->samp_keys + 2 * lane, k, sizeof(k), cudaMemcpyHostToDevice, c->stream));
+    RB_CUDA(cudaMemcpyAsync(s->samp_steps + lane, &zero, sizeof(int), cudaMemcpyHostToDevice, c->stream));
+    RB_CUDA(cudaMemcpyAsync(s->samp_hist + (size_t)lane * s->max_len, ids, (size_t)S * sizeof(int), cudaMemcpyHostToDevice, c->stream));
+    RB_CUDA(cudaMemcpyAsync(s->samp_hist_len + lane, &S, sizeof(int), cudaMemcpyHostToDevice, c->stream));
   }
   RB_CUDA(cudaEventRecord(s->ev0, c->stream));
   FwdOpts o;
@@ -2003,7 +2003,7 @@ int rewb200_lanes_feed(rewb200_session* s, int n_entries, const int32_t* lanes, 
     RB_TRY(lane_reserve(s, e.lane, e.pos0 + e.n));
     if (!s->lane_active[e.lane]) {
       const int one = 1;
-      RB_CUDA(cudaMemcpy(s->d_active + e.lane, &one, sizeof(int), cudaMemcpyHostToDevice));
+      RB_CUDA(cudaMemcpyAsync(s->d_active + e.lane, &one, sizeof(int), cudaMemcpyHostToDevice, c->stream));
       s->lane_active[e.lane] = 1;
       s->lane_len[e.lane] = 0;
       if (s->samp_on) {
@@ -2011,16 +2011,16 @@ int rewb200_lanes_feed(rewb200_session* s, int n_entries, const int32_t* lanes, 
         s->samp_seeds[e.lane] = seed;
         const uint32_t k[2] = {(uint32_t)(seed & 0xFFFFFFFFull), (uint32_t)(seed >> 32)};
         const int zero = 0;
-        RB_CUDA(cudaMemcpy(s->samp_keys + 2 * e.lane, k, sizeof(k), cudaMemcpyHostToDevice));
-        RB_CUDA(cudaMemcpy(s->samp_steps + e.lane, &zero, sizeof(int), cudaMemcpyHostToDevice));
+        RB_CUDA(cudaMemcpyAsync(s->samp_keys + 2 * e.lane, k, sizeof(k), cudaMemcpyHostToDevice, c->stream));
+        RB_CUDA(cudaMemcpyAsync(s->samp_steps + e.lane, &zero, sizeof(int), cudaMemcpyHostToDevice, c->stream));
       }
     }
     if (s->samp_on) {  // tokens seen so far = everything fed to the model
       const int n = e.pos0 + e.n;
-      RB_CUDA(cudaMemcpy(s->samp_hist + (size_t)e.lane * s->max_len + e.pos0, ids + e.row0, (size_t)e.n * sizeof(int), cudaMemcpyHostToDevice));
-      RB_CUDA(cudaMemcpy(s->samp_hist_len + e.lane, &n, sizeof(int), cudaMemcpyHostToDevice));
+      RB_CUDA(cudaMemcpyAsync(s->samp_hist + (size_t)e.lane * s->max_len + e.pos0, ids + e.row0, (size_t)e.n * sizeof(int), cudaMemcpyHostToDevice, c->stream));
+      RB_CUDA(cudaMemcpyAsync(s->samp_hist_len + e.lane, &n, sizeof(int), cudaMemcpyHostToDevice, c->stream));
     }
-    RB_CUDA(cudaMemcpy(s->d_pos + e.lane, &e.pos0, sizeof(int), cudaMemcpyHostToDevice));
+    RB_CUDA(cudaMemcpyAsync(s->d_pos + e.lane, &e.pos0, sizeof(int), cudaMemcpyHostToDevice, c->stream));
   }
   // one upload: ids | rows of the lm_head (wanted places, then every lane's last row) | sampled lanes
   std::vector<int> up((size_t)rows + n_want + s->B + s->B, 0);
@@ -2035,7 +2035,7 @@ int rewb200_lanes_feed(rewb200_session* s, int n_entries, const int32_t* lanes, 
     RB_CUDA(cudaMalloc((void**)&s->feed_dev, up.size() * sizeof(int)));
     s->feed_cap = up.size();
   }
-  RB_CUDA(cudaMemcpy(s->feed_dev, up.data(), up.size() * sizeof(int), cudaMemcpyHostToDevice));
+  RB_CUDA(cudaMemcpyAsync(s->feed_dev, up.data(), up.size() * sizeof(int), cudaMemcpyHostToDevice, c->stream));
   const int* d_rows = s->feed_dev + rows;
   const int* d_act = s->feed_dev + rows + n_want + s->B;
   RB_CUDA(cudaEventRecord(s->ev0, c->stream));
@@ -2087,7 +2087,7 @@ int rewb200_lanes_feed(rewb200_session* s, int n_entries, const int32_t* lanes, 
   RB_CUDA(cudaEventElapsedTime(&s->prefill_ms, s->ev0, s->ev1));
   for (const StepEntry& e : entries) {
     s->lane_len[e.lane] = e.pos0 + e.n;
-    RB_CUDA(cudaMemcpy(s->d_pos + e.lane, &s->lane_len[e.lane], sizeof(int), cudaMemcpyHostToDevice));
+    RB_CUDA(cudaMemcpyAsync(s->d_pos + e.lane, &s->lane_len[e.lane], sizeof(int), cudaMemcpyHostToDevice, c->stream));
   }
   if (next_ids)
     for (int e = 0; e < n_entries; ++e) next_ids[e] = act[lanes[e]] ? next[lanes[e]] : -1;
@@ -2101,10 +2101,10 @@ int rewb200_lane_release(rewb200_session* s, int lane) {
   RB_CUDA(cudaSetDevice(c->device));
   RB_CUDA(cudaStreamSynchronize(c->stream));
   const int zero = 0;
-  RB_CUDA(cudaMemcpy(s->d_active + lane, &zero, sizeof(int), cudaMemcpyHostToDevice));
-  RB_CUDA(cudaMemcpy(s->d_pos + lane, &zero, sizeof(int), cudaMemcpyHostToDevice));
+  RB_CUDA(cudaMemcpyAsync(s->d_active + lane, &zero, sizeof(int), cudaMemcpyHostToDevice, c->stream));
+  RB_CUDA(cudaMemcpyAsync(s->d_pos + lane, &zero, sizeof(int), cudaMemcpyHostToDevice, c->stream));
   std::vector<int> row((size_t)s->max_pages, 0);  // back on the scratch block
-  RB_CUDA(cudaMemcpy(s->block_table + (size_t)lane * s->max_pages, row.data(), row.size() * sizeof(int), cudaMemcpyHostToDevice));
+  RB_CUDA(cudaMemcpyAsync(s->block_table + (size_t)lane * s->max_pages, row.data(), row.size() * sizeof(int), cudaMemcpyHostToDevice, c->stream));
   for (int pg : s->lane_pages[lane]) s->free_blocks.push_back(pg);
   s->lane_pages[lane].clear();
   s->lane_active[lane] = 0;

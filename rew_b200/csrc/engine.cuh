@@ -190,7 +190,7 @@ struct rewb200_session {
   int* plan_dev = nullptr;             // row maps, tile lists and gather lists of a step that is no captured decode
   size_t plan_cap = 0;
   std::vector<int> plan_host;
-  int plan_abs_tiles = 0;
+  int plan_abs_tiles = 0, plan_chunks = 0;
   int* feed_dev = nullptr;             // ids and row lists of a rewb200_lanes_feed step
   size_t feed_cap = 0;
   int64_t route_rows = 0;              // rows of the forward recorded last

@@ -2,6 +2,8 @@
 // cached latents.  Scores, softmax, norms, rotations and gates are f32 throughout.
 #include <math.h>
 
+#include <algorithm>
+
 #include "latent.cuh"
 #include "ptx.cuh"
 
@@ -214,6 +216,440 @@ __global__ void __launch_bounds__(128) latent_out_plain_kernel(LatentAttnArgs a)
   }
 }
 
+// ------------------------------------------------------------------ bf16 kernels on the tensor cores
+// Three launches per layer: queries into the latent space, attention over the cache rows, values back out of it.
+
+__device__ __forceinline__ void cp_async16(uint32_t dst, const void* src) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(src) : "memory");
+}
+__device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_all;" ::: "memory"); }
+
+// rows x cols (bf16, row stride lds elements) -> shared memory with row stride ldd elements; columns up to cols_p
+// and rows up to rows_p are zero-filled.  Asynchronous where 16-byte copies are possible.
+__device__ __forceinline__ void stage_matrix(bf16* dst, int ldd, const bf16* src, int64_t lds, int rows, int cols, int rows_p, int cols_p,
+                                             bool vec) {
+  const int cpr = cols_p / 8;
+  for (int i = threadIdx.x; i < rows_p * cpr; i += blockDim.x) {
+    const int r = i / cpr, c = (i % cpr) * 8;
+    bf16* d = dst + (int64_t)r * ldd + c;
+    if (r < rows && c + 8 <= cols && vec) {
+      cp_async16(smem_u32(d), src + r * lds + c);
+    } else {
+#pragma unroll
+      for (int e = 0; e < 8; ++e) d[e] = (r < rows && c + e < cols) ? src[r * lds + c + e] : __float2bfloat16_rn(0.f);
+    }
+  }
+}
+
+__device__ __forceinline__ int2 chunk_rows(const LatentAttnArgs& a, int i) {
+  if (a.chunks.list) return a.chunks.list[i];
+  const int r0 = i * kChunkRows;
+  return make_int2(r0, (int)min((int64_t)kChunkRows, a.rows - r0));
+}
+
+// Two neighbouring query values of a row (col even) from the projection's slabs or its bf16 output.
+__device__ __forceinline__ float2 q_pair(const LatentAttnArgs& a, int64_t row, int64_t col) {
+  if (a.nsplit == 0) {
+    const __nv_bfloat162 v = *reinterpret_cast<const __nv_bfloat162*>(reinterpret_cast<const bf16*>(a.q) + row * a.ldq + col);
+    return make_float2(__low2float(v), __high2float(v));
+  }
+  float2 t = make_float2(0.f, 0.f);
+  const float* p = reinterpret_cast<const float*>(a.q) + row * a.ldq + col;
+  for (int s = 0; s < a.nsplit; ++s) {
+    const float2 v = *reinterpret_cast<const float2*>(p + s * a.split_stride);
+    t.x += v.x;
+    t.y += v.y;
+  }
+  return t;
+}
+
+constexpr int LQ_N = 64;   // latent features per CTA
+
+// grid (latent tiles, heads, chunks): qeff[row][head][n0 .. n0+63] = sum_i q[row][head][i] W_uk[n][i]; the first latent
+// tile also rotates the head's rot_dim part.
+__global__ void __launch_bounds__(128) latent_q_kernel(LatentAttnArgs a) {
+  extern __shared__ __align__(16) uint8_t smem_raw[];
+  const int h = blockIdx.y, dn = a.m.dim, dr = a.m.rot_dim, r = a.m.kv_rank;
+  const int kp = (dn + 15) / 16 * 16, ld = kp + 8;
+  bf16* sA = reinterpret_cast<bf16*>(smem_raw);
+  bf16* sB = sA + kChunkRows * ld;
+  const int n0 = blockIdx.x * LQ_N;
+  pdl_launch_dependents();
+  // the weights do not depend on earlier kernels
+  stage_matrix(sB, ld, reinterpret_cast<const bf16*>(a.ukv) + (int64_t)n0 * a.ld_ukv + (int64_t)h * dn, a.ld_ukv, min(LQ_N, r - n0), dn, LQ_N, kp,
+               dn % 8 == 0);
+  pdl_wait();
+  const int2 ch = chunk_rows(a, blockIdx.z);
+  const int64_t qcol = (int64_t)h * (dn + dr);
+  const bool even = (dn % 2 == 0) && (dr % 2 == 0);
+  const int hp = kp / 2, rows16 = (ch.y + 15) / 16 * 16;
+  for (int i = threadIdx.x; i < rows16 * hp; i += 128) {
+    const int row = i / hp, c = (i % hp) * 2;
+    float2 v = make_float2(0.f, 0.f);
+    if (row < ch.y && c < dn) {
+      if (even) v = q_pair(a, ch.x + row, qcol + c);
+      else {
+        v.x = q_at<bf16>(a, ch.x + row, qcol + c);
+        if (c + 1 < dn) v.y = q_at<bf16>(a, ch.x + row, qcol + c + 1);
+      }
+    }
+    *reinterpret_cast<uint32_t*>(sA + row * ld + c) = pack_bf16(v.x, v.y);
+  }
+  if (blockIdx.x == 0) {
+    const int half = a.m.rope_dims / 2, np = (dr + 1) / 2;
+    for (int i = threadIdx.x; i < ch.y * np; i += 128) {
+      const int64_t row = ch.x + i / np;
+      const int p = i % np;
+      float2 v;
+      if (even) v = q_pair(a, row, qcol + dn + 2 * p);
+      else v = make_float2(q_at<bf16>(a, row, qcol + dn + 2 * p), 2 * p + 1 < dr ? q_at<bf16>(a, row, qcol + dn + 2 * p + 1) : 0.f);
+      v = make_float2(ldf<bf16>(stf<bf16>(v.x)), ldf<bf16>(stf<bf16>(v.y)));   // the projection's bf16 output
+      if (p < half) {
+        const int pos = min(max(row_pos(a.map, row), 0), a.m.max_pos - 1);
+        v = rotate(v, a.m.rope[(int64_t)pos * half + p]);
+      }
+      bf16* qe = reinterpret_cast<bf16*>(a.qeff) + (row * a.m.heads + h) * a.ldc + r + 2 * p;
+      qe[0] = stf<bf16>(v.x);
+      if (2 * p + 1 < dr) qe[1] = stf<bf16>(v.y);
+    }
+  }
+  cp_async_wait();
+  __syncthreads();
+  // warps: wm along the rows (16 each), the others along the 64 latent features
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, l8 = lane & 7, lq = lane >> 3, g = lane >> 2, t = lane & 3;
+  const int wm = ch.y <= 16 ? 1 : ch.y <= 32 ? 2 : 4, wn = 4 / wm, nt_n = 8 / wn;
+  const int mrow = (warp % wm) * 16, ncol = (warp / wm) * nt_n * 8;
+  if (mrow >= rows16) return;
+  float acc[8][4];
+#pragma unroll
+  for (int i = 0; i < 8; ++i)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) acc[i][e] = 0.f;
+  const uint32_t aA = smem_u32(sA), aB = smem_u32(sB);
+  for (int k = 0; k < kp; k += 16) {
+    uint32_t af[4];
+    ldmatrix_x4(af[0], af[1], af[2], af[3], aA + ((mrow + (lq & 1) * 8 + l8) * ld + k + (lq >> 1) * 8) * 2);
+#pragma unroll
+    for (int i = 0; i < 8; i += 2) {
+      if (i >= nt_n) break;
+      uint32_t b0, b1, b2, b3;
+      ldmatrix_x4(b0, b1, b2, b3, aB + ((ncol + i * 8 + (lq >> 1) * 8 + l8) * ld + k + (lq & 1) * 8) * 2);
+      mma_bf16_16816(acc[i], af, b0, b1);
+      mma_bf16_16816(acc[i + 1], af, b2, b3);
+    }
+  }
+#pragma unroll
+  for (int i = 0; i < 8; ++i) {
+    if (i >= nt_n) break;
+#pragma unroll
+    for (int hf = 0; hf < 2; ++hf) {
+      const int row = mrow + g + hf * 8, n = n0 + ncol + i * 8 + 2 * t;
+      if (row >= ch.y || n >= r) continue;
+      bf16* qe = reinterpret_cast<bf16*>(a.qeff) + ((int64_t)(ch.x + row) * a.m.heads + h) * a.ldc + n;
+      if (n + 1 < r && (r & 1) == 0) *reinterpret_cast<uint32_t*>(qe) = pack_bf16(acc[i][2 * hf], acc[i][2 * hf + 1]);
+      else {
+        qe[0] = stf<bf16>(acc[i][2 * hf]);
+        if (n + 1 < r) qe[1] = stf<bf16>(acc[i][2 * hf + 1]);
+      }
+    }
+  }
+}
+
+// Attention of a few (token, head) rows over the cache rows of their lane.  grid (kv splits, tiles * subtiles, head
+// groups), 256 threads.  A CTA's 16 * MT rows are `heads_per` heads of up to `tokens_per` tokens.  Per 64-key page:
+//   S     warp w: keys 16 (w & 3) .. +15, half (w >> 2) of the features; the halves meet in shared memory
+//   P     online softmax in f32, 16 / MT threads per row
+//   O     warp w: value columns 16 (w + 8 i) .. +15, f32 in registers
+// The page's [64][kv_rank + rot_dim] rows are both keys and (their first kv_rank columns) values: one TMA load each.
+struct AbsCfg {
+  int boxes;       // 64-column boxes of a cache row
+  int stages;
+  int heads_per, tokens_per, subtiles;
+};
+constexpr int ABS_OG = 4;       // 16-column value groups per warp: kv_rank up to 512
+
+template <int MT>
+__global__ void __launch_bounds__(256) latent_attn_kernel(const __grid_constant__ CUtensorMap tm, LatentAttnArgs a, AbsCfg cf) {
+  extern __shared__ uint8_t smem_raw[];
+  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
+  constexpr int R = 16 * MT, TPR = 256 / R, KPT = 64 / TPR;   // rows, threads per row, keys per thread
+  const int stage_bytes = cf.boxes * 8192;
+  uint8_t* sKV = smem;
+  uint8_t* sQ = sKV + cf.stages * stage_bytes;                // [box][R rows][128 bytes]
+  uint8_t* sP = sQ + cf.boxes * R * 128;                      // [R rows][128 bytes]
+  float* sS = reinterpret_cast<float*>(sP + R * 128);         // [2][R][68]
+  float* sAl = sS + 2 * R * 68;                               // [R]
+  uint64_t* full = reinterpret_cast<uint64_t*>(sAl + R);
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, l8 = lane & 7, lq = lane >> 3, g = lane >> 2, t = lane & 3;
+  if (tid == 0) {
+    for (int i = 0; i < cf.stages; ++i) mbar_init(&full[i], 1);
+    fence_barrier_init();
+    tma_prefetch_desc(&tm);
+  }
+  pdl_launch_dependents();
+  pdl_wait();
+  const int2 tr = tile_rows(a.tiles, blockIdx.y / cf.subtiles);
+  const int tok0 = (blockIdx.y % cf.subtiles) * cf.tokens_per;
+  const int ntok = min(cf.tokens_per, tr.y - tok0);
+  if (ntok <= 0) return;
+  const int64_t row0 = tr.x + tok0;
+  const int head0 = blockIdx.z * cf.heads_per, nh = min(cf.heads_per, a.m.heads - head0);
+  const int lane_id = row_lane(a.map, row0);
+  const int cap = a.max_pages * PAGE_TOKENS;
+  const int pos_first = min(max(row_pos(a.map, row0), 0), cap - 1), pos_last = min(pos_first + ntok - 1, cap - 1);
+  const int k_lo = a.m.window > 0 ? max(0, pos_first - a.m.window + 1) : 0;
+  const int t_lo = k_lo / PAGE_TOKENS, nt_all = pos_last / PAGE_TOKENS - t_lo + 1;
+  const int per = (nt_all + gridDim.x - 1) / gridDim.x;
+  const int t0 = t_lo + blockIdx.x * per, nt = max(0, min(per, t_lo + nt_all - t0));
+  // queries
+  for (int i = tid; i < R * cf.boxes * 8; i += 256) {
+    const int m = i / (cf.boxes * 8), c = i % (cf.boxes * 8);
+    const int tok = m / cf.heads_per, hh = m % cf.heads_per;
+    uint4 v = make_uint4(0, 0, 0, 0);
+    if (tok < ntok && hh < nh && c * 8 < a.ldc)
+      v = *reinterpret_cast<const uint4*>(reinterpret_cast<const bf16*>(a.qeff) + ((row0 + tok) * a.m.heads + head0 + hh) * a.ldc + c * 8);
+    *reinterpret_cast<uint4*>(sQ + (c >> 3) * (R * 128) + swz128((uint32_t)m, (uint32_t)(c & 7))) = v;
+  }
+  __syncthreads();
+  auto load_page = [&](int i) {
+    const int st = i % cf.stages;
+    const int page = a.block_table[(int64_t)lane_id * a.max_pages + t0 + i];
+    mbar_expect_tx(&full[st], stage_bytes);
+    for (int b = 0; b < cf.boxes; ++b) tma_load_2d(sKV + st * stage_bytes + b * 8192, &tm, &full[st], b * 64, page * PAGE_TOKENS);
+  };
+  if (tid == 0)
+    for (int i = 0; i < min(cf.stages, nt); ++i) load_page(i);
+
+  // softmax ownership: thread -> (row, KPT keys)
+  const int srow = tid / TPR, skey = (tid % TPR) * KPT;
+  const int stok = srow / cf.heads_per;
+  const bool sval = stok < ntok && srow % cf.heads_per < nh;
+  const int spos = pos_first + stok, slo = a.m.window > 0 ? spos - a.m.window : -1;   // sees keys slo < key <= spos
+  float m_run = -INFINITY, l_run = 0.f;
+  float acc[MT][ABS_OG][2][4];
+#pragma unroll
+  for (int i = 0; i < MT; ++i)
+#pragma unroll
+    for (int j = 0; j < ABS_OG; ++j)
+#pragma unroll
+      for (int e = 0; e < 8; ++e) acc[i][j][e >> 2][e & 3] = 0.f;
+  const int groups = (a.m.kv_rank + 15) / 16;
+  const uint32_t q_base = smem_u32(sQ), p_base = smem_u32(sP);
+  const int kg = warp & 3, kh = warp >> 2;
+  const int ks0 = kh * cf.boxes * 2, ks1 = ks0 + cf.boxes * 2;   // 16-feature steps of this warp's half
+  bool ok = true;
+  for (int it = 0; it < nt; ++it) {
+    const int st = it % cf.stages;
+    ok = mbar_wait(&full[st], (it / cf.stages) & 1, a.status);
+    const uint32_t kv = smem_u32(sKV) + st * stage_bytes;
+    float sc[MT][2][4];
+#pragma unroll
+    for (int i = 0; i < MT; ++i)
+#pragma unroll
+      for (int e = 0; e < 8; ++e) sc[i][e >> 2][e & 3] = 0.f;
+    for (int k = ks0; k < ks1; ++k) {
+      const uint32_t box = k >> 2, ch = (k & 3) * 2;
+      uint32_t b0, b1, b2, b3;
+      ldmatrix_x4(b0, b1, b2, b3, kv + box * 8192 + swz128(kg * 16 + (lq >> 1) * 8 + l8, ch + (lq & 1)));
+#pragma unroll
+      for (int i = 0; i < MT; ++i) {
+        uint32_t af[4];
+        ldmatrix_x4(af[0], af[1], af[2], af[3], q_base + box * (R * 128) + swz128(i * 16 + (lq & 1) * 8 + l8, ch + (lq >> 1)));
+        mma_bf16_16816(sc[i][0], af, b0, b1);
+        mma_bf16_16816(sc[i][1], af, b2, b3);
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < MT; ++i)
+#pragma unroll
+      for (int n = 0; n < 2; ++n)
+#pragma unroll
+        for (int hf = 0; hf < 2; ++hf)
+          *reinterpret_cast<float2*>(sS + (kh * R + i * 16 + g + hf * 8) * 68 + kg * 16 + n * 8 + 2 * t) = make_float2(sc[i][n][2 * hf], sc[i][n][2 * hf + 1]);
+    __syncthreads();
+    {
+      const int key0 = (t0 + it) * PAGE_TOKENS + skey;
+      float x[KPT], mx = -INFINITY;
+#pragma unroll
+      for (int e = 0; e < KPT; ++e) {
+        const float v = (sS[srow * 68 + skey + e] + sS[(R + srow) * 68 + skey + e]) * a.m.scale;
+        x[e] = (sval && key0 + e <= spos && key0 + e > slo) ? v : -INFINITY;
+        mx = fmaxf(mx, x[e]);
+      }
+#pragma unroll
+      for (int o = TPR / 2; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
+      const float m_new = fmaxf(m_run, mx), m_use = m_new == -INFINITY ? 0.f : m_new;
+      const float alpha = __expf(m_run - m_use);
+      float ps = 0.f;
+      uint32_t pk[KPT / 2];
+#pragma unroll
+      for (int e = 0; e < KPT; e += 2) {
+        const float p0 = __expf(x[e] - m_use), p1 = __expf(x[e + 1] - m_use);
+        ps += p0 + p1;
+        pk[e / 2] = pack_bf16(p0, p1);
+      }
+#pragma unroll
+      for (int o = TPR / 2; o > 0; o >>= 1) ps += __shfl_xor_sync(0xffffffffu, ps, o);
+      l_run = l_run * alpha + ps;
+      m_run = m_new;
+      uint8_t* pd = sP + swz128((uint32_t)srow, (uint32_t)(skey >> 3)) + (skey & 7) * 2;
+#pragma unroll
+      for (int e = 0; e < KPT / 2; ++e) *reinterpret_cast<uint32_t*>(pd + e * 4) = pk[e];
+      if (tid % TPR == 0) sAl[srow] = alpha;
+    }
+    __syncthreads();
+#pragma unroll
+    for (int i = 0; i < MT; ++i) {
+      const float a0 = sAl[i * 16 + g], a1 = sAl[i * 16 + g + 8];
+#pragma unroll
+      for (int j = 0; j < ABS_OG; ++j)
+#pragma unroll
+        for (int n = 0; n < 2; ++n) {
+          acc[i][j][n][0] *= a0;
+          acc[i][j][n][1] *= a0;
+          acc[i][j][n][2] *= a1;
+          acc[i][j][n][3] *= a1;
+        }
+    }
+#pragma unroll
+    for (int k = 0; k < 4; ++k) {   // 16 keys a step
+      uint32_t pf[MT][4];
+#pragma unroll
+      for (int i = 0; i < MT; ++i)
+        ldmatrix_x4(pf[i][0], pf[i][1], pf[i][2], pf[i][3], p_base + swz128(i * 16 + (lq & 1) * 8 + l8, k * 2 + (lq >> 1)));
+#pragma unroll
+      for (int j = 0; j < ABS_OG; ++j) {
+        const int grp = warp + 8 * j;
+        if (grp >= groups) break;
+        uint32_t v0, v1, v2, v3;
+        ldmatrix_x4_trans(v0, v1, v2, v3, kv + (grp >> 2) * 8192 + swz128(k * 16 + (lq & 1) * 8 + l8, (grp & 3) * 2 + (lq >> 1)));
+#pragma unroll
+        for (int i = 0; i < MT; ++i) {
+          mma_bf16_16816(acc[i][j][0], pf[i], v0, v1);
+          mma_bf16_16816(acc[i][j][1], pf[i], v2, v3);
+        }
+      }
+    }
+    ok = __syncthreads_and(ok);   // everyone is done with the stage, the scores and the probabilities
+    if (!ok) break;
+    if (tid == 0 && it + cf.stages < nt) load_page(it + cf.stages);
+  }
+  if (!ok) return;
+#pragma unroll
+  for (int i = 0; i < MT; ++i)
+#pragma unroll
+    for (int hf = 0; hf < 2; ++hf) {
+      const int m = i * 16 + g + hf * 8, tok = m / cf.heads_per, hh = m % cf.heads_per;
+      if (tok >= ntok || hh >= nh) continue;
+      const int64_t u = ((row0 + tok) * a.m.heads + head0 + hh) * a.kv_splits + blockIdx.x;
+      float* o = a.olat + u * a.m.kv_rank;
+#pragma unroll
+      for (int j = 0; j < ABS_OG; ++j)
+#pragma unroll
+        for (int n = 0; n < 2; ++n) {
+          const int col = (warp + 8 * j) * 16 + n * 8 + 2 * t;
+          if (col + 1 < a.m.kv_rank && (a.m.kv_rank & 1) == 0)
+            *reinterpret_cast<float2*>(o + col) = make_float2(acc[i][j][n][2 * hf], acc[i][j][n][2 * hf + 1]);
+          else {
+            if (col < a.m.kv_rank) o[col] = acc[i][j][n][2 * hf];
+            if (col + 1 < a.m.kv_rank) o[col + 1] = acc[i][j][n][2 * hf + 1];
+          }
+        }
+    }
+  if (tid % TPR == 0 && sval)
+    a.ml[((row0 + stok) * a.m.heads + head0 + srow % cf.heads_per) * a.kv_splits + blockIdx.x] = make_float2(m_run, l_run);
+}
+
+constexpr int LO_ROWS = 32, LO_N = 32;
+
+// grid (value tiles, heads, chunks * 2): merges the kv splits, out[row][head][n0 .. n0+31] = gate * sum_k o[k] W_uv[k][n]
+__global__ void __launch_bounds__(128) latent_out_kernel(LatentAttnArgs a) {
+  extern __shared__ __align__(16) uint8_t smem_raw[];
+  const int h = blockIdx.y, r = a.m.kv_rank, dv = a.m.vdim;
+  const int kp = (r + 15) / 16 * 16, ld = kp + 8;
+  bf16* sA = reinterpret_cast<bf16*>(smem_raw);
+  bf16* sB = sA + LO_ROWS * ld;                 // [kp][LO_N + 8]
+  constexpr int ldb = LO_N + 8;
+  __shared__ float sw[LO_ROWS][17];
+  const int n0 = blockIdx.x * LO_N;
+  pdl_launch_dependents();
+  const int64_t c0 = (int64_t)a.m.heads * a.m.dim + (int64_t)h * dv + n0;
+  stage_matrix(sB, ldb, reinterpret_cast<const bf16*>(a.ukv) + c0, a.ld_ukv, r, min(LO_N, dv - n0), kp, LO_N, c0 % 8 == 0);
+  pdl_wait();
+  int2 ch = chunk_rows(a, (int)(blockIdx.z >> 1));
+  const int skip = (int)(blockIdx.z & 1) * LO_ROWS;
+  ch.x += skip;
+  ch.y = min(LO_ROWS, ch.y - skip);
+  if (ch.y <= 0) {
+    cp_async_wait();
+    return;
+  }
+  const int ns = a.kv_splits;
+  // weights of the splits: exp(m_s - M) / sum
+  if (threadIdx.x < LO_ROWS) {
+    const int row = threadIdx.x;
+    if (row < ch.y) {
+      const float2* ml = a.ml + ((int64_t)(ch.x + row) * a.m.heads + h) * ns;
+      float M = -INFINITY, L = 0.f;
+      for (int s = 0; s < ns; ++s) M = fmaxf(M, ml[s].x);
+      for (int s = 0; s < ns; ++s) {
+        const float f = ml[s].x == -INFINITY ? 0.f : __expf(ml[s].x - M);
+        sw[row][s] = f;
+        L += ml[s].y * f;
+      }
+      for (int s = 0; s < ns; ++s) sw[row][s] /= L;
+    }
+  }
+  __syncthreads();
+  const int hp = kp / 2, rows16 = (ch.y + 15) / 16 * 16;
+  for (int i = threadIdx.x; i < rows16 * hp; i += 128) {
+    const int row = i / hp, c = (i % hp) * 2;
+    float2 v = make_float2(0.f, 0.f);
+    if (row < ch.y && c < r) {
+      const float* o = a.olat + ((int64_t)(ch.x + row) * a.m.heads + h) * ns * r + c;
+      const bool pair = (r & 1) == 0;
+      for (int s = 0; s < ns; ++s) {
+        const float w = sw[row][s];
+        if (w == 0.f) continue;   // a split without keys of this row has written nothing that counts
+        if (pair) {
+          const float2 x = *reinterpret_cast<const float2*>(o + (int64_t)s * r);
+          v.x += w * x.x;
+          v.y += w * x.y;
+        } else {
+          v.x += w * o[(int64_t)s * r];
+          if (c + 1 < r) v.y += w * o[(int64_t)s * r + 1];
+        }
+      }
+    }
+    *reinterpret_cast<uint32_t*>(sA + row * ld + c) = pack_bf16(v.x, v.y);
+  }
+  cp_async_wait();
+  __syncthreads();
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, l8 = lane & 7, lq = lane >> 3, g = lane >> 2, t = lane & 3;
+  const int mrow = (warp & 1) * 16, ncol = (warp >> 1) * 16;
+  if (mrow >= rows16) return;
+  float acc[2][4] = {};
+  const uint32_t aA = smem_u32(sA), aB = smem_u32(sB);
+  for (int k = 0; k < kp; k += 16) {
+    uint32_t af[4], b0, b1, b2, b3;
+    ldmatrix_x4(af[0], af[1], af[2], af[3], aA + ((mrow + (lq & 1) * 8 + l8) * ld + k + (lq >> 1) * 8) * 2);
+    ldmatrix_x4_trans(b0, b1, b2, b3, aB + ((k + (lq & 1) * 8 + l8) * ldb + ncol + (lq >> 1) * 8) * 2);
+    mma_bf16_16816(acc[0], af, b0, b1);
+    mma_bf16_16816(acc[1], af, b2, b3);
+  }
+#pragma unroll
+  for (int i = 0; i < 2; ++i)
+#pragma unroll
+    for (int hf = 0; hf < 2; ++hf) {
+      const int row = mrow + g + hf * 8, n = n0 + ncol + i * 8 + 2 * t;
+      if (row >= ch.y || n >= dv) continue;
+      const float gt = a.m.gate ? a.gate[(int64_t)(ch.x + row) * a.m.heads + h] : 1.0f;
+      bf16* op = reinterpret_cast<bf16*>(a.out) + (int64_t)(ch.x + row) * a.ldo + (int64_t)h * dv + n;
+      op[0] = stf<bf16>(acc[i][2 * hf] * gt);
+      if (n + 1 < dv) op[1] = stf<bf16>(acc[i][2 * hf + 1] * gt);
+    }
+}
+
 template <typename T>
 __global__ void __launch_bounds__(128) gather_rows_kernel(const T* src, const int* index, T* dst, int64_t width) {
   pdl_launch_dependents();
@@ -249,14 +685,69 @@ int latent_post_launch(Ctx* c, const LatentPostArgs& a, int64_t rows) {
   return REWB200_OK;
 }
 
+namespace {
+
+constexpr size_t kSmemMax = 227 * 1024;
+
+// Sizes the tensor-core kernels take; everything else runs on the plain ones.
+bool abs_config(const LatentDims& m, int64_t ldc, int mt, AbsCfg* cf, size_t* smem) {
+  cf->boxes = (int)((m.kv_rank + m.rot_dim + 63) / 64);
+  const int R = 16 * mt;
+  const size_t fixed = (size_t)cf->boxes * R * 128 + R * 128 + 2 * R * 68 * 4 + R * 4 + 64 + 1024;
+  cf->stages = 4;
+  while (cf->stages > 1 && fixed + (size_t)cf->stages * cf->boxes * 8192 > kSmemMax) --cf->stages;
+  *smem = fixed + (size_t)cf->stages * cf->boxes * 8192;
+  const size_t q_smem = (size_t)2 * 64 * ((m.dim + 15) / 16 * 16 + 8) * 2;
+  const int kp = (m.kv_rank + 15) / 16 * 16;
+  const size_t o_smem = (size_t)LO_ROWS * (kp + 8) * 2 + (size_t)kp * (LO_N + 8) * 2;
+  (void)ldc;
+  return m.kv_rank <= 16 * 8 * ABS_OG && *smem <= kSmemMax && cf->stages >= 2 && q_smem <= kSmemMax && o_smem <= kSmemMax - 4096;
+}
+
+}  // namespace
+
 int latent_kv_splits(Ctx* c, const LatentDims& m, int64_t tiles, int64_t max_ctx) {
-  (void)c; (void)m; (void)tiles; (void)max_ctx;
-  return 1;
+  const int64_t ctx = m.window > 0 ? std::min<int64_t>(m.window, max_ctx) : max_ctx;
+  const int64_t pages = (ctx + PAGE_TOKENS - 1) / PAGE_TOKENS + 1;
+  const int64_t hg = (m.heads + 31) / 32;
+  const int64_t want = c->sm_count / std::max<int64_t>(1, tiles * hg);
+  return (int)std::max<int64_t>(1, std::min<int64_t>(std::min<int64_t>(want, pages / 2), 16));
 }
 
 int latent_attn_absorbed_launch(Ctx* c, const LatentAttnArgs& a) {
   if (a.tiles.count == 0) return REWB200_OK;
-  return a.dtype == REWB200_BF16 ? plain_launch<bf16>(c, a) : plain_launch<float>(c, a);
+  AbsCfg cf;
+  size_t smem = 0;
+  const int mt = a.m.heads <= 16 && a.max_tile_rows == 1 ? 1 : 2;
+  if (a.dtype != REWB200_BF16 || c->latent_impl == 1 || !abs_config(a.m, a.ldc, mt, &cf, &smem)) {
+    // the plain kernels do not split the keys: one partial per (row, head)
+    LatentAttnArgs p = a;
+    p.kv_splits = 1;
+    return a.dtype == REWB200_BF16 ? plain_launch<bf16>(c, p) : plain_launch<float>(c, p);
+  }
+  cf.heads_per = std::min(a.m.heads, 16 * mt);
+  cf.tokens_per = std::min(16 * mt / cf.heads_per, a.max_tile_rows);
+  cf.subtiles = (a.max_tile_rows + cf.tokens_per - 1) / cf.tokens_per;
+  const int kp = (a.m.dim + 15) / 16 * 16, rp = (a.m.kv_rank + 15) / 16 * 16;
+  const size_t q_smem = (size_t)(kChunkRows + LQ_N) * (kp + 8) * 2;
+  const size_t o_smem = (size_t)LO_ROWS * (rp + 8) * 2 + (size_t)rp * (LO_N + 8) * 2;
+  static bool attr_set = false;
+  if (!attr_set) {
+    RB_CUDA(cudaFuncSetAttribute(latent_q_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kSmemMax));
+    RB_CUDA(cudaFuncSetAttribute(latent_attn_kernel<1>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kSmemMax));
+    RB_CUDA(cudaFuncSetAttribute(latent_attn_kernel<2>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kSmemMax));
+    RB_CUDA(cudaFuncSetAttribute(latent_out_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kSmemMax - 4096));
+    attr_set = true;
+  }
+  const dim3 gq((unsigned)((a.m.kv_rank + LQ_N - 1) / LQ_N), (unsigned)a.m.heads, (unsigned)a.chunks.count);
+  RB_CUDA(launch_k(latent_q_kernel, gq, dim3(128), q_smem, c->stream, c->use_pdl, a));
+  const dim3 ga((unsigned)a.kv_splits, (unsigned)(a.tiles.count * cf.subtiles), (unsigned)((a.m.heads + cf.heads_per - 1) / cf.heads_per));
+  if (mt == 1) RB_CUDA(launch_k(latent_attn_kernel<1>, ga, dim3(256), smem, c->stream, c->use_pdl, *a.tm_cache, a, cf));
+  else RB_CUDA(launch_k(latent_attn_kernel<2>, ga, dim3(256), smem, c->stream, c->use_pdl, *a.tm_cache, a, cf));
+  const dim3 go((unsigned)((a.m.vdim + LO_N - 1) / LO_N), (unsigned)a.m.heads, (unsigned)(a.chunks.count * 2));
+  RB_CUDA(launch_k(latent_out_kernel, go, dim3(128), o_smem, c->stream, c->use_pdl, a));
+  g_launch_total += 3;
+  return REWB200_OK;
 }
 
 int gather_rows_launch(Ctx* c, const void* src, const int* index, void* dst, int64_t n, int64_t width, int dtype) {

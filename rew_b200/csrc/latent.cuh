@@ -28,6 +28,8 @@ struct RowTiles {
   int per_tile;   // rows per tile at most
 };
 
+constexpr int kChunkRows = 64;   // RowTiles of LatentAttnArgs::chunks
+
 struct LatentDims {
   int heads, dim, rot_dim, vdim, q_rank, kv_rank;
   int rope_dims;           // rotated features of the rot_dim part (interleaved pairs), the rest passes unchanged
@@ -65,8 +67,9 @@ int latent_post_launch(Ctx* c, const LatentPostArgs& a, int64_t rows);
 struct LatentAttnArgs {
   LatentDims m;
   RowMap map;
-  RowTiles tiles;
+  RowTiles tiles;          // runs of rows of one lane
   int max_tile_rows;       // rows of the longest tile
+  RowTiles chunks;         // the same rows in runs of up to kChunkRows, whatever their lanes
   int64_t rows;            // rows of the whole step
   // queries: either split-K slabs f32 [nsplit][rows][ldq] or (nsplit == 0) act dtype [rows][ldq]
   const void* q;
