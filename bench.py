@@ -19,6 +19,8 @@ N(0, 0.02) generated on the device, uniform random prompt ids):
 With --gpus N > 1 the l8 workloads run N independent replicas (sequences are independent units; no
 data-path collective): weak scaling.
     tiny     the tiny fp32 Llama of the parity tests
+    rezupel_b32, rezupel_b1, rezupel_b8_s2048, rezupel_moe_b64
+             Rezupel (latent attention) at the sizes of l8_b32, l8_b1, l8_b8_s2048 and moe_b64
 
 `value` is decode tokens/s of the whole job with ids, weights and cache resident
 in HBM (CUDA events around K graph replays); `e2e` is tokens/s of one generate()
@@ -62,6 +64,13 @@ WORKLOADS = {
     # 4 / 8, no exchange): what the sharded kernels cost without the all-reduce, measurable on one GPU
     "l70_tp4shape": dict(model="llama3_70b", batch=16, prompt=1024, shape_div=4),
     "l70_tp8shape": dict(model="llama3_70b", batch=16, prompt=1024, shape_div=8),
+    # layered models (latent attention, parallel blocks) beside l8_b32 and moe_b64 at equal size: same width, heads,
+    # feed-forward or experts, as many layer runs
+    "rezupel_b32": dict(model="rezupel.dense_8b", batch=32, prompt=512),
+    "rezupel_b1": dict(model="rezupel.dense_8b", batch=1, prompt=512),
+    "rezupel_b8_s2048": dict(model="rezupel.dense_8b", batch=8, prompt=2048),
+    "rezupel_moe_b64": dict(model="rezupel.moe_lite", batch=64, prompt=256),
+    "l8_b8_s2048": dict(model="llama3_8b", batch=8, prompt=2048),
     # the attention operator alone: batch 8, 32 query / 8 kv heads, head_dim 128, 4096 positions
     "attn_op": dict(model=None, batch=8, prompt=4096),
 }
@@ -169,8 +178,8 @@ def dist_env():
 
 
 def make_cfg(name):
-    from rew_b200 import weights as W
-    return getattr(W, name)()
+    from rew_b200 import rezupel, weights as W
+    return getattr(rezupel, name.split(".")[1])() if name.startswith("rezupel.") else getattr(W, name)()
 
 
 def product_config(args, wl, world, model_gb=None):
@@ -180,8 +189,8 @@ def product_config(args, wl, world, model_gb=None):
     cfg = make_cfg(wl["model"])
     return {"workload": args.workload + ("" if args.layers <= 0 else "_%dlayers" % args.layers), "batch_per_gpu": per_gpu,
             "prompt": wl["prompt"], "decode_steps": args.steps, "parallelism": parallel + (str(world) if world > 1 else ""),
-            "sampling": args.sampling, "mask": "conventional" if cfg.mask_kind == 1 else "as_written",
-            "norm": "rmsNorm" if cfg.norm_kind == 0 else "LayerNorm",
+            "sampling": args.sampling, "mask": "windows" if hasattr(cfg, "layer_runs") else "conventional" if cfg.mask_kind == 1 else "as_written",
+            "norm": "rmsNorm" if getattr(cfg, "norm_kind", 0) == 0 else "LayerNorm",
             "l2": "weights streamed per step exceed the 126 MB L2"}
 
 
@@ -341,7 +350,10 @@ def run_model(args, name, rank, local_rank, world, pg, K, Wm, with_e2e, with_pro
         dv = wl["shape_div"]
         cfg.n_heads, cfg.n_kv_heads, cfg.ffn = cfg.n_heads // dv, cfg.n_kv_heads // dv, cfg.ffn // dv
         cfg.vocab = cfg.vocab // dv // 8 * 8
-    if args.layers > 0:
+    layered = hasattr(cfg, "layer_runs")
+    if args.layers > 0 and layered:
+        cfg.layers, cfg.loop = cfg.layers[:args.layers], None
+    elif args.layers > 0:
         cfg.n_layers = args.layers
     B, S = wl["batch"], wl["prompt"]
     max_len = S + Wm + K + 16 + SETTLE_MAX_STEPS
@@ -450,12 +462,16 @@ def run_model(args, name, rank, local_rank, world, pg, K, Wm, with_e2e, with_pro
 
     # ---- rooflines: whole step (weights + KV read once per step per GPU), and the Linear launches alone
     peak, which = measured_peaks()
-    kv_bytes = 2 * cfg.n_layers * (cfg.n_kv_heads // cfg.tp_size) * cfg.head_dim * 2 * B * (S + Wm + settle + K / 2.0)
-    step_bytes = model.weight_bytes() - cfg.vocab * cfg.d_model * 2 + kv_bytes   # the embedding table is not streamed
+    ctx = S + Wm + settle + K / 2.0
+    if layered:
+        step_bytes = cfg.step_bytes(B, ctx)
+    else:
+        kv_bytes = 2 * cfg.n_layers * (cfg.n_kv_heads // cfg.tp_size) * cfg.head_dim * 2 * B * ctx
+        step_bytes = model.weight_bytes() - cfg.vocab * cfg.d_model * 2 + kv_bytes   # the embedding table is not streamed
     out["step_bytes_per_gpu"] = step_bytes
     out["step_frac"] = step_bytes / (decode_ms / K * 1e-3) / 1e9 / peak
     out["peak"], out["peak_source"] = peak, which
-    if with_profile and cfg.n_routed == 0 and cfg.dtype == _lib.BF16:
+    if with_profile and cfg.n_routed == 0 and cfg.dtype == _lib.BF16 and not layered:
         ms, nbytes, nl = C.c_float(), C.c_int64(), C.c_int32()
         _lib.check(L.rewb200_session_profile_linears(sess._h, 20, C.byref(ms), C.byref(nbytes), C.byref(nl)))
         out["linear"] = {"ms_per_step": ms.value, "bytes_per_step": nbytes.value, "launches_per_step": nl.value,
@@ -561,6 +577,10 @@ def main():
     if args.workload == "attn_op":
         run_attention_op(args, rank, local_rank)
         return
+    if args.impl == "reference" and wl["model"].startswith("rezupel."):
+        if rank == 0:
+            print(json.dumps({"impl": "reference", "unavailable": "the reference has no latent-attention model"}), flush=True)
+        return
     if args.impl == "reference":
         run_reference(args, wl, rank, world)
         return
@@ -660,7 +680,7 @@ def main():
     if "trace_ms" in r:
         line["trace_ms"] = r["trace_ms"]
     line.update(extra)
-    if world == 1 and not args.no_cpu_baseline:
+    if world == 1 and not args.no_cpu_baseline and not hasattr(cfg, "layer_runs"):
         line["cpu_baseline"] = cpu_baseline_leg(args, wl)
     print(json.dumps(line), flush=True)
 

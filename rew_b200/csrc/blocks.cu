@@ -474,7 +474,7 @@ int layered_prepare(rewb200_session* s, const FwdOpts& o, int64_t rows) {
 
 // The layer runs of a layered model over `rows` rows; na carries the residual, the embedding and the ids.  Leaves the
 // final norm's output in s->xn.
-int layered_blocks(rewb200_session* s, const FwdOpts& o, const NormArgs& na, int64_t rows) {
+int layered_blocks(rewb200_session* s, const FwdOpts& o, const NormArgs& na, int64_t rows, bool in_graph) {
   rewb200_model* m = s->m;
   Ctx* c = m->c;
   const int dt = m->cfg.dtype;
@@ -614,6 +614,7 @@ int layered_blocks(rewb200_session* s, const FwdOpts& o, const NormArgs& na, int
     aa.max_pages = s->max_pages;
     aa.ldc = A.ldc;
     aa.dtype = dt;
+    aa.early_kv = in_graph ? 1 : 0;
     aa.status = c->d_status;
     if (o.trace) RB_TRY(o.trace->mark(TC_QKV_POST));
     RB_TRY(latent_attn_absorbed_launch(c, aa));

@@ -956,7 +956,7 @@ int enqueue_forward(rewb200_session* s, const FwdOpts& o) {
     na.embed = m->embed;
     na.ids = o.ids_src ? o.ids_src : s->d_ids;
     if (d != cf.d_model) na.d_mean = cf.d_model;
-    RB_TRY(layered_blocks(s, o, na, rows));
+    RB_TRY(layered_blocks(s, o, na, rows, in_graph));
   } else {
     RB_TRY(gqa_blocks(s, o, na, rows, in_graph));
   }

@@ -313,6 +313,6 @@ int layered_acts(rewb200_session* s, int64_t rows);
 int layered_session(rewb200_session* s, int64_t n_pages);
 // Host-side preparation of a step: plan upload and scratch growth (never inside a capture).
 int layered_prepare(rewb200_session* s, const FwdOpts& o, int64_t rows);
-int layered_blocks(rewb200_session* s, const FwdOpts& o, const NormArgs& na, int64_t rows);
+int layered_blocks(rewb200_session* s, const FwdOpts& o, const NormArgs& na, int64_t rows, bool in_graph);
 
 }  // namespace rewb

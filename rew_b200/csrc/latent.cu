@@ -38,6 +38,8 @@ __device__ __forceinline__ float2 rotate(float2 v, float2 cs) {
   return make_float2(v.x * cs.x - v.y * cs.y, v.y * cs.x + v.x * cs.y);
 }
 
+__device__ __forceinline__ void add4(float4& v, const float4 w) { v.x += w.x; v.y += w.y; v.z += w.z; v.w += w.w; }
+
 __device__ __forceinline__ float block_sum256(float v, float* red) {
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
@@ -54,7 +56,7 @@ __device__ __forceinline__ float block_sum256(float v, float* red) {
 // One CTA per row.
 template <typename T>
 __global__ void __launch_bounds__(256) latent_post_kernel(LatentPostArgs a) {
-  extern __shared__ float sx[];
+  extern __shared__ __align__(16) float sx[];
   __shared__ float red[8];
   pdl_launch_dependents();
   pdl_wait();
@@ -62,12 +64,24 @@ __global__ void __launch_bounds__(256) latent_post_kernel(LatentPostArgs a) {
   const int nq = a.m.q_rank, nc = a.m.kv_rank, nr = a.m.rot_dim, n = nq + nc + nr + (a.m.gate ? a.m.heads : 0);
   const float* p = a.partial + row * a.ld;
   float sq = 0.f, sc = 0.f;
-  for (int i = threadIdx.x; i < n; i += 256) {
-    float v = 0.f;
-    for (int s = 0; s < a.nsplit; ++s) v += p[s * a.split_stride + i];
-    sx[i] = v;
-    if (i < nq) sq += v * v;
-    else if (i < nq + nc) sc += v * v;
+  for (int i = threadIdx.x * 4; i < n; i += 1024) {   // rows are padded to a multiple of 8 columns
+    float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+    int k = 0;
+    for (; k + 4 <= a.nsplit; k += 4) {
+      float4 w[4];
+#pragma unroll
+      for (int u = 0; u < 4; ++u) w[u] = *reinterpret_cast<const float4*>(p + (k + u) * a.split_stride + i);
+#pragma unroll
+      for (int u = 0; u < 4; ++u) add4(v, w[u]);
+    }
+    for (; k < a.nsplit; ++k) add4(v, *reinterpret_cast<const float4*>(p + k * a.split_stride + i));
+    *reinterpret_cast<float4*>(sx + i) = v;
+    const float e[4] = {v.x, v.y, v.z, v.w};
+#pragma unroll
+    for (int u = 0; u < 4; ++u) {
+      if (i + u < nq) sq += e[u] * e[u];
+      else if (i + u < nq + nc) sc += e[u] * e[u];
+    }
   }
   sq = block_sum256(sq, red);
   sc = block_sum256(sc, red);
@@ -265,9 +279,9 @@ __device__ __forceinline__ float2 q_pair(const LatentAttnArgs& a, int64_t row, i
 
 constexpr int LQ_N = 64;   // latent features per CTA
 
-// grid (latent tiles, heads, chunks): qeff[row][head][n0 .. n0+63] = sum_i q[row][head][i] W_uk[n][i]; the first latent
-// tile also rotates the head's rot_dim part.
-__global__ void __launch_bounds__(128) latent_q_kernel(LatentAttnArgs a) {
+// grid (latent tiles, heads, chunks): qeff[row][head][n0 .. n0+63] = sum_i q[row][head][i] W_uk[n][i]; the
+// head's rot_dim part is rotated on the way.
+__global__ void __launch_bounds__(256) latent_q_kernel(LatentAttnArgs a) {
   extern __shared__ __align__(16) uint8_t smem_raw[];
   const int h = blockIdx.y, dn = a.m.dim, dr = a.m.rot_dim, r = a.m.kv_rank;
   const int kp = (dn + 15) / 16 * 16, ld = kp + 8;
@@ -282,22 +296,47 @@ __global__ void __launch_bounds__(128) latent_q_kernel(LatentAttnArgs a) {
   const int2 ch = chunk_rows(a, blockIdx.z);
   const int64_t qcol = (int64_t)h * (dn + dr);
   const bool even = (dn % 2 == 0) && (dr % 2 == 0);
-  const int hp = kp / 2, rows16 = (ch.y + 15) / 16 * 16;
-  for (int i = threadIdx.x; i < rows16 * hp; i += 128) {
-    const int row = i / hp, c = (i % hp) * 2;
-    float2 v = make_float2(0.f, 0.f);
-    if (row < ch.y && c < dn) {
-      if (even) v = q_pair(a, ch.x + row, qcol + c);
-      else {
-        v.x = q_at<bf16>(a, ch.x + row, qcol + c);
-        if (c + 1 < dn) v.y = q_at<bf16>(a, ch.x + row, qcol + c + 1);
+  const int rows16 = (ch.y + 15) / 16 * 16;
+  if (a.nsplit > 0 && dn % 4 == 0 && qcol % 4 == 0) {
+    // four columns a thread, four independent chains of slab loads in flight
+    const int hp = kp / 4, items = rows16 * hp;
+    for (int i0 = threadIdx.x; i0 < items; i0 += 4 * 256) {
+      float4 v[4];
+      const float* src[4];
+#pragma unroll
+      for (int u = 0; u < 4; ++u) {
+        const int i = i0 + u * 256, row = i / hp, c = (i % hp) * 4;
+        src[u] = i < items && row < ch.y && c < dn ? reinterpret_cast<const float*>(a.q) + (int64_t)(ch.x + row) * a.ldq + qcol + c : nullptr;
+        v[u] = make_float4(0.f, 0.f, 0.f, 0.f);
+      }
+      for (int s = 0; s < a.nsplit; ++s)
+#pragma unroll
+        for (int u = 0; u < 4; ++u)
+          if (src[u]) add4(v[u], *reinterpret_cast<const float4*>(src[u] + s * a.split_stride));
+#pragma unroll
+      for (int u = 0; u < 4; ++u) {
+        const int i = i0 + u * 256;
+        if (i < items) *reinterpret_cast<uint2*>(sA + (i / hp) * ld + (i % hp) * 4) = make_uint2(pack_bf16(v[u].x, v[u].y), pack_bf16(v[u].z, v[u].w));
       }
     }
-    *reinterpret_cast<uint32_t*>(sA + row * ld + c) = pack_bf16(v.x, v.y);
+  } else {
+    const int hp = kp / 2;
+    for (int i = threadIdx.x; i < rows16 * hp; i += 256) {
+      const int row = i / hp, c = (i % hp) * 2;
+      float2 v = make_float2(0.f, 0.f);
+      if (row < ch.y && c < dn) {
+        if (even) v = q_pair(a, ch.x + row, qcol + c);
+        else {
+          v.x = q_at<bf16>(a, ch.x + row, qcol + c);
+          if (c + 1 < dn) v.y = q_at<bf16>(a, ch.x + row, qcol + c + 1);
+        }
+      }
+      *reinterpret_cast<uint32_t*>(sA + row * ld + c) = pack_bf16(v.x, v.y);
+    }
   }
-  if (blockIdx.x == 0) {
-    const int half = a.m.rope_dims / 2, np = (dr + 1) / 2;
-    for (int i = threadIdx.x; i < ch.y * np; i += 128) {
+  {
+    const int half = a.m.rope_dims / 2, np = (dr + 1) / 2;   // the rotations are shared out over the latent tiles
+    for (int i = blockIdx.x * 256 + threadIdx.x; i < ch.y * np; i += gridDim.x * 256) {
       const int64_t row = ch.x + i / np;
       const int p = i % np;
       float2 v;
@@ -319,7 +358,7 @@ __global__ void __launch_bounds__(128) latent_q_kernel(LatentAttnArgs a) {
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, l8 = lane & 7, lq = lane >> 3, g = lane >> 2, t = lane & 3;
   const int wm = ch.y <= 16 ? 1 : ch.y <= 32 ? 2 : 4, wn = 4 / wm, nt_n = 8 / wn;
   const int mrow = (warp % wm) * 16, ncol = (warp / wm) * nt_n * 8;
-  if (mrow >= rows16) return;
+  if (warp >= 4 || mrow >= rows16) return;
   float acc[8][4];
 #pragma unroll
   for (int i = 0; i < 8; ++i)
@@ -369,7 +408,7 @@ struct AbsCfg {
 constexpr int ABS_OG = 4;       // 16-column value groups per warp: kv_rank up to 512
 
 template <int MT>
-__global__ void __launch_bounds__(256) latent_attn_kernel(const __grid_constant__ CUtensorMap tm, LatentAttnArgs a, AbsCfg cf) {
+__global__ void __launch_bounds__(288) latent_attn_kernel(const __grid_constant__ CUtensorMap tm, LatentAttnArgs a, AbsCfg cf) {
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
   constexpr int R = 16 * MT, TPR = 256 / R, KPT = 64 / TPR;   // rows, threads per row, keys per thread
@@ -379,17 +418,23 @@ __global__ void __launch_bounds__(256) latent_attn_kernel(const __grid_constant_
   uint8_t* sP = sQ + cf.boxes * R * 128;                      // [R rows][128 bytes]
   float* sS = reinterpret_cast<float*>(sP + R * 128);         // [2][R][68]
   float* sAl = sS + 2 * R * 68;                               // [R]
-  uint64_t* full = reinterpret_cast<uint64_t*>(sAl + R);
+  uint64_t* full = reinterpret_cast<uint64_t*>(sAl + R);      // [stages] filled by TMA
+  uint64_t* empty = full + 4;                                 // [stages] released by the eight consumer warps
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, l8 = lane & 7, lq = lane >> 3, g = lane >> 2, t = lane & 3;
-  if (tid == 0) {
-    for (int i = 0; i < cf.stages; ++i) mbar_init(&full[i], 1);
+  if (tid == 256) {
+    for (int i = 0; i < cf.stages; ++i) {
+      mbar_init(&full[i], 1);
+      mbar_init(&empty[i], 8);
+    }
     fence_barrier_init();
     tma_prefetch_desc(&tm);
   }
   pdl_launch_dependents();
-  pdl_wait();
-  const int2 tr = tile_rows(a.tiles, blockIdx.y / cf.subtiles);
-  const int tok0 = (blockIdx.y % cf.subtiles) * cf.tokens_per;
+  __syncthreads();
+  // In a captured decode step positions and block tables predate the step, and so do all cache rows but the newest.
+  if (!a.early_kv) pdl_wait();
+  const int2 tr = tile_rows(a.tiles, (int)blockIdx.y / cf.subtiles);
+  const int tok0 = ((int)blockIdx.y % cf.subtiles) * cf.tokens_per;
   const int ntok = min(cf.tokens_per, tr.y - tok0);
   if (ntok <= 0) return;
   const int64_t row0 = tr.x + tok0;
@@ -399,8 +444,31 @@ __global__ void __launch_bounds__(256) latent_attn_kernel(const __grid_constant_
   const int pos_first = min(max(row_pos(a.map, row0), 0), cap - 1), pos_last = min(pos_first + ntok - 1, cap - 1);
   const int k_lo = a.m.window > 0 ? max(0, pos_first - a.m.window + 1) : 0;
   const int t_lo = k_lo / PAGE_TOKENS, nt_all = pos_last / PAGE_TOKENS - t_lo + 1;
-  const int per = (nt_all + gridDim.x - 1) / gridDim.x;
-  const int t0 = t_lo + blockIdx.x * per, nt = max(0, min(per, t_lo + nt_all - t0));
+  const int per = (nt_all + (int)gridDim.x - 1) / (int)gridDim.x;
+  const int t0 = t_lo + (int)blockIdx.x * per, nt = max(0, min(per, t_lo + nt_all - t0));
+  if (warp == 8) {
+    // ---- producer
+    if (lane == 0) {
+      auto load_page = [&](int i) {
+        const int st = i % cf.stages;
+        const int page = a.block_table[(int64_t)lane_id * a.max_pages + t0 + i];
+        mbar_expect_tx(&full[st], stage_bytes);
+        for (int b = 0; b < cf.boxes; ++b) tma_load_2d(sKV + st * stage_bytes + b * 8192, &tm, &full[st], b * 64, page * PAGE_TOKENS);
+      };
+      int i = 0;
+      if (a.early_kv) {
+        const int newest = pos_last / PAGE_TOKENS - t0;   // the page the step's own row is written to
+        for (; i < min(cf.stages, nt) && i < newest; ++i) load_page(i);
+        pdl_wait();
+      }
+      for (; i < nt; ++i) {
+        if (i >= cf.stages && !mbar_wait(&empty[i % cf.stages], ((i / cf.stages) - 1) & 1, a.status)) break;
+        load_page(i);
+      }
+    }
+    return;
+  }
+  if (a.early_kv) pdl_wait();
   // queries
   for (int i = tid; i < R * cf.boxes * 8; i += 256) {
     const int m = i / (cf.boxes * 8), c = i % (cf.boxes * 8);
@@ -410,15 +478,8 @@ __global__ void __launch_bounds__(256) latent_attn_kernel(const __grid_constant_
       v = *reinterpret_cast<const uint4*>(reinterpret_cast<const bf16*>(a.qeff) + ((row0 + tok) * a.m.heads + head0 + hh) * a.ldc + c * 8);
     *reinterpret_cast<uint4*>(sQ + (c >> 3) * (R * 128) + swz128((uint32_t)m, (uint32_t)(c & 7))) = v;
   }
-  __syncthreads();
-  auto load_page = [&](int i) {
-    const int st = i % cf.stages;
-    const int page = a.block_table[(int64_t)lane_id * a.max_pages + t0 + i];
-    mbar_expect_tx(&full[st], stage_bytes);
-    for (int b = 0; b < cf.boxes; ++b) tma_load_2d(sKV + st * stage_bytes + b * 8192, &tm, &full[st], b * 64, page * PAGE_TOKENS);
-  };
-  if (tid == 0)
-    for (int i = 0; i < min(cf.stages, nt); ++i) load_page(i);
+  auto consumers_sync = [] { asm volatile("bar.sync 1, 256;" ::: "memory"); };
+  consumers_sync();
 
   // softmax ownership: thread -> (row, KPT keys)
   const int srow = tid / TPR, skey = (tid % TPR) * KPT;
@@ -440,7 +501,7 @@ __global__ void __launch_bounds__(256) latent_attn_kernel(const __grid_constant_
   bool ok = true;
   for (int it = 0; it < nt; ++it) {
     const int st = it % cf.stages;
-    ok = mbar_wait(&full[st], (it / cf.stages) & 1, a.status);
+    if (ok) ok = mbar_wait(&full[st], (it / cf.stages) & 1, a.status);
     const uint32_t kv = smem_u32(sKV) + st * stage_bytes;
     float sc[MT][2][4];
 #pragma unroll
@@ -466,7 +527,7 @@ __global__ void __launch_bounds__(256) latent_attn_kernel(const __grid_constant_
 #pragma unroll
         for (int hf = 0; hf < 2; ++hf)
           *reinterpret_cast<float2*>(sS + (kh * R + i * 16 + g + hf * 8) * 68 + kg * 16 + n * 8 + 2 * t) = make_float2(sc[i][n][2 * hf], sc[i][n][2 * hf + 1]);
-    __syncthreads();
+    consumers_sync();
     {
       const int key0 = (t0 + it) * PAGE_TOKENS + skey;
       float x[KPT], mx = -INFINITY;
@@ -497,7 +558,7 @@ __global__ void __launch_bounds__(256) latent_attn_kernel(const __grid_constant_
       for (int e = 0; e < KPT / 2; ++e) *reinterpret_cast<uint32_t*>(pd + e * 4) = pk[e];
       if (tid % TPR == 0) sAl[srow] = alpha;
     }
-    __syncthreads();
+    consumers_sync();
 #pragma unroll
     for (int i = 0; i < MT; ++i) {
       const float a0 = sAl[i * 16 + g], a1 = sAl[i * 16 + g + 8];
@@ -530,9 +591,10 @@ __global__ void __launch_bounds__(256) latent_attn_kernel(const __grid_constant_
         }
       }
     }
-    ok = __syncthreads_and(ok);   // everyone is done with the stage, the scores and the probabilities
-    if (!ok) break;
-    if (tid == 0 && it + cf.stages < nt) load_page(it + cf.stages);
+    __syncwarp();
+    if (lane == 0) mbar_arrive(&empty[st]);
+    // the next scores go to a buffer every warp has left: the probabilities and factors are rewritten only behind
+    // the next barrier, which every warp reaches after this page's products
   }
   if (!ok) return;
 #pragma unroll
@@ -560,24 +622,26 @@ __global__ void __launch_bounds__(256) latent_attn_kernel(const __grid_constant_
     a.ml[((row0 + stok) * a.m.heads + head0 + srow % cf.heads_per) * a.kv_splits + blockIdx.x] = make_float2(m_run, l_run);
 }
 
-constexpr int LO_ROWS = 32, LO_N = 32;
+constexpr int LO_ROWS = 16, LO_N = 32, LO_PARTS = kChunkRows / LO_ROWS;
 
-// grid (value tiles, heads, chunks * 2): merges the kv splits, out[row][head][n0 .. n0+31] = gate * sum_k o[k] W_uv[k][n]
-__global__ void __launch_bounds__(128) latent_out_kernel(LatentAttnArgs a) {
+// grid (value tiles, heads, chunks * LO_PARTS), 256 threads: merges the kv splits, then
+// out[row][head][n0 .. n0+31] = gate * sum_k o[k] W_uv[k][n].  Warp w: columns 8 (w & 3) .. +7, half (w >> 2) of k.
+__global__ void __launch_bounds__(256) latent_out_kernel(LatentAttnArgs a) {
   extern __shared__ __align__(16) uint8_t smem_raw[];
   const int h = blockIdx.y, r = a.m.kv_rank, dv = a.m.vdim;
-  const int kp = (r + 15) / 16 * 16, ld = kp + 8;
+  const int kp = (r + 63) / 64 * 64, ld = kp + 8;   // two halves of whole 32-wide steps
   bf16* sA = reinterpret_cast<bf16*>(smem_raw);
   bf16* sB = sA + LO_ROWS * ld;                 // [kp][LO_N + 8]
   constexpr int ldb = LO_N + 8;
   __shared__ float sw[LO_ROWS][17];
-  const int n0 = blockIdx.x * LO_N;
+  __shared__ float sred[4][32][4];
+  const int n0 = blockIdx.x * LO_N, tid = threadIdx.x;
   pdl_launch_dependents();
   const int64_t c0 = (int64_t)a.m.heads * a.m.dim + (int64_t)h * dv + n0;
   stage_matrix(sB, ldb, reinterpret_cast<const bf16*>(a.ukv) + c0, a.ld_ukv, r, min(LO_N, dv - n0), kp, LO_N, c0 % 8 == 0);
   pdl_wait();
-  int2 ch = chunk_rows(a, (int)(blockIdx.z >> 1));
-  const int skip = (int)(blockIdx.z & 1) * LO_ROWS;
+  int2 ch = chunk_rows(a, (int)blockIdx.z / LO_PARTS);
+  const int skip = ((int)blockIdx.z % LO_PARTS) * LO_ROWS;
   ch.x += skip;
   ch.y = min(LO_ROWS, ch.y - skip);
   if (ch.y <= 0) {
@@ -585,69 +649,86 @@ __global__ void __launch_bounds__(128) latent_out_kernel(LatentAttnArgs a) {
     return;
   }
   const int ns = a.kv_splits;
-  // weights of the splits: exp(m_s - M) / sum
-  if (threadIdx.x < LO_ROWS) {
-    const int row = threadIdx.x;
-    if (row < ch.y) {
-      const float2* ml = a.ml + ((int64_t)(ch.x + row) * a.m.heads + h) * ns;
-      float M = -INFINITY, L = 0.f;
-      for (int s = 0; s < ns; ++s) M = fmaxf(M, ml[s].x);
-      for (int s = 0; s < ns; ++s) {
-        const float f = ml[s].x == -INFINITY ? 0.f : __expf(ml[s].x - M);
-        sw[row][s] = f;
-        L += ml[s].y * f;
-      }
-      for (int s = 0; s < ns; ++s) sw[row][s] /= L;
-    }
+  {
+    // weights of the splits, exp(m_s - M) / sum: 16 threads a row, one split each
+    const int row = tid >> 4, s = tid & 15;
+    const bool in = row < ch.y && s < ns;
+    const float2 ml = in ? a.ml[((int64_t)(ch.x + row) * a.m.heads + h) * ns + s] : make_float2(-INFINITY, 0.f);
+    float M = ml.x;
+#pragma unroll
+    for (int o = 8; o > 0; o >>= 1) M = fmaxf(M, __shfl_xor_sync(0xffffffffu, M, o));
+    const float f = ml.x == -INFINITY ? 0.f : __expf(ml.x - M);
+    float L = ml.y * f;
+#pragma unroll
+    for (int o = 8; o > 0; o >>= 1) L += __shfl_xor_sync(0xffffffffu, L, o);
+    sw[row][s] = L > 0.f ? f / L : 0.f;
   }
   __syncthreads();
-  const int hp = kp / 2, rows16 = (ch.y + 15) / 16 * 16;
-  for (int i = threadIdx.x; i < rows16 * hp; i += 128) {
-    const int row = i / hp, c = (i % hp) * 2;
-    float2 v = make_float2(0.f, 0.f);
-    if (row < ch.y && c < r) {
-      const float* o = a.olat + ((int64_t)(ch.x + row) * a.m.heads + h) * ns * r + c;
-      const bool pair = (r & 1) == 0;
-      for (int s = 0; s < ns; ++s) {
-        const float w = sw[row][s];
-        if (w == 0.f) continue;   // a split without keys of this row has written nothing that counts
-        if (pair) {
-          const float2 x = *reinterpret_cast<const float2*>(o + (int64_t)s * r);
-          v.x += w * x.x;
-          v.y += w * x.y;
-        } else {
-          v.x += w * o[(int64_t)s * r];
-          if (c + 1 < r) v.y += w * o[(int64_t)s * r + 1];
-        }
+  if (r % 4 == 0) {
+    // four columns a thread, eight independent chains of split loads in flight
+    constexpr int U = 8;
+    const int hp = kp / 4, items = LO_ROWS * hp;
+    for (int i0 = tid; i0 < items; i0 += U * 256) {
+      float4 v[U];
+      const float* src[U];
+#pragma unroll
+      for (int u = 0; u < U; ++u) {
+        const int i = i0 + u * 256, row = i / hp, c = (i % hp) * 4;
+        src[u] = row < ch.y && c < r ? a.olat + ((int64_t)(ch.x + row) * a.m.heads + h) * ns * r + c : nullptr;
+        v[u] = make_float4(0.f, 0.f, 0.f, 0.f);
+      }
+      for (int s = 0; s < ns; ++s)
+#pragma unroll
+        for (int u = 0; u < U; ++u)
+          if (src[u]) {
+            const float4 x = *reinterpret_cast<const float4*>(src[u] + (int64_t)s * r);
+            const float f = sw[min((i0 + u * 256) / hp, LO_ROWS - 1)][s];
+            v[u].x = fmaf(f, x.x, v[u].x);
+            v[u].y = fmaf(f, x.y, v[u].y);
+            v[u].z = fmaf(f, x.z, v[u].z);
+            v[u].w = fmaf(f, x.w, v[u].w);
+          }
+#pragma unroll
+      for (int u = 0; u < U; ++u) {
+        const int i = i0 + u * 256;
+        if (i < items) *reinterpret_cast<uint2*>(sA + (i / hp) * ld + (i % hp) * 4) = make_uint2(pack_bf16(v[u].x, v[u].y), pack_bf16(v[u].z, v[u].w));
       }
     }
-    *reinterpret_cast<uint32_t*>(sA + row * ld + c) = pack_bf16(v.x, v.y);
+  } else {
+    for (int i = tid; i < LO_ROWS * kp; i += 256) {
+      const int row = i / kp, c = i % kp;
+      float v = 0.f;
+      if (row < ch.y && c < r)
+        for (int s = 0; s < ns; ++s) v += sw[row][s] * a.olat[(((int64_t)(ch.x + row) * a.m.heads + h) * ns + s) * r + c];
+      sA[row * ld + c] = stf<bf16>(v);
+    }
   }
   cp_async_wait();
   __syncthreads();
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, l8 = lane & 7, lq = lane >> 3, g = lane >> 2, t = lane & 3;
-  const int mrow = (warp & 1) * 16, ncol = (warp >> 1) * 16;
-  if (mrow >= rows16) return;
-  float acc[2][4] = {};
+  const int warp = tid >> 5, lane = tid & 31, l8 = lane & 7, lq = lane >> 3, g = lane >> 2, t = lane & 3;
+  const int nq = warp & 3, kh = warp >> 2;
+  float acc[4] = {};
   const uint32_t aA = smem_u32(sA), aB = smem_u32(sB);
-  for (int k = 0; k < kp; k += 16) {
-    uint32_t af[4], b0, b1, b2, b3;
-    ldmatrix_x4(af[0], af[1], af[2], af[3], aA + ((mrow + (lq & 1) * 8 + l8) * ld + k + (lq >> 1) * 8) * 2);
-    ldmatrix_x4_trans(b0, b1, b2, b3, aB + ((k + (lq & 1) * 8 + l8) * ldb + ncol + (lq >> 1) * 8) * 2);
-    mma_bf16_16816(acc[0], af, b0, b1);
-    mma_bf16_16816(acc[1], af, b2, b3);
+  for (int k = kh * (kp / 2); k < (kh + 1) * (kp / 2); k += 32) {
+    uint32_t a0[4], a1[4], b0, b1, b2, b3;
+    ldmatrix_x4(a0[0], a0[1], a0[2], a0[3], aA + (((lq & 1) * 8 + l8) * ld + k + (lq >> 1) * 8) * 2);
+    ldmatrix_x4(a1[0], a1[1], a1[2], a1[3], aA + (((lq & 1) * 8 + l8) * ld + k + 16 + (lq >> 1) * 8) * 2);
+    ldmatrix_x4_trans(b0, b1, b2, b3, aB + ((k + lq * 8 + l8) * ldb + nq * 8) * 2);
+    mma_bf16_16816(acc, a0, b0, b1);
+    mma_bf16_16816(acc, a1, b2, b3);
   }
+  if (kh == 1) *reinterpret_cast<float4*>(sred[nq][lane]) = make_float4(acc[0], acc[1], acc[2], acc[3]);
+  __syncthreads();
+  if (kh == 1) return;
 #pragma unroll
-  for (int i = 0; i < 2; ++i)
-#pragma unroll
-    for (int hf = 0; hf < 2; ++hf) {
-      const int row = mrow + g + hf * 8, n = n0 + ncol + i * 8 + 2 * t;
-      if (row >= ch.y || n >= dv) continue;
-      const float gt = a.m.gate ? a.gate[(int64_t)(ch.x + row) * a.m.heads + h] : 1.0f;
-      bf16* op = reinterpret_cast<bf16*>(a.out) + (int64_t)(ch.x + row) * a.ldo + (int64_t)h * dv + n;
-      op[0] = stf<bf16>(acc[i][2 * hf] * gt);
-      if (n + 1 < dv) op[1] = stf<bf16>(acc[i][2 * hf + 1] * gt);
-    }
+  for (int hf = 0; hf < 2; ++hf) {
+    const int row = g + hf * 8, n = n0 + nq * 8 + 2 * t;
+    if (row >= ch.y || n >= dv) continue;
+    const float gt = a.m.gate ? a.gate[(int64_t)(ch.x + row) * a.m.heads + h] : 1.0f;
+    bf16* op = reinterpret_cast<bf16*>(a.out) + (int64_t)(ch.x + row) * a.ldo + (int64_t)h * dv + n;
+    op[0] = stf<bf16>((acc[2 * hf] + sred[nq][lane][2 * hf]) * gt);
+    if (n + 1 < dv) op[1] = stf<bf16>((acc[2 * hf + 1] + sred[nq][lane][2 * hf + 1]) * gt);
+  }
 }
 
 template <typename T>
@@ -675,8 +756,8 @@ int plain_launch(Ctx* c, const LatentAttnArgs& a) {
 
 int latent_post_launch(Ctx* c, const LatentPostArgs& a, int64_t rows) {
   if (rows == 0) return REWB200_OK;
-  const size_t smem = (size_t)(a.m.q_rank + a.m.kv_rank + a.m.rot_dim + a.m.heads) * sizeof(float);
-  RB_REQUIRE(smem <= 48 * 1024, "latent attention: the input projection is wider than 12288 columns");
+  const size_t smem = (size_t)a.ld * sizeof(float);
+  RB_REQUIRE(a.ld % 4 == 0 && smem <= 48 * 1024, "latent attention: the input projection is wider than 12288 columns");
   if (a.dtype == REWB200_BF16)
     RB_CUDA(launch_k(latent_post_kernel<bf16>, dim3((unsigned)rows), dim3(256), smem, c->stream, c->use_pdl, a));
   else
@@ -693,15 +774,15 @@ constexpr size_t kSmemMax = 227 * 1024;
 bool abs_config(const LatentDims& m, int64_t ldc, int mt, AbsCfg* cf, size_t* smem) {
   cf->boxes = (int)((m.kv_rank + m.rot_dim + 63) / 64);
   const int R = 16 * mt;
-  const size_t fixed = (size_t)cf->boxes * R * 128 + R * 128 + 2 * R * 68 * 4 + R * 4 + 64 + 1024;
+  const size_t fixed = (size_t)cf->boxes * R * 128 + R * 128 + 2 * R * 68 * 4 + R * 4 + 128 + 1024;
   cf->stages = 4;
   while (cf->stages > 1 && fixed + (size_t)cf->stages * cf->boxes * 8192 > kSmemMax) --cf->stages;
   *smem = fixed + (size_t)cf->stages * cf->boxes * 8192;
   const size_t q_smem = (size_t)2 * 64 * ((m.dim + 15) / 16 * 16 + 8) * 2;
-  const int kp = (m.kv_rank + 15) / 16 * 16;
+  const int kp = (m.kv_rank + 63) / 64 * 64;
   const size_t o_smem = (size_t)LO_ROWS * (kp + 8) * 2 + (size_t)kp * (LO_N + 8) * 2;
   (void)ldc;
-  return m.kv_rank <= 16 * 8 * ABS_OG && *smem <= kSmemMax && cf->stages >= 2 && q_smem <= kSmemMax && o_smem <= kSmemMax - 4096;
+  return m.kv_rank <= 16 * 8 * ABS_OG && *smem <= kSmemMax && cf->stages >= 2 && q_smem <= kSmemMax && o_smem <= kSmemMax - 8192;
 }
 
 }  // namespace
@@ -728,7 +809,7 @@ int latent_attn_absorbed_launch(Ctx* c, const LatentAttnArgs& a) {
   cf.heads_per = std::min(a.m.heads, 16 * mt);
   cf.tokens_per = std::min(16 * mt / cf.heads_per, a.max_tile_rows);
   cf.subtiles = (a.max_tile_rows + cf.tokens_per - 1) / cf.tokens_per;
-  const int kp = (a.m.dim + 15) / 16 * 16, rp = (a.m.kv_rank + 15) / 16 * 16;
+  const int kp = (a.m.dim + 15) / 16 * 16, rp = (a.m.kv_rank + 63) / 64 * 64;
   const size_t q_smem = (size_t)(kChunkRows + LQ_N) * (kp + 8) * 2;
   const size_t o_smem = (size_t)LO_ROWS * (rp + 8) * 2 + (size_t)rp * (LO_N + 8) * 2;
   static bool attr_set = false;
@@ -736,16 +817,16 @@ int latent_attn_absorbed_launch(Ctx* c, const LatentAttnArgs& a) {
     RB_CUDA(cudaFuncSetAttribute(latent_q_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kSmemMax));
     RB_CUDA(cudaFuncSetAttribute(latent_attn_kernel<1>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kSmemMax));
     RB_CUDA(cudaFuncSetAttribute(latent_attn_kernel<2>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kSmemMax));
-    RB_CUDA(cudaFuncSetAttribute(latent_out_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kSmemMax - 4096));
+    RB_CUDA(cudaFuncSetAttribute(latent_out_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kSmemMax - 8192));
     attr_set = true;
   }
   const dim3 gq((unsigned)((a.m.kv_rank + LQ_N - 1) / LQ_N), (unsigned)a.m.heads, (unsigned)a.chunks.count);
-  RB_CUDA(launch_k(latent_q_kernel, gq, dim3(128), q_smem, c->stream, c->use_pdl, a));
+  RB_CUDA(launch_k(latent_q_kernel, gq, dim3(256), q_smem, c->stream, c->use_pdl, a));
   const dim3 ga((unsigned)a.kv_splits, (unsigned)(a.tiles.count * cf.subtiles), (unsigned)((a.m.heads + cf.heads_per - 1) / cf.heads_per));
-  if (mt == 1) RB_CUDA(launch_k(latent_attn_kernel<1>, ga, dim3(256), smem, c->stream, c->use_pdl, *a.tm_cache, a, cf));
-  else RB_CUDA(launch_k(latent_attn_kernel<2>, ga, dim3(256), smem, c->stream, c->use_pdl, *a.tm_cache, a, cf));
-  const dim3 go((unsigned)((a.m.vdim + LO_N - 1) / LO_N), (unsigned)a.m.heads, (unsigned)(a.chunks.count * 2));
-  RB_CUDA(launch_k(latent_out_kernel, go, dim3(128), o_smem, c->stream, c->use_pdl, a));
+  if (mt == 1) RB_CUDA(launch_k(latent_attn_kernel<1>, ga, dim3(288), smem, c->stream, c->use_pdl, *a.tm_cache, a, cf));
+  else RB_CUDA(launch_k(latent_attn_kernel<2>, ga, dim3(288), smem, c->stream, c->use_pdl, *a.tm_cache, a, cf));
+  const dim3 go((unsigned)((a.m.vdim + LO_N - 1) / LO_N), (unsigned)a.m.heads, (unsigned)(a.chunks.count * LO_PARTS));
+  RB_CUDA(launch_k(latent_out_kernel, go, dim3(256), o_smem, c->stream, c->use_pdl, a));
   g_launch_total += 3;
   return REWB200_OK;
 }

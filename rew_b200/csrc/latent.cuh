@@ -90,6 +90,7 @@ struct LatentAttnArgs {
   int max_pages;
   int64_t ldc;
   int dtype;
+  int early_kv;            // captured decode step: cache pages other than the newest may be loaded ahead of the stream dependency
   int* status;
 };
 int latent_attn_absorbed_launch(Ctx* c, const LatentAttnArgs& a);

@@ -71,6 +71,23 @@ class LayeredConfig:
         a, b, k = self.loop
         return n[:a] + n[a:b] * k + n[b:]
 
+    def step_bytes(self, batch, ctx):
+        """Bytes a decode step of `batch` sequences streams at context ctx: every layer run's weights (a loop reads them once
+        a pass), the lm_head, and the cache rows the windows see."""
+        es = 2 if self.dtype == _lib.BF16 else 4
+        d, total = self.d_model, self.d_model * self.vocab
+        for i in self.layer_runs:
+            l = self.layers[i]
+            total += d * (l.q_rank + l.kv_rank + l.rot_dim + (l.heads if l.out_gate else 0)) + l.q_rank * l.heads * (l.dim + l.rot_dim)
+            total += l.kv_rank * l.heads * (l.dim + l.vdim) + l.heads * l.vdim * d
+            if l.ff == "dense":
+                total += 3 * d * l.ffn
+            elif l.ff == "experts":
+                total += d * l.experts + min(l.experts, batch * l.top_k) * (3 if l.expert_gated else 2) * d * l.ffn
+            seen = min(ctx, l.window) if l.window else ctx
+            total += batch * seen * (l.kv_rank + l.rot_dim)
+        return total * es
+
     def create(self, slot, out):
         """rewb200_model_create_layers into the handle `out`."""
         import ctypes as C

@@ -67,3 +67,20 @@ def load(model_dir, dtype, max_seq=None, slot=0):
     kw = {} if max_seq is None else dict(max_seq=int(max_seq))
     cfg = config_from_json(os.path.join(model_dir, "config.json"), dtype=dtype, **kw)
     return CausalLM(cfg, slot).load(canonical_tensors(cfg, st.read_safetensors_dir(model_dir)))
+
+
+# Benchmark configurations (shapes only; weights are synthetic).
+def dense_8b(**kw):
+    """Layers of the width, heads and feed-forward of the 8B Llama shape."""
+    from . import _lib
+    layer = LayerSpec(heads=32, dim=128, rot_dim=64, vdim=128, q_rank=1536, kv_rank=512, scale=192 ** -0.5, window=1024,
+                      rope_base=500000.0, ff="dense", ffn=14336)
+    return LayeredConfig(**{**dict(vocab=128256, d_model=4096, layers=[layer] * 32, eps=1e-5, max_seq=2048, dtype=_lib.BF16), **kw})
+
+
+def moe_lite(**kw):
+    """As many layer runs, the width, heads, experts and expert width of the DeepSeek-V2-Lite shape; 13 layers run twice."""
+    from . import _lib
+    mix = dict(heads=16, dim=128, rot_dim=64, vdim=128, q_rank=768, kv_rank=512, scale=192 ** -0.5, window=1024, rope_base=10000.0)
+    layers = [LayerSpec(ff="dense", ffn=10944, **mix)] + [LayerSpec(ff="experts", ffn=1408, experts=64, top_k=6, **mix)] * 13
+    return LayeredConfig(**{**dict(vocab=102400, d_model=2048, layers=layers, loop=(1, 14, 2), eps=1e-6, max_seq=2048, dtype=_lib.BF16), **kw})
