@@ -388,12 +388,10 @@ namespace {
 
 // Rows of one lane an absorbed-attention tile covers at most.
 constexpr int ABS_TILE_ROWS = 8;
-
-struct Plan {
-  int rows = 0;
-  bool uniform = true;   // one token per lane at the lanes' device-side positions: no lists
-  int n_abs = 0;         // absorbed tiles
-};
+// Portions of at least this many tokens attend to keys and values expanded per head.  Expanding costs a Linear over the
+// portion's keys, its own and its window's; the absorbed form costs (2 kv_rank + rot_dim) / (dim + rot_dim + vdim) times
+// the score and value products of every query, on the slower mma.sync pipe.
+constexpr int EXPAND_MIN_ROWS = 64;
 
 template <typename T>
 int regrow(rewb200_session* s, T** p, size_t bytes) {
@@ -419,29 +417,61 @@ int layered_prepare(rewb200_session* s, const FwdOpts& o, int64_t rows) {
   const size_t es = dtype_size(m->cfg.dtype);
   const bool uniform = o.entries == nullptr;
   RB_REQUIRE(!uniform || o.S == 1, "layered step: a step of several tokens per lane needs its portions");
-  // ---- lists of the step: [row lane | row position | absorbed tiles]
-  int64_t abs_rows = rows;
+  // ---- lists of the step: [row lane | row position | absorbed tiles | their chunks | expanded tiles | gathered keys]
+  int64_t abs_rows = rows, n_keys = 0;
   s->plan_host.clear();
-  s->plan_abs_tiles = 0;
+  s->plan_abs_tiles = s->plan_chunks = s->plan_exp_tiles = s->plan_keys = 0;
   if (!uniform) {
     std::vector<int>& h = s->plan_host;
     h.resize(2 * rows);
-    std::vector<int2> tiles;
+    std::vector<int2> tiles, chunks, keys;
+    std::vector<ExpTile> exps;
+    abs_rows = 0;
+    int64_t reach = 0;  // the widest window of any layer, 0: everything
+    bool exp_ok = m->cfg.dtype == REWB200_BF16 && c->latent_impl == 0;
+    for (const LayerDev& D : m->layers) {
+      exp_ok = exp_ok && latent_expanded_ok(D.a.m);
+      reach = D.a.m.window == 0 ? INT32_MAX : std::max<int64_t>(reach, D.a.m.window);
+    }
     for (const StepEntry& e : *o.entries) {
       for (int i = 0; i < e.n; ++i) {
         h[e.row0 + i] = e.lane;
         h[rows + e.row0 + i] = e.pos0 + i;
       }
+      if (exp_ok && e.n >= EXPAND_MIN_ROWS) {
+        const int key0 = (int)std::max<int64_t>(0, (int64_t)e.pos0 - reach + 1);
+        for (int i = 0; i < e.n; i += 256)
+          exps.push_back({e.row0 + i, std::min(256, e.n - i), e.pos0 + i, key0, (int)keys.size() - key0, {0, 0, 0}});
+        for (int p = key0; p < e.pos0 + e.n; ++p) keys.push_back(make_int2(e.lane, p));
+        continue;
+      }
+      abs_rows = e.row0 + e.n;
       for (int i = 0; i < e.n; i += ABS_TILE_ROWS) tiles.push_back(make_int2(e.row0 + i, std::min(ABS_TILE_ROWS, e.n - i)));
+      // the same rows in longer runs, whatever their lanes, for the per-head products around the attention
+      for (int i = 0; i < e.n;) {
+        const bool grow = !chunks.empty() && chunks.back().x + chunks.back().y == e.row0 + i && chunks.back().y < kChunkRows;
+        const int room = grow ? kChunkRows - chunks.back().y : kChunkRows, k = std::min(room, e.n - i);
+        if (grow) chunks.back().y += k;
+        else chunks.push_back(make_int2(e.row0 + i, k));
+        i += k;
+      }
     }
+    // long query tiles first: the last ones of a wave are then short
+    std::stable_sort(exps.begin(), exps.end(), [](const ExpTile& x, const ExpTile& y) { return x.pos0 + x.n - x.key0 > y.pos0 + y.n - y.key0; });
     s->plan_abs_tiles = (int)tiles.size();
-    // the same rows in longer runs, whatever their lanes, for the per-head products around the attention
-    s->plan_chunks = 0;
-    for (int64_t i = 0; i < rows; i += kChunkRows, ++s->plan_chunks)
-      tiles.push_back(make_int2((int)i, (int)std::min<int64_t>(kChunkRows, rows - i)));
-    const size_t at = h.size();
-    h.resize(at + 2 * tiles.size());
-    if (!tiles.empty()) memcpy(h.data() + at, tiles.data(), tiles.size() * sizeof(int2));
+    s->plan_chunks = (int)chunks.size();
+    s->plan_exp_tiles = (int)exps.size();
+    s->plan_keys = (int)keys.size();
+    n_keys = (int64_t)keys.size();
+    auto append = [&](const void* p, size_t bytes) {
+      const size_t at = h.size();
+      h.resize(at + bytes / sizeof(int));
+      if (bytes) memcpy(h.data() + at, p, bytes);
+    };
+    append(tiles.data(), tiles.size() * sizeof(int2));
+    append(chunks.data(), chunks.size() * sizeof(int2));
+    append(exps.data(), exps.size() * sizeof(ExpTile));
+    append(keys.data(), keys.size() * sizeof(int2));
     if (h.size() > s->plan_cap) {
       s->plan_cap = 0;
       RB_TRY(regrow(s, &s->plan_dev, h.size() * 2 * sizeof(int)));
@@ -449,19 +479,38 @@ int layered_prepare(rewb200_session* s, const FwdOpts& o, int64_t rows) {
     }
     RB_CUDA(cudaMemcpyAsync(s->plan_dev, h.data(), h.size() * sizeof(int), cudaMemcpyHostToDevice, c->stream));
   }
+  if (n_keys > s->kvx_rows) {
+    int64_t kv = 0, ldc = 0;
+    for (const LayerDev& D : m->layers) {
+      kv = std::max(kv, D.a.ukv.N);
+      ldc = std::max(ldc, D.a.ldc);
+    }
+    s->kvx_rows = 0;
+    RB_TRY(regrow(s, &s->kvx, (size_t)n_keys * kv * es));
+    RB_TRY(regrow(s, &s->latx, (size_t)n_keys * ldc * es));
+    // rows past a portion's last key are multiplied by zero probabilities: finite from the start
+    RB_CUDA(cudaMemsetAsync(s->kvx, 0, (size_t)n_keys * kv * es, c->stream));
+    RB_CUDA(cudaMemsetAsync(s->latx, 0, (size_t)n_keys * ldc * es, c->stream));
+    s->kvx_rows = n_keys;
+  }
   // ---- scratch of the absorbed path
-  int64_t units = 0, qe = 0;
+  int64_t units = 0, stats = 0, qe = 0;
   for (const LayerDev& D : m->layers) {
     const int64_t H = D.a.m.heads;
     const int sp = latent_kv_splits(c, D.a.m, rows, s->max_len);
-    units = std::max(units, H * sp * std::max<int64_t>(D.a.m.kv_rank, 1));
+    units = std::max(units, H * sp * D.a.m.kv_rank);
+    stats = std::max(stats, H * sp);
     qe = std::max(qe, H * D.a.ldc);
   }
   if (abs_rows * units > s->abs_units) {
     s->abs_units = 0;
     RB_TRY(regrow(s, &s->olat, (size_t)abs_rows * units * sizeof(float)));
-    RB_TRY(regrow(s, &s->ml, (size_t)abs_rows * units * sizeof(float2)));
     s->abs_units = abs_rows * units;
+  }
+  if (abs_rows * stats > s->abs_stats) {
+    s->abs_stats = 0;
+    RB_TRY(regrow(s, &s->ml, (size_t)abs_rows * stats * sizeof(float2)));
+    s->abs_stats = abs_rows * stats;
   }
   if (abs_rows * qe > s->abs_rows) {
     s->abs_rows = 0;
@@ -482,6 +531,9 @@ int layered_blocks(rewb200_session* s, const FwdOpts& o, const NormArgs& na, int
   const bool uniform = o.entries == nullptr;
   RowMap map = {nullptr, nullptr, s->d_pos, o.b0, o.S};
   RowTiles abs = {nullptr, (int)rows, 1, 1}, chunks = {nullptr, (int)((rows + kChunkRows - 1) / kChunkRows), 1, 1};
+  const ExpTile* exp_tiles = nullptr;
+  const int2* key_list = nullptr;
+  const bool expand = !uniform && s->plan_exp_tiles > 0;
   if (!uniform) {
     map.row_lane = s->plan_dev;
     map.row_pos = s->plan_dev + rows;
@@ -489,6 +541,8 @@ int layered_blocks(rewb200_session* s, const FwdOpts& o, const NormArgs& na, int
     abs.count = s->plan_abs_tiles;
     chunks.list = abs.list + abs.count;
     chunks.count = s->plan_chunks;
+    exp_tiles = reinterpret_cast<const ExpTile*>(chunks.list + chunks.count);
+    key_list = reinterpret_cast<const int2*>(exp_tiles + s->plan_exp_tiles);
   }
   auto ahead_of = [&](size_t r, NormArgs& a) {  // what the norm launch in front of run r adds and writes
     if (r == m->runs.size()) {
@@ -594,9 +648,15 @@ int layered_blocks(rewb200_session* s, const FwdOpts& o, const NormArgs& na, int
     aa.chunks = chunks;
     aa.max_tile_rows = uniform ? 1 : ABS_TILE_ROWS;
     aa.rows = rows;
-    RB_TRY(run_linear(s, A.uq, s->cq, A.uq.K, rows, true, 0, s->part, A.uq.N, &ks));
-    aa.q = s->part;
-    aa.nsplit = ks;
+    if (expand) {
+      RB_TRY(run_linear(s, A.uq, s->cq, A.uq.K, rows, false, EPI_BIAS_BF16, s->q, A.uq.N, nullptr));
+      aa.q = s->q;
+      aa.nsplit = 0;
+    } else {
+      RB_TRY(run_linear(s, A.uq, s->cq, A.uq.K, rows, true, 0, s->part, A.uq.N, &ks));
+      aa.q = s->part;
+      aa.nsplit = ks;
+    }
     aa.split_stride = rows * A.uq.N;
     aa.ldq = A.uq.N;
     aa.ukv = A.ukv.w;
@@ -618,6 +678,27 @@ int layered_blocks(rewb200_session* s, const FwdOpts& o, const NormArgs& na, int
     aa.status = c->d_status;
     if (o.trace) RB_TRY(o.trace->mark(TC_QKV_POST));
     RB_TRY(latent_attn_absorbed_launch(c, aa));
+    if (expand) {
+      LatentExpArgs ea;
+      memset(&ea, 0, sizeof(ea));
+      ea.m = A.m;
+      ea.tiles = exp_tiles;
+      ea.count = s->plan_exp_tiles;
+      ea.q = (const bf16*)s->q;
+      ea.ldq = A.uq.N;
+      ea.gate = s->gate;
+      ea.out = (bf16*)s->attn;
+      ea.ldo = D.o.K;
+      ea.kv = (const bf16*)s->kvx;
+      ea.ldkv = A.ukv.N;
+      ea.lat = (const bf16*)s->latx;
+      ea.ldc = A.ldc;
+      ea.keys = s->plan_keys;
+      ea.status = c->d_status;
+      RB_TRY(latent_gather_launch(c, (const bf16*)s->kc[r], s->block_table, s->max_pages, A.ldc, key_list, (bf16*)s->latx, s->plan_keys));
+      RB_TRY(linear_bf16_launch(c, A.ukv.plan, (const bf16*)s->latx, A.ldc, s->plan_keys, EPI_BIAS_BF16, 1, s->kvx, A.ukv.N, nullptr, nullptr, 0));
+      RB_TRY(latent_attn_expanded_launch(c, ea));
+    }
     if (o.trace) RB_TRY(o.trace->mark(TC_ATTN));
     RB_TRY(run_linear(s, D.o, s->attn, D.o.K, rows, true, 0, s->part, dp, &ks_o));
     if (o.trace) RB_TRY(o.trace->mark(TC_O));

@@ -179,7 +179,7 @@ struct rewb200_session {
   void* qeff = nullptr;                // absorbed queries, latent outputs and their row statistics (absorbed rows of a step)
   float* olat = nullptr;
   float2* ml = nullptr;
-  int64_t abs_units = 0, abs_rows = 0; // capacity of olat / ml and of qeff
+  int64_t abs_units = 0, abs_stats = 0, abs_rows = 0; // capacity of olat, ml and qeff
   void *kvx = nullptr, *latx = nullptr;  // keys / values expanded per head, and the gathered cache rows they come from
   int64_t kvx_rows = 0;
   float* layer_rec = nullptr;          // option record_layers: [runs][rows_cap][d]
@@ -190,7 +190,7 @@ struct rewb200_session {
   int* plan_dev = nullptr;             // row maps, tile lists and gather lists of a step that is no captured decode
   size_t plan_cap = 0;
   std::vector<int> plan_host;
-  int plan_abs_tiles = 0, plan_chunks = 0;
+  int plan_abs_tiles = 0, plan_chunks = 0, plan_exp_tiles = 0, plan_keys = 0;
   int* feed_dev = nullptr;             // ids and row lists of a rewb200_lanes_feed step
   size_t feed_cap = 0;
   int64_t route_rows = 0;              // rows of the forward recorded last

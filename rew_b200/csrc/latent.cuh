@@ -96,6 +96,35 @@ struct LatentAttnArgs {
 int latent_attn_absorbed_launch(Ctx* c, const LatentAttnArgs& a);
 int latent_kv_splits(Ctx* c, const LatentDims& m, int64_t tiles, int64_t max_ctx);
 
+// Expanded attention of large prompt portions: keys and values of every head are computed from the gathered cache rows by
+// one Linear, then attention runs on them with tcgen05.  One tile = up to 256 queries of one portion.
+struct ExpTile {
+  int row0, n;     // rows of the step
+  int pos0;        // position of the first one
+  int key0;        // first position of the portion's gathered keys
+  int off;         // row of the gathered buffers = position + off
+  int pad[3];
+};
+struct LatentExpArgs {
+  LatentDims m;
+  const ExpTile* tiles;
+  int count;
+  const bf16* q;           // [rows][ldq], unrotated
+  int64_t ldq;
+  const float* gate;       // [rows][heads]
+  bf16* out;               // [rows][ldo]
+  int64_t ldo;
+  const bf16* kv;          // [keys][ldkv]: heads*dim of keys, then heads*vdim of values
+  int64_t ldkv;
+  const bf16* lat;         // [keys][ldc] gathered cache rows (their rotated part is the shared key part)
+  int64_t ldc, keys;
+  int* status;
+};
+bool latent_expanded_ok(const LatentDims& m);
+int latent_attn_expanded_launch(Ctx* c, const LatentExpArgs& a);
+// dst[i] = cache row of position index[i].y of lane index[i].x
+int latent_gather_launch(Ctx* c, const bf16* cache, const int* block_table, int max_pages, int64_t ldc, const int2* index, bf16* dst, int64_t n);
+
 // Gathers rows of the step: dst[i] = src[index[i]] (width elements of `dtype`).
 int gather_rows_launch(Ctx* c, const void* src, const int* index, void* dst, int64_t n, int64_t width, int dtype);
 

@@ -130,7 +130,7 @@ def test_other_sizes(rb, dtype, i):
 # ---------------------------------------------------------------- cuts, batches, pages
 
 @pytest.mark.parametrize("impl", ["auto", "plain", "absorbed"])
-@pytest.mark.parametrize("cuts", [[300], [2], [1], [7, 2, 31], [64], [63, 2, 65], [130, 1, 129, 1]])
+@pytest.mark.parametrize("cuts", [[300], [2], [1], [7, 2, 31], [64], [63, 2, 65], [130, 1, 129, 1], [100, 160]])
 def test_portions_agree_with_the_whole_prompt(rb, dtype, cuts, impl):
     cfg = K.small()
     t = K.weights(cfg, seed=3, score_gain=2.5)
