@@ -40,70 +40,90 @@ __device__ __forceinline__ float2 rotate(float2 v, float2 cs) {
 
 __device__ __forceinline__ void add4(float4& v, const float4 w) { v.x += w.x; v.y += w.y; v.z += w.z; v.w += w.w; }
 
-__device__ __forceinline__ float block_sum256(float v, float* red) {
+// Sums of two values over the block; every thread gets both.
+__device__ __forceinline__ float2 block_sum2(float2 v, float2* red) {
 #pragma unroll
-  for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
-  const int w = threadIdx.x >> 5;
+  for (int o = 16; o > 0; o >>= 1) {
+    v.x += __shfl_xor_sync(0xffffffffu, v.x, o);
+    v.y += __shfl_xor_sync(0xffffffffu, v.y, o);
+  }
+  if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = v;
   __syncthreads();
-  if ((threadIdx.x & 31) == 0) red[w] = v;
-  __syncthreads();
-  float t = 0.f;
-#pragma unroll
-  for (int i = 0; i < 8; ++i) t += red[i];
+  float2 t = make_float2(0.f, 0.f);
+  for (int i = 0; i < (int)(blockDim.x >> 5); ++i) {
+    t.x += red[i].x;
+    t.y += red[i].y;
+  }
   return t;
 }
 
-// One CTA per row.
+// One CTA per row; small steps have a thread per four columns (up to 768 threads).
 template <typename T>
-__global__ void __launch_bounds__(256) latent_post_kernel(LatentPostArgs a) {
+__global__ void __launch_bounds__(768) latent_post_kernel(LatentPostArgs a) {
   extern __shared__ __align__(16) float sx[];
-  __shared__ float red[8];
+  __shared__ float2 red[32];
   pdl_launch_dependents();
   pdl_wait();
   const int64_t row = blockIdx.x;
+  const int nt = blockDim.x;
   const int nq = a.m.q_rank, nc = a.m.kv_rank, nr = a.m.rot_dim, n = nq + nc + nr + (a.m.gate ? a.m.heads : 0);
+  const int lane = row_lane(a.map, row), pos = row_pos(a.map, row);
+  const bool ok = pos >= 0 && pos < a.capacity && pos < a.m.max_pos;
+  const int page = a.block_table[(int64_t)lane * a.max_pages + (ok ? pos / PAGE_TOKENS : 0)];
   const float* p = a.partial + row * a.ld;
-  float sq = 0.f, sc = 0.f;
-  for (int i = threadIdx.x * 4; i < n; i += 1024) {   // rows are padded to a multiple of 8 columns
+  float2 sq = make_float2(0.f, 0.f);
+  for (int i = threadIdx.x * 4; i < n; i += nt * 4) {   // rows are padded to a multiple of 8 columns
     float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
-    int k = 0;
-    for (; k + 4 <= a.nsplit; k += 4) {
-      float4 w[4];
+    if (a.nsplit == 1) v = *reinterpret_cast<const float4*>(p + i);
+    else for (int k = 0; k < a.nsplit; k += 8) {
+      float4 w[8];
 #pragma unroll
-      for (int u = 0; u < 4; ++u) w[u] = *reinterpret_cast<const float4*>(p + (k + u) * a.split_stride + i);
+      for (int u = 0; u < 8; ++u)
+        w[u] = k + u < a.nsplit ? *reinterpret_cast<const float4*>(p + (k + u) * a.split_stride + i) : make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll
-      for (int u = 0; u < 4; ++u) add4(v, w[u]);
+      for (int u = 0; u < 8; ++u) add4(v, w[u]);
     }
-    for (; k < a.nsplit; ++k) add4(v, *reinterpret_cast<const float4*>(p + k * a.split_stride + i));
     *reinterpret_cast<float4*>(sx + i) = v;
     const float e[4] = {v.x, v.y, v.z, v.w};
 #pragma unroll
     for (int u = 0; u < 4; ++u) {
-      if (i + u < nq) sq += e[u] * e[u];
-      else if (i + u < nq + nc) sc += e[u] * e[u];
+      if (i + u < nq) sq.x += e[u] * e[u];
+      else if (i + u < nq + nc) sq.y += e[u] * e[u];
     }
   }
-  sq = block_sum256(sq, red);
-  sc = block_sum256(sc, red);
-  const float rq = sqrtf(sq / (float)nq + a.eps), rc = sqrtf(sc / (float)nc + a.eps);
-  const int lane = row_lane(a.map, row), pos = row_pos(a.map, row);
-  const bool ok = pos >= 0 && pos < a.capacity && pos < a.m.max_pos;
+  sq = block_sum2(sq, red);
+  const float rq = sqrtf(sq.x / (float)nq + a.eps), rc = sqrtf(sq.y / (float)nc + a.eps);
   if (!ok && threadIdx.x == 0) atomicExch(a.status, KS_BAD_INDEX);
   T* cq = reinterpret_cast<T*>(a.cq) + row * a.ldcq;
-  for (int i = threadIdx.x; i < nq; i += 256) cq[i] = stf<T>(a.q_norm[i] * (sx[i] / rq));
-  if (a.m.gate)
-    for (int i = threadIdx.x; i < a.m.heads; i += 256) a.gate[row * a.m.heads + i] = 1.0f / (1.0f + expf(-sx[nq + nc + nr + i]));
-  if (!ok) return;
-  const int page = a.block_table[(int64_t)lane * a.max_pages + pos / PAGE_TOKENS];
-  T* cr = reinterpret_cast<T*>(a.cache) + ((int64_t)page * PAGE_TOKENS + pos % PAGE_TOKENS) * a.ldc;
-  for (int i = threadIdx.x; i < nc; i += 256) cr[i] = stf<T>(a.kv_norm[i] * (sx[nq + i] / rc));
-  const int half = a.m.rope_dims / 2;
-  for (int i = threadIdx.x; i < half; i += 256) {
-    const float2 v = rotate(make_float2(sx[nq + nc + 2 * i], sx[nq + nc + 2 * i + 1]), a.m.rope[(int64_t)pos * half + i]);
-    cr[nc + 2 * i] = stf<T>(v.x);
-    cr[nc + 2 * i + 1] = stf<T>(v.y);
+  T* cr = reinterpret_cast<T*>(a.cache) + ((int64_t)page * PAGE_TOKENS + (ok ? pos % PAGE_TOKENS : 0)) * a.ldc;
+  // two columns a thread: the pairs of the query latent, of the key/value latent and of the rotated part
+  auto put = [](T* d, float x, float y) {
+    if constexpr (sizeof(T) == 2) {
+      if ((reinterpret_cast<uintptr_t>(d) & 3) == 0) {
+        *reinterpret_cast<uint32_t*>(d) = pack_bf16(x, y);
+        return;
+      }
+    }
+    d[0] = stf<T>(x);
+    d[1] = stf<T>(y);
+  };
+  for (int i = threadIdx.x * 2; i < nq; i += nt * 2) {
+    if (i + 1 < nq) put(cq + i, a.q_norm[i] * (sx[i] / rq), a.q_norm[i + 1] * (sx[i + 1] / rq));
+    else cq[i] = stf<T>(a.q_norm[i] * (sx[i] / rq));
   }
-  for (int i = 2 * half + threadIdx.x; i < nr; i += 256) cr[nc + i] = stf<T>(sx[nq + nc + i]);
+  if (a.m.gate)
+    for (int i = threadIdx.x; i < a.m.heads; i += nt) a.gate[row * a.m.heads + i] = 1.0f / (1.0f + expf(-sx[nq + nc + nr + i]));
+  if (!ok) return;
+  for (int i = threadIdx.x * 2; i < nc; i += nt * 2) {
+    if (i + 1 < nc) put(cr + i, a.kv_norm[i] * (sx[nq + i] / rc), a.kv_norm[i + 1] * (sx[nq + i + 1] / rc));
+    else cr[i] = stf<T>(a.kv_norm[i] * (sx[nq + i] / rc));
+  }
+  const int half = a.m.rope_dims / 2;
+  for (int i = threadIdx.x; i < half; i += nt) {
+    const float2 v = rotate(make_float2(sx[nq + nc + 2 * i], sx[nq + nc + 2 * i + 1]), a.m.rope[(int64_t)pos * half + i]);
+    put(cr + nc + 2 * i, v.x, v.y);
+  }
+  for (int i = 2 * half + threadIdx.x; i < nr; i += nt) cr[nc + i] = stf<T>(sx[nq + nc + i]);
 }
 
 // ------------------------------------------------------------------ plain kernels (f32 models, and shapes the
@@ -495,30 +515,58 @@ __global__ void __launch_bounds__(288) latent_attn_kernel(const __grid_constant_
 #pragma unroll
       for (int e = 0; e < 8; ++e) acc[i][j][e >> 2][e & 3] = 0.f;
   const int groups = (a.m.kv_rank + 15) / 16;
-  const uint32_t q_base = smem_u32(sQ), p_base = smem_u32(sP);
   const int kg = warp & 3, kh = warp >> 2;
-  const int ks0 = kh * cf.boxes * 2, ks1 = ks0 + cf.boxes * 2;   // 16-feature steps of this warp's half
+  // Lane addresses.  Every row an ldmatrix lane points at is l8 modulo 8, so the swizzle is a constant of the lane and
+  // the loops below add constants only.  Half kh of the features: 16-feature steps 2 kh and 2 kh + 1 of every box.
+  uint32_t k_off[2], q_off[2], p_off[4];
+#pragma unroll
+  for (int u = 0; u < 2; ++u) {
+    const uint32_t ch = (2 * kh + u) * 2;
+    k_off[u] = swz128(kg * 16 + (lq >> 1) * 8 + l8, ch + (lq & 1));
+    q_off[u] = smem_u32(sQ) + swz128((lq & 1) * 8 + l8, ch + (lq >> 1));
+  }
+#pragma unroll
+  for (int k = 0; k < 4; ++k) p_off[k] = smem_u32(sP) + swz128((lq & 1) * 8 + l8, k * 2 + (lq >> 1));
+  const uint32_t v_off = (warp >> 2) * 8192 + swz128((lq & 1) * 8 + l8, (warp & 3) * 2 + (lq >> 1));
+  const uint32_t kv_base = smem_u32(sKV);
+  float* const s_row = sS + (kh * R + g) * 68 + kg * 16 + 2 * t;
   bool ok = true;
   for (int it = 0; it < nt; ++it) {
     const int st = it % cf.stages;
     if (ok) ok = mbar_wait(&full[st], (it / cf.stages) & 1, a.status);
-    const uint32_t kv = smem_u32(sKV) + st * stage_bytes;
+    const uint32_t kv = kv_base + st * stage_bytes;
     float sc[MT][2][4];
 #pragma unroll
     for (int i = 0; i < MT; ++i)
 #pragma unroll
       for (int e = 0; e < 8; ++e) sc[i][e >> 2][e & 3] = 0.f;
-    for (int k = ks0; k < ks1; ++k) {
-      const uint32_t box = k >> 2, ch = (k & 3) * 2;
-      uint32_t b0, b1, b2, b3;
-      ldmatrix_x4(b0, b1, b2, b3, kv + box * 8192 + swz128(kg * 16 + (lq >> 1) * 8 + l8, ch + (lq & 1)));
+    // the fragments of the next box are requested ahead of this box's products
+    uint32_t bf[2][2][4], af[2][2][MT][4];
+    auto fetch = [&](int slot, uint32_t kb, uint32_t qb) {
 #pragma unroll
-      for (int i = 0; i < MT; ++i) {
-        uint32_t af[4];
-        ldmatrix_x4(af[0], af[1], af[2], af[3], q_base + box * (R * 128) + swz128(i * 16 + (lq & 1) * 8 + l8, ch + (lq >> 1)));
-        mma_bf16_16816(sc[i][0], af, b0, b1);
-        mma_bf16_16816(sc[i][1], af, b2, b3);
+      for (int u = 0; u < 2; ++u) {
+        ldmatrix_x4(bf[slot][u][0], bf[slot][u][1], bf[slot][u][2], bf[slot][u][3], kb + k_off[u]);
+#pragma unroll
+        for (int i = 0; i < MT; ++i)
+          ldmatrix_x4(af[slot][u][i][0], af[slot][u][i][1], af[slot][u][i][2], af[slot][u][i][3], qb + q_off[u] + i * 2048);
       }
+    };
+    auto products = [&](int slot) {
+#pragma unroll
+      for (int u = 0; u < 2; ++u)
+#pragma unroll
+        for (int i = 0; i < MT; ++i) {
+          mma_bf16_16816(sc[i][0], af[slot][u][i], bf[slot][u][0], bf[slot][u][1]);
+          mma_bf16_16816(sc[i][1], af[slot][u][i], bf[slot][u][2], bf[slot][u][3]);
+        }
+    };
+    fetch(0, kv, 0);
+    for (int b = 0; b < cf.boxes; b += 2) {
+      if (b + 1 < cf.boxes) fetch(1, kv + (b + 1) * 8192, (b + 1) * (R * 128));
+      products(0);
+      if (b + 1 >= cf.boxes) break;
+      if (b + 2 < cf.boxes) fetch(0, kv + (b + 2) * 8192, (b + 2) * (R * 128));
+      products(1);
     }
 #pragma unroll
     for (int i = 0; i < MT; ++i)
@@ -526,32 +574,37 @@ __global__ void __launch_bounds__(288) latent_attn_kernel(const __grid_constant_
       for (int n = 0; n < 2; ++n)
 #pragma unroll
         for (int hf = 0; hf < 2; ++hf)
-          *reinterpret_cast<float2*>(sS + (kh * R + i * 16 + g + hf * 8) * 68 + kg * 16 + n * 8 + 2 * t) = make_float2(sc[i][n][2 * hf], sc[i][n][2 * hf + 1]);
+          *reinterpret_cast<float2*>(s_row + (i * 16 + hf * 8) * 68 + n * 8) = make_float2(sc[i][n][2 * hf], sc[i][n][2 * hf + 1]);
     consumers_sync();
     {
       const int key0 = (t0 + it) * PAGE_TOKENS + skey;
       float x[KPT], mx = -INFINITY;
 #pragma unroll
+      for (int e = 0; e < KPT; e += 4) {
+        const float4 s0 = *reinterpret_cast<const float4*>(sS + srow * 68 + skey + e), s1 = *reinterpret_cast<const float4*>(sS + (R + srow) * 68 + skey + e);
+        x[e] = s0.x + s1.x;
+        x[e + 1] = s0.y + s1.y;
+        x[e + 2] = s0.z + s1.z;
+        x[e + 3] = s0.w + s1.w;
+      }
+#pragma unroll
       for (int e = 0; e < KPT; ++e) {
-        const float v = (sS[srow * 68 + skey + e] + sS[(R + srow) * 68 + skey + e]) * a.m.scale;
-        x[e] = (sval && key0 + e <= spos && key0 + e > slo) ? v : -INFINITY;
+        x[e] = (sval && key0 + e <= spos && key0 + e > slo) ? x[e] * a.m.scale : -INFINITY;
         mx = fmaxf(mx, x[e]);
       }
 #pragma unroll
       for (int o = TPR / 2; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
       const float m_new = fmaxf(m_run, mx), m_use = m_new == -INFINITY ? 0.f : m_new;
       const float alpha = __expf(m_run - m_use);
-      float ps = 0.f;
       uint32_t pk[KPT / 2];
+      float ps = 0.f;
 #pragma unroll
       for (int e = 0; e < KPT; e += 2) {
         const float p0 = __expf(x[e] - m_use), p1 = __expf(x[e + 1] - m_use);
         ps += p0 + p1;
         pk[e / 2] = pack_bf16(p0, p1);
       }
-#pragma unroll
-      for (int o = TPR / 2; o > 0; o >>= 1) ps += __shfl_xor_sync(0xffffffffu, ps, o);
-      l_run = l_run * alpha + ps;
+      l_run = l_run * alpha + ps;   // this thread's keys; the row's threads meet after the last page
       m_run = m_new;
       uint8_t* pd = sP + swz128((uint32_t)srow, (uint32_t)(skey >> 3)) + (skey & 7) * 2;
 #pragma unroll
@@ -562,32 +615,33 @@ __global__ void __launch_bounds__(288) latent_attn_kernel(const __grid_constant_
 #pragma unroll
     for (int i = 0; i < MT; ++i) {
       const float a0 = sAl[i * 16 + g], a1 = sAl[i * 16 + g + 8];
+      if (__any_sync(0xffffffffu, a0 != 1.f || a1 != 1.f)) {
 #pragma unroll
-      for (int j = 0; j < ABS_OG; ++j)
+        for (int j = 0; j < ABS_OG; ++j)
 #pragma unroll
-        for (int n = 0; n < 2; ++n) {
-          acc[i][j][n][0] *= a0;
-          acc[i][j][n][1] *= a0;
-          acc[i][j][n][2] *= a1;
-          acc[i][j][n][3] *= a1;
-        }
+          for (int n = 0; n < 2; ++n) {
+            acc[i][j][n][0] *= a0;
+            acc[i][j][n][1] *= a0;
+            acc[i][j][n][2] *= a1;
+            acc[i][j][n][3] *= a1;
+          }
+      }
     }
 #pragma unroll
     for (int k = 0; k < 4; ++k) {   // 16 keys a step
-      uint32_t pf[MT][4];
+      uint32_t pf[MT][4], vf[ABS_OG][4];
 #pragma unroll
-      for (int i = 0; i < MT; ++i)
-        ldmatrix_x4(pf[i][0], pf[i][1], pf[i][2], pf[i][3], p_base + swz128(i * 16 + (lq & 1) * 8 + l8, k * 2 + (lq >> 1)));
+      for (int i = 0; i < MT; ++i) ldmatrix_x4(pf[i][0], pf[i][1], pf[i][2], pf[i][3], p_off[k] + i * 2048);
+#pragma unroll
+      for (int j = 0; j < ABS_OG; ++j)   // value columns 16 (warp + 8 j) ..: box (warp >> 2) + 2 j
+        if (warp + 8 * j < groups) ldmatrix_x4_trans(vf[j][0], vf[j][1], vf[j][2], vf[j][3], kv + v_off + j * 16384 + k * 2048);
 #pragma unroll
       for (int j = 0; j < ABS_OG; ++j) {
-        const int grp = warp + 8 * j;
-        if (grp >= groups) break;
-        uint32_t v0, v1, v2, v3;
-        ldmatrix_x4_trans(v0, v1, v2, v3, kv + (grp >> 2) * 8192 + swz128(k * 16 + (lq & 1) * 8 + l8, (grp & 3) * 2 + (lq >> 1)));
+        if (warp + 8 * j >= groups) break;
 #pragma unroll
         for (int i = 0; i < MT; ++i) {
-          mma_bf16_16816(acc[i][j][0], pf[i], v0, v1);
-          mma_bf16_16816(acc[i][j][1], pf[i], v2, v3);
+          mma_bf16_16816(acc[i][j][0], pf[i], vf[j][0], vf[j][1]);
+          mma_bf16_16816(acc[i][j][1], pf[i], vf[j][2], vf[j][3]);
         }
       }
     }
@@ -596,6 +650,8 @@ __global__ void __launch_bounds__(288) latent_attn_kernel(const __grid_constant_
     // the next scores go to a buffer every warp has left: the probabilities and factors are rewritten only behind
     // the next barrier, which every warp reaches after this page's products
   }
+#pragma unroll
+  for (int o = TPR / 2; o > 0; o >>= 1) l_run += __shfl_xor_sync(0xffffffffu, l_run, o);
   if (!ok) return;
 #pragma unroll
   for (int i = 0; i < MT; ++i)
@@ -637,6 +693,7 @@ __global__ void __launch_bounds__(256) latent_out_kernel(LatentAttnArgs a) {
   __shared__ float sred[4][32][4];
   const int n0 = blockIdx.x * LO_N, tid = threadIdx.x;
   pdl_launch_dependents();
+  if (!a.chunks.list && (int64_t)blockIdx.z * LO_ROWS >= a.rows) return;   // a uniform step knows its rows without loading anything
   const int64_t c0 = (int64_t)a.m.heads * a.m.dim + (int64_t)h * dv + n0;
   stage_matrix(sB, ldb, reinterpret_cast<const bf16*>(a.ukv) + c0, a.ld_ukv, r, min(LO_N, dv - n0), kp, LO_N, c0 % 8 == 0);
   pdl_wait();
@@ -677,17 +734,20 @@ __global__ void __launch_bounds__(256) latent_out_kernel(LatentAttnArgs a) {
         src[u] = row < ch.y && c < r ? a.olat + ((int64_t)(ch.x + row) * a.m.heads + h) * ns * r + c : nullptr;
         v[u] = make_float4(0.f, 0.f, 0.f, 0.f);
       }
-      for (int s = 0; s < ns; ++s)
+#pragma unroll 2
+      for (int s = 0; s < ns; ++s) {
+        float4 x[U];
 #pragma unroll
-        for (int u = 0; u < U; ++u)
-          if (src[u]) {
-            const float4 x = *reinterpret_cast<const float4*>(src[u] + (int64_t)s * r);
-            const float f = sw[min((i0 + u * 256) / hp, LO_ROWS - 1)][s];
-            v[u].x = fmaf(f, x.x, v[u].x);
-            v[u].y = fmaf(f, x.y, v[u].y);
-            v[u].z = fmaf(f, x.z, v[u].z);
-            v[u].w = fmaf(f, x.w, v[u].w);
-          }
+        for (int u = 0; u < U; ++u) x[u] = src[u] ? *reinterpret_cast<const float4*>(src[u] + (int64_t)s * r) : make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+        for (int u = 0; u < U; ++u) {
+          const float f = sw[min((i0 + u * 256) / hp, LO_ROWS - 1)][s];
+          v[u].x = fmaf(f, x[u].x, v[u].x);
+          v[u].y = fmaf(f, x[u].y, v[u].y);
+          v[u].z = fmaf(f, x[u].z, v[u].z);
+          v[u].w = fmaf(f, x[u].w, v[u].w);
+        }
+      }
 #pragma unroll
       for (int u = 0; u < U; ++u) {
         const int i = i0 + u * 256;
@@ -758,10 +818,11 @@ int latent_post_launch(Ctx* c, const LatentPostArgs& a, int64_t rows) {
   if (rows == 0) return REWB200_OK;
   const size_t smem = (size_t)a.ld * sizeof(float);
   RB_REQUIRE(a.ld % 4 == 0 && smem <= 48 * 1024, "latent attention: the input projection is wider than 12288 columns");
+  const unsigned threads = rows > 256 ? 256 : (unsigned)std::min<int64_t>(768, std::max<int64_t>(64, (a.ld / 4 + 31) / 32 * 32));
   if (a.dtype == REWB200_BF16)
-    RB_CUDA(launch_k(latent_post_kernel<bf16>, dim3((unsigned)rows), dim3(256), smem, c->stream, c->use_pdl, a));
+    RB_CUDA(launch_k(latent_post_kernel<bf16>, dim3((unsigned)rows), dim3(threads), smem, c->stream, c->use_pdl, a));
   else
-    RB_CUDA(launch_k(latent_post_kernel<float>, dim3((unsigned)rows), dim3(256), smem, c->stream, c->use_pdl, a));
+    RB_CUDA(launch_k(latent_post_kernel<float>, dim3((unsigned)rows), dim3(threads), smem, c->stream, c->use_pdl, a));
   ++g_launch_total;
   return REWB200_OK;
 }
@@ -792,7 +853,7 @@ int latent_kv_splits(Ctx* c, const LatentDims& m, int64_t tiles, int64_t max_ctx
   const int64_t pages = (ctx + PAGE_TOKENS - 1) / PAGE_TOKENS + 1;
   const int64_t hg = (m.heads + 31) / 32;
   const int64_t want = c->sm_count / std::max<int64_t>(1, tiles * hg);
-  return (int)std::max<int64_t>(1, std::min<int64_t>(std::min<int64_t>(want, pages / 2), 16));
+  return (int)std::max<int64_t>(1, std::min<int64_t>(std::min<int64_t>(want, pages), 16));
 }
 
 int latent_attn_absorbed_launch(Ctx* c, const LatentAttnArgs& a) {
@@ -825,7 +886,7 @@ int latent_attn_absorbed_launch(Ctx* c, const LatentAttnArgs& a) {
   const dim3 ga((unsigned)a.kv_splits, (unsigned)(a.tiles.count * cf.subtiles), (unsigned)((a.m.heads + cf.heads_per - 1) / cf.heads_per));
   if (mt == 1) RB_CUDA(launch_k(latent_attn_kernel<1>, ga, dim3(288), smem, c->stream, c->use_pdl, *a.tm_cache, a, cf));
   else RB_CUDA(launch_k(latent_attn_kernel<2>, ga, dim3(288), smem, c->stream, c->use_pdl, *a.tm_cache, a, cf));
-  const dim3 go((unsigned)((a.m.vdim + LO_N - 1) / LO_N), (unsigned)a.m.heads, (unsigned)(a.chunks.count * LO_PARTS));
+  const dim3 go((unsigned)((a.m.vdim + LO_N - 1) / LO_N), (unsigned)a.m.heads, (unsigned)(a.chunks.list ? (int64_t)a.chunks.count * LO_PARTS : (a.rows + LO_ROWS - 1) / LO_ROWS));
   RB_CUDA(launch_k(latent_out_kernel, go, dim3(256), o_smem, c->stream, c->use_pdl, a));
   g_launch_total += 3;
   return REWB200_OK;
