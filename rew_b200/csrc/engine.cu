@@ -434,7 +434,8 @@ bool ep_uses_peer_heap(const rewb200_model* m, int64_t rows) {
          a2a_need(rows * cf.top_k * cf.ep_size, cf.d_model, dtype_size(cf.dtype), nullptr, nullptr) <= pi->a2a_bytes;
 }
 
-int moe_routed(rewb200_session* s, MoeDev& X, const void* x, int64_t d, int64_t rows, bool accumulate, float* out, int moe_index) {
+int moe_routed(rewb200_session* s, MoeDev& X, const void* x, int64_t d, int64_t rows, bool accumulate, float* out, int moe_index,
+               bool first_plain) {
   rewb200_model* m = s->m;
   Ctx* c = m->c;
   const rewb200_config& cf = m->cfg;
@@ -446,13 +447,17 @@ int moe_routed(rewb200_session* s, MoeDev& X, const void* x, int64_t d, int64_t 
   const bool peer = ep_uses_peer_heap(m, rows);
   int* const clear = peer ? s->moe_ints : nullptr;
   bool cleared = false;
+  const bool pdl = c->use_pdl;
+  if (first_plain) c->use_pdl = false;  // the router Linear follows an event wait: a plain dependency
   if (dt == REWB200_BF16 && rows <= 64) {
     // the router has one feature tile: split K over several CTAs, the routing kernel sums the slabs
     const int nkb = (int)((d + 63) / 64);
     int ks = 1;
     while (ks < 8 && nkb / (ks * 2) >= 4) ks *= 2;
-    RB_TRY(linear_bf16_launch(c, X.router.plan, (const bf16*)x, d, rows, EPI_PARTIAL_F32, ks, s->moe_logits, ldr,
-                              nullptr, nullptr, 0));
+    const int st = linear_bf16_launch(c, X.router.plan, (const bf16*)x, d, rows, EPI_PARTIAL_F32, ks, s->moe_logits, ldr,
+                                      nullptr, nullptr, 0);
+    c->use_pdl = pdl;
+    RB_TRY(st);
     RB_TRY(moe_route_slabs_launch(c, s->moe_logits, ks, rows * ldr, X.router.b, rows, X.E, ldr, k, X.renorm, s->moe_topw,
                                   s->moe_topi, clear, peer ? ep : 0));
     cleared = peer;
@@ -462,6 +467,7 @@ int moe_routed(rewb200_session* s, MoeDev& X, const void* x, int64_t d, int64_t 
                                 X.router.b, nullptr, 0));
     else
       RB_TRY(gemm_f32_launch(c, (const float*)x, (const float*)X.router.w, X.router.b, s->moe_logits, rows, d, ldr));
+    c->use_pdl = pdl;
     RB_TRY(moe_route_slabs_launch(c, s->moe_logits, 1, 0, nullptr, rows, X.E, ldr, k, X.renorm, s->moe_topw, s->moe_topi, nullptr, 0));
   }
   if (s->route_rec) {

@@ -300,7 +300,7 @@ int swiglu_rows_f32_launch(Ctx* c, const float* gu, float* out, int64_t rows, in
 // Routed experts of one MoE layer for the normalised rows x [rows][d]: router, top-k, expert Linears, weighted sum
 // into `out` (nullptr: slab 0 of s->part).
 int moe_routed(rewb200_session* s, MoeDev& X, const void* x, int64_t d, int64_t rows, bool accumulate, float* out = nullptr,
-               int moe_index = 0);
+               int moe_index = 0, bool first_plain = false);
 
 // ---- blocks.cu: layered models
 int layered_create(rewb200_model* m, const rewb200_layer* layers, const rewb200_stack* stack);

@@ -40,6 +40,8 @@ __device__ __forceinline__ float2 rotate(float2 v, float2 cs) {
 
 __device__ __forceinline__ void add4(float4& v, const float4 w) { v.x += w.x; v.y += w.y; v.z += w.z; v.w += w.w; }
 
+__device__ __forceinline__ void prefetch_l2(const void* p) { asm volatile("prefetch.global.L2 [%0];" ::"l"(p)); }
+
 // Sums of two values over the block; every thread gets both.
 __device__ __forceinline__ float2 block_sum2(float2 v, float2* red) {
 #pragma unroll
@@ -63,13 +65,19 @@ __global__ void __launch_bounds__(768) latent_post_kernel(LatentPostArgs a) {
   extern __shared__ __align__(16) float sx[];
   __shared__ float2 red[32];
   pdl_launch_dependents();
-  pdl_wait();
   const int64_t row = blockIdx.x;
   const int nt = blockDim.x;
   const int nq = a.m.q_rank, nc = a.m.kv_rank, nr = a.m.rot_dim, n = nq + nc + nr + (a.m.gate ? a.m.heads : 0);
+  // the norm weights depend on no earlier kernel; in a captured decode step neither do the position and its table row
+  if (threadIdx.x * 32 < nq) prefetch_l2(a.q_norm + threadIdx.x * 32);
+  if (threadIdx.x * 32 < nc) prefetch_l2(a.kv_norm + threadIdx.x * 32);
+  if (!a.early) pdl_wait();
   const int lane = row_lane(a.map, row), pos = row_pos(a.map, row);
   const bool ok = pos >= 0 && pos < a.capacity && pos < a.m.max_pos;
-  const int page = a.block_table[(int64_t)lane * a.max_pages + (ok ? pos / PAGE_TOKENS : 0)];
+  if (a.early) {
+    if (ok && a.m.rope_dims > 0 && threadIdx.x * 32 < a.m.rope_dims) prefetch_l2(a.m.rope + (int64_t)pos * (a.m.rope_dims / 2) + threadIdx.x * 16);
+    pdl_wait();
+  }
   const float* p = a.partial + row * a.ld;
   float2 sq = make_float2(0.f, 0.f);
   for (int i = threadIdx.x * 4; i < n; i += nt * 4) {   // rows are padded to a multiple of 8 columns
@@ -91,6 +99,7 @@ __global__ void __launch_bounds__(768) latent_post_kernel(LatentPostArgs a) {
       else if (i + u < nq + nc) sq.y += e[u] * e[u];
     }
   }
+  const int page = a.block_table[(int64_t)lane * a.max_pages + (ok ? pos / PAGE_TOKENS : 0)];
   sq = block_sum2(sq, red);
   const float rq = sqrtf(sq.x / (float)nq + a.eps), rc = sqrtf(sq.y / (float)nc + a.eps);
   if (!ok && threadIdx.x == 0) atomicExch(a.status, KS_BAD_INDEX);
@@ -853,7 +862,7 @@ int latent_kv_splits(Ctx* c, const LatentDims& m, int64_t tiles, int64_t max_ctx
   const int64_t pages = (ctx + PAGE_TOKENS - 1) / PAGE_TOKENS + 1;
   const int64_t hg = (m.heads + 31) / 32;
   const int64_t want = c->sm_count / std::max<int64_t>(1, tiles * hg);
-  return (int)std::max<int64_t>(1, std::min<int64_t>(std::min<int64_t>(want, pages), 16));
+  return (int)std::max<int64_t>(1, std::min<int64_t>(std::min<int64_t>(want, pages), 8));
 }
 
 int latent_attn_absorbed_launch(Ctx* c, const LatentAttnArgs& a) {

@@ -59,6 +59,7 @@ struct LatentPostArgs {
   int max_pages, capacity;
   int64_t ldc;
   int dtype;
+  int early;               // captured decode step: positions predate the step
   int* status;
 };
 int latent_post_launch(Ctx* c, const LatentPostArgs& a, int64_t rows);
