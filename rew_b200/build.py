@@ -3,6 +3,7 @@
 Usage: python -m rew_b200.build [--force]
 """
 import concurrent.futures
+import fcntl
 import os
 import subprocess
 import sys
@@ -43,6 +44,13 @@ def _compile(src, verbose):
 
 
 def build(force=False, verbose=False):
+    """Compiles what is missing or out of date; processes that start together wait for one another."""
+    with open(os.path.join(HERE, ".build.lock"), "w") as lock:
+        fcntl.flock(lock, fcntl.LOCK_EX)
+        return _build(force, verbose)
+
+
+def _build(force, verbose):
     srcs = sources()
     if force:
         for s in srcs:
@@ -54,10 +62,12 @@ def build(force=False, verbose=False):
     objs = [o for o, _ in results]
     log = "".join(l for _, l in results)
     if _stale(OUT, objs):
-        cmd = [NVCC, "-shared", "-o", OUT] + objs + ["-gencode", "arch=compute_100a,code=sm_100a", "-ldl"]
+        part = OUT + ".part"
+        cmd = [NVCC, "-shared", "-o", part] + objs + ["-gencode", "arch=compute_100a,code=sm_100a", "-ldl"]
         r = subprocess.run(cmd, capture_output=True, text=True)
         if r.returncode != 0:
             raise RuntimeError("link failed:\n%s\n%s" % (r.stdout, r.stderr))
+        os.replace(part, OUT)
     return OUT, log
 
 

@@ -59,9 +59,9 @@ __device__ __forceinline__ float2 block_sum2(float2 v, float2* red) {
   return t;
 }
 
-// One CTA per row; small steps have a thread per four columns (up to 768 threads).
-template <typename T>
-__global__ void __launch_bounds__(768) latent_post_kernel(LatentPostArgs a) {
+// One CTA per row; small steps (SMALL) have a thread per four columns, up to 768, and many slabs.
+template <typename T, bool SMALL>
+__global__ void __launch_bounds__(SMALL ? 768 : 128, SMALL ? 1 : 10) latent_post_kernel(LatentPostArgs a) {
   extern __shared__ __align__(16) float sx[];
   __shared__ float2 red[32];
   pdl_launch_dependents();
@@ -69,27 +69,30 @@ __global__ void __launch_bounds__(768) latent_post_kernel(LatentPostArgs a) {
   const int nt = blockDim.x;
   const int nq = a.m.q_rank, nc = a.m.kv_rank, nr = a.m.rot_dim, n = nq + nc + nr + (a.m.gate ? a.m.heads : 0);
   // the norm weights depend on no earlier kernel; in a captured decode step neither do the position and its table row
-  if (threadIdx.x * 32 < nq) prefetch_l2(a.q_norm + threadIdx.x * 32);
-  if (threadIdx.x * 32 < nc) prefetch_l2(a.kv_norm + threadIdx.x * 32);
+  if ((int)threadIdx.x * 32 < nq) prefetch_l2(a.q_norm + threadIdx.x * 32);
+  if ((int)threadIdx.x * 32 < nc) prefetch_l2(a.kv_norm + threadIdx.x * 32);
   if (!a.early) pdl_wait();
   const int lane = row_lane(a.map, row), pos = row_pos(a.map, row);
   const bool ok = pos >= 0 && pos < a.capacity && pos < a.m.max_pos;
   if (a.early) {
-    if (ok && a.m.rope_dims > 0 && threadIdx.x * 32 < a.m.rope_dims) prefetch_l2(a.m.rope + (int64_t)pos * (a.m.rope_dims / 2) + threadIdx.x * 16);
+    if (ok && a.m.rope_dims > 0 && (int)threadIdx.x * 32 < a.m.rope_dims) prefetch_l2(a.m.rope + (int64_t)pos * (a.m.rope_dims / 2) + threadIdx.x * 16);
     pdl_wait();
   }
   const float* p = a.partial + row * a.ld;
   float2 sq = make_float2(0.f, 0.f);
   for (int i = threadIdx.x * 4; i < n; i += nt * 4) {   // rows are padded to a multiple of 8 columns
     float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
-    if (a.nsplit == 1) v = *reinterpret_cast<const float4*>(p + i);
-    else for (int k = 0; k < a.nsplit; k += 8) {
-      float4 w[8];
+    if constexpr (SMALL) {
+      for (int k = 0; k < a.nsplit; k += 8) {
+        float4 w[8];
 #pragma unroll
-      for (int u = 0; u < 8; ++u)
-        w[u] = k + u < a.nsplit ? *reinterpret_cast<const float4*>(p + (k + u) * a.split_stride + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+        for (int u = 0; u < 8; ++u)
+          w[u] = k + u < a.nsplit ? *reinterpret_cast<const float4*>(p + (k + u) * a.split_stride + i) : make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll
-      for (int u = 0; u < 8; ++u) add4(v, w[u]);
+        for (int u = 0; u < 8; ++u) add4(v, w[u]);
+      }
+    } else {
+      for (int k = 0; k < a.nsplit; ++k) add4(v, *reinterpret_cast<const float4*>(p + k * a.split_stride + i));
     }
     *reinterpret_cast<float4*>(sx + i) = v;
     const float e[4] = {v.x, v.y, v.z, v.w};
@@ -101,7 +104,7 @@ __global__ void __launch_bounds__(768) latent_post_kernel(LatentPostArgs a) {
   }
   const int page = a.block_table[(int64_t)lane * a.max_pages + (ok ? pos / PAGE_TOKENS : 0)];
   sq = block_sum2(sq, red);
-  const float rq = sqrtf(sq.x / (float)nq + a.eps), rc = sqrtf(sq.y / (float)nc + a.eps);
+  const float rq = 1.0f / sqrtf(sq.x / (float)nq + a.eps), rc = 1.0f / sqrtf(sq.y / (float)nc + a.eps);
   if (!ok && threadIdx.x == 0) atomicExch(a.status, KS_BAD_INDEX);
   T* cq = reinterpret_cast<T*>(a.cq) + row * a.ldcq;
   T* cr = reinterpret_cast<T*>(a.cache) + ((int64_t)page * PAGE_TOKENS + (ok ? pos % PAGE_TOKENS : 0)) * a.ldc;
@@ -117,15 +120,15 @@ __global__ void __launch_bounds__(768) latent_post_kernel(LatentPostArgs a) {
     d[1] = stf<T>(y);
   };
   for (int i = threadIdx.x * 2; i < nq; i += nt * 2) {
-    if (i + 1 < nq) put(cq + i, a.q_norm[i] * (sx[i] / rq), a.q_norm[i + 1] * (sx[i + 1] / rq));
-    else cq[i] = stf<T>(a.q_norm[i] * (sx[i] / rq));
+    if (i + 1 < nq) put(cq + i, a.q_norm[i] * (sx[i] * rq), a.q_norm[i + 1] * (sx[i + 1] * rq));
+    else cq[i] = stf<T>(a.q_norm[i] * (sx[i] * rq));
   }
   if (a.m.gate)
     for (int i = threadIdx.x; i < a.m.heads; i += nt) a.gate[row * a.m.heads + i] = 1.0f / (1.0f + expf(-sx[nq + nc + nr + i]));
   if (!ok) return;
   for (int i = threadIdx.x * 2; i < nc; i += nt * 2) {
-    if (i + 1 < nc) put(cr + i, a.kv_norm[i] * (sx[nq + i] / rc), a.kv_norm[i + 1] * (sx[nq + i + 1] / rc));
-    else cr[i] = stf<T>(a.kv_norm[i] * (sx[nq + i] / rc));
+    if (i + 1 < nc) put(cr + i, a.kv_norm[i] * (sx[nq + i] * rc), a.kv_norm[i + 1] * (sx[nq + i + 1] * rc));
+    else cr[i] = stf<T>(a.kv_norm[i] * (sx[nq + i] * rc));
   }
   const int half = a.m.rope_dims / 2;
   for (int i = threadIdx.x; i < half; i += nt) {
@@ -827,11 +830,16 @@ int latent_post_launch(Ctx* c, const LatentPostArgs& a, int64_t rows) {
   if (rows == 0) return REWB200_OK;
   const size_t smem = (size_t)a.ld * sizeof(float);
   RB_REQUIRE(a.ld % 4 == 0 && smem <= 48 * 1024, "latent attention: the input projection is wider than 12288 columns");
-  const unsigned threads = rows > 256 ? 256 : (unsigned)std::min<int64_t>(768, std::max<int64_t>(64, (a.ld / 4 + 31) / 32 * 32));
+  const bool small = rows <= 256;
+  const dim3 grid((unsigned)rows), block(small ? (unsigned)std::min<int64_t>(768, std::max<int64_t>(64, (a.ld / 4 + 31) / 32 * 32)) : 128);
+  cudaError_t e;
   if (a.dtype == REWB200_BF16)
-    RB_CUDA(launch_k(latent_post_kernel<bf16>, dim3((unsigned)rows), dim3(threads), smem, c->stream, c->use_pdl, a));
+    e = small ? launch_k(latent_post_kernel<bf16, true>, grid, block, smem, c->stream, c->use_pdl, a)
+              : launch_k(latent_post_kernel<bf16, false>, grid, block, smem, c->stream, c->use_pdl, a);
   else
-    RB_CUDA(launch_k(latent_post_kernel<float>, dim3((unsigned)rows), dim3(threads), smem, c->stream, c->use_pdl, a));
+    e = small ? launch_k(latent_post_kernel<float, true>, grid, block, smem, c->stream, c->use_pdl, a)
+              : launch_k(latent_post_kernel<float, false>, grid, block, smem, c->stream, c->use_pdl, a);
+  RB_CUDA(e);
   ++g_launch_total;
   return REWB200_OK;
 }

@@ -83,3 +83,10 @@ def test_clock_record_counts_only_samples_inside_the_timed_region():
     assert rec["power_w"] == 610.0 and rec["power_limit_w"] == 1000.0
     short = bench.ClockSampler.summarise(text, base + 0.05, base + 0.31, base + 0.33)
     assert short["samples"] == 3 and short["window"].startswith("warm-up + timed region") and short["reasons"] == ["sw_power_cap"]
+
+
+def test_reference_arm_says_why_a_layered_workload_is_unavailable():
+    r = _run("--impl", "reference", "--workload", "rezupel_b32", "--steps", "1", "--warmup", "1")
+    assert r.returncode == 0, r.stderr[-2000:]
+    j = json.loads([l for l in r.stdout.splitlines() if l.startswith("{")][0])
+    assert j["impl"] == "reference" and "latent" in j["unavailable"]

@@ -111,20 +111,25 @@ SIZES = [
     dict(heads=5, dim=13, rot_dim=6, vdim=11, q_rank=19, kv_rank=27, window=30, rope_dims=4),     # nothing divides by 8
     dict(heads=2, dim=192, rot_dim=32, vdim=160, q_rank=64, kv_rank=256, window=129),
     dict(heads=8, dim=32, rot_dim=16, vdim=64, q_rank=64, kv_rank=640, window=100),
+    dict(heads=3, dim=192, rot_dim=64, vdim=128, q_rank=48, kv_rank=72, window=150),     # four score boxes: one query tile a CTA
+    dict(heads=2, dim=136, rot_dim=24, vdim=40, q_rank=32, kv_rank=56, window=300),      # ... two, with one value stage
+    dict(heads=4, dim=128, rot_dim=64, vdim=128, q_rank=80, kv_rank=256, window=130),
 ]
 
 
 @pytest.mark.parametrize("i", range(len(SIZES)))
 def test_other_sizes(rb, dtype, i):
-    width, vocab = [(40, 33), (96, 64), (256, 130), (320, 200), (136, 72), (61, 101), (128, 90), (200, 88)][i]
+    width, vocab = [(40, 33), (96, 64), (256, 130), (320, 200), (136, 72), (61, 101), (128, 90), (200, 88), (112, 70), (96, 50),
+                    (192, 96)][i]
     cfg = K.config([K.layer(K.dense(37), **SIZES[i]), K.layer(K.moe(6, 1, 13), **SIZES[i])], vocab=vocab, width=width, loop=(0, 2, 2))
     t = K.weights(cfg, seed=i, score_gain=2.0)
-    ids = K.tokens(cfg, 150, seed=i)
+    n = 150 if i < 8 else 400
+    ids = K.tokens(cfg, n, seed=i)
     want = R.forward(cfg, t, ids)
-    sess = build(rb, cfg, t, dtype).paged_session(1, 192, 4)
-    close(feed_all(sess, 0, ids, [150]), want, dtype)
+    sess = build(rb, cfg, t, dtype).paged_session(1, 448, 8)
+    close(feed_all(sess, 0, ids, [n]), want, dtype)
     sess.release(0)
-    close(feed_all(sess, 0, ids, [100, 1, 1, 3, 2, 1]), want, dtype)
+    close(feed_all(sess, 0, ids, [100, 1, 1, 3, 2, 80, 1]), want, dtype)
 
 
 # ---------------------------------------------------------------- cuts, batches, pages
