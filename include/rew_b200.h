@@ -286,7 +286,7 @@ typedef struct rewb200_layer {
   int32_t heads, dim, rot_dim, vdim, q_rank, kv_rank;
   int32_t window;       /* keys a query sees, itself included; 0: all before it */
   int32_t rope_dims;    /* rotated features of the rot_dim part, interleaved pairs */
-  int32_t out_gate;     /* 1: head h's output is multiplied by sigmoid(g . input)_h */
+  int32_t out_gate;     /* 1: every head's output is scaled by a sigmoid of its own projection of the input */
   int32_t ff;           /* 0 none, 1 dense gated SiLU, 2 routed experts */
   int32_t ffn;          /* hidden width of the dense feed-forward or of one expert */
   int32_t experts, top_k;
@@ -297,9 +297,10 @@ typedef struct rewb200_layer {
   int32_t reserved;
 } rewb200_layer;
 typedef struct rewb200_stack {
-  int32_t loop_start, loop_stop, loop_times; /* layers loop_start .. loop_stop - 1 run loop_times times (0: no loop);
-                                              * every pass has its own cache.  Before pass t the vector step[t] is added
-                                              * to x, before every pass but the first also the embedding output. */
+  int32_t loop_start, loop_stop, loop_times; /* the half-open range of layers that is repeated, and how often it runs
+                                              * (0: no loop).  Passes share weights and have a cache each; a pass opens by
+                                              * adding its row of `step` and, from the second on, the token embeddings
+                                              * to the residual. */
   int32_t norm_zero_centred;                 /* block and final norm weights are stored as the distance from one */
 } rewb200_stack;
 

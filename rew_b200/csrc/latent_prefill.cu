@@ -80,7 +80,7 @@ __device__ __forceinline__ void softmax_rows(const LatentExpArgs& a, const ExpCf
     xm[half * 128 + row] = mraw;
     pair_barrier(pair_bar);   // both warps hold their scores in registers now; P may overwrite them
     mraw = fmaxf(mraw, xm[(half ^ 1) * 128 + row]);
-    // the scale may be of either sign only in theory: maxima of raw scores need it positive, which the host requires
+    // the maximum of the raw scores is that of the scaled ones: the host requires a positive scale
     const float mx = fmaxf(m, mraw * sl2);
     const float m_use = mx == -INFINITY ? 0.f : mx;
     const float alpha = ex2(m - m_use);
@@ -315,8 +315,8 @@ __global__ void __launch_bounds__(64 + QT * 256, 1) latent_prefill_kernel(const 
           }
         }
         if (!ok) break;
-        // every active tile of this key tile has waited for V; a tile nobody looks at cannot occur (the tiles' key
-        // ranges overlap or touch), but its loads are waited for all the same
+        // the query tiles' key ranges overlap or touch, so some tile has waited for these loads already; if none had,
+        // the buffers must not be released before they have landed
         if (!v_ready) ok = mbar_wait(v_full + st, (j / cf.v_stages) & 1, a.status);
         if (ok && j + 1 < j_end && !k_ready) ok = mbar_wait(k_full, (j + 1) & 1, a.status);
         if (!ok) break;

@@ -47,7 +47,7 @@ class LayeredConfig:
     d_model: int
     layers: list                # LayerSpec
     eps: float = 1e-6
-    loop: tuple = None          # (start, stop, times): layers start .. stop - 1 run `times` times in a row
+    loop: tuple = None          # (start, stop, times): layers[start:stop] are repeated, `times` passes in all
     norm_zero_centred: bool = True   # block and final norm weights are stored as the distance from one
     max_seq: int = 4096
     dtype: int = _lib.F32

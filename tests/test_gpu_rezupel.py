@@ -191,6 +191,19 @@ def test_mixed_batches_against_each_request_alone(rb, dtype):
         close(np.concatenate(got[r]), want[r], dtype)
 
 
+def test_long_prompt_with_many_routed_pairs(rb, dtype):
+    """More (token, expert) pairs than the small-step sort takes, beside a decoding lane."""
+    cfg = K.config([K.layer(K.moe(6, 4, 16), window=90)], loop=(0, 1, 2))
+    t = K.weights(cfg, seed=17)
+    a, b = K.tokens(cfg, 700, seed=17), K.tokens(cfg, 30, seed=18)
+    wa, wb = R.forward(cfg, t, a), R.forward(cfg, t, b)
+    sess = build(rb, cfg, t, dtype).paged_session(2, 704, 13)
+    close(sess.feed([(1, b[:29])], want=range(29))[0], wb[:29], dtype)
+    lg, _ = sess.feed([(0, a[:640]), (1, b[29:])], want=range(641))
+    close(lg, np.concatenate([wa[:640], wb[29:]]), dtype)
+    close(sess.feed([(0, a[640:])], want=range(60))[0], wa[640:], dtype)
+
+
 def test_freed_pages_hold_nothing_over(rb):
     """A request on pages and a lane that others used gives the same bits as on a fresh session."""
     cfg = K.small()
