@@ -95,6 +95,12 @@ int rewb200_sync(int slot, int timeout_ms);
  *   "latent_attention" = "auto" | "plain" | "absorbed"   latent attention: keys and values expanded per head for large prompt
  *                                            portions and the cached latents themselves otherwise (default); always the
  *                                            plain kernels; always on the latents
+ *   "gqa_attention" = "auto" | "plain" | "paged"   grouped-query attention of layered models: the tcgen05 kernel for large prompt
+ *                                            portions and the paged kernel otherwise (default); always the plain kernel;
+ *                                            always the paged kernel
+ *   "linear_attention" = "auto" | "plain" | "recurrent"   gated linear attention: in chunks for large prompt portions and token
+ *                                            by token otherwise (default); token by token with the state in global
+ *                                            memory; always token by token
  *   "inject_alloc_fail" = "n"                test hook: the n-th activation-buffer allocation from now fails on the host
  *   "moe_overlap" = "on" | "off"             MoE layers on one rank, steps of at most 64 rows: the shared experts run on a
  *                                            second stream beside the routed experts (default on)
@@ -277,15 +283,24 @@ int rewb200_linear_noalloc(int slot, const void* x_bf16, const void* w_bf16, con
 
 /* ---- layered models ---------------------------------------------------------
  * Decoders whose layers are described one by one (rewb200_model_create_layers): which mixer a layer has and its
- * sizes, its feed-forward, and a range of layers that runs several times.  A layer is the parallel block
- * x += mixer(norm1(x)) + ff(norm2(x)).  `mixer` 1 is latent attention: queries through a latent of q_rank, keys and
- * values from a cached latent of kv_rank, a rotated key part of rot_dim shared by all heads, an optional sigmoid
- * gate per head on the output, a sliding window. */
+ * sizes, its feed-forward, how a block is put together, and a range of layers that runs several times.
+ *
+ * `mixer`
+ *   1  latent attention: queries through a latent of q_rank, keys and values from a cached latent of kv_rank, a
+ *      rotated key part of rot_dim shared by all heads, a sliding window.
+ *   2  grouped-query attention with a learned distance bias: per-head RMS norm of queries and keys (qk_norm), a
+ *      query temperature 1 + temp_coef ln(floor((p + 1) / temp_every) + 1), a bias per head and distance bucket
+ *      added to the scaled score (bias_rows, bias_max), a learned number per head in the softmax denominator (sink).
+ *      kv_from >= 0: the layer has no keys and values of its own and attends to those layer kv_from has cached.
+ *   3  gated linear attention: a state [dim, vdim] per head in f32 for every sequence, decayed per key channel by
+ *      sigmoid(z)^(1 / tau) with z a projection through decay_rank features, RMS norm per head on the output and a
+ *      SiLU gate.
+ * Mixers 1 and 2 have an optional sigmoid gate per head on the output (out_gate). */
 typedef struct rewb200_layer {
-  int32_t mixer;        /* 1: latent attention */
+  int32_t mixer;
   int32_t heads, dim, rot_dim, vdim, q_rank, kv_rank;
-  int32_t window;       /* keys a query sees, itself included; 0: all before it */
-  int32_t rope_dims;    /* rotated features of the rot_dim part, interleaved pairs */
+  int32_t window;       /* mixer 1: keys a query sees, itself included; 0: all before it */
+  int32_t rope_dims;    /* mixer 1: rotated features of the rot_dim part, interleaved pairs */
   int32_t out_gate;     /* 1: every head's output is scaled by a sigmoid of its own projection of the input */
   int32_t ff;           /* 0 none, 1 dense gated SiLU, 2 routed experts */
   int32_t ffn;          /* hidden width of the dense feed-forward or of one expert */
@@ -294,7 +309,18 @@ typedef struct rewb200_layer {
   int32_t expert_gated; /* 1: gated SiLU experts, 0: W_down relu(W_up x)^2 */
   double rope_base;
   float scale;          /* of the attention scores */
-  int32_t reserved;
+  int32_t kv_heads;     /* mixer 2: key/value heads */
+  int32_t kv_from;      /* mixer 2: layer whose keys and values are used; -1: its own */
+  int32_t qk_norm, sink;
+  int32_t bias_rows;    /* mixer 2: rows of the distance bias table (0: no bias): a bucket per distance below
+                         * bias_rows / 2, then logarithmic ones up to bias_max */
+  int32_t bias_max;
+  int32_t temp_every;   /* mixer 2: 0: no query temperature */
+  float temp_coef;
+  int32_t decay_rank;   /* mixer 3 */
+  float tau;
+  int32_t router_bias;  /* 1: the router has a bias per expert */
+  int32_t shared_ffn;   /* hidden width of a gated SiLU expert that runs for every token beside the routed ones; 0: none */
 } rewb200_layer;
 typedef struct rewb200_stack {
   int32_t loop_start, loop_stop, loop_times; /* the half-open range of layers that is repeated, and how often it runs
@@ -302,6 +328,9 @@ typedef struct rewb200_stack {
                                               * adding its row of `step` and, from the second on, the token embeddings
                                               * to the residual. */
   int32_t norm_zero_centred;                 /* block and final norm weights are stored as the distance from one */
+  int32_t block;                             /* 0: x += mixer(norm1(x)) + ff(norm2(x));
+                                              * 1: x += norm1(mixer(x)), then x += norm2(ff(x)) */
+  int32_t own_head;                          /* 1: the output head is a tensor of its own, 0: the embedding table */
 } rewb200_stack;
 
 /* ---- model + generate ------------------------------------------------------
@@ -324,10 +353,12 @@ typedef struct rewb200_config {
 
 int rewb200_model_create(int slot, const rewb200_config* cfg, rewb200_model** out);
 /* A layered model: `cfg` gives vocab, d_model, n_layers, max_seq, eps and dtype (its other fields are ignored),
- * `layers` n_layers descriptions.  The output head is the embedding table.  Canonical tensors (Linear weights
- * [in, out], see rew_b200/layered.py): embed, step [times, d] (with a loop); per layer norm1, dq, dq.norm, uq, dkv,
- * dkv.norm, uk, uv, g (with out_gate), o, then with a feed-forward norm2 and gate, up, down (dense) or router and per
- * expert [gate,] up, down; final norm. */
+ * `layers` n_layers descriptions.  Canonical tensors (Linear weights [in, out], see rew_b200/layered.py): embed,
+ * step [times, d] (with a loop); per layer norm1, the mixer (1: dq, dq.norm, uq, dkv, dkv.norm, uk, uv; 2: q, then
+ * with keys and values of its own k, v, then q.norm and (own) k.norm with qk_norm, rel [bias_rows, heads], sink;
+ * 3: q, k, v, a1, a2, a2.b, g, norm), g (mixers 1 and 2 with out_gate), o, then with a feed-forward norm2 and gate,
+ * up, down (dense) or router, [router.b,] per expert [gate,] up, down and the shared expert's gate, up, down; final
+ * norm; head [d, vocab] (with own_head). */
 int rewb200_model_create_layers(int slot, const rewb200_config* cfg, const rewb200_layer* layers, const rewb200_stack* stack,
                                 rewb200_model** out);
 void rewb200_model_free(rewb200_model* m);

@@ -2,13 +2,14 @@
 // one by one.  They share the engine's sessions, lanes, page pool, captured decode step, sampler and lm_head
 // (engine.cu); this file has what differs per layer.
 //
-// A layer is the parallel block x += mixer(norm1(x)) + ff(norm2(x)).  One launch (residual_norm) adds both branches'
-// f32 slabs to the residual, adds what a loop adds ahead of a pass, and leaves both norms of the next layer run.
-// In small steps the feed-forward branch runs on the slot's second stream beside the mixer.
+// A block is the parallel x += mixer(norm1(x)) + ff(norm2(x)), where one launch (residual_norm) adds both branches' f32
+// slabs to the residual, adds what a loop adds ahead of a pass, and leaves both norms of the next layer run, and in small
+// steps the feed-forward branch runs on the slot's second stream beside the mixer; or x += norm1(mixer(x)), then
+// x += norm2(ff(x)), where one launch (output_norm) per sublayer sums its slabs, norms the sum and adds it.
 //
 // Device layouts beyond engine.cu's: rows and Linear outputs are padded to multiples of 8 elements (zero weights, zero
-// norm weights), so any width can be loaded by TMA; the mixer's four input projections are one matrix; the key and value
-// projections of the latent are one matrix; a loop's passes share weights and have a cache each.
+// norm weights), so any width can be loaded by TMA; a mixer's input projections are one matrix; the key and value
+// projections of a latent are one matrix; a loop's passes share weights and have a cache each.
 #include <cmath>
 #include <map>
 
@@ -22,8 +23,10 @@ int64_t pad8(int64_t v) { return (v + 7) / 8 * 8; }
 
 enum Slot : int {
   SL_NORM1, SL_DQ, SL_DQ_NORM, SL_UQ, SL_DKV, SL_DKV_NORM, SL_UK, SL_UV, SL_G, SL_O, SL_NORM2, SL_GATE, SL_UP, SL_DOWN, SL_ROUTER,
-  SL_E_GATE, SL_E_UP, SL_E_DOWN, SL_EMBED, SL_STEP, SL_FINAL
+  SL_E_GATE, SL_E_UP, SL_E_DOWN, SL_EMBED, SL_STEP, SL_FINAL, SL_HEAD, SL_Q, SL_K, SL_V, SL_Q_NORM, SL_K_NORM, SL_REL, SL_SINK, SL_A1, SL_A2,
+  SL_A2_B, SL_V_GATE, SL_V_NORM, SL_ROUTER_B, SL_S_GATE, SL_S_UP, SL_S_DOWN
 };
+enum Mixer : int { MIX_LATENT = 1, MIX_GQA = 2, MIX_GLA = 3 };
 struct TensorAt {
   Slot slot;
   int layer, expert;
@@ -35,22 +38,39 @@ void tensors_of(const rewb200_model* m, std::vector<TensorAt>* out) {
   if (m->stack.loop_times > 0) out->push_back({SL_STEP, -1, -1});
   for (int l = 0; l < m->cfg.n_layers; ++l) {
     const rewb200_layer& L = m->spec[l];
-    for (Slot s : {SL_NORM1, SL_DQ, SL_DQ_NORM, SL_UQ, SL_DKV, SL_DKV_NORM, SL_UK, SL_UV}) out->push_back({s, l, -1});
+    auto add = [&](std::initializer_list<Slot> slots) {
+      for (Slot s : slots) out->push_back({s, l, -1});
+    };
+    add({SL_NORM1});
+    if (L.mixer == MIX_LATENT) add({SL_DQ, SL_DQ_NORM, SL_UQ, SL_DKV, SL_DKV_NORM, SL_UK, SL_UV});
+    if (L.mixer == MIX_GQA) {
+      const bool own = L.kv_from < 0;
+      add({SL_Q});
+      if (own) add({SL_K, SL_V});
+      if (L.qk_norm) add({SL_Q_NORM});
+      if (L.qk_norm && own) add({SL_K_NORM});
+      if (L.bias_rows > 0) add({SL_REL});
+      if (L.sink) add({SL_SINK});
+    }
+    if (L.mixer == MIX_GLA) add({SL_Q, SL_K, SL_V, SL_A1, SL_A2, SL_A2_B, SL_V_GATE, SL_V_NORM});
     if (L.out_gate) out->push_back({SL_G, l, -1});
     out->push_back({SL_O, l, -1});
     if (L.ff) out->push_back({SL_NORM2, l, -1});
     if (L.ff == 1)
       for (Slot s : {SL_GATE, SL_UP, SL_DOWN}) out->push_back({s, l, -1});
     if (L.ff == 2) {
-      out->push_back({SL_ROUTER, l, -1});
+      add({SL_ROUTER});
+      if (L.router_bias) add({SL_ROUTER_B});
       for (int e = 0; e < L.experts; ++e) {
         if (L.expert_gated) out->push_back({SL_E_GATE, l, e});
         out->push_back({SL_E_UP, l, e});
         out->push_back({SL_E_DOWN, l, e});
       }
+      if (L.shared_ffn > 0) add({SL_S_GATE, SL_S_UP, SL_S_DOWN});
     }
   }
   out->push_back({SL_FINAL, -1, -1});
+  if (m->stack.own_head) out->push_back({SL_HEAD, -1, -1});
 }
 
 int shape_of(const rewb200_model* m, const TensorAt& t, int64_t* rows, int64_t* cols, bool* vec) {
@@ -75,6 +95,21 @@ int shape_of(const rewb200_model* m, const TensorAt& t, int64_t* rows, int64_t* 
     case SL_GATE: case SL_UP: case SL_E_GATE: case SL_E_UP: mat(d, L->ffn); break;
     case SL_DOWN: case SL_E_DOWN: mat(L->ffn, d); break;
     case SL_ROUTER: mat(d, L->experts); break;
+    case SL_ROUTER_B: v(L->experts); break;
+    case SL_S_GATE: case SL_S_UP: mat(d, L->shared_ffn); break;
+    case SL_S_DOWN: mat(L->shared_ffn, d); break;
+    case SL_HEAD: mat(d, m->cfg.vocab); break;
+    case SL_Q: mat(d, (int64_t)L->heads * L->dim); break;
+    case SL_K: mat(d, (int64_t)(L->mixer == MIX_GQA ? L->kv_heads : L->heads) * L->dim); break;
+    case SL_V: mat(d, (int64_t)(L->mixer == MIX_GQA ? L->kv_heads : L->heads) * L->vdim); break;
+    case SL_Q_NORM: case SL_K_NORM: v(L->dim); break;
+    case SL_REL: mat(L->bias_rows, L->heads); break;
+    case SL_SINK: v(L->heads); break;
+    case SL_A1: mat(d, L->decay_rank); break;
+    case SL_A2: mat(L->decay_rank, (int64_t)L->heads * L->dim); break;
+    case SL_A2_B: v((int64_t)L->heads * L->dim); break;
+    case SL_V_GATE: mat(d, (int64_t)L->heads * L->vdim); break;
+    case SL_V_NORM: v(L->vdim); break;
   }
   return REWB200_OK;
 }
@@ -125,6 +160,42 @@ int rope_table(rewb200_model* m, double base, int dims, float2** out) {
   return REWB200_OK;
 }
 
+// Row of a bias table of B rows for a key n tokens back: a row per distance below B / 2, then logarithmic ones up to D.
+// The small allowance keeps distances that lie exactly on a border on its far side.
+int distance_bucket(int n, int B, int D) {
+  const int h = B / 2;
+  if (n < h) return n;
+  if (h == 0 || D <= h) return B - 1;
+  const double v = std::log((double)n / h) / std::log((double)D / h) * (B - h);
+  return (int)std::min<double>(B - 1, h + std::floor(v + 1e-9));
+}
+// Distances a bias table tells apart: 0 .. bias_distances - 1, the last one standing for all longer ones.
+int bias_distances(int B, int D) {
+  int n = 0;
+  while (distance_bucket(n, B, D) < B - 1) ++n;
+  return n + 1;
+}
+
+// Tables of a mixer-2 layer by distance: [heads][n_bias] from the stored [rows][heads].
+int upload_bias(rewb200_model* m, const rewb200_layer& L, GqaDev& G, const float* host) {
+  std::vector<float> t((size_t)L.heads * G.m.n_bias);
+  for (int n = 0; n < G.m.n_bias; ++n) {
+    const int b = distance_bucket(n, L.bias_rows, L.bias_max);
+    for (int h = 0; h < L.heads; ++h) t[(size_t)h * G.m.n_bias + n] = host[(size_t)b * L.heads + h];
+  }
+  RB_CUDA(cudaMemcpyAsync(G.bias, t.data(), t.size() * sizeof(float), cudaMemcpyHostToDevice, m->c->stream));
+  RB_CUDA(cudaStreamSynchronize(m->c->stream));
+  return REWB200_OK;
+}
+
+// The Linear weights of a layer's mixer that are no routed experts (all of them padded matrices of the model dtype).
+std::vector<LinW*> mixer_linears(LayerDev& D) {
+  if (D.mixer == MIX_LATENT) return {&D.a.in, &D.a.uq, &D.a.ukv, &D.o};
+  if (D.mixer == MIX_GQA) return {&D.g.in, &D.o};
+  return {&D.l.in, &D.o};
+}
+bool has_dense(const LayerDev& D) { return D.ffn_local > 0; }
+
 }  // namespace
 
 int layered_create(rewb200_model* m, const rewb200_layer* layers, const rewb200_stack* stack) {
@@ -139,11 +210,27 @@ int layered_create(rewb200_model* m, const rewb200_layer* layers, const rewb200_
   for (int l = 0; l < n; ++l) {
     const rewb200_layer& L = m->spec[l];
     const std::string who = "layer " + std::to_string(l) + ": ";
-    RB_REQUIRE(L.mixer == 1, who + "unknown mixer");
-    RB_REQUIRE(L.heads > 0 && L.dim > 0 && L.rot_dim >= 0 && L.vdim > 0 && L.q_rank > 0 && L.kv_rank > 0, who + "mixer sizes must be positive");
-    RB_REQUIRE(L.rope_dims >= 0 && L.rope_dims % 2 == 0 && L.rope_dims <= L.rot_dim, who + "rotated features must be pairs within rot_dim");
-    RB_REQUIRE(L.window >= 0, who + "the window must not be negative");
+    RB_REQUIRE(L.mixer >= MIX_LATENT && L.mixer <= MIX_GLA, who + "unknown mixer");
+    RB_REQUIRE(L.heads > 0 && L.dim > 0 && L.vdim > 0, who + "mixer sizes must be positive");
+    if (L.mixer == MIX_LATENT) {
+      RB_REQUIRE(L.rot_dim >= 0 && L.q_rank > 0 && L.kv_rank > 0, who + "mixer sizes must be positive");
+      RB_REQUIRE(L.rope_dims >= 0 && L.rope_dims % 2 == 0 && L.rope_dims <= L.rot_dim, who + "rotated features must be pairs within rot_dim");
+      RB_REQUIRE(L.window >= 0, who + "the window must not be negative");
+    } else if (L.mixer == MIX_GQA) {
+      RB_REQUIRE(L.kv_heads > 0 && L.heads % L.kv_heads == 0, who + "heads must be divisible by kv_heads");
+      RB_REQUIRE(L.bias_rows >= 0 && (L.bias_rows == 0 || (L.bias_max > 0 && L.bias_max <= 1 << 20)), who + "the distance bias needs a positive bias_max");
+      RB_REQUIRE(L.temp_every >= 0, who + "temp_every must not be negative");
+      if (L.kv_from >= 0) {
+        RB_REQUIRE(L.kv_from < l, who + "kv_from must name an earlier layer");
+        const rewb200_layer& S = m->spec[L.kv_from];
+        RB_REQUIRE(S.mixer == MIX_GQA && S.kv_from < 0 && S.kv_heads == L.kv_heads && S.dim == L.dim && S.vdim == L.vdim,
+                   who + "kv_from must name an attention layer with keys and values of its own and the same head sizes");
+      }
+    } else {
+      RB_REQUIRE(L.decay_rank > 0 && L.tau > 0.f, who + "decay_rank and tau must be positive");
+    }
     RB_REQUIRE(L.ff >= 0 && L.ff <= 2 && (L.ff == 0 || L.ffn > 0), who + "unknown feed-forward");
+    RB_REQUIRE(L.shared_ffn >= 0 && (L.ff == 2 || L.shared_ffn == 0), who + "a shared expert stands beside routed ones");
     RB_REQUIRE(L.ff != 2 || (L.experts > 0 && L.experts <= 256 && L.top_k > 0 && L.top_k <= L.experts),
                who + "experts must be in 1..256 and top in 1..experts");
   }
@@ -157,24 +244,50 @@ int layered_create(rewb200_model* m, const rewb200_layer* layers, const rewb200_
   for (int l = 0; l < n; ++l) {
     const rewb200_layer& L = m->spec[l];
     LayerDev& D = m->layers[l];
-    LatentDev& A = D.a;
+    D.mixer = L.mixer;
     RB_TRY(zero_weights(m, (void**)&D.ln1g, dp * sizeof(float)));
     if (L.ff) RB_TRY(zero_weights(m, (void**)&D.ln2g, dp * sizeof(float)));
-    A.m = LatentDims{L.heads, L.dim, L.rot_dim, L.vdim, L.q_rank, L.kv_rank, L.rope_dims, L.window, L.out_gate, L.scale, nullptr, m->cfg.max_seq};
-    if (L.rope_dims > 0) {
-      float2*& t = tables[{L.rope_base, L.rope_dims}];
-      if (!t) RB_TRY(rope_table(m, L.rope_base, L.rope_dims, &t));
-      A.m.rope = t;
+    if (L.mixer == MIX_LATENT) {
+      LatentDev& A = D.a;
+      A.m = LatentDims{L.heads, L.dim, L.rot_dim, L.vdim, L.q_rank, L.kv_rank, L.rope_dims, L.window, L.out_gate, L.scale, nullptr, m->cfg.max_seq};
+      if (L.rope_dims > 0) {
+        float2*& t = tables[{L.rope_base, L.rope_dims}];
+        if (!t) RB_TRY(rope_table(m, L.rope_base, L.rope_dims, &t));
+        A.m.rope = t;
+      }
+      RB_TRY(zero_lin(m, &A.in, dp, pad8((int64_t)L.q_rank + L.kv_rank + L.rot_dim + (L.out_gate ? L.heads : 0))));
+      RB_TRY(zero_lin(m, &A.uq, pad8(L.q_rank), pad8((int64_t)L.heads * (L.dim + L.rot_dim))));
+      RB_TRY(zero_lin(m, &A.ukv, L.kv_rank, pad8((int64_t)L.heads * (L.dim + L.vdim))));
+      RB_TRY(zero_weights(m, (void**)&A.q_norm, L.q_rank * sizeof(float)));
+      RB_TRY(zero_weights(m, (void**)&A.kv_norm, L.kv_rank * sizeof(float)));
+      A.ldc = pad8(L.kv_rank + L.rot_dim);
+      widest = std::max(widest, std::max(A.in.N, A.uq.N));
+      q_cols = std::max(q_cols, A.uq.N);
+    } else if (L.mixer == MIX_GQA) {
+      GqaDev& G = D.g;
+      const bool own = L.kv_from < 0;
+      G.ldk = pad8(L.dim);
+      G.ldv = pad8(L.vdim);
+      RB_TRY(zero_lin(m, &G.in, dp, pad8((int64_t)L.heads * L.dim + (own ? (int64_t)L.kv_heads * (L.dim + L.vdim) : 0) + (L.out_gate ? L.heads : 0))));
+      if (L.qk_norm) RB_TRY(zero_weights(m, (void**)&G.q_norm, L.dim * sizeof(float)));
+      if (L.qk_norm && own) RB_TRY(zero_weights(m, (void**)&G.k_norm, L.dim * sizeof(float)));
+      const int nb = L.bias_rows > 0 ? bias_distances(L.bias_rows, L.bias_max) : 0;
+      if (nb > 0) RB_TRY(zero_weights(m, (void**)&G.bias, (size_t)L.heads * nb * sizeof(float)));
+      if (L.sink) RB_TRY(zero_weights(m, (void**)&G.sink, L.heads * sizeof(float)));
+      G.m = GqaDims{L.heads, L.kv_heads, L.dim, L.vdim, own ? 1 : 0, L.out_gate, L.scale, G.q_norm, G.k_norm, L.temp_every, L.temp_coef, G.bias, nb, G.sink};
+      widest = std::max(widest, G.in.N);
+      q_cols = std::max(q_cols, pad8((int64_t)L.heads * L.dim));
+    } else {
+      GlaDev& A = D.l;
+      const int64_t hk = (int64_t)L.heads * L.dim, hv = (int64_t)L.heads * L.vdim;
+      RB_TRY(zero_lin(m, &A.in, dp, pad8(2 * hk + 2 * hv + L.decay_rank)));
+      RB_TRY(zero_weights(m, (void**)&A.a2, hk * L.decay_rank * sizeof(float)));
+      RB_TRY(zero_weights(m, (void**)&A.a2_b, hk * sizeof(float)));
+      RB_TRY(zero_weights(m, (void**)&A.norm, L.vdim * sizeof(float)));
+      A.m = GlaDims{L.heads, L.dim, L.vdim, L.decay_rank, L.tau, A.a2, A.a2_b, A.norm};
+      widest = std::max(widest, A.in.N);
     }
-    RB_TRY(zero_lin(m, &A.in, dp, pad8((int64_t)L.q_rank + L.kv_rank + L.rot_dim + (L.out_gate ? L.heads : 0))));
-    RB_TRY(zero_lin(m, &A.uq, pad8(L.q_rank), pad8((int64_t)L.heads * (L.dim + L.rot_dim))));
-    RB_TRY(zero_lin(m, &A.ukv, L.kv_rank, pad8((int64_t)L.heads * (L.dim + L.vdim))));
-    RB_TRY(zero_weights(m, (void**)&A.q_norm, L.q_rank * sizeof(float)));
-    RB_TRY(zero_weights(m, (void**)&A.kv_norm, L.kv_rank * sizeof(float)));
-    A.ldc = pad8(L.kv_rank + L.rot_dim);
     RB_TRY(zero_lin(m, &D.o, pad8((int64_t)L.heads * L.vdim), dp));
-    widest = std::max(widest, std::max(A.in.N, A.uq.N));
-    q_cols = std::max(q_cols, A.uq.N);
     attn_cols = std::max(attn_cols, D.o.K);
     D.ff = L.ff;
     const int64_t fp = pad8(L.ffn);
@@ -200,6 +313,12 @@ int layered_create(rewb200_model* m, const rewb200_layer* layers, const rewb200_
       m->max_moe_ffn = std::max(m->max_moe_ffn, fp);
       m->max_experts = std::max<int>(m->max_experts, (int)X.router.N);
       m->max_topk = std::max(m->max_topk, X.top_k);
+      if (L.shared_ffn > 0) {
+        D.ffn_local = pad8(L.shared_ffn);
+        m->max_ffn = std::max(m->max_ffn, D.ffn_local);
+        RB_TRY(zero_lin(m, &D.gu, dp, 2 * D.ffn_local));
+        RB_TRY(zero_lin(m, &D.down, D.ffn_local, dp));
+      }
     }
   }
   m->nq = std::max(q_cols, attn_cols);  // sizes the query and attention-output buffers
@@ -208,11 +327,21 @@ int layered_create(rewb200_model* m, const rewb200_layer* layers, const rewb200_
   RB_TRY(zero_lin(m, &m->lm, dp, m->vp));
   const int a = st.loop_times > 0 ? st.loop_start : n, b = st.loop_times > 0 ? st.loop_stop : n;
   for (int l = 0; l < a; ++l) m->runs.push_back({l, false, -1});
+  RB_REQUIRE(st.block == 0 || (st.block == 1 && st.loop_times == 0), "layered model: blocks normed on the way back run without a loop");
+  RB_REQUIRE(st.block == 1 || m->max_topk == 0 || std::none_of(m->spec.begin(), m->spec.end(), [](const rewb200_layer& L) { return L.shared_ffn > 0; }),
+             "layered model: a shared expert needs blocks normed on the way back");
   for (int p = 0; p < st.loop_times; ++p)
     for (int l = a; l < b; ++l) m->runs.push_back({l, l == a && p > 0, l == a ? p : -1});
   for (int l = b; l < n; ++l) m->runs.push_back({l, false, -1});
-  for (const LayerRun& r : m->runs)
-    if (m->layers[r.layer].moe) ++m->n_moe;
+  for (size_t r = 0; r < m->runs.size(); ++r) {
+    LayerRun& R = m->runs[r];
+    if (m->layers[R.layer].moe) ++m->n_moe;
+    R.cache = (int)r;
+    const rewb200_layer& L = m->spec[R.layer];
+    if (L.mixer == MIX_GQA && L.kv_from >= 0)   // the latest run of that layer: in a loop, the one of the same pass
+      for (size_t q = 0; q < r; ++q)
+        if (m->runs[q].layer == L.kv_from) R.cache = (int)q;
+  }
   RB_CUDA(cudaStreamSynchronize(m->c->stream));
   return REWB200_OK;
 }
@@ -257,6 +386,7 @@ int layered_set_tensor(rewb200_model* m, int64_t index, const float* host, int64
   const bool zc = m->stack.norm_zero_centred != 0;
   if (t.slot == SL_EMBED) {
     RB_TRY(cols(m->embed, m->dp, 0));
+    if (m->stack.own_head) return REWB200_OK;
     // the output head is the same table: the lm_head matrix is its transpose
     const int64_t n = R * C;
     if (bf)
@@ -268,13 +398,53 @@ int layered_set_tensor(rewb200_model* m, int64_t index, const float* host, int64
   }
   if (t.slot == SL_STEP) return scatter(m, C, 0, 0, R, C, m->step_vec, false, m->dp, C, C, 0);
   if (t.slot == SL_FINAL) return norm(m->ng, zc);
+  if (t.slot == SL_HEAD) return cols(m->lm.w, m->vp, 0);
   LayerDev& D = m->layers[t.layer];
   const rewb200_layer& L = m->spec[t.layer];
   LatentDev& A = D.a;
   const int64_t fp = pad8(L.ffn);
-  // gate / up columns: bf16 interleaves groups of 8, f32 concatenates
-  const int64_t gran = bf ? 8 : L.ffn, gst = bf ? 16 : L.ffn, uoff = bf ? 8 : fp;
-  auto gate_up = [&](void* w, bool up) { return scatter(m, C, 0, 0, R, C, w, true, 2 * fp, gran, gst, up ? uoff : 0); };
+  // gate / up columns of `f` logical ones: bf16 interleaves groups of 8, f32 concatenates
+  auto gate_up = [&](void* w, bool up, int64_t f) {
+    return scatter(m, C, 0, 0, R, C, w, true, 2 * pad8(f), bf ? 8 : f, bf ? 16 : f, up ? (bf ? 8 : pad8(f)) : 0);
+  };
+  auto vector = [&](float* dst) { return scatter(m, C, 0, 0, 1, R * C, dst, false, R * C, R * C, R * C, 0); };
+  const int64_t hk = (int64_t)L.heads * L.dim, hv = (int64_t)L.heads * L.vdim;
+  if (L.mixer == MIX_GQA) {
+    GqaDev& G = D.g;
+    const int64_t kv = L.kv_from < 0 ? (int64_t)L.kv_heads : 0;
+    switch (t.slot) {
+      case SL_Q: return cols(G.in.w, G.in.N, 0);
+      case SL_K: return cols(G.in.w, G.in.N, hk);
+      case SL_V: return cols(G.in.w, G.in.N, hk + kv * L.dim);
+      case SL_G: return cols(G.in.w, G.in.N, hk + kv * (L.dim + L.vdim));
+      case SL_Q_NORM: return norm(G.q_norm, false);
+      case SL_K_NORM: return norm(G.k_norm, false);
+      case SL_SINK: return vector(G.sink);
+      case SL_REL: return upload_bias(m, L, G, host);
+      default: break;
+    }
+  }
+  if (L.mixer == MIX_GLA) {
+    GlaDev& G = D.l;
+    switch (t.slot) {
+      case SL_Q: return cols(G.in.w, G.in.N, 0);
+      case SL_K: return cols(G.in.w, G.in.N, hk);
+      case SL_V: return cols(G.in.w, G.in.N, 2 * hk);
+      case SL_V_GATE: return cols(G.in.w, G.in.N, 2 * hk + hv);
+      case SL_A1: return cols(G.in.w, G.in.N, 2 * hk + 2 * hv);
+      case SL_A2: {   // stored [rank, heads * dim], used row by row of its transpose
+        std::vector<float> w((size_t)numel);
+        for (int64_t r = 0; r < R; ++r)
+          for (int64_t i = 0; i < C; ++i) w[i * R + r] = host[r * C + i];
+        RB_CUDA(cudaMemcpyAsync(G.a2, w.data(), w.size() * sizeof(float), cudaMemcpyHostToDevice, m->c->stream));
+        RB_CUDA(cudaStreamSynchronize(m->c->stream));
+        return REWB200_OK;
+      }
+      case SL_A2_B: return vector(G.a2_b);
+      case SL_V_NORM: return norm(G.norm, false);
+      default: break;
+    }
+  }
   switch (t.slot) {
     case SL_NORM1: return norm(D.ln1g, zc);
     case SL_NORM2: return norm(D.ln2g, zc);
@@ -287,14 +457,18 @@ int layered_set_tensor(rewb200_model* m, int64_t index, const float* host, int64
     case SL_UK: return cols(A.ukv.w, A.ukv.N, 0);
     case SL_UV: return cols(A.ukv.w, A.ukv.N, (int64_t)L.heads * L.dim);
     case SL_O: return cols(D.o.w, m->dp, 0);
-    case SL_GATE: return gate_up(D.gu.w, false);
-    case SL_UP: return gate_up(D.gu.w, true);
+    case SL_GATE: return gate_up(D.gu.w, false, L.ffn);
+    case SL_UP: return gate_up(D.gu.w, true, L.ffn);
     case SL_DOWN: return cols(D.down.w, m->dp, 0);
     case SL_ROUTER: return cols(D.x.router.w, D.x.router.N, 0);
+    case SL_ROUTER_B: return vector(D.x.router.b);
+    case SL_S_GATE: return gate_up(D.gu.w, false, L.shared_ffn);
+    case SL_S_UP: return gate_up(D.gu.w, true, L.shared_ffn);
+    case SL_S_DOWN: return cols(D.down.w, m->dp, 0);
     case SL_E_DOWN: return cols((char*)D.x.down + (size_t)t.expert * fp * m->dp * es, m->dp, 0);
-    case SL_E_GATE: return gate_up((char*)D.x.gu + (size_t)t.expert * m->dp * 2 * fp * es, false);
+    case SL_E_GATE: return gate_up((char*)D.x.gu + (size_t)t.expert * m->dp * 2 * fp * es, false, L.ffn);
     case SL_E_UP:
-      if (D.x.gated) return gate_up((char*)D.x.gu + (size_t)t.expert * m->dp * 2 * fp * es, true);
+      if (D.x.gated) return gate_up((char*)D.x.gu + (size_t)t.expert * m->dp * 2 * fp * es, true, L.ffn);
       return cols((char*)D.x.gu + (size_t)t.expert * m->dp * fp * es, fp, 0);
     default: return fail("tensor slot not supported");
   }
@@ -313,10 +487,20 @@ int layered_init_random(rewb200_model* m, uint64_t seed, float std) {
   for (LayerDev& D : m->layers) {
     RB_TRY(fill_const_launch(c, D.ln1g, REWB200_F32, m->dp, 1.f));
     if (D.ff) RB_TRY(fill_const_launch(c, D.ln2g, REWB200_F32, m->dp, 1.f));
-    RB_TRY(fill_const_launch(c, D.a.q_norm, REWB200_F32, D.a.m.q_rank, 1.f));
-    RB_TRY(fill_const_launch(c, D.a.kv_norm, REWB200_F32, D.a.m.kv_rank, 1.f));
-    for (LinW* w : {&D.a.in, &D.a.uq, &D.a.ukv, &D.o}) RB_TRY(fill(w->w, w->K * w->N));
-    if (D.ff == 1)
+    if (D.mixer == MIX_LATENT) {
+      RB_TRY(fill_const_launch(c, D.a.q_norm, REWB200_F32, D.a.m.q_rank, 1.f));
+      RB_TRY(fill_const_launch(c, D.a.kv_norm, REWB200_F32, D.a.m.kv_rank, 1.f));
+    } else if (D.mixer == MIX_GQA) {
+      if (D.g.q_norm) RB_TRY(fill_const_launch(c, D.g.q_norm, REWB200_F32, D.g.m.dim, 1.f));
+      if (D.g.k_norm) RB_TRY(fill_const_launch(c, D.g.k_norm, REWB200_F32, D.g.m.dim, 1.f));
+      if (D.g.bias) RB_TRY(fill_normal_launch(c, D.g.bias, REWB200_F32, (int64_t)D.g.m.heads * D.g.m.n_bias, ++k, 1.f));
+    } else {
+      RB_TRY(fill_const_launch(c, D.l.norm, REWB200_F32, D.l.m.vdim, 1.f));
+      RB_TRY(fill_const_launch(c, D.l.a2_b, REWB200_F32, (int64_t)D.l.m.heads * D.l.m.dim, 2.f));
+      RB_TRY(fill_normal_launch(c, D.l.a2, REWB200_F32, (int64_t)D.l.m.heads * D.l.m.dim * D.l.m.rank, ++k, std));
+    }
+    for (LinW* w : mixer_linears(D)) RB_TRY(fill(w->w, w->K * w->N));
+    if (has_dense(D))
       for (LinW* w : {&D.gu, &D.down}) RB_TRY(fill(w->w, w->K * w->N));
     if (D.ff == 2) {
       RB_TRY(fill(D.x.router.w, D.x.router.K * D.x.router.N));
@@ -332,8 +516,8 @@ int layered_plans(rewb200_model* m) {
   if (m->cfg.dtype != REWB200_BF16) return REWB200_OK;
   auto plan = [&](LinW& w) { return linear_bf16_plan(&w.plan, (const bf16*)w.w, w.K, w.N, 0); };
   for (LayerDev& D : m->layers) {
-    for (LinW* w : {&D.a.in, &D.a.uq, &D.a.ukv, &D.o}) RB_TRY(plan(*w));
-    if (D.ff == 1)
+    for (LinW* w : mixer_linears(D)) RB_TRY(plan(*w));
+    if (has_dense(D))
       for (LinW* w : {&D.gu, &D.down}) RB_TRY(plan(*w));
     if (D.ff == 2) {
       RB_TRY(plan(D.x.router));
@@ -349,11 +533,12 @@ int layered_acts(rewb200_session* s, int64_t rows) {
   rewb200_model* m = s->m;
   Ctx* c = m->c;
   const size_t es = dtype_size(m->cfg.dtype);
-  int64_t cq = 0, heads = 0;
+  int64_t cq = 1, heads = 0;
   for (const LayerDev& D : m->layers) {
     cq = std::max(cq, D.a.uq.K);
-    heads = std::max<int64_t>(heads, D.a.m.heads);
+    heads = std::max<int64_t>(heads, std::max(D.a.m.heads, D.g.m.heads));
   }
+  heads = std::max<int64_t>(heads, 1);
   RB_TRY(acts_alloc(c, &s->xn2, (size_t)rows * m->dp * es));
   RB_TRY(acts_alloc(c, &s->cq, (size_t)rows * cq * es));
   RB_TRY(acts_alloc(c, (void**)&s->gate, (size_t)rows * heads * sizeof(float)));
@@ -366,20 +551,36 @@ int layered_acts(rewb200_session* s, int64_t rows) {
   return REWB200_OK;
 }
 
-// One cache of latents per layer run.
+// One cache of latents, of keys and values, or one recurrent state per lane, for every layer run that has its own.
 int layered_session(rewb200_session* s, int64_t n_pages) {
   rewb200_model* m = s->m;
+  const bool bf = m->cfg.dtype == REWB200_BF16;
   const size_t es = dtype_size(m->cfg.dtype);
   const size_t n = m->runs.size();
   s->kc.resize(n, nullptr);
+  s->vc.resize(n, nullptr);
   s->tmK.resize(n);
+  s->tmV.resize(n);
+  s->state.resize(n, nullptr);
+  auto zeroed = [&](void** p, size_t bytes) -> int {
+    RB_CUDA(cudaMalloc(p, bytes));
+    RB_CUDA(cudaMemsetAsync(*p, 0, bytes, m->c->stream));
+    return REWB200_OK;
+  };
+  auto pages = [&](void** p, CUtensorMap* tm, int64_t rows, int64_t ld) -> int {
+    RB_TRY(zeroed(p, (size_t)rows * ld * es));
+    return bf ? make_tmap_2d_bf16(tm, *p, (uint64_t)ld, (uint64_t)rows, (uint64_t)ld * 2, 64, 64) : REWB200_OK;
+  };
   for (size_t r = 0; r < n; ++r) {
-    const int64_t ldc = m->layers[m->runs[r].layer].a.ldc;
-    const size_t bytes = (size_t)n_pages * PAGE * ldc * es;
-    RB_CUDA(cudaMalloc(&s->kc[r], bytes));
-    RB_CUDA(cudaMemsetAsync(s->kc[r], 0, bytes, m->c->stream));
-    if (m->cfg.dtype == REWB200_BF16)
-      RB_TRY(make_tmap_2d_bf16(&s->tmK[r], s->kc[r], (uint64_t)ldc, (uint64_t)n_pages * PAGE, (uint64_t)ldc * 2, 64, 64));
+    const LayerDev& D = m->layers[m->runs[r].layer];
+    if (D.mixer == MIX_LATENT) RB_TRY(pages(&s->kc[r], &s->tmK[r], n_pages * PAGE, D.a.ldc));
+    if (D.mixer == MIX_GQA && D.g.m.own_kv) {
+      RB_TRY(pages(&s->kc[r], &s->tmK[r], n_pages * D.g.m.kv_heads * PAGE, D.g.ldk));
+      RB_TRY(pages(&s->vc[r], &s->tmV[r], n_pages * D.g.m.kv_heads * PAGE, D.g.ldv));
+    }
+    // a state needs no clearing between sequences: a portion that starts at position 0 does not read it
+    if (D.mixer == MIX_GLA)
+      RB_TRY(zeroed((void**)&s->state[r], (size_t)s->B * D.l.m.heads * D.l.m.dim * gla_state_ld(D.l.m.vdim) * sizeof(float)));
   }
   return REWB200_OK;
 }
@@ -388,10 +589,14 @@ namespace {
 
 // Rows of one lane an absorbed-attention tile covers at most.
 constexpr int ABS_TILE_ROWS = 8;
+// Rows of one lane a tile of the paged grouped-query kernel covers at most.
+constexpr int GQA_TILE_ROWS = 16;
 // Portions of at least this many tokens attend to keys and values expanded per head.  Expanding costs a Linear over the
 // portion's keys, its own and its window's; the absorbed form costs (2 kv_rank + rot_dim) / (dim + rot_dim + vdim) times
 // the score and value products of every query, on the slower mma.sync pipe.
 constexpr int EXPAND_MIN_ROWS = 64;
+// Portions of at least this many tokens run grouped-query attention on tcgen05 and gated linear attention in chunks.
+constexpr int LARGE_MIN_ROWS = 64, CHUNK_MIN_ROWS = 32;
 
 template <typename T>
 int regrow(rewb200_session* s, T** p, size_t bytes) {
@@ -417,27 +622,51 @@ int layered_prepare(rewb200_session* s, const FwdOpts& o, int64_t rows) {
   const size_t es = dtype_size(m->cfg.dtype);
   const bool uniform = o.entries == nullptr;
   RB_REQUIRE(!uniform || o.S == 1, "layered step: a step of several tokens per lane needs its portions");
-  // ---- lists of the step: [row lane | row position | absorbed tiles | their chunks | expanded tiles | gathered keys]
+  // ---- lists of the step: [row lane | row position | absorbed tiles | their chunks | expanded tiles | gathered keys |
+  // small and large tiles of grouped-query attention | small and large portions of gated linear attention]
   int64_t abs_rows = rows, n_keys = 0;
   s->plan_host.clear();
   s->plan_abs_tiles = s->plan_chunks = s->plan_exp_tiles = s->plan_keys = 0;
   if (!uniform) {
     std::vector<int>& h = s->plan_host;
-    h.resize(2 * rows);
+    h.assign(2 * rows, 0);
     std::vector<int2> tiles, chunks, keys;
     std::vector<ExpTile> exps;
     abs_rows = 0;
     int64_t reach = 0;  // the widest window of any layer, 0: everything
-    bool exp_ok = m->cfg.dtype == REWB200_BF16 && c->latent_impl == 0;
+    const bool bf = m->cfg.dtype == REWB200_BF16;
+    bool exp_ok = bf && c->latent_impl == 0, gqa_ok = bf && c->gqa_impl == 0, gla_ok = bf && c->gla_impl == 0;
+    bool has_latent = false, has_gqa = false, has_gla = false;
     for (const LayerDev& D : m->layers) {
+      if (D.mixer == MIX_GQA) {
+        has_gqa = true;
+        gqa_ok = gqa_ok && gqa_prefill_ok(D.g.m);
+      }
+      if (D.mixer == MIX_GLA) {
+        has_gla = true;
+        gla_ok = gla_ok && gla_chunk_ok(D.l.m);
+      }
+      if (D.mixer != MIX_LATENT) continue;
+      has_latent = true;
       exp_ok = exp_ok && latent_expanded_ok(D.a.m);
       reach = D.a.m.window == 0 ? INT32_MAX : std::max<int64_t>(reach, D.a.m.window);
     }
+    std::vector<int2> gqa_small;
+    std::vector<GqaTile> gqa_large;
+    std::vector<GlaPortion> gla_small, gla_large;
     for (const StepEntry& e : *o.entries) {
       for (int i = 0; i < e.n; ++i) {
         h[e.row0 + i] = e.lane;
         h[rows + e.row0 + i] = e.pos0 + i;
       }
+      if (has_gqa) {
+        if (gqa_ok && e.n >= LARGE_MIN_ROWS)
+          for (int i = 0; i < e.n; i += 256) gqa_large.push_back({e.row0 + i, std::min(256, e.n - i), e.pos0 + i, e.lane});
+        else
+          for (int i = 0; i < e.n; i += GQA_TILE_ROWS) gqa_small.push_back(make_int2(e.row0 + i, std::min(GQA_TILE_ROWS, e.n - i)));
+      }
+      if (has_gla) (gla_ok && e.n >= CHUNK_MIN_ROWS ? gla_large : gla_small).push_back({e.row0, e.n, e.pos0, e.lane});
+      if (!has_latent) continue;
       if (exp_ok && e.n >= EXPAND_MIN_ROWS) {
         const int key0 = (int)std::max<int64_t>(0, (int64_t)e.pos0 - reach + 1);
         for (int i = 0; i < e.n; i += 256)
@@ -458,6 +687,11 @@ int layered_prepare(rewb200_session* s, const FwdOpts& o, int64_t rows) {
     }
     // long query tiles first: the last ones of a wave are then short
     std::stable_sort(exps.begin(), exps.end(), [](const ExpTile& x, const ExpTile& y) { return x.pos0 + x.n - x.key0 > y.pos0 + y.n - y.key0; });
+    std::stable_sort(gqa_large.begin(), gqa_large.end(), [](const GqaTile& x, const GqaTile& y) { return x.pos0 + x.n > y.pos0 + y.n; });
+    s->plan_gqa_small = (int)gqa_small.size();
+    s->plan_gqa_large = (int)gqa_large.size();
+    s->plan_gla_small = (int)gla_small.size();
+    s->plan_gla_large = (int)gla_large.size();
     s->plan_abs_tiles = (int)tiles.size();
     s->plan_chunks = (int)chunks.size();
     s->plan_exp_tiles = (int)exps.size();
@@ -472,6 +706,10 @@ int layered_prepare(rewb200_session* s, const FwdOpts& o, int64_t rows) {
     append(chunks.data(), chunks.size() * sizeof(int2));
     append(exps.data(), exps.size() * sizeof(ExpTile));
     append(keys.data(), keys.size() * sizeof(int2));
+    append(gqa_small.data(), gqa_small.size() * sizeof(int2));
+    append(gqa_large.data(), gqa_large.size() * sizeof(GqaTile));
+    append(gla_small.data(), gla_small.size() * sizeof(GlaPortion));
+    append(gla_large.data(), gla_large.size() * sizeof(GlaPortion));
     if (h.size() > s->plan_cap) {
       s->plan_cap = 0;
       RB_TRY(regrow(s, &s->plan_dev, h.size() * 2 * sizeof(int)));
@@ -495,12 +733,29 @@ int layered_prepare(rewb200_session* s, const FwdOpts& o, int64_t rows) {
   }
   // ---- scratch of the absorbed path
   int64_t units = 0, stats = 0, qe = 0;
+  int64_t g_units = 0, g_stats = 0;
   for (const LayerDev& D : m->layers) {
+    if (D.mixer == MIX_GQA) {
+      const int sp = gqa_kv_splits(c, D.g.m, uniform ? rows : s->plan_gqa_small, s->max_len);
+      g_stats = std::max<int64_t>(g_stats, (int64_t)D.g.m.heads * sp);
+      g_units = std::max<int64_t>(g_units, (int64_t)D.g.m.heads * sp * D.g.m.vdim);
+    }
+    if (D.mixer != MIX_LATENT) continue;
     const int64_t H = D.a.m.heads;
     const int sp = latent_kv_splits(c, D.a.m, rows, s->max_len);
     units = std::max(units, H * sp * D.a.m.kv_rank);
     stats = std::max(stats, H * sp);
     qe = std::max(qe, H * D.a.ldc);
+  }
+  if (rows * g_units > s->gqa_units) {
+    s->gqa_units = 0;
+    RB_TRY(regrow(s, &s->gqa_part, (size_t)rows * g_units * sizeof(float)));
+    s->gqa_units = rows * g_units;
+  }
+  if (rows * g_stats > s->gqa_stats) {
+    s->gqa_stats = 0;
+    RB_TRY(regrow(s, &s->gqa_ml, (size_t)rows * g_stats * sizeof(float2)));
+    s->gqa_stats = rows * g_stats;
   }
   if (abs_rows * units > s->abs_units) {
     s->abs_units = 0;
@@ -521,6 +776,391 @@ int layered_prepare(rewb200_session* s, const FwdOpts& o, int64_t rows) {
   return REWB200_OK;
 }
 
+namespace {
+
+// The lists of a step on the device (layered_prepare's upload, or none for a captured decode step).
+struct StepLists {
+  bool uniform = true;
+  RowMap map = {};
+  RowTiles abs = {}, chunks = {};
+  const ExpTile* exp_tiles = nullptr;
+  const int2* key_list = nullptr;
+  RowTiles gqa_small = {};
+  const GqaTile* gqa_large = nullptr;
+  const GlaPortion *gla_small = nullptr, *gla_large = nullptr;
+};
+
+StepLists step_lists(const rewb200_session* s, const FwdOpts& o, int64_t rows) {
+  StepLists t;
+  t.uniform = o.entries == nullptr;
+  t.map = {nullptr, nullptr, s->d_pos, o.b0, o.S};
+  t.abs = t.gqa_small = {nullptr, (int)rows, 1, 1};
+  t.chunks = {nullptr, (int)((rows + kChunkRows - 1) / kChunkRows), 1, 1};
+  if (t.uniform) return t;
+  t.map.row_lane = s->plan_dev;
+  t.map.row_pos = s->plan_dev + rows;
+  t.abs.list = reinterpret_cast<const int2*>(s->plan_dev + 2 * rows);
+  t.abs.count = s->plan_abs_tiles;
+  t.chunks.list = t.abs.list + t.abs.count;
+  t.chunks.count = s->plan_chunks;
+  t.exp_tiles = reinterpret_cast<const ExpTile*>(t.chunks.list + t.chunks.count);
+  t.key_list = reinterpret_cast<const int2*>(t.exp_tiles + s->plan_exp_tiles);
+  t.gqa_small.list = t.key_list + s->plan_keys;
+  t.gqa_small.count = s->plan_gqa_small;
+  t.gqa_large = reinterpret_cast<const GqaTile*>(t.gqa_small.list + t.gqa_small.count);
+  t.gla_small = reinterpret_cast<const GlaPortion*>(t.gqa_large + s->plan_gqa_large);
+  t.gla_large = t.gla_small + s->plan_gla_small;
+  return t;
+}
+
+// The mixers read s->xn and leave their output (ahead of the output projection) in s->attn.
+
+int gqa_mixer(rewb200_session* s, const FwdOpts& o, const StepLists& t, size_t r, int64_t rows, bool in_graph) {
+  rewb200_model* m = s->m;
+  Ctx* c = m->c;
+  const int dt = m->cfg.dtype;
+  const LayerRun& R = m->runs[r];
+  LayerDev& D = m->layers[R.layer];
+  GqaDev& G = D.g;
+  const int64_t ldq = pad8((int64_t)G.m.heads * G.m.dim);
+  int ks = 1;
+  RB_TRY(run_linear(s, G.in, s->xn, m->dp, rows, true, 0, s->part, G.in.N, &ks));
+  if (o.trace) RB_TRY(o.trace->mark(TC_QKV));
+  GqaPostArgs pa;
+  memset(&pa, 0, sizeof(pa));
+  pa.m = G.m;
+  pa.partial = s->part;
+  pa.nsplit = ks;
+  pa.split_stride = rows * G.in.N;
+  pa.ld = G.in.N;
+  pa.eps = m->cfg.eps;
+  pa.map = t.map;
+  pa.q = s->q;
+  pa.ldq = ldq;
+  pa.gate = s->gate;
+  pa.kc = s->kc[R.cache];
+  pa.vc = s->vc[R.cache];
+  pa.ldk = G.ldk;
+  pa.ldv = G.ldv;
+  pa.block_table = s->block_table;
+  pa.max_pages = s->max_pages;
+  pa.capacity = s->max_len;
+  pa.dtype = dt;
+  pa.early = in_graph ? 1 : 0;
+  pa.status = c->d_status;
+  RB_TRY(gqa_post_launch(c, pa, rows));
+  if (o.trace) RB_TRY(o.trace->mark(TC_QKV_POST));
+  GqaAttnArgs aa;
+  memset(&aa, 0, sizeof(aa));
+  aa.m = G.m;
+  aa.map = t.map;
+  aa.tiles = t.gqa_small;
+  aa.max_tile_rows = t.uniform ? 1 : GQA_TILE_ROWS;
+  aa.q = s->q;
+  aa.ldq = ldq;
+  aa.gate = s->gate;
+  aa.out = s->attn;
+  aa.ldo = D.o.K;
+  aa.kc = pa.kc;
+  aa.vc = pa.vc;
+  if (dt == REWB200_BF16) {
+    aa.tm_k = &s->tmK[R.cache];
+    aa.tm_v = &s->tmV[R.cache];
+  }
+  aa.ldk = G.ldk;
+  aa.ldv = G.ldv;
+  aa.block_table = s->block_table;
+  aa.max_pages = s->max_pages;
+  aa.dtype = dt;
+  aa.o_part = s->gqa_part;
+  aa.ml = s->gqa_ml;
+  aa.kv_splits = gqa_kv_splits(c, G.m, aa.tiles.count, s->max_len);
+  aa.rows = rows;
+  aa.early_kv = in_graph ? 1 : 0;
+  aa.status = c->d_status;
+  RB_TRY(gqa_attn_launch(c, aa));
+  if (!t.uniform && s->plan_gqa_large > 0) {
+    GqaPrefillArgs fa;
+    memset(&fa, 0, sizeof(fa));
+    fa.m = G.m;
+    fa.tiles = t.gqa_large;
+    fa.count = s->plan_gqa_large;
+    fa.q = (const bf16*)s->q;
+    fa.ldq = ldq;
+    fa.gate = s->gate;
+    fa.out = (bf16*)s->attn;
+    fa.ldo = D.o.K;
+    fa.tm_k = aa.tm_k;
+    fa.tm_v = aa.tm_v;
+    fa.block_table = s->block_table;
+    fa.max_pages = s->max_pages;
+    fa.status = c->d_status;
+    RB_TRY(gqa_prefill_launch(c, fa));
+  }
+  if (o.trace) RB_TRY(o.trace->mark(TC_ATTN));
+  return REWB200_OK;
+}
+
+int gla_mixer(rewb200_session* s, const FwdOpts& o, const StepLists& t, size_t r, int64_t rows, bool in_graph) {
+  rewb200_model* m = s->m;
+  Ctx* c = m->c;
+  LayerDev& D = m->layers[m->runs[r].layer];
+  GlaDev& A = D.l;
+  int ks = 1;
+  RB_TRY(run_linear(s, A.in, s->xn, m->dp, rows, true, 0, s->part, A.in.N, &ks));
+  if (o.trace) RB_TRY(o.trace->mark(TC_QKV));
+  GlaArgs ga;
+  memset(&ga, 0, sizeof(ga));
+  ga.m = A.m;
+  ga.list = t.gla_small;
+  ga.count = t.uniform ? (int)rows : s->plan_gla_small;
+  ga.pos0 = s->d_pos;
+  ga.b0 = o.b0;
+  ga.partial = s->part;
+  ga.nsplit = ks;
+  ga.split_stride = rows * A.in.N;
+  ga.ld = A.in.N;
+  ga.eps = m->cfg.eps;
+  ga.state = s->state[r];
+  ga.ldv = (int)gla_state_ld(A.m.vdim);
+  ga.out = s->attn;
+  ga.ldo = D.o.K;
+  ga.dtype = m->cfg.dtype;
+  ga.early = in_graph ? 1 : 0;
+  ga.status = c->d_status;
+  RB_TRY(gla_recurrent_launch(c, ga));
+  if (!t.uniform && s->plan_gla_large > 0) {
+    ga.list = t.gla_large;
+    ga.count = s->plan_gla_large;
+    RB_TRY(gla_chunk_launch(c, ga));
+  }
+  if (o.trace) RB_TRY(o.trace->mark(TC_ATTN));
+  return REWB200_OK;
+}
+
+int latent_mixer(rewb200_session* s, const FwdOpts& o, const StepLists& t, size_t r, int64_t rows, bool in_graph) {
+  rewb200_model* m = s->m;
+  Ctx* c = m->c;
+  const int dt = m->cfg.dtype;
+  LayerDev& D = m->layers[m->runs[r].layer];
+  LatentDev& A = D.a;
+  const bool expand = !t.uniform && s->plan_exp_tiles > 0;
+  int ks = 1;
+  RB_TRY(run_linear(s, A.in, s->xn, m->dp, rows, true, 0, s->part, A.in.N, &ks));
+  if (o.trace) RB_TRY(o.trace->mark(TC_QKV));
+  LatentPostArgs pa;
+  memset(&pa, 0, sizeof(pa));
+  pa.m = A.m;
+  pa.partial = s->part;
+  pa.nsplit = ks;
+  pa.split_stride = rows * A.in.N;
+  pa.ld = A.in.N;
+  pa.q_norm = A.q_norm;
+  pa.kv_norm = A.kv_norm;
+  pa.eps = m->cfg.eps;
+  pa.map = t.map;
+  pa.cq = s->cq;
+  pa.ldcq = A.uq.K;
+  pa.gate = s->gate;
+  pa.cache = s->kc[r];
+  pa.block_table = s->block_table;
+  pa.max_pages = s->max_pages;
+  pa.capacity = s->max_len;
+  pa.ldc = A.ldc;
+  pa.dtype = dt;
+  pa.early = in_graph ? 1 : 0;
+  pa.status = c->d_status;
+  RB_TRY(latent_post_launch(c, pa, rows));
+  LatentAttnArgs aa;
+  memset(&aa, 0, sizeof(aa));
+  aa.m = A.m;
+  aa.map = t.map;
+  aa.tiles = t.abs;
+  aa.chunks = t.chunks;
+  aa.max_tile_rows = t.uniform ? 1 : ABS_TILE_ROWS;
+  aa.rows = rows;
+  if (expand) {
+    RB_TRY(run_linear(s, A.uq, s->cq, A.uq.K, rows, false, EPI_BIAS_BF16, s->q, A.uq.N, nullptr));
+    aa.q = s->q;
+    aa.nsplit = 0;
+  } else {
+    RB_TRY(run_linear(s, A.uq, s->cq, A.uq.K, rows, true, 0, s->part, A.uq.N, &ks));
+    aa.q = s->part;
+    aa.nsplit = ks;
+  }
+  aa.split_stride = rows * A.uq.N;
+  aa.ldq = A.uq.N;
+  aa.ukv = A.ukv.w;
+  aa.ld_ukv = A.ukv.N;
+  aa.qeff = s->qeff;
+  aa.olat = s->olat;
+  aa.ml = s->ml;
+  aa.kv_splits = latent_kv_splits(c, A.m, rows, s->max_len);
+  aa.gate = s->gate;
+  aa.out = s->attn;
+  aa.ldo = D.o.K;
+  aa.cache = s->kc[r];
+  aa.tm_cache = dt == REWB200_BF16 ? &s->tmK[r] : nullptr;
+  aa.block_table = s->block_table;
+  aa.max_pages = s->max_pages;
+  aa.ldc = A.ldc;
+  aa.dtype = dt;
+  aa.early_kv = in_graph ? 1 : 0;
+  aa.status = c->d_status;
+  if (o.trace) RB_TRY(o.trace->mark(TC_QKV_POST));
+  RB_TRY(latent_attn_absorbed_launch(c, aa));
+  if (expand) {
+    LatentExpArgs ea;
+    memset(&ea, 0, sizeof(ea));
+    ea.m = A.m;
+    ea.tiles = t.exp_tiles;
+    ea.count = s->plan_exp_tiles;
+    ea.q = (const bf16*)s->q;
+    ea.ldq = A.uq.N;
+    ea.gate = s->gate;
+    ea.out = (bf16*)s->attn;
+    ea.ldo = D.o.K;
+    ea.kv = (const bf16*)s->kvx;
+    ea.ldkv = A.ukv.N;
+    ea.lat = (const bf16*)s->latx;
+    ea.ldc = A.ldc;
+    ea.keys = s->plan_keys;
+    ea.status = c->d_status;
+    RB_TRY(latent_gather_launch(c, (const bf16*)s->kc[r], s->block_table, s->max_pages, A.ldc, t.key_list, (bf16*)s->latx, s->plan_keys));
+    RB_TRY(linear_bf16_launch(c, A.ukv.plan, (const bf16*)s->latx, A.ldc, s->plan_keys, EPI_BIAS_BF16, 1, s->kvx, A.ukv.N, nullptr, nullptr, 0));
+    RB_TRY(latent_attn_expanded_launch(c, ea));
+  }
+  if (o.trace) RB_TRY(o.trace->mark(TC_ATTN));
+  return REWB200_OK;
+}
+
+int mixer(rewb200_session* s, const FwdOpts& o, const StepLists& t, size_t r, int64_t rows, bool in_graph) {
+  switch (s->m->layers[s->m->runs[r].layer].mixer) {
+    case MIX_GQA: return gqa_mixer(s, o, t, r, rows, in_graph);
+    case MIX_GLA: return gla_mixer(s, o, t, r, rows, in_graph);
+    default: return latent_mixer(s, o, t, r, rows, in_graph);
+  }
+}
+
+// A gated SiLU feed-forward (dense, or the shared expert beside routed ones): f32 slabs of the result in `out`.
+int dense_ff(rewb200_session* s, const FwdOpts& o, LayerDev& D, const void* x, int64_t rows, float* out, int* ks) {
+  rewb200_model* m = s->m;
+  const int64_t dp = m->dp;
+  if (m->cfg.dtype == REWB200_BF16) {
+    RB_TRY(run_linear(s, D.gu, x, dp, rows, false, EPI_SWIGLU_BF16, s->h, D.ffn_local, nullptr));
+  } else {
+    RB_TRY(run_linear(s, D.gu, x, dp, rows, false, EPI_BIAS_F32, s->gu32, 2 * D.ffn_local, nullptr));
+    RB_TRY(swiglu_rows_f32_launch(m->c, s->gu32, (float*)s->h, rows, D.ffn_local));
+  }
+  if (o.trace) RB_TRY(o.trace->mark(TC_GATE_UP));
+  RB_TRY(run_linear(s, D.down, s->h, D.ffn_local, rows, true, 0, out, dp, ks));
+  if (o.trace) RB_TRY(o.trace->mark(TC_DOWN));
+  return REWB200_OK;
+}
+
+// Runs `body` on the slot's second stream, after everything enqueued so far; the caller waits for c->ev_join.
+template <typename F>
+int on_side_stream(Ctx* c, F&& body) {
+  RB_CUDA(cudaEventRecord(c->ev_fork, c->stream));
+  RB_CUDA(cudaStreamWaitEvent(c->side, c->ev_fork, 0));
+  cudaStream_t main_stream = c->stream;
+  c->stream = c->side;
+  const int st = body();
+  c->stream = main_stream;
+  RB_TRY(st);
+  RB_CUDA(cudaEventRecord(c->ev_join, c->side));
+  return REWB200_OK;
+}
+
+// Blocks normed on the way back: x += norm1(mixer(x)), x += norm2(ff(x)).
+int output_norm_blocks(rewb200_session* s, const FwdOpts& o, const NormArgs& na, int64_t rows, bool in_graph) {
+  rewb200_model* m = s->m;
+  Ctx* c = m->c;
+  const int dt = m->cfg.dtype;
+  const int64_t dp = m->dp;
+  const StepLists t = step_lists(s, o, rows);
+  OutputNormArgs base;
+  memset(&base, 0, sizeof(base));
+  base.x_res = s->x_res;
+  base.split_stride = rows * dp;
+  base.eps = m->cfg.eps;
+  base.d = dp;
+  base.d_mean = na.d_mean;
+  base.out = s->xn;
+  base.dtype = dt;
+  base.status = c->d_status;
+  if (o.trace) RB_TRY(o.trace->begin(c->stream));
+  {
+    OutputNormArgs a = base;
+    a.embed = na.embed;
+    a.ids = na.ids;
+    a.vocab = na.vocab;
+    RB_TRY(output_norm_launch(c, a, rows));
+    if (o.trace) RB_TRY(o.trace->mark(TC_EMBED));
+  }
+  int moe_seen = 0;
+  for (size_t r = 0; r < m->runs.size(); ++r) {
+    LayerDev& D = m->layers[m->runs[r].layer];
+    const bool last = r + 1 == m->runs.size();
+    int ks_o = 1;
+    RB_TRY(mixer(s, o, t, r, rows, in_graph));
+    RB_TRY(run_linear(s, D.o, s->attn, D.o.K, rows, true, 0, s->part, dp, &ks_o));
+    if (o.trace) RB_TRY(o.trace->mark(TC_O));
+    {
+      OutputNormArgs a = base;
+      a.partial = s->part;
+      a.nsplit = ks_o;
+      a.gamma = D.ln1g;
+      if (last && !D.ff) a.final_gamma = m->ng;
+      RB_TRY(output_norm_launch(c, a, rows));
+      if (o.trace) RB_TRY(o.trace->mark(TC_NORM_ATTN));
+    }
+    if (D.ff) {
+      // slabs of a dense feed-forward or shared expert in part, the sum of the routed experts in part2
+      OutputNormArgs a = base;
+      const bool fork = D.ff == 2 && has_dense(D) && dt == REWB200_BF16 && rows <= 64 && c->moe_overlap && !o.trace;
+      const bool pdl = c->use_pdl;
+      auto dense = [&]() -> int { return dense_ff(s, o, D, s->xn, rows, s->part, &a.nsplit); };
+      if (has_dense(D)) {
+        a.partial = s->part;
+        if (fork) {
+          RB_TRY(on_side_stream(c, [&]() -> int {
+            c->use_pdl = false;   // follows an event wait: plain launches
+            const int st = dense();
+            c->use_pdl = pdl;
+            return st;
+          }));
+        } else {
+          RB_TRY(dense());
+        }
+      }
+      if (D.ff == 2) {
+        RB_TRY(moe_routed(s, D.x, s->xn, dp, rows, false, s->part2, moe_seen++, false));
+        a.partial2 = s->part2;
+        a.nsplit2 = 1;
+        if (o.trace) RB_TRY(o.trace->mark(TC_MOE));
+      }
+      if (fork) {
+        RB_CUDA(cudaStreamWaitEvent(c->stream, c->ev_join, 0));
+        c->use_pdl = false;       // two predecessors: a plain dependency
+      }
+      a.gamma = D.ln2g;
+      if (last) a.final_gamma = m->ng;
+      const int st = output_norm_launch(c, a, rows);
+      c->use_pdl = pdl;
+      RB_TRY(st);
+      if (o.trace) RB_TRY(o.trace->mark(TC_NORM_FFN));
+    }
+    if (s->layer_rec && !t.uniform) {
+      RB_CUDA(cudaMemcpyAsync(s->layer_rec + r * s->rows_cap * dp, s->x_res, (size_t)rows * dp * sizeof(float), cudaMemcpyDeviceToDevice, c->stream));
+      s->layer_rows = rows;
+    }
+  }
+  return REWB200_OK;
+}
+
+}  // namespace
+
 // The layer runs of a layered model over `rows` rows; na carries the residual, the embedding and the ids.  Leaves the
 // final norm's output in s->xn.
 int layered_blocks(rewb200_session* s, const FwdOpts& o, const NormArgs& na, int64_t rows, bool in_graph) {
@@ -528,22 +1168,8 @@ int layered_blocks(rewb200_session* s, const FwdOpts& o, const NormArgs& na, int
   Ctx* c = m->c;
   const int dt = m->cfg.dtype;
   const int64_t dp = m->dp;
-  const bool uniform = o.entries == nullptr;
-  RowMap map = {nullptr, nullptr, s->d_pos, o.b0, o.S};
-  RowTiles abs = {nullptr, (int)rows, 1, 1}, chunks = {nullptr, (int)((rows + kChunkRows - 1) / kChunkRows), 1, 1};
-  const ExpTile* exp_tiles = nullptr;
-  const int2* key_list = nullptr;
-  const bool expand = !uniform && s->plan_exp_tiles > 0;
-  if (!uniform) {
-    map.row_lane = s->plan_dev;
-    map.row_pos = s->plan_dev + rows;
-    abs.list = reinterpret_cast<const int2*>(s->plan_dev + 2 * rows);
-    abs.count = s->plan_abs_tiles;
-    chunks.list = abs.list + abs.count;
-    chunks.count = s->plan_chunks;
-    exp_tiles = reinterpret_cast<const ExpTile*>(chunks.list + chunks.count);
-    key_list = reinterpret_cast<const int2*>(exp_tiles + s->plan_exp_tiles);
-  }
+  if (m->stack.block == 1) return output_norm_blocks(s, o, na, rows, in_graph);
+  const StepLists t = step_lists(s, o, rows);
   auto ahead_of = [&](size_t r, NormArgs& a) {  // what the norm launch in front of run r adds and writes
     if (r == m->runs.size()) {
       a.gamma = m->ng;
@@ -572,8 +1198,7 @@ int layered_blocks(rewb200_session* s, const FwdOpts& o, const NormArgs& na, int
   int moe_seen = 0;
   for (size_t r = 0; r < m->runs.size(); ++r) {
     LayerDev& D = m->layers[m->runs[r].layer];
-    LatentDev& A = D.a;
-    int ks = 1, ks_o = 1, ks_f = 0;
+    int ks_o = 1, ks_f = 0;
     const bool fork = D.ff != 0 && dt == REWB200_BF16 && rows <= 64 && c->moe_overlap && !o.trace;
     // ---- feed-forward branch: slabs in part2
     auto ff_branch = [&]() -> int {
@@ -591,122 +1216,17 @@ int layered_blocks(rewb200_session* s, const FwdOpts& o, const NormArgs& na, int
         // mixer's short kernels then wait for (measured, 8B shape: 3.69 instead of 3.53 ms per step at batch 32)
         const bool pdl = c->use_pdl;
         if (fork) c->use_pdl = false;
-        auto dense = [&]() -> int {
-          if (dt == REWB200_BF16) {
-            RB_TRY(run_linear(s, D.gu, s->xn2, dp, rows, false, EPI_SWIGLU_BF16, s->h, D.ffn_local, nullptr));
-          } else {
-            RB_TRY(run_linear(s, D.gu, s->xn2, dp, rows, false, EPI_BIAS_F32, s->gu32, 2 * D.ffn_local, nullptr));
-            RB_TRY(swiglu_rows_f32_launch(c, s->gu32, (float*)s->h, rows, D.ffn_local));
-          }
-          if (o.trace) RB_TRY(o.trace->mark(TC_GATE_UP));
-          return run_linear(s, D.down, s->h, D.ffn_local, rows, true, 0, s->part2, dp, &ks_f);
-        };
-        const int st = dense();
+        const int st = dense_ff(s, o, D, s->xn2, rows, s->part2, &ks_f);
         c->use_pdl = pdl;
-        RB_TRY(st);
-        if (o.trace) RB_TRY(o.trace->mark(TC_DOWN));
-        return REWB200_OK;
+        return st;
       };
       const int st = body();
       s->part = keep;
       return st;
     };
-    if (fork) {
-      RB_CUDA(cudaEventRecord(c->ev_fork, c->stream));
-      RB_CUDA(cudaStreamWaitEvent(c->side, c->ev_fork, 0));
-      cudaStream_t main_stream = c->stream;
-      c->stream = c->side;
-      const int st = ff_branch();
-      c->stream = main_stream;
-      RB_TRY(st);
-      RB_CUDA(cudaEventRecord(c->ev_join, c->side));
-    }
+    if (fork) RB_TRY(on_side_stream(c, ff_branch));
     // ---- mixer
-    RB_TRY(run_linear(s, A.in, s->xn, dp, rows, true, 0, s->part, A.in.N, &ks));
-    if (o.trace) RB_TRY(o.trace->mark(TC_QKV));
-    LatentPostArgs pa;
-    memset(&pa, 0, sizeof(pa));
-    pa.m = A.m;
-    pa.partial = s->part;
-    pa.nsplit = ks;
-    pa.split_stride = rows * A.in.N;
-    pa.ld = A.in.N;
-    pa.q_norm = A.q_norm;
-    pa.kv_norm = A.kv_norm;
-    pa.eps = m->cfg.eps;
-    pa.map = map;
-    pa.cq = s->cq;
-    pa.ldcq = A.uq.K;
-    pa.gate = s->gate;
-    pa.cache = s->kc[r];
-    pa.block_table = s->block_table;
-    pa.max_pages = s->max_pages;
-    pa.capacity = s->max_len;
-    pa.ldc = A.ldc;
-    pa.dtype = dt;
-    pa.early = in_graph ? 1 : 0;
-    pa.status = c->d_status;
-    RB_TRY(latent_post_launch(c, pa, rows));
-    LatentAttnArgs aa;
-    memset(&aa, 0, sizeof(aa));
-    aa.m = A.m;
-    aa.map = map;
-    aa.tiles = abs;
-    aa.chunks = chunks;
-    aa.max_tile_rows = uniform ? 1 : ABS_TILE_ROWS;
-    aa.rows = rows;
-    if (expand) {
-      RB_TRY(run_linear(s, A.uq, s->cq, A.uq.K, rows, false, EPI_BIAS_BF16, s->q, A.uq.N, nullptr));
-      aa.q = s->q;
-      aa.nsplit = 0;
-    } else {
-      RB_TRY(run_linear(s, A.uq, s->cq, A.uq.K, rows, true, 0, s->part, A.uq.N, &ks));
-      aa.q = s->part;
-      aa.nsplit = ks;
-    }
-    aa.split_stride = rows * A.uq.N;
-    aa.ldq = A.uq.N;
-    aa.ukv = A.ukv.w;
-    aa.ld_ukv = A.ukv.N;
-    aa.qeff = s->qeff;
-    aa.olat = s->olat;
-    aa.ml = s->ml;
-    aa.kv_splits = latent_kv_splits(c, A.m, rows, s->max_len);
-    aa.gate = s->gate;
-    aa.out = s->attn;
-    aa.ldo = D.o.K;
-    aa.cache = s->kc[r];
-    aa.tm_cache = dt == REWB200_BF16 ? &s->tmK[r] : nullptr;
-    aa.block_table = s->block_table;
-    aa.max_pages = s->max_pages;
-    aa.ldc = A.ldc;
-    aa.dtype = dt;
-    aa.early_kv = in_graph ? 1 : 0;
-    aa.status = c->d_status;
-    if (o.trace) RB_TRY(o.trace->mark(TC_QKV_POST));
-    RB_TRY(latent_attn_absorbed_launch(c, aa));
-    if (expand) {
-      LatentExpArgs ea;
-      memset(&ea, 0, sizeof(ea));
-      ea.m = A.m;
-      ea.tiles = exp_tiles;
-      ea.count = s->plan_exp_tiles;
-      ea.q = (const bf16*)s->q;
-      ea.ldq = A.uq.N;
-      ea.gate = s->gate;
-      ea.out = (bf16*)s->attn;
-      ea.ldo = D.o.K;
-      ea.kv = (const bf16*)s->kvx;
-      ea.ldkv = A.ukv.N;
-      ea.lat = (const bf16*)s->latx;
-      ea.ldc = A.ldc;
-      ea.keys = s->plan_keys;
-      ea.status = c->d_status;
-      RB_TRY(latent_gather_launch(c, (const bf16*)s->kc[r], s->block_table, s->max_pages, A.ldc, key_list, (bf16*)s->latx, s->plan_keys));
-      RB_TRY(linear_bf16_launch(c, A.ukv.plan, (const bf16*)s->latx, A.ldc, s->plan_keys, EPI_BIAS_BF16, 1, s->kvx, A.ukv.N, nullptr, nullptr, 0));
-      RB_TRY(latent_attn_expanded_launch(c, ea));
-    }
-    if (o.trace) RB_TRY(o.trace->mark(TC_ATTN));
+    RB_TRY(mixer(s, o, t, r, rows, in_graph));
     RB_TRY(run_linear(s, D.o, s->attn, D.o.K, rows, true, 0, s->part, dp, &ks_o));
     if (o.trace) RB_TRY(o.trace->mark(TC_O));
     if (!fork) RB_TRY(ff_branch());
@@ -725,7 +1245,7 @@ int layered_blocks(rewb200_session* s, const FwdOpts& o, const NormArgs& na, int
     if (a.add_embed) a.embed = m->embed;
     const bool pdl = c->use_pdl;
     if (fork) c->use_pdl = false;  // two predecessors: a plain dependency
-    if (s->layer_rec && !uniform) {
+    if (s->layer_rec && !t.uniform) {
       // the residual as the layer leaves it, ahead of what a loop adds
       NormArgs b = a;
       b.norm_kind = -1;

@@ -76,6 +76,8 @@ struct Ctx {
   bool record_routing = false;  // sessions keep every MoE layer's top-k expert ids of their last forward (a test aid)
   bool record_layers = false;   // layered models keep the residual stream after every layer run (a test aid)
   int latent_impl = 0;          // latent attention: 0 by step size, 1 plain kernels, 2 always on the cached latents
+  int gqa_impl = 0;             // layered grouped-query attention: 0 by step size, 1 plain kernels, 2 never the large-portion kernel
+  int gla_impl = 0;             // gated linear attention: 0 by step size, 1 plain kernels, 2 always token by token
   int inject_alloc_fail = 0;  // test hook: the n-th activation allocation from now fails on the host
   int option_epoch = 0;      // bumped by rewb200_set_option; captured graphs from older epochs are rebuilt
   void* pinned = nullptr;    // pinned host staging for H2D/D2H of buffers
@@ -277,6 +279,29 @@ struct NormArgs {
   int64_t d_mean;         // width the row statistics divide by when rows are padded (0: d); the padding is zero
 };
 int residual_norm_launch(Ctx* c, const NormArgs& a, int64_t rows);
+
+// Blocks whose sublayers read the residual itself and are normed on the way back: x += gamma * y / rms(y), y the sum of two
+// sets of f32 slabs.  Leaves x (or, with final_gamma, its RMS norm) in `out`.  Without slabs the row is only written out;
+// with an embedding table it starts from the row of its id.
+struct OutputNormArgs {
+  float* x_res;            // [rows][d]
+  const void* embed;       // [vocab][d] act dtype or nullptr
+  const int* ids;
+  int vocab;
+  const float* partial;    // [nsplit][rows][d]
+  int nsplit;
+  const float* partial2;
+  int nsplit2;
+  int64_t split_stride;
+  const float* gamma;
+  const float* final_gamma;
+  float eps;
+  int64_t d, d_mean;       // d_mean: width the statistics divide by when rows are padded with zeros (0: d)
+  void* out;
+  int dtype;
+  int* status;
+};
+int output_norm_launch(Ctx* c, const OutputNormArgs& a, int64_t rows);
 
 struct KvLayout {
   void* k;                // [n_pages][kvh][page][hd]

@@ -447,6 +447,88 @@ __global__ void __launch_bounds__(NORMV_THREADS) residual_norm_vec_kernel(NormAr
   }
 }
 
+// Sublayers normed on the way back (OutputNormArgs): x += gamma * y / rms(y), y the sum of the slabs.  CL CTAs of a
+// cluster share a row (decode-size steps), their sums of squares meet through distributed shared memory.
+template <typename T, int CL, int NCH>
+__global__ void __launch_bounds__(CL == 1 ? 512 : 256) output_norm_kernel(OutputNormArgs a) {
+  constexpr int THREADS = CL == 1 ? 512 : 256;
+  __shared__ float red[33];
+  __shared__ float part[2];
+  pdl_launch_dependents();
+  const int64_t row = blockIdx.x / CL, d = a.d, dq = d / CL, col0 = (int64_t)(blockIdx.x % CL) * dq;
+  pdl_wait();
+  float* xr = a.x_res + row * d + col0;
+  const T* erow = nullptr;
+  if (a.embed) {
+    int64_t id = a.ids[row];
+    if (id < 0 || id >= a.vocab) {
+      if (threadIdx.x == 0) atomicExch(a.status, KS_BAD_INDEX);
+      id = 0;
+    }
+    erow = reinterpret_cast<const T*>(a.embed) + id * d + col0;
+  }
+  // sum of squares over the row
+  auto row_sum = [&](float v, int slot) -> float {
+    v = block_sum(v, red);
+    if constexpr (CL > 1) {
+      cg::cluster_group cl = cg::this_cluster();
+      if (threadIdx.x == 0) part[slot] = v;
+      cl.sync();
+      v = 0.f;
+#pragma unroll
+      for (int r = 0; r < CL; ++r) v += cl.map_shared_rank(part, r)[slot];
+    }
+    return v;
+  };
+  const float dm = (float)(a.d_mean > 0 ? a.d_mean : d);
+  float4 x[NCH], y[NCH];
+  float ss = 0.f;
+#pragma unroll
+  for (int c = 0; c < NCH; ++c) {
+    const int64_t i = ((int64_t)c * THREADS + threadIdx.x) * 4;
+    x[c] = y[c] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (i >= dq) continue;
+    x[c] = erow ? Vec4<T>::load(erow + i) : *reinterpret_cast<const float4*>(xr + i);
+    const int64_t at = row * d + col0 + i;
+#pragma unroll 8
+    for (int s = 0; s < a.nsplit; ++s) add4(y[c], *reinterpret_cast<const float4*>(a.partial + s * a.split_stride + at));
+#pragma unroll 4
+    for (int s = 0; s < a.nsplit2; ++s) add4(y[c], *reinterpret_cast<const float4*>(a.partial2 + s * a.split_stride + at));
+    ss += y[c].x * y[c].x + y[c].y * y[c].y + y[c].z * y[c].z + y[c].w * y[c].w;
+  }
+  if (a.nsplit + a.nsplit2 > 0) {
+    const float f = 1.0f / sqrtf(row_sum(ss, 0) / dm + a.eps);
+#pragma unroll
+    for (int c = 0; c < NCH; ++c) {
+      const int64_t i = ((int64_t)c * THREADS + threadIdx.x) * 4;
+      if (i >= dq) continue;
+      const float4 g = *reinterpret_cast<const float4*>(a.gamma + col0 + i);
+      add4(x[c], make_float4(g.x * (y[c].x * f), g.y * (y[c].y * f), g.z * (y[c].z * f), g.w * (y[c].w * f)));
+    }
+  }
+  float f2 = 1.0f;
+  if (a.final_gamma) {
+    ss = 0.f;
+#pragma unroll
+    for (int c = 0; c < NCH; ++c) ss += x[c].x * x[c].x + x[c].y * x[c].y + x[c].z * x[c].z + x[c].w * x[c].w;
+    f2 = 1.0f / sqrtf(row_sum(ss, 1) / dm + a.eps);
+  }
+  T* orow = reinterpret_cast<T*>(a.out) + row * d + col0;
+#pragma unroll
+  for (int c = 0; c < NCH; ++c) {
+    const int64_t i = ((int64_t)c * THREADS + threadIdx.x) * 4;
+    if (i >= dq) continue;
+    *reinterpret_cast<float4*>(xr + i) = x[c];
+    float4 o = x[c];
+    if (a.final_gamma) {
+      const float4 g = *reinterpret_cast<const float4*>(a.final_gamma + col0 + i);
+      o = make_float4(g.x * (o.x * f2), g.y * (o.y * f2), g.z * (o.z * f2), g.w * (o.w * f2));
+    }
+    Vec4<T>::store(orow + i, o);
+  }
+  if constexpr (CL > 1) cg::this_cluster().sync();   // a peer may still read this CTA's partial sums
+}
+
 // Decode-size variant: a cluster of four CTAs per row, each on a quarter of the columns; the row
 // statistics meet through distributed shared memory.  With 32 rows the one-CTA-per-row kernel keeps 32
 // SMs busy reading 8 slabs of 16 KB each; this one spreads the same reads over 128 SMs.
@@ -1026,6 +1108,28 @@ __global__ void fill_const_kernel(T* dst, int64_t n, float v) {
 }
 
 }  // namespace
+
+int output_norm_launch(Ctx* c, const OutputNormArgs& a, int64_t rows) {
+  if (rows == 0) return REWB200_OK;
+  RB_REQUIRE(a.d % 8 == 0 && a.d <= 16384, "output norm: rows of a multiple of 8 elements, at most 16384");
+  const bool bf = a.dtype == REWB200_BF16, cluster = rows <= 64 && a.d % 16 == 0 && c->norm_cluster;
+  auto go = [&](auto kernel, int cl) -> int {
+    const dim3 g((unsigned)(rows * cl)), b(cl == 1 ? 512 : 256);
+    RB_CUDA(cl == 1 ? launch_k(kernel, g, b, 0, c->stream, c->use_pdl, a) : launch_k_cluster(kernel, g, b, 0, c->stream, c->use_pdl, dim3(4), a));
+    ++g_launch_total;
+    return REWB200_OK;
+  };
+#define RB_ONORM(T, CL)                                                                                         \
+  (nch <= 1 ? go(output_norm_kernel<T, CL, 1>, CL) : nch <= 2 ? go(output_norm_kernel<T, CL, 2>, CL)            \
+   : nch <= 4 ? go(output_norm_kernel<T, CL, 4>, CL) : go(output_norm_kernel<T, CL, 8>, CL))
+  if (cluster) {
+    const int nch = (int)((a.d / 16 + 255) / 256);
+    return bf ? RB_ONORM(bf16, 4) : RB_ONORM(float, 4);
+  }
+  const int nch = (int)((a.d / 4 + 511) / 512);
+  return bf ? RB_ONORM(bf16, 1) : RB_ONORM(float, 1);
+#undef RB_ONORM
+}
 
 int residual_norm_launch(Ctx* c, const NormArgs& a, int64_t rows) {
   if (rows == 0) return REWB200_OK;

@@ -5,6 +5,8 @@
 #include <cstring>
 
 #include "common.cuh"
+#include "gla.cuh"
+#include "gqa.cuh"
 #include "latent.cuh"
 #include "ptx.cuh"
 
@@ -77,12 +79,27 @@ struct MoeDev {
 
 // Latent attention of one layer (latent.cuh).
 struct LatentDev {
-  LatentDims m;
+  LatentDims m = {};
   LinW in;                     // [d, q_rank | kv_rank | rot_dim | heads]: query latent, key/value latent, shared key part, gate
   LinW uq;                     // [q_rank, heads * (dim + rot_dim)]
   LinW ukv;                    // [kv_rank, heads * dim | heads * vdim]
   float *q_norm = nullptr, *kv_norm = nullptr;
   int64_t ldc = 0;             // elements of a cache row: kv_rank + rot_dim, padded
+};
+
+// Grouped-query attention of one layer of a layered model (gqa.cuh).
+struct GqaDev {
+  GqaDims m = {};
+  LinW in;                     // [d, heads * dim | kv_heads * dim | kv_heads * vdim | heads]: queries, keys, values, gate
+  float *q_norm = nullptr, *k_norm = nullptr, *bias = nullptr, *sink = nullptr;
+  int64_t ldk = 0, ldv = 0;    // elements of a cached key / value row, padded
+};
+
+// Gated linear attention of one layer (gla.cuh).
+struct GlaDev {
+  GlaDims m = {};
+  LinW in;                     // [d, heads * dim | heads * dim | heads * vdim | heads * vdim | rank]: q, k, v, gate, decay features
+  float *a2 = nullptr, *a2_b = nullptr, *norm = nullptr;
 };
 
 struct LayerDev {
@@ -91,7 +108,10 @@ struct LayerDev {
   int64_t ffn_local = 0;
   bool moe = false;
   MoeDev x;
-  LatentDev a;                 // layered models
+  int mixer = 0;               // layered models: rewb200_layer::mixer, and what it has
+  LatentDev a;
+  GqaDev g;
+  GlaDev l;
   int ff = 0;                  // layered models: rewb200_layer::ff
 };
 
@@ -100,6 +120,7 @@ struct LayerRun {
   int layer = 0;
   bool add_embed = false;      // the embedding output is added to the residual ahead of this run
   int step = -1;               // row of the model's step vectors added ahead of this run
+  int cache = -1;              // run whose cache this one reads (its own unless the layer shares another's keys and values)
 };
 
 }  // namespace rewb
@@ -141,6 +162,7 @@ struct rewb200_session {
   int B = 0, max_len = 0, max_pages = 0;
   std::vector<void*> kc, vc;           // per layer
   std::vector<CUtensorMap> tmK, tmV;   // per layer (bf16)
+  std::vector<float*> state;           // layered models: recurrent state per layer run [B][heads][dim][ldv] f32, or nullptr
   int* block_table = nullptr;
   int *d_pos = nullptr, *d_ids = nullptr, *d_next = nullptr, *d_out = nullptr, *d_step = nullptr;
   int out_capacity = 0;
@@ -180,6 +202,9 @@ struct rewb200_session {
   float* olat = nullptr;
   float2* ml = nullptr;
   int64_t abs_units = 0, abs_stats = 0, abs_rows = 0; // capacity of olat, ml and qeff
+  float* gqa_part = nullptr;           // partial outputs of split attention and their row statistics
+  float2* gqa_ml = nullptr;
+  int64_t gqa_units = 0, gqa_stats = 0;
   void *kvx = nullptr, *latx = nullptr;  // keys / values expanded per head, and the gathered cache rows they come from
   int64_t kvx_rows = 0;
   float* layer_rec = nullptr;          // option record_layers: [runs][rows_cap][d]
@@ -191,6 +216,7 @@ struct rewb200_session {
   size_t plan_cap = 0;
   std::vector<int> plan_host;
   int plan_abs_tiles = 0, plan_chunks = 0, plan_exp_tiles = 0, plan_keys = 0;
+  int plan_gqa_small = 0, plan_gqa_large = 0, plan_gla_small = 0, plan_gla_large = 0;
   int* feed_dev = nullptr;             // ids and row lists of a rewb200_lanes_feed step
   size_t feed_cap = 0;
   int64_t route_rows = 0;              // rows of the forward recorded last

@@ -1,0 +1,441 @@
+// Gated linear attention of large prompt portions, in chunks of 32 tokens on the tensor cores.
+//
+// With b_t the running sum of the log decays of a key channel and r its value in the middle of the chunk,
+//   q~_t = q_t e^(b_t - r)      k~_s = k_s e^(r - b_s)      A_ts = q~_t . k~_s  (s <= t)
+//   o_t  = q~_t (e^r S) + sum_s A_ts v_s                    S <- e^(b_end - r) (e^r S + sum_s k~_s v_s^T)
+// so one pair of scaled operands serves the scores, the output and the state.  A CTA walks the chunks of one portion
+// with the state of one head (or of a slice of its value columns; a cluster shares the head) in registers: warp w holds
+// the transposed state [16 value rows][dim], whose accumulator fragments are also the A operand of q~ S.  Products are
+// bf16 with operands split in two (high part and remainder) where they carry the decays, the state or the scores, and
+// f32 sums; decays, their sums and the state itself are f32.
+//
+// The two halves of a chunk bound the exponents: if a channel decays by more than 2^MAX_DECAY in one of them, the
+// chunk runs token by token on the same registers.
+#include <cooperative_groups.h>
+#include <math.h>
+
+#include <algorithm>
+
+#include "gla.cuh"
+#include "ptx.cuh"
+
+namespace cg = cooperative_groups;
+
+namespace rewb {
+
+extern int64_t g_launch_total;
+
+namespace {
+
+constexpr int C = 32;             // tokens of a chunk
+constexpr int NT = 256;
+constexpr float MAX_DECAY = 50.f;
+constexpr float LOG2E = 1.4426950408889634f;
+
+__device__ __forceinline__ float ex2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+__device__ __forceinline__ void ldmatrix_x2(uint32_t& r0, uint32_t& r1, uint32_t addr) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x2.shared.b16 {%0,%1}, [%2];" : "=r"(r0), "=r"(r1) : "r"(addr));
+}
+// x = hi + lo, both bf16
+__device__ __forceinline__ void split(float x, bf16& hi, bf16& lo) {
+  hi = __float2bfloat16_rn(x);
+  lo = __float2bfloat16_rn(x - __bfloat162float(hi));
+}
+__device__ __forceinline__ void split2(float x, float y, uint32_t& hi, uint32_t& lo) {
+  hi = pack_bf16(x, y);
+  const __nv_bfloat162 h = *reinterpret_cast<const __nv_bfloat162*>(&hi);
+  lo = pack_bf16(x - __low2float(h), y - __high2float(h));
+}
+__device__ __forceinline__ float slab(const GlaArgs& a, const float* p) {
+  float v = *p;
+  for (int s = 1; s < a.nsplit; ++s) v += p[s * a.split_stride];
+  return v;
+}
+__device__ __forceinline__ float4 slab4(const GlaArgs& a, const float* p) {
+  float4 v = *reinterpret_cast<const float4*>(p);
+  for (int s = 1; s < a.nsplit; ++s) {
+    const float4 w = *reinterpret_cast<const float4*>(p + s * a.split_stride);
+    v.x += w.x; v.y += w.y; v.z += w.z; v.w += w.w;
+  }
+  return v;
+}
+
+struct ChunkCfg {
+  int kt;        // 16-channel steps of a key: dim padded to 16 kt
+  int vs;        // value columns of the CTA, a multiple of 16
+  int rp;        // decay features padded to a multiple of 4
+  int ldq;       // elements of a row of the q~ / k~ buffers
+  int off_k, off_v, off_a, off_a1, off_a2, off_f, off_ss;   // byte offsets in shared memory (q~ and the staged output at 0)
+};
+
+// KT: capacity of the register state in 16-channel steps.
+template <int KT, bool CLUSTER>
+__global__ void __launch_bounds__(NT, 2) gla_chunk_kernel(GlaArgs a, ChunkCfg cf) {
+  extern __shared__ __align__(16) uint8_t smem[];
+  const GlaDims& m = a.m;
+  const int K = m.dim, V = m.vdim, Kp = cf.kt * 16, vs = cf.vs, rp = cf.rp, ldq = cf.ldq, ldv = vs + 8, ldO = vs + 4;
+  bf16* sQ = reinterpret_cast<bf16*>(smem);                    // [hi, lo][C][ldq]
+  float* sO = reinterpret_cast<float*>(smem);                  // [C][ldO], once q~ has been read
+  bf16* sK = reinterpret_cast<bf16*>(smem + cf.off_k);         // [hi, lo][C][ldq]
+  bf16* sV = reinterpret_cast<bf16*>(smem + cf.off_v);         // [C][ldv]
+  bf16* sA = reinterpret_cast<bf16*>(smem + cf.off_a);         // [hi, lo][C][C + 8]
+  float* sA1 = reinterpret_cast<float*>(smem + cf.off_a1);     // [2][C][rp]
+  float* sA2 = reinterpret_cast<float*>(smem + cf.off_a2);     // [rp][Kp]
+  float* sF = reinterpret_cast<float*>(smem + cf.off_f);       // [2][Kp] decays of the halves
+  float* sS = reinterpret_cast<float*>(smem + cf.off_ss);      // [2][C] sums of squares (cluster), then [8 warps][C]
+  constexpr int ldA = C + 8;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, l8 = lane & 7, lq = lane >> 3, g = lane >> 2, t4 = lane & 3;
+  const int h = blockIdx.y, v0 = blockIdx.x * vs;
+  const int64_t HK = (int64_t)m.heads * K, HV = (int64_t)m.heads * V;
+  const bool state_warp = warp * 16 < vs;
+  pdl_launch_dependents();
+  // weights of the decay projection do not depend on earlier kernels
+  for (int i = tid; i < rp * Kp; i += NT) {
+    const int r = i / Kp, k = i % Kp;
+    sA2[i] = r < m.rank && k < K ? m.a2[((int64_t)h * K + k) * m.rank + r] : 0.f;
+  }
+  const int kc = tid & 127, half = tid >> 7;                   // this thread's key channel and half of the chunk
+  const float kbias = kc < K ? m.a2_b[(int64_t)h * K + kc] : 0.f;
+  pdl_wait();
+  const GlaPortion p = a.list[blockIdx.z];
+  float* st = a.state + ((int64_t)p.lane * m.heads + h) * K * a.ldv;
+  // S[j][e]: value row v0 + 16 warp + g + 8 (e >> 1), channel 8 j + 2 t4 + (e & 1)
+  float S[2 * KT][4];
+#pragma unroll
+  for (int j = 0; j < 2 * KT; ++j)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int v = v0 + warp * 16 + g + 8 * (e >> 1), k = 8 * j + 2 * t4 + (e & 1);
+      S[j][e] = p.pos0 > 0 && state_warp && v < V && k < K ? st[(int64_t)k * a.ldv + v] : 0.f;
+    }
+  auto load_a1 = [&](int t0, float* dst) {
+    for (int i = tid; i < C * rp; i += NT) {
+      const int t = i / rp, r = i % rp;
+      dst[i] = t0 + t < p.n && r < m.rank ? slab(a, a.partial + (int64_t)(p.row0 + t0 + t) * a.ld + 2 * HK + 2 * HV + r) : 0.f;
+    }
+  };
+  load_a1(0, sA1);
+  __syncthreads();
+  const float qscale = rsqrtf((float)K), dscale = -LOG2E / m.tau;
+  for (int t0 = 0, it = 0; t0 < p.n; t0 += C, ++it) {
+    const int nt = min(C, p.n - t0);
+    const float* a1 = sA1 + (it & 1) * C * rp;
+    const float* base = a.partial + (int64_t)(p.row0 + t0) * a.ld;
+    // ---- values
+    for (int i = tid; i < C * vs / 4; i += NT) {
+      const int t = i / (vs / 4), v = (i % (vs / 4)) * 4;
+      float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (t < nt && v0 + v < V) x = slab4(a, base + (int64_t)t * a.ld + 2 * HK + (int64_t)h * V + v0 + v);
+      *reinterpret_cast<uint2*>(sV + t * ldv + v) = make_uint2(pack_bf16(x.x, x.y), pack_bf16(x.z, x.w));
+    }
+    // ---- decays and scaled queries and keys of this thread's channel, 16 tokens
+    bool far = false;
+    if (kc < Kp) {
+      float e[16];
+#pragma unroll
+      for (int u = 0; u < 16; ++u) e[u] = kbias;
+      for (int r = 0; r < rp; r += 4) {
+        const float w0 = sA2[r * Kp + kc], w1 = sA2[(r + 1) * Kp + kc], w2 = sA2[(r + 2) * Kp + kc], w3 = sA2[(r + 3) * Kp + kc];
+#pragma unroll
+        for (int u = 0; u < 16; ++u) {
+          const float4 x = *reinterpret_cast<const float4*>(a1 + (half * 16 + u) * rp + r);
+          e[u] = fmaf(x.x, w0, fmaf(x.y, w1, fmaf(x.z, w2, fmaf(x.w, w3, e[u]))));
+        }
+      }
+      // log2 of the decays, then their sums from the middle of the chunk
+      float tot = 0.f;
+#pragma unroll
+      for (int u = 0; u < 16; ++u) {
+        const float z = e[u];
+        const float la = half * 16 + u < nt && kc < K ? (fmaxf(-z, 0.f) + log1pf(ex2(-LOG2E * fabsf(z)))) * dscale : 0.f;
+        tot += la;
+        e[u] = la;
+      }
+      far = tot < -MAX_DECAY;
+      sF[half * Kp + kc] = ex2(tot);
+      float run = half ? 0.f : tot;
+#pragma unroll
+      for (int u = 0; u < 16; ++u) {
+        // first half: minus the decays still ahead of the middle; second half: the decays since
+        if (half) {
+          run += e[u];
+          e[u] = run;
+        } else {
+          run -= e[u];
+          e[u] = -run;
+        }
+      }
+      const float* qp = base + (int64_t)half * 16 * a.ld + (int64_t)h * K + kc;
+#pragma unroll
+      for (int u = 0; u < 16; ++u) {
+        const int t = half * 16 + u;
+        float q = 0.f, k = 0.f;
+        if (t < nt && kc < K) {
+          q = slab(a, qp + (int64_t)u * a.ld);
+          k = slab(a, qp + (int64_t)u * a.ld + HK);
+        }
+        const float f = far ? 0.f : ex2(e[u]), fi = far ? 0.f : ex2(-e[u]);
+        bf16* dq = sQ + t * ldq + kc;
+        bf16* dk = sK + t * ldq + kc;
+        split(q * qscale * f, dq[0], dq[C * ldq]);
+        split(k * fi, dk[0], dk[C * ldq]);
+      }
+    }
+    const bool slow = __syncthreads_or(far ? 1 : 0) != 0;
+    if (t0 + C < p.n) load_a1(t0 + C, sA1 + ((it + 1) & 1) * C * rp);
+    float o[4][4];
+#pragma unroll
+    for (int j = 0; j < 4; ++j)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) o[j][e] = 0.f;
+    if (!slow) {
+      const uint32_t aQ = smem_u32(sQ), aK = smem_u32(sK), aV = smem_u32(sV), aA = smem_u32(sA);
+      const uint32_t lo = C * ldq * 2;   // bytes from the high parts to the remainders
+      // ---- scores: six 16 x 8 tiles on and below the diagonal
+      if (warp < 6) {
+        const int mt = warp < 2 ? 0 : 1, nn = warp < 2 ? warp : warp - 2;
+        float s[4] = {0.f, 0.f, 0.f, 0.f};
+        const uint32_t qa = aQ + ((mt * 16 + (lq & 1) * 8 + l8) * ldq + (lq >> 1) * 8) * 2;
+        const uint32_t ka = aK + ((nn * 8 + l8) * ldq + (lq & 1) * 8) * 2;
+        for (int k = 0; k < cf.kt; ++k) {
+          uint32_t qh[4], ql[4], b0, b1, c0, c1;
+          ldmatrix_x4(qh[0], qh[1], qh[2], qh[3], qa + k * 32);
+          ldmatrix_x4(ql[0], ql[1], ql[2], ql[3], qa + k * 32 + lo);
+          ldmatrix_x2(b0, b1, ka + k * 32);
+          ldmatrix_x2(c0, c1, ka + k * 32 + lo);
+          mma_bf16_16816(s, qh, b0, b1);
+          mma_bf16_16816(s, qh, c0, c1);
+          mma_bf16_16816(s, ql, b0, b1);
+        }
+#pragma unroll
+        for (int r = 0; r < 2; ++r) {
+          const int t = mt * 16 + g + 8 * r, sc = nn * 8 + 2 * t4;
+          uint32_t hi, lw;
+          split2(sc <= t ? s[2 * r] : 0.f, sc + 1 <= t ? s[2 * r + 1] : 0.f, hi, lw);
+          *reinterpret_cast<uint32_t*>(sA + t * ldA + sc) = hi;
+          *reinterpret_cast<uint32_t*>(sA + (C + t) * ldA + sc) = lw;
+        }
+      } else {
+        // tokens 0 .. 15 see none of 16 .. 31
+        for (int i = tid - 192; i < 2 * 16 * 8; i += 64)
+          *reinterpret_cast<uint32_t*>(sA + ((i >> 7) * C + ((i >> 3) & 15)) * ldA + 16 + (i & 7) * 2) = 0u;
+      }
+      // ---- the state as every earlier token left it: o^T [16 value rows][C] = (e^r S)^T q~^T
+      if (state_warp) {
+        const uint32_t qb = aQ + (((lq >> 1) * 8 + l8) * ldq + (lq & 1) * 8) * 2;
+#pragma unroll
+        for (int k = 0; k < KT; ++k) {
+          if (k >= cf.kt) break;
+          const float2 f0 = *reinterpret_cast<const float2*>(sF + k * 16 + 2 * t4), f1 = *reinterpret_cast<const float2*>(sF + k * 16 + 8 + 2 * t4);
+          uint32_t sh[4], sl[4];
+#pragma unroll
+          for (int r = 0; r < 2; ++r) {
+            S[2 * k][2 * r] *= f0.x;
+            S[2 * k][2 * r + 1] *= f0.y;
+            S[2 * k + 1][2 * r] *= f1.x;
+            S[2 * k + 1][2 * r + 1] *= f1.y;
+            split2(S[2 * k][2 * r], S[2 * k][2 * r + 1], sh[r], sl[r]);
+            split2(S[2 * k + 1][2 * r], S[2 * k + 1][2 * r + 1], sh[2 + r], sl[2 + r]);
+          }
+#pragma unroll
+          for (int j = 0; j < 4; j += 2) {
+            uint32_t b[4], c[4];
+            ldmatrix_x4(b[0], b[1], b[2], b[3], qb + j * 8 * ldq * 2 + k * 32);
+            ldmatrix_x4(c[0], c[1], c[2], c[3], qb + j * 8 * ldq * 2 + k * 32 + lo);
+            mma_bf16_16816(o[j], sh, b[0], b[1]);
+            mma_bf16_16816(o[j + 1], sh, b[2], b[3]);
+            mma_bf16_16816(o[j], sl, b[0], b[1]);
+            mma_bf16_16816(o[j + 1], sl, b[2], b[3]);
+            mma_bf16_16816(o[j], sh, c[0], c[1]);
+            mma_bf16_16816(o[j + 1], sh, c[2], c[3]);
+          }
+        }
+      }
+      __syncthreads();
+      // ---- o^T += v^T A^T, S^T += v^T k~, then the rest of the decay
+      if (state_warp) {
+        const uint32_t ab = aA + (((lq >> 1) * 8 + l8) * ldA + (lq & 1) * 8) * 2;
+        const uint32_t kb = aK + (((lq & 1) * 8 + l8) * ldq + (lq >> 1) * 8) * 2;
+#pragma unroll
+        for (int s = 0; s < 2; ++s) {
+          uint32_t vf[4];
+          ldmatrix_x4_trans(vf[0], vf[1], vf[2], vf[3], aV + ((s * 16 + (lq >> 1) * 8 + l8) * ldv + warp * 16 + (lq & 1) * 8) * 2);
+#pragma unroll
+          for (int j = 0; j < 4; j += 2) {
+            uint32_t b[4], c[4];
+            ldmatrix_x4(b[0], b[1], b[2], b[3], ab + j * 8 * ldA * 2 + s * 32);
+            ldmatrix_x4(c[0], c[1], c[2], c[3], ab + j * 8 * ldA * 2 + s * 32 + C * ldA * 2);
+            mma_bf16_16816(o[j], vf, b[0], b[1]);
+            mma_bf16_16816(o[j + 1], vf, b[2], b[3]);
+            mma_bf16_16816(o[j], vf, c[0], c[1]);
+            mma_bf16_16816(o[j + 1], vf, c[2], c[3]);
+          }
+#pragma unroll
+          for (int k = 0; k < KT; ++k) {
+            if (k >= cf.kt) break;
+            uint32_t b[4], c[4];
+            ldmatrix_x4_trans(b[0], b[1], b[2], b[3], kb + s * 16 * ldq * 2 + k * 32);
+            ldmatrix_x4_trans(c[0], c[1], c[2], c[3], kb + s * 16 * ldq * 2 + k * 32 + lo);
+            mma_bf16_16816(S[2 * k], vf, b[0], b[1]);
+            mma_bf16_16816(S[2 * k + 1], vf, b[2], b[3]);
+            mma_bf16_16816(S[2 * k], vf, c[0], c[1]);
+            mma_bf16_16816(S[2 * k + 1], vf, c[2], c[3]);
+          }
+        }
+#pragma unroll
+        for (int j = 0; j < 2 * KT; ++j) {
+          if (j >= 2 * cf.kt) break;
+          const float2 f = *reinterpret_cast<const float2*>(sF + Kp + j * 8 + 2 * t4);
+          S[j][0] *= f.x;
+          S[j][1] *= f.y;
+          S[j][2] *= f.x;
+          S[j][3] *= f.y;
+        }
+        // output and its sums of squares over this warp's value rows
+#pragma unroll
+        for (int j = 0; j < 4; ++j)
+#pragma unroll
+          for (int e = 0; e < 2; ++e) {
+            const int t = j * 8 + 2 * t4 + e;
+            float ss = o[j][e] * o[j][e] + o[j][e + 2] * o[j][e + 2];
+            ss += __shfl_xor_sync(0xffffffffu, ss, 4);
+            ss += __shfl_xor_sync(0xffffffffu, ss, 8);
+            ss += __shfl_xor_sync(0xffffffffu, ss, 16);
+            if (g == 0) sS[2 * C + warp * C + t] = ss;
+            sO[t * ldO + warp * 16 + g] = o[j][e];
+            sO[t * ldO + warp * 16 + g + 8] = o[j][e + 2];
+          }
+      }
+    } else {
+      // ---- token by token: q | k | alpha in the k~ buffer
+      float* x = reinterpret_cast<float*>(sK);
+      for (int t = 0; t < nt; ++t) {
+        for (int k = tid; k < Kp; k += NT) {
+          float q = 0.f, kk = 0.f, al = 0.f;
+          if (k < K) {
+            const float* qp = base + (int64_t)t * a.ld + (int64_t)h * K + k;
+            q = slab(a, qp) * qscale;
+            kk = slab(a, qp + HK);
+            float z = m.a2_b[(int64_t)h * K + k];
+            for (int r = 0; r < rp; ++r) z = fmaf(a1[t * rp + r], sA2[r * Kp + k], z);
+            al = ex2((fmaxf(-z, 0.f) + log1pf(ex2(-LOG2E * fabsf(z)))) * dscale);
+          }
+          x[k] = q;
+          x[Kp + k] = kk;
+          x[2 * Kp + k] = al;
+        }
+        __syncthreads();
+        if (state_warp) {
+          const float va = __bfloat162float(sV[t * ldv + warp * 16 + g]), vb = __bfloat162float(sV[t * ldv + warp * 16 + g + 8]);
+          float oa = 0.f, ob = 0.f;
+#pragma unroll
+          for (int j = 0; j < 2 * KT; ++j) {
+            if (j >= 2 * cf.kt) break;
+            const float2 q = *reinterpret_cast<const float2*>(x + j * 8 + 2 * t4), k = *reinterpret_cast<const float2*>(x + Kp + j * 8 + 2 * t4),
+                         al = *reinterpret_cast<const float2*>(x + 2 * Kp + j * 8 + 2 * t4);
+            S[j][0] = fmaf(al.x, S[j][0], k.x * va);
+            S[j][1] = fmaf(al.y, S[j][1], k.y * va);
+            S[j][2] = fmaf(al.x, S[j][2], k.x * vb);
+            S[j][3] = fmaf(al.y, S[j][3], k.y * vb);
+            oa = fmaf(q.x, S[j][0], fmaf(q.y, S[j][1], oa));
+            ob = fmaf(q.x, S[j][2], fmaf(q.y, S[j][3], ob));
+          }
+          oa += __shfl_xor_sync(0xffffffffu, oa, 1);
+          oa += __shfl_xor_sync(0xffffffffu, oa, 2);
+          ob += __shfl_xor_sync(0xffffffffu, ob, 1);
+          ob += __shfl_xor_sync(0xffffffffu, ob, 2);
+          float ss = oa * oa + ob * ob;
+          ss += __shfl_xor_sync(0xffffffffu, ss, 4);
+          ss += __shfl_xor_sync(0xffffffffu, ss, 8);
+          ss += __shfl_xor_sync(0xffffffffu, ss, 16);
+          if (t4 == 0) {
+            sO[t * ldO + warp * 16 + g] = oa;
+            sO[t * ldO + warp * 16 + g + 8] = ob;
+          }
+          if (lane == 0) sS[2 * C + warp * C + t] = ss;
+        }
+        __syncthreads();
+      }
+    }
+    __syncthreads();
+    // ---- norm over the head, gate, store
+    if (tid < C) {
+      float ss = 0.f;
+      for (int w = 0; w * 16 < vs; ++w) ss += sS[2 * C + w * C + tid];
+      sS[(it & 1) * C + tid] = ss;
+    }
+    if constexpr (CLUSTER) cg::this_cluster().sync();
+    else __syncthreads();
+    for (int i = tid; i < nt * vs / 4; i += NT) {
+      const int t = i / (vs / 4), v = (i % (vs / 4)) * 4;
+      if (v0 + v >= V) continue;
+      float ss = sS[(it & 1) * C + t];
+      if constexpr (CLUSTER) {
+        ss = 0.f;
+        for (unsigned r = 0; r < gridDim.x; ++r) ss += cg::this_cluster().map_shared_rank(sS, r)[(it & 1) * C + t];
+      }
+      const float f = 1.0f / sqrtf(ss / (float)V + a.eps);
+      const float4 gz = slab4(a, base + (int64_t)t * a.ld + 2 * HK + HV + (int64_t)h * V + v0 + v);
+      const float4 x = *reinterpret_cast<const float4*>(sO + t * ldO + v), w = *reinterpret_cast<const float4*>(m.norm + v0 + v);
+      auto silu = [](float z) { return z / (1.0f + __expf(-z)); };
+      *reinterpret_cast<uint2*>(reinterpret_cast<bf16*>(a.out) + (int64_t)(p.row0 + t0 + t) * a.ldo + (int64_t)h * V + v0 + v) =
+          make_uint2(pack_bf16(x.x * f * w.x * silu(gz.x), x.y * f * w.y * silu(gz.y)), pack_bf16(x.z * f * w.z * silu(gz.z), x.w * f * w.w * silu(gz.w)));
+    }
+    __syncthreads();
+  }
+  if (state_warp) {
+#pragma unroll
+    for (int j = 0; j < 2 * KT; ++j)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int v = v0 + warp * 16 + g + 8 * (e >> 1), k = 8 * j + 2 * t4 + (e & 1);
+        if (v < V && k < K) st[(int64_t)k * a.ldv + v] = S[j][e];
+      }
+  }
+  if constexpr (CLUSTER) cg::this_cluster().sync();   // a peer may still read this CTA's sums
+}
+
+}  // namespace
+
+bool gla_chunk_ok(const GlaDims& m) { return m.dim % 8 == 0 && m.vdim % 8 == 0 && m.dim <= 128 && m.vdim <= 128 && m.rank <= 64; }
+
+int gla_chunk_launch(Ctx* c, const GlaArgs& a) {
+  if (a.count == 0) return REWB200_OK;
+  RB_REQUIRE(gla_chunk_ok(a.m) && a.dtype == REWB200_BF16 && a.list, "gated linear attention: sizes without a chunk kernel");
+  const int vp = (a.m.vdim + 15) / 16 * 16;
+  // few portions: a cluster of CTAs shares a head's value columns
+  int nv = 1;
+  while (nv < 4 && vp % (nv * 2 * 16) == 0 && (int64_t)nv * a.m.heads * a.count < c->sm_count) nv *= 2;
+  ChunkCfg cf;
+  cf.kt = (a.m.dim + 15) / 16;
+  cf.vs = vp / nv;
+  cf.rp = (a.m.rank + 3) / 4 * 4;
+  const int Kp = cf.kt * 16;
+  cf.ldq = Kp + 8;
+  auto up = [](int v) { return (v + 127) / 128 * 128; };
+  const int ops = 2 * C * cf.ldq * 2;
+  cf.off_k = up(std::max(ops, C * (cf.vs + 4) * 4));
+  cf.off_v = cf.off_k + up(std::max(ops, 3 * Kp * 4));
+  cf.off_a = cf.off_v + up(C * (cf.vs + 8) * 2);
+  cf.off_a1 = cf.off_a + up(2 * C * (C + 8) * 2);
+  cf.off_a2 = cf.off_a1 + up(2 * C * cf.rp * 4);
+  cf.off_f = cf.off_a2 + up(cf.rp * Kp * 4);
+  cf.off_ss = cf.off_f + up(2 * Kp * 4);
+  const int smem = cf.off_ss + up((2 + 8) * C * 4);
+  const dim3 grid((unsigned)nv, (unsigned)a.m.heads, (unsigned)a.count);
+  auto go = [&](auto kernel, bool cluster) -> int {
+    RB_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
+    RB_CUDA(cluster ? launch_k_cluster(kernel, grid, dim3(NT), smem, c->stream, c->use_pdl, dim3(nv), a, cf)
+                    : launch_k(kernel, grid, dim3(NT), smem, c->stream, c->use_pdl, a, cf));
+    ++g_launch_total;
+    return REWB200_OK;
+  };
+  if (cf.kt <= 4) return nv > 1 ? go(gla_chunk_kernel<4, true>, true) : go(gla_chunk_kernel<4, false>, false);
+  return nv > 1 ? go(gla_chunk_kernel<8, true>, true) : go(gla_chunk_kernel<8, false>, false);
+}
+
+}  // namespace rewb

@@ -1,0 +1,542 @@
+// Kernels of gqa.cuh: the fused post-processing of the input projection, attention of decoded tokens and small portions
+// on mma.sync, and plain kernels for f32 models and head sizes the tensor-core kernels do not take.  Norms, scores,
+// biases, softmax and gates are f32 throughout.
+#include <math.h>
+
+#include <algorithm>
+
+#include "gqa.cuh"
+#include "ptx.cuh"
+
+namespace rewb {
+
+extern int64_t g_launch_total;
+
+namespace {
+
+constexpr int PAGE_TOKENS = 64;
+constexpr float LOG2E = 1.4426950408889634f;
+
+__device__ __forceinline__ float warp_sum(float v) {
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
+  return v;
+}
+__device__ __forceinline__ float ex2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+__device__ __forceinline__ float sigmoid(float z) { return 1.0f / (1.0f + expf(-z)); }
+
+// Four neighbouring columns of a row, summed over the slabs in slab order; columns past `n` read as zero.
+__device__ __forceinline__ float4 slab4(const GqaPostArgs& a, const float* p, int i, int n, bool vec) {
+  float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+  if (i >= n) return v;
+  if (vec && i + 4 <= n) {
+#pragma unroll 4
+    for (int s = 0; s < a.nsplit; ++s) {
+      const float4 w = *reinterpret_cast<const float4*>(p + s * a.split_stride + i);
+      v.x += w.x; v.y += w.y; v.z += w.z; v.w += w.w;
+    }
+    return v;
+  }
+  float e[4] = {0.f, 0.f, 0.f, 0.f};
+  for (int u = 0; u < 4 && i + u < n; ++u)
+    for (int s = 0; s < a.nsplit; ++s) e[u] += p[s * a.split_stride + i + u];
+  return make_float4(e[0], e[1], e[2], e[3]);
+}
+template <typename T>
+__device__ __forceinline__ void put4(T* d, int i, int n, float4 v) {
+  if (i >= n) return;
+  if constexpr (sizeof(T) == 2) {
+    if (i + 4 <= n && (reinterpret_cast<uintptr_t>(d + i) & 7) == 0) {
+      *reinterpret_cast<uint2*>(d + i) = make_uint2(pack_bf16(v.x, v.y), pack_bf16(v.z, v.w));
+      return;
+    }
+  }
+  const float e[4] = {v.x, v.y, v.z, v.w};
+  for (int u = 0; u < 4 && i + u < n; ++u) d[i + u] = stf<T>(e[u]);
+}
+
+// One warp per head: query heads, key heads, value heads, then one warp for all gates.  A lane holds four columns at a
+// time, PC of them (dim and vdim up to 128 PC).
+template <typename T, int PC>
+__global__ void __launch_bounds__(256) gqa_post_kernel(GqaPostArgs a) {
+  pdl_launch_dependents();
+  const int64_t row = blockIdx.x;
+  const int unit = blockIdx.y * 8 + (threadIdx.x >> 5), ln = threadIdx.x & 31;
+  const int H = a.m.heads, G = a.m.own_kv ? a.m.kv_heads : 0, K = a.m.dim, V = a.m.vdim;
+  if (!a.early) pdl_wait();
+  const int pos = row_pos(a.map, row), lane = row_lane(a.map, row);
+  const bool ok = pos >= 0 && pos < a.capacity;
+  const int page = a.block_table[(int64_t)lane * a.max_pages + (ok ? pos / PAGE_TOKENS : 0)];
+  if (a.early) pdl_wait();
+  if (unit > H + 2 * G || (unit == H + 2 * G && !a.m.gate)) return;
+  if (!ok && unit == 0 && ln == 0) atomicExch(a.status, KS_BAD_INDEX);
+  const float* p = a.partial + row * a.ld;
+  if (unit == H + 2 * G) {
+    p += (int64_t)H * K + (int64_t)G * (K + V);
+    for (int h = ln; h < H; h += 32) {
+      float z = 0.f;
+      for (int s = 0; s < a.nsplit; ++s) z += p[s * a.split_stride + h];
+      a.gate[row * H + h] = sigmoid(z);
+    }
+    return;
+  }
+  const bool is_q = unit < H, is_v = unit >= H + G;
+  const int n = is_v ? V : K;
+  const int64_t col = is_v ? (int64_t)(H + G) * K + (int64_t)(unit - H - G) * V : (int64_t)unit * K;
+  const bool vec = col % 4 == 0 && a.ld % 4 == 0 && a.split_stride % 4 == 0;
+  float4 x[PC];
+  float ss = 0.f;
+#pragma unroll
+  for (int c = 0; c < PC; ++c) {
+    x[c] = slab4(a, p + col, (c * 32 + ln) * 4, n, vec);
+    ss += x[c].x * x[c].x + x[c].y * x[c].y + x[c].z * x[c].z + x[c].w * x[c].w;
+  }
+  const float* w = is_q ? a.m.q_norm : a.m.k_norm;
+  if (!is_v && w) {
+    float f = 1.0f / sqrtf(warp_sum(ss) / (float)K + a.eps);
+    if (is_q && a.m.temp_every > 0) f *= 1.0f + a.m.temp_coef * logf((float)((pos + 1) / a.m.temp_every + 1));
+#pragma unroll
+    for (int c = 0; c < PC; ++c) {
+      const int i = (c * 32 + ln) * 4;
+      float4 g = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (i < n) g.x = w[i];
+      if (i + 1 < n) g.y = w[i + 1];
+      if (i + 2 < n) g.z = w[i + 2];
+      if (i + 3 < n) g.w = w[i + 3];
+      x[c] = make_float4(x[c].x * f * g.x, x[c].y * f * g.y, x[c].z * f * g.z, x[c].w * f * g.w);
+    }
+  } else if (is_q && a.m.temp_every > 0) {
+    const float f = 1.0f + a.m.temp_coef * logf((float)((pos + 1) / a.m.temp_every + 1));
+#pragma unroll
+    for (int c = 0; c < PC; ++c) x[c] = make_float4(x[c].x * f, x[c].y * f, x[c].z * f, x[c].w * f);
+  }
+  T* dst;
+  if (is_q) {
+    dst = reinterpret_cast<T*>(a.q) + row * a.ldq + (int64_t)unit * K;
+  } else {
+    if (!ok) return;
+    const int g = is_v ? unit - H - G : unit - H;
+    const int64_t crow = ((int64_t)page * G + g) * PAGE_TOKENS + pos % PAGE_TOKENS;
+    dst = is_v ? reinterpret_cast<T*>(a.vc) + crow * a.ldv : reinterpret_cast<T*>(a.kc) + crow * a.ldk;
+  }
+#pragma unroll
+  for (int c = 0; c < PC; ++c) put4<T>(dst, (c * 32 + ln) * 4, n, x[c]);
+}
+
+// ------------------------------------------------------------------ plain attention: one CTA per (row of a tile, head),
+// online softmax over 64-key pages
+template <typename T>
+__global__ void __launch_bounds__(128) gqa_plain_kernel(GqaAttnArgs a) {
+  extern __shared__ float sm[];  // [dim] query, [vdim] accumulator, [64] scores
+  pdl_launch_dependents();
+  pdl_wait();
+  const int2 tr = tile_rows(a.tiles, blockIdx.x / a.max_tile_rows);
+  const int k_in = blockIdx.x % a.max_tile_rows;
+  if (k_in >= tr.y) return;
+  const int64_t row = tr.x + k_in;
+  const int h = blockIdx.y, K = a.m.dim, V = a.m.vdim, G = a.m.kv_heads, hk = h / (a.m.heads / G);
+  float *q = sm, *acc = sm + K, *sc = acc + V;
+  const T* qp = reinterpret_cast<const T*>(a.q) + row * a.ldq + (int64_t)h * K;
+  for (int i = threadIdx.x; i < K; i += 128) q[i] = ldf<T>(qp[i]);
+  for (int i = threadIdx.x; i < V; i += 128) acc[i] = 0.f;
+  const int lane = row_lane(a.map, row), pos = min(max(row_pos(a.map, row), 0), a.max_pages * PAGE_TOKENS - 1);
+  const int w = threadIdx.x >> 5, ln = threadIdx.x & 31;
+  const float* tab = a.m.bias ? a.m.bias + (int64_t)h * a.m.n_bias : nullptr;
+  float mx = a.m.sink ? a.m.sink[h] : -INFINITY, l = a.m.sink ? 1.f : 0.f;
+  __syncthreads();
+  for (int t = 0; t <= pos / PAGE_TOKENS; ++t) {
+    const int page = a.block_table[(int64_t)lane * a.max_pages + t];
+    const T* kb = reinterpret_cast<const T*>(a.kc) + ((int64_t)page * G + hk) * PAGE_TOKENS * a.ldk;
+    const T* vb = reinterpret_cast<const T*>(a.vc) + ((int64_t)page * G + hk) * PAGE_TOKENS * a.ldv;
+    for (int j = w; j < PAGE_TOKENS; j += 4) {
+      const int key = t * PAGE_TOKENS + j;
+      float s = 0.f;
+      if (key <= pos)
+        for (int i = ln; i < K; i += 32) s = fmaf(q[i], ldf<T>(kb[(int64_t)j * a.ldk + i]), s);
+      s = warp_sum(s);
+      if (ln == 0) sc[j] = key <= pos ? s * a.m.scale + (tab ? tab[min(pos - key, a.m.n_bias - 1)] : 0.f) : -INFINITY;
+    }
+    __syncthreads();
+    float tm = mx;
+    for (int j = 0; j < PAGE_TOKENS; ++j) tm = fmaxf(tm, sc[j]);
+    const float alpha = mx == -INFINITY ? 0.f : expf(mx - tm);
+    __syncthreads();
+    if (threadIdx.x < PAGE_TOKENS) sc[threadIdx.x] = sc[threadIdx.x] == -INFINITY ? 0.f : expf(sc[threadIdx.x] - tm);
+    __syncthreads();
+    float ps = 0.f;
+    for (int j = 0; j < PAGE_TOKENS; ++j) ps += sc[j];
+    l = l * alpha + ps;
+    mx = tm;
+    const int j1 = min(PAGE_TOKENS - 1, pos - t * PAGE_TOKENS);
+    for (int i = threadIdx.x; i < V; i += 128) {
+      float v = acc[i] * alpha;
+      for (int j = 0; j <= j1; ++j) v = fmaf(sc[j], ldf<T>(vb[(int64_t)j * a.ldv + i]), v);
+      acc[i] = v;
+    }
+    __syncthreads();
+  }
+  const float g = (a.m.gate ? a.gate[row * a.m.heads + h] : 1.0f) / l;
+  T* op = reinterpret_cast<T*>(a.out) + row * a.ldo + (int64_t)h * V;
+  for (int i = threadIdx.x; i < V; i += 128) op[i] = stf<T>(acc[i] * g);
+}
+
+// ------------------------------------------------------------------ bf16 on the tensor cores
+// grid (kv splits, tiles * subtiles, kv heads * head groups), four consumer warps and a TMA warp.  A CTA's 16 rows are
+// `heads_per` query heads of one kv head times `tokens_per` tokens; every K / V page is loaded once for all of them.
+// Warp w owns keys 16 w .. 16 w + 15 of every page with a softmax state of its own in registers (no barrier between
+// warps but the ring's); the warps meet after the last page.
+struct GqaCfg {
+  int nb_k, nb_v;     // 64-column boxes of a key / value row
+  int stages;
+  int heads_per, hgroups, tokens_per, subtiles;
+};
+
+// Shared tail of the attention and merge kernels: the sink joins the softmax, the gate scales the output.
+__device__ __forceinline__ float sink_l2(const GqaDims& m, int h) { return m.sink ? m.sink[h] * LOG2E : -INFINITY; }
+
+// KS: 16-feature steps of a key row, VG: 16-column groups of a value row.
+template <int KS, int VG>
+__global__ void __launch_bounds__(160) gqa_attn_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_constant__ CUtensorMap tm_v,
+                                                       GqaAttnArgs a, GqaCfg cf) {
+  extern __shared__ uint8_t smem_raw[];
+  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
+  const int kb = cf.nb_k * 8192, stage_bytes = kb + cf.nb_v * 8192;
+  uint8_t* sKV = smem;
+  uint8_t* sQ = sKV + cf.stages * stage_bytes;                      // [box][16 rows][128 bytes]
+  float* sM = reinterpret_cast<float*>(sQ + cf.nb_k * 2048);        // [4 warps][16] maxima, [4][16] sums
+  uint64_t* full = reinterpret_cast<uint64_t*>(sM + 128);
+  uint64_t* empty = full + 8;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, l8 = lane & 7, lq = lane >> 3, g = lane >> 2, t = lane & 3;
+  if (tid == 128) {
+    for (int i = 0; i < cf.stages; ++i) {
+      mbar_init(&full[i], 1);
+      mbar_init(&empty[i], 4);
+    }
+    fence_barrier_init();
+    tma_prefetch_desc(&tm_k);
+    tma_prefetch_desc(&tm_v);
+  }
+  pdl_launch_dependents();
+  __syncthreads();
+  if (!a.early_kv) pdl_wait();
+  const int2 tr = tile_rows(a.tiles, (int)blockIdx.y / cf.subtiles);
+  const int tok0 = ((int)blockIdx.y % cf.subtiles) * cf.tokens_per;
+  const int ntok = min(cf.tokens_per, tr.y - tok0);
+  if (ntok <= 0) return;
+  const int64_t row0 = tr.x + tok0;
+  const int hk = blockIdx.z / cf.hgroups, group = a.m.heads / a.m.kv_heads;
+  const int hsub = ((int)blockIdx.z % cf.hgroups) * cf.heads_per, nh = min(cf.heads_per, group - hsub), head0 = hk * group + hsub;
+  const int lane_id = row_lane(a.map, row0);
+  const int cap = a.max_pages * PAGE_TOKENS;
+  const int pos_first = min(max(row_pos(a.map, row0), 0), cap - 1), pos_last = min(pos_first + ntok - 1, cap - 1);
+  const int nt_all = pos_last / PAGE_TOKENS + 1;
+  const int per = (nt_all + (int)gridDim.x - 1) / (int)gridDim.x;
+  const int t0 = (int)blockIdx.x * per, nt = max(0, min(per, nt_all - t0));
+  if (warp == 4) {
+    if (lane == 0) {
+      auto load_page = [&](int i) {
+        const int st = i % cf.stages;
+        const int y = (a.block_table[(int64_t)lane_id * a.max_pages + t0 + i] * a.m.kv_heads + hk) * PAGE_TOKENS;
+        mbar_expect_tx(&full[st], stage_bytes);
+        for (int b = 0; b < cf.nb_k; ++b) tma_load_2d(sKV + st * stage_bytes + b * 8192, &tm_k, &full[st], b * 64, y);
+        for (int b = 0; b < cf.nb_v; ++b) tma_load_2d(sKV + st * stage_bytes + kb + b * 8192, &tm_v, &full[st], b * 64, y);
+      };
+      int i = 0;
+      if (a.early_kv) {
+        const int newest = pos_last / PAGE_TOKENS - t0;   // the page the step's own row is written to
+        for (; i < min(cf.stages, nt) && i < newest; ++i) load_page(i);
+        pdl_wait();
+      }
+      for (; i < nt; ++i) {
+        if (i >= cf.stages && !mbar_wait(&empty[i % cf.stages], ((i / cf.stages) - 1) & 1, a.status)) break;
+        load_page(i);
+      }
+    }
+    return;
+  }
+  if (a.early_kv) pdl_wait();
+  auto consumers_sync = [] { asm volatile("bar.sync 1, 128;" ::: "memory"); };
+  for (int i = tid; i < 16 * cf.nb_k * 8; i += 128) {
+    const int m = i / (cf.nb_k * 8), c = i % (cf.nb_k * 8);
+    const int tok = m / cf.heads_per, hh = m % cf.heads_per;
+    uint4 v = make_uint4(0, 0, 0, 0);
+    if (tok < ntok && hh < nh && c * 8 < a.m.dim)   // dim is a multiple of 8
+      v = *reinterpret_cast<const uint4*>(reinterpret_cast<const bf16*>(a.q) + (row0 + tok) * a.ldq + (int64_t)(head0 + hh) * a.m.dim + c * 8);
+    *reinterpret_cast<uint4*>(sQ + (c >> 3) * 2048 + swz128((uint32_t)m, (uint32_t)(c & 7))) = v;
+  }
+  consumers_sync();
+  const int ks = (a.m.dim + 15) / 16, vg = (a.m.vdim + 15) / 16;
+  uint32_t qf[KS][4];
+  const uint32_t q_base = smem_u32(sQ);
+#pragma unroll
+  for (int k = 0; k < KS; ++k)
+    if (k < ks)
+      ldmatrix_x4(qf[k][0], qf[k][1], qf[k][2], qf[k][3], q_base + (k >> 2) * 2048 + swz128((lq & 1) * 8 + l8, (k & 3) * 2 + (lq >> 1)));
+  // this thread's rows: g and g + 8
+  const float sl2 = a.m.scale * LOG2E;
+  int spos[2];
+  const float* tab[2];
+  float far[2];
+#pragma unroll
+  for (int r = 0; r < 2; ++r) {
+    const int m = g + 8 * r, tok = m / cf.heads_per, hh = m % cf.heads_per;
+    spos[r] = tok < ntok && hh < nh ? pos_first + tok : -1;   // -1: sees no key
+    tab[r] = a.m.bias ? a.m.bias + (int64_t)(head0 + min(hh, nh - 1)) * a.m.n_bias : nullptr;
+    far[r] = tab[r] ? tab[r][a.m.n_bias - 1] * LOG2E : 0.f;
+  }
+  float mrun[2] = {-INFINITY, -INFINITY}, lrun[2] = {0.f, 0.f};
+  float acc[VG][2][4];
+#pragma unroll
+  for (int j = 0; j < VG; ++j)
+#pragma unroll
+    for (int e = 0; e < 8; ++e) acc[j][e >> 2][e & 3] = 0.f;
+  uint32_t k_off[4], v_off[4];
+#pragma unroll
+  for (int u = 0; u < 4; ++u) {
+    k_off[u] = swz128(warp * 16 + (lq >> 1) * 8 + l8, u * 2 + (lq & 1));
+    v_off[u] = swz128(warp * 16 + (lq & 1) * 8 + l8, u * 2 + (lq >> 1));
+  }
+  const uint32_t kv_base = smem_u32(sKV);
+  bool ok = true;
+  for (int it = 0; it < nt; ++it) {
+    const int st = it % cf.stages;
+    if (ok) ok = mbar_wait(&full[st], (it / cf.stages) & 1, a.status);
+    const uint32_t kp = kv_base + st * stage_bytes, vp = kp + kb;
+    float sc[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
+#pragma unroll
+    for (int k = 0; k < KS; ++k) {
+      if (k >= ks) break;
+      uint32_t b0, b1, b2, b3;
+      ldmatrix_x4(b0, b1, b2, b3, kp + (k >> 2) * 8192 + k_off[k & 3]);
+      mma_bf16_16816(sc[0], qf[k], b0, b1);
+      mma_bf16_16816(sc[1], qf[k], b2, b3);
+    }
+    const int key0 = (t0 + it) * PAGE_TOKENS + warp * 16 + 2 * t;
+    const bool inside = (t0 + it) * PAGE_TOKENS + PAGE_TOKENS - 1 <= pos_first - (a.m.bias ? a.m.n_bias - 1 : 0);   // every distance has the far bias
+    float mx[2] = {-INFINITY, -INFINITY};
+#pragma unroll
+    for (int n = 0; n < 2; ++n)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int r = e >> 1, dist = spos[r] - (key0 + n * 8 + (e & 1));
+        float b = far[r];
+        if (!inside && tab[r] && dist >= 0) b = __ldg(tab[r] + min(dist, a.m.n_bias - 1)) * LOG2E;
+        sc[n][e] = dist >= 0 ? fmaf(sc[n][e], sl2, b) : -INFINITY;
+        mx[r] = fmaxf(mx[r], sc[n][e]);
+      }
+    float alpha[2], muse[2];
+#pragma unroll
+    for (int r = 0; r < 2; ++r) {
+      mx[r] = fmaxf(mx[r], __shfl_xor_sync(0xffffffffu, mx[r], 1));
+      mx[r] = fmaxf(mx[r], __shfl_xor_sync(0xffffffffu, mx[r], 2));
+      const float mn = fmaxf(mrun[r], mx[r]);
+      muse[r] = mn == -INFINITY ? 0.f : mn;
+      alpha[r] = ex2(mrun[r] - muse[r]);
+      mrun[r] = mn;
+    }
+    uint32_t pf[4];
+    float ps[2] = {0.f, 0.f};
+#pragma unroll
+    for (int n = 0; n < 2; ++n)
+#pragma unroll
+      for (int r = 0; r < 2; ++r) {
+        const float p0 = ex2(sc[n][2 * r] - muse[r]), p1 = ex2(sc[n][2 * r + 1] - muse[r]);
+        ps[r] += p0 + p1;
+        pf[n * 2 + r] = pack_bf16(p0, p1);
+      }
+    lrun[0] = lrun[0] * alpha[0] + ps[0];
+    lrun[1] = lrun[1] * alpha[1] + ps[1];
+    if (__any_sync(0xffffffffu, alpha[0] != 1.f || alpha[1] != 1.f)) {
+#pragma unroll
+      for (int j = 0; j < VG; ++j)
+#pragma unroll
+        for (int n = 0; n < 2; ++n) {
+          acc[j][n][0] *= alpha[0];
+          acc[j][n][1] *= alpha[0];
+          acc[j][n][2] *= alpha[1];
+          acc[j][n][3] *= alpha[1];
+        }
+    }
+#pragma unroll
+    for (int j = 0; j < VG; ++j) {
+      if (j >= vg) break;
+      uint32_t v0, v1, v2, v3;
+      ldmatrix_x4_trans(v0, v1, v2, v3, vp + (j >> 2) * 8192 + v_off[j & 3]);
+      mma_bf16_16816(acc[j][0], pf, v0, v1);
+      mma_bf16_16816(acc[j][1], pf, v2, v3);
+    }
+    __syncwarp();
+    if (lane == 0) mbar_arrive(&empty[st]);
+  }
+#pragma unroll
+  for (int r = 0; r < 2; ++r) {
+    lrun[r] += __shfl_xor_sync(0xffffffffu, lrun[r], 1);
+    lrun[r] += __shfl_xor_sync(0xffffffffu, lrun[r], 2);
+    if (t == 0) {
+      sM[warp * 16 + g + 8 * r] = mrun[r];
+      sM[64 + warp * 16 + g + 8 * r] = lrun[r];
+    }
+  }
+  // the stages are read out: they hold the warps' accumulators now, [4][16][vg * 16 + 4]
+  consumers_sync();
+  float* sO = reinterpret_cast<float*>(sKV);
+  const int ldO = vg * 16 + 4;
+#pragma unroll
+  for (int j = 0; j < VG; ++j) {
+    if (j >= vg) break;
+#pragma unroll
+    for (int n = 0; n < 2; ++n)
+#pragma unroll
+      for (int r = 0; r < 2; ++r)
+        *reinterpret_cast<float2*>(sO + (warp * 16 + g + 8 * r) * ldO + j * 16 + n * 8 + 2 * t) = make_float2(acc[j][n][2 * r], acc[j][n][2 * r + 1]);
+  }
+  consumers_sync();
+  const int V = a.m.vdim, v2 = V / 2;   // vdim is a multiple of 8
+  for (int i = tid; i < 16 * v2; i += 128) {
+    const int m = i / v2, c = (i % v2) * 2, tok = m / cf.heads_per, hh = m % cf.heads_per;
+    if (tok >= ntok || hh >= nh) continue;
+    const int h = head0 + hh;
+    const int64_t row = row0 + tok;
+    const bool last = gridDim.x == 1;
+    float M = last ? sink_l2(a.m, h) : -INFINITY;
+#pragma unroll
+    for (int w = 0; w < 4; ++w) M = fmaxf(M, sM[w * 16 + m]);
+    const float mu = M == -INFINITY ? 0.f : M;
+    float l = 0.f;
+    float2 o = make_float2(0.f, 0.f);
+#pragma unroll
+    for (int w = 0; w < 4; ++w) {
+      const float f = ex2(sM[w * 16 + m] - mu);
+      const float2 x = *reinterpret_cast<const float2*>(sO + (w * 16 + m) * ldO + c);
+      l += f * sM[64 + w * 16 + m];
+      o.x += f * x.x;
+      o.y += f * x.y;
+    }
+    if (last) {
+      if (a.m.sink) l += ex2(sink_l2(a.m, h) - mu);
+      const float inv = (a.m.gate ? a.gate[row * a.m.heads + h] : 1.0f) / l;
+      *reinterpret_cast<uint32_t*>(reinterpret_cast<bf16*>(a.out) + row * a.ldo + (int64_t)h * V + c) = pack_bf16(o.x * inv, o.y * inv);
+    } else {
+      const int64_t u = (row * a.m.heads + h) * a.kv_splits + blockIdx.x;
+      *reinterpret_cast<float2*>(a.o_part + u * V + c) = o;
+      if (c == 0) a.ml[u] = make_float2(M, l);
+    }
+  }
+}
+
+// One warp per (row of a tile, head): the kv splits, the sink and the gate.
+__global__ void __launch_bounds__(256) gqa_merge_kernel(GqaAttnArgs a) {
+  pdl_launch_dependents();
+  const int64_t u = (int64_t)blockIdx.x * 8 + (threadIdx.x >> 5);
+  const int ln = threadIdx.x & 31, H = a.m.heads, V = a.m.vdim, ns = a.kv_splits;
+  const int64_t slot = u / H;
+  const int h = (int)(u % H);
+  if (slot >= (int64_t)a.tiles.count * a.max_tile_rows) return;
+  pdl_wait();
+  const int2 tr = tile_rows(a.tiles, (int)(slot / a.max_tile_rows));
+  const int k = (int)(slot % a.max_tile_rows);
+  if (k >= tr.y) return;
+  const int64_t row = tr.x + k, at = (row * H + h) * ns;
+  const float2 e = ln < ns ? a.ml[at + ln] : make_float2(-INFINITY, 0.f);   // at most 32 splits
+  float M = e.x;
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) M = fmaxf(M, __shfl_xor_sync(0xffffffffu, M, o));
+  const float sk = sink_l2(a.m, h);
+  M = fmaxf(M, sk);
+  const float mu = M == -INFINITY ? 0.f : M;
+  const float f = ex2(e.x - mu);
+  float l = warp_sum(f * e.y);
+  if (a.m.sink) l += ex2(sk - mu);
+  const float inv = (a.m.gate ? a.gate[row * H + h] : 1.0f) / l;
+  for (int c0 = 0; c0 < V; c0 += 128) {
+    const int c = c0 + ln * 4;
+    float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 4
+    for (int s = 0; s < ns; ++s) {
+      const float w = __shfl_sync(0xffffffffu, f, s);
+      if (c < V) {
+        const float4 x = *reinterpret_cast<const float4*>(a.o_part + (at + s) * V + c);
+        o.x += w * x.x; o.y += w * x.y; o.z += w * x.z; o.w += w * x.w;
+      }
+    }
+    if (c < V)
+      *reinterpret_cast<uint2*>(reinterpret_cast<bf16*>(a.out) + row * a.ldo + (int64_t)h * V + c) =
+          make_uint2(pack_bf16(o.x * inv, o.y * inv), pack_bf16(o.z * inv, o.w * inv));
+  }
+}
+
+bool mma_ok(const GqaDims& m) { return m.dim % 8 == 0 && m.vdim % 8 == 0 && m.dim <= 256 && m.vdim <= 256; }
+
+GqaCfg config(const GqaDims& m, int max_tile_rows) {
+  GqaCfg cf;
+  const int group = m.heads / m.kv_heads;
+  cf.nb_k = (m.dim + 63) / 64;
+  cf.nb_v = (m.vdim + 63) / 64;
+  cf.heads_per = std::min(group, 16);
+  cf.hgroups = (group + cf.heads_per - 1) / cf.heads_per;
+  cf.tokens_per = std::min(max_tile_rows, std::max(1, 16 / cf.heads_per));
+  cf.subtiles = (max_tile_rows + cf.tokens_per - 1) / cf.tokens_per;
+  cf.stages = std::min(4, std::max(2, (int)(104 * 1024 / ((cf.nb_k + cf.nb_v) * 8192))));
+  return cf;
+}
+
+}  // namespace
+
+int gqa_post_launch(Ctx* c, const GqaPostArgs& a, int64_t rows) {
+  if (rows == 0) return REWB200_OK;
+  const int units = a.m.heads + (a.m.own_kv ? 2 * a.m.kv_heads : 0) + (a.m.gate ? 1 : 0);
+  RB_REQUIRE(a.m.dim <= 512 && a.m.vdim <= 512, "grouped-query attention: head sizes above 512");
+  const dim3 grid((unsigned)rows, (unsigned)((units + 7) / 8));
+  const bool small = a.m.dim <= 128 && a.m.vdim <= 128, bf = a.dtype == REWB200_BF16;
+  RB_CUDA(bf ? (small ? launch_k(gqa_post_kernel<bf16, 1>, grid, dim3(256), 0, c->stream, c->use_pdl, a)
+                      : launch_k(gqa_post_kernel<bf16, 4>, grid, dim3(256), 0, c->stream, c->use_pdl, a))
+             : (small ? launch_k(gqa_post_kernel<float, 1>, grid, dim3(256), 0, c->stream, c->use_pdl, a)
+                      : launch_k(gqa_post_kernel<float, 4>, grid, dim3(256), 0, c->stream, c->use_pdl, a)));
+  ++g_launch_total;
+  return REWB200_OK;
+}
+
+// KV splits of a launch over `tiles` row tiles: enough CTAs for two per SM, no more than a split per page.
+int gqa_kv_splits(Ctx* c, const GqaDims& m, int64_t tiles, int64_t max_ctx) {
+  const int group = m.heads / m.kv_heads;
+  const int64_t ctas = std::max<int64_t>(1, tiles * m.kv_heads * ((group + 15) / 16)), pages = (max_ctx + PAGE_TOKENS - 1) / PAGE_TOKENS;
+  return (int)std::max<int64_t>(1, std::min<int64_t>({(2 * c->sm_count + ctas - 1) / ctas, pages, 16}));
+}
+
+int gqa_attn_launch(Ctx* c, const GqaAttnArgs& a) {
+  if (a.tiles.count == 0) return REWB200_OK;
+  if (a.dtype != REWB200_BF16 || c->gqa_impl == 1 || !mma_ok(a.m)) {
+    const dim3 grid((unsigned)a.tiles.count * a.max_tile_rows, (unsigned)a.m.heads);
+    const size_t smem = (a.m.dim + a.m.vdim + PAGE_TOKENS) * sizeof(float);
+    RB_CUDA(a.dtype == REWB200_BF16 ? launch_k(gqa_plain_kernel<bf16>, grid, dim3(128), smem, c->stream, c->use_pdl, a)
+                                    : launch_k(gqa_plain_kernel<float>, grid, dim3(128), smem, c->stream, c->use_pdl, a));
+    ++g_launch_total;
+    return REWB200_OK;
+  }
+  const GqaCfg cf = config(a.m, a.max_tile_rows);
+  const size_t kv = (size_t)cf.stages * (cf.nb_k + cf.nb_v) * 8192, merge = (size_t)64 * ((a.m.vdim + 15) / 16 * 16 + 4) * 4;
+  const size_t smem = std::max(kv, (merge + 1023) / 1024 * 1024) + cf.nb_k * 2048 + 512 + 256 + 1024;
+  RB_REQUIRE(kv >= merge, "grouped-query attention: value heads too large for the merge buffer");
+  const dim3 grid((unsigned)a.kv_splits, (unsigned)(a.tiles.count * cf.subtiles), (unsigned)(a.m.kv_heads * cf.hgroups));
+  const int ks = (a.m.dim + 15) / 16, vg = (a.m.vdim + 15) / 16;
+  auto go = [&](auto kernel) -> int {
+    RB_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    RB_CUDA(launch_k(kernel, grid, dim3(160), smem, c->stream, c->use_pdl, *a.tm_k, *a.tm_v, a, cf));
+    ++g_launch_total;
+    return REWB200_OK;
+  };
+  if (ks <= 4 && vg <= 4) RB_TRY(go(gqa_attn_kernel<4, 4>));
+  else if (ks <= 8 && vg <= 8) RB_TRY(go(gqa_attn_kernel<8, 8>));
+  else RB_TRY(go(gqa_attn_kernel<16, 16>));
+  if (a.kv_splits == 1) return REWB200_OK;
+  const int64_t units = (int64_t)a.tiles.count * a.max_tile_rows * a.m.heads;
+  RB_CUDA(launch_k(gqa_merge_kernel, dim3((unsigned)((units + 7) / 8)), dim3(256), 0, c->stream, c->use_pdl, a));
+  ++g_launch_total;
+  return REWB200_OK;
+}
+
+}  // namespace rewb

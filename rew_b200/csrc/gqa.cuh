@@ -1,0 +1,95 @@
+// Grouped-query attention of layered models: per-head RMS norms of queries and keys, a query temperature that grows
+// with the position, a learned bias per head and distance bucket, a learned number per head in the softmax denominator
+// ("sink"), an output gate per head.  Argument structs and launchers of gqa.cu and gqa_prefill.cu.
+//
+// Caches: keys [pages][kv_heads][64][ldk], values [pages][kv_heads][64][ldv].
+#pragma once
+#include "steprows.cuh"
+
+namespace rewb {
+
+struct GqaDims {
+  int heads, kv_heads, dim, vdim;
+  int own_kv;              // 0: another layer's keys and values
+  int gate;
+  float scale;
+  const float* q_norm;     // [dim] or nullptr: no norm
+  const float* k_norm;
+  int temp_every;          // queries times 1 + temp_coef ln(floor((p + 1) / temp_every) + 1); 0: no temperature
+  float temp_coef;
+  const float* bias;       // [heads][n_bias] by distance; the last entry holds for every longer distance; nullptr: none
+  int n_bias;
+  const float* sink;       // [heads] or nullptr
+};
+
+// Finishes the fused input projection [q | k | v | gate] (q | gate without keys of its own): sums the split-K slabs,
+// norms queries and keys, applies the temperature, appends keys and values to the cache.
+struct GqaPostArgs {
+  GqaDims m;
+  const float* partial;    // [nsplit][rows][ld]
+  int nsplit;
+  int64_t split_stride, ld;
+  float eps;
+  RowMap map;
+  void* q;                 // [rows][ldq] act dtype
+  int64_t ldq;
+  float* gate;             // [rows][heads]
+  void *kc, *vc;
+  int64_t ldk, ldv;
+  const int* block_table;
+  int max_pages, capacity;
+  int dtype;
+  int early;               // captured decode step: positions predate the step
+  int* status;
+};
+int gqa_post_launch(Ctx* c, const GqaPostArgs& a, int64_t rows);
+
+// Attention of the rows in `tiles` (decoded tokens, small portions).
+struct GqaAttnArgs {
+  GqaDims m;
+  RowMap map;
+  RowTiles tiles;
+  int max_tile_rows;
+  const void* q;
+  int64_t ldq;
+  const float* gate;
+  void* out;               // [rows][ldo] act dtype, head-major columns
+  int64_t ldo;
+  const void *kc, *vc;
+  const CUtensorMap *tm_k, *tm_v;  // bf16: box 64 x 64
+  int64_t ldk, ldv;
+  const int* block_table;
+  int max_pages;
+  int dtype;
+  float* o_part;           // scratch [rows][heads][kv splits][vdim], not yet divided by the row sum
+  float2* ml;              // scratch [rows][heads][kv splits] running maximum (base 2) and sum
+  int kv_splits;
+  int64_t rows;            // rows of the whole step
+  int early_kv;            // captured decode step: cache pages other than the newest may be loaded ahead of the stream dependency
+  int* status;
+};
+int gqa_attn_launch(Ctx* c, const GqaAttnArgs& a);
+int gqa_kv_splits(Ctx* c, const GqaDims& m, int64_t tiles, int64_t max_ctx);
+
+// Attention of large prompt portions on tcgen05; one tile = up to 256 queries of one portion.
+struct GqaTile {
+  int row0, n, pos0, lane;
+};
+struct GqaPrefillArgs {
+  GqaDims m;
+  const GqaTile* tiles;
+  int count;
+  const bf16* q;
+  int64_t ldq;
+  const float* gate;
+  bf16* out;
+  int64_t ldo;
+  const CUtensorMap *tm_k, *tm_v;
+  const int* block_table;
+  int max_pages;
+  int* status;
+};
+bool gqa_prefill_ok(const GqaDims& m);
+int gqa_prefill_launch(Ctx* c, const GqaPrefillArgs& a);
+
+}  // namespace rewb

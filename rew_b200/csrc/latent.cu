@@ -15,25 +15,6 @@ namespace {
 
 constexpr int PAGE_TOKENS = 64;
 
-template <typename T> __device__ __forceinline__ float ldf(T v);
-template <> __device__ __forceinline__ float ldf<float>(float v) { return v; }
-template <> __device__ __forceinline__ float ldf<bf16>(bf16 v) { return __bfloat162float(v); }
-template <typename T> __device__ __forceinline__ T stf(float v);
-template <> __device__ __forceinline__ float stf<float>(float v) { return v; }
-template <> __device__ __forceinline__ bf16 stf<bf16>(float v) { return __float2bfloat16_rn(v); }
-
-__device__ __forceinline__ int row_lane(const RowMap& m, int64_t row) {
-  return m.row_lane ? m.row_lane[row] : m.b0 + (int)(row / m.S);
-}
-__device__ __forceinline__ int row_pos(const RowMap& m, int64_t row) {
-  return m.row_pos ? m.row_pos[row] : m.pos0[m.b0 + row / m.S] + (int)(row % m.S);
-}
-__device__ __forceinline__ int2 tile_rows(const RowTiles& t, int i) {
-  if (t.list) return t.list[i];
-  const int per_lane = (t.S + t.per_tile - 1) / t.per_tile;
-  const int lane = i / per_lane, k = (i % per_lane) * t.per_tile;
-  return make_int2(lane * t.S + k, min(t.per_tile, t.S - k));
-}
 __device__ __forceinline__ float2 rotate(float2 v, float2 cs) {
   return make_float2(v.x * cs.x - v.y * cs.y, v.y * cs.x + v.x * cs.y);
 }

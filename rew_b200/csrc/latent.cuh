@@ -6,27 +6,9 @@
 // W_uv (sum_j p_j c_j), so attention can run on the cache rows themselves ("absorbed": small steps, decode) or on
 // keys and values expanded from them per head (large prompt portions).
 #pragma once
-#include "common.cuh"
+#include "steprows.cuh"
 
 namespace rewb {
-
-// Which sequence (lane) and position a row of the step belongs to: explicit arrays (a step of unequal portions), or
-// S consecutive tokens for every lane from b0 on, starting at the lane's position pos0[lane].
-struct RowMap {
-  const int* row_lane;
-  const int* row_pos;
-  const int* pos0;
-  int b0, S;
-};
-
-// Runs of consecutive rows of one lane: an explicit list of (first row, rows), or (list == nullptr) the rows of
-// every lane of a uniform step in pieces of `per_tile`.
-struct RowTiles {
-  const int2* list;
-  int count;      // tiles
-  int S;          // rows per lane (list == nullptr)
-  int per_tile;   // rows per tile at most
-};
 
 constexpr int kChunkRows = 64;   // RowTiles of LatentAttnArgs::chunks
 

@@ -1,345 +1,70 @@
-// Latent attention of large prompt portions on keys and values expanded per head, on tcgen05.
-//
-// A CTA owns one head of up to QT x 128 queries of one portion (QT 2 where shared memory allows it, else 1); both query
-// tiles share every 128-key K / V tile.  Warp roles:
-//   warp 0        TMA: K tiles (per-head features from the expanded keys, then the rotated features all heads share from
-//                 the gathered cache rows) and V tiles
-//   warp 1        one thread issues S_t = Q_t K^T and O_t += P_t V; while the softmax warps of one query tile work, the
-//                 tensor core runs the other tile's products
-//   warps 2 ..    eight softmax warps per query tile: thread = query row, two warps share a row's keys.  Scores, maxima,
-//                 sums and rotations are f32; P goes back to tensor memory as bf16.
-// Tensor memory: S_t (P overwrites it) 128 columns each, O_t 64 x value boxes columns each.  Every wait is bounded.
-// A query sees the keys of its window only: key tiles outside a query tile's windows are skipped, tiles across an edge
-// are masked.
-#include <math.h>
-
-#include <algorithm>
-
+// Latent attention of large prompt portions on keys and values expanded per head: the tcgen05 kernel of flash_tc.cuh.  The
+// rotated features all heads share come from the gathered cache rows; queries are rotated on the way in.
+#include "flash_tc.cuh"
 #include "latent.cuh"
-#include "ptx.cuh"
-#include "tc.cuh"
 
 namespace rewb {
 
-extern int64_t g_launch_total;
-
 namespace {
 
-constexpr int BOX_BYTES = 128 * 128;   // 128 rows x 64 bf16 columns
-constexpr int XCH_FLOATS = 3 * 2 * 128;   // per query tile: two buffers of half-row maxima, half-row sums
+struct LatentPolicy {
+  static constexpr bool kBias = false;
+  LatentExpArgs a;
+  int nb_n;                // boxes of unrotated features
+  int heads, vdim;
+  float scale;
+  const float* gate;
+  bf16* out;
+  int64_t ldo;
+  int* status;
 
-struct ExpCfg {
-  int nb_n, nb_r, nb_v;   // 64-column boxes of unrotated / rotated features and of values
-  int v_stages;
+  __device__ __forceinline__ ExpTile tile(int i, int skip) const {
+    ExpTile t = a.tiles[i];
+    t.row0 += skip;
+    t.n -= skip;
+    t.pos0 += skip;
+    return t;
+  }
+  __device__ __forceinline__ int window() const { return a.m.window; }
+  __device__ __forceinline__ int k_base(const ExpTile& t) const { return max(t.key0, a.m.window > 0 ? t.pos0 - a.m.window + 1 : 0); }
+  __device__ __forceinline__ int n_bias() const { return 1; }
+  __device__ __forceinline__ uint4 q_chunk(const ExpTile& t, int qi, int head, int box, int c) const {
+    const bf16* qp = a.q + (int64_t)(t.row0 + qi) * a.ldq + (int64_t)head * (a.m.dim + a.m.rot_dim);
+    uint4 v = make_uint4(0, 0, 0, 0);
+    if (box < nb_n) {
+      const int f = box * 64 + c;
+      if (f < a.m.dim) v = *reinterpret_cast<const uint4*>(qp + f);
+      return v;
+    }
+    const int f = (box - nb_n) * 64 + c, half_r = a.m.rope_dims / 2;
+    if (f >= a.m.rot_dim) return v;
+    const float2* rope = a.m.rope + (int64_t)min(t.pos0 + qi, a.m.max_pos - 1) * half_r;
+    v = *reinterpret_cast<const uint4*>(qp + a.m.dim + f);
+    uint32_t w[4] = {v.x, v.y, v.z, v.w};
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int p = f / 2 + e;
+      if (p < half_r) {
+        const __nv_bfloat162 x = *reinterpret_cast<const __nv_bfloat162*>(&w[e]);
+        const float2 cs = rope[p];
+        const float u = __low2float(x), s = __high2float(x);
+        w[e] = pack_bf16(u * cs.x - s * cs.y, s * cs.x + u * cs.y);
+      }
+    }
+    return make_uint4(w[0], w[1], w[2], w[3]);
+  }
+  __device__ __forceinline__ void load_k(uint8_t* dst, const CUtensorMap& tm_kv, const CUtensorMap& tm_lat, uint64_t* bar, const ExpTile& t, int head,
+                                         int j, int k_base, const flash::Cfg& cf) const {
+    const int krow = k_base + j * 128 + t.off;
+    for (int b = 0; b < nb_n; ++b) tma_load_2d(dst + b * flash::BOX_BYTES, &tm_kv, bar, head * a.m.dim + b * 64, krow);
+    for (int b = nb_n; b < cf.nb_k; ++b) tma_load_2d(dst + b * flash::BOX_BYTES, &tm_lat, bar, a.m.kv_rank + (b - nb_n) * 64, krow);
+  }
+  __device__ __forceinline__ void load_v(uint8_t* dst, const CUtensorMap& tm_kv, const CUtensorMap&, uint64_t* bar, const ExpTile& t, int head, int j,
+                                         int k_base, const flash::Cfg& cf) const {
+    const int krow = k_base + j * 128 + t.off;
+    for (int b = 0; b < cf.nb_v; ++b) tma_load_2d(dst + b * flash::BOX_BYTES, &tm_kv, bar, heads * a.m.dim + head * vdim + b * 64, krow);
+  }
 };
-
-__device__ __forceinline__ float ex2(float x) {
-  float y;
-  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-  return y;
-}
-__device__ __forceinline__ void pair_barrier(int id) { asm volatile("bar.sync %0, 64;" ::"r"(id) : "memory"); }
-
-// The softmax of one query tile (see attention.cu for the exchange between the two warps of a lane quarter).  Key tiles
-// j_lo .. j_hi - 1, tile j = keys k_base + 128 j ..; first / last: positions of the tile's first and last query.
-__device__ __forceinline__ void softmax_rows(const LatentExpArgs& a, const ExpCfg& cf, uint32_t s_addr, uint32_t o_addr, float* xmax, float* xsum,
-                                             uint64_t* s_full, uint64_t* p_full, uint64_t* o_done, int j_lo, int j_hi, int k_base, int row0,
-                                             int n, int first, int quarter, int half, int lane, int pair_bar, int head) {
-  const int row = quarter * 32 + lane;
-  const int hi = first + row;                                        // last visible key
-  const int lo = a.m.window > 0 ? hi - a.m.window : -1;              // the key before the first visible one
-  const int last = first + min(n, 128) - 1;
-  const float sl2 = a.m.scale * 1.4426950408889634f;
-  float m = -INFINITY, l = 0.f;
-  bool ok = true;
-  for (int j = j_lo; j < j_hi; ++j) {
-    const int it = j - j_lo;
-    if (ok) ok = mbar_wait(s_full, it & 1, a.status);
-    __syncwarp();
-    tc::fence_after();
-    const int kt = k_base + j * 128, k0 = kt + half * 64;
-    const bool edge = kt + 127 > first || (a.m.window > 0 && kt <= last - a.m.window);
-    uint32_t r0[32], r1[32];
-    tc::ld32_issue(s_addr + half * 64, r0);
-    tc::ld32_issue(s_addr + half * 64 + 32, r1);
-    tc::wait_ld();
-    if (edge) {
-#pragma unroll
-      for (int e = 0; e < 32; ++e) {
-        if (k0 + e > hi || k0 + e <= lo) r0[e] = 0xff800000u;            // -inf
-        if (k0 + 32 + e > hi || k0 + 32 + e <= lo) r1[e] = 0xff800000u;
-      }
-    }
-    float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
-#pragma unroll
-    for (int e = 0; e < 32; e += 4)
-#pragma unroll
-      for (int u = 0; u < 4; ++u) mx4[u] = fmaxf(fmaxf(mx4[u], __uint_as_float(r0[e + u])), __uint_as_float(r1[e + u]));
-    float mraw = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3]));
-    float* xm = xmax + (it & 1) * 256;
-    xm[half * 128 + row] = mraw;
-    pair_barrier(pair_bar);   // both warps hold their scores in registers now; P may overwrite them
-    mraw = fmaxf(mraw, xm[(half ^ 1) * 128 + row]);
-    // the maximum of the raw scores is that of the scaled ones: the host requires a positive scale
-    const float mx = fmaxf(m, mraw * sl2);
-    const float m_use = mx == -INFINITY ? 0.f : mx;
-    const float alpha = ex2(m - m_use);
-    float ls[4] = {0.f, 0.f, 0.f, 0.f};
-    uint32_t pk[32];
-#pragma unroll
-    for (int cc = 0; cc < 2; ++cc) {
-      const uint32_t* rr = cc ? r1 : r0;
-#pragma unroll
-      for (int e = 0; e < 32; e += 2) {
-        const float p0 = ex2(fmaf(__uint_as_float(rr[e]), sl2, -m_use));
-        const float p1 = ex2(fmaf(__uint_as_float(rr[e + 1]), sl2, -m_use));
-        ls[(e >> 1) & 3] += p0 + p1;
-        pk[cc * 16 + (e >> 1)] = pack_bf16(p0, p1);
-      }
-    }
-    tc::st32(s_addr + half * 32, pk);
-    l = l * alpha + ((ls[0] + ls[1]) + (ls[2] + ls[3]));
-    m = mx;
-    // S of this tile was announced after P V of the one before it, so O is complete up to there
-    if (it > 0 && __any_sync(0xffffffffu, alpha != 1.0f)) {
-#pragma unroll 1
-      for (int c = 0; c < cf.nb_v; ++c) {
-        const uint32_t at = o_addr + half * 32 * cf.nb_v + c * 32;
-        tc::ld32_issue(at, r0);
-        tc::wait_ld();
-#pragma unroll
-        for (int e = 0; e < 32; ++e) r0[e] = __float_as_uint(__uint_as_float(r0[e]) * alpha);
-        tc::st32_issue(at, r0);
-        tc::wait_st();
-      }
-    }
-    tc::fence_before();
-    __syncwarp();
-    if (lane == 0) mbar_arrive(p_full);
-  }
-  xsum[half * 128 + row] = l;
-  pair_barrier(pair_bar);
-  l += xsum[(half ^ 1) * 128 + row];
-  const int tiles = j_hi - j_lo;
-  if (tiles > 0 && ok) ok = mbar_wait(o_done, (tiles - 1) & 1, a.status);
-  __syncwarp();
-  tc::fence_after();
-  if (tiles <= 0) return;
-  const bool store = row < n && ok;
-  const int64_t grow = row0 + min(row, n - 1);
-  const float gt = a.m.gate ? a.gate[grow * a.m.heads + head] : 1.0f;
-  const float inv = l > 0.f ? gt / l : 0.f;
-  bf16* op = a.out + grow * a.ldo + (int64_t)head * a.m.vdim;
-  uint32_t r[32];
-#pragma unroll 1
-  for (int c = 0; c < cf.nb_v; ++c) {
-    const int col = half * 32 * cf.nb_v + c * 32;
-    tc::ld32(o_addr + col, r);
-    if (!store) continue;
-#pragma unroll
-    for (int e = 0; e < 32; e += 8) {
-      if (col + e >= a.m.vdim) continue;   // vdim is a multiple of 8
-      uint4 v;
-      v.x = pack_bf16(__uint_as_float(r[e]) * inv, __uint_as_float(r[e + 1]) * inv);
-      v.y = pack_bf16(__uint_as_float(r[e + 2]) * inv, __uint_as_float(r[e + 3]) * inv);
-      v.z = pack_bf16(__uint_as_float(r[e + 4]) * inv, __uint_as_float(r[e + 5]) * inv);
-      v.w = pack_bf16(__uint_as_float(r[e + 6]) * inv, __uint_as_float(r[e + 7]) * inv);
-      *reinterpret_cast<uint4*>(op + col + e) = v;
-    }
-  }
-}
-
-template <int QT>
-__global__ void __launch_bounds__(64 + QT * 256, 1) latent_prefill_kernel(const __grid_constant__ CUtensorMap tm_kv,
-                                                                           const __grid_constant__ CUtensorMap tm_lat, LatentExpArgs a,
-                                                                           ExpCfg cf) {
-  extern __shared__ uint8_t smem_raw[];
-  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
-  const int nb = cf.nb_n + cf.nb_r;
-  const int q_bytes = nb * BOX_BYTES, k_bytes = nb * BOX_BYTES, v_bytes = cf.nb_v * BOX_BYTES;
-  uint8_t* sQ = smem;
-  uint8_t* sK = sQ + QT * q_bytes;
-  uint8_t* sV = sK + k_bytes;
-  float* xch = reinterpret_cast<float*>(sV + cf.v_stages * v_bytes);
-  uint64_t* bars = reinterpret_cast<uint64_t*>(xch + QT * XCH_FLOATS);
-  uint64_t *k_full = bars, *k_empty = bars + 1, *v_full = bars + 2, *v_empty = bars + 4, *s_full = bars + 6, *p_full = bars + 8,
-           *o_done = bars + 10;
-  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 12);
-  constexpr uint32_t TM_COLS = QT * 256;
-
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int head = blockIdx.y;
-  if (threadIdx.x == 0) {
-    mbar_init(k_full, 1);
-    mbar_init(k_empty, 1);
-    for (int i = 0; i < 2; ++i) {
-      mbar_init(v_full + i, 1);
-      mbar_init(v_empty + i, 1);
-      mbar_init(s_full + i, 1);
-      mbar_init(p_full + i, 8);
-      mbar_init(o_done + i, 1);
-    }
-    fence_barrier_init();
-    pdl_launch_dependents();
-  }
-  if (warp == 1) tc::alloc(tmem_slot, TM_COLS);
-  tc::fence_before();
-  __syncthreads();
-  tc::fence_after();
-  const uint32_t tmem_base = *tmem_slot;
-  pdl_wait();
-
-  // QT == 1: two CTAs per listed tile, 128 queries each
-  const ExpTile et = a.tiles[QT == 2 ? blockIdx.x : blockIdx.x >> 1];
-  const int q_skip = QT == 2 ? 0 : (int)(blockIdx.x & 1) * 128;
-  const int row0 = et.row0 + q_skip, n = et.n - q_skip, pos0 = et.pos0 + q_skip;   // n may be <= 0 (uniform over the CTA)
-  const int W = a.m.window;
-  const int k_base = max(et.key0, W > 0 ? pos0 - W + 1 : 0);
-  int jlo[2] = {0, 0}, jhi[2] = {0, 0};
-#pragma unroll
-  for (int t = 0; t < QT; ++t) {
-    const int first = pos0 + t * 128, nt = min(n - t * 128, 128);
-    if (nt <= 0) continue;
-    jlo[t] = W > 0 ? max(0, first - W + 1 - k_base) >> 7 : 0;
-    jhi[t] = ((first + nt - 1 - k_base) >> 7) + 1;
-  }
-  const int j_end = max(jhi[0], jhi[1]);
-
-  if (warp >= 2 && n > 0) {
-    // queries: one row per two threads of a tile, rotated on the way, in the layout a 128-byte-swizzled TMA would leave
-    const int idx = threadIdx.x - 64, r = idx & 127, part = (idx >> 7) & 1, t = idx >> 8;
-    const int qi = t * 128 + r;
-    const bool in = qi < n;
-    const bf16* qp = a.q + (int64_t)(row0 + min(qi, n - 1)) * a.ldq + (int64_t)head * (a.m.dim + a.m.rot_dim);
-    const int half_r = a.m.rope_dims / 2;
-    const float2* rope = a.m.rope + (int64_t)min(pos0 + qi, a.m.max_pos - 1) * half_r;
-    for (int ch = part; ch < nb * 8; ch += 2) {
-      const int box = ch >> 3, c = (ch & 7) * 8;
-      uint4 v = make_uint4(0, 0, 0, 0);
-      if (box < cf.nb_n) {
-        const int f = box * 64 + c;
-        if (in && f < a.m.dim) v = *reinterpret_cast<const uint4*>(qp + f);
-      } else {
-        const int f = (box - cf.nb_n) * 64 + c;
-        if (in && f < a.m.rot_dim) {
-          v = *reinterpret_cast<const uint4*>(qp + a.m.dim + f);
-          uint32_t w[4] = {v.x, v.y, v.z, v.w};
-#pragma unroll
-          for (int e = 0; e < 4; ++e) {
-            const int p = f / 2 + e;
-            if (p < half_r) {
-              const __nv_bfloat162 x = *reinterpret_cast<const __nv_bfloat162*>(&w[e]);
-              const float2 cs = rope[p];
-              const float u = __low2float(x), s = __high2float(x);
-              w[e] = pack_bf16(u * cs.x - s * cs.y, s * cs.x + u * cs.y);
-            }
-          }
-          v = make_uint4(w[0], w[1], w[2], w[3]);
-        }
-      }
-      *reinterpret_cast<uint4*>(sQ + t * q_bytes + box * BOX_BYTES + swz128((uint32_t)r, (uint32_t)(ch & 7))) = v;
-    }
-    fence_proxy_async();
-  }
-  __syncthreads();
-
-  if (warp == 0) {
-    if (lane == 0 && n > 0) {
-      tma_prefetch_desc(&tm_kv);
-      tma_prefetch_desc(&tm_lat);
-      bool ok = true;
-      for (int j = 0; j < j_end && ok; ++j) {
-        const int krow = k_base + j * 128 + et.off;
-        if (j > 0) ok = mbar_wait(k_empty, (j - 1) & 1, a.status);
-        if (!ok) break;
-        mbar_expect_tx(k_full, k_bytes);
-        for (int b = 0; b < cf.nb_n; ++b) tma_load_2d(sK + b * BOX_BYTES, &tm_kv, k_full, head * a.m.dim + b * 64, krow);
-        for (int b = 0; b < cf.nb_r; ++b) tma_load_2d(sK + (cf.nb_n + b) * BOX_BYTES, &tm_lat, k_full, a.m.kv_rank + b * 64, krow);
-        const int st = j % cf.v_stages;
-        if (j >= cf.v_stages) ok = mbar_wait(v_empty + st, (j / cf.v_stages - 1) & 1, a.status);
-        if (!ok) break;
-        mbar_expect_tx(v_full + st, v_bytes);
-        for (int b = 0; b < cf.nb_v; ++b)
-          tma_load_2d(sV + st * v_bytes + b * BOX_BYTES, &tm_kv, v_full + st, a.m.heads * a.m.dim + head * a.m.vdim + b * 64, krow);
-      }
-    }
-  } else if (warp == 1) {
-    if (lane == 0 && n > 0) {
-      const uint32_t idesc_qk = (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(128 >> 3) << 17) | ((uint32_t)(128 >> 4) << 24);
-      const uint32_t idesc_pv = (1u << 4) | (1u << 7) | (1u << 10) | (1u << 16) | ((uint32_t)(cf.nb_v * 8) << 17) | ((uint32_t)(128 >> 4) << 24);
-      constexpr uint32_t hi = tc::desc_hi(1024);
-      const uint32_t q_lo = tc::desc_lo(smem_u32(sQ), 16), k_lo = tc::desc_lo(smem_u32(sK), 16), v_lo = tc::desc_lo(smem_u32(sV), BOX_BYTES);
-      auto active = [&](int t, int j) { return j >= jlo[t] && j < jhi[t]; };
-      auto issue_qk = [&](int t) {
-        const uint32_t qa = q_lo + t * (q_bytes >> 4);
-        for (int b = 0; b < nb; ++b)
-#pragma unroll
-          for (int kk = 0; kk < 4; ++kk) {
-            const uint32_t off = b * (BOX_BYTES >> 4) + kk * 2;
-            tc::umma_bf16_ss_lh(tmem_base + t * 128, qa + off, k_lo + off, hi, idesc_qk, (b > 0 || kk > 0) ? 1u : 0u);
-          }
-        tc::commit(s_full + t);
-      };
-      bool ok = mbar_wait(k_full, 0, a.status);
-      if (ok) {
-        tc::fence_after();
-#pragma unroll
-        for (int t = 0; t < QT; ++t)
-          if (active(t, 0)) issue_qk(t);
-        tc::commit(k_empty);
-      }
-      for (int j = 0; j < j_end && ok; ++j) {
-        const int st = j % cf.v_stages;
-        bool v_ready = false, k_ready = false;
-#pragma unroll
-        for (int t = 0; t < QT; ++t) {
-          if (!ok) break;
-          if (active(t, j)) {
-            ok = mbar_wait(p_full + t, (j - jlo[t]) & 1, a.status);
-            if (ok && !v_ready) ok = v_ready = mbar_wait(v_full + st, (j / cf.v_stages) & 1, a.status);
-            if (!ok) break;
-            tc::fence_after();
-            const uint32_t va = v_lo + st * (v_bytes >> 4);
-            const uint32_t acc0 = j > jlo[t] ? 1u : 0u;
-#pragma unroll
-            for (int kk = 0; kk < 8; ++kk)
-              tc::umma_bf16_ta_lh(tmem_base + QT * 128 + t * 128, tmem_base + t * 128 + kk * 8, va + kk * (2048 >> 4), hi, idesc_pv,
-                                  kk > 0 ? 1u : acc0);
-            tc::commit(o_done + t);
-          }
-          if (active(t, j + 1)) {
-            if (!k_ready) ok = k_ready = mbar_wait(k_full, (j + 1) & 1, a.status);
-            if (!ok) break;
-            tc::fence_after();
-            issue_qk(t);
-          }
-        }
-        if (!ok) break;
-        // the query tiles' key ranges overlap or touch, so some tile has waited for these loads already; if none had,
-        // the buffers must not be released before they have landed
-        if (!v_ready) ok = mbar_wait(v_full + st, (j / cf.v_stages) & 1, a.status);
-        if (ok && j + 1 < j_end && !k_ready) ok = mbar_wait(k_full, (j + 1) & 1, a.status);
-        if (!ok) break;
-        tc::commit(v_empty + st);
-        if (j + 1 < j_end) tc::commit(k_empty);
-      }
-    }
-  } else {
-    const int t = (warp - 2) >> 3;
-    const int quarter = warp & 3, half = ((warp - 2) >> 2) & 1;
-    const uint32_t lane_addr = tmem_base + ((uint32_t)(quarter * 32) << 16);
-    float* xmax = xch + t * XCH_FLOATS;
-    softmax_rows(a, cf, lane_addr + t * 128, lane_addr + QT * 128 + t * 128, xmax, xmax + 2 * 2 * 128, s_full + t, p_full + t, o_done + t,
-                 t == 0 ? jlo[0] : jlo[1], t == 0 ? jhi[0] : jhi[1], k_base, row0 + t * 128, n - t * 128, pos0 + t * 128, quarter, half, lane,
-                 1 + t * 4 + quarter, head);
-  }
-  tc::fence_before();
-  __syncthreads();
-  if (warp == 1) {
-    tc::fence_after();
-    tc::dealloc(tmem_base, TM_COLS);
-  }
-}
 
 __global__ void __launch_bounds__(256) latent_gather_kernel(const bf16* cache, const int* block_table, int max_pages, int64_t ldc, const int2* index,
                                                             bf16* dst, int64_t n) {
@@ -352,12 +77,6 @@ __global__ void __launch_bounds__(256) latent_gather_kernel(const bf16* cache, c
   const uint4* src = reinterpret_cast<const uint4*>(cache + ((int64_t)page * 64 + lp.y % 64) * ldc);
   uint4* d = reinterpret_cast<uint4*>(dst + i * ldc);
   for (int c = threadIdx.x & 31; c < ldc / 8; c += 32) d[c] = src[c];
-}
-
-constexpr size_t kSmemMax = 227 * 1024;
-
-size_t exp_smem(int nb, int nb_v, int qt, int v_stages) {
-  return (size_t)(qt * nb + nb + v_stages * nb_v) * BOX_BYTES + (size_t)qt * XCH_FLOATS * 4 + 256 + 1024;
 }
 
 }  // namespace
@@ -373,35 +92,12 @@ bool latent_expanded_ok(const LatentDims& m) {
 int latent_attn_expanded_launch(Ctx* c, const LatentExpArgs& a) {
   if (a.count == 0) return REWB200_OK;
   RB_REQUIRE(latent_expanded_ok(a.m), "latent attention: head sizes without an expanded kernel");
-  ExpCfg cf;
-  cf.nb_n = (a.m.dim + 63) / 64;
-  cf.nb_r = (a.m.rot_dim + 63) / 64;
-  cf.nb_v = (a.m.vdim + 63) / 64;
-  const int nb = cf.nb_n + cf.nb_r;
-  int qt = 2;
-  cf.v_stages = 2;
-  if (exp_smem(nb, cf.nb_v, 2, 2) > kSmemMax) cf.v_stages = 1;
-  if (exp_smem(nb, cf.nb_v, 2, cf.v_stages) > kSmemMax) {
-    qt = 1;
-    cf.v_stages = 2;
-  }
-  const size_t smem = exp_smem(nb, cf.nb_v, qt, cf.v_stages);
-  RB_REQUIRE(smem <= kSmemMax, "latent attention: head sizes too large for the expanded kernel");
   CUtensorMap tm_kv, tm_lat;
   RB_TRY(make_tmap_2d_bf16(&tm_kv, a.kv, (uint64_t)a.m.heads * (a.m.dim + a.m.vdim), (uint64_t)a.keys, (uint64_t)a.ldkv * 2, 64, 128));
   RB_TRY(make_tmap_2d_bf16(&tm_lat, a.lat, (uint64_t)a.m.kv_rank + a.m.rot_dim, (uint64_t)a.keys, (uint64_t)a.ldc * 2, 64, 128));
-  static bool attr_set = false;
-  if (!attr_set) {
-    RB_CUDA(cudaFuncSetAttribute(latent_prefill_kernel<1>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kSmemMax));
-    RB_CUDA(cudaFuncSetAttribute(latent_prefill_kernel<2>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kSmemMax));
-    attr_set = true;
-  }
-  if (qt == 2)
-    RB_CUDA(launch_k(latent_prefill_kernel<2>, dim3((unsigned)a.count, (unsigned)a.m.heads), dim3(64 + 2 * 256), smem, c->stream, c->use_pdl, tm_kv, tm_lat, a, cf));
-  else
-    RB_CUDA(launch_k(latent_prefill_kernel<1>, dim3((unsigned)a.count * 2, (unsigned)a.m.heads), dim3(64 + 256), smem, c->stream, c->use_pdl, tm_kv, tm_lat, a, cf));
-  ++g_launch_total;
-  return REWB200_OK;
+  const int nb_n = (a.m.dim + 63) / 64;
+  const LatentPolicy p = {a, nb_n, a.m.heads, a.m.vdim, a.m.scale, a.m.gate ? a.gate : nullptr, a.out, a.ldo, a.status};
+  return flash::launch(c, p, tm_kv, tm_lat, a.count, nb_n + (a.m.rot_dim + 63) / 64, (a.m.vdim + 63) / 64, 0);
 }
 
 int latent_gather_launch(Ctx* c, const bf16* cache, const int* block_table, int max_pages, int64_t ldc, const int2* index, bf16* dst, int64_t n) {

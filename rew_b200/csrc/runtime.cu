@@ -295,6 +295,12 @@ int rewb200_set_option(int slot, const char* key, const char* value) {
   } else if (k == "latent_attention") {
     RB_REQUIRE(v == "auto" || v == "plain" || v == "absorbed", "option latent_attention: expected auto, plain or absorbed");
     c->latent_impl = v == "plain" ? 1 : v == "absorbed" ? 2 : 0;
+  } else if (k == "gqa_attention") {
+    RB_REQUIRE(v == "auto" || v == "plain" || v == "paged", "option gqa_attention: expected auto, plain or paged");
+    c->gqa_impl = v == "plain" ? 1 : v == "paged" ? 2 : 0;
+  } else if (k == "linear_attention") {
+    RB_REQUIRE(v == "auto" || v == "plain" || v == "recurrent", "option linear_attention: expected auto, plain or recurrent");
+    c->gla_impl = v == "plain" ? 1 : v == "recurrent" ? 2 : 0;
   } else if (k == "inject_alloc_fail") {
     const int n = atoi(v.c_str());
     RB_REQUIRE(n >= 0, "option inject_alloc_fail: a non-negative count");

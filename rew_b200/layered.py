@@ -5,40 +5,112 @@ logical tensors in the order rewb200_model_set_tensor indexes them; Linear weigh
 """
 from dataclasses import dataclass, field
 
+import numpy as np
+
 from . import _lib
+
+
+MIXERS = {"latent": 1, "attention": 2, "gla": 3}
 
 
 @dataclass
 class LayerSpec:
-    """Latent attention and a feed-forward, both reading their own norm of the layer's input."""
+    """One layer: a mixer and a feed-forward.
+
+    mixer "latent": latent attention; "attention": grouped-query attention with a learned distance bias, query / key
+    norms, a query temperature and a softmax sink; "gla": gated linear attention with a state per sequence.
+    """
     heads: int
-    dim: int                    # unrotated query / key features per head
-    rot_dim: int                # rotated ones; the key part is shared by all heads
+    dim: int                    # query / key features per head (latent: the unrotated ones)
     vdim: int
-    q_rank: int
-    kv_rank: int
-    scale: float
+    mixer: str = "latent"
+    scale: float = 1.0          # of the attention scores
+    out_gate: bool = True       # latent, attention: a sigmoid gate per head on the output
+    # latent
+    rot_dim: int = 0            # rotated features per head; the key part is shared by all heads
+    q_rank: int = 0
+    kv_rank: int = 0
     window: int = 0             # keys a query sees, itself included; 0: all
     rope_base: float = 10000.0
     rope_dims: int = None       # rotated features of the rot_dim part (None: all)
-    out_gate: bool = True
+    # attention
+    kv_heads: int = 0
+    kv_from: int = -1           # layer whose keys and values are used; -1: its own
+    qk_norm: bool = True
+    sink: bool = True           # a learned number per head in the softmax denominator
+    bias_rows: int = 0          # rows of the distance bias table; 0: no bias
+    bias_max: int = 0           # distance at which the buckets end
+    temp_every: int = 0         # query temperature 1 + temp_coef ln(floor((p + 1) / temp_every) + 1); 0: none
+    temp_coef: float = 0.0
+    # gla
+    decay_rank: int = 0
+    tau: float = 1.0
+    # feed-forward
     ff: str = "dense"           # "none", "dense" (gated SiLU) or "experts"
     ffn: int = 0                # hidden width of the dense feed-forward or of one expert
     experts: int = 0
     top_k: int = 0
     renormalize: bool = False   # routing weights divided by the sum of the chosen ones
     expert_gated: bool = False  # gated SiLU experts; False: W_down relu(W_up x)^2
+    router_bias: bool = False
+    shared_ffn: int = 0         # hidden width of the shared expert; 0: none
 
     def to_c(self):
         kinds = ("none", "dense", "experts")
         if self.ff not in kinds:
             raise ValueError("unknown feed-forward %r" % (self.ff,))
-        return _lib.Layer(mixer=1, heads=self.heads, dim=self.dim, rot_dim=self.rot_dim, vdim=self.vdim, q_rank=self.q_rank,
+        if self.mixer not in MIXERS:
+            raise ValueError("unknown mixer %r" % (self.mixer,))
+        return _lib.Layer(mixer=MIXERS[self.mixer], heads=self.heads, dim=self.dim, rot_dim=self.rot_dim, vdim=self.vdim, q_rank=self.q_rank,
                           kv_rank=self.kv_rank, window=self.window,
-                          rope_dims=self.rot_dim if self.rope_dims is None else self.rope_dims, out_gate=int(self.out_gate),
-                          ff=kinds.index(self.ff), ffn=self.ffn, experts=self.experts, top_k=self.top_k,
-                          renormalize=int(self.renormalize), expert_gated=int(self.expert_gated), rope_base=self.rope_base,
-                          scale=self.scale, reserved=0)
+                          rope_dims=self.rot_dim if self.rope_dims is None else self.rope_dims,
+                          out_gate=int(self.out_gate and self.mixer != "gla"), ff=kinds.index(self.ff), ffn=self.ffn,
+                          experts=self.experts, top_k=self.top_k, renormalize=int(self.renormalize),
+                          expert_gated=int(self.expert_gated), rope_base=self.rope_base, scale=self.scale, kv_heads=self.kv_heads,
+                          kv_from=self.kv_from, qk_norm=int(self.qk_norm), sink=int(self.sink), bias_rows=self.bias_rows,
+                          bias_max=self.bias_max, temp_every=self.temp_every, temp_coef=self.temp_coef, decay_rank=self.decay_rank,
+                          tau=self.tau, router_bias=int(self.router_bias), shared_ffn=self.shared_ffn)
+
+    def mixer_specs(self, d):
+        """[(name, shape)] of the mixer's tensors, Linear weights [in, out]."""
+        H, K, V = self.heads, self.dim, self.vdim
+        if self.mixer == "latent":
+            specs = [("dq", (d, self.q_rank)), ("dq.norm", (self.q_rank,)), ("uq", (self.q_rank, H * (K + self.rot_dim))),
+                     ("dkv", (d, self.kv_rank + self.rot_dim)), ("dkv.norm", (self.kv_rank,)), ("uk", (self.kv_rank, H * K)),
+                     ("uv", (self.kv_rank, H * V))]
+        elif self.mixer == "attention":
+            own = self.kv_from < 0
+            specs = [("q", (d, H * K))]
+            if own:
+                specs += [("k", (d, self.kv_heads * K)), ("v", (d, self.kv_heads * V))]
+            if self.qk_norm:
+                specs += [("q.norm", (K,))] + ([("k.norm", (K,))] if own else [])
+            if self.bias_rows:
+                specs.append(("rel", (self.bias_rows, H)))
+            if self.sink:
+                specs.append(("sink", (H,)))
+        else:
+            specs = [("q", (d, H * K)), ("k", (d, H * K)), ("v", (d, H * V)), ("a1", (d, self.decay_rank)),
+                     ("a2", (self.decay_rank, H * K)), ("a2.b", (H * K,)), ("g", (d, H * V)), ("norm", (V,))]
+        if self.out_gate and self.mixer != "gla":
+            specs.append(("g", (d, H)))
+        return specs + [("o", (H * V, d))]
+
+    def step_traffic(self, d, batch, ctx):
+        """Elements a decode step of `batch` sequences at context ctx reads or writes for the mixer, without
+        recurrent state."""
+        n = sum(s[0] * s[1] for _, s in self.mixer_specs(d) if len(s) == 2)
+        if self.mixer == "latent":
+            seen = min(ctx, self.window) if self.window else ctx
+            return n + batch * seen * (self.kv_rank + self.rot_dim)
+        if self.mixer == "attention":
+            return n + batch * ctx * self.kv_heads * (self.dim + self.vdim)
+        return n
+
+    @property
+    def state_elements(self):
+        """f32 elements of recurrent state per sequence."""
+        return self.heads * self.dim * self.vdim if self.mixer == "gla" else 0
 
 
 @dataclass
@@ -49,6 +121,8 @@ class LayeredConfig:
     eps: float = 1e-6
     loop: tuple = None          # (start, stop, times): layers[start:stop] are repeated, `times` passes in all
     norm_zero_centred: bool = True   # block and final norm weights are stored as the distance from one
+    block: str = "parallel"     # "parallel": x += mixer(norm1 x) + ff(norm2 x); "output_norm": x += norm1(mixer x), x += norm2(ff x)
+    own_head: bool = False      # the output head is a tensor of its own; False: the embedding table
     max_seq: int = 4096
     dtype: int = _lib.F32
     tp_size: int = field(default=1, init=False)
@@ -73,20 +147,18 @@ class LayeredConfig:
 
     def step_bytes(self, batch, ctx):
         """Bytes a decode step of `batch` sequences streams at context ctx: every layer run's weights (a loop reads them once
-        a pass), the lm_head, and the cache rows the windows see."""
+        a pass), the lm_head, the cache rows the windows see and the recurrent state."""
         es = 2 if self.dtype == _lib.BF16 else 4
-        d, total = self.d_model, self.d_model * self.vocab
+        d, total, state = self.d_model, self.d_model * self.vocab, 0
         for i in self.layer_runs:
             l = self.layers[i]
-            total += d * (l.q_rank + l.kv_rank + l.rot_dim + (l.heads if l.out_gate else 0)) + l.q_rank * l.heads * (l.dim + l.rot_dim)
-            total += l.kv_rank * l.heads * (l.dim + l.vdim) + l.heads * l.vdim * d
+            total += l.step_traffic(d, batch, ctx)
+            state += 2 * batch * l.state_elements          # read and written
             if l.ff == "dense":
                 total += 3 * d * l.ffn
             elif l.ff == "experts":
-                total += d * l.experts + min(l.experts, batch * l.top_k) * (3 if l.expert_gated else 2) * d * l.ffn
-            seen = min(ctx, l.window) if l.window else ctx
-            total += batch * seen * (l.kv_rank + l.rot_dim)
-        return total * es
+                total += d * l.experts + min(l.experts, batch * l.top_k) * (3 if l.expert_gated else 2) * d * l.ffn + 3 * d * l.shared_ffn
+        return total * es + state * 4
 
     def create(self, slot, out):
         """rewb200_model_create_layers into the handle `out`."""
@@ -95,7 +167,8 @@ class LayeredConfig:
                            dtype=self.dtype, tp_size=1, ep_size=1)
         arr = (_lib.Layer * self.n_layers)(*[l.to_c() for l in self.layers])
         a, b, k = self.loop or (0, 0, 0)
-        stack = _lib.Stack(loop_start=a, loop_stop=b, loop_times=k, norm_zero_centred=int(self.norm_zero_centred))
+        stack = _lib.Stack(loop_start=a, loop_stop=b, loop_times=k, norm_zero_centred=int(self.norm_zero_centred),
+                           block=("parallel", "output_norm").index(self.block), own_head=int(self.own_head))
         _lib.check(_lib.lib().rewb200_model_create_layers(slot, C.byref(base), arr, C.byref(stack), out))
 
     def tensor_specs(self):
@@ -106,14 +179,8 @@ class LayeredConfig:
             specs.append(("loop.step", (self.loop[2], d)))
         for i, l in enumerate(self.layers):
             p = "l%d." % i
-            x = p + "mix."
-            specs += [(p + "norm1", (d,)), (x + "dq", (d, l.q_rank)), (x + "dq.norm", (l.q_rank,)),
-                      (x + "uq", (l.q_rank, l.heads * (l.dim + l.rot_dim))), (x + "dkv", (d, l.kv_rank + l.rot_dim)),
-                      (x + "dkv.norm", (l.kv_rank,)), (x + "uk", (l.kv_rank, l.heads * l.dim)),
-                      (x + "uv", (l.kv_rank, l.heads * l.vdim))]
-            if l.out_gate:
-                specs.append((x + "g", (d, l.heads)))
-            specs.append((x + "o", (l.heads * l.vdim, d)))
+            specs.append((p + "norm1", (d,)))
+            specs += [(p + "mix." + n, shape) for n, shape in l.mixer_specs(d)]
             if l.ff == "none":
                 continue
             specs.append((p + "norm2", (d,)))
@@ -121,10 +188,32 @@ class LayeredConfig:
                 specs += [(p + "mlp.gate", (d, l.ffn)), (p + "mlp.up", (d, l.ffn)), (p + "mlp.down", (l.ffn, d))]
             else:
                 specs.append((p + "mlp.router", (d, l.experts)))
+                if l.router_bias:
+                    specs.append((p + "mlp.router.b", (l.experts,)))
                 for e in range(l.experts):
                     q = p + "mlp.e%d." % e
                     if l.expert_gated:
                         specs.append((q + "gate", (d, l.ffn)))
                     specs += [(q + "up", (d, l.ffn)), (q + "down", (l.ffn, d))]
+                if l.shared_ffn:
+                    q = p + "mlp.shared."
+                    specs += [(q + "gate", (d, l.shared_ffn)), (q + "up", (d, l.shared_ffn)), (q + "down", (l.shared_ffn, d))]
         specs.append(("final.norm", (d,)))
+        if self.own_head:
+            specs.append(("head", (d, self.vocab)))
         return specs
+
+    def canonical_tensors(self, tensors, tables=("embed", "loop.step", "mix.rel")):
+        """The canonical list from {name: array} of a file whose Linear weights are [out, in]; names that end in one of
+        `tables` are matrices that are no Linear and stay as they are."""
+        out = []
+        for name, shape in self.tensor_specs():
+            if name not in tensors:
+                raise KeyError("model.safetensors: missing tensor " + name)
+            t = np.asarray(tensors[name], np.float32)
+            if t.ndim == 2 and not name.endswith(tables):
+                t = t.T
+            if tuple(t.shape) != tuple(shape):
+                raise ValueError("model.safetensors: %s is %r, config.json asks for %r" % (name, t.shape, tuple(shape)))
+            out.append(np.ascontiguousarray(t))
+        return out

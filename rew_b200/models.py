@@ -19,6 +19,15 @@ def _load_rezupel(path, dtype, max_seq, slot):
     return rezupel.load(path, dtype, max_seq, slot)
 
 
+def _is_girulorn(cfg):
+    return cfg.get("architecture") == "Girulorn"
+
+
+def _load_girulorn(path, dtype, max_seq, slot):
+    from . import girulorn
+    return girulorn.load(path, dtype, max_seq, slot)
+
+
 def _is_hf_llama(cfg):
     return cfg.get("model_type") == "llama" or "LlamaForCausalLM" in (cfg.get("architectures") or [])
 
@@ -32,6 +41,7 @@ def _load_hf_llama(path, dtype, max_seq, slot):
 # (family, does this config.json name it, loader)
 FAMILIES = [
     ("rezupel", _is_rezupel, _load_rezupel),
+    ("girulorn", _is_girulorn, _load_girulorn),
     ("llama", _is_hf_llama, _load_hf_llama),
 ]
 

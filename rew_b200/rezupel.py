@@ -4,8 +4,6 @@ layers that runs several times.  Reads its config.json and maps its tensors onto
 import json
 import os
 
-import numpy as np
-
 from .layered import LayeredConfig, LayerSpec
 
 ARCHITECTURE = "Rezupel"
@@ -47,17 +45,7 @@ def config_from_json(path_or_dict, **overrides):
 
 def canonical_tensors(cfg, tensors):
     """The canonical list from {name: array}; the file's Linear weights are [out, in], the backend's [in, out]."""
-    out = []
-    for name, shape in cfg.tensor_specs():
-        if name not in tensors:
-            raise KeyError("model.safetensors: missing tensor " + name)
-        t = np.asarray(tensors[name], np.float32)
-        if t.ndim == 2 and name not in ("embed", "loop.step"):
-            t = t.T
-        if tuple(t.shape) != tuple(shape):
-            raise ValueError("model.safetensors: %s is %r, config.json asks for %r" % (name, t.shape, tuple(shape)))
-        out.append(np.ascontiguousarray(t))
-    return out
+    return cfg.canonical_tensors(tensors)
 
 
 def load(model_dir, dtype, max_seq=None, slot=0):
