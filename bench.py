@@ -21,6 +21,9 @@ data-path collective): weak scaling.
     tiny     the tiny fp32 Llama of the parity tests
     rezupel_b32, rezupel_b1, rezupel_b8_s2048, rezupel_moe_b64
              Rezupel (latent attention) at the sizes of l8_b32, l8_b1, l8_b8_s2048 and moe_b64
+    girulorn_b64, girulorn_b1, girulorn_b8_s2048
+             Girulorn (gated linear attention and attention with distance bias in turn, routed and
+             shared experts) at the sizes of moe_b64, moe_b1 and moe_b8_s2048
 
 `value` is decode tokens/s of the whole job with ids, weights and cache resident
 in HBM (CUDA events around K graph replays); `e2e` is tokens/s of one generate()
@@ -64,13 +67,18 @@ WORKLOADS = {
     # 4 / 8, no exchange): what the sharded kernels cost without the all-reduce, measurable on one GPU
     "l70_tp4shape": dict(model="llama3_70b", batch=16, prompt=1024, shape_div=4),
     "l70_tp8shape": dict(model="llama3_70b", batch=16, prompt=1024, shape_div=8),
-    # layered models (latent attention, parallel blocks) beside l8_b32 and moe_b64 at equal size: same width, heads,
-    # feed-forward or experts, as many layer runs
+    # layered models beside l8_b32 and moe_b64 at equal size: same width, heads, feed-forward or experts, as many layer
+    # runs
     "rezupel_b32": dict(model="rezupel.dense_8b", batch=32, prompt=512),
     "rezupel_b1": dict(model="rezupel.dense_8b", batch=1, prompt=512),
     "rezupel_b8_s2048": dict(model="rezupel.dense_8b", batch=8, prompt=2048),
     "rezupel_moe_b64": dict(model="rezupel.moe_lite", batch=64, prompt=256),
     "l8_b8_s2048": dict(model="llama3_8b", batch=8, prompt=2048),
+    "girulorn_b64": dict(model="girulorn.moe_lite", batch=64, prompt=256),
+    "girulorn_b1": dict(model="girulorn.moe_lite", batch=1, prompt=512),
+    "girulorn_b8_s2048": dict(model="girulorn.moe_lite", batch=8, prompt=2048),
+    "moe_b1": dict(model="deepseek_v2_lite", batch=1, prompt=512),
+    "moe_b8_s2048": dict(model="deepseek_v2_lite", batch=8, prompt=2048),
     # the attention operator alone: batch 8, 32 query / 8 kv heads, head_dim 128, 4096 positions
     "attn_op": dict(model=None, batch=8, prompt=4096),
 }
@@ -178,8 +186,9 @@ def dist_env():
 
 
 def make_cfg(name):
-    from rew_b200 import rezupel, weights as W
-    return getattr(rezupel, name.split(".")[1])() if name.startswith("rezupel.") else getattr(W, name)()
+    import importlib
+    family, _, shape = name.rpartition(".")      # "family.shape" of a layered model, or a shape of rew_b200/weights.py
+    return getattr(importlib.import_module("rew_b200." + (family or "weights")), shape)()
 
 
 def product_config(args, wl, world, model_gb=None):
@@ -189,7 +198,7 @@ def product_config(args, wl, world, model_gb=None):
     cfg = make_cfg(wl["model"])
     return {"workload": args.workload + ("" if args.layers <= 0 else "_%dlayers" % args.layers), "batch_per_gpu": per_gpu,
             "prompt": wl["prompt"], "decode_steps": args.steps, "parallelism": parallel + (str(world) if world > 1 else ""),
-            "sampling": args.sampling, "mask": "windows" if hasattr(cfg, "layer_runs") else "conventional" if cfg.mask_kind == 1 else "as_written",
+            "sampling": args.sampling, "mask": "windows" if any(getattr(l, "window", 0) for l in getattr(cfg, "layers", ())) else "conventional" if getattr(cfg, "mask_kind", 1) == 1 else "as_written",
             "norm": "rmsNorm" if getattr(cfg, "norm_kind", 0) == 0 else "LayerNorm",
             "l2": "weights streamed per step exceed the 126 MB L2"}
 
@@ -577,9 +586,9 @@ def main():
     if args.workload == "attn_op":
         run_attention_op(args, rank, local_rank)
         return
-    if args.impl == "reference" and wl["model"].startswith("rezupel."):
+    if args.impl == "reference" and "." in wl["model"]:
         if rank == 0:
-            print(json.dumps({"impl": "reference", "unavailable": "the reference has no latent-attention model"}), flush=True)
+            print(json.dumps({"impl": "reference", "unavailable": "the reference has no model of the family %s" % wl["model"].split(".")[0]}), flush=True)
         return
     if args.impl == "reference":
         run_reference(args, wl, rank, world)

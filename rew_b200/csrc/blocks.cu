@@ -432,14 +432,7 @@ int layered_set_tensor(rewb200_model* m, int64_t index, const float* host, int64
       case SL_V: return cols(G.in.w, G.in.N, 2 * hk);
       case SL_V_GATE: return cols(G.in.w, G.in.N, 2 * hk + hv);
       case SL_A1: return cols(G.in.w, G.in.N, 2 * hk + 2 * hv);
-      case SL_A2: {   // stored [rank, heads * dim], used row by row of its transpose
-        std::vector<float> w((size_t)numel);
-        for (int64_t r = 0; r < R; ++r)
-          for (int64_t i = 0; i < C; ++i) w[i * R + r] = host[r * C + i];
-        RB_CUDA(cudaMemcpyAsync(G.a2, w.data(), w.size() * sizeof(float), cudaMemcpyHostToDevice, m->c->stream));
-        RB_CUDA(cudaStreamSynchronize(m->c->stream));
-        return REWB200_OK;
-      }
+      case SL_A2: return vector(G.a2);
       case SL_A2_B: return vector(G.a2_b);
       case SL_V_NORM: return norm(G.norm, false);
       default: break;

@@ -24,15 +24,11 @@ __device__ __forceinline__ float warp_sum(float v) {
 // ln(sigmoid(z)) / tau
 __device__ __forceinline__ float log_decay(float z, float inv_tau) { return -(fmaxf(-z, 0.f) + log1pf(expf(-fabsf(z)))) * inv_tau; }
 
-__device__ __forceinline__ float slab_sum(const GlaArgs& a, const float* p, int64_t col) {
+// A column of a row summed over the slabs, in slab order.
+__device__ __forceinline__ float slab_sum(const GlaArgs& a, const float* p) {
   float v = 0.f;
-  for (int s0 = 0; s0 < a.nsplit; s0 += 8) {
-    float w[8];
-#pragma unroll
-    for (int u = 0; u < 8; ++u) w[u] = s0 + u < a.nsplit ? p[(s0 + u) * a.split_stride + col] : 0.f;
-#pragma unroll
-    for (int u = 0; u < 8; ++u) v += w[u];
-  }
+#pragma unroll 4
+  for (int s = 0; s < a.nsplit; ++s) v += p[s * a.split_stride];
   return v;
 }
 
@@ -53,23 +49,26 @@ __device__ __forceinline__ TokenSmem carve(float* sm, const GlaDims& m) {
 }
 __device__ __forceinline__ void load_token(const GlaArgs& a, const TokenSmem& s, int h, int64_t row) {
   const GlaDims& m = a.m;
+  const float qscale = rsqrtf((float)m.dim), inv_tau = 1.0f / m.tau;
   const int K = m.dim, V = m.vdim;
   const int64_t HK = (int64_t)m.heads * K, HV = (int64_t)m.heads * V;
   const float* p = a.partial + row * a.ld;
-  const int n = 2 * K + 2 * V + m.rank;
-  for (int i = threadIdx.x; i < n; i += NT) {
-    if (i < K) s.q[i] = slab_sum(a, p, (int64_t)h * K + i) * rsqrtf((float)K);
-    else if (i < 2 * K) s.k[i - K] = slab_sum(a, p, HK + (int64_t)h * K + i - K);
-    else if (i < 2 * K + V) s.v[i - 2 * K] = slab_sum(a, p, 2 * HK + (int64_t)h * V + i - 2 * K);
-    else if (i < 2 * K + 2 * V) s.g[i - 2 * K - V] = slab_sum(a, p, 2 * HK + HV + (int64_t)h * V + i - 2 * K - V);
-    else s.a1[i - 2 * K - 2 * V] = slab_sum(a, p, 2 * HK + 2 * HV + i - 2 * K - 2 * V);
+  // the decay features feed a longer chain: the last warp loads them, q, k, v and the gate go to all threads
+  if (threadIdx.x >= NT - 32)
+    for (int i = threadIdx.x - (NT - 32); i < m.rank; i += 32) s.a1[i] = slab_sum(a, p + 2 * HK + 2 * HV + i);
+  for (int i = threadIdx.x; i < 2 * K + 2 * V; i += NT) {
+    const bool key = i < 2 * K;
+    const int j = key ? i : i - 2 * K, n = key ? K : V, second = j >= n ? 1 : 0, at = j - second * n;
+    const float v = slab_sum(a, p + (key ? 0 : 2 * HK) + second * (key ? HK : HV) + (int64_t)h * n + at);
+    (key ? (second ? s.k : s.q) : (second ? s.g : s.v))[at] = key && !second ? v * qscale : v;
   }
   __syncthreads();
   for (int i = threadIdx.x; i < K; i += NT) {
-    const float* w = m.a2 + ((int64_t)h * K + i) * m.rank;
+    const float* w = m.a2 + (int64_t)h * K + i;
     float z = m.a2_b[(int64_t)h * K + i];
-    for (int r = 0; r < m.rank; ++r) z = fmaf(s.a1[r], w[r], z);
-    s.al[i] = expf(log_decay(z, 1.0f / m.tau));
+#pragma unroll 8
+    for (int r = 0; r < m.rank; ++r) z = fmaf(s.a1[r], w[r * HK], z);
+    s.al[i] = expf(log_decay(z, inv_tau));
   }
   __syncthreads();
 }

@@ -9,7 +9,7 @@ namespace rewb {
 struct GlaDims {
   int heads, dim, vdim, rank;
   float tau;
-  const float* a2;         // [heads * dim][rank] second decay projection
+  const float* a2;         // [rank][heads * dim] second decay projection
   const float* a2_b;       // [heads * dim]
   const float* norm;       // [vdim]
 };

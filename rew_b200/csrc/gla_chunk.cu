@@ -50,18 +50,17 @@ __device__ __forceinline__ void split2(float x, float y, uint32_t& hi, uint32_t&
   const __nv_bfloat162 h = *reinterpret_cast<const __nv_bfloat162*>(&hi);
   lo = pack_bf16(x - __low2float(h), y - __high2float(h));
 }
-__device__ __forceinline__ float slab(const GlaArgs& a, const float* p) {
-  float v = *p;
-  for (int s = 1; s < a.nsplit; ++s) v += p[s * a.split_stride];
-  return v;
-}
-__device__ __forceinline__ float4 slab4(const GlaArgs& a, const float* p) {
-  float4 v = *reinterpret_cast<const float4*>(p);
+// N values, `step` elements apart from one another, summed over the slabs; all loads of a slab are in flight together.
+template <int N>
+__device__ __forceinline__ void slab_n(const GlaArgs& a, const float* p, int64_t step, int n, float (&v)[N]) {
+#pragma unroll
+  for (int u = 0; u < N; ++u) v[u] = u < n ? p[u * step] : 0.f;
   for (int s = 1; s < a.nsplit; ++s) {
-    const float4 w = *reinterpret_cast<const float4*>(p + s * a.split_stride);
-    v.x += w.x; v.y += w.y; v.z += w.z; v.w += w.w;
+    p += a.split_stride;
+#pragma unroll
+    for (int u = 0; u < N; ++u)
+      if (u < n) v[u] += p[u * step];
   }
-  return v;
 }
 
 struct ChunkCfg {
@@ -96,7 +95,7 @@ __global__ void __launch_bounds__(NT, 2) gla_chunk_kernel(GlaArgs a, ChunkCfg cf
   // weights of the decay projection do not depend on earlier kernels
   for (int i = tid; i < rp * Kp; i += NT) {
     const int r = i / Kp, k = i % Kp;
-    sA2[i] = r < m.rank && k < K ? m.a2[((int64_t)h * K + k) * m.rank + r] : 0.f;
+    sA2[i] = r < m.rank && k < K ? m.a2[(int64_t)r * HK + (int64_t)h * K + k] : 0.f;
   }
   const int kc = tid & 127, half = tid >> 7;                   // this thread's key channel and half of the chunk
   const float kbias = kc < K ? m.a2_b[(int64_t)h * K + kc] : 0.f;
@@ -112,10 +111,30 @@ __global__ void __launch_bounds__(NT, 2) gla_chunk_kernel(GlaArgs a, ChunkCfg cf
       const int v = v0 + warp * 16 + g + 8 * (e >> 1), k = 8 * j + 2 * t4 + (e & 1);
       S[j][e] = p.pos0 > 0 && state_warp && v < V && k < K ? st[(int64_t)k * a.ldv + v] : 0.f;
     }
+  // items of four columns this thread handles of a [C][vs] tile: one column group, tokens vt, vt + vstep, ..
+  const int vq = vs / 4, vt = tid / vq, vc = (tid % vq) * 4, vstep = NT / vq;   // vs <= 128: at most 4 items
+  auto tile4 = [&](const float* base, int nt, float4 (&x)[4]) {
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const int t = vt + i * vstep;
+      x[i] = vt < vstep && t < nt && v0 + vc < V ? *reinterpret_cast<const float4*>(base + (int64_t)t * a.ld + vc) : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+    for (int s = 1; s < a.nsplit; ++s)
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        const int t = vt + i * vstep;
+        if (vt < vstep && t < nt && v0 + vc < V) {
+          const float4 w = *reinterpret_cast<const float4*>(base + s * a.split_stride + (int64_t)t * a.ld + vc);
+          x[i].x += w.x; x[i].y += w.y; x[i].z += w.z; x[i].w += w.w;
+        }
+      }
+  };
   auto load_a1 = [&](int t0, float* dst) {
     for (int i = tid; i < C * rp; i += NT) {
       const int t = i / rp, r = i % rp;
-      dst[i] = t0 + t < p.n && r < m.rank ? slab(a, a.partial + (int64_t)(p.row0 + t0 + t) * a.ld + 2 * HK + 2 * HV + r) : 0.f;
+      float v[1] = {0.f};
+      if (t0 + t < p.n && r < m.rank) slab_n<1>(a, a.partial + (int64_t)(p.row0 + t0 + t) * a.ld + 2 * HK + 2 * HV + r, 0, 1, v);
+      dst[i] = v[0];
     }
   };
   load_a1(0, sA1);
@@ -126,11 +145,14 @@ __global__ void __launch_bounds__(NT, 2) gla_chunk_kernel(GlaArgs a, ChunkCfg cf
     const float* a1 = sA1 + (it & 1) * C * rp;
     const float* base = a.partial + (int64_t)(p.row0 + t0) * a.ld;
     // ---- values
-    for (int i = tid; i < C * vs / 4; i += NT) {
-      const int t = i / (vs / 4), v = (i % (vs / 4)) * 4;
-      float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
-      if (t < nt && v0 + v < V) x = slab4(a, base + (int64_t)t * a.ld + 2 * HK + (int64_t)h * V + v0 + v);
-      *reinterpret_cast<uint2*>(sV + t * ldv + v) = make_uint2(pack_bf16(x.x, x.y), pack_bf16(x.z, x.w));
+    {
+      float4 x[4];
+      tile4(base + 2 * HK + (int64_t)h * V + v0, nt, x);
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        const int t = vt + i * vstep;
+        if (vt < vstep && t < C) *reinterpret_cast<uint2*>(sV + t * ldv + vc) = make_uint2(pack_bf16(x[i].x, x[i].y), pack_bf16(x[i].z, x[i].w));
+      }
     }
     // ---- decays and scaled queries and keys of this thread's channel, 16 tokens
     bool far = false;
@@ -170,19 +192,21 @@ __global__ void __launch_bounds__(NT, 2) gla_chunk_kernel(GlaArgs a, ChunkCfg cf
         }
       }
       const float* qp = base + (int64_t)half * 16 * a.ld + (int64_t)h * K + kc;
+      const int nu = kc < K ? nt - half * 16 : 0;
 #pragma unroll
-      for (int u = 0; u < 16; ++u) {
-        const int t = half * 16 + u;
-        float q = 0.f, k = 0.f;
-        if (t < nt && kc < K) {
-          q = slab(a, qp + (int64_t)u * a.ld);
-          k = slab(a, qp + (int64_t)u * a.ld + HK);
+      for (int w = 0; w < 16; w += 8) {
+        float q[8], k[8];
+        slab_n<8>(a, qp + (int64_t)w * a.ld, a.ld, nu - w, q);
+        slab_n<8>(a, qp + (int64_t)w * a.ld + HK, a.ld, nu - w, k);
+#pragma unroll
+        for (int u = 0; u < 8; ++u) {
+          const int t = half * 16 + w + u;
+          const float f = far ? 0.f : ex2(e[w + u]), fi = far ? 0.f : ex2(-e[w + u]);
+          bf16* dq = sQ + t * ldq + kc;
+          bf16* dk = sK + t * ldq + kc;
+          split(q[u] * qscale * f, dq[0], dq[C * ldq]);
+          split(k[u] * fi, dk[0], dk[C * ldq]);
         }
-        const float f = far ? 0.f : ex2(e[u]), fi = far ? 0.f : ex2(-e[u]);
-        bf16* dq = sQ + t * ldq + kc;
-        bf16* dk = sK + t * ldq + kc;
-        split(q * qscale * f, dq[0], dq[C * ldq]);
-        split(k * fi, dk[0], dk[C * ldq]);
       }
     }
     const bool slow = __syncthreads_or(far ? 1 : 0) != 0;
@@ -318,8 +342,10 @@ __global__ void __launch_bounds__(NT, 2) gla_chunk_kernel(GlaArgs a, ChunkCfg cf
           float q = 0.f, kk = 0.f, al = 0.f;
           if (k < K) {
             const float* qp = base + (int64_t)t * a.ld + (int64_t)h * K + k;
-            q = slab(a, qp) * qscale;
-            kk = slab(a, qp + HK);
+            float y[2];
+            slab_n<2>(a, qp, HK, 2, y);
+            q = y[0] * qscale;
+            kk = y[1];
             float z = m.a2_b[(int64_t)h * K + k];
             for (int r = 0; r < rp; ++r) z = fmaf(a1[t * rp + r], sA2[r * Kp + k], z);
             al = ex2((fmaxf(-z, 0.f) + log1pf(ex2(-LOG2E * fabsf(z)))) * dscale);
@@ -361,6 +387,9 @@ __global__ void __launch_bounds__(NT, 2) gla_chunk_kernel(GlaArgs a, ChunkCfg cf
         __syncthreads();
       }
     }
+    // the gates are requested ahead of the barrier
+    float4 gz[4];
+    tile4(base + 2 * HK + HV + (int64_t)h * V + v0, nt, gz);
     __syncthreads();
     // ---- norm over the head, gate, store
     if (tid < C) {
@@ -370,20 +399,21 @@ __global__ void __launch_bounds__(NT, 2) gla_chunk_kernel(GlaArgs a, ChunkCfg cf
     }
     if constexpr (CLUSTER) cg::this_cluster().sync();
     else __syncthreads();
-    for (int i = tid; i < nt * vs / 4; i += NT) {
-      const int t = i / (vs / 4), v = (i % (vs / 4)) * 4;
-      if (v0 + v >= V) continue;
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const int t = vt + i * vstep;
+      if (vt >= vstep || t >= nt || v0 + vc >= V) continue;
       float ss = sS[(it & 1) * C + t];
       if constexpr (CLUSTER) {
         ss = 0.f;
         for (unsigned r = 0; r < gridDim.x; ++r) ss += cg::this_cluster().map_shared_rank(sS, r)[(it & 1) * C + t];
       }
       const float f = 1.0f / sqrtf(ss / (float)V + a.eps);
-      const float4 gz = slab4(a, base + (int64_t)t * a.ld + 2 * HK + HV + (int64_t)h * V + v0 + v);
-      const float4 x = *reinterpret_cast<const float4*>(sO + t * ldO + v), w = *reinterpret_cast<const float4*>(m.norm + v0 + v);
+      const float4 x = *reinterpret_cast<const float4*>(sO + t * ldO + vc), w = *reinterpret_cast<const float4*>(m.norm + v0 + vc);
       auto silu = [](float z) { return z / (1.0f + __expf(-z)); };
-      *reinterpret_cast<uint2*>(reinterpret_cast<bf16*>(a.out) + (int64_t)(p.row0 + t0 + t) * a.ldo + (int64_t)h * V + v0 + v) =
-          make_uint2(pack_bf16(x.x * f * w.x * silu(gz.x), x.y * f * w.y * silu(gz.y)), pack_bf16(x.z * f * w.z * silu(gz.z), x.w * f * w.w * silu(gz.w)));
+      *reinterpret_cast<uint2*>(reinterpret_cast<bf16*>(a.out) + (int64_t)(p.row0 + t0 + t) * a.ldo + (int64_t)h * V + v0 + vc) =
+          make_uint2(pack_bf16(x.x * f * w.x * silu(gz[i].x), x.y * f * w.y * silu(gz[i].y)),
+                     pack_bf16(x.z * f * w.z * silu(gz[i].z), x.w * f * w.w * silu(gz[i].w)));
     }
     __syncthreads();
   }

@@ -59,72 +59,101 @@ __device__ __forceinline__ void put4(T* d, int i, int n, float4 v) {
   for (int u = 0; u < 4 && i + u < n; ++u) d[i + u] = stf<T>(e[u]);
 }
 
-// One warp per head: query heads, key heads, value heads, then one warp for all gates.  A lane holds four columns at a
-// time, PC of them (dim and vdim up to 128 PC).
-template <typename T, int PC>
-__global__ void __launch_bounds__(256) gqa_post_kernel(GqaPostArgs a) {
+// One warp per head: query heads, key heads, value heads, then one warp for all gates; RW rows each, requested together.
+// A lane holds four columns at a time, PC of them (dim and vdim up to 128 PC).
+template <typename T, int PC, int RW>
+__global__ void __launch_bounds__(256) gqa_post_kernel(GqaPostArgs a, int64_t rows) {
   pdl_launch_dependents();
-  const int64_t row = blockIdx.x;
+  const int64_t row0 = (int64_t)blockIdx.x * RW;
+  const int nr = (int)min((int64_t)RW, rows - row0);
   const int unit = blockIdx.y * 8 + (threadIdx.x >> 5), ln = threadIdx.x & 31;
   const int H = a.m.heads, G = a.m.own_kv ? a.m.kv_heads : 0, K = a.m.dim, V = a.m.vdim;
   if (!a.early) pdl_wait();
-  const int pos = row_pos(a.map, row), lane = row_lane(a.map, row);
-  const bool ok = pos >= 0 && pos < a.capacity;
-  const int page = a.block_table[(int64_t)lane * a.max_pages + (ok ? pos / PAGE_TOKENS : 0)];
+  int pos[RW], page[RW];
+  bool ok[RW];
+#pragma unroll
+  for (int r = 0; r < RW; ++r) {
+    const int64_t row = row0 + min(r, nr - 1);
+    pos[r] = row_pos(a.map, row);
+    ok[r] = pos[r] >= 0 && pos[r] < a.capacity;
+    page[r] = a.block_table[(int64_t)row_lane(a.map, row) * a.max_pages + (ok[r] ? pos[r] / PAGE_TOKENS : 0)];
+    if (!ok[r] && unit == 0 && ln == 0) atomicExch(a.status, KS_BAD_INDEX);
+  }
   if (a.early) pdl_wait();
   if (unit > H + 2 * G || (unit == H + 2 * G && !a.m.gate)) return;
-  if (!ok && unit == 0 && ln == 0) atomicExch(a.status, KS_BAD_INDEX);
-  const float* p = a.partial + row * a.ld;
+  const float* p = a.partial + row0 * a.ld;
   if (unit == H + 2 * G) {
     p += (int64_t)H * K + (int64_t)G * (K + V);
-    for (int h = ln; h < H; h += 32) {
+    for (int i = ln; i < nr * H; i += 32) {
+      const int r = i / H, h = i % H;
       float z = 0.f;
-      for (int s = 0; s < a.nsplit; ++s) z += p[s * a.split_stride + h];
-      a.gate[row * H + h] = sigmoid(z);
+      for (int s = 0; s < a.nsplit; ++s) z += p[s * a.split_stride + r * a.ld + h];
+      a.gate[(row0 + r) * H + h] = sigmoid(z);
     }
     return;
   }
   const bool is_q = unit < H, is_v = unit >= H + G;
   const int n = is_v ? V : K;
   const int64_t col = is_v ? (int64_t)(H + G) * K + (int64_t)(unit - H - G) * V : (int64_t)unit * K;
-  const bool vec = col % 4 == 0 && a.ld % 4 == 0 && a.split_stride % 4 == 0;
-  float4 x[PC];
-  float ss = 0.f;
+  const bool vec = col % 4 == 0 && n % 4 == 0 && a.ld % 4 == 0;
+  float4 x[RW][PC];
+  if (vec) {
+#pragma unroll
+    for (int r = 0; r < RW; ++r)
+#pragma unroll
+      for (int c = 0; c < PC; ++c) {
+        const int i = (c * 32 + ln) * 4;
+        x[r][c] = r < nr && i < n ? *reinterpret_cast<const float4*>(p + r * a.ld + col + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+      }
+#pragma unroll 4
+    for (int s = 1; s < a.nsplit; ++s)
+#pragma unroll
+      for (int r = 0; r < RW; ++r)
+#pragma unroll
+        for (int c = 0; c < PC; ++c) {
+          const int i = (c * 32 + ln) * 4;
+          if (r < nr && i < n) {
+            const float4 w = *reinterpret_cast<const float4*>(p + s * a.split_stride + r * a.ld + col + i);
+            x[r][c].x += w.x; x[r][c].y += w.y; x[r][c].z += w.z; x[r][c].w += w.w;
+          }
+        }
+  } else {
+#pragma unroll
+    for (int r = 0; r < RW; ++r)
+#pragma unroll
+      for (int c = 0; c < PC; ++c) x[r][c] = r < nr ? slab4(a, p + r * a.ld + col, (c * 32 + ln) * 4, n, false) : make_float4(0.f, 0.f, 0.f, 0.f);
+  }
+  const float* w = is_v ? nullptr : is_q ? a.m.q_norm : a.m.k_norm;
+  float4 g[PC];
 #pragma unroll
   for (int c = 0; c < PC; ++c) {
-    x[c] = slab4(a, p + col, (c * 32 + ln) * 4, n, vec);
-    ss += x[c].x * x[c].x + x[c].y * x[c].y + x[c].z * x[c].z + x[c].w * x[c].w;
+    const int i = (c * 32 + ln) * 4;
+    g[c] = make_float4(1.f, 1.f, 1.f, 1.f);
+    if (w) g[c] = make_float4(i < n ? w[i] : 0.f, i + 1 < n ? w[i + 1] : 0.f, i + 2 < n ? w[i + 2] : 0.f, i + 3 < n ? w[i + 3] : 0.f);
   }
-  const float* w = is_q ? a.m.q_norm : a.m.k_norm;
-  if (!is_v && w) {
-    float f = 1.0f / sqrtf(warp_sum(ss) / (float)K + a.eps);
-    if (is_q && a.m.temp_every > 0) f *= 1.0f + a.m.temp_coef * logf((float)((pos + 1) / a.m.temp_every + 1));
 #pragma unroll
-    for (int c = 0; c < PC; ++c) {
-      const int i = (c * 32 + ln) * 4;
-      float4 g = make_float4(0.f, 0.f, 0.f, 0.f);
-      if (i < n) g.x = w[i];
-      if (i + 1 < n) g.y = w[i + 1];
-      if (i + 2 < n) g.z = w[i + 2];
-      if (i + 3 < n) g.w = w[i + 3];
-      x[c] = make_float4(x[c].x * f * g.x, x[c].y * f * g.y, x[c].z * f * g.z, x[c].w * f * g.w);
+  for (int r = 0; r < RW; ++r) {
+    if (r >= nr) break;
+    float f = 1.f;
+    if (w) {
+      float ss = 0.f;
+#pragma unroll
+      for (int c = 0; c < PC; ++c) ss += x[r][c].x * x[r][c].x + x[r][c].y * x[r][c].y + x[r][c].z * x[r][c].z + x[r][c].w * x[r][c].w;
+      f = 1.0f / sqrtf(warp_sum(ss) / (float)K + a.eps);
     }
-  } else if (is_q && a.m.temp_every > 0) {
-    const float f = 1.0f + a.m.temp_coef * logf((float)((pos + 1) / a.m.temp_every + 1));
+    if (is_q && a.m.temp_every > 0) f *= 1.0f + a.m.temp_coef * logf((float)((pos[r] + 1) / a.m.temp_every + 1));
+    T* dst;
+    if (is_q) {
+      dst = reinterpret_cast<T*>(a.q) + (row0 + r) * a.ldq + (int64_t)unit * K;
+    } else {
+      if (!ok[r]) continue;
+      const int64_t crow = ((int64_t)page[r] * G + (is_v ? unit - H - G : unit - H)) * PAGE_TOKENS + pos[r] % PAGE_TOKENS;
+      dst = is_v ? reinterpret_cast<T*>(a.vc) + crow * a.ldv : reinterpret_cast<T*>(a.kc) + crow * a.ldk;
+    }
 #pragma unroll
-    for (int c = 0; c < PC; ++c) x[c] = make_float4(x[c].x * f, x[c].y * f, x[c].z * f, x[c].w * f);
+    for (int c = 0; c < PC; ++c)
+      put4<T>(dst, (c * 32 + ln) * 4, n, make_float4(x[r][c].x * f * g[c].x, x[r][c].y * f * g[c].y, x[r][c].z * f * g[c].z, x[r][c].w * f * g[c].w));
   }
-  T* dst;
-  if (is_q) {
-    dst = reinterpret_cast<T*>(a.q) + row * a.ldq + (int64_t)unit * K;
-  } else {
-    if (!ok) return;
-    const int g = is_v ? unit - H - G : unit - H;
-    const int64_t crow = ((int64_t)page * G + g) * PAGE_TOKENS + pos % PAGE_TOKENS;
-    dst = is_v ? reinterpret_cast<T*>(a.vc) + crow * a.ldv : reinterpret_cast<T*>(a.kc) + crow * a.ldk;
-  }
-#pragma unroll
-  for (int c = 0; c < PC; ++c) put4<T>(dst, (c * 32 + ln) * 4, n, x[c]);
 }
 
 // ------------------------------------------------------------------ plain attention: one CTA per (row of a tile, head),
@@ -276,6 +305,8 @@ __global__ void __launch_bounds__(160) gqa_attn_kernel(const __grid_constant__ C
   for (int k = 0; k < KS; ++k)
     if (k < ks)
       ldmatrix_x4(qf[k][0], qf[k][1], qf[k][2], qf[k][3], q_base + (k >> 2) * 2048 + swz128((lq & 1) * 8 + l8, (k & 3) * 2 + (lq >> 1)));
+  const int rows_in = ntok * cf.heads_per;          // rows in use come first
+  const int nr = rows_in > 8 ? 2 : 1;
   // this thread's rows: g and g + 8
   const float sl2 = a.m.scale * LOG2E;
   int spos[2];
@@ -322,15 +353,17 @@ __global__ void __launch_bounds__(160) gqa_attn_kernel(const __grid_constant__ C
     for (int n = 0; n < 2; ++n)
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
+        if ((e >> 1) >= nr) continue;
         const int r = e >> 1, dist = spos[r] - (key0 + n * 8 + (e & 1));
         float b = far[r];
         if (!inside && tab[r] && dist >= 0) b = __ldg(tab[r] + min(dist, a.m.n_bias - 1)) * LOG2E;
         sc[n][e] = dist >= 0 ? fmaf(sc[n][e], sl2, b) : -INFINITY;
         mx[r] = fmaxf(mx[r], sc[n][e]);
       }
-    float alpha[2], muse[2];
+    float alpha[2] = {1.f, 1.f}, muse[2] = {0.f, 0.f};
 #pragma unroll
     for (int r = 0; r < 2; ++r) {
+      if (r >= nr) break;
       mx[r] = fmaxf(mx[r], __shfl_xor_sync(0xffffffffu, mx[r], 1));
       mx[r] = fmaxf(mx[r], __shfl_xor_sync(0xffffffffu, mx[r], 2));
       const float mn = fmaxf(mrun[r], mx[r]);
@@ -338,12 +371,13 @@ __global__ void __launch_bounds__(160) gqa_attn_kernel(const __grid_constant__ C
       alpha[r] = ex2(mrun[r] - muse[r]);
       mrun[r] = mn;
     }
-    uint32_t pf[4];
+    uint32_t pf[4] = {0u, 0u, 0u, 0u};
     float ps[2] = {0.f, 0.f};
 #pragma unroll
     for (int n = 0; n < 2; ++n)
 #pragma unroll
       for (int r = 0; r < 2; ++r) {
+        if (r >= nr) break;
         const float p0 = ex2(sc[n][2 * r] - muse[r]), p1 = ex2(sc[n][2 * r + 1] - muse[r]);
         ps[r] += p0 + p1;
         pf[n * 2 + r] = pack_bf16(p0, p1);
@@ -357,8 +391,10 @@ __global__ void __launch_bounds__(160) gqa_attn_kernel(const __grid_constant__ C
         for (int n = 0; n < 2; ++n) {
           acc[j][n][0] *= alpha[0];
           acc[j][n][1] *= alpha[0];
-          acc[j][n][2] *= alpha[1];
-          acc[j][n][3] *= alpha[1];
+          if (nr > 1) {
+            acc[j][n][2] *= alpha[1];
+            acc[j][n][3] *= alpha[1];
+          }
         }
     }
 #pragma unroll
@@ -392,38 +428,49 @@ __global__ void __launch_bounds__(160) gqa_attn_kernel(const __grid_constant__ C
     for (int n = 0; n < 2; ++n)
 #pragma unroll
       for (int r = 0; r < 2; ++r)
-        *reinterpret_cast<float2*>(sO + (warp * 16 + g + 8 * r) * ldO + j * 16 + n * 8 + 2 * t) = make_float2(acc[j][n][2 * r], acc[j][n][2 * r + 1]);
+        if (g + 8 * r < rows_in) *reinterpret_cast<float2*>(sO + (warp * 16 + g + 8 * r) * ldO + j * 16 + n * 8 + 2 * t) = make_float2(acc[j][n][2 * r], acc[j][n][2 * r + 1]);
   }
   consumers_sync();
-  const int V = a.m.vdim, v2 = V / 2;   // vdim is a multiple of 8
-  for (int i = tid; i < 16 * v2; i += 128) {
-    const int m = i / v2, c = (i % v2) * 2, tok = m / cf.heads_per, hh = m % cf.heads_per;
-    if (tok >= ntok || hh >= nh) continue;
+  const int V = a.m.vdim;   // a multiple of 8
+  const bool last = gridDim.x == 1;
+  for (int mrow = warp; mrow < rows_in; mrow += 4) {
+    const int tok = mrow / cf.heads_per, hh = mrow - tok * cf.heads_per;
+    if (hh >= nh) continue;
     const int h = head0 + hh;
     const int64_t row = row0 + tok;
-    const bool last = gridDim.x == 1;
-    float M = last ? sink_l2(a.m, h) : -INFINITY;
-#pragma unroll
-    for (int w = 0; w < 4; ++w) M = fmaxf(M, sM[w * 16 + m]);
-    const float mu = M == -INFINITY ? 0.f : M;
-    float l = 0.f;
-    float2 o = make_float2(0.f, 0.f);
+    float mw[4], M = last ? sink_l2(a.m, h) : -INFINITY;
 #pragma unroll
     for (int w = 0; w < 4; ++w) {
-      const float f = ex2(sM[w * 16 + m] - mu);
-      const float2 x = *reinterpret_cast<const float2*>(sO + (w * 16 + m) * ldO + c);
-      l += f * sM[64 + w * 16 + m];
-      o.x += f * x.x;
-      o.y += f * x.y;
+      mw[w] = sM[w * 16 + mrow];
+      M = fmaxf(M, mw[w]);
     }
+    const float mu = M == -INFINITY ? 0.f : M;
+    float l = 0.f;
+#pragma unroll
+    for (int w = 0; w < 4; ++w) {
+      mw[w] = ex2(mw[w] - mu);
+      l += mw[w] * sM[64 + w * 16 + mrow];
+    }
+    float inv = 1.f;
+    const int64_t u = (row * a.m.heads + h) * a.kv_splits + blockIdx.x;
     if (last) {
       if (a.m.sink) l += ex2(sink_l2(a.m, h) - mu);
-      const float inv = (a.m.gate ? a.gate[row * a.m.heads + h] : 1.0f) / l;
-      *reinterpret_cast<uint32_t*>(reinterpret_cast<bf16*>(a.out) + row * a.ldo + (int64_t)h * V + c) = pack_bf16(o.x * inv, o.y * inv);
-    } else {
-      const int64_t u = (row * a.m.heads + h) * a.kv_splits + blockIdx.x;
-      *reinterpret_cast<float2*>(a.o_part + u * V + c) = o;
-      if (c == 0) a.ml[u] = make_float2(M, l);
+      inv = (a.m.gate ? a.gate[row * a.m.heads + h] : 1.0f) / l;
+    } else if (lane == 0) {
+      a.ml[u] = make_float2(M, l);
+    }
+    for (int c = lane * 4; c < V; c += 128) {
+      float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+      for (int w = 0; w < 4; ++w) {
+        const float4 x = *reinterpret_cast<const float4*>(sO + (w * 16 + mrow) * ldO + c);
+        o.x += mw[w] * x.x; o.y += mw[w] * x.y; o.z += mw[w] * x.z; o.w += mw[w] * x.w;
+      }
+      if (last)
+        *reinterpret_cast<uint2*>(reinterpret_cast<bf16*>(a.out) + row * a.ldo + (int64_t)h * V + c) =
+            make_uint2(pack_bf16(o.x * inv, o.y * inv), pack_bf16(o.z * inv, o.w * inv));
+      else
+        *reinterpret_cast<float4*>(a.o_part + u * V + c) = o;
     }
   }
 }
@@ -490,12 +537,11 @@ int gqa_post_launch(Ctx* c, const GqaPostArgs& a, int64_t rows) {
   if (rows == 0) return REWB200_OK;
   const int units = a.m.heads + (a.m.own_kv ? 2 * a.m.kv_heads : 0) + (a.m.gate ? 1 : 0);
   RB_REQUIRE(a.m.dim <= 512 && a.m.vdim <= 512, "grouped-query attention: head sizes above 512");
-  const dim3 grid((unsigned)rows, (unsigned)((units + 7) / 8));
-  const bool small = a.m.dim <= 128 && a.m.vdim <= 128, bf = a.dtype == REWB200_BF16;
-  RB_CUDA(bf ? (small ? launch_k(gqa_post_kernel<bf16, 1>, grid, dim3(256), 0, c->stream, c->use_pdl, a)
-                      : launch_k(gqa_post_kernel<bf16, 4>, grid, dim3(256), 0, c->stream, c->use_pdl, a))
-             : (small ? launch_k(gqa_post_kernel<float, 1>, grid, dim3(256), 0, c->stream, c->use_pdl, a)
-                      : launch_k(gqa_post_kernel<float, 4>, grid, dim3(256), 0, c->stream, c->use_pdl, a)));
+  const bool small = a.m.dim <= 128 && a.m.vdim <= 128, bf = a.dtype == REWB200_BF16, many = small && bf && rows >= 512;
+  const dim3 grid((unsigned)(many ? (rows + 3) / 4 : rows), (unsigned)((units + 7) / 8));
+  auto go = [&](auto kernel) { return launch_k(kernel, grid, dim3(256), 0, c->stream, c->use_pdl, a, rows); };
+  RB_CUDA(many ? go(gqa_post_kernel<bf16, 1, 4>) : bf ? (small ? go(gqa_post_kernel<bf16, 1, 1>) : go(gqa_post_kernel<bf16, 4, 1>))
+          : small ? go(gqa_post_kernel<float, 1, 1>) : go(gqa_post_kernel<float, 4, 1>));
   ++g_launch_total;
   return REWB200_OK;
 }
