@@ -229,7 +229,7 @@ __device__ __forceinline__ float sink_l2(const GqaDims& m, int h) { return m.sin
 
 // KS: 16-feature steps of a key row, VG: 16-column groups of a value row.
 template <int KS, int VG>
-__global__ void __launch_bounds__(160) gqa_attn_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_constant__ CUtensorMap tm_v,
+__global__ void __launch_bounds__(160, KS <= 8 ? 3 : 1) gqa_attn_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_constant__ CUtensorMap tm_v,
                                                        GqaAttnArgs a, GqaCfg cf) {
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
@@ -527,7 +527,7 @@ GqaCfg config(const GqaDims& m, int max_tile_rows) {
   cf.hgroups = (group + cf.heads_per - 1) / cf.heads_per;
   cf.tokens_per = std::min(max_tile_rows, std::max(1, 16 / cf.heads_per));
   cf.subtiles = (max_tile_rows + cf.tokens_per - 1) / cf.tokens_per;
-  cf.stages = std::min(4, std::max(2, (int)(104 * 1024 / ((cf.nb_k + cf.nb_v) * 8192))));
+  cf.stages = std::min(4, std::max(2, (int)(64 * 1024 / ((cf.nb_k + cf.nb_v) * 8192))));
   return cf;
 }
 
