@@ -40,29 +40,21 @@ __device__ __forceinline__ float ex2(float x) {
 __device__ __forceinline__ void ldmatrix_x2(uint32_t& r0, uint32_t& r1, uint32_t addr) {
   asm volatile("ldmatrix.sync.aligned.m8n8.x2.shared.b16 {%0,%1}, [%2];" : "=r"(r0), "=r"(r1) : "r"(addr));
 }
-// x = hi + lo, both bf16
-__device__ __forceinline__ void split(float x, bf16& hi, bf16& lo) {
-  hi = __float2bfloat16_rn(x);
-  lo = __float2bfloat16_rn(x - __bfloat162float(hi));
+// -log2(sigmoid(z)): log1p of a small argument by its series, where 1 + u would round it away
+__device__ __forceinline__ float neg_log2_sigmoid(float z) {
+  const float u = ex2(-LOG2E * fabsf(z));
+  float l;
+  asm("lg2.approx.ftz.f32 %0, %1;" : "=f"(l) : "f"(1.0f + u));
+  const float series = u * LOG2E * fmaf(u, fmaf(u, 0.33333333f, -0.5f), 1.0f);
+  return fmaf(fmaxf(-z, 0.f), LOG2E, u < 0.015625f ? series : l);
 }
+__device__ __forceinline__ void prefetch_l2(const void* p) { asm volatile("prefetch.global.L2 [%0];" ::"l"(p)); }
+// x, y = hi + lo, packed bf16 pairs
 __device__ __forceinline__ void split2(float x, float y, uint32_t& hi, uint32_t& lo) {
   hi = pack_bf16(x, y);
   const __nv_bfloat162 h = *reinterpret_cast<const __nv_bfloat162*>(&hi);
   lo = pack_bf16(x - __low2float(h), y - __high2float(h));
 }
-// N values, `step` elements apart from one another, summed over the slabs; all loads of a slab are in flight together.
-template <int N>
-__device__ __forceinline__ void slab_n(const GlaArgs& a, const float* p, int64_t step, int n, float (&v)[N]) {
-#pragma unroll
-  for (int u = 0; u < N; ++u) v[u] = u < n ? p[u * step] : 0.f;
-  for (int s = 1; s < a.nsplit; ++s) {
-    p += a.split_stride;
-#pragma unroll
-    for (int u = 0; u < N; ++u)
-      if (u < n) v[u] += p[u * step];
-  }
-}
-
 struct ChunkCfg {
   int kt;        // 16-channel steps of a key: dim padded to 16 kt
   int vs;        // value columns of the CTA, a multiple of 16
@@ -82,9 +74,10 @@ __global__ void __launch_bounds__(NT, 2) gla_chunk_kernel(GlaArgs a, ChunkCfg cf
   bf16* sK = reinterpret_cast<bf16*>(smem + cf.off_k);         // [hi, lo][C][ldq]
   bf16* sV = reinterpret_cast<bf16*>(smem + cf.off_v);         // [C][ldv]
   bf16* sA = reinterpret_cast<bf16*>(smem + cf.off_a);         // [hi, lo][C][C + 8]
-  float* sA1 = reinterpret_cast<float*>(smem + cf.off_a1);     // [2][C][rp]
+  float* sA1 = reinterpret_cast<float*>(smem + cf.off_a1);     // [2][a1_at(C, 0)]
   float* sA2 = reinterpret_cast<float*>(smem + cf.off_a2);     // [rp][Kp]
-  float* sF = reinterpret_cast<float*>(smem + cf.off_f);       // [2][Kp] decays of the halves
+  float* sF = reinterpret_cast<float*>(smem + cf.off_f);       // [Kp] decay up to the middle since the state was scaled last
+  float* sEnd = sF + Kp;                                       // [2][Kp] decay after the middle, by chunk parity
   float* sS = reinterpret_cast<float*>(smem + cf.off_ss);      // [2][C] sums of squares (cluster), then [8 warps][C]
   constexpr int ldA = C + 8;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, l8 = lane & 7, lq = lane >> 3, g = lane >> 2, t4 = lane & 3;
@@ -97,8 +90,16 @@ __global__ void __launch_bounds__(NT, 2) gla_chunk_kernel(GlaArgs a, ChunkCfg cf
     const int r = i / Kp, k = i % Kp;
     sA2[i] = r < m.rank && k < K ? m.a2[(int64_t)r * HK + (int64_t)h * K + k] : 0.f;
   }
-  const int kc = tid & 127, half = tid >> 7;                   // this thread's key channel and half of the chunk
-  const float kbias = kc < K ? m.a2_b[(int64_t)h * K + kc] : 0.f;
+  // this thread's pair of key channels and eight tokens: a warp has 32 channels of one half of the chunk, its upper lanes
+  // the later eight tokens
+  const int half = warp >> 2, kc = (warp & 3) * 32 + (lane & 15) * 2, late = lane >> 4, tb = half * 16 + late * 8;
+  const bool mine = kc < Kp, live = kc < K;
+  const uint32_t pair = __ballot_sync(0xffffffffu, mine);      // both lanes of a channel pair are in or out together
+  const float2 kbias = live ? *reinterpret_cast<const float2*>(m.a2_b + (int64_t)h * K + kc) : make_float2(0.f, 0.f);
+  for (int k = tid; k < Kp; k += NT) sEnd[Kp + k] = 1.f;       // the chunk before the first one
+  // rows of decay features, with a gap every eight of them so that two groups of lanes read different banks
+  auto a1_at = [rp](int t, int r) { return t * rp + (t >> 3) * 4 + r; };
+  const int a1_size = a1_at(C, 0), ld = (int)a.ld;
   pdl_wait();
   const GlaPortion p = a.list[blockIdx.z];
   float* st = a.state + ((int64_t)p.lane * m.heads + h) * K * a.ldv;
@@ -117,14 +118,14 @@ __global__ void __launch_bounds__(NT, 2) gla_chunk_kernel(GlaArgs a, ChunkCfg cf
 #pragma unroll
     for (int i = 0; i < 4; ++i) {
       const int t = vt + i * vstep;
-      x[i] = vt < vstep && t < nt && v0 + vc < V ? *reinterpret_cast<const float4*>(base + (int64_t)t * a.ld + vc) : make_float4(0.f, 0.f, 0.f, 0.f);
+      x[i] = vt < vstep && t < nt && v0 + vc < V ? *reinterpret_cast<const float4*>(base + (int64_t)t * ld + vc) : make_float4(0.f, 0.f, 0.f, 0.f);
     }
     for (int s = 1; s < a.nsplit; ++s)
 #pragma unroll
       for (int i = 0; i < 4; ++i) {
         const int t = vt + i * vstep;
         if (vt < vstep && t < nt && v0 + vc < V) {
-          const float4 w = *reinterpret_cast<const float4*>(base + s * a.split_stride + (int64_t)t * a.ld + vc);
+          const float4 w = *reinterpret_cast<const float4*>(base + s * a.split_stride + (int64_t)t * ld + vc);
           x[i].x += w.x; x[i].y += w.y; x[i].z += w.z; x[i].w += w.w;
         }
       }
@@ -132,17 +133,22 @@ __global__ void __launch_bounds__(NT, 2) gla_chunk_kernel(GlaArgs a, ChunkCfg cf
   auto load_a1 = [&](int t0, float* dst) {
     for (int i = tid; i < C * rp; i += NT) {
       const int t = i / rp, r = i % rp;
-      float v[1] = {0.f};
-      if (t0 + t < p.n && r < m.rank) slab_n<1>(a, a.partial + (int64_t)(p.row0 + t0 + t) * a.ld + 2 * HK + 2 * HV + r, 0, 1, v);
-      dst[i] = v[0];
+      float v = 0.f;
+      if (t0 + t < p.n && r < m.rank) {
+        const float* x = a.partial + (int64_t)(p.row0 + t0 + t) * a.ld + 2 * HK + 2 * HV + r;
+        for (int s = 0; s < a.nsplit; ++s) v += x[s * a.split_stride];
+      }
+      dst[a1_at(t, r)] = v;
     }
   };
   load_a1(0, sA1);
   __syncthreads();
-  const float qscale = rsqrtf((float)K), dscale = -LOG2E / m.tau;
+  const float qscale = rsqrtf((float)K), dscale = -1.0f / m.tau;
   for (int t0 = 0, it = 0; t0 < p.n; t0 += C, ++it) {
     const int nt = min(C, p.n - t0);
-    const float* a1 = sA1 + (it & 1) * C * rp;
+    const float* a1 = sA1 + (it & 1) * a1_size;
+    float* const end_prev = sEnd + ((it & 1) ^ 1) * Kp;
+    float* const end_now = sEnd + (it & 1) * Kp;
     const float* base = a.partial + (int64_t)(p.row0 + t0) * a.ld;
     // ---- values
     {
@@ -154,63 +160,103 @@ __global__ void __launch_bounds__(NT, 2) gla_chunk_kernel(GlaArgs a, ChunkCfg cf
         if (vt < vstep && t < C) *reinterpret_cast<uint2*>(sV + t * ldv + vc) = make_uint2(pack_bf16(x[i].x, x[i].y), pack_bf16(x[i].z, x[i].w));
       }
     }
-    // ---- decays and scaled queries and keys of this thread's channel, 16 tokens
+    // ---- decays and scaled queries and keys of this thread's channels and tokens
     bool far = false;
-    if (kc < Kp) {
-      float e[16];
+    if (mine) {
+      const float* qp = base + (int64_t)tb * ld + (int64_t)h * K + kc;
+      const int nu = live ? nt - tb : 0;
+      auto rows8 = [&](const float* x, float2 (&y)[8]) {
 #pragma unroll
-      for (int u = 0; u < 16; ++u) e[u] = kbias;
+        for (int u = 0; u < 8; ++u) y[u] = u < nu ? *reinterpret_cast<const float2*>(x + u * ld) : make_float2(0.f, 0.f);
+        for (int s = 1; s < a.nsplit; ++s)
+#pragma unroll
+          for (int u = 0; u < 8; ++u)
+            if (u < nu) {
+              const float2 w = *reinterpret_cast<const float2*>(x + s * a.split_stride + u * ld);
+              y[u].x += w.x;
+              y[u].y += w.y;
+            }
+      };
+      float2 e[8];
+#pragma unroll
+      for (int u = 0; u < 8; ++u) e[u] = kbias;
       for (int r = 0; r < rp; r += 4) {
-        const float w0 = sA2[r * Kp + kc], w1 = sA2[(r + 1) * Kp + kc], w2 = sA2[(r + 2) * Kp + kc], w3 = sA2[(r + 3) * Kp + kc];
+        float2 w[4];
 #pragma unroll
-        for (int u = 0; u < 16; ++u) {
-          const float4 x = *reinterpret_cast<const float4*>(a1 + (half * 16 + u) * rp + r);
-          e[u] = fmaf(x.x, w0, fmaf(x.y, w1, fmaf(x.z, w2, fmaf(x.w, w3, e[u]))));
+        for (int i = 0; i < 4; ++i) w[i] = *reinterpret_cast<const float2*>(sA2 + (r + i) * Kp + kc);
+#pragma unroll
+        for (int u = 0; u < 8; ++u) {
+          const float4 x = *reinterpret_cast<const float4*>(a1 + a1_at(tb + u, r));
+          e[u].x = fmaf(x.x, w[0].x, fmaf(x.y, w[1].x, fmaf(x.z, w[2].x, fmaf(x.w, w[3].x, e[u].x))));
+          e[u].y = fmaf(x.x, w[0].y, fmaf(x.y, w[1].y, fmaf(x.z, w[2].y, fmaf(x.w, w[3].y, e[u].y))));
         }
       }
       // log2 of the decays, then their sums from the middle of the chunk
-      float tot = 0.f;
+      float2 part = make_float2(0.f, 0.f);
 #pragma unroll
-      for (int u = 0; u < 16; ++u) {
-        const float z = e[u];
-        const float la = half * 16 + u < nt && kc < K ? (fmaxf(-z, 0.f) + log1pf(ex2(-LOG2E * fabsf(z)))) * dscale : 0.f;
-        tot += la;
-        e[u] = la;
+      for (int u = 0; u < 8; ++u) {
+        e[u].x = u < nu ? neg_log2_sigmoid(e[u].x) * dscale : 0.f;
+        e[u].y = u < nu ? neg_log2_sigmoid(e[u].y) * dscale : 0.f;
+        part.x += e[u].x;
+        part.y += e[u].y;
       }
-      far = tot < -MAX_DECAY;
-      sF[half * Kp + kc] = ex2(tot);
-      float run = half ? 0.f : tot;
-#pragma unroll
-      for (int u = 0; u < 16; ++u) {
-        // first half: minus the decays still ahead of the middle; second half: the decays since
+      const float2 other = make_float2(__shfl_xor_sync(pair, part.x, 16), __shfl_xor_sync(pair, part.y, 16));
+      const float2 tot = make_float2(part.x + other.x, part.y + other.y);
+      far = fminf(tot.x, tot.y) < -MAX_DECAY;
+      if (!late) {
+        const float2 f = make_float2(ex2(tot.x), ex2(tot.y));
         if (half) {
-          run += e[u];
+          *reinterpret_cast<float2*>(end_now + kc) = f;
+        } else {
+          const float2 g0 = *reinterpret_cast<const float2*>(end_prev + kc);
+          *reinterpret_cast<float2*>(sF + kc) = make_float2(f.x * g0.x, f.y * g0.y);
+        }
+      }
+      // first half: minus the decays still ahead of the middle; second half: the decays since
+      float2 run = half ? (late ? other : make_float2(0.f, 0.f)) : (late ? part : tot);
+      bf16* dq = sQ + tb * ldq + kc;
+      bf16* dk = sK + tb * ldq + kc;
+#pragma unroll
+      for (int u = 0; u < 8; ++u) {
+        if (half) {
+          run.x += e[u].x;
+          run.y += e[u].y;
           e[u] = run;
         } else {
-          run -= e[u];
-          e[u] = -run;
+          run.x -= e[u].x;
+          run.y -= e[u].y;
+          e[u] = make_float2(-run.x, -run.y);
         }
+        if (far) e[u] = make_float2(0.f, 0.f);
       }
-      const float* qp = base + (int64_t)half * 16 * a.ld + (int64_t)h * K + kc;
-      const int nu = kc < K ? nt - half * 16 : 0;
+      float2 x[8];
+      rows8(qp, x);
+      uint32_t hi, lo;
 #pragma unroll
-      for (int w = 0; w < 16; w += 8) {
-        float q[8], k[8];
-        slab_n<8>(a, qp + (int64_t)w * a.ld, a.ld, nu - w, q);
-        slab_n<8>(a, qp + (int64_t)w * a.ld + HK, a.ld, nu - w, k);
+      for (int u = 0; u < 8; ++u) {
+        split2(x[u].x * qscale * ex2(e[u].x), x[u].y * qscale * ex2(e[u].y), hi, lo);
+        *reinterpret_cast<uint32_t*>(dq + u * ldq) = hi;
+        *reinterpret_cast<uint32_t*>(dq + (C + u) * ldq) = lo;
+      }
+      rows8(qp + HK, x);
 #pragma unroll
-        for (int u = 0; u < 8; ++u) {
-          const int t = half * 16 + w + u;
-          const float f = far ? 0.f : ex2(e[w + u]), fi = far ? 0.f : ex2(-e[w + u]);
-          bf16* dq = sQ + t * ldq + kc;
-          bf16* dk = sK + t * ldq + kc;
-          split(q[u] * qscale * f, dq[0], dq[C * ldq]);
-          split(k[u] * fi, dk[0], dk[C * ldq]);
-        }
+      for (int u = 0; u < 8; ++u) {
+        split2(x[u].x * ex2(-e[u].x), x[u].y * ex2(-e[u].y), hi, lo);
+        *reinterpret_cast<uint32_t*>(dk + u * ldq) = hi;
+        *reinterpret_cast<uint32_t*>(dk + (C + u) * ldq) = lo;
       }
     }
     const bool slow = __syncthreads_or(far ? 1 : 0) != 0;
-    if (t0 + C < p.n) load_a1(t0 + C, sA1 + ((it + 1) & 1) * C * rp);
+    if (t0 + C < p.n) {
+      load_a1(t0 + C, sA1 + ((it + 1) & 1) * a1_size);
+      // the next chunk's rows of this head move into L2 under this chunk's products
+      for (int i = tid; i < C * 16; i += NT) {
+        const int t = i >> 4, part = (i >> 2) & 3, line = (i & 3) * 32;
+        const int n = part < 2 ? K : vs;
+        if (t0 + C + t < p.n && line < n)
+          prefetch_l2(base + (int64_t)(C + t) * ld + (part < 2 ? part * HK + (int64_t)h * K : 2 * HK + (part - 2) * HV + (int64_t)h * V + v0) + line);
+      }
+    }
     float o[4][4];
 #pragma unroll
     for (int j = 0; j < 4; ++j)
@@ -280,7 +326,7 @@ __global__ void __launch_bounds__(NT, 2) gla_chunk_kernel(GlaArgs a, ChunkCfg cf
         }
       }
       __syncthreads();
-      // ---- o^T += v^T A^T, S^T += v^T k~, then the rest of the decay
+      // ---- o^T += v^T A^T, S^T += v^T k~; the decay after the middle joins the next scaling of the state
       if (state_warp) {
         const uint32_t ab = aA + (((lq >> 1) * 8 + l8) * ldA + (lq & 1) * 8) * 2;
         const uint32_t kb = aK + (((lq & 1) * 8 + l8) * ldq + (lq >> 1) * 8) * 2;
@@ -310,15 +356,6 @@ __global__ void __launch_bounds__(NT, 2) gla_chunk_kernel(GlaArgs a, ChunkCfg cf
             mma_bf16_16816(S[2 * k + 1], vf, c[2], c[3]);
           }
         }
-#pragma unroll
-        for (int j = 0; j < 2 * KT; ++j) {
-          if (j >= 2 * cf.kt) break;
-          const float2 f = *reinterpret_cast<const float2*>(sF + Kp + j * 8 + 2 * t4);
-          S[j][0] *= f.x;
-          S[j][1] *= f.y;
-          S[j][2] *= f.x;
-          S[j][3] *= f.y;
-        }
         // output and its sums of squares over this warp's value rows
 #pragma unroll
         for (int j = 0; j < 4; ++j)
@@ -337,18 +374,29 @@ __global__ void __launch_bounds__(NT, 2) gla_chunk_kernel(GlaArgs a, ChunkCfg cf
     } else {
       // ---- token by token: q | k | alpha in the k~ buffer
       float* x = reinterpret_cast<float*>(sK);
+#pragma unroll
+      for (int j = 0; j < 2 * KT; ++j) {
+        if (j >= 2 * cf.kt) break;
+        const float2 f = *reinterpret_cast<const float2*>(end_prev + j * 8 + 2 * t4);
+        S[j][0] *= f.x;
+        S[j][1] *= f.y;
+        S[j][2] *= f.x;
+        S[j][3] *= f.y;
+      }
+      for (int k = tid; k < Kp; k += NT) end_now[k] = 1.f;
       for (int t = 0; t < nt; ++t) {
         for (int k = tid; k < Kp; k += NT) {
           float q = 0.f, kk = 0.f, al = 0.f;
           if (k < K) {
-            const float* qp = base + (int64_t)t * a.ld + (int64_t)h * K + k;
-            float y[2];
-            slab_n<2>(a, qp, HK, 2, y);
-            q = y[0] * qscale;
-            kk = y[1];
+            const float* qp = base + (int64_t)t * ld + (int64_t)h * K + k;
+            for (int s = 0; s < a.nsplit; ++s) {
+              q += qp[s * a.split_stride];
+              kk += qp[s * a.split_stride + HK];
+            }
+            q *= qscale;
             float z = m.a2_b[(int64_t)h * K + k];
-            for (int r = 0; r < rp; ++r) z = fmaf(a1[t * rp + r], sA2[r * Kp + k], z);
-            al = ex2((fmaxf(-z, 0.f) + log1pf(ex2(-LOG2E * fabsf(z)))) * dscale);
+            for (int r = 0; r < rp; ++r) z = fmaf(a1[a1_at(t, r)], sA2[r * Kp + k], z);
+            al = ex2(neg_log2_sigmoid(z) * dscale);
           }
           x[k] = q;
           x[Kp + k] = kk;
@@ -408,9 +456,9 @@ __global__ void __launch_bounds__(NT, 2) gla_chunk_kernel(GlaArgs a, ChunkCfg cf
         ss = 0.f;
         for (unsigned r = 0; r < gridDim.x; ++r) ss += cg::this_cluster().map_shared_rank(sS, r)[(it & 1) * C + t];
       }
-      const float f = 1.0f / sqrtf(ss / (float)V + a.eps);
+      const float f = rsqrtf(ss / (float)V + a.eps);
       const float4 x = *reinterpret_cast<const float4*>(sO + t * ldO + vc), w = *reinterpret_cast<const float4*>(m.norm + v0 + vc);
-      auto silu = [](float z) { return z / (1.0f + __expf(-z)); };
+      auto silu = [](float z) { return __fdividef(z, 1.0f + __expf(-z)); };
       *reinterpret_cast<uint2*>(reinterpret_cast<bf16*>(a.out) + (int64_t)(p.row0 + t0 + t) * a.ldo + (int64_t)h * V + v0 + vc) =
           make_uint2(pack_bf16(x.x * f * w.x * silu(gz[i].x), x.y * f * w.y * silu(gz[i].y)),
                      pack_bf16(x.z * f * w.z * silu(gz[i].z), x.w * f * w.w * silu(gz[i].w)));
@@ -418,12 +466,13 @@ __global__ void __launch_bounds__(NT, 2) gla_chunk_kernel(GlaArgs a, ChunkCfg cf
     __syncthreads();
   }
   if (state_warp) {
+    const float* f = sEnd + (((p.n + C - 1) / C - 1) & 1) * Kp;
 #pragma unroll
     for (int j = 0; j < 2 * KT; ++j)
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         const int v = v0 + warp * 16 + g + 8 * (e >> 1), k = 8 * j + 2 * t4 + (e & 1);
-        if (v < V && k < K) st[(int64_t)k * a.ldv + v] = S[j][e];
+        if (v < V && k < K) st[(int64_t)k * a.ldv + v] = S[j][e] * f[k];
       }
   }
   if constexpr (CLUSTER) cg::this_cluster().sync();   // a peer may still read this CTA's sums
@@ -452,9 +501,9 @@ int gla_chunk_launch(Ctx* c, const GlaArgs& a) {
   cf.off_v = cf.off_k + up(std::max(ops, 3 * Kp * 4));
   cf.off_a = cf.off_v + up(C * (cf.vs + 8) * 2);
   cf.off_a1 = cf.off_a + up(2 * C * (C + 8) * 2);
-  cf.off_a2 = cf.off_a1 + up(2 * C * cf.rp * 4);
+  cf.off_a2 = cf.off_a1 + up(2 * (C * cf.rp + C / 8 * 4) * 4);
   cf.off_f = cf.off_a2 + up(cf.rp * Kp * 4);
-  cf.off_ss = cf.off_f + up(2 * Kp * 4);
+  cf.off_ss = cf.off_f + up(3 * Kp * 4);
   const int smem = cf.off_ss + up((2 + 8) * C * 4);
   const dim3 grid((unsigned)nv, (unsigned)a.m.heads, (unsigned)a.count);
   auto go = [&](auto kernel, bool cluster) -> int {
