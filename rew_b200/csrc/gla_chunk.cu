@@ -5,9 +5,8 @@
 //   o_t  = q~_t (e^r S) + sum_s A_ts v_s                    S <- e^(b_end - r) (e^r S + sum_s k~_s v_s^T)
 // so one pair of scaled operands serves the scores, the output and the state.  A CTA walks the chunks of one portion
 // with the state of one head (or of a slice of its value columns; a cluster shares the head) in registers: warp w holds
-// the transposed state [16 value rows][dim], whose accumulator fragments are also the A operand of q~ S.  Products are
-// bf16 with operands split in two (high part and remainder) where they carry the decays, the state or the scores, and
-// f32 sums; decays, their sums and the state itself are f32.
+// the transposed state [16 value rows][dim], whose accumulator fragments are also the A operand of q~ S.  Decays, their
+// sums and the state are f32; operands of products are bf16 (the state as a high part and a remainder) and sums f32.
 //
 // The two halves of a chunk bound the exponents: if a channel decays by more than 2^MAX_DECAY in one of them, the
 // chunk runs token by token on the same registers.
@@ -69,11 +68,11 @@ __global__ void __launch_bounds__(NT, 2) gla_chunk_kernel(GlaArgs a, ChunkCfg cf
   extern __shared__ __align__(16) uint8_t smem[];
   const GlaDims& m = a.m;
   const int K = m.dim, V = m.vdim, Kp = cf.kt * 16, vs = cf.vs, rp = cf.rp, ldq = cf.ldq, ldv = vs + 8, ldO = vs + 4;
-  bf16* sQ = reinterpret_cast<bf16*>(smem);                    // [hi, lo][C][ldq]
+  bf16* sQ = reinterpret_cast<bf16*>(smem);                    // [C][ldq]
   float* sO = reinterpret_cast<float*>(smem);                  // [C][ldO], once q~ has been read
-  bf16* sK = reinterpret_cast<bf16*>(smem + cf.off_k);         // [hi, lo][C][ldq]
+  bf16* sK = reinterpret_cast<bf16*>(smem + cf.off_k);         // [C][ldq]
   bf16* sV = reinterpret_cast<bf16*>(smem + cf.off_v);         // [C][ldv]
-  bf16* sA = reinterpret_cast<bf16*>(smem + cf.off_a);         // [hi, lo][C][C + 8]
+  bf16* sA = reinterpret_cast<bf16*>(smem + cf.off_a);         // [C][C + 8]
   float* sA1 = reinterpret_cast<float*>(smem + cf.off_a1);     // [2][a1_at(C, 0)]
   float* sA2 = reinterpret_cast<float*>(smem + cf.off_a2);     // [rp][Kp]
   float* sF = reinterpret_cast<float*>(smem + cf.off_f);       // [Kp] decay up to the middle since the state was scaled last
@@ -82,27 +81,26 @@ __global__ void __launch_bounds__(NT, 2) gla_chunk_kernel(GlaArgs a, ChunkCfg cf
   constexpr int ldA = C + 8;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, l8 = lane & 7, lq = lane >> 3, g = lane >> 2, t4 = lane & 3;
   const int h = blockIdx.y, v0 = blockIdx.x * vs;
-  const int64_t HK = (int64_t)m.heads * K, HV = (int64_t)m.heads * V;
+  const int HK = m.heads * K, HV = m.heads * V;
   const bool state_warp = warp * 16 < vs;
   pdl_launch_dependents();
   // weights of the decay projection do not depend on earlier kernels
   for (int i = tid; i < rp * Kp; i += NT) {
     const int r = i / Kp, k = i % Kp;
-    sA2[i] = r < m.rank && k < K ? m.a2[(int64_t)r * HK + (int64_t)h * K + k] : 0.f;
+    sA2[i] = r < m.rank && k < K ? m.a2[r * HK + h * K + k] : 0.f;
   }
   // this thread's pair of key channels and eight tokens: a warp has 32 channels of one half of the chunk, its upper lanes
   // the later eight tokens
   const int half = warp >> 2, kc = (warp & 3) * 32 + (lane & 15) * 2, late = lane >> 4, tb = half * 16 + late * 8;
   const bool mine = kc < Kp, live = kc < K;
   const uint32_t pair = __ballot_sync(0xffffffffu, mine);      // both lanes of a channel pair are in or out together
-  const float2 kbias = live ? *reinterpret_cast<const float2*>(m.a2_b + (int64_t)h * K + kc) : make_float2(0.f, 0.f);
   for (int k = tid; k < Kp; k += NT) sEnd[Kp + k] = 1.f;       // the chunk before the first one
   // rows of decay features, with a gap every eight of them so that two groups of lanes read different banks
   auto a1_at = [rp](int t, int r) { return t * rp + (t >> 3) * 4 + r; };
   const int a1_size = a1_at(C, 0), ld = (int)a.ld;
   pdl_wait();
   const GlaPortion p = a.list[blockIdx.z];
-  float* st = a.state + ((int64_t)p.lane * m.heads + h) * K * a.ldv;
+  auto state = [&]() -> float* { return a.state + ((int64_t)p.lane * m.heads + h) * K * a.ldv; };
   // S[j][e]: value row v0 + 16 warp + g + 8 (e >> 1), channel 8 j + 2 t4 + (e & 1)
   float S[2 * KT][4];
 #pragma unroll
@@ -110,25 +108,28 @@ __global__ void __launch_bounds__(NT, 2) gla_chunk_kernel(GlaArgs a, ChunkCfg cf
 #pragma unroll
     for (int e = 0; e < 4; ++e) {
       const int v = v0 + warp * 16 + g + 8 * (e >> 1), k = 8 * j + 2 * t4 + (e & 1);
-      S[j][e] = p.pos0 > 0 && state_warp && v < V && k < K ? st[(int64_t)k * a.ldv + v] : 0.f;
+      S[j][e] = p.pos0 > 0 && state_warp && v < V && k < K ? state()[k * a.ldv + v] : 0.f;
     }
   // items of four columns this thread handles of a [C][vs] tile: one column group, tokens vt, vt + vstep, ..
   const int vq = vs / 4, vt = tid / vq, vc = (tid % vq) * 4, vstep = NT / vq;   // vs <= 128: at most 4 items
+  const bool exact = NT % vq == 0 && C % vstep == 0 && v0 + vs <= V;
   auto tile4 = [&](const float* base, int nt, float4 (&x)[4]) {
+    const float* b = base + vt * ld + vc;
+    if (exact && nt == C && a.nsplit == 1) {
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+        if (i * vstep < C) x[i] = *reinterpret_cast<const float4*>(b + i * vstep * ld);
+      return;
+    }
 #pragma unroll
     for (int i = 0; i < 4; ++i) {
-      const int t = vt + i * vstep;
-      x[i] = vt < vstep && t < nt && v0 + vc < V ? *reinterpret_cast<const float4*>(base + (int64_t)t * ld + vc) : make_float4(0.f, 0.f, 0.f, 0.f);
-    }
-    for (int s = 1; s < a.nsplit; ++s)
-#pragma unroll
-      for (int i = 0; i < 4; ++i) {
-        const int t = vt + i * vstep;
-        if (vt < vstep && t < nt && v0 + vc < V) {
-          const float4 w = *reinterpret_cast<const float4*>(base + s * a.split_stride + (int64_t)t * ld + vc);
+      x[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (vt < vstep && vt + i * vstep < nt && v0 + vc < V)
+        for (int s = 0; s < a.nsplit; ++s) {
+          const float4 w = *reinterpret_cast<const float4*>(b + s * a.split_stride + i * vstep * ld);
           x[i].x += w.x; x[i].y += w.y; x[i].z += w.z; x[i].w += w.w;
         }
-      }
+    }
   };
   auto load_a1 = [&](int t0, float* dst) {
     for (int i = tid; i < C * rp; i += NT) {
@@ -143,7 +144,7 @@ __global__ void __launch_bounds__(NT, 2) gla_chunk_kernel(GlaArgs a, ChunkCfg cf
   };
   load_a1(0, sA1);
   __syncthreads();
-  const float qscale = rsqrtf((float)K), dscale = -1.0f / m.tau;
+  const float qscale = rsqrtf((float)K), dscale = -1.0f / m.tau, inv_v = 1.0f / (float)V;
   for (int t0 = 0, it = 0; t0 < p.n; t0 += C, ++it) {
     const int nt = min(C, p.n - t0);
     const float* a1 = sA1 + (it & 1) * a1_size;
@@ -153,7 +154,7 @@ __global__ void __launch_bounds__(NT, 2) gla_chunk_kernel(GlaArgs a, ChunkCfg cf
     // ---- values
     {
       float4 x[4];
-      tile4(base + 2 * HK + (int64_t)h * V + v0, nt, x);
+      tile4(base + 2 * HK + h * V + v0, nt, x);
 #pragma unroll
       for (int i = 0; i < 4; ++i) {
         const int t = vt + i * vstep;
@@ -163,21 +164,27 @@ __global__ void __launch_bounds__(NT, 2) gla_chunk_kernel(GlaArgs a, ChunkCfg cf
     // ---- decays and scaled queries and keys of this thread's channels and tokens
     bool far = false;
     if (mine) {
-      const float* qp = base + (int64_t)tb * ld + (int64_t)h * K + kc;
+      const float* qp = base + tb * ld + h * K + kc;
       const int nu = live ? nt - tb : 0;
       auto rows8 = [&](const float* x, float2 (&y)[8]) {
+        if (nu >= 8 && a.nsplit == 1) {
 #pragma unroll
-        for (int u = 0; u < 8; ++u) y[u] = u < nu ? *reinterpret_cast<const float2*>(x + u * ld) : make_float2(0.f, 0.f);
-        for (int s = 1; s < a.nsplit; ++s)
+          for (int u = 0; u < 8; ++u) y[u] = *reinterpret_cast<const float2*>(x + u * ld);
+          return;
+        }
 #pragma unroll
-          for (int u = 0; u < 8; ++u)
-            if (u < nu) {
+        for (int u = 0; u < 8; ++u) {
+          y[u] = make_float2(0.f, 0.f);
+          if (u < nu)
+            for (int s = 0; s < a.nsplit; ++s) {
               const float2 w = *reinterpret_cast<const float2*>(x + s * a.split_stride + u * ld);
               y[u].x += w.x;
               y[u].y += w.y;
             }
+        }
       };
       float2 e[8];
+      const float2 kbias = live ? *reinterpret_cast<const float2*>(m.a2_b + h * K + kc) : make_float2(0.f, 0.f);
 #pragma unroll
       for (int u = 0; u < 8; ++u) e[u] = kbias;
       for (int r = 0; r < rp; r += 4) {
@@ -195,8 +202,9 @@ __global__ void __launch_bounds__(NT, 2) gla_chunk_kernel(GlaArgs a, ChunkCfg cf
       float2 part = make_float2(0.f, 0.f);
 #pragma unroll
       for (int u = 0; u < 8; ++u) {
-        e[u].x = u < nu ? neg_log2_sigmoid(e[u].x) * dscale : 0.f;
-        e[u].y = u < nu ? neg_log2_sigmoid(e[u].y) * dscale : 0.f;
+        e[u].x = neg_log2_sigmoid(e[u].x) * dscale;
+        e[u].y = neg_log2_sigmoid(e[u].y) * dscale;
+        if (u >= nu) e[u] = make_float2(0.f, 0.f);
         part.x += e[u].x;
         part.y += e[u].y;
       }
@@ -231,30 +239,22 @@ __global__ void __launch_bounds__(NT, 2) gla_chunk_kernel(GlaArgs a, ChunkCfg cf
       }
       float2 x[8];
       rows8(qp, x);
-      uint32_t hi, lo;
 #pragma unroll
-      for (int u = 0; u < 8; ++u) {
-        split2(x[u].x * qscale * ex2(e[u].x), x[u].y * qscale * ex2(e[u].y), hi, lo);
-        *reinterpret_cast<uint32_t*>(dq + u * ldq) = hi;
-        *reinterpret_cast<uint32_t*>(dq + (C + u) * ldq) = lo;
-      }
+      for (int u = 0; u < 8; ++u)
+        *reinterpret_cast<uint32_t*>(dq + u * ldq) = pack_bf16(x[u].x * (qscale * ex2(e[u].x)), x[u].y * (qscale * ex2(e[u].y)));
       rows8(qp + HK, x);
 #pragma unroll
-      for (int u = 0; u < 8; ++u) {
-        split2(x[u].x * ex2(-e[u].x), x[u].y * ex2(-e[u].y), hi, lo);
-        *reinterpret_cast<uint32_t*>(dk + u * ldq) = hi;
-        *reinterpret_cast<uint32_t*>(dk + (C + u) * ldq) = lo;
-      }
+      for (int u = 0; u < 8; ++u) *reinterpret_cast<uint32_t*>(dk + u * ldq) = pack_bf16(x[u].x * ex2(-e[u].x), x[u].y * ex2(-e[u].y));
     }
     const bool slow = __syncthreads_or(far ? 1 : 0) != 0;
     if (t0 + C < p.n) {
       load_a1(t0 + C, sA1 + ((it + 1) & 1) * a1_size);
       // the next chunk's rows of this head move into L2 under this chunk's products
-      for (int i = tid; i < C * 16; i += NT) {
-        const int t = i >> 4, part = (i >> 2) & 3, line = (i & 3) * 32;
-        const int n = part < 2 ? K : vs;
-        if (t0 + C + t < p.n && line < n)
-          prefetch_l2(base + (int64_t)(C + t) * ld + (part < 2 ? part * HK + (int64_t)h * K : 2 * HK + (part - 2) * HV + (int64_t)h * V + v0) + line);
+      const int line = (tid & 3) * 32, part = (tid >> 2) & 3;
+      if (line < (part < 2 ? K : vs)) {
+        const float* x = base + (C + (tid >> 4)) * ld + (part < 2 ? part * HK + h * K : 2 * HK + (part - 2) * HV + h * V + v0) + line;
+        if (t0 + C + (tid >> 4) < p.n) prefetch_l2(x);
+        if (t0 + C + 16 + (tid >> 4) < p.n) prefetch_l2(x + 16 * ld);
       }
     }
     float o[4][4];
@@ -264,39 +264,29 @@ __global__ void __launch_bounds__(NT, 2) gla_chunk_kernel(GlaArgs a, ChunkCfg cf
       for (int e = 0; e < 4; ++e) o[j][e] = 0.f;
     if (!slow) {
       const uint32_t aQ = smem_u32(sQ), aK = smem_u32(sK), aV = smem_u32(sV), aA = smem_u32(sA);
-      const uint32_t lo = C * ldq * 2;   // bytes from the high parts to the remainders
       // ---- scores: six 16 x 8 tiles on and below the diagonal
       if (warp < 6) {
         const int mt = warp < 2 ? 0 : 1, nn = warp < 2 ? warp : warp - 2;
         float s[4] = {0.f, 0.f, 0.f, 0.f};
         const uint32_t qa = aQ + ((mt * 16 + (lq & 1) * 8 + l8) * ldq + (lq >> 1) * 8) * 2;
         const uint32_t ka = aK + ((nn * 8 + l8) * ldq + (lq & 1) * 8) * 2;
-        for (int k = 0; k < cf.kt; ++k) {
-          uint32_t qh[4], ql[4], b0, b1, c0, c1;
-          ldmatrix_x4(qh[0], qh[1], qh[2], qh[3], qa + k * 32);
-          ldmatrix_x4(ql[0], ql[1], ql[2], ql[3], qa + k * 32 + lo);
+#pragma unroll
+        for (int k = 0; k < KT; ++k) {
+          if (k >= cf.kt) break;
+          uint32_t q[4], b0, b1;
+          ldmatrix_x4(q[0], q[1], q[2], q[3], qa + k * 32);
           ldmatrix_x2(b0, b1, ka + k * 32);
-          ldmatrix_x2(c0, c1, ka + k * 32 + lo);
-          mma_bf16_16816(s, qh, b0, b1);
-          mma_bf16_16816(s, qh, c0, c1);
-          mma_bf16_16816(s, ql, b0, b1);
+          mma_bf16_16816(s, q, b0, b1);
         }
 #pragma unroll
         for (int r = 0; r < 2; ++r) {
           const int t = mt * 16 + g + 8 * r, sc = nn * 8 + 2 * t4;
-          uint32_t hi, lw;
-          split2(sc <= t ? s[2 * r] : 0.f, sc + 1 <= t ? s[2 * r + 1] : 0.f, hi, lw);
-          *reinterpret_cast<uint32_t*>(sA + t * ldA + sc) = hi;
-          *reinterpret_cast<uint32_t*>(sA + (C + t) * ldA + sc) = lw;
+          *reinterpret_cast<uint32_t*>(sA + t * ldA + sc) = pack_bf16(sc <= t ? s[2 * r] : 0.f, sc + 1 <= t ? s[2 * r + 1] : 0.f);
         }
-      } else {
-        // tokens 0 .. 15 see none of 16 .. 31
-        for (int i = tid - 192; i < 2 * 16 * 8; i += 64)
-          *reinterpret_cast<uint32_t*>(sA + ((i >> 7) * C + ((i >> 3) & 15)) * ldA + 16 + (i & 7) * 2) = 0u;
       }
       // ---- the state as every earlier token left it: o^T [16 value rows][C] = (e^r S)^T q~^T
       if (state_warp) {
-        const uint32_t qb = aQ + (((lq >> 1) * 8 + l8) * ldq + (lq & 1) * 8) * 2;
+        const uint32_t qb = aQ + (((lq >> 1) * 8 + l8) * ldq + (lq & 1) * 8) * 2, qb2 = qb + 16 * ldq * 2;
 #pragma unroll
         for (int k = 0; k < KT; ++k) {
           if (k >= cf.kt) break;
@@ -313,15 +303,12 @@ __global__ void __launch_bounds__(NT, 2) gla_chunk_kernel(GlaArgs a, ChunkCfg cf
           }
 #pragma unroll
           for (int j = 0; j < 4; j += 2) {
-            uint32_t b[4], c[4];
-            ldmatrix_x4(b[0], b[1], b[2], b[3], qb + j * 8 * ldq * 2 + k * 32);
-            ldmatrix_x4(c[0], c[1], c[2], c[3], qb + j * 8 * ldq * 2 + k * 32 + lo);
+            uint32_t b[4];
+            ldmatrix_x4(b[0], b[1], b[2], b[3], (j ? qb2 : qb) + k * 32);
             mma_bf16_16816(o[j], sh, b[0], b[1]);
             mma_bf16_16816(o[j + 1], sh, b[2], b[3]);
             mma_bf16_16816(o[j], sl, b[0], b[1]);
             mma_bf16_16816(o[j + 1], sl, b[2], b[3]);
-            mma_bf16_16816(o[j], sh, c[0], c[1]);
-            mma_bf16_16816(o[j + 1], sh, c[2], c[3]);
           }
         }
       }
@@ -329,31 +316,26 @@ __global__ void __launch_bounds__(NT, 2) gla_chunk_kernel(GlaArgs a, ChunkCfg cf
       // ---- o^T += v^T A^T, S^T += v^T k~; the decay after the middle joins the next scaling of the state
       if (state_warp) {
         const uint32_t ab = aA + (((lq >> 1) * 8 + l8) * ldA + (lq & 1) * 8) * 2;
-        const uint32_t kb = aK + (((lq & 1) * 8 + l8) * ldq + (lq >> 1) * 8) * 2;
+        const uint32_t kb = aK + (((lq & 1) * 8 + l8) * ldq + (lq >> 1) * 8) * 2, kb2 = kb + 16 * ldq * 2;
 #pragma unroll
         for (int s = 0; s < 2; ++s) {
           uint32_t vf[4];
           ldmatrix_x4_trans(vf[0], vf[1], vf[2], vf[3], aV + ((s * 16 + (lq >> 1) * 8 + l8) * ldv + warp * 16 + (lq & 1) * 8) * 2);
 #pragma unroll
           for (int j = 0; j < 4; j += 2) {
-            uint32_t b[4], c[4];
+            if (s == 1 && j == 0) continue;   // tokens 0 .. 15 see none of 16 .. 31
+            uint32_t b[4];
             ldmatrix_x4(b[0], b[1], b[2], b[3], ab + j * 8 * ldA * 2 + s * 32);
-            ldmatrix_x4(c[0], c[1], c[2], c[3], ab + j * 8 * ldA * 2 + s * 32 + C * ldA * 2);
             mma_bf16_16816(o[j], vf, b[0], b[1]);
             mma_bf16_16816(o[j + 1], vf, b[2], b[3]);
-            mma_bf16_16816(o[j], vf, c[0], c[1]);
-            mma_bf16_16816(o[j + 1], vf, c[2], c[3]);
           }
 #pragma unroll
           for (int k = 0; k < KT; ++k) {
             if (k >= cf.kt) break;
-            uint32_t b[4], c[4];
-            ldmatrix_x4_trans(b[0], b[1], b[2], b[3], kb + s * 16 * ldq * 2 + k * 32);
-            ldmatrix_x4_trans(c[0], c[1], c[2], c[3], kb + s * 16 * ldq * 2 + k * 32 + lo);
+            uint32_t b[4];
+            ldmatrix_x4_trans(b[0], b[1], b[2], b[3], (s ? kb2 : kb) + k * 32);
             mma_bf16_16816(S[2 * k], vf, b[0], b[1]);
             mma_bf16_16816(S[2 * k + 1], vf, b[2], b[3]);
-            mma_bf16_16816(S[2 * k], vf, c[0], c[1]);
-            mma_bf16_16816(S[2 * k + 1], vf, c[2], c[3]);
           }
         }
         // output and its sums of squares over this warp's value rows
@@ -388,13 +370,13 @@ __global__ void __launch_bounds__(NT, 2) gla_chunk_kernel(GlaArgs a, ChunkCfg cf
         for (int k = tid; k < Kp; k += NT) {
           float q = 0.f, kk = 0.f, al = 0.f;
           if (k < K) {
-            const float* qp = base + (int64_t)t * ld + (int64_t)h * K + k;
+            const float* qp = base + t * ld + h * K + k;
             for (int s = 0; s < a.nsplit; ++s) {
               q += qp[s * a.split_stride];
               kk += qp[s * a.split_stride + HK];
             }
             q *= qscale;
-            float z = m.a2_b[(int64_t)h * K + k];
+            float z = m.a2_b[h * K + k];
             for (int r = 0; r < rp; ++r) z = fmaf(a1[a1_at(t, r)], sA2[r * Kp + k], z);
             al = ex2(neg_log2_sigmoid(z) * dscale);
           }
@@ -437,42 +419,47 @@ __global__ void __launch_bounds__(NT, 2) gla_chunk_kernel(GlaArgs a, ChunkCfg cf
     }
     // the gates are requested ahead of the barrier
     float4 gz[4];
-    tile4(base + 2 * HK + HV + (int64_t)h * V + v0, nt, gz);
+    tile4(base + 2 * HK + HV + h * V + v0, nt, gz);
     __syncthreads();
     // ---- norm over the head, gate, store
     if (tid < C) {
       float ss = 0.f;
       for (int w = 0; w * 16 < vs; ++w) ss += sS[2 * C + w * C + tid];
-      sS[(it & 1) * C + tid] = ss;
+      sS[(it & 1) * C + tid] = CLUSTER ? ss : rsqrtf(fmaf(ss, inv_v, a.eps));
     }
     if constexpr (CLUSTER) cg::this_cluster().sync();
     else __syncthreads();
+    if (vt < vstep && v0 + vc < V) {
+      const float4 w = *reinterpret_cast<const float4*>(m.norm + v0 + vc);
+      bf16* op = reinterpret_cast<bf16*>(a.out) + (int64_t)(p.row0 + t0 + vt) * a.ldo + h * V + v0 + vc;
+      const int ldo = (int)a.ldo;
+      auto silu = [](float z) { return __fdividef(z, 1.0f + ex2(-LOG2E * z)); };
 #pragma unroll
-    for (int i = 0; i < 4; ++i) {
-      const int t = vt + i * vstep;
-      if (vt >= vstep || t >= nt || v0 + vc >= V) continue;
-      float ss = sS[(it & 1) * C + t];
-      if constexpr (CLUSTER) {
-        ss = 0.f;
-        for (unsigned r = 0; r < gridDim.x; ++r) ss += cg::this_cluster().map_shared_rank(sS, r)[(it & 1) * C + t];
+      for (int i = 0; i < 4; ++i) {
+        const int t = vt + i * vstep;
+        if (t >= nt) break;
+        float f = sS[(it & 1) * C + t];
+        if constexpr (CLUSTER) {
+          f = 0.f;
+          for (unsigned r = 0; r < gridDim.x; ++r) f += cg::this_cluster().map_shared_rank(sS, r)[(it & 1) * C + t];
+          f = rsqrtf(fmaf(f, inv_v, a.eps));
+        }
+        const float4 x = *reinterpret_cast<const float4*>(sO + t * ldO + vc);
+        *reinterpret_cast<uint2*>(op + i * vstep * ldo) = make_uint2(pack_bf16(x.x * f * w.x * silu(gz[i].x), x.y * f * w.y * silu(gz[i].y)),
+                                                                     pack_bf16(x.z * f * w.z * silu(gz[i].z), x.w * f * w.w * silu(gz[i].w)));
       }
-      const float f = rsqrtf(ss / (float)V + a.eps);
-      const float4 x = *reinterpret_cast<const float4*>(sO + t * ldO + vc), w = *reinterpret_cast<const float4*>(m.norm + v0 + vc);
-      auto silu = [](float z) { return __fdividef(z, 1.0f + __expf(-z)); };
-      *reinterpret_cast<uint2*>(reinterpret_cast<bf16*>(a.out) + (int64_t)(p.row0 + t0 + t) * a.ldo + (int64_t)h * V + v0 + vc) =
-          make_uint2(pack_bf16(x.x * f * w.x * silu(gz[i].x), x.y * f * w.y * silu(gz[i].y)),
-                     pack_bf16(x.z * f * w.z * silu(gz[i].z), x.w * f * w.w * silu(gz[i].w)));
     }
     __syncthreads();
   }
   if (state_warp) {
     const float* f = sEnd + (((p.n + C - 1) / C - 1) & 1) * Kp;
+    float* to = state();
 #pragma unroll
     for (int j = 0; j < 2 * KT; ++j)
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         const int v = v0 + warp * 16 + g + 8 * (e >> 1), k = 8 * j + 2 * t4 + (e & 1);
-        if (v < V && k < K) st[(int64_t)k * a.ldv + v] = S[j][e] * f[k];
+        if (v < V && k < K) to[k * a.ldv + v] = S[j][e] * f[k];
       }
   }
   if constexpr (CLUSTER) cg::this_cluster().sync();   // a peer may still read this CTA's sums
@@ -496,11 +483,11 @@ int gla_chunk_launch(Ctx* c, const GlaArgs& a) {
   const int Kp = cf.kt * 16;
   cf.ldq = Kp + 8;
   auto up = [](int v) { return (v + 127) / 128 * 128; };
-  const int ops = 2 * C * cf.ldq * 2;
+  const int ops = C * cf.ldq * 2;
   cf.off_k = up(std::max(ops, C * (cf.vs + 4) * 4));
   cf.off_v = cf.off_k + up(std::max(ops, 3 * Kp * 4));
   cf.off_a = cf.off_v + up(C * (cf.vs + 8) * 2);
-  cf.off_a1 = cf.off_a + up(2 * C * (C + 8) * 2);
+  cf.off_a1 = cf.off_a + up(C * (C + 8) * 2);
   cf.off_a2 = cf.off_a1 + up(2 * (C * cf.rp + C / 8 * 4) * 4);
   cf.off_f = cf.off_a2 + up(cf.rp * Kp * 4);
   cf.off_ss = cf.off_f + up(3 * Kp * 4);
