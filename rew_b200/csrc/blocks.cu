@@ -616,10 +616,10 @@ int layered_prepare(rewb200_session* s, const FwdOpts& o, int64_t rows) {
   const bool uniform = o.entries == nullptr;
   RB_REQUIRE(!uniform || o.S == 1, "layered step: a step of several tokens per lane needs its portions");
   // ---- lists of the step: [row lane | row position | absorbed tiles | their chunks | expanded tiles | gathered keys |
-  // small and large tiles of grouped-query attention | small and large portions of gated linear attention]
+  // chunks of gated linear attention | small and large tiles of grouped-query attention | small and large portions of gated linear attention]
   int64_t abs_rows = rows, n_keys = 0;
   s->plan_host.clear();
-  s->plan_abs_tiles = s->plan_chunks = s->plan_exp_tiles = s->plan_keys = 0;
+  s->plan_abs_tiles = s->plan_chunks = s->plan_exp_tiles = s->plan_keys = s->plan_gla_chunks = 0;
   if (!uniform) {
     std::vector<int>& h = s->plan_host;
     h.assign(2 * rows, 0);
@@ -647,6 +647,7 @@ int layered_prepare(rewb200_session* s, const FwdOpts& o, int64_t rows) {
     std::vector<int2> gqa_small;
     std::vector<GqaTile> gqa_large;
     std::vector<GlaPortion> gla_small, gla_large;
+    std::vector<int2> gla_chunk;
     for (const StepEntry& e : *o.entries) {
       for (int i = 0; i < e.n; ++i) {
         h[e.row0 + i] = e.lane;
@@ -658,7 +659,13 @@ int layered_prepare(rewb200_session* s, const FwdOpts& o, int64_t rows) {
         else
           for (int i = 0; i < e.n; i += GQA_TILE_ROWS) gqa_small.push_back(make_int2(e.row0 + i, std::min(GQA_TILE_ROWS, e.n - i)));
       }
-      if (has_gla) (gla_ok && e.n >= CHUNK_MIN_ROWS ? gla_large : gla_small).push_back({e.row0, e.n, e.pos0, e.lane});
+      if (has_gla) {
+        const bool large = gla_ok && e.n >= CHUNK_MIN_ROWS;
+        const GlaPortion p = {e.row0, e.n, e.pos0, e.lane, large ? (int)gla_chunk.size() : 0};
+        (large ? gla_large : gla_small).push_back(p);
+        if (large)
+          for (int i = 0; i < gla_chunks(e.n); ++i) gla_chunk.push_back(gla_chunk_rows(p, i));
+      }
       if (!has_latent) continue;
       if (exp_ok && e.n >= EXPAND_MIN_ROWS) {
         const int key0 = (int)std::max<int64_t>(0, (int64_t)e.pos0 - reach + 1);
@@ -685,6 +692,7 @@ int layered_prepare(rewb200_session* s, const FwdOpts& o, int64_t rows) {
     s->plan_gqa_large = (int)gqa_large.size();
     s->plan_gla_small = (int)gla_small.size();
     s->plan_gla_large = (int)gla_large.size();
+    s->plan_gla_chunks = (int)gla_chunk.size();
     s->plan_abs_tiles = (int)tiles.size();
     s->plan_chunks = (int)chunks.size();
     s->plan_exp_tiles = (int)exps.size();
@@ -699,6 +707,7 @@ int layered_prepare(rewb200_session* s, const FwdOpts& o, int64_t rows) {
     append(chunks.data(), chunks.size() * sizeof(int2));
     append(exps.data(), exps.size() * sizeof(ExpTile));
     append(keys.data(), keys.size() * sizeof(int2));
+    append(gla_chunk.data(), gla_chunk.size() * sizeof(int2));
     append(gqa_small.data(), gqa_small.size() * sizeof(int2));
     append(gqa_large.data(), gqa_large.size() * sizeof(GqaTile));
     append(gla_small.data(), gla_small.size() * sizeof(GlaPortion));
@@ -725,6 +734,14 @@ int layered_prepare(rewb200_session* s, const FwdOpts& o, int64_t rows) {
     s->kvx_rows = n_keys;
   }
   // ---- scratch of the absorbed path
+  size_t chunk = 0;
+  for (const LayerDev& D : m->layers)
+    if (D.mixer == MIX_GLA) chunk = std::max(chunk, gla_chunk_bytes(D.l.m));
+  if (chunk * s->plan_gla_chunks > s->gla_work_bytes) {
+    s->gla_work_bytes = 0;
+    RB_TRY(regrow(s, &s->gla_work, chunk * s->plan_gla_chunks));
+    s->gla_work_bytes = chunk * s->plan_gla_chunks;
+  }
   int64_t units = 0, stats = 0, qe = 0;
   int64_t g_units = 0, g_stats = 0;
   for (const LayerDev& D : m->layers) {
@@ -777,7 +794,7 @@ struct StepLists {
   RowMap map = {};
   RowTiles abs = {}, chunks = {};
   const ExpTile* exp_tiles = nullptr;
-  const int2* key_list = nullptr;
+  const int2 *key_list = nullptr, *gla_chunks = nullptr;
   RowTiles gqa_small = {};
   const GqaTile* gqa_large = nullptr;
   const GlaPortion *gla_small = nullptr, *gla_large = nullptr;
@@ -798,7 +815,8 @@ StepLists step_lists(const rewb200_session* s, const FwdOpts& o, int64_t rows) {
   t.chunks.count = s->plan_chunks;
   t.exp_tiles = reinterpret_cast<const ExpTile*>(t.chunks.list + t.chunks.count);
   t.key_list = reinterpret_cast<const int2*>(t.exp_tiles + s->plan_exp_tiles);
-  t.gqa_small.list = t.key_list + s->plan_keys;
+  t.gla_chunks = t.key_list + s->plan_keys;
+  t.gqa_small.list = t.gla_chunks + s->plan_gla_chunks;
   t.gqa_small.count = s->plan_gqa_small;
   t.gqa_large = reinterpret_cast<const GqaTile*>(t.gqa_small.list + t.gqa_small.count);
   t.gla_small = reinterpret_cast<const GlaPortion*>(t.gqa_large + s->plan_gqa_large);
@@ -925,6 +943,9 @@ int gla_mixer(rewb200_session* s, const FwdOpts& o, const StepLists& t, size_t r
   if (!t.uniform && s->plan_gla_large > 0) {
     ga.list = t.gla_large;
     ga.count = s->plan_gla_large;
+    ga.chunks = t.gla_chunks;
+    ga.n_chunks = s->plan_gla_chunks;
+    ga.work = s->gla_work;
     RB_TRY(gla_chunk_launch(c, ga));
   }
   if (o.trace) RB_TRY(o.trace->mark(TC_ATTN));

@@ -216,7 +216,9 @@ struct rewb200_session {
   size_t plan_cap = 0;
   std::vector<int> plan_host;
   int plan_abs_tiles = 0, plan_chunks = 0, plan_exp_tiles = 0, plan_keys = 0;
-  int plan_gqa_small = 0, plan_gqa_large = 0, plan_gla_small = 0, plan_gla_large = 0;
+  int plan_gqa_small = 0, plan_gqa_large = 0, plan_gla_small = 0, plan_gla_large = 0, plan_gla_chunks = 0;
+  uint8_t* gla_work = nullptr;         // blocks of the chunks of gated linear attention
+  size_t gla_work_bytes = 0;
   int* feed_dev = nullptr;             // ids and row lists of a rewb200_lanes_feed step
   size_t feed_cap = 0;
   int64_t route_rows = 0;              // rows of the forward recorded last

@@ -108,7 +108,7 @@ __device__ __forceinline__ void finish_token(const GlaArgs& a, const TokenSmem& 
 
 __device__ __forceinline__ GlaPortion portion_of(const GlaArgs& a, int i) {
   if (a.list) return a.list[i];
-  return GlaPortion{i, 1, a.pos0[a.b0 + i], a.b0 + i};
+  return GlaPortion{i, 1, a.pos0[a.b0 + i], a.b0 + i, 0};
 }
 
 // grid (heads, portions).  The head's state stays in registers over the portion: a thread owns four neighbouring value

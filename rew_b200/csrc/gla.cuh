@@ -17,6 +17,7 @@ struct GlaDims {
 // A portion of a step: rows row0 .. row0 + n - 1 are the tokens at positions pos0 .. of `lane`.
 struct GlaPortion {
   int row0, n, pos0, lane;
+  int chunk0;              // large portions: the first of its chunks in GlaArgs::chunks
 };
 
 struct GlaArgs {
@@ -25,6 +26,9 @@ struct GlaArgs {
   int count;
   const int* pos0;
   int b0;
+  const int2* chunks;      // large portions: (first row, tokens) of every chunk
+  int n_chunks;
+  uint8_t* work;           // ... scratch, gla_chunk_bytes a chunk
   // fused input projection [q heads*dim | k heads*dim | v heads*vdim | gate heads*vdim | decay rank], split-K slabs
   const float* partial;    // [nsplit][rows][ld]
   int nsplit;
@@ -41,6 +45,9 @@ struct GlaArgs {
 int64_t gla_state_ld(int vdim);
 int gla_recurrent_launch(Ctx* c, const GlaArgs& a);
 bool gla_chunk_ok(const GlaDims& m);
+int gla_chunks(int n);                                  // chunks of a portion of n tokens
+int2 gla_chunk_rows(const GlaPortion& p, int i);        // first row and tokens of its i-th chunk
+size_t gla_chunk_bytes(const GlaDims& m);               // scratch of one chunk, all heads
 int gla_chunk_launch(Ctx* c, const GlaArgs& a);
 
 }  // namespace rewb
