@@ -456,6 +456,8 @@ __global__ void __launch_bounds__(CL == 1 ? 512 : 256) output_norm_kernel(Output
   __shared__ float part[2];
   pdl_launch_dependents();
   const int64_t row = blockIdx.x / CL, d = a.d, dq = d / CL, col0 = (int64_t)(blockIdx.x % CL) * dq;
+  if (CL > 1 && a.gamma) prefetch_floats(a.gamma + col0, (int)dq);   // depends on no earlier kernel
+  if (CL > 1 && a.final_gamma) prefetch_floats(a.final_gamma + col0, (int)dq);
   pdl_wait();
   float* xr = a.x_res + row * d + col0;
   const T* erow = nullptr;

@@ -114,12 +114,17 @@ __device__ __forceinline__ GlaPortion portion_of(const GlaArgs& a, int i) {
 // grid (heads, portions).  The head's state stays in registers over the portion: a thread owns four neighbouring value
 // columns of up to KI key channels, `slices` apart.
 template <typename T, int NT, int KI>
-__global__ void __launch_bounds__(NT, NT == 128 ? (KI <= 16 ? 4 : 3) : 1) gla_recurrent_kernel(GlaArgs a, int slices) {
+__global__ void __launch_bounds__(NT, NT == 128 ? (KI <= 16 ? 4 : 3) : KI <= 8 ? 2 : 1) gla_recurrent_kernel(GlaArgs a, int slices) {
   extern __shared__ __align__(16) float sm[];
   __shared__ float red[NT / 32];
   pdl_launch_dependents();
   const GlaDims& m = a.m;
   const int h = blockIdx.x, K = m.dim, V = m.vdim, vq = a.ldv / 4;
+  // weights depend on no earlier kernel
+  for (int r = threadIdx.x / 8; r < m.rank; r += NT / 8)
+    for (int i = (threadIdx.x % 8) * 32; i < K; i += 256) prefetch_l2(m.a2 + ((int64_t)r * m.heads + h) * K + i);
+  prefetch_floats(m.a2_b + (int64_t)h * K, K);
+  prefetch_floats(m.norm, V);
   if (!a.early) pdl_wait();
   const GlaPortion p = portion_of(a, blockIdx.y);
   const TokenSmem s = carve(sm, m, a.ldv);
@@ -221,6 +226,8 @@ int gla_recurrent_launch(Ctx* c, const GlaArgs& a) {
   (bf ? go(gla_recurrent_kernel<bf16, NT, KI>, NT, slices_of(NT), slices_of(NT))                  \
       : go(gla_recurrent_kernel<float, NT, KI>, NT, slices_of(NT), slices_of(NT)))
   if (c->gla_impl != 1) {
+    // few heads and sequences: more threads on each, for latency
+    if ((int64_t)a.m.heads * a.count <= 2 * c->sm_count && ki_of(512) <= 8) return RB_GLA(512, 8);
     if (ki_of(128) <= 8) return RB_GLA(128, 8);
     if (ki_of(128) <= 16) return RB_GLA(128, 16);
     if (ki_of(128) <= 32) return RB_GLA(128, 32);

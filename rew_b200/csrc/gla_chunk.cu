@@ -251,20 +251,20 @@ __global__ void __launch_bounds__(NT, 3) gla_prepare_kernel(GlaArgs a, ChunkLayo
   }
 }
 
-// grid (value slices, heads, portions).  KT: capacity of the register state in 16-channel steps; vs: value columns of the
-// CTA, a multiple of 16.
+// grid (value slices, heads, portions), a warp per 16 value columns.  KT: capacity of the register state in 16-channel steps;
+// vs: value columns of the CTA, a multiple of 16.
 template <int KT, bool CLUSTER>
 __global__ void __launch_bounds__(NT, 2) gla_scan_kernel(GlaArgs a, ChunkLayout cl, int vs) {
   extern __shared__ __align__(128) uint8_t smem[];
   const GlaDims& m = a.m;
   const int K = m.dim, V = m.vdim, Kp = cl.kt * 16, ldq = cl.ldq, ldv = cl.ldv, ldO = vs + 4, ld = (int)a.ld;
   float* sO = reinterpret_cast<float*>(smem + 2 * cl.bytes);                 // [2][C][ldO]
-  float* sS = sO + 2 * C * ldO;                                              // [2][C] norms (cluster: sums), [2][8 warps][C] sums of squares
-  float* sX = sS + 2 * C + 2 * 8 * C;                                        // [3][Kp] q, k, alpha of a token (token-by-token path)
+  float* sS = sO + 2 * C * ldO;                                              // [2][C] sums of squares, [C] norms, [2][8 warps][C] sums of squares
+  float* sX = sS + 3 * C + 2 * 8 * C;                                        // [3][Kp] q, k, alpha of a token (token-by-token path)
   uint64_t* full = reinterpret_cast<uint64_t*>(sX + 3 * Kp);
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, l8 = lane & 7, lq = lane >> 3, g = lane >> 2, t4 = lane & 3;
   const int h = blockIdx.y, v0 = blockIdx.x * vs, HK = m.heads * K, HV = m.heads * V;
-  const bool state_warp = warp * 16 < vs;
+  const int nthreads = 2 * vs;                                               // the block
   if (tid == 0) {
     mbar_init(full, 1);
     mbar_init(full + 1, 1);
@@ -289,7 +289,7 @@ __global__ void __launch_bounds__(NT, 2) gla_scan_kernel(GlaArgs a, ChunkLayout 
 #pragma unroll
     for (int e = 0; e < 4; ++e) {
       const int v = v0 + warp * 16 + g + 8 * (e >> 1), k = 8 * j + 2 * t4 + (e & 1);
-      S[j][e] = p.pos0 > 0 && state_warp && v < V && k < K ? st[k * a.ldv + v] : 0.f;
+      S[j][e] = p.pos0 > 0 && v < V && k < K ? st[k * a.ldv + v] : 0.f;
     }
   auto scale_state = [&](const float* f) {
 #pragma unroll
@@ -303,8 +303,9 @@ __global__ void __launch_bounds__(NT, 2) gla_scan_kernel(GlaArgs a, ChunkLayout 
     }
   };
   // output: one group of four columns, tokens vt, vt + vstep, ..
-  const int vq = vs / 4, vt = tid / vq, vc = (tid - vt * vq) * 4, vstep = NT / vq;
-  const bool writes = vt < vstep && v0 + vc < V;
+  constexpr int vstep = 8;   // 2 vs threads, vs / 4 column groups
+  const int vq = vs / 4, vt = tid / vq, vc = (tid - vt * vq) * 4;
+  const bool writes = v0 + vc < V;
   const float inv_v = 1.0f / (float)V;
   const int ldo = (int)a.ldo;
   bool ok = true;
@@ -313,7 +314,7 @@ __global__ void __launch_bounds__(NT, 2) gla_scan_kernel(GlaArgs a, ChunkLayout 
     uint8_t* const blk = smem + (it & 1) * cl.bytes;
     const float* const base = a.partial + (int64_t)(p.row0 + it * C) * a.ld;
     float* const o_buf = sO + (it & 1) * C * ldO;
-    float* const ss_buf = sS + 2 * C + (it & 1) * 8 * C;
+    float* const ss_buf = sS + 3 * C + (it & 1) * 8 * C;
     // the gates of the chunk are requested ahead of its products
     float4 gz[4];
 #pragma unroll
@@ -330,7 +331,7 @@ __global__ void __launch_bounds__(NT, 2) gla_scan_kernel(GlaArgs a, ChunkLayout 
         }
     if (ok) ok = mbar_wait(full + (it & 1), (it >> 1) & 1, a.status);
     if (*reinterpret_cast<const int*>(blk + cl.far) == 0) {
-      if (state_warp) {
+      {
         const uint32_t aQ = smem_u32(blk), aK = aQ + cl.k, aV = aQ + cl.v, aA = aQ + cl.a;
         const float* f = reinterpret_cast<const float*>(blk + cl.f);
         float o[4][4];
@@ -410,7 +411,7 @@ __global__ void __launch_bounds__(NT, 2) gla_scan_kernel(GlaArgs a, ChunkLayout 
       // ---- token by token
       const bf16* sV = reinterpret_cast<const bf16*>(blk + cl.v);
       for (int t = 0; t < nt; ++t) {
-        for (int k = tid; k < Kp; k += NT) {
+        for (int k = tid; k < Kp; k += nthreads) {
           float q = 0.f, kk = 0.f, al = 0.f;
           if (k < K) {
             const float* x = base + t * ld;
@@ -427,7 +428,7 @@ __global__ void __launch_bounds__(NT, 2) gla_scan_kernel(GlaArgs a, ChunkLayout 
           sX[2 * Kp + k] = al;
         }
         __syncthreads();
-        if (state_warp) {
+        {
           const float va = __bfloat162float(sV[t * ldv + v0 + warp * 16 + g]), vb = __bfloat162float(sV[t * ldv + v0 + warp * 16 + g + 8]);
           float oa = 0.f, ob = 0.f;
 #pragma unroll
@@ -462,14 +463,26 @@ __global__ void __launch_bounds__(NT, 2) gla_scan_kernel(GlaArgs a, ChunkLayout 
     __syncthreads();   // the block has been read, the output stands in o_buf
     if (tid == 0 && it + 2 < chunks) load(it + 2);
     // ---- norm over the head, gate, store
+    float* const norms = sS + 2 * C;
+    auto warps_sum = [&]() -> float {
+      float x[8];
+#pragma unroll
+      for (int w = 0; w < 8; ++w) x[w] = w * 16 < vs ? ss_buf[w * C + tid] : 0.f;
+      return ((x[0] + x[1]) + (x[2] + x[3])) + ((x[4] + x[5]) + (x[6] + x[7]));
+    };
     if constexpr (CLUSTER) {
-      if (tid < C) {
-        float ss = 0.f;
-        for (int w = 0; w * 16 < vs; ++w) ss += ss_buf[w * C + tid];
-        sS[(it & 1) * C + tid] = ss;
-      }
+      if (tid < C) sS[(it & 1) * C + tid] = warps_sum();
       cg::this_cluster().sync();
+      if (tid < C) {
+        float x[4];
+#pragma unroll
+        for (unsigned r = 0; r < 4; ++r) x[r] = r < gridDim.x ? cg::this_cluster().map_shared_rank(sS, r)[(it & 1) * C + tid] : 0.f;
+        norms[tid] = rsqrtf(fmaf((x[0] + x[1]) + (x[2] + x[3]), inv_v, a.eps));
+      }
+    } else {
+      if (tid < C) norms[tid] = rsqrtf(fmaf(warps_sum(), inv_v, a.eps));
     }
+    __syncthreads();
     if (writes) {
       const float4 w = *reinterpret_cast<const float4*>(m.norm + v0 + vc);
       bf16* op = reinterpret_cast<bf16*>(a.out) + (int64_t)(p.row0 + it * C + vt) * a.ldo + h * V + v0 + vc;
@@ -478,20 +491,14 @@ __global__ void __launch_bounds__(NT, 2) gla_scan_kernel(GlaArgs a, ChunkLayout 
       for (int i = 0; i < 4; ++i) {
         const int t = vt + i * vstep;
         if (t >= nt) break;
-        float f = 0.f;
-        if constexpr (CLUSTER) {
-          for (unsigned r = 0; r < gridDim.x; ++r) f += cg::this_cluster().map_shared_rank(sS, r)[(it & 1) * C + t];
-        } else {
-          for (int u = 0; u * 16 < vs; ++u) f += ss_buf[u * C + t];
-        }
-        f = rsqrtf(fmaf(f, inv_v, a.eps));
+        const float f = norms[t];
         const float4 x = *reinterpret_cast<const float4*>(o_buf + t * ldO + vc);
         *reinterpret_cast<uint2*>(op + i * vstep * ldo) = make_uint2(pack_bf16(x.x * f * w.x * silu(gz[i].x), x.y * f * w.y * silu(gz[i].y)),
                                                                      pack_bf16(x.z * f * w.z * silu(gz[i].z), x.w * f * w.w * silu(gz[i].w)));
       }
     }
   }
-  if (state_warp) {
+  {
 #pragma unroll
     for (int j = 0; j < 2 * KT; ++j)
 #pragma unroll
@@ -521,12 +528,12 @@ int gla_chunk_launch(Ctx* c, const GlaArgs& a) {
   // few portions: a cluster of CTAs shares a head's value columns
   int nv = 1;
   while (nv < 4 && cl.vp % (nv * 2 * 16) == 0 && (int64_t)nv * a.m.heads * a.count < c->sm_count) nv *= 2;
-  const int vs = cl.vp / nv, smem = 2 * cl.bytes + (2 * C * (vs + 4) + 2 * C + 2 * 8 * C + 3 * cl.kt * 16) * 4 + 16;
+  const int vs = cl.vp / nv, smem = 2 * cl.bytes + (2 * C * (vs + 4) + 3 * C + 2 * 8 * C + 3 * cl.kt * 16) * 4 + 16;
   const dim3 grid((unsigned)nv, (unsigned)a.m.heads, (unsigned)a.count);
   auto go = [&](auto kernel, bool cluster) -> int {
     RB_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
-    RB_CUDA(cluster ? launch_k_cluster(kernel, grid, dim3(NT), smem, c->stream, c->use_pdl, dim3(nv), a, cl, vs)
-                    : launch_k(kernel, grid, dim3(NT), smem, c->stream, c->use_pdl, a, cl, vs));
+    RB_CUDA(cluster ? launch_k_cluster(kernel, grid, dim3(2 * vs), smem, c->stream, c->use_pdl, dim3(nv), a, cl, vs)
+                    : launch_k(kernel, grid, dim3(2 * vs), smem, c->stream, c->use_pdl, a, cl, vs));
     ++g_launch_total;
     return REWB200_OK;
   };

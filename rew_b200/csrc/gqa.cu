@@ -68,18 +68,23 @@ __global__ void __launch_bounds__(256) gqa_post_kernel(GqaPostArgs a, int64_t ro
   const int nr = (int)min((int64_t)RW, rows - row0);
   const int unit = blockIdx.y * 8 + (threadIdx.x >> 5), ln = threadIdx.x & 31;
   const int H = a.m.heads, G = a.m.own_kv ? a.m.kv_heads : 0, K = a.m.dim, V = a.m.vdim;
-  if (!a.early) pdl_wait();
+  // norm weights depend on no earlier kernel
+  if (a.m.q_norm) prefetch_floats(a.m.q_norm, K);
+  if (a.m.k_norm) prefetch_floats(a.m.k_norm, K);
   int pos[RW], page[RW];
   bool ok[RW];
+  auto lookup = [&]() {
 #pragma unroll
-  for (int r = 0; r < RW; ++r) {
-    const int64_t row = row0 + min(r, nr - 1);
-    pos[r] = row_pos(a.map, row);
-    ok[r] = pos[r] >= 0 && pos[r] < a.capacity;
-    page[r] = a.block_table[(int64_t)row_lane(a.map, row) * a.max_pages + (ok[r] ? pos[r] / PAGE_TOKENS : 0)];
-    if (!ok[r] && unit == 0 && ln == 0) atomicExch(a.status, KS_BAD_INDEX);
-  }
-  if (a.early) pdl_wait();
+    for (int r = 0; r < RW; ++r) {
+      const int64_t row = row0 + min(r, nr - 1);
+      pos[r] = row_pos(a.map, row);
+      ok[r] = pos[r] >= 0 && pos[r] < a.capacity;
+      page[r] = a.block_table[(int64_t)row_lane(a.map, row) * a.max_pages + (ok[r] ? pos[r] / PAGE_TOKENS : 0)];
+      if (!ok[r] && unit == 0 && ln == 0) atomicExch(a.status, KS_BAD_INDEX);
+    }
+  };
+  if (a.early) lookup();   // captured decode step: while the projection still runs
+  pdl_wait();
   if (unit > H + 2 * G || (unit == H + 2 * G && !a.m.gate)) return;
   const float* p = a.partial + row0 * a.ld;
   if (unit == H + 2 * G) {
@@ -123,6 +128,7 @@ __global__ void __launch_bounds__(256) gqa_post_kernel(GqaPostArgs a, int64_t ro
 #pragma unroll
       for (int c = 0; c < PC; ++c) x[r][c] = r < nr ? slab4(a, p + r * a.ld + col, (c * 32 + ln) * 4, n, false) : make_float4(0.f, 0.f, 0.f, 0.f);
   }
+  if (!a.early) lookup();  // ... or behind the loads above
   const float* w = is_v ? nullptr : is_q ? a.m.q_norm : a.m.k_norm;
   float4 g[PC];
 #pragma unroll
@@ -250,6 +256,12 @@ __global__ void __launch_bounds__(160, KS <= 8 ? 3 : 1) gqa_attn_kernel(const __
     tma_prefetch_desc(&tm_v);
   }
   pdl_launch_dependents();
+  {
+    // bias tables and sinks depend on no earlier kernel
+    const int group = a.m.heads / a.m.kv_heads, first = (int)blockIdx.z / cf.hgroups * group + ((int)blockIdx.z % cf.hgroups) * cf.heads_per;
+    if (a.m.bias) prefetch_floats(a.m.bias + (int64_t)first * a.m.n_bias, min(cf.heads_per, a.m.heads - first) * a.m.n_bias);
+    if (a.m.sink) prefetch_floats(a.m.sink + first, 1);
+  }
   __syncthreads();
   if (!a.early_kv) pdl_wait();
   const int2 tr = tile_rows(a.tiles, (int)blockIdx.y / cf.subtiles);

@@ -21,8 +21,6 @@ __device__ __forceinline__ float2 rotate(float2 v, float2 cs) {
 
 __device__ __forceinline__ void add4(float4& v, const float4 w) { v.x += w.x; v.y += w.y; v.z += w.z; v.w += w.w; }
 
-__device__ __forceinline__ void prefetch_l2(const void* p) { asm volatile("prefetch.global.L2 [%0];" ::"l"(p)); }
-
 // Sums of two values over the block; every thread gets both.
 __device__ __forceinline__ float2 block_sum2(float2 v, float2* red) {
 #pragma unroll

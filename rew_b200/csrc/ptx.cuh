@@ -119,6 +119,12 @@ __device__ __forceinline__ uint64_t policy_evict_last() {
   return p;
 }
 
+__device__ __forceinline__ void prefetch_l2(const void* p) { asm volatile("prefetch.global.L2 [%0];" ::"l"(p)); }
+// The lines of n floats, shared out over the threads of a block.
+__device__ __forceinline__ void prefetch_floats(const float* p, int n) {
+  for (int i = threadIdx.x * 32; i < n; i += blockDim.x * 32) prefetch_l2(p + i);
+}
+
 // Programmatic dependent launch: let the next kernel in the stream start its
 // prologue early / wait until every prior kernel's writes are visible.
 __device__ __forceinline__ void pdl_launch_dependents() {

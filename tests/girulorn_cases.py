@@ -96,8 +96,9 @@ def weights(cfg, seed=0, score_gain=1.0, decay=2.0):
         r = rng.normal(0, 0.002, size=(e_n, d))
         r[np.arange(e_n), rng.permutation(E)[:e_n]] += 1.5
         t[q + "router"] = r
-        t[q + "router.b"] = rng.permutation(e_n) * (6.0 * 1.5 / max(E - 1, 1))     # moves the choice, by whole rungs of the ladder and half
-        t[q + "router.b"] += np.where(np.arange(e_n) % 2, 1.5 / max(E - 1, 1), 0.0)
+        # the bias moves the choice: by whole rungs of the ladder, plus a fraction of one of its own for every expert
+        rung = 1.5 * 4.0 / max(E - 1, 1)
+        t[q + "router.b"] = rung * (rng.integers(-1, 2, size=e_n) + rng.permutation(e_n) / (e_n + 1.0))
         for e in ["e%d." % e for e in range(e_n)]:
             t[q + e + "gate"], t[q + e + "up"], t[q + e + "down"] = lin(f, d, 1.5), lin(f, d, 1.5), lin(d, f, 1.5)
         if L["mlp"].get("shared"):
