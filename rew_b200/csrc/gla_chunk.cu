@@ -254,7 +254,7 @@ __global__ void __launch_bounds__(NT, 3) gla_prepare_kernel(GlaArgs a, ChunkLayo
 // grid (value slices, heads, portions), a warp per 16 value columns.  KT: capacity of the register state in 16-channel steps;
 // vs: value columns of the CTA, a multiple of 16.
 template <int KT, bool CLUSTER>
-__global__ void __launch_bounds__(NT, 2) gla_scan_kernel(GlaArgs a, ChunkLayout cl, int vs) {
+__global__ void __launch_bounds__(CLUSTER ? NT / 2 : NT, CLUSTER ? 3 : 2) gla_scan_kernel(GlaArgs a, ChunkLayout cl, int vs) {
   extern __shared__ __align__(128) uint8_t smem[];
   const GlaDims& m = a.m;
   const int K = m.dim, V = m.vdim, Kp = cl.kt * 16, ldq = cl.ldq, ldv = cl.ldv, ldO = vs + 4, ld = (int)a.ld;
@@ -334,11 +334,13 @@ __global__ void __launch_bounds__(NT, 2) gla_scan_kernel(GlaArgs a, ChunkLayout 
       {
         const uint32_t aQ = smem_u32(blk), aK = aQ + cl.k, aV = aQ + cl.v, aA = aQ + cl.a;
         const float* f = reinterpret_cast<const float*>(blk + cl.f);
-        float o[4][4];
+        // (a slice has registers for a second set of sums: two shorter chains of products)
+        float o[4][4], o2[4][4];
 #pragma unroll
         for (int j = 0; j < 4; ++j)
 #pragma unroll
-          for (int e = 0; e < 4; ++e) o[j][e] = 0.f;
+          for (int e = 0; e < 4; ++e) o[j][e] = o2[j][e] = 0.f;
+        float(&ol)[4][4] = CLUSTER ? o2 : o;
         // ---- the state as every earlier token left it: o^T [16 value rows][C] = (e^r S)^T q~^T
         const uint32_t qb = aQ + (((lq >> 1) * 8 + l8) * ldq + (lq & 1) * 8) * 2, qb2 = qb + 16 * ldq * 2;
 #pragma unroll
@@ -362,10 +364,10 @@ __global__ void __launch_bounds__(NT, 2) gla_scan_kernel(GlaArgs a, ChunkLayout 
           mma_bf16_16816(o[1], sh, b[2], b[3]);
           mma_bf16_16816(o[2], sh, c[0], c[1]);
           mma_bf16_16816(o[3], sh, c[2], c[3]);
-          mma_bf16_16816(o[0], sl, b[0], b[1]);
-          mma_bf16_16816(o[1], sl, b[2], b[3]);
-          mma_bf16_16816(o[2], sl, c[0], c[1]);
-          mma_bf16_16816(o[3], sl, c[2], c[3]);
+          mma_bf16_16816(ol[0], sl, b[0], b[1]);
+          mma_bf16_16816(ol[1], sl, b[2], b[3]);
+          mma_bf16_16816(ol[2], sl, c[0], c[1]);
+          mma_bf16_16816(ol[3], sl, c[2], c[3]);
         }
         // ---- o^T += v^T A^T, S^T += v^T k~, then the decay after the middle
         const uint32_t ab = aA + (((lq >> 1) * 8 + l8) * LDA + (lq & 1) * 8) * 2;
@@ -392,6 +394,12 @@ __global__ void __launch_bounds__(NT, 2) gla_scan_kernel(GlaArgs a, ChunkLayout 
           }
         }
         scale_state(f + Kp);
+        if constexpr (CLUSTER) {
+#pragma unroll
+          for (int j = 0; j < 4; ++j)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) o[j][e] += o2[j][e];
+        }
         // output and its sums of squares over this warp's value rows
 #pragma unroll
         for (int j = 0; j < 4; ++j)

@@ -69,8 +69,8 @@ __global__ void __launch_bounds__(256) gqa_post_kernel(GqaPostArgs a, int64_t ro
   const int unit = blockIdx.y * 8 + (threadIdx.x >> 5), ln = threadIdx.x & 31;
   const int H = a.m.heads, G = a.m.own_kv ? a.m.kv_heads : 0, K = a.m.dim, V = a.m.vdim;
   // norm weights depend on no earlier kernel
-  if (a.m.q_norm) prefetch_floats(a.m.q_norm, K);
-  if (a.m.k_norm) prefetch_floats(a.m.k_norm, K);
+  if (RW == 1 && a.m.q_norm) prefetch_floats(a.m.q_norm, K);
+  if (RW == 1 && a.m.k_norm) prefetch_floats(a.m.k_norm, K);
   int pos[RW], page[RW];
   bool ok[RW];
   auto lookup = [&]() {

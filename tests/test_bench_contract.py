@@ -6,6 +6,8 @@ import os
 import subprocess
 import sys
 
+import pytest
+
 ROOT = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
 
 
@@ -85,8 +87,9 @@ def test_clock_record_counts_only_samples_inside_the_timed_region():
     assert short["samples"] == 3 and short["window"].startswith("warm-up + timed region") and short["reasons"] == ["sw_power_cap"]
 
 
-def test_reference_arm_says_why_a_layered_workload_is_unavailable():
-    r = _run("--impl", "reference", "--workload", "rezupel_b32", "--steps", "1", "--warmup", "1")
+@pytest.mark.parametrize("workload", ["rezupel_b32", "girulorn_b64"])
+def test_reference_arm_says_why_a_layered_workload_is_unavailable(workload):
+    r = _run("--impl", "reference", "--workload", workload, "--steps", "1", "--warmup", "1")
     assert r.returncode == 0, r.stderr[-2000:]
     j = json.loads([l for l in r.stdout.splitlines() if l.startswith("{")][0])
-    assert j["impl"] == "reference" and "latent" in j["unavailable"]
+    assert j["impl"] == "reference" and workload.split("_")[0] in j["unavailable"]
