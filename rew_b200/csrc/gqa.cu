@@ -83,8 +83,9 @@ __global__ void __launch_bounds__(256) gqa_post_kernel(GqaPostArgs a, int64_t ro
       if (!ok[r] && unit == 0 && ln == 0) atomicExch(a.status, KS_BAD_INDEX);
     }
   };
-  if (a.early) lookup();   // captured decode step: while the projection still runs
-  pdl_wait();
+  if (!a.early) pdl_wait();
+  lookup();                // in a captured decode step while the projection still runs
+  if (a.early) pdl_wait();
   if (unit > H + 2 * G || (unit == H + 2 * G && !a.m.gate)) return;
   const float* p = a.partial + row0 * a.ld;
   if (unit == H + 2 * G) {
@@ -128,7 +129,6 @@ __global__ void __launch_bounds__(256) gqa_post_kernel(GqaPostArgs a, int64_t ro
 #pragma unroll
       for (int c = 0; c < PC; ++c) x[r][c] = r < nr ? slab4(a, p + r * a.ld + col, (c * 32 + ln) * 4, n, false) : make_float4(0.f, 0.f, 0.f, 0.f);
   }
-  if (!a.early) lookup();  // ... or behind the loads above
   const float* w = is_v ? nullptr : is_q ? a.m.q_norm : a.m.k_norm;
   float4 g[PC];
 #pragma unroll

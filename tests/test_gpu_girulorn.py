@@ -14,7 +14,7 @@ from oracle import girulorn as G
 
 pytestmark = pytest.mark.gpu
 ROOT = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
-TOL = {"float32": 2e-5, "bfloat16": 4e-2}
+TOL = {"float32": 2e-5, "bfloat16": 3e-2}
 IMPLS = {"auto": ("auto", "auto"), "plain": ("plain", "plain"), "small": ("paged", "recurrent")}
 
 
@@ -46,16 +46,22 @@ def build(rb, cfg, t, dtype, max_seq=2048):
     return rb.CausalLM(c).load(c.canonical_tensors(t))
 
 
-def err(got, want):
-    """Worst row: rms of the difference over the rms of all wanted values."""
+def row_errors(got, want):
+    """rms of every row's difference over the rms of all wanted values."""
     got, want = np.asarray(got, np.float64), np.asarray(want, np.float64)
     assert got.shape == want.shape and np.isfinite(got).all()
-    return float(np.sqrt(((got - want) ** 2).mean(-1)).max() / max(np.sqrt((want ** 2).mean()), 1e-30))
+    return np.sqrt(((got - want) ** 2).mean(-1)) / max(np.sqrt((want ** 2).mean()), 1e-30)
 
 
-def close(got, want, dtype, slack=1.0):
-    e = err(got, want)
-    assert e <= TOL[dtype] * slack, e
+def err(got, want):
+    return float(np.sqrt((row_errors(got, want) ** 2).mean()))
+
+
+def close(got, want, dtype):
+    """All rows together within the tolerance, and no row far above it (16-bit rounding can move a sharp softmax at one
+    position)."""
+    e = row_errors(got, want)
+    assert np.sqrt((e ** 2).mean()) <= TOL[dtype] and e.max() <= 2.5 * TOL[dtype], (np.sqrt((e ** 2).mean()), e.max())
 
 
 def feed_all(sess, lane, ids, cuts):
