@@ -886,7 +886,6 @@ int gqa_mixer(rewb200_session* s, const FwdOpts& o, const StepLists& t, size_t r
   aa.o_part = s->gqa_part;
   aa.ml = s->gqa_ml;
   aa.kv_splits = gqa_kv_splits(c, G.m, aa.tiles.count, s->max_len);
-  aa.rows = rows;
   aa.early_kv = in_graph ? 1 : 0;
   aa.status = c->d_status;
   RB_TRY(gqa_attn_launch(c, aa));

@@ -29,18 +29,8 @@ __device__ __forceinline__ float ex2(float x) {
 }
 __device__ __forceinline__ float sigmoid(float z) { return 1.0f / (1.0f + expf(-z)); }
 
-// Four neighbouring columns of a row, summed over the slabs in slab order; columns past `n` read as zero.
-__device__ __forceinline__ float4 slab4(const GqaPostArgs& a, const float* p, int i, int n, bool vec) {
-  float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
-  if (i >= n) return v;
-  if (vec && i + 4 <= n) {
-#pragma unroll 4
-    for (int s = 0; s < a.nsplit; ++s) {
-      const float4 w = *reinterpret_cast<const float4*>(p + s * a.split_stride + i);
-      v.x += w.x; v.y += w.y; v.z += w.z; v.w += w.w;
-    }
-    return v;
-  }
+// Four neighbouring columns of a row that need not be aligned, summed over the slabs; columns past `n` read as zero.
+__device__ __forceinline__ float4 slab4(const GqaPostArgs& a, const float* p, int i, int n) {
   float e[4] = {0.f, 0.f, 0.f, 0.f};
   for (int u = 0; u < 4 && i + u < n; ++u)
     for (int s = 0; s < a.nsplit; ++s) e[u] += p[s * a.split_stride + i + u];
@@ -127,7 +117,7 @@ __global__ void __launch_bounds__(256) gqa_post_kernel(GqaPostArgs a, int64_t ro
 #pragma unroll
     for (int r = 0; r < RW; ++r)
 #pragma unroll
-      for (int c = 0; c < PC; ++c) x[r][c] = r < nr ? slab4(a, p + r * a.ld + col, (c * 32 + ln) * 4, n, false) : make_float4(0.f, 0.f, 0.f, 0.f);
+      for (int c = 0; c < PC; ++c) x[r][c] = r < nr ? slab4(a, p + r * a.ld + col, (c * 32 + ln) * 4, n) : make_float4(0.f, 0.f, 0.f, 0.f);
   }
   const float* w = is_v ? nullptr : is_q ? a.m.q_norm : a.m.k_norm;
   float4 g[PC];
@@ -230,7 +220,7 @@ struct GqaCfg {
   int heads_per, hgroups, tokens_per, subtiles;
 };
 
-// Shared tail of the attention and merge kernels: the sink joins the softmax, the gate scales the output.
+// A head's sink in base 2, -inf without one.
 __device__ __forceinline__ float sink_l2(const GqaDims& m, int h) { return m.sink ? m.sink[h] * LOG2E : -INFINITY; }
 
 // KS: 16-feature steps of a key row, VG: 16-column groups of a value row.

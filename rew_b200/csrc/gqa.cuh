@@ -64,7 +64,6 @@ struct GqaAttnArgs {
   float* o_part;           // scratch [rows][heads][kv splits][vdim], not yet divided by the row sum
   float2* ml;              // scratch [rows][heads][kv splits] running maximum (base 2) and sum
   int kv_splits;
-  int64_t rows;            // rows of the whole step
   int early_kv;            // captured decode step: cache pages other than the newest may be loaded ahead of the stream dependency
   int* status;
 };
