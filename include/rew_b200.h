@@ -300,7 +300,8 @@ typedef struct rewb200_layer {
   int32_t mixer;
   int32_t heads, dim, rot_dim, vdim, q_rank, kv_rank;
   int32_t window;       /* mixer 1: keys a query sees, itself included; 0: all before it */
-  int32_t rope_dims;    /* mixer 1: rotated features of the rot_dim part, interleaved pairs */
+  int32_t rope_dims;    /* mixer 1: rotated features of the rot_dim part, interleaved pairs; mixer 2: rotated features at the
+                         * start of a head, feature i paired with i + rope_dims / 2 */
   int32_t out_gate;     /* 1: every head's output is scaled by a sigmoid of its own projection of the input */
   int32_t ff;           /* 0 none, 1 dense gated SiLU, 2 routed experts */
   int32_t ffn;          /* hidden width of the dense feed-forward or of one expert */
@@ -310,8 +311,10 @@ typedef struct rewb200_layer {
   double rope_base;
   float scale;          /* of the attention scores */
   int32_t kv_heads;     /* mixer 2: key/value heads */
-  int32_t kv_from;      /* mixer 2: layer whose keys and values are used; -1: its own */
-  int32_t qk_norm, sink;
+  int32_t kv_from;      /* mixers 1 and 2: layer whose cached latents, or keys and values, are used; -1: its own */
+  int32_t qk_norm;
+  int32_t sink;         /* mixers 1 and 2, a term of the softmax denominator without a value: 0 none, 1 exp of a learned
+                         * number per head, 2 one (a score of zero) */
   int32_t bias_rows;    /* mixer 2: rows of the distance bias table (0: no bias): a bucket per distance below
                          * bias_rows / 2, then logarithmic ones up to bias_max */
   int32_t bias_max;
@@ -321,6 +324,10 @@ typedef struct rewb200_layer {
   float tau;
   int32_t router_bias;  /* 1: the router has a bias per expert */
   int32_t shared_ffn;   /* hidden width of a gated SiLU expert that runs for every token beside the routed ones; 0: none */
+  int32_t conv_taps;    /* mixer 2: taps of a causal convolution over time per channel of queries and keys; 0: none */
+  int32_t values_from_keys; /* mixer 2: 1: the values are the keys as they leave the convolution (vdim == dim) */
+  float router_scale;   /* factor of the routing weights; 0 reads as 1 */
+  int32_t shared_gate;  /* 1: the shared expert's output is scaled by a sigmoid of its own projection of the input */
 } rewb200_layer;
 typedef struct rewb200_stack {
   int32_t loop_start, loop_stop, loop_times; /* the half-open range of layers that is repeated, and how often it runs
@@ -329,8 +336,10 @@ typedef struct rewb200_stack {
                                               * to the residual. */
   int32_t norm_zero_centred;                 /* block and final norm weights are stored as the distance from one */
   int32_t block;                             /* 0: x += mixer(norm1(x)) + ff(norm2(x));
-                                              * 1: x += norm1(mixer(x)), then x += norm2(ff(x)) */
+                                              * 1: x += norm1(mixer(x)), then x += norm2(ff(x));
+                                              * 2: x += mixer(h) + ff(h), h = norm1(x) */
   int32_t own_head;                          /* 1: the output head is a tensor of its own, 0: the embedding table */
+  float logit_softcap;                       /* logits <- cap * tanh(logits / cap); 0: none */
 } rewb200_stack;
 
 /* ---- model + generate ------------------------------------------------------
@@ -354,11 +363,12 @@ typedef struct rewb200_config {
 int rewb200_model_create(int slot, const rewb200_config* cfg, rewb200_model** out);
 /* A layered model: `cfg` gives vocab, d_model, n_layers, max_seq, eps and dtype (its other fields are ignored),
  * `layers` n_layers descriptions.  Canonical tensors (Linear weights [in, out], see rew_b200/layered.py): embed,
- * step [times, d] (with a loop); per layer norm1, the mixer (1: dq, dq.norm, uq, dkv, dkv.norm, uk, uv; 2: q, then
- * with keys and values of its own k, v, then q.norm and (own) k.norm with qk_norm, rel [bias_rows, heads], sink;
- * 3: q, k, v, a1, a2, a2.b, g, norm), g (mixers 1 and 2 with out_gate), o, then with a feed-forward norm2 and gate,
- * up, down (dense) or router, [router.b,] per expert [gate,] up, down and the shared expert's gate, up, down; final
- * norm; head [d, vocab] (with own_head). */
+ * step [times, d] (with a loop); per layer norm1, the mixer (1: dq, dq.norm, uq, with latents of its own dkv, dkv.norm,
+ * then uk, uv, sink (1); 2: q, then with keys and values of its own k, v (v unless they are the keys), with a convolution
+ * q.conv and (own) k.conv [channels, taps], q.norm and (own) k.norm with qk_norm, rel [bias_rows, heads], sink (1);
+ * 3: q, k, v, a1, a2, a2.b, g, norm), g (mixers 1 and 2 with out_gate), o, then with a feed-forward norm2 (blocks 0 and 1)
+ * and gate, up, down (dense) or router, [router.b,] per expert [gate,] up, down and the shared expert's gate, up, down
+ * [, sg]; final norm; head [d, vocab] (with own_head). */
 int rewb200_model_create_layers(int slot, const rewb200_config* cfg, const rewb200_layer* layers, const rewb200_stack* stack,
                                 rewb200_model** out);
 void rewb200_model_free(rewb200_model* m);

@@ -36,12 +36,14 @@ class Layer(C.Structure):
                                          "out_gate", "ff", "ffn", "experts", "top_k", "renormalize", "expert_gated")] + [
         ("rope_base", C.c_double), ("scale", C.c_float)] + [
         (n, C.c_int32) for n in ("kv_heads", "kv_from", "qk_norm", "sink", "bias_rows", "bias_max", "temp_every")] + [
-        ("temp_coef", C.c_float), ("decay_rank", C.c_int32), ("tau", C.c_float), ("router_bias", C.c_int32), ("shared_ffn", C.c_int32)]
+        ("temp_coef", C.c_float), ("decay_rank", C.c_int32), ("tau", C.c_float), ("router_bias", C.c_int32), ("shared_ffn", C.c_int32),
+        ("conv_taps", C.c_int32), ("values_from_keys", C.c_int32), ("router_scale", C.c_float), ("shared_gate", C.c_int32)]
 
 
 class Stack(C.Structure):
     """struct rewb200_stack"""
-    _fields_ = [(n, C.c_int32) for n in ("loop_start", "loop_stop", "loop_times", "norm_zero_centred", "block", "own_head")]
+    _fields_ = [(n, C.c_int32) for n in ("loop_start", "loop_stop", "loop_times", "norm_zero_centred", "block", "own_head")] + [
+        ("logit_softcap", C.c_float)]
 
 
 _lib = None

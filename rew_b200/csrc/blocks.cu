@@ -5,7 +5,8 @@
 // A block is the parallel x += mixer(norm1(x)) + ff(norm2(x)), where one launch (residual_norm) adds both branches' f32
 // slabs to the residual, adds what a loop adds ahead of a pass, and leaves both norms of the next layer run, and in small
 // steps the feed-forward branch runs on the slot's second stream beside the mixer; or x += norm1(mixer(x)), then
-// x += norm2(ff(x)), where one launch (output_norm) per sublayer sums its slabs, norms the sum and adds it.
+// x += norm2(ff(x)), where one launch (output_norm) per sublayer sums its slabs, norms the sum and adds it; or the parallel
+// block with one norm that both branches read.
 //
 // Device layouts beyond engine.cu's: rows and Linear outputs are padded to multiples of 8 elements (zero weights, zero
 // norm weights), so any width can be loaded by TMA; a mixer's input projections are one matrix; the key and value
@@ -24,8 +25,10 @@ int64_t pad8(int64_t v) { return (v + 7) / 8 * 8; }
 enum Slot : int {
   SL_NORM1, SL_DQ, SL_DQ_NORM, SL_UQ, SL_DKV, SL_DKV_NORM, SL_UK, SL_UV, SL_G, SL_O, SL_NORM2, SL_GATE, SL_UP, SL_DOWN, SL_ROUTER,
   SL_E_GATE, SL_E_UP, SL_E_DOWN, SL_EMBED, SL_STEP, SL_FINAL, SL_HEAD, SL_Q, SL_K, SL_V, SL_Q_NORM, SL_K_NORM, SL_REL, SL_SINK, SL_A1, SL_A2,
-  SL_A2_B, SL_V_GATE, SL_V_NORM, SL_ROUTER_B, SL_S_GATE, SL_S_UP, SL_S_DOWN
+  SL_A2_B, SL_V_GATE, SL_V_NORM, SL_ROUTER_B, SL_S_GATE, SL_S_UP, SL_S_DOWN, SL_Q_CONV, SL_K_CONV, SL_S_SG
 };
+enum Block : int { BLOCK_PARALLEL = 0, BLOCK_OUTPUT_NORM = 1, BLOCK_ONE_NORM = 2 };
+enum Sink : int { SINK_NONE = 0, SINK_LEARNED = 1, SINK_ONE = 2 };
 enum Mixer : int { MIX_LATENT = 1, MIX_GQA = 2, MIX_GLA = 3 };
 struct TensorAt {
   Slot slot;
@@ -42,20 +45,28 @@ void tensors_of(const rewb200_model* m, std::vector<TensorAt>* out) {
       for (Slot s : slots) out->push_back({s, l, -1});
     };
     add({SL_NORM1});
-    if (L.mixer == MIX_LATENT) add({SL_DQ, SL_DQ_NORM, SL_UQ, SL_DKV, SL_DKV_NORM, SL_UK, SL_UV});
+    const bool own = L.kv_from < 0;
+    if (L.mixer == MIX_LATENT) {
+      add({SL_DQ, SL_DQ_NORM, SL_UQ});
+      if (own) add({SL_DKV, SL_DKV_NORM});
+      add({SL_UK, SL_UV});
+      if (L.sink == SINK_LEARNED) add({SL_SINK});
+    }
     if (L.mixer == MIX_GQA) {
-      const bool own = L.kv_from < 0;
       add({SL_Q});
-      if (own) add({SL_K, SL_V});
+      if (own) add({SL_K});
+      if (own && !L.values_from_keys) add({SL_V});
+      if (L.conv_taps > 0) add({SL_Q_CONV});
+      if (L.conv_taps > 0 && own) add({SL_K_CONV});
       if (L.qk_norm) add({SL_Q_NORM});
       if (L.qk_norm && own) add({SL_K_NORM});
       if (L.bias_rows > 0) add({SL_REL});
-      if (L.sink) add({SL_SINK});
+      if (L.sink == SINK_LEARNED) add({SL_SINK});
     }
     if (L.mixer == MIX_GLA) add({SL_Q, SL_K, SL_V, SL_A1, SL_A2, SL_A2_B, SL_V_GATE, SL_V_NORM});
     if (L.out_gate) out->push_back({SL_G, l, -1});
     out->push_back({SL_O, l, -1});
-    if (L.ff) out->push_back({SL_NORM2, l, -1});
+    if (L.ff && m->stack.block != BLOCK_ONE_NORM) out->push_back({SL_NORM2, l, -1});
     if (L.ff == 1)
       for (Slot s : {SL_GATE, SL_UP, SL_DOWN}) out->push_back({s, l, -1});
     if (L.ff == 2) {
@@ -67,6 +78,7 @@ void tensors_of(const rewb200_model* m, std::vector<TensorAt>* out) {
         out->push_back({SL_E_DOWN, l, e});
       }
       if (L.shared_ffn > 0) add({SL_S_GATE, SL_S_UP, SL_S_DOWN});
+      if (L.shared_gate) add({SL_S_SG});
     }
   }
   out->push_back({SL_FINAL, -1, -1});
@@ -110,6 +122,9 @@ int shape_of(const rewb200_model* m, const TensorAt& t, int64_t* rows, int64_t* 
     case SL_A2_B: v((int64_t)L->heads * L->dim); break;
     case SL_V_GATE: mat(d, (int64_t)L->heads * L->vdim); break;
     case SL_V_NORM: v(L->vdim); break;
+    case SL_Q_CONV: mat((int64_t)L->heads * L->dim, L->conv_taps); break;
+    case SL_K_CONV: mat((int64_t)L->kv_heads * L->dim, L->conv_taps); break;
+    case SL_S_SG: mat(d, 1); break;
   }
   return REWB200_OK;
 }
@@ -188,6 +203,17 @@ int upload_bias(rewb200_model* m, const rewb200_layer& L, GqaDev& G, const float
   return REWB200_OK;
 }
 
+// Convolution weights [taps][channels] from the stored [channels][taps] of queries or keys, whose first channel is c0.
+int upload_conv(rewb200_model* m, const GqaDev& G, int64_t c0, int64_t channels, const float* host) {
+  std::vector<float> t((size_t)G.m.taps * channels);
+  for (int64_t ch = 0; ch < channels; ++ch)
+    for (int j = 0; j < G.m.taps; ++j) t[(size_t)j * channels + ch] = host[ch * G.m.taps + j];
+  RB_CUDA(cudaMemcpy2DAsync(G.conv + c0, gqa_channels(G.m) * sizeof(float), t.data(), channels * sizeof(float), channels * sizeof(float), G.m.taps,
+                            cudaMemcpyHostToDevice, m->c->stream));
+  RB_CUDA(cudaStreamSynchronize(m->c->stream));
+  return REWB200_OK;
+}
+
 // The Linear weights of a layer's mixer that are no routed experts (all of them padded matrices of the model dtype).
 std::vector<LinW*> mixer_linears(LayerDev& D) {
   if (D.mixer == MIX_LATENT) return {&D.a.in, &D.a.uq, &D.a.ukv, &D.o};
@@ -207,11 +233,22 @@ int layered_create(rewb200_model* m, const rewb200_layer* layers, const rewb200_
   const rewb200_stack& st = m->stack;
   RB_REQUIRE(st.loop_times >= 0 && (st.loop_times == 0 || (st.loop_start >= 0 && st.loop_start < st.loop_stop && st.loop_stop <= n)),
              "layered model: the loop must cover layers start .. stop - 1 of the stack");
+  RB_REQUIRE(st.block >= BLOCK_PARALLEL && st.block <= BLOCK_ONE_NORM, "layered model: unknown block");
+  RB_REQUIRE(st.block != BLOCK_OUTPUT_NORM || st.loop_times == 0, "layered model: blocks normed on the way back run without a loop");
+  RB_REQUIRE(st.logit_softcap >= 0.f, "layered model: the cap of the logits must not be negative");
   for (int l = 0; l < n; ++l) {
     const rewb200_layer& L = m->spec[l];
     const std::string who = "layer " + std::to_string(l) + ": ";
     RB_REQUIRE(L.mixer >= MIX_LATENT && L.mixer <= MIX_GLA, who + "unknown mixer");
     RB_REQUIRE(L.heads > 0 && L.dim > 0 && L.vdim > 0, who + "mixer sizes must be positive");
+    RB_REQUIRE(L.sink >= SINK_NONE && L.sink <= SINK_ONE, who + "unknown sink");
+    RB_REQUIRE(L.conv_taps >= 0 && (L.mixer == MIX_GQA || (L.conv_taps == 0 && !L.values_from_keys)), who + "convolutions and values from keys belong to grouped-query attention");
+    if (L.kv_from >= 0) {
+      RB_REQUIRE(L.mixer != MIX_GLA && L.kv_from < l, who + "kv_from must name an earlier layer");
+      const rewb200_layer& S = m->spec[L.kv_from];
+      const bool same = L.mixer == MIX_LATENT ? S.kv_rank == L.kv_rank && S.rot_dim == L.rot_dim : S.kv_heads == L.kv_heads && S.dim == L.dim && S.vdim == L.vdim;
+      RB_REQUIRE(S.mixer == L.mixer && S.kv_from < 0 && same, who + "kv_from must name a layer of the same mixer with latents, or keys and values, of its own and the same sizes");
+    }
     if (L.mixer == MIX_LATENT) {
       RB_REQUIRE(L.rot_dim >= 0 && L.q_rank > 0 && L.kv_rank > 0, who + "mixer sizes must be positive");
       RB_REQUIRE(L.rope_dims >= 0 && L.rope_dims % 2 == 0 && L.rope_dims <= L.rot_dim, who + "rotated features must be pairs within rot_dim");
@@ -220,17 +257,14 @@ int layered_create(rewb200_model* m, const rewb200_layer* layers, const rewb200_
       RB_REQUIRE(L.kv_heads > 0 && L.heads % L.kv_heads == 0, who + "heads must be divisible by kv_heads");
       RB_REQUIRE(L.bias_rows >= 0 && (L.bias_rows == 0 || (L.bias_max > 0 && L.bias_max <= 1 << 20)), who + "the distance bias needs a positive bias_max");
       RB_REQUIRE(L.temp_every >= 0, who + "temp_every must not be negative");
-      if (L.kv_from >= 0) {
-        RB_REQUIRE(L.kv_from < l, who + "kv_from must name an earlier layer");
-        const rewb200_layer& S = m->spec[L.kv_from];
-        RB_REQUIRE(S.mixer == MIX_GQA && S.kv_from < 0 && S.kv_heads == L.kv_heads && S.dim == L.dim && S.vdim == L.vdim,
-                   who + "kv_from must name an attention layer with keys and values of its own and the same head sizes");
-      }
+      RB_REQUIRE(L.rope_dims >= 0 && L.rope_dims % 2 == 0 && L.rope_dims <= L.dim, who + "rotated features must be pairs within the head");
+      RB_REQUIRE(!L.values_from_keys || L.vdim == L.dim, who + "values that are the keys have their size");
     } else {
       RB_REQUIRE(L.decay_rank > 0 && L.tau > 0.f, who + "decay_rank and tau must be positive");
     }
     RB_REQUIRE(L.ff >= 0 && L.ff <= 2 && (L.ff == 0 || L.ffn > 0), who + "unknown feed-forward");
     RB_REQUIRE(L.shared_ffn >= 0 && (L.ff == 2 || L.shared_ffn == 0), who + "a shared expert stands beside routed ones");
+    RB_REQUIRE(!L.shared_gate || (L.shared_ffn > 0 && st.block != BLOCK_OUTPUT_NORM), who + "the gate of a shared expert needs one, in a parallel block");
     RB_REQUIRE(L.ff != 2 || (L.experts > 0 && L.experts <= 256 && L.top_k > 0 && L.top_k <= L.experts),
                who + "experts must be in 1..256 and top in 1..experts");
   }
@@ -239,6 +273,15 @@ int layered_create(rewb200_model* m, const rewb200_layer* layers, const rewb200_
   RB_TRY(zero_weights(m, &m->embed, (size_t)m->cfg.vocab * dp * es));
   if (st.loop_times > 0) RB_TRY(zero_weights(m, (void**)&m->step_vec, (size_t)st.loop_times * dp * sizeof(float)));
   std::map<std::pair<double, int>, float2*> tables;
+  auto rope_of = [&](const rewb200_layer& L, const float2** out) -> int {
+    if (L.rope_dims == 0) return REWB200_OK;
+    float2*& t = tables[{L.rope_base, L.rope_dims}];
+    if (!t) RB_TRY(rope_table(m, L.rope_base, L.rope_dims, &t));
+    *out = t;
+    return REWB200_OK;
+  };
+  // a sink of one is a score of zero: the zeros the array starts with
+  auto sink_of = [&](const rewb200_layer& L, float** out) { return L.sink ? zero_weights(m, (void**)out, L.heads * sizeof(float)) : REWB200_OK; };
   m->layers.resize(n);
   int64_t widest = dp, q_cols = 0, attn_cols = 0;
   for (int l = 0; l < n; ++l) {
@@ -246,35 +289,37 @@ int layered_create(rewb200_model* m, const rewb200_layer* layers, const rewb200_
     LayerDev& D = m->layers[l];
     D.mixer = L.mixer;
     RB_TRY(zero_weights(m, (void**)&D.ln1g, dp * sizeof(float)));
-    if (L.ff) RB_TRY(zero_weights(m, (void**)&D.ln2g, dp * sizeof(float)));
+    if (L.ff && st.block != BLOCK_ONE_NORM) RB_TRY(zero_weights(m, (void**)&D.ln2g, dp * sizeof(float)));
+    const bool own = L.kv_from < 0;
     if (L.mixer == MIX_LATENT) {
       LatentDev& A = D.a;
-      A.m = LatentDims{L.heads, L.dim, L.rot_dim, L.vdim, L.q_rank, L.kv_rank, L.rope_dims, L.window, L.out_gate, L.scale, nullptr, m->cfg.max_seq};
-      if (L.rope_dims > 0) {
-        float2*& t = tables[{L.rope_base, L.rope_dims}];
-        if (!t) RB_TRY(rope_table(m, L.rope_base, L.rope_dims, &t));
-        A.m.rope = t;
-      }
-      RB_TRY(zero_lin(m, &A.in, dp, pad8((int64_t)L.q_rank + L.kv_rank + L.rot_dim + (L.out_gate ? L.heads : 0))));
+      A.m = LatentDims{L.heads, L.dim, L.rot_dim, L.vdim, L.q_rank, L.kv_rank, L.rope_dims, L.window, L.out_gate, L.scale, nullptr, m->cfg.max_seq, own ? 1 : 0, nullptr};
+      RB_TRY(rope_of(L, &A.m.rope));
+      RB_TRY(sink_of(L, &A.sink));
+      A.m.sink = A.sink;
+      RB_TRY(zero_lin(m, &A.in, dp, pad8((int64_t)L.q_rank + (own ? L.kv_rank + L.rot_dim : 0) + (L.out_gate ? L.heads : 0))));
       RB_TRY(zero_lin(m, &A.uq, pad8(L.q_rank), pad8((int64_t)L.heads * (L.dim + L.rot_dim))));
       RB_TRY(zero_lin(m, &A.ukv, L.kv_rank, pad8((int64_t)L.heads * (L.dim + L.vdim))));
       RB_TRY(zero_weights(m, (void**)&A.q_norm, L.q_rank * sizeof(float)));
-      RB_TRY(zero_weights(m, (void**)&A.kv_norm, L.kv_rank * sizeof(float)));
+      if (own) RB_TRY(zero_weights(m, (void**)&A.kv_norm, L.kv_rank * sizeof(float)));
       A.ldc = pad8(L.kv_rank + L.rot_dim);
       widest = std::max(widest, std::max(A.in.N, A.uq.N));
       q_cols = std::max(q_cols, A.uq.N);
     } else if (L.mixer == MIX_GQA) {
       GqaDev& G = D.g;
-      const bool own = L.kv_from < 0;
       G.ldk = pad8(L.dim);
       G.ldv = pad8(L.vdim);
-      RB_TRY(zero_lin(m, &G.in, dp, pad8((int64_t)L.heads * L.dim + (own ? (int64_t)L.kv_heads * (L.dim + L.vdim) : 0) + (L.out_gate ? L.heads : 0))));
+      RB_TRY(zero_lin(m, &G.in, dp, pad8((int64_t)L.heads * L.dim + (own ? (int64_t)L.kv_heads * (L.dim + (L.values_from_keys ? 0 : L.vdim)) : 0) + (L.out_gate ? L.heads : 0))));
       if (L.qk_norm) RB_TRY(zero_weights(m, (void**)&G.q_norm, L.dim * sizeof(float)));
       if (L.qk_norm && own) RB_TRY(zero_weights(m, (void**)&G.k_norm, L.dim * sizeof(float)));
       const int nb = L.bias_rows > 0 ? bias_distances(L.bias_rows, L.bias_max) : 0;
       if (nb > 0) RB_TRY(zero_weights(m, (void**)&G.bias, (size_t)L.heads * nb * sizeof(float)));
-      if (L.sink) RB_TRY(zero_weights(m, (void**)&G.sink, L.heads * sizeof(float)));
-      G.m = GqaDims{L.heads, L.kv_heads, L.dim, L.vdim, own ? 1 : 0, L.out_gate, L.scale, G.q_norm, G.k_norm, L.temp_every, L.temp_coef, G.bias, nb, G.sink};
+      RB_TRY(sink_of(L, &G.sink));
+      G.m = GqaDims{L.heads, L.kv_heads, L.dim, L.vdim, own ? 1 : 0, L.out_gate, L.scale, G.q_norm, G.k_norm, L.temp_every, L.temp_coef, G.bias, nb, G.sink,
+                    L.values_from_keys, L.conv_taps, nullptr, L.rope_dims, nullptr};
+      RB_TRY(rope_of(L, &G.m.rope));
+      if (L.conv_taps > 0) RB_TRY(zero_weights(m, (void**)&G.conv, (size_t)L.conv_taps * gqa_channels(G.m) * sizeof(float)));
+      G.m.conv = G.conv;
       widest = std::max(widest, G.in.N);
       q_cols = std::max(q_cols, pad8((int64_t)L.heads * L.dim));
     } else {
@@ -302,10 +347,12 @@ int layered_create(rewb200_model* m, const rewb200_layer* layers, const rewb200_
       X.E = X.E_l = L.experts;
       X.top_k = L.top_k;
       X.renorm = L.renormalize;
+      X.scale = L.router_scale == 0.f ? 1.f : L.router_scale;
+      X.shared_gate = L.shared_gate != 0;
       X.gated = L.expert_gated != 0;
       X.f = fp;
       const int64_t up = X.gated ? 2 * fp : fp;
-      RB_TRY(zero_lin(m, &X.router, dp, pad8(L.experts)));
+      RB_TRY(zero_lin(m, &X.router, dp, pad8(L.experts + (X.shared_gate ? 1 : 0))));
       RB_TRY(zero_weights(m, &X.gu, (size_t)L.experts * dp * up * es));
       RB_TRY(zero_weights(m, &X.down, (size_t)L.experts * fp * dp * es));
       RB_TRY(zero_weights(m, (void**)&X.gu_b, (size_t)L.experts * up * sizeof(float)));
@@ -327,9 +374,6 @@ int layered_create(rewb200_model* m, const rewb200_layer* layers, const rewb200_
   RB_TRY(zero_lin(m, &m->lm, dp, m->vp));
   const int a = st.loop_times > 0 ? st.loop_start : n, b = st.loop_times > 0 ? st.loop_stop : n;
   for (int l = 0; l < a; ++l) m->runs.push_back({l, false, -1});
-  RB_REQUIRE(st.block == 0 || (st.block == 1 && st.loop_times == 0), "layered model: blocks normed on the way back run without a loop");
-  RB_REQUIRE(st.block == 1 || m->max_topk == 0 || std::none_of(m->spec.begin(), m->spec.end(), [](const rewb200_layer& L) { return L.shared_ffn > 0; }),
-             "layered model: a shared expert needs blocks normed on the way back");
   for (int p = 0; p < st.loop_times; ++p)
     for (int l = a; l < b; ++l) m->runs.push_back({l, l == a && p > 0, l == a ? p : -1});
   for (int l = b; l < n; ++l) m->runs.push_back({l, false, -1});
@@ -338,7 +382,7 @@ int layered_create(rewb200_model* m, const rewb200_layer* layers, const rewb200_
     if (m->layers[R.layer].moe) ++m->n_moe;
     R.cache = (int)r;
     const rewb200_layer& L = m->spec[R.layer];
-    if (L.mixer == MIX_GQA && L.kv_from >= 0)   // the latest run of that layer: in a loop, the one of the same pass
+    if (L.mixer != MIX_GLA && L.kv_from >= 0)   // the latest run of that layer: in a loop, the one of the same pass
       for (size_t q = 0; q < r; ++q)
         if (m->runs[q].layer == L.kv_from) R.cache = (int)q;
   }
@@ -416,7 +460,9 @@ int layered_set_tensor(rewb200_model* m, int64_t index, const float* host, int64
       case SL_Q: return cols(G.in.w, G.in.N, 0);
       case SL_K: return cols(G.in.w, G.in.N, hk);
       case SL_V: return cols(G.in.w, G.in.N, hk + kv * L.dim);
-      case SL_G: return cols(G.in.w, G.in.N, hk + kv * (L.dim + L.vdim));
+      case SL_G: return cols(G.in.w, G.in.N, hk + kv * (L.dim + (L.values_from_keys ? 0 : L.vdim)));
+      case SL_Q_CONV: return upload_conv(m, G, 0, hk, host);
+      case SL_K_CONV: return upload_conv(m, G, hk, kv * L.dim, host);
       case SL_Q_NORM: return norm(G.q_norm, false);
       case SL_K_NORM: return norm(G.k_norm, false);
       case SL_SINK: return vector(G.sink);
@@ -445,7 +491,8 @@ int layered_set_tensor(rewb200_model* m, int64_t index, const float* host, int64
     case SL_DKV_NORM: return norm(A.kv_norm, false);
     case SL_DQ: return cols(A.in.w, A.in.N, 0);
     case SL_DKV: return cols(A.in.w, A.in.N, L.q_rank);
-    case SL_G: return cols(A.in.w, A.in.N, (int64_t)L.q_rank + L.kv_rank + L.rot_dim);
+    case SL_G: return cols(A.in.w, A.in.N, (int64_t)L.q_rank + (L.kv_from < 0 ? L.kv_rank + L.rot_dim : 0));
+    case SL_SINK: return vector(A.sink);
     case SL_UQ: return cols(A.uq.w, A.uq.N, 0);
     case SL_UK: return cols(A.ukv.w, A.ukv.N, 0);
     case SL_UV: return cols(A.ukv.w, A.ukv.N, (int64_t)L.heads * L.dim);
@@ -458,6 +505,7 @@ int layered_set_tensor(rewb200_model* m, int64_t index, const float* host, int64
     case SL_S_GATE: return gate_up(D.gu.w, false, L.shared_ffn);
     case SL_S_UP: return gate_up(D.gu.w, true, L.shared_ffn);
     case SL_S_DOWN: return cols(D.down.w, m->dp, 0);
+    case SL_S_SG: return cols(D.x.router.w, D.x.router.N, L.experts);
     case SL_E_DOWN: return cols((char*)D.x.down + (size_t)t.expert * fp * m->dp * es, m->dp, 0);
     case SL_E_GATE: return gate_up((char*)D.x.gu + (size_t)t.expert * m->dp * 2 * fp * es, false, L.ffn);
     case SL_E_UP:
@@ -479,13 +527,14 @@ int layered_init_random(rewb200_model* m, uint64_t seed, float std) {
   RB_TRY(fill_const_launch(c, m->ng, REWB200_F32, m->dp, 1.f));
   for (LayerDev& D : m->layers) {
     RB_TRY(fill_const_launch(c, D.ln1g, REWB200_F32, m->dp, 1.f));
-    if (D.ff) RB_TRY(fill_const_launch(c, D.ln2g, REWB200_F32, m->dp, 1.f));
+    if (D.ln2g) RB_TRY(fill_const_launch(c, D.ln2g, REWB200_F32, m->dp, 1.f));
     if (D.mixer == MIX_LATENT) {
       RB_TRY(fill_const_launch(c, D.a.q_norm, REWB200_F32, D.a.m.q_rank, 1.f));
-      RB_TRY(fill_const_launch(c, D.a.kv_norm, REWB200_F32, D.a.m.kv_rank, 1.f));
+      if (D.a.kv_norm) RB_TRY(fill_const_launch(c, D.a.kv_norm, REWB200_F32, D.a.m.kv_rank, 1.f));
     } else if (D.mixer == MIX_GQA) {
       if (D.g.q_norm) RB_TRY(fill_const_launch(c, D.g.q_norm, REWB200_F32, D.g.m.dim, 1.f));
       if (D.g.k_norm) RB_TRY(fill_const_launch(c, D.g.k_norm, REWB200_F32, D.g.m.dim, 1.f));
+      if (D.g.conv) RB_TRY(fill_normal_launch(c, D.g.conv, REWB200_F32, D.g.m.taps * gqa_channels(D.g.m), ++k, 0.5f));
       if (D.g.bias) RB_TRY(fill_normal_launch(c, D.g.bias, REWB200_F32, (int64_t)D.g.m.heads * D.g.m.n_bias, ++k, 1.f));
     } else {
       RB_TRY(fill_const_launch(c, D.l.norm, REWB200_F32, D.l.m.vdim, 1.f));
@@ -536,6 +585,10 @@ int layered_acts(rewb200_session* s, int64_t rows) {
   RB_TRY(acts_alloc(c, &s->cq, (size_t)rows * cq * es));
   RB_TRY(acts_alloc(c, (void**)&s->gate, (size_t)rows * heads * sizeof(float)));
   RB_TRY(acts_alloc(c, (void**)&s->part2, s->part_bytes));
+  if (m->stack.block != BLOCK_OUTPUT_NORM && std::any_of(m->spec.begin(), m->spec.end(), [](const rewb200_layer& L) { return L.shared_ffn > 0; })) {
+    RB_TRY(acts_alloc(c, (void**)&s->part3, s->part_bytes));
+    RB_TRY(acts_alloc(c, (void**)&s->shared_gate, (size_t)rows * sizeof(float)));
+  }
   if (c->record_layers) RB_TRY(acts_alloc(c, (void**)&s->layer_rec, m->runs.size() * (size_t)rows * m->dp * sizeof(float)));
   // padding columns are multiplied by zero weights, so they must hold finite values from the start
   RB_CUDA(cudaMemsetAsync(s->cq, 0, (size_t)rows * cq * es, c->stream));
@@ -566,11 +619,12 @@ int layered_session(rewb200_session* s, int64_t n_pages) {
   };
   for (size_t r = 0; r < n; ++r) {
     const LayerDev& D = m->layers[m->runs[r].layer];
-    if (D.mixer == MIX_LATENT) RB_TRY(pages(&s->kc[r], &s->tmK[r], n_pages * PAGE, D.a.ldc));
+    if (D.mixer == MIX_LATENT && D.a.m.own_kv) RB_TRY(pages(&s->kc[r], &s->tmK[r], n_pages * PAGE, D.a.ldc));
     if (D.mixer == MIX_GQA && D.g.m.own_kv) {
       RB_TRY(pages(&s->kc[r], &s->tmK[r], n_pages * D.g.m.kv_heads * PAGE, D.g.ldk));
       RB_TRY(pages(&s->vc[r], &s->tmV[r], n_pages * D.g.m.kv_heads * PAGE, D.g.ldv));
     }
+    if (D.mixer == MIX_GQA && gqa_state_elems(D.g.m) > 0) RB_TRY(zeroed((void**)&s->state[r], (size_t)s->B * gqa_state_elems(D.g.m) * sizeof(float)));
     // a state needs no clearing between sequences: a portion that starts at position 0 does not read it
     if (D.mixer == MIX_GLA)
       RB_TRY(zeroed((void**)&s->state[r], (size_t)s->B * D.l.m.heads * D.l.m.dim * gla_state_ld(D.l.m.vdim) * sizeof(float)));
@@ -616,10 +670,11 @@ int layered_prepare(rewb200_session* s, const FwdOpts& o, int64_t rows) {
   const bool uniform = o.entries == nullptr;
   RB_REQUIRE(!uniform || o.S == 1, "layered step: a step of several tokens per lane needs its portions");
   // ---- lists of the step: [row lane | row position | absorbed tiles | their chunks | expanded tiles | gathered keys |
-  // chunks of gated linear attention | small and large tiles of grouped-query attention | small and large portions of gated linear attention]
+  // chunks of gated linear attention | last rows of the portions | small and large tiles of grouped-query attention | small and
+  // large portions of gated linear attention]
   int64_t abs_rows = rows, n_keys = 0;
   s->plan_host.clear();
-  s->plan_abs_tiles = s->plan_chunks = s->plan_exp_tiles = s->plan_keys = s->plan_gla_chunks = 0;
+  s->plan_abs_tiles = s->plan_chunks = s->plan_exp_tiles = s->plan_keys = s->plan_gla_chunks = s->plan_tails = 0;
   if (!uniform) {
     std::vector<int>& h = s->plan_host;
     h.assign(2 * rows, 0);
@@ -630,10 +685,12 @@ int layered_prepare(rewb200_session* s, const FwdOpts& o, int64_t rows) {
     const bool bf = m->cfg.dtype == REWB200_BF16;
     bool exp_ok = bf && c->latent_impl == 0, gqa_ok = bf && c->gqa_impl == 0, gla_ok = bf && c->gla_impl == 0;
     bool has_latent = false, has_gqa = false, has_gla = false;
+    int taps = 0;           // of the longest convolution
     for (const LayerDev& D : m->layers) {
       if (D.mixer == MIX_GQA) {
         has_gqa = true;
         gqa_ok = gqa_ok && gqa_prefill_ok(D.g.m);
+        taps = std::max(taps, D.g.m.taps);
       }
       if (D.mixer == MIX_GLA) {
         has_gla = true;
@@ -647,12 +704,13 @@ int layered_prepare(rewb200_session* s, const FwdOpts& o, int64_t rows) {
     std::vector<int2> gqa_small;
     std::vector<GqaTile> gqa_large;
     std::vector<GlaPortion> gla_small, gla_large;
-    std::vector<int2> gla_chunk;
+    std::vector<int2> gla_chunk, tails;
     for (const StepEntry& e : *o.entries) {
       for (int i = 0; i < e.n; ++i) {
         h[e.row0 + i] = e.lane;
         h[rows + e.row0 + i] = e.pos0 + i;
       }
+      for (int i = 0; i < std::min(taps - 1, e.n); ++i) tails.push_back(make_int2(e.row0 + e.n - 1 - i, i));
       if (has_gqa) {
         if (gqa_ok && e.n >= LARGE_MIN_ROWS)
           for (int i = 0; i < e.n; i += 256) gqa_large.push_back({e.row0 + i, std::min(256, e.n - i), e.pos0 + i, e.lane});
@@ -693,6 +751,7 @@ int layered_prepare(rewb200_session* s, const FwdOpts& o, int64_t rows) {
     s->plan_gla_small = (int)gla_small.size();
     s->plan_gla_large = (int)gla_large.size();
     s->plan_gla_chunks = (int)gla_chunk.size();
+    s->plan_tails = (int)tails.size();
     s->plan_abs_tiles = (int)tiles.size();
     s->plan_chunks = (int)chunks.size();
     s->plan_exp_tiles = (int)exps.size();
@@ -708,6 +767,7 @@ int layered_prepare(rewb200_session* s, const FwdOpts& o, int64_t rows) {
     append(exps.data(), exps.size() * sizeof(ExpTile));
     append(keys.data(), keys.size() * sizeof(int2));
     append(gla_chunk.data(), gla_chunk.size() * sizeof(int2));
+    append(tails.data(), tails.size() * sizeof(int2));
     append(gqa_small.data(), gqa_small.size() * sizeof(int2));
     append(gqa_large.data(), gqa_large.size() * sizeof(GqaTile));
     append(gla_small.data(), gla_small.size() * sizeof(GlaPortion));
@@ -794,7 +854,7 @@ struct StepLists {
   RowMap map = {};
   RowTiles abs = {}, chunks = {};
   const ExpTile* exp_tiles = nullptr;
-  const int2 *key_list = nullptr, *gla_chunks = nullptr;
+  const int2 *key_list = nullptr, *gla_chunks = nullptr, *tails = nullptr;
   RowTiles gqa_small = {};
   const GqaTile* gqa_large = nullptr;
   const GlaPortion *gla_small = nullptr, *gla_large = nullptr;
@@ -816,7 +876,8 @@ StepLists step_lists(const rewb200_session* s, const FwdOpts& o, int64_t rows) {
   t.exp_tiles = reinterpret_cast<const ExpTile*>(t.chunks.list + t.chunks.count);
   t.key_list = reinterpret_cast<const int2*>(t.exp_tiles + s->plan_exp_tiles);
   t.gla_chunks = t.key_list + s->plan_keys;
-  t.gqa_small.list = t.gla_chunks + s->plan_gla_chunks;
+  t.tails = t.gla_chunks + s->plan_gla_chunks;
+  t.gqa_small.list = t.tails + s->plan_tails;
   t.gqa_small.count = s->plan_gqa_small;
   t.gqa_large = reinterpret_cast<const GqaTile*>(t.gqa_small.list + t.gqa_small.count);
   t.gla_small = reinterpret_cast<const GlaPortion*>(t.gqa_large + s->plan_gqa_large);
@@ -859,7 +920,11 @@ int gqa_mixer(rewb200_session* s, const FwdOpts& o, const StepLists& t, size_t r
   pa.dtype = dt;
   pa.early = in_graph ? 1 : 0;
   pa.status = c->d_status;
+  pa.state = s->state[r];
+  pa.tails = t.tails;
+  pa.n_tails = s->plan_tails;
   RB_TRY(gqa_post_launch(c, pa, rows));
+  if (!t.uniform) RB_TRY(gqa_conv_state_launch(c, pa));
   if (o.trace) RB_TRY(o.trace->mark(TC_QKV_POST));
   GqaAttnArgs aa;
   memset(&aa, 0, sizeof(aa));
@@ -955,7 +1020,8 @@ int latent_mixer(rewb200_session* s, const FwdOpts& o, const StepLists& t, size_
   rewb200_model* m = s->m;
   Ctx* c = m->c;
   const int dt = m->cfg.dtype;
-  LayerDev& D = m->layers[m->runs[r].layer];
+  const LayerRun& R = m->runs[r];
+  LayerDev& D = m->layers[R.layer];
   LatentDev& A = D.a;
   const bool expand = !t.uniform && s->plan_exp_tiles > 0;
   int ks = 1;
@@ -975,7 +1041,7 @@ int latent_mixer(rewb200_session* s, const FwdOpts& o, const StepLists& t, size_
   pa.cq = s->cq;
   pa.ldcq = A.uq.K;
   pa.gate = s->gate;
-  pa.cache = s->kc[r];
+  pa.cache = s->kc[R.cache];
   pa.block_table = s->block_table;
   pa.max_pages = s->max_pages;
   pa.capacity = s->max_len;
@@ -1012,8 +1078,8 @@ int latent_mixer(rewb200_session* s, const FwdOpts& o, const StepLists& t, size_
   aa.gate = s->gate;
   aa.out = s->attn;
   aa.ldo = D.o.K;
-  aa.cache = s->kc[r];
-  aa.tm_cache = dt == REWB200_BF16 ? &s->tmK[r] : nullptr;
+  aa.cache = s->kc[R.cache];
+  aa.tm_cache = dt == REWB200_BF16 ? &s->tmK[R.cache] : nullptr;
   aa.block_table = s->block_table;
   aa.max_pages = s->max_pages;
   aa.ldc = A.ldc;
@@ -1039,7 +1105,7 @@ int latent_mixer(rewb200_session* s, const FwdOpts& o, const StepLists& t, size_
     ea.ldc = A.ldc;
     ea.keys = s->plan_keys;
     ea.status = c->d_status;
-    RB_TRY(latent_gather_launch(c, (const bf16*)s->kc[r], s->block_table, s->max_pages, A.ldc, t.key_list, (bf16*)s->latx, s->plan_keys));
+    RB_TRY(latent_gather_launch(c, (const bf16*)s->kc[R.cache], s->block_table, s->max_pages, A.ldc, t.key_list, (bf16*)s->latx, s->plan_keys));
     RB_TRY(linear_bf16_launch(c, A.ukv.plan, (const bf16*)s->latx, A.ldc, s->plan_keys, EPI_BIAS_BF16, 1, s->kvx, A.ukv.N, nullptr, nullptr, 0));
     RB_TRY(latent_attn_expanded_launch(c, ea));
   }
@@ -1181,7 +1247,8 @@ int layered_blocks(rewb200_session* s, const FwdOpts& o, const NormArgs& na, int
   Ctx* c = m->c;
   const int dt = m->cfg.dtype;
   const int64_t dp = m->dp;
-  if (m->stack.block == 1) return output_norm_blocks(s, o, na, rows, in_graph);
+  if (m->stack.block == BLOCK_OUTPUT_NORM) return output_norm_blocks(s, o, na, rows, in_graph);
+  void* const ff_in = m->stack.block == BLOCK_ONE_NORM ? s->xn : s->xn2;   // what the feed-forward reads
   const StepLists t = step_lists(s, o, rows);
   auto ahead_of = [&](size_t r, NormArgs& a) {  // what the norm launch in front of run r adds and writes
     if (r == m->runs.size()) {
@@ -1191,7 +1258,7 @@ int layered_blocks(rewb200_session* s, const FwdOpts& o, const NormArgs& na, int
     const LayerRun& R = m->runs[r];
     const LayerDev& D = m->layers[R.layer];
     a.gamma = D.ln1g;
-    if (D.ff) {
+    if (D.ln2g) {
       a.gamma2 = D.ln2g;
       a.out2 = s->xn2;
     }
@@ -1211,27 +1278,29 @@ int layered_blocks(rewb200_session* s, const FwdOpts& o, const NormArgs& na, int
   int moe_seen = 0;
   for (size_t r = 0; r < m->runs.size(); ++r) {
     LayerDev& D = m->layers[m->runs[r].layer];
-    int ks_o = 1, ks_f = 0;
+    int ks_o = 1, ks_f = 0, ks_s = 0;
     const bool fork = D.ff != 0 && dt == REWB200_BF16 && rows <= 64 && c->moe_overlap && !o.trace;
-    // ---- feed-forward branch: slabs in part2
+    const bool pdl = c->use_pdl;
+    // ---- feed-forward branch: slabs in part2, those of a shared expert in part3
     auto ff_branch = [&]() -> int {
       if (D.ff == 0) return REWB200_OK;
       float* const keep = s->part;
-      s->part = s->part2;  // scratch and slabs of this branch
-      auto body = [&]() -> int {
-        if (D.ff == 2) {
-          RB_TRY(moe_routed(s, D.x, s->xn2, dp, rows, false, s->part2, moe_seen++, fork));
-          ks_f = 1;
-          if (o.trace) RB_TRY(o.trace->mark(TC_MOE));
-          return REWB200_OK;
-        }
-        // beside the mixer both Linears are plain launches: a down projection launched early holds shared memory that the
-        // mixer's short kernels then wait for (measured, 8B shape: 3.69 instead of 3.53 ms per step at batch 32)
-        const bool pdl = c->use_pdl;
+      // beside the mixer both Linears are plain launches: a down projection launched early holds shared memory that the
+      // mixer's short kernels then wait for (measured, 8B shape: 3.69 instead of 3.53 ms per step at batch 32)
+      auto dense = [&](float* out, int* ks) -> int {
+        s->part = out;   // scratch and slabs of this branch
         if (fork) c->use_pdl = false;
-        const int st = dense_ff(s, o, D, s->xn2, rows, s->part2, &ks_f);
+        const int st = dense_ff(s, o, D, ff_in, rows, out, ks);
         c->use_pdl = pdl;
         return st;
+      };
+      auto body = [&]() -> int {
+        if (D.ff != 2) return dense(s->part2, &ks_f);
+        s->part = s->part2;
+        RB_TRY(moe_routed(s, D.x, ff_in, dp, rows, false, s->part2, moe_seen++, fork));
+        ks_f = 1;
+        if (o.trace) RB_TRY(o.trace->mark(TC_MOE));
+        return has_dense(D) ? dense(s->part3, &ks_s) : REWB200_OK;
       };
       const int st = body();
       s->part = keep;
@@ -1254,9 +1323,13 @@ int layered_blocks(rewb200_session* s, const FwdOpts& o, const NormArgs& na, int
       a.partial2 = s->part2;
       a.nsplit2 = ks_f;
     }
+    if (ks_s > 0) {
+      a.partial3 = s->part3;
+      a.nsplit3 = ks_s;
+      a.scale3 = D.x.shared_gate ? s->shared_gate : nullptr;
+    }
     ahead_of(r + 1, a);
     if (a.add_embed) a.embed = m->embed;
-    const bool pdl = c->use_pdl;
     if (fork) c->use_pdl = false;  // two predecessors: a plain dependency
     if (s->layer_rec && !t.uniform) {
       // the residual as the layer leaves it, ahead of what a loop adds
@@ -1269,8 +1342,8 @@ int layered_blocks(rewb200_session* s, const FwdOpts& o, const NormArgs& na, int
       RB_TRY(residual_norm_launch(c, b, rows));
       RB_CUDA(cudaMemcpyAsync(s->layer_rec + r * s->rows_cap * dp, s->x_res, (size_t)rows * dp * sizeof(float), cudaMemcpyDeviceToDevice, c->stream));
       s->layer_rows = rows;
-      a.partial = a.partial2 = nullptr;
-      a.nsplit = a.nsplit2 = 0;
+      a.partial = a.partial2 = a.partial3 = nullptr;
+      a.nsplit = a.nsplit2 = a.nsplit3 = 0;
     }
     const int st = residual_norm_launch(c, a, rows);
     c->use_pdl = pdl;

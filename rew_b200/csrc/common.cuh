@@ -272,6 +272,9 @@ struct NormArgs {
   // Blocks whose branches read two norms of one x, and stacks that run a range of layers several times:
   const float* partial2;  // a second set of f32 slabs added like `partial` (same split_stride), or nullptr
   int nsplit2;
+  const float* partial3;  // a third set whose sum is multiplied by scale3[row] (nullptr: by one), or nullptr
+  int nsplit3;
+  const float* scale3;
   const float* gamma2;    // a second RMS norm of the same row: out2 = gamma2 * x / rms, or nullptr
   void* out2;
   int add_embed;          // 1: the embedding row of ids[row] is ADDED to the residual instead of replacing it
@@ -279,6 +282,8 @@ struct NormArgs {
   int64_t d_mean;         // width the row statistics divide by when rows are padded (0: d); the padding is zero
 };
 int residual_norm_launch(Ctx* c, const NormArgs& a, int64_t rows);
+// dst = cap * tanh(src / cap), n columns of `rows` rows; src may be dst.
+int softcap_launch(Ctx* c, const float* src, int64_t lds, float* dst, int64_t ldd, int64_t rows, int64_t n, float cap);
 
 // Blocks whose sublayers read the residual itself and are normed on the way back: x += gamma * y / rms(y), y the sum of two
 // sets of f32 slabs.  Leaves x (or, with final_gamma, its RMS norm) in `out`.  Without slabs the row is only written out;

@@ -85,6 +85,11 @@ __global__ void __launch_bounds__(NORM_THREADS) residual_norm_kernel(NormArgs a)
       float p = 0.f;
       for (int s = 0; s < a.nsplit; ++s) p += a.partial[s * a.split_stride + row * d + i];
       for (int s = 0; s < a.nsplit2; ++s) p += a.partial2[s * a.split_stride + row * d + i];
+      if (a.nsplit3 > 0) {
+        float z = 0.f;
+        for (int s = 0; s < a.nsplit3; ++s) z += a.partial3[s * a.split_stride + row * d + i];
+        p += a.scale3 ? z * a.scale3[row] : z;
+      }
       if (a.bias) p += a.bias[i];
       v += p;
     }
@@ -182,7 +187,7 @@ __device__ __forceinline__ float4 partial_sum4(const NormArgs& a, int64_t idx) {
   return p;
 }
 
-// What a block with two branches, or a stack that runs layers several times, adds on top (NormArgs::partial2,
+// What a block with several branches, or a stack that runs layers several times, adds on top (NormArgs::partial2, partial3,
 // add_embed, add_vec) at column i of a row; idx = row * d + i.
 __device__ __forceinline__ void add4(float4& v, const float4 w) { v.x += w.x; v.y += w.y; v.z += w.z; v.w += w.w; }
 __device__ __forceinline__ float4 partial2_sum4(const NormArgs& a, int64_t idx) {
@@ -190,6 +195,13 @@ __device__ __forceinline__ float4 partial2_sum4(const NormArgs& a, int64_t idx) 
 #pragma unroll 4
   for (int s = 0; s < a.nsplit2; ++s) add4(p, *reinterpret_cast<const float4*>(a.partial2 + s * a.split_stride + idx));
   return p;
+}
+__device__ __forceinline__ float4 partial3_sum4(const NormArgs& a, int64_t row, int64_t idx) {
+  float4 p = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 4
+  for (int s = 0; s < a.nsplit3; ++s) add4(p, *reinterpret_cast<const float4*>(a.partial3 + s * a.split_stride + idx));
+  const float f = a.scale3 ? a.scale3[row] : 1.0f;
+  return make_float4(p.x * f, p.y * f, p.z * f, p.w * f);
 }
 
 // One 16-byte line of the one-shot exchange: two 4-byte payload words, each followed by the flag of this
@@ -387,6 +399,7 @@ __global__ void __launch_bounds__(NORMV_THREADS) residual_norm_vec_kernel(NormAr
       if (summed) {
         float4 p = vals[c];
         if (a.nsplit2 > 0) add4(p, partial2_sum4(a, row * d + i));
+        if (a.nsplit3 > 0) add4(p, partial3_sum4(a, row, row * d + i));
         if (a.bias) {
           const float4 b = *reinterpret_cast<const float4*>(a.bias + i);
           p.x += b.x; p.y += b.y; p.z += b.z; p.w += b.w;
@@ -591,6 +604,7 @@ __global__ void __cluster_dims__(4, 1, 1) __launch_bounds__(256) residual_norm_c
       if (summed) {
         float4 p = vals[c];
         if (a.nsplit2 > 0) add4(p, partial2_sum4(a, row * d + i));
+        if (a.nsplit3 > 0) add4(p, partial3_sum4(a, row, row * d + i));
         if (a.bias) {
           const float4 b = *reinterpret_cast<const float4*>(a.bias + i);
           p.x += b.x; p.y += b.y; p.z += b.z; p.w += b.w;
@@ -1131,6 +1145,31 @@ int output_norm_launch(Ctx* c, const OutputNormArgs& a, int64_t rows) {
   const int nch = (int)((a.d / 4 + 511) / 512);
   return bf ? RB_ONORM(bf16, 1) : RB_ONORM(float, 1);
 #undef RB_ONORM
+}
+
+// dst[r][i] = cap * tanh(src[r][i] / cap) for the first n columns of every row; src may be dst
+__global__ void __launch_bounds__(256) softcap_kernel(const float* src, int64_t lds, float* dst, int64_t ldd, int64_t n, float cap) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int64_t r = blockIdx.y, i = ((int64_t)blockIdx.x * 256 + threadIdx.x) * 4;
+  if (i >= n) return;
+  const float* s = src + r * lds + i;
+  float* d = dst + r * ldd + i;
+  if (i + 4 <= n && lds % 4 == 0 && ldd % 4 == 0) {
+    const float4 v = *reinterpret_cast<const float4*>(s);
+    *reinterpret_cast<float4*>(d) = make_float4(cap * tanhf(v.x / cap), cap * tanhf(v.y / cap), cap * tanhf(v.z / cap), cap * tanhf(v.w / cap));
+    return;
+  }
+  for (int u = 0; u < 4 && i + u < n; ++u) d[u] = cap * tanhf(s[u] / cap);
+}
+
+int softcap_launch(Ctx* c, const float* src, int64_t lds, float* dst, int64_t ldd, int64_t rows, int64_t n, float cap) {
+  for (int64_t r = 0; r < rows; r += 32768) {
+    const dim3 grid((unsigned)((n + 1023) / 1024), (unsigned)std::min<int64_t>(32768, rows - r));
+    RB_CUDA(launch_k(softcap_kernel, grid, dim3(256), 0, c->stream, c->use_pdl, src + r * lds, lds, dst + r * ldd, ldd, n, cap));
+    ++g_launch_total;
+  }
+  return REWB200_OK;
 }
 
 int residual_norm_launch(Ctx* c, const NormArgs& a, int64_t rows) {

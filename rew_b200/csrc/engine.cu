@@ -276,7 +276,7 @@ int ensure_acts(rewb200_session* s, int64_t rows, int64_t logits_rows) {
                      (void**)&s->moe_logits, (void**)&s->moe_topw, (void**)&s->moe_topi, (void**)&s->moe_ints, &s->moe_send,
                      &s->moe_recv, &s->moe_xs, &s->moe_hs, (void**)&s->moe_ys, (void**)&s->moe_ret, (void**)&s->moe_back,
                      (void**)&s->moe_tmp, (void**)&s->route_rec, &s->xn2, &s->cq, (void**)&s->gate, (void**)&s->part2,
-                     (void**)&s->layer_rec};
+                     (void**)&s->part3, (void**)&s->shared_gate, (void**)&s->layer_rec};
     // From here until every allocation below has succeeded the session holds no activation buffers: a failed
     // growth must leave it in a state where the next call allocates again instead of launching on NULL.
     s->rows_cap = 0;
@@ -446,6 +446,7 @@ int moe_routed(rewb200_session* s, MoeDev& X, const void* x, int64_t d, int64_t 
   // expert parallel over the peer heap: the routing kernel also clears the dispatch kernel's per-peer cursors
   const bool peer = ep_uses_peer_heap(m, rows);
   int* const clear = peer ? s->moe_ints : nullptr;
+  float* const gate = X.shared_gate ? s->shared_gate : nullptr;
   bool cleared = false;
   const bool pdl = c->use_pdl;
   if (first_plain) c->use_pdl = false;  // the router Linear follows an event wait: a plain dependency
@@ -458,7 +459,7 @@ int moe_routed(rewb200_session* s, MoeDev& X, const void* x, int64_t d, int64_t 
                                       nullptr, nullptr, 0);
     c->use_pdl = pdl;
     RB_TRY(st);
-    RB_TRY(moe_route_slabs_launch(c, s->moe_logits, ks, rows * ldr, X.router.b, rows, X.E, ldr, k, X.renorm, s->moe_topw,
+    RB_TRY(moe_route_slabs_launch(c, s->moe_logits, ks, rows * ldr, X.router.b, rows, X.E, ldr, k, X.renorm, X.scale, gate, s->moe_topw,
                                   s->moe_topi, clear, peer ? ep : 0));
     cleared = peer;
   } else {
@@ -468,7 +469,7 @@ int moe_routed(rewb200_session* s, MoeDev& X, const void* x, int64_t d, int64_t 
     else
       RB_TRY(gemm_f32_launch(c, (const float*)x, (const float*)X.router.w, X.router.b, s->moe_logits, rows, d, ldr));
     c->use_pdl = pdl;
-    RB_TRY(moe_route_slabs_launch(c, s->moe_logits, 1, 0, nullptr, rows, X.E, ldr, k, X.renorm, s->moe_topw, s->moe_topi, nullptr, 0));
+    RB_TRY(moe_route_slabs_launch(c, s->moe_logits, 1, 0, nullptr, rows, X.E, ldr, k, X.renorm, X.scale, gate, s->moe_topw, s->moe_topi, nullptr, 0));
   }
   if (s->route_rec) {
     RB_CUDA(cudaMemcpyAsync(s->route_rec + (size_t)moe_index * s->rows_cap * m->max_topk, s->moe_topi, (size_t)rows * k * sizeof(int),
@@ -986,7 +987,9 @@ int enqueue_forward(rewb200_session* s, const FwdOpts& o) {
     } else {
       RB_TRY(gemm_f32_ld_launch(c, (const float*)xl, ldx, (const float*)m->lm.w, vp, m->lm.b, lm_out, vp, lrows, m->lm.K, vp));
     }
-    if (vp != V)
+    if (m->layered && m->stack.logit_softcap > 0.f)
+      RB_TRY(softcap_launch(c, lm_out, vp, lout, V, lrows, V, m->stack.logit_softcap));
+    else if (vp != V)
       RB_CUDA(cudaMemcpy2DAsync(lout, V * sizeof(float), lm_out, vp * sizeof(float), V * sizeof(float), lrows, cudaMemcpyDeviceToDevice,
                                 c->stream));
   }
@@ -1640,7 +1643,7 @@ void rewb200_session_free(rewb200_session* s) {
                   s->attn, s->h, s->part, s->gu32, s->logits, s->attn_scratch, s->argmax_scratch, s->gather_scratch,
                   s->samp_hist, s->samp_hist_len, s->samp_steps, s->samp_keys, s->samp_work, s->samp_logprob, s->moe_logits, s->moe_topw, s->moe_topi, s->moe_ints,
                   s->moe_send, s->moe_recv, s->moe_xs, s->moe_hs, s->moe_ys, s->moe_ret, s->moe_back, s->moe_tmp, s->route_rec,
-                  s->xn2, s->cq, s->gate, s->part2, s->qeff, s->olat, s->ml, s->gqa_part, s->gqa_ml, s->gla_work, s->kvx, s->latx, s->layer_rec, s->xg, s->logits_pad, s->plan_dev, s->feed_dev};
+                  s->xn2, s->cq, s->gate, s->part2, s->part3, s->shared_gate, s->qeff, s->olat, s->ml, s->gqa_part, s->gqa_ml, s->gla_work, s->kvx, s->latx, s->layer_rec, s->xg, s->logits_pad, s->plan_dev, s->feed_dev};
   for (void* p : ptrs)
     if (p) cudaFree(p);
   if (s->h_ids) cudaFreeHost(s->h_ids);

@@ -24,7 +24,7 @@ int comm_alltoallv_rows(Ctx* c, int slot, const void* send, void* recv, size_t p
                         const int* send_rows, const int* recv_rows);
 int moe_route_launch(Ctx* c, const float* logits, int64_t N, int E, int k, float* topw, int* topi);
 int moe_route_slabs_launch(Ctx* c, const float* logits, int nsplit, int64_t split_stride, const float* bias, int64_t N, int E,
-                           int64_t ld, int k, int renorm, float* topw, int* topi, int* zero, int n_zero);
+                           int64_t ld, int k, int renorm, float scale, float* shared_gate, float* topw, int* topi, int* zero, int n_zero);
 int moe_group_local_launch(Ctx* c, const void* x, int dtype, const int* topi, int64_t tokens, int k, int64_t d, int n_experts,
                            int* offsets, void* xs, int* pair_pos);
 int moe_reset_launch(Ctx* c, int* cursor, int n_cursor, int* count, int n_count, int* meta, int n_meta);
@@ -72,6 +72,8 @@ struct MoeDev {
   int E = 0;                   // routed experts of the layer, all ranks
   int top_k = 0;
   int renorm = 1;              // routing weights divided by their sum
+  float scale = 1.f;           // ... times this
+  bool shared_gate = false;    // column E of the router projects the gate of the shared expert
   bool gated = true;           // SwiGLU experts; false: W_down relu(W_up x)^2
   int64_t f = 0;
   std::vector<float> shared_down_bias;  // sum of the shared experts' down biases (uploaded at finalize)
@@ -80,18 +82,18 @@ struct MoeDev {
 // Latent attention of one layer (latent.cuh).
 struct LatentDev {
   LatentDims m = {};
-  LinW in;                     // [d, q_rank | kv_rank | rot_dim | heads]: query latent, key/value latent, shared key part, gate
+  LinW in;                     // [d, q_rank | kv_rank | rot_dim | heads]: query latent, key/value latent, shared key part (own_kv), gate
   LinW uq;                     // [q_rank, heads * (dim + rot_dim)]
   LinW ukv;                    // [kv_rank, heads * dim | heads * vdim]
-  float *q_norm = nullptr, *kv_norm = nullptr;
+  float *q_norm = nullptr, *kv_norm = nullptr, *sink = nullptr;
   int64_t ldc = 0;             // elements of a cache row: kv_rank + rot_dim, padded
 };
 
 // Grouped-query attention of one layer of a layered model (gqa.cuh).
 struct GqaDev {
   GqaDims m = {};
-  LinW in;                     // [d, heads * dim | kv_heads * dim | kv_heads * vdim | heads]: queries, keys, values, gate
-  float *q_norm = nullptr, *k_norm = nullptr, *bias = nullptr, *sink = nullptr;
+  LinW in;                     // [d, heads * dim | kv_heads * dim | kv_heads * vdim | heads]: queries, keys, values (unless v_from_k), gate
+  float *q_norm = nullptr, *k_norm = nullptr, *bias = nullptr, *sink = nullptr, *conv = nullptr;
   int64_t ldk = 0, ldv = 0;    // elements of a cached key / value row, padded
 };
 
@@ -120,7 +122,7 @@ struct LayerRun {
   int layer = 0;
   bool add_embed = false;      // the embedding output is added to the residual ahead of this run
   int step = -1;               // row of the model's step vectors added ahead of this run
-  int cache = -1;              // run whose cache this one reads (its own unless the layer shares another's keys and values)
+  int cache = -1;              // run whose cache this one reads (its own unless the layer shares another's latents or keys and values)
 };
 
 }  // namespace rewb
@@ -162,7 +164,7 @@ struct rewb200_session {
   int B = 0, max_len = 0, max_pages = 0;
   std::vector<void*> kc, vc;           // per layer
   std::vector<CUtensorMap> tmK, tmV;   // per layer (bf16)
-  std::vector<float*> state;           // layered models: recurrent state per layer run [B][heads][dim][ldv] f32, or nullptr
+  std::vector<float*> state;           // layered models: recurrent or convolution state per layer run [B][..] f32, or nullptr
   int* block_table = nullptr;
   int *d_pos = nullptr, *d_ids = nullptr, *d_next = nullptr, *d_out = nullptr, *d_step = nullptr;
   int out_capacity = 0;
@@ -198,6 +200,8 @@ struct rewb200_session {
   void* cq = nullptr;                  // normed query latents
   float* gate = nullptr;               // output gates [rows][heads]
   float* part2 = nullptr;              // slabs and scratch of the feed-forward branch
+  float* part3 = nullptr;              // ... of a shared expert beside routed ones in a parallel block
+  float* shared_gate = nullptr;        // its gate [rows]
   void* qeff = nullptr;                // absorbed queries, latent outputs and their row statistics (absorbed rows of a step)
   float* olat = nullptr;
   float2* ml = nullptr;
@@ -215,7 +219,7 @@ struct rewb200_session {
   int* plan_dev = nullptr;             // row maps, tile lists and gather lists of a step that is no captured decode
   size_t plan_cap = 0;
   std::vector<int> plan_host;
-  int plan_abs_tiles = 0, plan_chunks = 0, plan_exp_tiles = 0, plan_keys = 0;
+  int plan_abs_tiles = 0, plan_chunks = 0, plan_exp_tiles = 0, plan_keys = 0, plan_tails = 0;
   int plan_gqa_small = 0, plan_gqa_large = 0, plan_gla_small = 0, plan_gla_large = 0, plan_gla_chunks = 0;
   uint8_t* gla_work = nullptr;         // blocks of the chunks of gated linear attention
   size_t gla_work_bytes = 0;

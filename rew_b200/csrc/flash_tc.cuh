@@ -13,13 +13,14 @@
 // are masked.
 //
 // P has
-//   kBias                      the scores get an f32 bias by distance, the softmax denominator a number per head
+//   kBias                      the scores get an f32 bias by distance
+//   sink(head)                 score of the softmax denominator's term without a value, -inf for none
 //   tile(i, skip)              tile i without its first `skip` queries: row0, n (may be <= 0), pos0 and what P itself needs
 //   k_base(tile)               position of the first key the tile's key tiles count from
 //   window()                   keys a query sees, itself included; 0: all
 //   q_chunk(tile, qi, head, box, col)   eight score features of a query (16 bytes), zero where there are none
 //   load_k / load_v(dst, tm_a, tm_b, bar, tile, head, j, k_base, cf)   issue the TMA loads of key tile j
-//   bias_table(head, table), n_bias(), sink(head)      (kBias) fill the table of biases by distance (see bias_slots)
+//   bias_table(head, table), n_bias()      (kBias) fill the table of biases by distance (see bias_slots)
 //   and the fields heads, vdim, scale, gate, out, ldo, status.
 #pragma once
 #include <math.h>
@@ -66,12 +67,10 @@ __device__ __forceinline__ void softmax_rows(const P& a, const Cfg& cf, const fl
   const int lo = W > 0 ? hi - W : -1;                                // the key before the first visible one
   const int last = first + min(n, 128) - 1;
   const float sl2 = a.scale * LOG2E;
-  float m = -INFINITY, l = 0.f, far = 0.f;
-  if constexpr (P::kBias) {
-    far = tab[BIAS_PAD + a.n_bias() - 1];
-    m = a.sink(head) * LOG2E;          // the sink: one more term of the denominator, -inf without one
-    l = half == 0 && m != -INFINITY ? 1.f : 0.f;
-  }
+  float m, l, far = 0.f;
+  if constexpr (P::kBias) far = tab[BIAS_PAD + a.n_bias() - 1];
+  m = a.sink(head) * LOG2E;            // the sink: one more term of the denominator, -inf without one
+  l = half == 0 && m != -INFINITY ? 1.f : 0.f;
   bool ok = true;
   for (int j = j_lo; j < j_hi; ++j) {
     const int it = j - j_lo;

@@ -29,13 +29,20 @@ __device__ __forceinline__ float ex2(float x) {
 }
 __device__ __forceinline__ float sigmoid(float z) { return 1.0f / (1.0f + expf(-z)); }
 
+__device__ __forceinline__ void fma4(float4& y, float4 w, float4 x) {
+  y.x = fmaf(w.x, x.x, y.x);
+  y.y = fmaf(w.y, x.y, y.y);
+  y.z = fmaf(w.z, x.z, y.z);
+  y.w = fmaf(w.w, x.w, y.w);
+}
 // Four neighbouring columns of a row that need not be aligned, summed over the slabs; columns past `n` read as zero.
-__device__ __forceinline__ float4 slab4(const GqaPostArgs& a, const float* p, int i, int n) {
+__device__ __forceinline__ float4 slab4(const float* p, int nsplit, int64_t split_stride, int i, int n) {
   float e[4] = {0.f, 0.f, 0.f, 0.f};
   for (int u = 0; u < 4 && i + u < n; ++u)
-    for (int s = 0; s < a.nsplit; ++s) e[u] += p[s * a.split_stride + i + u];
+    for (int s = 0; s < nsplit; ++s) e[u] += p[s * split_stride + i + u];
   return make_float4(e[0], e[1], e[2], e[3]);
 }
+__device__ __forceinline__ float4 slab4(const GqaPostArgs& a, const float* p, int i, int n) { return slab4(p, a.nsplit, a.split_stride, i, n); }
 template <typename T>
 __device__ __forceinline__ void put4(T* d, int i, int n, float4 v) {
   if (i >= n) return;
@@ -49,15 +56,27 @@ __device__ __forceinline__ void put4(T* d, int i, int n, float4 v) {
   for (int u = 0; u < 4 && i + u < n; ++u) d[i + u] = stf<T>(e[u]);
 }
 
-// One warp per head: query heads, key heads, value heads, then one warp for all gates; RW rows each, requested together.
-// A lane holds four columns at a time, PC of them (dim and vdim up to 128 PC).
-template <typename T, int PC, int RW>
+// Rows of the same portion ahead of `row` in this step, at most taps - 1.
+__device__ __forceinline__ int rows_ahead(const GqaPostArgs& a, int64_t row, int pos) {
+  int n = 0;
+  if (a.map.row_lane)
+    while (n + 1 < a.m.taps && row - n - 1 >= 0 && a.map.row_lane[row - n - 1] == a.map.row_lane[row] && a.map.row_pos[row - n - 1] == pos - n - 1) ++n;
+  return n;
+}
+
+constexpr int CONV_REG_TAPS = 4;   // convolutions up to this long run on registers
+
+// One warp per head: query heads, key heads, value heads (none where the values are the keys: a key warp writes both), then
+// one warp for all gates; RW rows each, requested together.  A lane holds four columns at a time, PC of them (dim and vdim up
+// to 128 PC).  TIME: the head has a convolution, rotated features or values that are its keys.
+template <typename T, int PC, int RW, bool TIME>
 __global__ void __launch_bounds__(256) gqa_post_kernel(GqaPostArgs a, int64_t rows) {
+  __shared__ __align__(16) float s_rot[TIME ? 8 : 1][TIME ? PC * 128 : 4];
   pdl_launch_dependents();
   const int64_t row0 = (int64_t)blockIdx.x * RW;
   const int nr = (int)min((int64_t)RW, rows - row0);
   const int unit = blockIdx.y * 8 + (threadIdx.x >> 5), ln = threadIdx.x & 31;
-  const int H = a.m.heads, G = a.m.own_kv ? a.m.kv_heads : 0, K = a.m.dim, V = a.m.vdim;
+  const int H = a.m.heads, G = a.m.own_kv ? a.m.kv_heads : 0, K = a.m.dim, V = a.m.vdim, GV = TIME && a.m.v_from_k ? 0 : G;
   // norm weights depend on no earlier kernel
   if (RW == 1 && a.m.q_norm) prefetch_floats(a.m.q_norm, K);
   if (RW == 1 && a.m.k_norm) prefetch_floats(a.m.k_norm, K);
@@ -75,11 +94,40 @@ __global__ void __launch_bounds__(256) gqa_post_kernel(GqaPostArgs a, int64_t ro
   };
   if (!a.early) pdl_wait();
   lookup();                // in a captured decode step while the projection still runs
+  const bool is_q = unit < H, is_v = unit >= H + G;
+  const int n = is_v ? V : K;
+  const int64_t col = is_v ? (int64_t)(H + G) * K + (int64_t)(unit - H - G) * V : (int64_t)unit * K;
+  const bool vec = col % 4 == 0 && n % 4 == 0 && a.ld % 4 == 0;
+  // convolution of queries and keys: its weights, and (single tokens) the values that the state holds
+  const int64_t C = TIME ? gqa_channels(a.m) : 0;
+  const bool conv = TIME && a.m.taps > 0 && !is_v, conv_reg = conv && vec && a.m.taps <= CONV_REG_TAPS;
+  float4 cw[TIME ? CONV_REG_TAPS : 1][PC], past[TIME ? CONV_REG_TAPS : 1][PC];   // by tokens ago; past[0] is not used
+  // the projected value of `back` tokens ahead of a row, from the state
+  auto state_at = [&](int r, int back) -> float* {
+    return a.state + ((int64_t)row_lane(a.map, row0 + r) * (a.m.taps - 1) + (pos[r] - back) % (a.m.taps - 1)) * C + col;
+  };
+  auto state4 = [&](int r, int back, int i) {
+    return back < a.m.taps && pos[r] - back >= 0 && r < nr && i < n ? *reinterpret_cast<const float4*>(state_at(r, back) + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+  };
+  if constexpr (TIME) {
+    if (conv_reg) {
+#pragma unroll
+      for (int b = 0; b < CONV_REG_TAPS; ++b)
+#pragma unroll
+        for (int c = 0; c < PC; ++c) {
+          const int i = (c * 32 + ln) * 4;
+          cw[b][c] = b < a.m.taps && i < n ? *reinterpret_cast<const float4*>(a.m.conv + (a.m.taps - 1 - b) * C + col + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+          if (RW == 1 && b > 0 && !a.map.row_lane) past[b][c] = state4(0, b, i);
+        }
+    }
+    if (RW == 1 && a.early && a.m.rope_dims > 0 && ln * 16 < a.m.rope_dims / 2)
+      prefetch_l2(a.m.rope + (int64_t)max(pos[0], 0) * (a.m.rope_dims / 2) * (ok[0] ? 1 : 0) + ln * 16);
+  }
   if (a.early) pdl_wait();
-  if (unit > H + 2 * G || (unit == H + 2 * G && !a.m.gate)) return;
+  if (unit > H + G + GV || (unit == H + G + GV && !a.m.gate)) return;
   const float* p = a.partial + row0 * a.ld;
-  if (unit == H + 2 * G) {
-    p += (int64_t)H * K + (int64_t)G * (K + V);
+  if (unit == H + G + GV) {
+    p += (int64_t)H * K + (int64_t)G * K + (int64_t)GV * V;
     for (int i = ln; i < nr * H; i += 32) {
       const int r = i / H, h = i % H;
       float z = 0.f;
@@ -88,10 +136,6 @@ __global__ void __launch_bounds__(256) gqa_post_kernel(GqaPostArgs a, int64_t ro
     }
     return;
   }
-  const bool is_q = unit < H, is_v = unit >= H + G;
-  const int n = is_v ? V : K;
-  const int64_t col = is_v ? (int64_t)(H + G) * K + (int64_t)(unit - H - G) * V : (int64_t)unit * K;
-  const bool vec = col % 4 == 0 && n % 4 == 0 && a.ld % 4 == 0;
   float4 x[RW][PC];
   if (vec) {
 #pragma unroll
@@ -118,6 +162,66 @@ __global__ void __launch_bounds__(256) gqa_post_kernel(GqaPostArgs a, int64_t ro
     for (int r = 0; r < RW; ++r)
 #pragma unroll
       for (int c = 0; c < PC; ++c) x[r][c] = r < nr ? slab4(a, p + r * a.ld + col, (c * 32 + ln) * 4, n) : make_float4(0.f, 0.f, 0.f, 0.f);
+  }
+  if constexpr (TIME) {
+    if (conv) {
+      int ahead[RW];
+#pragma unroll
+      for (int r = 0; r < RW; ++r) ahead[r] = r < nr ? rows_ahead(a, row0 + r, pos[r]) : 0;
+      if (conv_reg) {
+        if (RW > 1 || a.map.row_lane) {
+          // rows of the step ahead of the first one here
+#pragma unroll
+          for (int b = 1; b < CONV_REG_TAPS; ++b)
+#pragma unroll
+            for (int c = 0; c < PC; ++c) {
+              const int i = (c * 32 + ln) * 4;
+              past[b][c] = make_float4(0.f, 0.f, 0.f, 0.f);
+              if (b > ahead[0] || i >= n) continue;
+              for (int s = 0; s < a.nsplit; ++s) {
+                const float4 w = *reinterpret_cast<const float4*>(p + s * a.split_stride - b * a.ld + col + i);
+                past[b][c].x += w.x; past[b][c].y += w.y; past[b][c].z += w.z; past[b][c].w += w.w;
+              }
+            }
+        }
+#pragma unroll
+        for (int c = 0; c < PC; ++c) {
+          const int i = (c * 32 + ln) * 4;
+#pragma unroll
+          for (int r = RW - 1; r >= 0; --r) {     // backwards: the values ahead of a row are still the projected ones
+            const float4 u = x[r][c];
+            float4 y = make_float4(cw[0][c].x * u.x, cw[0][c].y * u.y, cw[0][c].z * u.z, cw[0][c].w * u.w);
+#pragma unroll
+            for (int b = 1; b < CONV_REG_TAPS; ++b) {
+              const bool given = RW == 1 && !a.map.row_lane;      // requested above
+              float4 h = r >= b ? x[r >= b ? r - b : 0][c] : past[r < b ? b - r : 0][c];
+              if (!given && b > ahead[r]) h = state4(r, b, i);
+              fma4(y, cw[b][c], h);
+            }
+            x[r][c] = y;
+            if (!a.tails && a.m.taps > 1 && r < nr && i < n && ok[r]) *reinterpret_cast<float4*>(state_at(r, 0) + i) = u;
+          }
+        }
+      } else {
+#pragma unroll
+        for (int r = 0; r < RW; ++r) {
+          if (r >= nr) break;
+#pragma unroll
+          for (int c = 0; c < PC; ++c) {
+            const int i = (c * 32 + ln) * 4;
+            float4 u = x[r][c], y = make_float4(0.f, 0.f, 0.f, 0.f);
+            for (int b = 0; b < a.m.taps; ++b) {
+              const float4 w = slab4(a.m.conv + (a.m.taps - 1 - b) * C + col, 1, 0, i, n);
+              if (b == 0) fma4(y, w, u);
+              else if (b <= ahead[r]) fma4(y, w, slab4(a, p + (r - b) * a.ld + col, i, n));
+              else if (pos[r] - b >= 0) fma4(y, w, slab4(state_at(r, b), 1, 0, i, n));
+            }
+            x[r][c] = y;
+            if (!a.tails && a.m.taps > 1 && ok[r]) put4<float>(state_at(r, 0), i, n, u);
+          }
+        }
+      }
+    }
   }
   const float* w = is_v ? nullptr : is_q ? a.m.q_norm : a.m.k_norm;
   float4 g[PC];
@@ -146,9 +250,79 @@ __global__ void __launch_bounds__(256) gqa_post_kernel(GqaPostArgs a, int64_t ro
       const int64_t crow = ((int64_t)page[r] * G + (is_v ? unit - H - G : unit - H)) * PAGE_TOKENS + pos[r] % PAGE_TOKENS;
       dst = is_v ? reinterpret_cast<T*>(a.vc) + crow * a.ldv : reinterpret_cast<T*>(a.kc) + crow * a.ldk;
     }
+    if constexpr (TIME) {
+      if (!is_q && !is_v && a.m.v_from_k) {
+        const int64_t crow = ((int64_t)page[r] * G + unit - H) * PAGE_TOKENS + pos[r] % PAGE_TOKENS;
+#pragma unroll
+        for (int c = 0; c < PC; ++c) put4<T>(reinterpret_cast<T*>(a.vc) + crow * a.ldv, (c * 32 + ln) * 4, n, x[r][c]);
+      }
+      if (!is_v && a.m.rope_dims > 0) {
+        float* s = s_rot[threadIdx.x >> 5];
+        const int half = a.m.rope_dims / 2;
+        const float2* cs = a.m.rope + (int64_t)(ok[r] ? pos[r] : 0) * half;
+#pragma unroll
+        for (int c = 0; c < PC; ++c) {
+          x[r][c] = make_float4(x[r][c].x * f * g[c].x, x[r][c].y * f * g[c].y, x[r][c].z * f * g[c].z, x[r][c].w * f * g[c].w);
+          *reinterpret_cast<float4*>(s + (c * 32 + ln) * 4) = x[r][c];
+        }
+        __syncwarp();
+#pragma unroll
+        for (int c = 0; c < PC; ++c) {
+          const int i = (c * 32 + ln) * 4;
+          float e[4] = {x[r][c].x, x[r][c].y, x[r][c].z, x[r][c].w};
+          if (half % 4 == 0 && i < 2 * half) {      // the four columns lie in one half, the table row starts on 32 bytes
+            const bool lo = i < half;
+            const int j = lo ? i : i - half;
+            const float4 o = *reinterpret_cast<const float4*>(s + (lo ? i + half : j));
+            const float4 t0 = *reinterpret_cast<const float4*>(cs + j), t1 = *reinterpret_cast<const float4*>(cs + j + 2);
+            const float sg = lo ? -1.f : 1.f;
+            e[0] = e[0] * t0.x + sg * (o.x * t0.y);
+            e[1] = e[1] * t0.z + sg * (o.y * t0.w);
+            e[2] = e[2] * t1.x + sg * (o.z * t1.y);
+            e[3] = e[3] * t1.z + sg * (o.w * t1.w);
+          } else if (half % 4 != 0) {
+#pragma unroll
+            for (int u = 0; u < 4; ++u) {
+              if (i + u >= 2 * half) continue;
+              const bool lo = i + u < half;
+              const float2 t = cs[lo ? i + u : i + u - half];
+              e[u] = lo ? e[u] * t.x - s[i + u + half] * t.y : e[u] * t.x + s[i + u - half] * t.y;
+            }
+          }
+          put4<T>(dst, i, n, make_float4(e[0], e[1], e[2], e[3]));
+        }
+        __syncwarp();
+        continue;
+      }
+    }
 #pragma unroll
     for (int c = 0; c < PC; ++c)
       put4<T>(dst, (c * 32 + ln) * 4, n, make_float4(x[r][c].x * f * g[c].x, x[r][c].y * f * g[c].y, x[r][c].z * f * g[c].z, x[r][c].w * f * g[c].w));
+  }
+}
+
+// The last values of every portion into the convolution state.  grid (tails, channels / 512)
+__global__ void __launch_bounds__(128) gqa_conv_state_kernel(GqaPostArgs a) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int2 tail = a.tails[blockIdx.x];
+  const int slots = a.m.taps - 1;
+  if (tail.y >= slots) return;
+  const int64_t C = gqa_channels(a.m), i = ((int64_t)blockIdx.y * 128 + threadIdx.x) * 4;
+  const int pos = row_pos(a.map, tail.x);
+  if (i >= C || pos < 0 || pos >= a.capacity) return;
+  const float* p = a.partial + tail.x * a.ld;
+  float* s = a.state + ((int64_t)row_lane(a.map, tail.x) * slots + pos % slots) * C;
+  if (C % 4 == 0 && a.ld % 4 == 0) {
+    float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 4
+    for (int k = 0; k < a.nsplit; ++k) {
+      const float4 w = *reinterpret_cast<const float4*>(p + k * a.split_stride + i);
+      v.x += w.x; v.y += w.y; v.z += w.z; v.w += w.w;
+    }
+    *reinterpret_cast<float4*>(s + i) = v;
+  } else {
+    put4<float>(s, (int)i, (int)C, slab4(a, p, (int)i, (int)C));
   }
 }
 
@@ -537,13 +711,25 @@ GqaCfg config(const GqaDims& m, int max_tile_rows) {
 
 int gqa_post_launch(Ctx* c, const GqaPostArgs& a, int64_t rows) {
   if (rows == 0) return REWB200_OK;
-  const int units = a.m.heads + (a.m.own_kv ? 2 * a.m.kv_heads : 0) + (a.m.gate ? 1 : 0);
+  const int units = a.m.heads + (a.m.own_kv ? (a.m.v_from_k ? 1 : 2) * a.m.kv_heads : 0) + (a.m.gate ? 1 : 0);
+  const bool time = a.m.taps > 0 || a.m.rope_dims > 0 || a.m.v_from_k;
   RB_REQUIRE(a.m.dim <= 512 && a.m.vdim <= 512, "grouped-query attention: head sizes above 512");
   const bool small = a.m.dim <= 128 && a.m.vdim <= 128, bf = a.dtype == REWB200_BF16, many = small && bf && rows >= 512;
   const dim3 grid((unsigned)(many ? (rows + 3) / 4 : rows), (unsigned)((units + 7) / 8));
   auto go = [&](auto kernel) { return launch_k(kernel, grid, dim3(256), 0, c->stream, c->use_pdl, a, rows); };
-  RB_CUDA(many ? go(gqa_post_kernel<bf16, 1, 4>) : bf ? (small ? go(gqa_post_kernel<bf16, 1, 1>) : go(gqa_post_kernel<bf16, 4, 1>))
-          : small ? go(gqa_post_kernel<float, 1, 1>) : go(gqa_post_kernel<float, 4, 1>));
+#define RB_POST(TIME)                                                                                                                \
+  (many ? go(gqa_post_kernel<bf16, 1, 4, TIME>) : bf ? (small ? go(gqa_post_kernel<bf16, 1, 1, TIME>) : go(gqa_post_kernel<bf16, 4, 1, TIME>)) \
+   : small ? go(gqa_post_kernel<float, 1, 1, TIME>) : go(gqa_post_kernel<float, 4, 1, TIME>))
+  RB_CUDA(time ? RB_POST(true) : RB_POST(false));
+#undef RB_POST
+  ++g_launch_total;
+  return REWB200_OK;
+}
+
+int gqa_conv_state_launch(Ctx* c, const GqaPostArgs& a) {
+  if (a.n_tails == 0 || a.m.taps < 2) return REWB200_OK;
+  const dim3 grid((unsigned)a.n_tails, (unsigned)((gqa_channels(a.m) + 511) / 512));
+  RB_CUDA(launch_k(gqa_conv_state_kernel, grid, dim3(128), 0, c->stream, c->use_pdl, a));
   ++g_launch_total;
   return REWB200_OK;
 }

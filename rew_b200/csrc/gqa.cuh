@@ -1,6 +1,7 @@
-// Grouped-query attention of layered models: per-head RMS norms of queries and keys, a query temperature that grows
-// with the position, a learned bias per head and distance bucket, a learned number per head in the softmax denominator
-// ("sink"), an output gate per head.  Argument structs and launchers of gqa.cu and gqa_prefill.cu.
+// Grouped-query attention of layered models: a short causal convolution over time on queries and keys, per-head RMS norms,
+// a query temperature that grows with the position, rotated features, a learned bias per head and distance bucket, a number
+// per head in the softmax denominator ("sink"), an output gate per head, each of them optional.  Argument structs and
+// launchers of gqa.cu and gqa_prefill.cu.
 //
 // Caches: keys [pages][kv_heads][64][ldk], values [pages][kv_heads][64][ldv].
 #pragma once
@@ -20,10 +21,22 @@ struct GqaDims {
   const float* bias;       // [heads][n_bias] by distance; the last entry holds for every longer distance; nullptr: none
   int n_bias;
   const float* sink;       // [heads] or nullptr
+  int v_from_k;            // the values are the keys as they leave the convolution: no value projection
+  int taps;                // of the convolution per channel of queries and keys; 0: none
+  const float* conv;       // [taps][gqa_channels]: the weight of the value taps - 1 - j tokens ago is row j
+  int rope_dims;           // rotated features at the start of a head, pairs (i, i + rope_dims / 2); 0: none
+  const float2* rope;      // [max_pos][rope_dims / 2] (cos, sin)
 };
 
-// Finishes the fused input projection [q | k | v | gate] (q | gate without keys of its own): sums the split-K slabs,
-// norms queries and keys, applies the temperature, appends keys and values to the cache.
+// Channels of the projection the convolution runs on: queries, then keys of its own.
+inline __host__ __device__ int64_t gqa_channels(const GqaDims& m) { return (int64_t)(m.heads + (m.own_kv ? m.kv_heads : 0)) * m.dim; }
+// f32 elements of convolution state per sequence: the projected values of the last taps - 1 tokens, that of position p in
+// slot p % (taps - 1).  A portion that starts at position 0 reads none of them, so a lane needs no clearing.
+inline int64_t gqa_state_elems(const GqaDims& m) { return m.taps > 1 ? (m.taps - 1) * gqa_channels(m) : 0; }
+
+// Finishes the fused input projection [q | k | v | gate] (q | gate without keys of its own, no v where the values are the
+// keys): sums the split-K slabs, runs the convolution, norms queries and keys, applies the temperature, rotates, appends keys
+// and values to the cache.
 struct GqaPostArgs {
   GqaDims m;
   const float* partial;    // [nsplit][rows][ld]
@@ -40,9 +53,15 @@ struct GqaPostArgs {
   int max_pages, capacity;
   int dtype;
   int early;               // captured decode step: positions predate the step
+  float* state;            // convolution state [lanes][taps - 1][gqa_channels], or nullptr
+  // Rows whose values enter the state: every row of a step of single tokens (tails == nullptr), written on the way, or the
+  // last rows of every portion, (row, rows of the portion behind it), written by gqa_conv_state_launch.
+  const int2* tails;
+  int n_tails;
   int* status;
 };
 int gqa_post_launch(Ctx* c, const GqaPostArgs& a, int64_t rows);
+int gqa_conv_state_launch(Ctx* c, const GqaPostArgs& a);
 
 // Attention of the rows in `tiles` (decoded tokens, small portions).
 struct GqaAttnArgs {

@@ -1,5 +1,5 @@
-// Grouped-query attention of large prompt portions: the tcgen05 kernel of flash_tc.cuh on the cache's pages, with a bias by
-// distance and a sink.  Key tiles further back than the bias table reaches add one number; the others read the table in
+// Grouped-query attention of large prompt portions: the tcgen05 kernel of flash_tc.cuh on the cache's pages, with a sink and,
+// where the layer has one, a bias by distance.  With a bias, key tiles further back than the bias table reaches add one number; the others read the table in
 // shared memory, whose entries for keys after the query are -inf.
 #include <algorithm>
 
@@ -10,8 +10,9 @@ namespace rewb {
 
 namespace {
 
+template <bool BIAS>
 struct GqaPolicy {
-  static constexpr bool kBias = true;
+  static constexpr bool kBias = BIAS;
   GqaPrefillArgs a;
   int nb;                  // distances the bias tells apart
   int heads, vdim;
@@ -35,7 +36,7 @@ struct GqaPolicy {
   __device__ __forceinline__ void bias_table(int head, float* tab, int tid, int nt) const {
     for (int i = tid; i < flash::bias_slots(nb); i += nt) {
       const int d = i - flash::BIAS_PAD;
-      tab[i] = d < 0 ? -INFINITY : a.m.bias ? a.m.bias[(int64_t)head * nb + min(d, nb - 1)] * flash::LOG2E : 0.f;
+      tab[i] = d < 0 ? -INFINITY : a.m.bias[(int64_t)head * nb + min(d, nb - 1)] * flash::LOG2E;
     }
   }
   __device__ __forceinline__ uint4 q_chunk(const GqaTile& t, int qi, int head, int box, int c) const {
@@ -62,7 +63,7 @@ struct GqaPolicy {
   }
 };
 
-size_t table_bytes(const GqaDims& m) { return (size_t)flash::bias_slots(std::max(m.n_bias, 1)) * sizeof(float); }
+size_t table_bytes(const GqaDims& m) { return m.bias ? (size_t)flash::bias_slots(m.n_bias) * sizeof(float) : 0; }
 
 }  // namespace
 
@@ -73,8 +74,12 @@ bool gqa_prefill_ok(const GqaDims& m) {
 int gqa_prefill_launch(Ctx* c, const GqaPrefillArgs& a) {
   if (a.count == 0) return REWB200_OK;
   RB_REQUIRE(gqa_prefill_ok(a.m), "grouped-query attention: head sizes without a tcgen05 kernel");
-  const GqaPolicy p = {a, std::max(a.m.n_bias, 1), a.m.heads, a.m.vdim, a.m.scale, a.m.gate ? a.gate : nullptr, a.out, a.ldo, a.status};
-  return flash::launch(c, p, *a.tm_k, *a.tm_v, a.count, (a.m.dim + 63) / 64, (a.m.vdim + 63) / 64, table_bytes(a.m));
+  auto go = [&](auto p, size_t table) {
+    return flash::launch(c, p, *a.tm_k, *a.tm_v, a.count, (a.m.dim + 63) / 64, (a.m.vdim + 63) / 64, table);
+  };
+  const float* gate = a.m.gate ? a.gate : nullptr;
+  if (a.m.bias) return go(GqaPolicy<true>{a, a.m.n_bias, a.m.heads, a.m.vdim, a.m.scale, gate, a.out, a.ldo, a.status}, table_bytes(a.m));
+  return go(GqaPolicy<false>{a, 1, a.m.heads, a.m.vdim, a.m.scale, gate, a.out, a.ldo, a.status}, 0);
 }
 
 }  // namespace rewb

@@ -46,7 +46,7 @@ __global__ void __launch_bounds__(SMALL ? 768 : 128, SMALL ? 1 : 10) latent_post
   pdl_launch_dependents();
   const int64_t row = blockIdx.x;
   const int nt = blockDim.x;
-  const int nq = a.m.q_rank, nc = a.m.kv_rank, nr = a.m.rot_dim, n = nq + nc + nr + (a.m.gate ? a.m.heads : 0);
+  const int nq = a.m.q_rank, nc = a.m.own_kv ? a.m.kv_rank : 0, nr = a.m.own_kv ? a.m.rot_dim : 0, n = nq + nc + nr + (a.m.gate ? a.m.heads : 0);
   // the norm weights depend on no earlier kernel; in a captured decode step neither do the position and its table row
   if ((int)threadIdx.x * 32 < nq) prefetch_l2(a.q_norm + threadIdx.x * 32);
   if ((int)threadIdx.x * 32 < nc) prefetch_l2(a.kv_norm + threadIdx.x * 32);
@@ -83,7 +83,7 @@ __global__ void __launch_bounds__(SMALL ? 768 : 128, SMALL ? 1 : 10) latent_post
   }
   const int page = a.block_table[(int64_t)lane * a.max_pages + (ok ? pos / PAGE_TOKENS : 0)];
   sq = block_sum2(sq, red);
-  const float rq = 1.0f / sqrtf(sq.x / (float)nq + a.eps), rc = 1.0f / sqrtf(sq.y / (float)nc + a.eps);
+  const float rq = 1.0f / sqrtf(sq.x / (float)nq + a.eps), rc = 1.0f / sqrtf(sq.y / (float)max(nc, 1) + a.eps);
   if (!ok && threadIdx.x == 0) atomicExch(a.status, KS_BAD_INDEX);
   T* cq = reinterpret_cast<T*>(a.cq) + row * a.ldcq;
   T* cr = reinterpret_cast<T*>(a.cache) + ((int64_t)page * PAGE_TOKENS + (ok ? pos % PAGE_TOKENS : 0)) * a.ldc;
@@ -104,7 +104,7 @@ __global__ void __launch_bounds__(SMALL ? 768 : 128, SMALL ? 1 : 10) latent_post
   }
   if (a.m.gate)
     for (int i = threadIdx.x; i < a.m.heads; i += nt) a.gate[row * a.m.heads + i] = 1.0f / (1.0f + expf(-sx[nq + nc + nr + i]));
-  if (!ok) return;
+  if (!ok || !a.m.own_kv) return;
   for (int i = threadIdx.x * 2; i < nc; i += nt * 2) {
     if (i + 1 < nc) put(cr + i, a.kv_norm[i] * (sx[nq + i] * rc), a.kv_norm[i + 1] * (sx[nq + i + 1] * rc));
     else cr[i] = stf<T>(a.kv_norm[i] * (sx[nq + i] * rc));
@@ -180,7 +180,7 @@ __global__ void __launch_bounds__(128) latent_attn_plain_kernel(LatentAttnArgs a
   const int lane = row_lane(a.map, row), pos = min(max(row_pos(a.map, row), 0), a.max_pages * PAGE_TOKENS - 1);
   const int k0 = a.m.window > 0 ? max(0, pos - a.m.window + 1) : 0;
   const int w = threadIdx.x >> 5, ln = threadIdx.x & 31;
-  float mx = -INFINITY, l = 0.f;
+  float mx = a.m.sink ? a.m.sink[h] : -INFINITY, l = a.m.sink ? 1.f : 0.f;
   __syncthreads();
   for (int t = k0 / PAGE_TOKENS; t <= pos / PAGE_TOKENS; ++t) {
     const int page = a.block_table[(int64_t)lane * a.max_pages + t];
@@ -702,13 +702,15 @@ __global__ void __launch_bounds__(256) latent_out_kernel(LatentAttnArgs a) {
     const int row = tid >> 4, s = tid & 15;
     const bool in = row < ch.y && s < ns;
     const float2 ml = in ? a.ml[((int64_t)(ch.x + row) * a.m.heads + h) * ns + s] : make_float2(-INFINITY, 0.f);
-    float M = ml.x;
+    const float sink = a.m.sink ? a.m.sink[h] : -INFINITY;
+    float M = fmaxf(ml.x, sink);
 #pragma unroll
     for (int o = 8; o > 0; o >>= 1) M = fmaxf(M, __shfl_xor_sync(0xffffffffu, M, o));
     const float f = ml.x == -INFINITY ? 0.f : __expf(ml.x - M);
     float L = ml.y * f;
 #pragma unroll
     for (int o = 8; o > 0; o >>= 1) L += __shfl_xor_sync(0xffffffffu, L, o);
+    if (a.m.sink) L += __expf(sink - M);
     sw[row][s] = L > 0.f ? f / L : 0.f;
   }
   __syncthreads();

@@ -20,9 +20,11 @@ struct LatentDims {
   float scale;
   const float2* rope;      // [max_pos][rope_dims / 2] (cos, sin)
   int max_pos;
+  int own_kv;              // 0: another layer's cached latents
+  const float* sink;       // [heads] a score without a key or value in the softmax denominator, or nullptr
 };
 
-// Finishes the fused input projection [q_rank | kv_rank | rot_dim | heads]: sums the split-K slabs, norms the query
+// Finishes the fused input projection [q_rank | kv_rank | rot_dim | heads] (q_rank | heads without latents of its own): sums the split-K slabs, norms the query
 // latent and the key/value latent, rotates the shared key part, appends [c | k_rot] to the cache, applies the
 // sigmoid of the output gate.
 struct LatentPostArgs {

@@ -28,6 +28,7 @@ struct LatentPolicy {
   __device__ __forceinline__ int window() const { return a.m.window; }
   __device__ __forceinline__ int k_base(const ExpTile& t) const { return max(t.key0, a.m.window > 0 ? t.pos0 - a.m.window + 1 : 0); }
   __device__ __forceinline__ int n_bias() const { return 1; }
+  __device__ __forceinline__ float sink(int head) const { return a.m.sink ? a.m.sink[head] : -INFINITY; }
   __device__ __forceinline__ uint4 q_chunk(const ExpTile& t, int qi, int head, int box, int c) const {
     const bf16* qp = a.q + (int64_t)(t.row0 + qi) * a.ldq + (int64_t)head * (a.m.dim + a.m.rot_dim);
     uint4 v = make_uint4(0, 0, 0, 0);
@@ -85,7 +86,7 @@ __global__ void __launch_bounds__(256) latent_gather_kernel(const bf16* cache, c
 // values in at most two.
 bool latent_expanded_ok(const LatentDims& m) {
   const int nb = (m.dim + 63) / 64 + (m.rot_dim + 63) / 64;
-  return m.dim % 8 == 0 && m.rot_dim % 8 == 0 && m.vdim % 8 == 0 && m.kv_rank % 8 == 0 && m.rope_dims % 2 == 0 && m.rot_dim > 0 && nb <= 4 &&
+  return m.dim % 8 == 0 && m.rot_dim % 8 == 0 && m.vdim % 8 == 0 && m.kv_rank % 8 == 0 && m.rope_dims % 2 == 0 && nb <= 4 &&
          m.vdim <= 128 && m.scale > 0.f;
 }
 

@@ -19,10 +19,12 @@ namespace {
 constexpr int MAX_E_PER_LANE = 8;  // E <= 256
 
 // logits: nsplit slabs [N][ld] split_stride apart, summed in slab order, plus bias (may be null).  renorm 0: the
-// weights are the chosen experts' probabilities themselves, not divided by their sum.
+// weights are the chosen experts' probabilities themselves, not divided by their sum.  scale: factor of the weights.
+// shared_gate (may be null) [N]: sigmoid of logit E, the gate of a shared expert.
 __global__ void __launch_bounds__(128) moe_route_kernel(const float* __restrict__ logits, int nsplit, int64_t split_stride,
                                                         const float* __restrict__ bias, int64_t N, int E, int64_t ld, int k, int renorm,
-                                                        float* __restrict__ topw, int* __restrict__ topi, int* zero, int n_zero) {
+                                                        float scale, float* __restrict__ shared_gate, float* __restrict__ topw,
+                                                        int* __restrict__ topi, int* zero, int n_zero) {
   pdl_launch_dependents();
   pdl_wait();
   if (blockIdx.x == 0 && (int)threadIdx.x < n_zero) zero[threadIdx.x] = 0;  // the dispatch kernel's per-peer cursors
@@ -30,6 +32,11 @@ __global__ void __launch_bounds__(128) moe_route_kernel(const float* __restrict_
   const int64_t tok = (int64_t)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
   if (tok >= N) return;
   const float* lr = logits + tok * ld;
+  if (shared_gate && lane == 0) {
+    float z = 0.f;
+    for (int sp = 0; sp < nsplit; ++sp) z += lr[sp * split_stride + E];
+    shared_gate[tok] = 1.0f / (1.0f + expf(-z));
+  }
   float p[MAX_E_PER_LANE];
   float mx = -INFINITY;
 #pragma unroll
@@ -98,9 +105,9 @@ __global__ void __launch_bounds__(128) moe_route_kernel(const float* __restrict_
       }
     }
   }
-  if (!renorm) return;
+  if (!renorm && scale == 1.0f) return;
   __syncwarp();
-  for (int j = lane; j < k; j += 32) topw[tok * k + j] = topw[tok * k + j] / denom;
+  for (int j = lane; j < k; j += 32) topw[tok * k + j] = topw[tok * k + j] / (renorm ? denom : 1.0f) * scale;
 }
 
 
@@ -528,18 +535,18 @@ int moe_combine_peer_launch(Ctx* c, const int* pair_slot, const float* topw, int
 }
 
 int moe_route_slabs_launch(Ctx* c, const float* logits, int nsplit, int64_t split_stride, const float* bias, int64_t N, int E,
-                           int64_t ld, int k, int renorm, float* topw, int* topi, int* zero, int n_zero) {
+                           int64_t ld, int k, int renorm, float scale, float* shared_gate, float* topw, int* topi, int* zero, int n_zero) {
   RB_REQUIRE(E >= 1 && E <= 32 * MAX_E_PER_LANE, "MoE routing supports up to 256 experts");
   RB_REQUIRE(k >= 1 && k <= E, "initDeepSeekMoE: numExpertsPerTok must be in 1..numRouted");
   RB_REQUIRE(n_zero >= 0 && n_zero <= 128, "at most 128 counters can be cleared by the routing kernel");
   if (N == 0) return REWB200_OK;
   RB_CUDA(launch_k(moe_route_kernel, dim3((unsigned)((N + 3) / 4)), dim3(128), 0, c->stream, c->use_pdl, logits, nsplit,
-                   split_stride, bias, N, E, ld, k, renorm, topw, topi, zero, n_zero));
+                   split_stride, bias, N, E, ld, k, renorm, scale, shared_gate, topw, topi, zero, n_zero));
   ++g_launch_total;
   return REWB200_OK;
 }
 int moe_route_launch(Ctx* c, const float* logits, int64_t N, int E, int k, float* topw, int* topi) {
-  return moe_route_slabs_launch(c, logits, 1, 0, nullptr, N, E, E, k, 1, topw, topi, nullptr, 0);
+  return moe_route_slabs_launch(c, logits, 1, 0, nullptr, N, E, E, k, 1, 1.0f, nullptr, topw, topi, nullptr, 0);
 }
 
 // One rank owning every expert: pos[pair] = row of pair (token, j) in the expert-sorted activation matrix

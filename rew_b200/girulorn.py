@@ -67,7 +67,7 @@ def moe_lite(**kw):
     moe = dict(ff="experts", ffn=1408, experts=64, top_k=6, renormalize=True, expert_gated=True, router_bias=True, shared_ffn=2816)
     gla = LayerSpec(mixer="gla", heads=16, dim=128, vdim=128, tau=16.0, decay_rank=16, **moe)
     att = LayerSpec(mixer="attention", heads=16, kv_heads=16, dim=128, vdim=128, scale=128 ** -0.5, bias_rows=32, bias_max=128,
-                    temp_every=1024, temp_coef=0.1, **moe)
+                    temp_every=1024, temp_coef=0.1, sink=True, **moe)
     layers = [att if i % 2 else gla for i in range(27)]
     return LayeredConfig(**{**dict(vocab=102400, d_model=2048, layers=layers, eps=1e-6, norm_zero_centred=False, block="output_norm",
                                    own_head=True, max_seq=2304, dtype=_lib.BF16), **kw})

@@ -11,14 +11,17 @@ from . import _lib
 
 
 MIXERS = {"latent": 1, "attention": 2, "gla": 3}
+BLOCKS = ("parallel", "output_norm", "parallel_one_norm")
+SINKS = {False: 0, True: 1, "one": 2}
 
 
 @dataclass
 class LayerSpec:
     """One layer: a mixer and a feed-forward.
 
-    mixer "latent": latent attention; "attention": grouped-query attention with a learned distance bias, query / key
-    norms, a query temperature and a softmax sink; "gla": gated linear attention with a state per sequence.
+    mixer "latent": latent attention; "attention": grouped-query attention with a short convolution, rotation, a learned
+    distance bias, query / key norms, a query temperature and a softmax sink, each optional; "gla": gated linear attention
+    with a state per sequence.
     """
     heads: int
     dim: int                    # query / key features per head (latent: the unrotated ones)
@@ -26,18 +29,22 @@ class LayerSpec:
     mixer: str = "latent"
     scale: float = 1.0          # of the attention scores
     out_gate: bool = True       # latent, attention: a sigmoid gate per head on the output
+    sink: object = False        # latent, attention: a further term of the softmax denominator, exp of a learned number per
+                                # head (True) or one ("one")
+    kv_from: int = -1           # latent, attention: layer whose cached latents, or keys and values, are used; -1: its own
+    rope_base: float = 10000.0
+    rope_dims: int = None       # latent: rotated features of the rot_dim part, interleaved pairs (None: all); attention:
+                                # rotated features of every head, pairs (i, i + rope_dims / 2) (None: none)
     # latent
     rot_dim: int = 0            # rotated features per head; the key part is shared by all heads
     q_rank: int = 0
     kv_rank: int = 0
     window: int = 0             # keys a query sees, itself included; 0: all
-    rope_base: float = 10000.0
-    rope_dims: int = None       # rotated features of the rot_dim part (None: all)
     # attention
     kv_heads: int = 0
-    kv_from: int = -1           # layer whose keys and values are used; -1: its own
+    conv_taps: int = 0          # causal convolution over time per channel of queries and keys; 0: none
+    values_from_keys: bool = False   # the values are the keys as they leave the convolution; there is no value projection
     qk_norm: bool = True
-    sink: bool = True           # a learned number per head in the softmax denominator
     bias_rows: int = 0          # rows of the distance bias table; 0: no bias
     bias_max: int = 0           # distance at which the buckets end
     temp_every: int = 0         # query temperature 1 + temp_coef ln(floor((p + 1) / temp_every) + 1); 0: none
@@ -51,9 +58,11 @@ class LayerSpec:
     experts: int = 0
     top_k: int = 0
     renormalize: bool = False   # routing weights divided by the sum of the chosen ones
+    router_scale: float = 1.0   # ... times this
     expert_gated: bool = False  # gated SiLU experts; False: W_down relu(W_up x)^2
     router_bias: bool = False
     shared_ffn: int = 0         # hidden width of the shared expert; 0: none
+    shared_gate: bool = False   # its output is scaled by a sigmoid of a projection of the input
 
     def to_c(self):
         kinds = ("none", "dense", "experts")
@@ -63,31 +72,36 @@ class LayerSpec:
             raise ValueError("unknown mixer %r" % (self.mixer,))
         return _lib.Layer(mixer=MIXERS[self.mixer], heads=self.heads, dim=self.dim, rot_dim=self.rot_dim, vdim=self.vdim, q_rank=self.q_rank,
                           kv_rank=self.kv_rank, window=self.window,
-                          rope_dims=self.rot_dim if self.rope_dims is None else self.rope_dims,
+                          rope_dims=self.rope_dims if self.rope_dims is not None else self.rot_dim,
                           out_gate=int(self.out_gate and self.mixer != "gla"), ff=kinds.index(self.ff), ffn=self.ffn,
                           experts=self.experts, top_k=self.top_k, renormalize=int(self.renormalize),
                           expert_gated=int(self.expert_gated), rope_base=self.rope_base, scale=self.scale, kv_heads=self.kv_heads,
-                          kv_from=self.kv_from, qk_norm=int(self.qk_norm), sink=int(self.sink), bias_rows=self.bias_rows,
+                          kv_from=self.kv_from, qk_norm=int(self.qk_norm), sink=SINKS[self.sink], bias_rows=self.bias_rows,
                           bias_max=self.bias_max, temp_every=self.temp_every, temp_coef=self.temp_coef, decay_rank=self.decay_rank,
-                          tau=self.tau, router_bias=int(self.router_bias), shared_ffn=self.shared_ffn)
+                          tau=self.tau, router_bias=int(self.router_bias), shared_ffn=self.shared_ffn, conv_taps=self.conv_taps,
+                          values_from_keys=int(self.values_from_keys), router_scale=self.router_scale, shared_gate=int(self.shared_gate))
 
     def mixer_specs(self, d):
         """[(name, shape)] of the mixer's tensors, Linear weights [in, out]."""
-        H, K, V = self.heads, self.dim, self.vdim
+        H, K, V, own = self.heads, self.dim, self.vdim, self.kv_from < 0
         if self.mixer == "latent":
-            specs = [("dq", (d, self.q_rank)), ("dq.norm", (self.q_rank,)), ("uq", (self.q_rank, H * (K + self.rot_dim))),
-                     ("dkv", (d, self.kv_rank + self.rot_dim)), ("dkv.norm", (self.kv_rank,)), ("uk", (self.kv_rank, H * K)),
-                     ("uv", (self.kv_rank, H * V))]
+            specs = [("dq", (d, self.q_rank)), ("dq.norm", (self.q_rank,)), ("uq", (self.q_rank, H * (K + self.rot_dim)))]
+            if own:
+                specs += [("dkv", (d, self.kv_rank + self.rot_dim)), ("dkv.norm", (self.kv_rank,))]
+            specs += [("uk", (self.kv_rank, H * K)), ("uv", (self.kv_rank, H * V))]
+            if self.sink is True:
+                specs.append(("sink", (H,)))
         elif self.mixer == "attention":
-            own = self.kv_from < 0
             specs = [("q", (d, H * K))]
             if own:
-                specs += [("k", (d, self.kv_heads * K)), ("v", (d, self.kv_heads * V))]
+                specs += [("k", (d, self.kv_heads * K))] + ([] if self.values_from_keys else [("v", (d, self.kv_heads * V))])
+            if self.conv_taps:
+                specs += [("q.conv", (H * K, self.conv_taps))] + ([("k.conv", (self.kv_heads * K, self.conv_taps))] if own else [])
             if self.qk_norm:
                 specs += [("q.norm", (K,))] + ([("k.norm", (K,))] if own else [])
             if self.bias_rows:
                 specs.append(("rel", (self.bias_rows, H)))
-            if self.sink:
+            if self.sink is True:
                 specs.append(("sink", (H,)))
         else:
             specs = [("q", (d, H * K)), ("k", (d, H * K)), ("v", (d, H * V)), ("a1", (d, self.decay_rank)),
@@ -110,6 +124,8 @@ class LayerSpec:
     @property
     def state_elements(self):
         """f32 elements of recurrent state per sequence."""
+        if self.mixer == "attention" and self.conv_taps:
+            return (self.conv_taps - 1) * (self.heads + (self.kv_heads if self.kv_from < 0 else 0)) * self.dim
         return self.heads * self.dim * self.vdim if self.mixer == "gla" else 0
 
 
@@ -121,8 +137,10 @@ class LayeredConfig:
     eps: float = 1e-6
     loop: tuple = None          # (start, stop, times): layers[start:stop] are repeated, `times` passes in all
     norm_zero_centred: bool = True   # block and final norm weights are stored as the distance from one
-    block: str = "parallel"     # "parallel": x += mixer(norm1 x) + ff(norm2 x); "output_norm": x += norm1(mixer x), x += norm2(ff x)
+    block: str = "parallel"     # "parallel": x += mixer(norm1 x) + ff(norm2 x); "output_norm": x += norm1(mixer x), x += norm2(ff x);
+                                # "parallel_one_norm": x += mixer(h) + ff(h), h = norm1 x
     own_head: bool = False      # the output head is a tensor of its own; False: the embedding table
+    logit_softcap: float = 0.0  # logits <- cap * tanh(logits / cap); 0: none
     max_seq: int = 4096
     dtype: int = _lib.F32
     tp_size: int = field(default=1, init=False)
@@ -168,7 +186,7 @@ class LayeredConfig:
         arr = (_lib.Layer * self.n_layers)(*[l.to_c() for l in self.layers])
         a, b, k = self.loop or (0, 0, 0)
         stack = _lib.Stack(loop_start=a, loop_stop=b, loop_times=k, norm_zero_centred=int(self.norm_zero_centred),
-                           block=("parallel", "output_norm").index(self.block), own_head=int(self.own_head))
+                           block=BLOCKS.index(self.block), own_head=int(self.own_head), logit_softcap=self.logit_softcap)
         _lib.check(_lib.lib().rewb200_model_create_layers(slot, C.byref(base), arr, C.byref(stack), out))
 
     def tensor_specs(self):
@@ -183,7 +201,8 @@ class LayeredConfig:
             specs += [(p + "mix." + n, shape) for n, shape in l.mixer_specs(d)]
             if l.ff == "none":
                 continue
-            specs.append((p + "norm2", (d,)))
+            if self.block != "parallel_one_norm":
+                specs.append((p + "norm2", (d,)))
             if l.ff == "dense":
                 specs += [(p + "mlp.gate", (d, l.ffn)), (p + "mlp.up", (d, l.ffn)), (p + "mlp.down", (l.ffn, d))]
             else:
@@ -198,12 +217,14 @@ class LayeredConfig:
                 if l.shared_ffn:
                     q = p + "mlp.shared."
                     specs += [(q + "gate", (d, l.shared_ffn)), (q + "up", (d, l.shared_ffn)), (q + "down", (l.shared_ffn, d))]
+                    if l.shared_gate:
+                        specs.append((q + "sg", (d, 1)))
         specs.append(("final.norm", (d,)))
         if self.own_head:
             specs.append(("head", (d, self.vocab)))
         return specs
 
-    def canonical_tensors(self, tensors, tables=("embed", "loop.step", "mix.rel")):
+    def canonical_tensors(self, tensors, tables=("embed", "loop.step", "mix.rel", ".conv")):
         """The canonical list from {name: array} of a file whose Linear weights are [out, in]; names that end in one of
         `tables` are matrices that are no Linear and stay as they are."""
         out = []

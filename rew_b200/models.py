@@ -28,6 +28,15 @@ def _load_girulorn(path, dtype, max_seq, slot):
     return girulorn.load(path, dtype, max_seq, slot)
 
 
+def _is_kugirax(cfg):
+    return cfg.get("architecture") == "Kugirax"
+
+
+def _load_kugirax(path, dtype, max_seq, slot):
+    from . import kugirax
+    return kugirax.load(path, dtype, max_seq, slot)
+
+
 def _is_hf_llama(cfg):
     return cfg.get("model_type") == "llama" or "LlamaForCausalLM" in (cfg.get("architectures") or [])
 
@@ -42,6 +51,7 @@ def _load_hf_llama(path, dtype, max_seq, slot):
 FAMILIES = [
     ("rezupel", _is_rezupel, _load_rezupel),
     ("girulorn", _is_girulorn, _load_girulorn),
+    ("kugirax", _is_kugirax, _load_kugirax),
     ("llama", _is_hf_llama, _load_hf_llama),
 ]
 
