@@ -24,6 +24,9 @@ data-path collective): weak scaling.
     girulorn_b64, girulorn_b1, girulorn_b8_s2048
              Girulorn (gated linear attention and attention with distance bias in turn, routed and
              shared experts) at the sizes of moe_b64, moe_b1 and moe_b8_s2048
+    kugirax_b32, kugirax_b1, kugirax_b8_s2048, kugirax_moe_b64
+             Kugirax (attention with a short convolution and latent attention with sinks in turn, one-norm
+             blocks) at the sizes of l8_b32, l8_b1, l8_b8_s2048 and moe_b64
 
 `value` is decode tokens/s of the whole job with ids, weights and cache resident
 in HBM (CUDA events around K graph replays); `e2e` is tokens/s of one generate()
@@ -77,6 +80,10 @@ WORKLOADS = {
     "girulorn_b64": dict(model="girulorn.moe_lite", batch=64, prompt=256),
     "girulorn_b1": dict(model="girulorn.moe_lite", batch=1, prompt=512),
     "girulorn_b8_s2048": dict(model="girulorn.moe_lite", batch=8, prompt=2048),
+    "kugirax_b32": dict(model="kugirax.dense_8b", batch=32, prompt=512),
+    "kugirax_b1": dict(model="kugirax.dense_8b", batch=1, prompt=512),
+    "kugirax_b8_s2048": dict(model="kugirax.dense_8b", batch=8, prompt=2048),
+    "kugirax_moe_b64": dict(model="kugirax.moe_lite", batch=64, prompt=256),
     "moe_b1": dict(model="deepseek_v2_lite", batch=1, prompt=512),
     "moe_b8_s2048": dict(model="deepseek_v2_lite", batch=8, prompt=2048),
     # the attention operator alone: batch 8, 32 query / 8 kv heads, head_dim 128, 4096 positions

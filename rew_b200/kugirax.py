@@ -58,3 +58,37 @@ def load(model_dir, dtype, max_seq=None, slot=0):
     kw = {} if max_seq is None else dict(max_seq=int(max_seq))
     cfg = config_from_json(os.path.join(model_dir, "config.json"), dtype=dtype, **kw)
     return CausalLM(cfg, slot).load(cfg.canonical_tensors(st.read_safetensors_dir(model_dir)))
+
+
+# Benchmark configurations (shapes only; weights are synthetic).
+def _turns(n, attention, latent, first_ff, ff):
+    """n layers, attention and latent attention in turn; every other latent layer reads the latents of the one before it."""
+    layers, own = [], -1
+    for i in range(n):
+        f = first_ff if i == 0 else ff
+        if i % 2 == 0:
+            layers.append(LayerSpec(mixer="attention", conv_taps=4, values_from_keys=True, qk_norm=False, sink="one", out_gate=False, **attention, **f))
+        else:
+            src, own = (own, -1) if own >= 0 else (-1, i)
+            layers.append(LayerSpec(mixer="latent", sink=True, out_gate=False, kv_from=src, **latent, **f))
+    return layers
+
+
+def dense_8b(**kw):
+    """Layers of the width, heads and feed-forward of the 8B Llama shape."""
+    from . import _lib
+    ff = dict(ff="dense", ffn=14336)
+    layers = _turns(32, dict(heads=32, kv_heads=8, dim=128, vdim=128, scale=128 ** -0.5, rope_base=500000.0, rope_dims=128),
+                    dict(heads=32, dim=128, vdim=128, q_rank=1536, kv_rank=512, scale=128 ** -0.5, window=1024), ff, ff)
+    return LayeredConfig(**{**dict(vocab=128256, d_model=4096, layers=layers, eps=1e-5, norm_zero_centred=False, block="parallel_one_norm",
+                                   own_head=True, logit_softcap=30.0, max_seq=2560, dtype=_lib.BF16), **kw})
+
+
+def moe_lite(**kw):
+    """As many layers, the width, heads, experts, expert and shared expert widths of the DeepSeek-V2-Lite shape."""
+    from . import _lib
+    moe = dict(ff="experts", ffn=1408, experts=64, top_k=6, renormalize=True, router_scale=2.5, expert_gated=True, shared_ffn=2816, shared_gate=True)
+    layers = _turns(27, dict(heads=16, kv_heads=16, dim=128, vdim=128, scale=128 ** -0.5, rope_base=10000.0, rope_dims=128),
+                    dict(heads=16, dim=128, vdim=128, q_rank=768, kv_rank=512, scale=128 ** -0.5, window=1024), dict(ff="dense", ffn=10944), moe)
+    return LayeredConfig(**{**dict(vocab=102400, d_model=2048, layers=layers, eps=1e-6, norm_zero_centred=False, block="parallel_one_norm",
+                                   own_head=True, logit_softcap=30.0, max_seq=1024, dtype=_lib.BF16), **kw})
