@@ -29,6 +29,7 @@ __device__ __forceinline__ float ex2(float x) {
 }
 __device__ __forceinline__ float sigmoid(float z) { return 1.0f / (1.0f + expf(-z)); }
 
+__device__ __forceinline__ void add4(float4& v, float4 w) { v.x += w.x; v.y += w.y; v.z += w.z; v.w += w.w; }
 __device__ __forceinline__ void fma4(float4& y, float4 w, float4 x) {
   y.x = fmaf(w.x, x.x, y.x);
   y.y = fmaf(w.y, x.y, y.y);
@@ -64,6 +65,7 @@ __device__ __forceinline__ int rows_ahead(const GqaPostArgs& a, int64_t row, int
   return n;
 }
 
+constexpr int POST_ROWS = 8;       // rows a warp of gqa_post_kernel takes in large steps
 constexpr int CONV_REG_TAPS = 4;   // convolutions up to this long run on registers
 
 // One warp per head: query heads, key heads, value heads (none where the values are the keys: a key warp writes both), then
@@ -71,60 +73,83 @@ constexpr int CONV_REG_TAPS = 4;   // convolutions up to this long run on regist
 // to 128 PC).  TIME: the head has a convolution, rotated features or values that are its keys.
 template <typename T, int PC, int RW, bool TIME>
 __global__ void __launch_bounds__(256) gqa_post_kernel(GqaPostArgs a, int64_t rows) {
+  constexpr int HIST = TIME ? CONV_REG_TAPS - 1 : 0, BACK = TIME ? CONV_REG_TAPS : 1;
+  constexpr unsigned ALL = 0xffffffffu;
   __shared__ __align__(16) float s_rot[TIME ? 8 : 1][TIME ? PC * 128 : 4];
   pdl_launch_dependents();
   const int64_t row0 = (int64_t)blockIdx.x * RW;
   const int nr = (int)min((int64_t)RW, rows - row0);
   const int unit = blockIdx.y * 8 + (threadIdx.x >> 5), ln = threadIdx.x & 31;
   const int H = a.m.heads, G = a.m.own_kv ? a.m.kv_heads : 0, K = a.m.dim, V = a.m.vdim, GV = TIME && a.m.v_from_k ? 0 : G;
-  // norm weights depend on no earlier kernel
-  if (RW == 1 && a.m.q_norm) prefetch_floats(a.m.q_norm, K);
-  if (RW == 1 && a.m.k_norm) prefetch_floats(a.m.k_norm, K);
-  int pos[RW], page[RW];
-  bool ok[RW];
-  auto lookup = [&]() {
-#pragma unroll
-    for (int r = 0; r < RW; ++r) {
-      const int64_t row = row0 + min(r, nr - 1);
-      pos[r] = row_pos(a.map, row);
-      ok[r] = pos[r] >= 0 && pos[r] < a.capacity;
-      page[r] = a.block_table[(int64_t)row_lane(a.map, row) * a.max_pages + (ok[r] ? pos[r] / PAGE_TOKENS : 0)];
-      if (!ok[r] && unit == 0 && ln == 0) atomicExch(a.status, KS_BAD_INDEX);
-    }
-  };
-  if (!a.early) pdl_wait();
-  lookup();                // in a captured decode step while the projection still runs
+  if (unit > H + G + GV || (unit == H + G + GV && !a.m.gate)) return;
   const bool is_q = unit < H, is_v = unit >= H + G;
   const int n = is_v ? V : K;
   const int64_t col = is_v ? (int64_t)(H + G) * K + (int64_t)(unit - H - G) * V : (int64_t)unit * K;
   const bool vec = col % 4 == 0 && n % 4 == 0 && a.ld % 4 == 0;
-  // convolution of queries and keys: its weights, and (single tokens) the values that the state holds
+  // norm and convolution weights depend on no earlier kernel
+  if (RW == 1 && a.m.q_norm) prefetch_floats(a.m.q_norm, K);
+  if (RW == 1 && a.m.k_norm) prefetch_floats(a.m.k_norm, K);
   const int64_t C = TIME ? gqa_channels(a.m) : 0;
   const bool conv = TIME && a.m.taps > 0 && !is_v, conv_reg = conv && vec && a.m.taps <= CONV_REG_TAPS;
-  float4 cw[TIME ? CONV_REG_TAPS : 1][PC], past[TIME ? CONV_REG_TAPS : 1][PC];   // by tokens ago; past[0] is not used
-  // the projected value of `back` tokens ahead of a row, from the state
-  auto state_at = [&](int r, int back) -> float* {
-    return a.state + ((int64_t)row_lane(a.map, row0 + r) * (a.m.taps - 1) + (pos[r] - back) % (a.m.taps - 1)) * C + col;
-  };
-  auto state4 = [&](int r, int back, int i) {
-    return back < a.m.taps && pos[r] - back >= 0 && r < nr && i < n ? *reinterpret_cast<const float4*>(state_at(r, back) + i) : make_float4(0.f, 0.f, 0.f, 0.f);
-  };
+  const int half = TIME && !is_v ? a.m.rope_dims / 2 : 0;
+  float4 cw[BACK][PC], past[BACK][PC];   // weights and values by tokens ago; past[0] is not used
   if constexpr (TIME) {
     if (conv_reg) {
 #pragma unroll
-      for (int b = 0; b < CONV_REG_TAPS; ++b)
+      for (int b = 0; b < BACK; ++b)
 #pragma unroll
         for (int c = 0; c < PC; ++c) {
           const int i = (c * 32 + ln) * 4;
-          cw[b][c] = b < a.m.taps && i < n ? *reinterpret_cast<const float4*>(a.m.conv + (a.m.taps - 1 - b) * C + col + i) : make_float4(0.f, 0.f, 0.f, 0.f);
-          if (RW == 1 && b > 0 && !a.map.row_lane) past[b][c] = state4(0, b, i);
+          past[b][c] = make_float4(0.f, 0.f, 0.f, 0.f);
+          cw[b][c] = b < a.m.taps && i < n ? *reinterpret_cast<const float4*>(a.m.conv + (a.m.taps - 1 - b) * C + col + i) : past[b][c];
         }
     }
-    if (RW == 1 && a.early && a.m.rope_dims > 0 && ln * 16 < a.m.rope_dims / 2)
-      prefetch_l2(a.m.rope + (int64_t)max(pos[0], 0) * (a.m.rope_dims / 2) * (ok[0] ? 1 : 0) + ln * 16);
+  }
+  if (!a.early) pdl_wait();
+  // Lane l looks up row0 - HIST + l, in a captured decode step while the projection still runs.
+  const int64_t my_row = row0 - HIST + ln;
+  int my_lane = -1, my_pos = -1, my_page = 0;
+  if (my_row >= 0 && my_row < row0 + nr && ln < RW + HIST) {
+    my_lane = row_lane(a.map, my_row);
+    my_pos = row_pos(a.map, my_row);
+    const bool in = my_pos >= 0 && my_pos < a.capacity;
+    my_page = a.block_table[(int64_t)my_lane * a.max_pages + (in ? my_pos / PAGE_TOKENS : 0)];
+    if (!in && unit == 0 && ln >= HIST) atomicExch(a.status, KS_BAD_INDEX);
+  }
+  auto pos_of = [&](int r) { return __shfl_sync(ALL, my_pos, min(r, nr - 1) + HIST); };
+  auto ok_at = [&](int pos) { return pos >= 0 && pos < a.capacity; };
+  // which rows go on where the row ahead of them ended
+  unsigned cont = 0;
+  if constexpr (TIME) {
+    const int pl = __shfl_up_sync(ALL, my_lane, 1), pp = __shfl_up_sync(ALL, my_pos, 1);
+    cont = __ballot_sync(ALL, a.map.row_lane && ln > 0 && my_lane >= 0 && pl == my_lane && pp == my_pos - 1);
+  }
+  auto ahead_of = [&](int r) { return min(__clz(~(cont << (31 - HIST - r))), HIST); };   // rows of the portion ahead of row r, at most HIST
+  auto state_at = [&](int lane, int pos) -> float* { return a.state + ((int64_t)lane * (a.m.taps - 1) + pos % (a.m.taps - 1)) * C + col; };
+  float4 t0 = make_float4(0.f, 0.f, 0.f, 0.f), t1 = t0;   // (cos, sin) of this lane's four features (RW == 1)
+  const bool rot_reg = PC == 1 && half > 0 && half % 4 == 0;
+  auto rope_row = [&](int pos) { return a.m.rope + (int64_t)(ok_at(pos) ? pos : 0) * half; };
+  auto rope_load = [&](int pos) {
+    const int i = ln * 4;
+    if (i >= 2 * half) return;
+    const float2* cs = rope_row(pos) + (i < half ? i : i - half);
+    t0 = *reinterpret_cast<const float4*>(cs);
+    t1 = *reinterpret_cast<const float4*>(cs + 2);
+  };
+  if constexpr (TIME && RW == 1) {
+    const int pos = pos_of(0);
+    const int lane = __shfl_sync(ALL, my_lane, HIST);
+    if (conv_reg && !a.map.row_lane)
+#pragma unroll
+      for (int b = 1; b < BACK; ++b)
+#pragma unroll
+        for (int c = 0; c < PC; ++c) {
+          const int i = (c * 32 + ln) * 4;
+          if (b < a.m.taps && pos - b >= 0 && i < n) past[b][c] = *reinterpret_cast<const float4*>(state_at(lane, pos - b) + i);
+        }
+    if (rot_reg) rope_load(pos);
   }
   if (a.early) pdl_wait();
-  if (unit > H + G + GV || (unit == H + G + GV && !a.m.gate)) return;
   const float* p = a.partial + row0 * a.ld;
   if (unit == H + G + GV) {
     p += (int64_t)H * K + (int64_t)G * K + (int64_t)GV * V;
@@ -145,18 +170,26 @@ __global__ void __launch_bounds__(256) gqa_post_kernel(GqaPostArgs a, int64_t ro
         const int i = (c * 32 + ln) * 4;
         x[r][c] = r < nr && i < n ? *reinterpret_cast<const float4*>(p + r * a.ld + col + i) : make_float4(0.f, 0.f, 0.f, 0.f);
       }
-#pragma unroll 4
-    for (int s = 1; s < a.nsplit; ++s)
+    constexpr int SU = RW == 1 ? 8 / PC : 1;   // slabs requested together
+    for (int s = 1; s < a.nsplit; s += SU) {
+      float4 w[SU][RW][PC];
 #pragma unroll
-      for (int r = 0; r < RW; ++r)
+      for (int u = 0; u < SU; ++u)
 #pragma unroll
-        for (int c = 0; c < PC; ++c) {
-          const int i = (c * 32 + ln) * 4;
-          if (r < nr && i < n) {
-            const float4 w = *reinterpret_cast<const float4*>(p + s * a.split_stride + r * a.ld + col + i);
-            x[r][c].x += w.x; x[r][c].y += w.y; x[r][c].z += w.z; x[r][c].w += w.w;
+        for (int r = 0; r < RW; ++r)
+#pragma unroll
+          for (int c = 0; c < PC; ++c) {
+            const int i = (c * 32 + ln) * 4;
+            w[u][r][c] = s + u < a.nsplit && r < nr && i < n ? *reinterpret_cast<const float4*>(p + (s + u) * a.split_stride + r * a.ld + col + i)
+                                                             : make_float4(0.f, 0.f, 0.f, 0.f);
           }
-        }
+#pragma unroll
+      for (int u = 0; u < SU; ++u)
+#pragma unroll
+        for (int r = 0; r < RW; ++r)
+#pragma unroll
+          for (int c = 0; c < PC; ++c) add4(x[r][c], w[u][r][c]);
+    }
   } else {
 #pragma unroll
     for (int r = 0; r < RW; ++r)
@@ -164,61 +197,58 @@ __global__ void __launch_bounds__(256) gqa_post_kernel(GqaPostArgs a, int64_t ro
       for (int c = 0; c < PC; ++c) x[r][c] = r < nr ? slab4(a, p + r * a.ld + col, (c * 32 + ln) * 4, n) : make_float4(0.f, 0.f, 0.f, 0.f);
   }
   if constexpr (TIME) {
-    if (conv) {
-      int ahead[RW];
+    if (conv_reg) {
+      if (RW > 1 || a.map.row_lane) {
+        const int ahead = ahead_of(0);   // rows of the step ahead of the first one here
 #pragma unroll
-      for (int r = 0; r < RW; ++r) ahead[r] = r < nr ? rows_ahead(a, row0 + r, pos[r]) : 0;
-      if (conv_reg) {
-        if (RW > 1 || a.map.row_lane) {
-          // rows of the step ahead of the first one here
-#pragma unroll
-          for (int b = 1; b < CONV_REG_TAPS; ++b)
-#pragma unroll
-            for (int c = 0; c < PC; ++c) {
-              const int i = (c * 32 + ln) * 4;
-              past[b][c] = make_float4(0.f, 0.f, 0.f, 0.f);
-              if (b > ahead[0] || i >= n) continue;
-              for (int s = 0; s < a.nsplit; ++s) {
-                const float4 w = *reinterpret_cast<const float4*>(p + s * a.split_stride - b * a.ld + col + i);
-                past[b][c].x += w.x; past[b][c].y += w.y; past[b][c].z += w.z; past[b][c].w += w.w;
-              }
-            }
-        }
-#pragma unroll
-        for (int c = 0; c < PC; ++c) {
-          const int i = (c * 32 + ln) * 4;
-#pragma unroll
-          for (int r = RW - 1; r >= 0; --r) {     // backwards: the values ahead of a row are still the projected ones
-            const float4 u = x[r][c];
-            float4 y = make_float4(cw[0][c].x * u.x, cw[0][c].y * u.y, cw[0][c].z * u.z, cw[0][c].w * u.w);
-#pragma unroll
-            for (int b = 1; b < CONV_REG_TAPS; ++b) {
-              const bool given = RW == 1 && !a.map.row_lane;      // requested above
-              float4 h = r >= b ? x[r >= b ? r - b : 0][c] : past[r < b ? b - r : 0][c];
-              if (!given && b > ahead[r]) h = state4(r, b, i);
-              fma4(y, cw[b][c], h);
-            }
-            x[r][c] = y;
-            if (!a.tails && a.m.taps > 1 && r < nr && i < n && ok[r]) *reinterpret_cast<float4*>(state_at(r, 0) + i) = u;
-          }
-        }
-      } else {
-#pragma unroll
-        for (int r = 0; r < RW; ++r) {
-          if (r >= nr) break;
+        for (int b = 1; b < BACK; ++b)
 #pragma unroll
           for (int c = 0; c < PC; ++c) {
             const int i = (c * 32 + ln) * 4;
-            float4 u = x[r][c], y = make_float4(0.f, 0.f, 0.f, 0.f);
-            for (int b = 0; b < a.m.taps; ++b) {
-              const float4 w = slab4(a.m.conv + (a.m.taps - 1 - b) * C + col, 1, 0, i, n);
-              if (b == 0) fma4(y, w, u);
-              else if (b <= ahead[r]) fma4(y, w, slab4(a, p + (r - b) * a.ld + col, i, n));
-              else if (pos[r] - b >= 0) fma4(y, w, slab4(state_at(r, b), 1, 0, i, n));
-            }
-            x[r][c] = y;
-            if (!a.tails && a.m.taps > 1 && ok[r]) put4<float>(state_at(r, 0), i, n, u);
+            if (b > ahead || i >= n) continue;
+            for (int s = 0; s < a.nsplit; ++s) add4(past[b][c], *reinterpret_cast<const float4*>(p + s * a.split_stride - b * a.ld + col + i));
           }
+      }
+#pragma unroll
+      for (int r = RW - 1; r >= 0; --r) {     // backwards: the values ahead of a row are still the projected ones
+        const int pos = pos_of(r), lane = __shfl_sync(ALL, my_lane, min(r, nr - 1) + HIST);
+        const int given = RW == 1 && !a.map.row_lane ? HIST : ahead_of(r);   // values at hand; older ones are the state's
+#pragma unroll
+        for (int c = 0; c < PC; ++c) {
+          const int i = (c * 32 + ln) * 4;
+          const float4 u = x[r][c];
+          float4 y = make_float4(cw[0][c].x * u.x, cw[0][c].y * u.y, cw[0][c].z * u.z, cw[0][c].w * u.w);
+#pragma unroll
+          for (int b = 1; b < BACK; ++b) {
+            float4 h = r >= b ? x[r >= b ? r - b : 0][c] : past[r < b ? b - r : 0][c];
+            if (b > given) {
+              h = make_float4(0.f, 0.f, 0.f, 0.f);
+              if (b < a.m.taps && pos - b >= 0 && r < nr && i < n) h = *reinterpret_cast<const float4*>(state_at(lane, pos - b) + i);
+            }
+            fma4(y, cw[b][c], h);
+          }
+          x[r][c] = y;
+          if (!a.tails && a.m.taps > 1 && r < nr && i < n && ok_at(pos)) *reinterpret_cast<float4*>(state_at(lane, pos) + i) = u;
+        }
+      }
+    } else if (conv) {
+#pragma unroll
+      for (int r = 0; r < RW; ++r) {
+        if (r >= nr) break;
+        const int pos = pos_of(r), lane = __shfl_sync(ALL, my_lane, r + HIST), ahead = rows_ahead(a, row0 + r, pos);
+#pragma unroll
+        for (int c = 0; c < PC; ++c) {
+          const int i = (c * 32 + ln) * 4;
+          const float4 u = x[r][c];
+          float4 y = make_float4(0.f, 0.f, 0.f, 0.f);
+          for (int b = 0; b < a.m.taps; ++b) {
+            const float4 w = slab4(a.m.conv + (a.m.taps - 1 - b) * C + col, 1, 0, i, n);
+            if (b == 0) fma4(y, w, u);
+            else if (b <= ahead) fma4(y, w, slab4(a, p + (r - b) * a.ld + col, i, n));
+            else if (pos - b >= 0) fma4(y, w, slab4(state_at(lane, pos - b), 1, 0, i, n));
+          }
+          x[r][c] = y;
+          if (!a.tails && a.m.taps > 1 && ok_at(pos)) put4<float>(state_at(lane, pos), i, n, u);
         }
       }
     }
@@ -234,6 +264,7 @@ __global__ void __launch_bounds__(256) gqa_post_kernel(GqaPostArgs a, int64_t ro
 #pragma unroll
   for (int r = 0; r < RW; ++r) {
     if (r >= nr) break;
+    const int pos = pos_of(r), page = __shfl_sync(ALL, my_page, r + HIST);
     float f = 1.f;
     if (w) {
       float ss = 0.f;
@@ -241,64 +272,174 @@ __global__ void __launch_bounds__(256) gqa_post_kernel(GqaPostArgs a, int64_t ro
       for (int c = 0; c < PC; ++c) ss += x[r][c].x * x[r][c].x + x[r][c].y * x[r][c].y + x[r][c].z * x[r][c].z + x[r][c].w * x[r][c].w;
       f = 1.0f / sqrtf(warp_sum(ss) / (float)K + a.eps);
     }
-    if (is_q && a.m.temp_every > 0) f *= 1.0f + a.m.temp_coef * logf((float)((pos[r] + 1) / a.m.temp_every + 1));
+    if (is_q && a.m.temp_every > 0) f *= 1.0f + a.m.temp_coef * logf((float)((pos + 1) / a.m.temp_every + 1));
     T* dst;
     if (is_q) {
       dst = reinterpret_cast<T*>(a.q) + (row0 + r) * a.ldq + (int64_t)unit * K;
     } else {
-      if (!ok[r]) continue;
-      const int64_t crow = ((int64_t)page[r] * G + (is_v ? unit - H - G : unit - H)) * PAGE_TOKENS + pos[r] % PAGE_TOKENS;
+      if (!ok_at(pos)) continue;
+      const int64_t crow = ((int64_t)page * G + (is_v ? unit - H - G : unit - H)) * PAGE_TOKENS + pos % PAGE_TOKENS;
       dst = is_v ? reinterpret_cast<T*>(a.vc) + crow * a.ldv : reinterpret_cast<T*>(a.kc) + crow * a.ldk;
-    }
-    if constexpr (TIME) {
-      if (!is_q && !is_v && a.m.v_from_k) {
-        const int64_t crow = ((int64_t)page[r] * G + unit - H) * PAGE_TOKENS + pos[r] % PAGE_TOKENS;
+      if (TIME && !is_v && a.m.v_from_k)
 #pragma unroll
         for (int c = 0; c < PC; ++c) put4<T>(reinterpret_cast<T*>(a.vc) + crow * a.ldv, (c * 32 + ln) * 4, n, x[r][c]);
-      }
-      if (!is_v && a.m.rope_dims > 0) {
+    }
+#pragma unroll
+    for (int c = 0; c < PC; ++c) x[r][c] = make_float4(x[r][c].x * f * g[c].x, x[r][c].y * f * g[c].y, x[r][c].z * f * g[c].z, x[r][c].w * f * g[c].w);
+    if constexpr (TIME) {
+      if (rot_reg) {
+        // the four features of a lane lie in one half; the other half is half / 4 lanes away
+        if (RW > 1) rope_load(pos);
+        const bool lo = ln * 4 < half;
+        const int from = (lo ? ln + half / 4 : ln - half / 4) & 31;
+        const float sg = lo ? -1.f : 1.f;
+        const float4 e = x[r][0];
+        const float4 o = make_float4(__shfl_sync(ALL, e.x, from), __shfl_sync(ALL, e.y, from), __shfl_sync(ALL, e.z, from), __shfl_sync(ALL, e.w, from));
+        if (ln * 4 < 2 * half)
+          x[r][0] = make_float4(e.x * t0.x + sg * (o.x * t0.y), e.y * t0.z + sg * (o.y * t0.w), e.z * t1.x + sg * (o.z * t1.y), e.w * t1.z + sg * (o.w * t1.w));
+      } else if (half > 0) {
         float* s = s_rot[threadIdx.x >> 5];
-        const int half = a.m.rope_dims / 2;
-        const float2* cs = a.m.rope + (int64_t)(ok[r] ? pos[r] : 0) * half;
+        const float2* cs = rope_row(pos);
 #pragma unroll
-        for (int c = 0; c < PC; ++c) {
-          x[r][c] = make_float4(x[r][c].x * f * g[c].x, x[r][c].y * f * g[c].y, x[r][c].z * f * g[c].z, x[r][c].w * f * g[c].w);
-          *reinterpret_cast<float4*>(s + (c * 32 + ln) * 4) = x[r][c];
-        }
+        for (int c = 0; c < PC; ++c) *reinterpret_cast<float4*>(s + (c * 32 + ln) * 4) = x[r][c];
         __syncwarp();
 #pragma unroll
         for (int c = 0; c < PC; ++c) {
-          const int i = (c * 32 + ln) * 4;
-          float e[4] = {x[r][c].x, x[r][c].y, x[r][c].z, x[r][c].w};
-          if (half % 4 == 0 && i < 2 * half) {      // the four columns lie in one half, the table row starts on 32 bytes
-            const bool lo = i < half;
-            const int j = lo ? i : i - half;
-            const float4 o = *reinterpret_cast<const float4*>(s + (lo ? i + half : j));
-            const float4 t0 = *reinterpret_cast<const float4*>(cs + j), t1 = *reinterpret_cast<const float4*>(cs + j + 2);
-            const float sg = lo ? -1.f : 1.f;
-            e[0] = e[0] * t0.x + sg * (o.x * t0.y);
-            e[1] = e[1] * t0.z + sg * (o.y * t0.w);
-            e[2] = e[2] * t1.x + sg * (o.z * t1.y);
-            e[3] = e[3] * t1.z + sg * (o.w * t1.w);
-          } else if (half % 4 != 0) {
+          float* e = reinterpret_cast<float*>(&x[r][c]);
 #pragma unroll
-            for (int u = 0; u < 4; ++u) {
-              if (i + u >= 2 * half) continue;
-              const bool lo = i + u < half;
-              const float2 t = cs[lo ? i + u : i + u - half];
-              e[u] = lo ? e[u] * t.x - s[i + u + half] * t.y : e[u] * t.x + s[i + u - half] * t.y;
-            }
+          for (int u = 0; u < 4; ++u) {
+            const int i = (c * 32 + ln) * 4 + u;
+            if (i >= 2 * half) continue;
+            const float2 t = cs[i < half ? i : i - half];
+            e[u] = i < half ? e[u] * t.x - s[i + half] * t.y : e[u] * t.x + s[i - half] * t.y;
           }
-          put4<T>(dst, i, n, make_float4(e[0], e[1], e[2], e[3]));
         }
         __syncwarp();
-        continue;
       }
     }
 #pragma unroll
-    for (int c = 0; c < PC; ++c)
-      put4<T>(dst, (c * 32 + ln) * 4, n, make_float4(x[r][c].x * f * g[c].x, x[r][c].y * f * g[c].y, x[r][c].z * f * g[c].z, x[r][c].w * f * g[c].w));
+    for (int c = 0; c < PC; ++c) put4<T>(dst, (c * 32 + ln) * 4, n, x[r][c]);
   }
+}
+
+// The same for large steps of heads with a convolution, rotation or values that are their keys, where `rows_post_ok`: a warp
+// owns four columns a lane of one head and walks down TR rows with the last values in registers.
+constexpr int TR = 32;
+template <typename T>
+__global__ void __launch_bounds__(256, 4) gqa_post_rows_kernel(GqaPostArgs a, int64_t rows) {
+  constexpr unsigned ALL = 0xffffffffu;
+  __shared__ int4 info[TR];      // per row: lane, position (-1: outside the cache), page, rows of its portion ahead of it in this step (up to three)
+  pdl_launch_dependents();
+  const int64_t row0 = (int64_t)blockIdx.x * TR;
+  const int nr = (int)min((int64_t)TR, rows - row0);
+  const int unit = blockIdx.y * 8 + (threadIdx.x >> 5), ln = threadIdx.x & 31;
+  const int H = a.m.heads, G = a.m.own_kv ? a.m.kv_heads : 0, K = a.m.dim, V = a.m.vdim, GV = a.m.v_from_k ? 0 : G;
+  const bool is_q = unit < H, is_v = unit >= H + G;
+  const int n = is_v ? V : K, i = ln * 4, half = is_v ? 0 : a.m.rope_dims / 2;
+  const bool on = i < n && unit < H + G + GV;
+  const int64_t col = (is_v ? (int64_t)(H + G) * K + (int64_t)(unit - H - G) * V : (int64_t)unit * K) + i, C = gqa_channels(a.m);
+  const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f), one = make_float4(1.f, 1.f, 1.f, 1.f);
+  float4 cw[CONV_REG_TAPS];
+#pragma unroll
+  for (int b = 0; b < CONV_REG_TAPS; ++b) {
+    cw[b] = b == 0 && (is_v || a.m.taps == 0) ? one : zero;
+    if (on && !is_v && b < a.m.taps) cw[b] = *reinterpret_cast<const float4*>(a.m.conv + (a.m.taps - 1 - b) * C + col);
+  }
+  const float* w = is_v ? nullptr : is_q ? a.m.q_norm : a.m.k_norm;
+  const float4 g = w && on ? make_float4(w[i], w[i + 1], w[i + 2], w[i + 3]) : one;
+  pdl_wait();
+  if ((int)threadIdx.x < nr) {
+    const int64_t row = row0 + threadIdx.x;
+    const int lane = row_lane(a.map, row), pos = row_pos(a.map, row);
+    const bool in = pos >= 0 && pos < a.capacity;
+    int ahead = 0;
+    if (a.map.row_lane)
+#pragma unroll
+      for (int b = 1; b < CONV_REG_TAPS; ++b)
+        if (row >= b && a.map.row_lane[row - b] == lane && a.map.row_pos[row - b] == pos - b) ahead = b;
+    info[threadIdx.x] = make_int4(lane, in ? pos : -1, a.block_table[(int64_t)lane * a.max_pages + (in ? pos / PAGE_TOKENS : 0)], ahead);
+    if (!in && blockIdx.y == 0) atomicExch(a.status, KS_BAD_INDEX);
+  }
+  __syncthreads();
+  if (unit > H + G + GV || (unit == H + G + GV && !a.m.gate)) return;
+  if (unit == H + G + GV) {
+    const float* p = a.partial + row0 * a.ld + (int64_t)(H + G) * K + (int64_t)GV * V;
+    for (int k = ln; k < nr * H; k += 32) {
+      const int r = k / H, h = k % H;
+      float z = 0.f;
+      for (int s = 0; s < a.nsplit; ++s) z += p[s * a.split_stride + r * a.ld + h];
+      a.gate[(row0 + r) * H + h] = sigmoid(z);
+    }
+    return;
+  }
+  const float* p = a.partial + row0 * a.ld + col;
+  auto value = [&](int r) {
+    float4 v = on ? *reinterpret_cast<const float4*>(p + r * a.ld) : zero;
+    for (int s = 1; s < a.nsplit; ++s)
+      if (on) add4(v, *reinterpret_cast<const float4*>(p + s * a.split_stride + r * a.ld));
+    return v;
+  };
+  float4 h[CONV_REG_TAPS];   // projected values by tokens ago
+  // those ahead of row r that no row at hand gives, from `first` tokens ago on
+  auto from_state = [&](const int4& in, int first) {
+#pragma unroll
+    for (int b = 1; b < CONV_REG_TAPS; ++b) {
+      if (b < first) continue;
+      h[b] = zero;
+      if (on && !is_v && b < a.m.taps && in.y - b >= 0)
+        h[b] = *reinterpret_cast<const float4*>(a.state + ((int64_t)in.x * (a.m.taps - 1) + (in.y - b) % (a.m.taps - 1)) * C + col);
+    }
+  };
+  from_state(info[0], info[0].w + 1);
+#pragma unroll
+  for (int b = 1; b < CONV_REG_TAPS; ++b)
+    if (b <= info[0].w) h[b] = value(-b);
+  const bool lo = i < half, turned = i < 2 * half;
+  const int from = (lo ? ln + half / 4 : ln - half / 4) & 31, j = lo ? i : i - half;
+  const float sg = lo ? -1.f : 1.f;
+  T* const q = reinterpret_cast<T*>(a.q) + row0 * a.ldq + (int64_t)unit * K + i;
+  auto put = [&](T* d, float4 v) {
+    if constexpr (sizeof(T) == 2) *reinterpret_cast<uint2*>(d) = make_uint2(pack_bf16(v.x, v.y), pack_bf16(v.z, v.w));
+    else *reinterpret_cast<float4*>(d) = v;
+  };
+  for (int r = 0; r < nr; ++r) {
+    const float4 x = value(r);
+    const int4 in = info[r];
+    float4 t0 = zero, t1 = zero;
+    if (turned) {
+      const float2* cs = a.m.rope + (int64_t)max(in.y, 0) * half + j;
+      t0 = *reinterpret_cast<const float4*>(cs);
+      t1 = *reinterpret_cast<const float4*>(cs + 2);
+    }
+    if (in.w == 0 && r > 0) from_state(in, 1);      // a portion starts here
+    float4 y = make_float4(cw[0].x * x.x, cw[0].y * x.y, cw[0].z * x.z, cw[0].w * x.w);
+#pragma unroll
+    for (int b = 1; b < CONV_REG_TAPS; ++b) fma4(y, cw[b], h[b]);
+#pragma unroll
+    for (int b = CONV_REG_TAPS - 1; b > 1; --b) h[b] = h[b - 1];
+    h[1] = x;
+    if (!a.tails && a.m.taps > 1 && on && !is_v && in.y >= 0)
+      *reinterpret_cast<float4*>(a.state + ((int64_t)in.x * (a.m.taps - 1) + in.y % (a.m.taps - 1)) * C + col) = x;
+    const int64_t crow = ((int64_t)in.z * G + (is_v ? unit - H - G : unit - H)) * PAGE_TOKENS + in.y % PAGE_TOKENS;
+    if (!is_q && !is_v && a.m.v_from_k && on && in.y >= 0) put(reinterpret_cast<T*>(a.vc) + crow * a.ldv + i, y);
+    float f = 1.f;
+    if (w) f = 1.0f / sqrtf(warp_sum(y.x * y.x + y.y * y.y + y.z * y.z + y.w * y.w) / (float)K + a.eps);
+    if (is_q && a.m.temp_every > 0) f *= 1.0f + a.m.temp_coef * logf((float)((in.y + 1) / a.m.temp_every + 1));
+    if (w || f != 1.f) y = make_float4(y.x * f * g.x, y.y * f * g.y, y.z * f * g.z, y.w * f * g.w);
+    if (half > 0) {
+      const float4 o = make_float4(__shfl_sync(ALL, y.x, from), __shfl_sync(ALL, y.y, from), __shfl_sync(ALL, y.z, from), __shfl_sync(ALL, y.w, from));
+      if (turned) y = make_float4(y.x * t0.x + sg * (o.x * t0.y), y.y * t0.z + sg * (o.y * t0.w), y.z * t1.x + sg * (o.z * t1.y), y.w * t1.z + sg * (o.w * t1.w));
+    }
+    if (is_q) {
+      if (on) put(q + r * a.ldq, y);
+    } else if (on && in.y >= 0) {
+      put(is_v ? reinterpret_cast<T*>(a.vc) + crow * a.ldv + i : reinterpret_cast<T*>(a.kc) + crow * a.ldk + i, y);
+    }
+  }
+}
+bool rows_post_ok(const GqaPostArgs& a) {
+  const GqaDims& m = a.m;
+  return m.dim <= 128 && m.vdim <= 128 && m.dim % 4 == 0 && m.vdim % 4 == 0 && a.ld % 4 == 0 && a.ldq % 4 == 0 && m.taps <= CONV_REG_TAPS && m.rope_dims % 8 == 0;
 }
 
 // The last values of every portion into the convolution state.  grid (tails, channels / 512)
@@ -714,13 +855,20 @@ int gqa_post_launch(Ctx* c, const GqaPostArgs& a, int64_t rows) {
   const int units = a.m.heads + (a.m.own_kv ? (a.m.v_from_k ? 1 : 2) * a.m.kv_heads : 0) + (a.m.gate ? 1 : 0);
   const bool time = a.m.taps > 0 || a.m.rope_dims > 0 || a.m.v_from_k;
   RB_REQUIRE(a.m.dim <= 512 && a.m.vdim <= 512, "grouped-query attention: head sizes above 512");
-  const bool small = a.m.dim <= 128 && a.m.vdim <= 128, bf = a.dtype == REWB200_BF16, many = small && bf && rows >= 512;
-  const dim3 grid((unsigned)(many ? (rows + 3) / 4 : rows), (unsigned)((units + 7) / 8));
+  const bool small = a.m.dim <= 128 && a.m.vdim <= 128, bf = a.dtype == REWB200_BF16, many = small && bf && rows >= 512 && !time;
+  const dim3 grid((unsigned)(many ? (rows + POST_ROWS - 1) / POST_ROWS : rows), (unsigned)((units + 7) / 8));
   auto go = [&](auto kernel) { return launch_k(kernel, grid, dim3(256), 0, c->stream, c->use_pdl, a, rows); };
-#define RB_POST(TIME)                                                                                                                \
-  (many ? go(gqa_post_kernel<bf16, 1, 4, TIME>) : bf ? (small ? go(gqa_post_kernel<bf16, 1, 1, TIME>) : go(gqa_post_kernel<bf16, 4, 1, TIME>)) \
+  if (time && rows >= 512 && rows_post_ok(a)) {
+    const dim3 g((unsigned)((rows + TR - 1) / TR), grid.y);
+    RB_CUDA(bf ? launch_k(gqa_post_rows_kernel<bf16>, g, dim3(256), 0, c->stream, c->use_pdl, a, rows)
+               : launch_k(gqa_post_rows_kernel<float>, g, dim3(256), 0, c->stream, c->use_pdl, a, rows));
+    ++g_launch_total;
+    return REWB200_OK;
+  }
+#define RB_POST(TIME)                                                                                      \
+  (bf ? (small ? go(gqa_post_kernel<bf16, 1, 1, TIME>) : go(gqa_post_kernel<bf16, 4, 1, TIME>))            \
    : small ? go(gqa_post_kernel<float, 1, 1, TIME>) : go(gqa_post_kernel<float, 4, 1, TIME>))
-  RB_CUDA(time ? RB_POST(true) : RB_POST(false));
+  RB_CUDA(many ? go(gqa_post_kernel<bf16, 1, POST_ROWS, false>) : time ? RB_POST(true) : RB_POST(false));
 #undef RB_POST
   ++g_launch_total;
   return REWB200_OK;

@@ -455,16 +455,21 @@ def test_wide_batches_of_decoding_lanes(rb):
         close(lg[i:i + 1], G.forward(cfg, t, reqs[i])[-1:], "bfloat16")
 
 
-def test_hundreds_of_sequences_in_one_captured_step(rb):
-    cfg = K.config([K.attention(K.dense(), conv=3), K.latent(K.dense())], cap=30.0)
+@pytest.mark.parametrize("conv,rot", [(3, 16), (4, 20), (7, 24), (1, 8)])
+def test_hundreds_of_sequences_in_one_step(rb, dtype, conv, rot):
+    """Short portions, each starting inside a tile of rows, from the state of the step ahead; then captured decode steps."""
+    cfg = K.config([K.attention(K.dense(), conv=conv, rot=rot), K.latent(K.dense())], cap=30.0)
     t = K.weights(cfg, seed=14)
-    s = build(rb, cfg, t, "bfloat16", max_seq=64).session(516, 64)
-    ids = np.stack([K.tokens(cfg, 6, seed=i) for i in range(516)])
-    first, _ = s.forward(ids, want_logits=True)
+    s = build(rb, cfg, t, dtype, max_seq=64).session(516, 64)
+    ids = np.stack([K.tokens(cfg, 19, seed=i) for i in range(516)])
+    some = (0, 1, 2, 3, 255, 511, 512, 515)
+    for lo, hi in ((0, 6), (6, 8), (8, 9), (9, 19)):
+        first, logits = s.forward(ids[:, lo:hi], want_logits=True)
+        close(logits[list(some)], np.stack([G.forward(cfg, t, ids[i, :hi])[-1] for i in some]), dtype)
     got, logits = s.decode(5, want_logits=True)
-    for i in (0, 1, 2, 3, 255, 511, 512, 515):
+    for i in some:
         full = np.concatenate([ids[i], [first[i]], got[i][:-1]])
-        close(logits[i:i + 1], G.forward(cfg, t, full)[-1:], "bfloat16")
+        close(logits[i:i + 1], G.forward(cfg, t, full)[-1:], dtype)
 
 
 def test_forward_all_and_chunked_session_forward(rb, dtype):
