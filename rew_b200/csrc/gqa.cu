@@ -323,15 +323,15 @@ __global__ void __launch_bounds__(256) gqa_post_kernel(GqaPostArgs a, int64_t ro
 }
 
 // The same for large steps of heads with a convolution, rotation or values that are their keys, where `rows_post_ok`: a warp
-// owns four columns a lane of one head and walks down TR rows with the last values in registers.
-constexpr int TR = 32;
+// owns four columns a lane of one head and walks down tr rows with the last values in registers.
+constexpr int MAX_TR = 32, ROWS_POST_MIN = 512;
 template <typename T>
-__global__ void __launch_bounds__(256, 4) gqa_post_rows_kernel(GqaPostArgs a, int64_t rows) {
+__global__ void __launch_bounds__(256, 4) gqa_post_rows_kernel(GqaPostArgs a, int64_t rows, int tr) {
   constexpr unsigned ALL = 0xffffffffu;
-  __shared__ int4 info[TR];      // per row: lane, position (-1: outside the cache), page, rows of its portion ahead of it in this step (up to three)
+  __shared__ int4 info[MAX_TR];      // per row: lane, position (-1: outside the cache), page, rows of its portion ahead of it in this step (up to three)
   pdl_launch_dependents();
-  const int64_t row0 = (int64_t)blockIdx.x * TR;
-  const int nr = (int)min((int64_t)TR, rows - row0);
+  const int64_t row0 = (int64_t)blockIdx.x * tr;
+  const int nr = (int)min((int64_t)tr, rows - row0);
   const int unit = blockIdx.y * 8 + (threadIdx.x >> 5), ln = threadIdx.x & 31;
   const int H = a.m.heads, G = a.m.own_kv ? a.m.kv_heads : 0, K = a.m.dim, V = a.m.vdim, GV = a.m.v_from_k ? 0 : G;
   const bool is_q = unit < H, is_v = unit >= H + G;
@@ -858,10 +858,12 @@ int gqa_post_launch(Ctx* c, const GqaPostArgs& a, int64_t rows) {
   const bool small = a.m.dim <= 128 && a.m.vdim <= 128, bf = a.dtype == REWB200_BF16, many = small && bf && rows >= 512 && !time;
   const dim3 grid((unsigned)(many ? (rows + POST_ROWS - 1) / POST_ROWS : rows), (unsigned)((units + 7) / 8));
   auto go = [&](auto kernel) { return launch_k(kernel, grid, dim3(256), 0, c->stream, c->use_pdl, a, rows); };
-  if (time && rows >= 512 && rows_post_ok(a)) {
-    const dim3 g((unsigned)((rows + TR - 1) / TR), grid.y);
-    RB_CUDA(bf ? launch_k(gqa_post_rows_kernel<bf16>, g, dim3(256), 0, c->stream, c->use_pdl, a, rows)
-               : launch_k(gqa_post_rows_kernel<float>, g, dim3(256), 0, c->stream, c->use_pdl, a, rows));
+  if (time && rows >= ROWS_POST_MIN && rows_post_ok(a)) {
+    int tr = MAX_TR;         // long walks, but four CTAs for every SM
+    while (tr > 4 && (rows + tr - 1) / tr * grid.y < 4 * c->sm_count) tr /= 2;
+    const dim3 g((unsigned)((rows + tr - 1) / tr), grid.y);
+    RB_CUDA(bf ? launch_k(gqa_post_rows_kernel<bf16>, g, dim3(256), 0, c->stream, c->use_pdl, a, rows, tr)
+               : launch_k(gqa_post_rows_kernel<float>, g, dim3(256), 0, c->stream, c->use_pdl, a, rows, tr));
     ++g_launch_total;
     return REWB200_OK;
   }
