@@ -325,16 +325,18 @@ __global__ void __launch_bounds__(256) gqa_post_kernel(GqaPostArgs a, int64_t ro
 // The same for large steps of heads with a convolution, rotation or values that are their keys, where `rows_post_ok`: a warp
 // owns four columns a lane of one head and walks down tr rows with the last values in registers.
 constexpr int MAX_TR = 32, ROWS_POST_MIN = 512;
-template <typename T>
+template <typename T, bool NORM>     // NORM: RMS norms or a query temperature
 __global__ void __launch_bounds__(256, 4) gqa_post_rows_kernel(GqaPostArgs a, int64_t rows, int tr) {
   constexpr unsigned ALL = 0xffffffffu;
-  __shared__ int4 info[MAX_TR];      // per row: lane, position (-1: outside the cache), page, rows of its portion ahead of it in this step (up to three)
+  // per row: position (-1: outside the cache), row of its page's first head in the cache, rows of its portion ahead of it in
+  // this step (up to three), lane
+  __shared__ int4 info[MAX_TR];
   pdl_launch_dependents();
   const int64_t row0 = (int64_t)blockIdx.x * tr;
   const int nr = (int)min((int64_t)tr, rows - row0);
   const int unit = blockIdx.y * 8 + (threadIdx.x >> 5), ln = threadIdx.x & 31;
   const int H = a.m.heads, G = a.m.own_kv ? a.m.kv_heads : 0, K = a.m.dim, V = a.m.vdim, GV = a.m.v_from_k ? 0 : G;
-  const bool is_q = unit < H, is_v = unit >= H + G;
+  const bool is_q = unit < H, is_v = unit >= H + G, twice = !is_q && !is_v && a.m.v_from_k;   // twice: key and value
   const int n = is_v ? V : K, i = ln * 4, half = is_v ? 0 : a.m.rope_dims / 2;
   const bool on = i < n && unit < H + G + GV;
   const int64_t col = (is_v ? (int64_t)(H + G) * K + (int64_t)(unit - H - G) * V : (int64_t)unit * K) + i, C = gqa_channels(a.m);
@@ -346,7 +348,7 @@ __global__ void __launch_bounds__(256, 4) gqa_post_rows_kernel(GqaPostArgs a, in
     if (on && !is_v && b < a.m.taps) cw[b] = *reinterpret_cast<const float4*>(a.m.conv + (a.m.taps - 1 - b) * C + col);
   }
   const float* w = is_v ? nullptr : is_q ? a.m.q_norm : a.m.k_norm;
-  const float4 g = w && on ? make_float4(w[i], w[i + 1], w[i + 2], w[i + 3]) : one;
+  const float4 g = NORM && w && on ? make_float4(w[i], w[i + 1], w[i + 2], w[i + 3]) : one;
   pdl_wait();
   if ((int)threadIdx.x < nr) {
     const int64_t row = row0 + threadIdx.x;
@@ -357,7 +359,8 @@ __global__ void __launch_bounds__(256, 4) gqa_post_rows_kernel(GqaPostArgs a, in
 #pragma unroll
       for (int b = 1; b < CONV_REG_TAPS; ++b)
         if (row >= b && a.map.row_lane[row - b] == lane && a.map.row_pos[row - b] == pos - b) ahead = b;
-    info[threadIdx.x] = make_int4(lane, in ? pos : -1, a.block_table[(int64_t)lane * a.max_pages + (in ? pos / PAGE_TOKENS : 0)], ahead);
+    const int page = a.block_table[(int64_t)lane * a.max_pages + (in ? pos / PAGE_TOKENS : 0)];
+    info[threadIdx.x] = make_int4(in ? pos : -1, page * G * PAGE_TOKENS + (in ? pos % PAGE_TOKENS : 0), ahead, lane);
     if (!in && blockIdx.y == 0) atomicExch(a.status, KS_BAD_INDEX);
   }
   __syncthreads();
@@ -372,68 +375,74 @@ __global__ void __launch_bounds__(256, 4) gqa_post_rows_kernel(GqaPostArgs a, in
     }
     return;
   }
-  const float* p = a.partial + row0 * a.ld + col;
-  auto value = [&](int r) {
-    float4 v = on ? *reinterpret_cast<const float4*>(p + r * a.ld) : zero;
+  auto value = [&](const float* p) {
+    float4 v = on ? *reinterpret_cast<const float4*>(p) : zero;
     for (int s = 1; s < a.nsplit; ++s)
-      if (on) add4(v, *reinterpret_cast<const float4*>(p + s * a.split_stride + r * a.ld));
+      if (on) add4(v, *reinterpret_cast<const float4*>(p + s * a.split_stride));
     return v;
   };
-  float4 h[CONV_REG_TAPS];   // projected values by tokens ago
-  // those ahead of row r that no row at hand gives, from `first` tokens ago on
+  auto state_at = [&](int lane, int pos) { return reinterpret_cast<float4*>(a.state + ((int64_t)lane * (a.m.taps - 1) + pos % (a.m.taps - 1)) * C + col); };
+  const float* xp = a.partial + row0 * a.ld + col;
+  float4 h1 = zero, h2 = zero, h3 = zero;   // projected values by tokens ago
+  // those that no row at hand gives, from `first` tokens ago on
   auto from_state = [&](const int4& in, int first) {
-#pragma unroll
-    for (int b = 1; b < CONV_REG_TAPS; ++b) {
-      if (b < first) continue;
-      h[b] = zero;
-      if (on && !is_v && b < a.m.taps && in.y - b >= 0)
-        h[b] = *reinterpret_cast<const float4*>(a.state + ((int64_t)in.x * (a.m.taps - 1) + (in.y - b) % (a.m.taps - 1)) * C + col);
-    }
+    auto at = [&](int b) { return on && !is_v && b < a.m.taps && in.x - b >= 0 ? *state_at(in.w, in.x - b) : zero; };
+    if (first <= 1) h1 = at(1);
+    if (first <= 2) h2 = at(2);
+    if (first <= 3) h3 = at(3);
   };
-  from_state(info[0], info[0].w + 1);
-#pragma unroll
-  for (int b = 1; b < CONV_REG_TAPS; ++b)
-    if (b <= info[0].w) h[b] = value(-b);
+  from_state(info[0], info[0].z + 1);
+  if (info[0].z >= 1) h1 = value(xp - a.ld);
+  if (info[0].z >= 2) h2 = value(xp - 2 * a.ld);
+  if (info[0].z >= 3) h3 = value(xp - 3 * a.ld);
   const bool lo = i < half, turned = i < 2 * half;
-  const int from = (lo ? ln + half / 4 : ln - half / 4) & 31, j = lo ? i : i - half;
+  const int from = (lo ? ln + half / 4 : ln - half / 4) & 31;
   const float sg = lo ? -1.f : 1.f;
+  const float2* const rope = a.m.rope + (lo ? i : i - half);
+  const int hk = is_v ? unit - H - G : unit - H;
   T* const q = reinterpret_cast<T*>(a.q) + row0 * a.ldq + (int64_t)unit * K + i;
-  auto put = [&](T* d, float4 v) {
+  T* const kc = reinterpret_cast<T*>(a.kc) + (int64_t)hk * PAGE_TOKENS * a.ldk + i;
+  T* const vc = reinterpret_cast<T*>(a.vc) + (int64_t)hk * PAGE_TOKENS * a.ldv + i;
+  const bool keep = !a.tails && a.m.taps > 1 && on && !is_v;
+  auto put = [&](T* d, const float4& v) {
     if constexpr (sizeof(T) == 2) *reinterpret_cast<uint2*>(d) = make_uint2(pack_bf16(v.x, v.y), pack_bf16(v.z, v.w));
     else *reinterpret_cast<float4*>(d) = v;
   };
+#pragma unroll 1
   for (int r = 0; r < nr; ++r) {
-    const float4 x = value(r);
+    const float4 x = value(xp);
+    xp += a.ld;
     const int4 in = info[r];
-    float4 t0 = zero, t1 = zero;
+    float4 t0, t1;
     if (turned) {
-      const float2* cs = a.m.rope + (int64_t)max(in.y, 0) * half + j;
+      const float2* cs = rope + (int64_t)max(in.x, 0) * half;
       t0 = *reinterpret_cast<const float4*>(cs);
       t1 = *reinterpret_cast<const float4*>(cs + 2);
     }
-    if (in.w == 0 && r > 0) from_state(in, 1);      // a portion starts here
+    if (in.z == 0 && r > 0) from_state(in, 1);      // a portion starts here
     float4 y = make_float4(cw[0].x * x.x, cw[0].y * x.y, cw[0].z * x.z, cw[0].w * x.w);
-#pragma unroll
-    for (int b = 1; b < CONV_REG_TAPS; ++b) fma4(y, cw[b], h[b]);
-#pragma unroll
-    for (int b = CONV_REG_TAPS - 1; b > 1; --b) h[b] = h[b - 1];
-    h[1] = x;
-    if (!a.tails && a.m.taps > 1 && on && !is_v && in.y >= 0)
-      *reinterpret_cast<float4*>(a.state + ((int64_t)in.x * (a.m.taps - 1) + in.y % (a.m.taps - 1)) * C + col) = x;
-    const int64_t crow = ((int64_t)in.z * G + (is_v ? unit - H - G : unit - H)) * PAGE_TOKENS + in.y % PAGE_TOKENS;
-    if (!is_q && !is_v && a.m.v_from_k && on && in.y >= 0) put(reinterpret_cast<T*>(a.vc) + crow * a.ldv + i, y);
-    float f = 1.f;
-    if (w) f = 1.0f / sqrtf(warp_sum(y.x * y.x + y.y * y.y + y.z * y.z + y.w * y.w) / (float)K + a.eps);
-    if (is_q && a.m.temp_every > 0) f *= 1.0f + a.m.temp_coef * logf((float)((in.y + 1) / a.m.temp_every + 1));
-    if (w || f != 1.f) y = make_float4(y.x * f * g.x, y.y * f * g.y, y.z * f * g.z, y.w * f * g.w);
+    fma4(y, cw[1], h1);
+    fma4(y, cw[2], h2);
+    fma4(y, cw[3], h3);
+    h3 = h2;
+    h2 = h1;
+    h1 = x;
+    if (keep && in.x >= 0) *state_at(in.w, in.x) = x;
+    if (twice && on && in.x >= 0) put(vc + (int64_t)in.y * a.ldv, y);
+    if constexpr (NORM) {
+      float f = 1.f;
+      if (w) f = 1.0f / sqrtf(warp_sum(y.x * y.x + y.y * y.y + y.z * y.z + y.w * y.w) / (float)K + a.eps);
+      if (is_q && a.m.temp_every > 0) f *= 1.0f + a.m.temp_coef * logf((float)((in.x + 1) / a.m.temp_every + 1));
+      y = make_float4(y.x * f * g.x, y.y * f * g.y, y.z * f * g.z, y.w * f * g.w);
+    }
     if (half > 0) {
       const float4 o = make_float4(__shfl_sync(ALL, y.x, from), __shfl_sync(ALL, y.y, from), __shfl_sync(ALL, y.z, from), __shfl_sync(ALL, y.w, from));
-      if (turned) y = make_float4(y.x * t0.x + sg * (o.x * t0.y), y.y * t0.z + sg * (o.y * t0.w), y.z * t1.x + sg * (o.z * t1.y), y.w * t1.z + sg * (o.w * t1.w));
+      if (turned) y = make_float4(y.x * t0.x + o.x * (sg * t0.y), y.y * t0.z + o.y * (sg * t0.w), y.z * t1.x + o.z * (sg * t1.y), y.w * t1.z + o.w * (sg * t1.w));
     }
     if (is_q) {
       if (on) put(q + r * a.ldq, y);
-    } else if (on && in.y >= 0) {
-      put(is_v ? reinterpret_cast<T*>(a.vc) + crow * a.ldv + i : reinterpret_cast<T*>(a.kc) + crow * a.ldk + i, y);
+    } else if (on && in.x >= 0) {
+      put(is_v ? vc + (int64_t)in.y * a.ldv : kc + (int64_t)in.y * a.ldk, y);
     }
   }
 }
@@ -862,8 +871,10 @@ int gqa_post_launch(Ctx* c, const GqaPostArgs& a, int64_t rows) {
     int tr = MAX_TR;         // long walks, but four CTAs for every SM
     while (tr > 4 && (rows + tr - 1) / tr * grid.y < 4 * c->sm_count) tr /= 2;
     const dim3 g((unsigned)((rows + tr - 1) / tr), grid.y);
-    RB_CUDA(bf ? launch_k(gqa_post_rows_kernel<bf16>, g, dim3(256), 0, c->stream, c->use_pdl, a, rows, tr)
-               : launch_k(gqa_post_rows_kernel<float>, g, dim3(256), 0, c->stream, c->use_pdl, a, rows, tr));
+    const bool norm = a.m.q_norm || a.m.k_norm || a.m.temp_every > 0;
+    auto go_rows = [&](auto kernel) { return launch_k(kernel, g, dim3(256), 0, c->stream, c->use_pdl, a, rows, tr); };
+    RB_CUDA(bf ? (norm ? go_rows(gqa_post_rows_kernel<bf16, true>) : go_rows(gqa_post_rows_kernel<bf16, false>))
+               : (norm ? go_rows(gqa_post_rows_kernel<float, true>) : go_rows(gqa_post_rows_kernel<float, false>)));
     ++g_launch_total;
     return REWB200_OK;
   }
