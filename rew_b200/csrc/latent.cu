@@ -117,6 +117,88 @@ __global__ void __launch_bounds__(SMALL ? 768 : 128, SMALL ? 1 : 10) latent_post
   for (int i = 2 * half + threadIdx.x; i < nr; i += nt) cr[nc + i] = stf<T>(sx[nq + nc + i]);
 }
 
+// Large steps: a warp per row, which it holds in registers, four columns at a time (up to 128 NV; the parts of a row are
+// multiples of four columns wide).
+template <typename T, int NV>
+__global__ void __launch_bounds__(256, NV <= 10 ? 3 : 2) latent_post_rows_kernel(LatentPostArgs a, int64_t rows) {
+  pdl_launch_dependents();
+  const int64_t row = (int64_t)blockIdx.x * 8 + (threadIdx.x >> 5);
+  const int ln = threadIdx.x & 31;
+  if (row >= rows) return;
+  const int nq = a.m.q_rank, nc = a.m.own_kv ? a.m.kv_rank : 0, nr = a.m.own_kv ? a.m.rot_dim : 0, n = nq + nc + nr + (a.m.gate ? a.m.heads : 0);
+  pdl_wait();
+  const float* p = a.partial + row * a.ld;
+  float4 v[NV];
+#pragma unroll
+  for (int k = 0; k < NV; ++k) {
+    const int i = (k * 32 + ln) * 4;
+    v[k] = i < n ? *reinterpret_cast<const float4*>(p + i) : make_float4(0.f, 0.f, 0.f, 0.f);   // rows are padded to a multiple of 8 columns
+  }
+  const int lane = row_lane(a.map, row), pos = row_pos(a.map, row);
+  const bool ok = pos >= 0 && pos < a.capacity && pos < a.m.max_pos;
+  const int page = a.block_table[(int64_t)lane * a.max_pages + (ok ? pos / PAGE_TOKENS : 0)];
+  if (!ok && ln == 0) atomicExch(a.status, KS_BAD_INDEX);
+  for (int s = 1; s < a.nsplit; ++s)
+#pragma unroll
+    for (int k = 0; k < NV; ++k) {
+      const int i = (k * 32 + ln) * 4;
+      if (i < n) add4(v[k], *reinterpret_cast<const float4*>(p + s * a.split_stride + i));
+    }
+  float sq = 0.f, sc = 0.f;
+#pragma unroll
+  for (int k = 0; k < NV; ++k) {
+    const int i = (k * 32 + ln) * 4;
+    const float t = v[k].x * v[k].x + v[k].y * v[k].y + v[k].z * v[k].z + v[k].w * v[k].w;
+    if (i < nq) sq += t;
+    else if (i < nq + nc) sc += t;
+  }
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) {
+    sq += __shfl_xor_sync(0xffffffffu, sq, o);
+    sc += __shfl_xor_sync(0xffffffffu, sc, o);
+  }
+  const float rq = 1.0f / sqrtf(sq / (float)nq + a.eps), rc = 1.0f / sqrtf(sc / (float)max(nc, 1) + a.eps);
+  auto put = [](T* d, float4 y) {
+    if constexpr (sizeof(T) == 2) *reinterpret_cast<uint2*>(d) = make_uint2(pack_bf16(y.x, y.y), pack_bf16(y.z, y.w));
+    else *reinterpret_cast<float4*>(d) = y;
+  };
+  auto normed = [](const float* w, float4 x, float r) {
+    const float4 g = *reinterpret_cast<const float4*>(w);
+    return make_float4(g.x * (x.x * r), g.y * (x.y * r), g.z * (x.z * r), g.w * (x.w * r));
+  };
+  T* cq = reinterpret_cast<T*>(a.cq) + row * a.ldcq;
+  T* cr = reinterpret_cast<T*>(a.cache) + ((int64_t)page * PAGE_TOKENS + (ok ? pos % PAGE_TOKENS : 0)) * a.ldc;
+  const int half = a.m.rope_dims / 2;
+#pragma unroll
+  for (int k = 0; k < NV; ++k) {
+    const int i = (k * 32 + ln) * 4;
+    if (i >= n) break;
+    if (i < nq) {
+      put(cq + i, normed(a.q_norm + i, v[k], rq));
+    } else if (i < nq + nc) {
+      if (ok) put(cr + i - nq, normed(a.kv_norm + i - nq, v[k], rc));
+    } else if (i < nq + nc + nr) {
+      const int f = i - nq - nc;
+      float4 y = v[k];
+      const float2* cs = a.m.rope + (int64_t)(ok ? pos : 0) * half + f / 2;
+      if (f < 2 * half) {
+        const float2 t = rotate(make_float2(y.x, y.y), cs[0]);
+        y.x = t.x;
+        y.y = t.y;
+      }
+      if (f + 2 < 2 * half) {
+        const float2 t = rotate(make_float2(y.z, y.w), cs[1]);
+        y.z = t.x;
+        y.w = t.y;
+      }
+      if (ok) put(cr + nc + f, y);
+    } else {
+      const float e[4] = {v[k].x, v[k].y, v[k].z, v[k].w};
+      for (int u = 0; u < 4 && i + u < n; ++u) a.gate[row * a.m.heads + i + u - nq - nc - nr] = 1.0f / (1.0f + expf(-e[u]));
+    }
+  }
+}
+
 // ------------------------------------------------------------------ plain kernels (f32 models, and shapes the
 // tensor-core kernels do not take): one CTA per (row of a tile, head)
 
@@ -812,6 +894,15 @@ int latent_post_launch(Ctx* c, const LatentPostArgs& a, int64_t rows) {
   const size_t smem = (size_t)a.ld * sizeof(float);
   RB_REQUIRE(a.ld % 4 == 0 && smem <= 48 * 1024, "latent attention: the input projection is wider than 12288 columns");
   const bool small = rows <= 256;
+  const int nv = (int)((a.ld + 127) / 128);
+  if (rows >= 1024 && nv <= 20 && a.m.q_rank % 4 == 0 && a.m.kv_rank % 4 == 0 && a.m.rot_dim % 4 == 0) {
+    auto go = [&](auto kernel) { return launch_k(kernel, dim3((unsigned)((rows + 7) / 8)), dim3(256), 0, c->stream, c->use_pdl, a, rows); };
+#define RB_LPOST(T) (nv <= 5 ? go(latent_post_rows_kernel<T, 5>) : nv <= 10 ? go(latent_post_rows_kernel<T, 10>) : nv <= 16 ? go(latent_post_rows_kernel<T, 16>) : go(latent_post_rows_kernel<T, 20>))
+    RB_CUDA(a.dtype == REWB200_BF16 ? RB_LPOST(bf16) : RB_LPOST(float));
+#undef RB_LPOST
+    ++g_launch_total;
+    return REWB200_OK;
+  }
   const dim3 grid((unsigned)rows), block(small ? (unsigned)std::min<int64_t>(768, std::max<int64_t>(64, (a.ld / 4 + 31) / 32 * 32)) : 128);
   cudaError_t e;
   if (a.dtype == REWB200_BF16)

@@ -351,6 +351,48 @@ def test_rotation_at_far_positions(rb, dtype):
     close(np.concatenate(got), want, dtype)
 
 
+def mixed_attention(T, spec, t, p, h, kv):
+    """Attention with every option of the layered one: convolution, norms, temperature, rotation, values of their own, a
+    learned sink and a gate per head, keys and values of another layer (kv)"""
+    from oracle import girulorn as GG
+    H, N, D, V = spec.heads, spec.kv_heads, spec.dim, spec.vdim
+    w = lambda n: t[p + "mix." + n].astype(np.float64)
+    turn = lambda x: G.rotated_halves(x, np.arange(T), spec.rope_base, spec.rope_dims)
+    q = GG.rms_norm(G.short_conv(h @ w("q"), w("q.conv")).reshape(T, H, D), w("q.norm"), 1e-5)
+    q = turn(q * GG.query_temperature(range(T), dict(coef=spec.temp_coef, every=spec.temp_every))[:, None, None])
+    if kv is None:
+        kv = (turn(GG.rms_norm(G.short_conv(h @ w("k"), w("k.conv")).reshape(T, N, D), w("k.norm"), 1e-5)), (h @ w("v")).reshape(T, N, V))
+    gate = G.sigmoid(h @ w("g"))
+    out = np.stack([G.sink_softmax(q[:, a] @ kv[0][:, a // (H // N)].T * spec.scale, G.visible(T), w("sink")[a]) @ kv[1][:, a // (H // N)] * gate[:, a:a + 1]
+                    for a in range(H)], 1)
+    return out.reshape(T, H * V) @ w("o"), kv
+
+
+@pytest.mark.parametrize("dim,vdim,taps,rope", [(24, 40, 3, 16), (16, 16, 4, 12), (40, 24, 6, 40), (136, 64, 2, 64)])
+def test_convolution_norms_temperature_rotation_and_values_together(rb, dtype, dim, vdim, taps, rope):
+    from rew_b200 import models
+    from rew_b200.layered import LayeredConfig, LayerSpec
+    from rew_b200.weights import bf16_round
+    base = dict(mixer="attention", heads=4, kv_heads=2, dim=dim, vdim=vdim, scale=dim ** -0.5, conv_taps=taps, rope_base=90.0, rope_dims=rope, qk_norm=True,
+                sink=True, out_gate=True, temp_every=7, temp_coef=0.3, ff="none")
+    cfg = LayeredConfig(vocab=72, d_model=64, layers=[LayerSpec(**base), LayerSpec(kv_from=0, **base)], eps=1e-5, norm_zero_centred=False,
+                        block="parallel_one_norm", own_head=True, max_seq=640, dtype=models.DTYPES[dtype])
+    rng = np.random.default_rng(dim)
+    t = {n: bf16_round(rng.normal(1.0 if n.endswith("norm") or n.endswith("norm1") else 0.0, 0.2 if "norm" in n else 1.2 if n.endswith("conv") or n == "embed"
+                                  else shape[0] ** -0.5, size=shape).astype(np.float32)) for n, shape in cfg.tensor_specs()}
+    ids = rng.integers(0, 72, size=600).astype(np.int32)
+    f = {k: v.astype(np.float64) for k, v in t.items()}
+    x, kv = f["embed"][ids], None
+    for i, spec in enumerate(cfg.layers):
+        y, kv = mixed_attention(600, spec, t, "l%d." % i, G.rms_norm(x, f["l%d.norm1" % i], 1e-5), kv)
+        x = x + y
+    want = G.rms_norm(x, f["final.norm"], 1e-5) @ f["head"]
+    sess = rb.CausalLM(cfg).load([t[n] for n, _ in cfg.tensor_specs()]).paged_session(1, 640, 11)
+    for cuts in ([600], [520, 1, 2, 70, 1], [3, 597]):
+        close(feed_all(sess, 0, ids, cuts), want, dtype)
+        sess.release(0)
+
+
 def test_long_decoding(rb, dtype):
     cfg = K.config([K.attention(K.moe()), K.latent(K.moe(), window=80), K.latent(None, window=120, kv_from=1)])
     t = K.weights(cfg, seed=8, score_gain=1.5)

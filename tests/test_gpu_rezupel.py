@@ -387,6 +387,19 @@ def test_bf16_decode_step_matches_the_fed_step(rb):
     assert err(lg[-1:], logits) < 1e-2
 
 
+@pytest.mark.parametrize("rope_dims,heads", [(12, 3), (6, 5), (0, 4)])
+def test_hundreds_of_sequences_in_one_step(rb, dtype, rope_dims, heads):
+    """Large steps of short portions: rotated pairs whole and in part, gates of any number of heads."""
+    cfg = K.config([K.layer(K.dense(), heads=heads, rope_dims=rope_dims), K.layer(None, heads=2, window=9)])
+    t = K.weights(cfg, seed=21, score_gain=2.0)
+    s = build(rb, cfg, t, dtype, max_seq=64).session(260, 64)
+    ids = np.stack([K.tokens(cfg, 11, seed=i) for i in range(260)])
+    some = [0, 1, 7, 128, 255, 259]
+    for lo, hi in ((0, 5), (5, 11)):
+        _, logits = s.forward(ids[:, lo:hi], want_logits=True)
+        close(logits[some], np.stack([R.forward(cfg, t, ids[i, :hi])[-1] for i in some]), dtype)
+
+
 def test_forward_all_and_chunked_session_forward(rb, dtype):
     cfg = K.small()
     t = K.weights(cfg, seed=12)
