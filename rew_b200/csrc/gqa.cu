@@ -70,9 +70,11 @@ constexpr int CONV_REG_TAPS = 4;   // convolutions up to this long run on regist
 
 // One warp per head: query heads, key heads, value heads (none where the values are the keys: a key warp writes both), then
 // one warp for all gates; RW rows each, requested together.  A lane holds four columns at a time, PC of them (dim and vdim up
-// to 128 PC).  TIME: the head has a convolution, rotated features or values that are its keys.
+// to 128 PC).  TIME: the head has a convolution, rotated features or values that are its keys (one row a warp; large steps:
+// gqa_post_rows_kernel).
 template <typename T, int PC, int RW, bool TIME>
 __global__ void __launch_bounds__(256) gqa_post_kernel(GqaPostArgs a, int64_t rows) {
+  static_assert(!TIME || RW == 1, "one row a warp");
   constexpr int HIST = TIME ? CONV_REG_TAPS - 1 : 0, BACK = TIME ? CONV_REG_TAPS : 1;
   constexpr unsigned ALL = 0xffffffffu;
   __shared__ __align__(16) float s_rot[TIME ? 8 : 1][TIME ? PC * 128 : 4];
@@ -124,9 +126,9 @@ __global__ void __launch_bounds__(256) gqa_post_kernel(GqaPostArgs a, int64_t ro
     const int pl = __shfl_up_sync(ALL, my_lane, 1), pp = __shfl_up_sync(ALL, my_pos, 1);
     cont = __ballot_sync(ALL, a.map.row_lane && ln > 0 && my_lane >= 0 && pl == my_lane && pp == my_pos - 1);
   }
-  auto ahead_of = [&](int r) { return min(__clz(~(cont << (31 - HIST - r))), HIST); };   // rows of the portion ahead of row r, at most HIST
+  auto ahead_of = [&](int r) { return min(__clz(~(cont << (31 - HIST - r))), HIST); };   // rows of its portion ahead of row r in this step, at most HIST
   auto state_at = [&](int lane, int pos) -> float* { return a.state + ((int64_t)lane * (a.m.taps - 1) + pos % (a.m.taps - 1)) * C + col; };
-  float4 t0 = make_float4(0.f, 0.f, 0.f, 0.f), t1 = t0;   // (cos, sin) of this lane's four features (RW == 1)
+  float4 t0 = make_float4(0.f, 0.f, 0.f, 0.f), t1 = t0;   // (cos, sin) of this lane's four features
   const bool rot_reg = PC == 1 && half > 0 && half % 4 == 0;
   auto rope_row = [&](int pos) { return a.m.rope + (int64_t)(ok_at(pos) ? pos : 0) * half; };
   auto rope_load = [&](int pos) {
@@ -136,7 +138,7 @@ __global__ void __launch_bounds__(256) gqa_post_kernel(GqaPostArgs a, int64_t ro
     t0 = *reinterpret_cast<const float4*>(cs);
     t1 = *reinterpret_cast<const float4*>(cs + 2);
   };
-  if constexpr (TIME && RW == 1) {
+  if constexpr (TIME) {
     const int pos = pos_of(0);
     const int lane = __shfl_sync(ALL, my_lane, HIST);
     if (conv_reg && !a.map.row_lane)
@@ -198,8 +200,8 @@ __global__ void __launch_bounds__(256) gqa_post_kernel(GqaPostArgs a, int64_t ro
   }
   if constexpr (TIME) {
     if (conv_reg) {
-      if (RW > 1 || a.map.row_lane) {
-        const int ahead = ahead_of(0);   // rows of the step ahead of the first one here
+      if (a.map.row_lane) {
+        const int ahead = ahead_of(0);
 #pragma unroll
         for (int b = 1; b < BACK; ++b)
 #pragma unroll
@@ -209,47 +211,37 @@ __global__ void __launch_bounds__(256) gqa_post_kernel(GqaPostArgs a, int64_t ro
             for (int s = 0; s < a.nsplit; ++s) add4(past[b][c], *reinterpret_cast<const float4*>(p + s * a.split_stride - b * a.ld + col + i));
           }
       }
+      const int pos = pos_of(0), lane = __shfl_sync(ALL, my_lane, HIST);
+      const int given = a.map.row_lane ? ahead_of(0) : HIST;   // values at hand; older ones are the state's
 #pragma unroll
-      for (int r = RW - 1; r >= 0; --r) {     // backwards: the values ahead of a row are still the projected ones
-        const int pos = pos_of(r), lane = __shfl_sync(ALL, my_lane, min(r, nr - 1) + HIST);
-        const int given = RW == 1 && !a.map.row_lane ? HIST : ahead_of(r);   // values at hand; older ones are the state's
+      for (int c = 0; c < PC; ++c) {
+        const int i = (c * 32 + ln) * 4;
+        const float4 u = x[0][c];
+        float4 y = make_float4(cw[0][c].x * u.x, cw[0][c].y * u.y, cw[0][c].z * u.z, cw[0][c].w * u.w);
 #pragma unroll
-        for (int c = 0; c < PC; ++c) {
-          const int i = (c * 32 + ln) * 4;
-          const float4 u = x[r][c];
-          float4 y = make_float4(cw[0][c].x * u.x, cw[0][c].y * u.y, cw[0][c].z * u.z, cw[0][c].w * u.w);
-#pragma unroll
-          for (int b = 1; b < BACK; ++b) {
-            float4 h = r >= b ? x[r >= b ? r - b : 0][c] : past[r < b ? b - r : 0][c];
-            if (b > given) {
-              h = make_float4(0.f, 0.f, 0.f, 0.f);
-              if (b < a.m.taps && pos - b >= 0 && r < nr && i < n) h = *reinterpret_cast<const float4*>(state_at(lane, pos - b) + i);
-            }
-            fma4(y, cw[b][c], h);
-          }
-          x[r][c] = y;
-          if (!a.tails && a.m.taps > 1 && r < nr && i < n && ok_at(pos)) *reinterpret_cast<float4*>(state_at(lane, pos) + i) = u;
+        for (int b = 1; b < BACK; ++b) {
+          float4 h = past[b][c];
+          if (b > given && b < a.m.taps && pos - b >= 0 && i < n) h = *reinterpret_cast<const float4*>(state_at(lane, pos - b) + i);
+          fma4(y, cw[b][c], h);
         }
+        x[0][c] = y;
+        if (!a.tails && a.m.taps > 1 && i < n && ok_at(pos)) *reinterpret_cast<float4*>(state_at(lane, pos) + i) = u;
       }
     } else if (conv) {
+      const int pos = pos_of(0), lane = __shfl_sync(ALL, my_lane, HIST), ahead = rows_ahead(a, row0, pos);
 #pragma unroll
-      for (int r = 0; r < RW; ++r) {
-        if (r >= nr) break;
-        const int pos = pos_of(r), lane = __shfl_sync(ALL, my_lane, r + HIST), ahead = rows_ahead(a, row0 + r, pos);
-#pragma unroll
-        for (int c = 0; c < PC; ++c) {
-          const int i = (c * 32 + ln) * 4;
-          const float4 u = x[r][c];
-          float4 y = make_float4(0.f, 0.f, 0.f, 0.f);
-          for (int b = 0; b < a.m.taps; ++b) {
-            const float4 w = slab4(a.m.conv + (a.m.taps - 1 - b) * C + col, 1, 0, i, n);
-            if (b == 0) fma4(y, w, u);
-            else if (b <= ahead) fma4(y, w, slab4(a, p + (r - b) * a.ld + col, i, n));
-            else if (pos - b >= 0) fma4(y, w, slab4(state_at(lane, pos - b), 1, 0, i, n));
-          }
-          x[r][c] = y;
-          if (!a.tails && a.m.taps > 1 && ok_at(pos)) put4<float>(state_at(lane, pos), i, n, u);
+      for (int c = 0; c < PC; ++c) {
+        const int i = (c * 32 + ln) * 4;
+        const float4 u = x[0][c];
+        float4 y = make_float4(0.f, 0.f, 0.f, 0.f);
+        for (int b = 0; b < a.m.taps; ++b) {
+          const float4 w = slab4(a.m.conv + (a.m.taps - 1 - b) * C + col, 1, 0, i, n);
+          if (b == 0) fma4(y, w, u);
+          else if (b <= ahead) fma4(y, w, slab4(a, p - b * a.ld + col, i, n));
+          else if (pos - b >= 0) fma4(y, w, slab4(state_at(lane, pos - b), 1, 0, i, n));
         }
+        x[0][c] = y;
+        if (!a.tails && a.m.taps > 1 && ok_at(pos)) put4<float>(state_at(lane, pos), i, n, u);
       }
     }
   }
@@ -289,7 +281,6 @@ __global__ void __launch_bounds__(256) gqa_post_kernel(GqaPostArgs a, int64_t ro
     if constexpr (TIME) {
       if (rot_reg) {
         // the four features of a lane lie in one half; the other half is half / 4 lanes away
-        if (RW > 1) rope_load(pos);
         const bool lo = ln * 4 < half;
         const int from = (lo ? ln + half / 4 : ln - half / 4) & 31;
         const float sg = lo ? -1.f : 1.f;

@@ -81,14 +81,14 @@ def dense_8b(**kw):
     layers = _turns(32, dict(heads=32, kv_heads=8, dim=128, vdim=128, scale=128 ** -0.5, rope_base=500000.0, rope_dims=128),
                     dict(heads=32, dim=128, vdim=128, q_rank=1536, kv_rank=512, scale=128 ** -0.5, window=1024), ff, ff)
     return LayeredConfig(**{**dict(vocab=128256, d_model=4096, layers=layers, eps=1e-5, norm_zero_centred=False, block="parallel_one_norm",
-                                   own_head=True, logit_softcap=30.0, max_seq=2560, dtype=_lib.BF16), **kw})
+                                   own_head=True, logit_softcap=50.0, max_seq=2560, dtype=_lib.BF16), **kw})
 
 
 def moe_lite(**kw):
     """As many layers, the width, heads, experts, expert and shared expert widths of the DeepSeek-V2-Lite shape."""
     from . import _lib
-    moe = dict(ff="experts", ffn=1408, experts=64, top_k=6, renormalize=True, router_scale=2.5, expert_gated=True, shared_ffn=2816, shared_gate=True)
+    moe = dict(ff="experts", ffn=1408, experts=64, top_k=6, renormalize=True, router_scale=1.5, expert_gated=True, shared_ffn=2816, shared_gate=True)
     layers = _turns(27, dict(heads=16, kv_heads=16, dim=128, vdim=128, scale=128 ** -0.5, rope_base=10000.0, rope_dims=128),
                     dict(heads=16, dim=128, vdim=128, q_rank=768, kv_rank=512, scale=128 ** -0.5, window=1024), dict(ff="dense", ffn=10944), moe)
     return LayeredConfig(**{**dict(vocab=102400, d_model=2048, layers=layers, eps=1e-6, norm_zero_centred=False, block="parallel_one_norm",
-                                   own_head=True, logit_softcap=30.0, max_seq=1024, dtype=_lib.BF16), **kw})
+                                   own_head=True, logit_softcap=50.0, max_seq=1024, dtype=_lib.BF16), **kw})

@@ -468,7 +468,7 @@ def test_greedy_generation_follows_the_oracle(rb):
 
 def test_bf16_decode_step_matches_the_fed_step(rb):
     """The captured decode step against rewb200_lanes_feed of the same tokens: same kernels up to the launch shapes."""
-    cfg = K.small(cap=30.0)
+    cfg = K.small(cap=25.0)
     t = K.weights(cfg, seed=11, score_gain=1.5)
     model = build(rb, cfg, t, "bfloat16")
     p = K.tokens(cfg, 90, seed=11)
@@ -500,7 +500,7 @@ def test_wide_batches_of_decoding_lanes(rb):
 @pytest.mark.parametrize("conv,rot", [(3, 16), (4, 20), (7, 24), (1, 8)])
 def test_hundreds_of_sequences_in_one_step(rb, dtype, conv, rot):
     """Short portions, each starting inside a tile of rows, from the state of the step ahead; then captured decode steps."""
-    cfg = K.config([K.attention(K.dense(), conv=conv, rot=rot), K.latent(K.dense())], cap=30.0)
+    cfg = K.config([K.attention(K.dense(), conv=conv, rot=rot), K.latent(K.dense())], cap=25.0)
     t = K.weights(cfg, seed=14)
     s = build(rb, cfg, t, dtype, max_seq=64).session(516, 64)
     ids = np.stack([K.tokens(cfg, 19, seed=i) for i in range(516)])
