@@ -295,15 +295,25 @@ int rewb200_linear_noalloc(int slot, const void* x_bf16, const void* w_bf16, con
  *   3  gated linear attention: a state [dim, vdim] per head in f32 for every sequence, decayed per key channel by
  *      sigmoid(z)^(1 / tau) with z a projection through decay_rank features, RMS norm per head on the output and a
  *      SiLU gate.
- * Mixers 1 and 2 have an optional sigmoid gate per head on the output (out_gate). */
+ *   4  gated delta rule: a short convolution and SiLU on queries, keys and values, unit queries and keys of kv_heads
+ *      shared by groups of heads; per head a state S [dim, vdim] in f32 that decays by one number a token
+ *      (exp(-exp(A_log) softplus(a + dt_bias))) and is corrected towards v at the key: S += k (beta (v - S^T k))^T,
+ *      beta a sigmoid; RMS norm per head on the output and a SiLU gate.
+ *   5  linear recurrent unit: two projections of heads * dim channels; one goes through a short convolution, its
+ *      blocks of dim channels ("heads") through two square matrices whose sigmoids r, i gate the recurrence
+ *      S = a S + sqrt(1 - a^2) i u, log a = -8 r softplus(lam); the other, through a tanh GELU, scales the output.
+ * Mixers 1 and 2 have an optional sigmoid gate per head on the output (out_gate).
+ * A layer may have a second mixer beside the first (`beside`): both read the same input, their outputs are scaled
+ * by mix_scale and added. */
 typedef struct rewb200_layer {
   int32_t mixer;
   int32_t heads, dim, rot_dim, vdim, q_rank, kv_rank;
-  int32_t window;       /* mixer 1: keys a query sees, itself included; 0: all before it */
+  int32_t window;       /* mixers 1 and 2: keys a query sees, itself included; 0: all before it */
   int32_t rope_dims;    /* mixer 1: rotated features of the rot_dim part, interleaved pairs; mixer 2: rotated features at the
-                         * start of a head, feature i paired with i + rope_dims / 2 */
-  int32_t out_gate;     /* 1: every head's output is scaled by a sigmoid of its own projection of the input */
-  int32_t ff;           /* 0 none, 1 dense gated SiLU, 2 routed experts */
+                         * start of a head, feature i paired with i + rope_dims / 2, or with its neighbour (rope_pairs) */
+  int32_t out_gate;     /* 1: every head's output is scaled by a sigmoid of its own projection of the input; 2 (mixer 2):
+                         * every feature of the output by its own */
+  int32_t ff;           /* 0 none, 1 dense, 2 routed experts */
   int32_t ffn;          /* hidden width of the dense feed-forward or of one expert */
   int32_t experts, top_k;
   int32_t renormalize;  /* 1: routing weights divided by the sum of the chosen ones */
@@ -324,22 +334,40 @@ typedef struct rewb200_layer {
   float tau;
   int32_t router_bias;  /* 1: the router has a bias per expert */
   int32_t shared_ffn;   /* hidden width of a gated SiLU expert that runs for every token beside the routed ones; 0: none */
-  int32_t conv_taps;    /* mixer 2: taps of a causal convolution over time per channel of queries and keys; 0: none */
+  int32_t conv_taps;    /* mixer 2: taps of a causal convolution over time per channel of queries and keys; 0: none;
+                         * mixers 4 and 5: of theirs */
   int32_t values_from_keys; /* mixer 2: 1: the values are the keys as they leave the convolution (vdim == dim) */
   float router_scale;   /* factor of the routing weights; 0 reads as 1 */
   int32_t shared_gate;  /* 1: the shared expert's output is scaled by a sigmoid of its own projection of the input */
+  int32_t qkv_bias;     /* mixer 2: queries, keys and values have biases */
+  int32_t rope_pairs;   /* mixer 2: 1: feature 2i is rotated with 2i + 1 */
+  int32_t v_norm;       /* mixer 2: 1: values are divided by their root mean square (and cached so) */
+  int32_t keep_first;   /* mixer 2 with a window: the first keys of the sequence every query sees besides */
+  int32_t head_mix;     /* mixer 2: 1: after the softmax head h weighs keys with sum_g T[h, g] (weights of head g) */
+  int32_t ff_act;       /* dense feed-forward: 0 gated SiLU, 1 W_down gelu(W_up x) with the tanh form of gelu */
+  int32_t ff_bias;      /* dense feed-forward with ff_act 1: both projections have biases */
+  int32_t beside;       /* 1 + index of a second mixer among rewb200_stack.n_beside, 0: none */
+  float mix_scale;      /* mixers 2, 4 and 5: factor of the mixer's output; 0 reads as 1 */
 } rewb200_layer;
 typedef struct rewb200_stack {
   int32_t loop_start, loop_stop, loop_times; /* the half-open range of layers that is repeated, and how often it runs
                                               * (0: no loop).  Passes share weights and have a cache each; a pass opens by
                                               * adding its row of `step` and, from the second on, the token embeddings
-                                              * to the residual. */
+                                              * to the residual, or as loop_in says. */
   int32_t norm_zero_centred;                 /* block and final norm weights are stored as the distance from one */
   int32_t block;                             /* 0: x += mixer(norm1(x)) + ff(norm2(x));
                                               * 1: x += norm1(mixer(x)), then x += norm2(ff(x));
-                                              * 2: x += mixer(h) + ff(h), h = norm1(x) */
+                                              * 2: x += mixer(h) + ff(h), h = norm1(x);
+                                              * 3: x += norm1b(mixer(norm1(x))), then x += norm2b(ff(norm2(x))) */
   int32_t own_head;                          /* 1: the output head is a tensor of its own, 0: the embedding table */
   float logit_softcap;                       /* logits <- cap * tanh(logits / cap); 0: none */
+  float embed_scale;                         /* block 3: factor of the token embeddings; 0 reads as 1 */
+  int32_t bigram_buckets;                    /* block 3: > 0: a table [bigram_buckets + 1, d] is added to the embeddings: row
+                                              * (previous id * bigram_mul_prev + id * bigram_mul_cur) mod bigram_buckets, the
+                                              * last row for the first token of a sequence */
+  int64_t bigram_mul_prev, bigram_mul_cur;
+  int32_t loop_in;                           /* block 3: 1: every pass opens with x <- W [x; x0], x0 the embeddings */
+  int32_t n_beside;                          /* descriptions of second mixers behind those of the layers */
 } rewb200_stack;
 
 /* ---- model + generate ------------------------------------------------------
@@ -362,12 +390,16 @@ typedef struct rewb200_config {
 
 int rewb200_model_create(int slot, const rewb200_config* cfg, rewb200_model** out);
 /* A layered model: `cfg` gives vocab, d_model, n_layers, max_seq, eps and dtype (its other fields are ignored),
- * `layers` n_layers descriptions.  Canonical tensors (Linear weights [in, out], see rew_b200/layered.py): embed,
- * step [times, d] (with a loop); per layer norm1, the mixer (1: dq, dq.norm, uq, with latents of its own dkv, dkv.norm,
+ * `layers` n_layers descriptions, then those of the second mixers (of which only the mixer's fields are read).  Canonical
+ * tensors (Linear weights [in, out], see rew_b200/layered.py): embed, bigram (with buckets), step [times, d] (with a loop)
+ * or loop.in [2 d, d] (with loop_in); per layer norm1 (block 3: norm1, norm1b), the mixer (1: dq, dq.norm, uq, with latents of its own dkv, dkv.norm,
  * then uk, uv, sink (1); 2: q, then with keys and values of its own k, v (v unless they are the keys), with a convolution
- * q.conv and (own) k.conv [channels, taps], q.norm and (own) k.norm with qk_norm, rel [bias_rows, heads], sink (1);
- * 3: q, k, v, a1, a2, a2.b, g, norm), g (mixers 1 and 2 with out_gate), o, then with a feed-forward norm2 (blocks 0 and 1)
- * and gate, up, down (dense) or router, [router.b,] per expert [gate,] up, down and the shared expert's gate, up, down
+ * q.conv and (own) k.conv [channels, taps], q.norm and (own) k.norm with qk_norm, rel [bias_rows, heads], sink (1),
+ * talk [heads, heads] (head_mix), q.b, (own) k.b and v.b (qkv_bias); 3: q, k, v, a1, a2, a2.b, g, norm; 4: q, k, v, q.conv,
+ * k.conv, v.conv [channels, taps], b, a, A_log, dt_bias, g, norm; 5: y, y.b, x, x.b, conv, conv.b, ra and ri
+ * [heads, dim, dim] as [heads * dim, dim] (out, in), ra.b, ri.b, lam), g (mixers 1 and 2 with out_gate), o, the same for a
+ * second mixer, then with a feed-forward norm2 (blocks 0, 1 and 3; 3: norm2b) and gate, up, down (dense; ff_act 1: up, up.b,
+ * down, down.b without gate) or router, [router.b,] per expert [gate,] up, down and the shared expert's gate, up, down
  * [, sg]; final norm; head [d, vocab] (with own_head). */
 int rewb200_model_create_layers(int slot, const rewb200_config* cfg, const rewb200_layer* layers, const rewb200_stack* stack,
                                 rewb200_model** out);

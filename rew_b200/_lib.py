@@ -37,13 +37,16 @@ class Layer(C.Structure):
         ("rope_base", C.c_double), ("scale", C.c_float)] + [
         (n, C.c_int32) for n in ("kv_heads", "kv_from", "qk_norm", "sink", "bias_rows", "bias_max", "temp_every")] + [
         ("temp_coef", C.c_float), ("decay_rank", C.c_int32), ("tau", C.c_float), ("router_bias", C.c_int32), ("shared_ffn", C.c_int32),
-        ("conv_taps", C.c_int32), ("values_from_keys", C.c_int32), ("router_scale", C.c_float), ("shared_gate", C.c_int32)]
+        ("conv_taps", C.c_int32), ("values_from_keys", C.c_int32), ("router_scale", C.c_float)] + [
+        (n, C.c_int32) for n in ("shared_gate", "qkv_bias", "rope_pairs", "v_norm", "keep_first", "head_mix", "ff_act", "ff_bias", "beside")] + [
+        ("mix_scale", C.c_float)]
 
 
 class Stack(C.Structure):
     """struct rewb200_stack"""
     _fields_ = [(n, C.c_int32) for n in ("loop_start", "loop_stop", "loop_times", "norm_zero_centred", "block", "own_head")] + [
-        ("logit_softcap", C.c_float)]
+        ("logit_softcap", C.c_float), ("embed_scale", C.c_float), ("bigram_buckets", C.c_int32), ("bigram_mul_prev", C.c_int64),
+        ("bigram_mul_cur", C.c_int64), ("loop_in", C.c_int32), ("n_beside", C.c_int32)]
 
 
 _lib = None

@@ -6,7 +6,9 @@
 // slabs to the residual, adds what a loop adds ahead of a pass, and leaves both norms of the next layer run, and in small
 // steps the feed-forward branch runs on the slot's second stream beside the mixer; or x += norm1(mixer(x)), then
 // x += norm2(ff(x)), where one launch (output_norm) per sublayer sums its slabs, norms the sum and adds it; or the parallel
-// block with one norm that both branches read.
+// block with one norm that both branches read; or x += norm1b(mixer(norm1(x))), x += norm2b(ff(norm2(x))), where the same
+// output_norm launch also leaves the next sublayer's norm, and a pass of a loop may open with a Linear over the stream and
+// the embeddings side by side.
 //
 // Device layouts beyond engine.cu's: rows and Linear outputs are padded to multiples of 8 elements (zero weights, zero
 // norm weights), so any width can be loaded by TMA; a mixer's input projections are one matrix; the key and value
@@ -25,49 +27,79 @@ int64_t pad8(int64_t v) { return (v + 7) / 8 * 8; }
 enum Slot : int {
   SL_NORM1, SL_DQ, SL_DQ_NORM, SL_UQ, SL_DKV, SL_DKV_NORM, SL_UK, SL_UV, SL_G, SL_O, SL_NORM2, SL_GATE, SL_UP, SL_DOWN, SL_ROUTER,
   SL_E_GATE, SL_E_UP, SL_E_DOWN, SL_EMBED, SL_STEP, SL_FINAL, SL_HEAD, SL_Q, SL_K, SL_V, SL_Q_NORM, SL_K_NORM, SL_REL, SL_SINK, SL_A1, SL_A2,
-  SL_A2_B, SL_V_GATE, SL_V_NORM, SL_ROUTER_B, SL_S_GATE, SL_S_UP, SL_S_DOWN, SL_Q_CONV, SL_K_CONV, SL_S_SG
+  SL_A2_B, SL_V_GATE, SL_V_NORM, SL_ROUTER_B, SL_S_GATE, SL_S_UP, SL_S_DOWN, SL_Q_CONV, SL_K_CONV, SL_S_SG,
+  SL_BIGRAM, SL_LOOP_IN, SL_BACK1, SL_BACK2, SL_UP_B, SL_DOWN_B, SL_TALK, SL_Q_B, SL_K_B, SL_V_B, SL_V_CONV, SL_BETA, SL_ALPHA, SL_RATE, SL_DT_BIAS,
+  SL_Y, SL_Y_B, SL_X, SL_X_B, SL_CONV, SL_CONV_B, SL_RA, SL_RI, SL_RA_B, SL_RI_B, SL_LAM
 };
-enum Block : int { BLOCK_PARALLEL = 0, BLOCK_OUTPUT_NORM = 1, BLOCK_ONE_NORM = 2 };
+enum Block : int { BLOCK_PARALLEL = 0, BLOCK_OUTPUT_NORM = 1, BLOCK_ONE_NORM = 2, BLOCK_SANDWICH = 3 };
 enum Sink : int { SINK_NONE = 0, SINK_LEARNED = 1, SINK_ONE = 2 };
-enum Mixer : int { MIX_LATENT = 1, MIX_GQA = 2, MIX_GLA = 3 };
+enum Mixer : int { MIX_LATENT = 1, MIX_GQA = 2, MIX_GLA = 3, MIX_DELTA = 4, MIX_LRU = 5 };
 struct TensorAt {
   Slot slot;
   int layer, expert;
+  bool second = false;   // of the layer's second mixer
 };
+// The description of a layer's first or second mixer.
+const rewb200_layer& mixer_spec(const rewb200_model* m, int layer, bool second) {
+  return second ? m->spec[m->cfg.n_layers + m->spec[layer].beside - 1] : m->spec[layer];
+}
+bool has_loop_in(const rewb200_model* m) { return m->stack.loop_times > 0 && m->stack.loop_in; }
 
 // The canonical tensors of a layered model (rew_b200/layered.py lists the same).
 void tensors_of(const rewb200_model* m, std::vector<TensorAt>* out) {
   out->push_back({SL_EMBED, -1, -1});
-  if (m->stack.loop_times > 0) out->push_back({SL_STEP, -1, -1});
+  if (m->stack.bigram_buckets > 0) out->push_back({SL_BIGRAM, -1, -1});
+  if (m->stack.loop_times > 0) out->push_back({has_loop_in(m) ? SL_LOOP_IN : SL_STEP, -1, -1});
+  const bool sandwich = m->stack.block == BLOCK_SANDWICH;
   for (int l = 0; l < m->cfg.n_layers; ++l) {
     const rewb200_layer& L = m->spec[l];
     auto add = [&](std::initializer_list<Slot> slots) {
       for (Slot s : slots) out->push_back({s, l, -1});
     };
     add({SL_NORM1});
-    const bool own = L.kv_from < 0;
-    if (L.mixer == MIX_LATENT) {
-      add({SL_DQ, SL_DQ_NORM, SL_UQ});
-      if (own) add({SL_DKV, SL_DKV_NORM});
-      add({SL_UK, SL_UV});
-      if (L.sink == SINK_LEARNED) add({SL_SINK});
+    if (sandwich) add({SL_BACK1});
+    for (int k = 0; k < (L.beside ? 2 : 1); ++k) {
+      const rewb200_layer& M = mixer_spec(m, l, k == 1);
+      auto add = [&](std::initializer_list<Slot> slots) {
+        for (Slot s : slots) out->push_back({s, l, -1, k == 1});
+      };
+      const bool own = M.kv_from < 0;
+      if (M.mixer == MIX_LATENT) {
+        add({SL_DQ, SL_DQ_NORM, SL_UQ});
+        if (own) add({SL_DKV, SL_DKV_NORM});
+        add({SL_UK, SL_UV});
+        if (M.sink == SINK_LEARNED) add({SL_SINK});
+      }
+      if (M.mixer == MIX_GQA) {
+        add({SL_Q});
+        if (own) add({SL_K});
+        if (own && !M.values_from_keys) add({SL_V});
+        if (M.conv_taps > 0) add({SL_Q_CONV});
+        if (M.conv_taps > 0 && own) add({SL_K_CONV});
+        if (M.qk_norm) add({SL_Q_NORM});
+        if (M.qk_norm && own) add({SL_K_NORM});
+        if (M.bias_rows > 0) add({SL_REL});
+        if (M.sink == SINK_LEARNED) add({SL_SINK});
+        if (M.head_mix) add({SL_TALK});
+        if (M.qkv_bias) add({SL_Q_B});
+        if (M.qkv_bias && own) add({SL_K_B});
+        if (M.qkv_bias && own && !M.values_from_keys) add({SL_V_B});
+      }
+      if (M.mixer == MIX_GLA) add({SL_Q, SL_K, SL_V, SL_A1, SL_A2, SL_A2_B, SL_V_GATE, SL_V_NORM});
+      if (M.mixer == MIX_DELTA)
+        add({SL_Q, SL_K, SL_V, SL_Q_CONV, SL_K_CONV, SL_V_CONV, SL_BETA, SL_ALPHA, SL_RATE, SL_DT_BIAS, SL_V_GATE, SL_V_NORM});
+      if (M.mixer == MIX_LRU) add({SL_Y, SL_Y_B, SL_X, SL_X_B, SL_CONV, SL_CONV_B, SL_RA, SL_RI, SL_RA_B, SL_RI_B, SL_LAM});
+      if (M.out_gate) add({SL_G});
+      add({SL_O});
     }
-    if (L.mixer == MIX_GQA) {
-      add({SL_Q});
-      if (own) add({SL_K});
-      if (own && !L.values_from_keys) add({SL_V});
-      if (L.conv_taps > 0) add({SL_Q_CONV});
-      if (L.conv_taps > 0 && own) add({SL_K_CONV});
-      if (L.qk_norm) add({SL_Q_NORM});
-      if (L.qk_norm && own) add({SL_K_NORM});
-      if (L.bias_rows > 0) add({SL_REL});
-      if (L.sink == SINK_LEARNED) add({SL_SINK});
-    }
-    if (L.mixer == MIX_GLA) add({SL_Q, SL_K, SL_V, SL_A1, SL_A2, SL_A2_B, SL_V_GATE, SL_V_NORM});
-    if (L.out_gate) out->push_back({SL_G, l, -1});
-    out->push_back({SL_O, l, -1});
     if (L.ff && m->stack.block != BLOCK_ONE_NORM) out->push_back({SL_NORM2, l, -1});
-    if (L.ff == 1)
+    if (L.ff && sandwich) add({SL_BACK2});
+    if (L.ff == 1 && L.ff_act == 1) {
+      add({SL_UP});
+      if (L.ff_bias) add({SL_UP_B});
+      add({SL_DOWN});
+      if (L.ff_bias) add({SL_DOWN_B});
+    } else if (L.ff == 1)
       for (Slot s : {SL_GATE, SL_UP, SL_DOWN}) out->push_back({s, l, -1});
     if (L.ff == 2) {
       add({SL_ROUTER});
@@ -87,14 +119,17 @@ void tensors_of(const rewb200_model* m, std::vector<TensorAt>* out) {
 
 int shape_of(const rewb200_model* m, const TensorAt& t, int64_t* rows, int64_t* cols, bool* vec) {
   const int64_t d = m->cfg.d_model;
-  const rewb200_layer* L = t.layer >= 0 ? &m->spec[t.layer] : nullptr;
+  const rewb200_layer* L = t.layer >= 0 ? &mixer_spec(m, t.layer, t.second) : nullptr;
+  const bool grouped = L && (L->mixer == MIX_GQA || L->mixer == MIX_DELTA);   // kv_heads of keys
   *vec = false;
   auto mat = [&](int64_t r, int64_t c) { *rows = r; *cols = c; };
   auto v = [&](int64_t n) { *rows = 1; *cols = n; *vec = true; };
   switch (t.slot) {
     case SL_EMBED: mat(m->cfg.vocab, d); break;
     case SL_STEP: mat(m->stack.loop_times, d); break;
-    case SL_FINAL: case SL_NORM1: case SL_NORM2: v(d); break;
+    case SL_BIGRAM: mat(m->stack.bigram_buckets + 1, d); break;
+    case SL_LOOP_IN: mat(2 * d, d); break;
+    case SL_FINAL: case SL_NORM1: case SL_NORM2: case SL_BACK1: case SL_BACK2: v(d); break;
     case SL_DQ: mat(d, L->q_rank); break;
     case SL_DQ_NORM: v(L->q_rank); break;
     case SL_UQ: mat(L->q_rank, (int64_t)L->heads * (L->dim + L->rot_dim)); break;
@@ -102,7 +137,7 @@ int shape_of(const rewb200_model* m, const TensorAt& t, int64_t* rows, int64_t* 
     case SL_DKV_NORM: v(L->kv_rank); break;
     case SL_UK: mat(L->kv_rank, (int64_t)L->heads * L->dim); break;
     case SL_UV: mat(L->kv_rank, (int64_t)L->heads * L->vdim); break;
-    case SL_G: mat(d, L->heads); break;
+    case SL_G: mat(d, L->out_gate == 2 ? (int64_t)L->heads * L->vdim : L->heads); break;
     case SL_O: mat((int64_t)L->heads * L->vdim, d); break;
     case SL_GATE: case SL_UP: case SL_E_GATE: case SL_E_UP: mat(d, L->ffn); break;
     case SL_DOWN: case SL_E_DOWN: mat(L->ffn, d); break;
@@ -111,8 +146,8 @@ int shape_of(const rewb200_model* m, const TensorAt& t, int64_t* rows, int64_t* 
     case SL_S_GATE: case SL_S_UP: mat(d, L->shared_ffn); break;
     case SL_S_DOWN: mat(L->shared_ffn, d); break;
     case SL_HEAD: mat(d, m->cfg.vocab); break;
-    case SL_Q: mat(d, (int64_t)L->heads * L->dim); break;
-    case SL_K: mat(d, (int64_t)(L->mixer == MIX_GQA ? L->kv_heads : L->heads) * L->dim); break;
+    case SL_Q: mat(d, (int64_t)(L->mixer == MIX_DELTA ? L->kv_heads : L->heads) * L->dim); break;
+    case SL_K: mat(d, (int64_t)(grouped ? L->kv_heads : L->heads) * L->dim); break;
     case SL_V: mat(d, (int64_t)(L->mixer == MIX_GQA ? L->kv_heads : L->heads) * L->vdim); break;
     case SL_Q_NORM: case SL_K_NORM: v(L->dim); break;
     case SL_REL: mat(L->bias_rows, L->heads); break;
@@ -122,7 +157,19 @@ int shape_of(const rewb200_model* m, const TensorAt& t, int64_t* rows, int64_t* 
     case SL_A2_B: v((int64_t)L->heads * L->dim); break;
     case SL_V_GATE: mat(d, (int64_t)L->heads * L->vdim); break;
     case SL_V_NORM: v(L->vdim); break;
-    case SL_Q_CONV: mat((int64_t)L->heads * L->dim, L->conv_taps); break;
+    case SL_Q_CONV: mat((int64_t)(L->mixer == MIX_DELTA ? L->kv_heads : L->heads) * L->dim, L->conv_taps); break;
+    case SL_V_CONV: mat((int64_t)L->heads * L->vdim, L->conv_taps); break;
+    case SL_UP_B: v(L->ffn); break;
+    case SL_DOWN_B: v(d); break;
+    case SL_TALK: mat(L->heads, L->heads); break;
+    case SL_Q_B: case SL_Y_B: case SL_X_B: case SL_CONV_B: case SL_RA_B: case SL_RI_B: case SL_LAM: v((int64_t)L->heads * L->dim); break;
+    case SL_K_B: v((int64_t)L->kv_heads * L->dim); break;
+    case SL_V_B: v((int64_t)L->kv_heads * L->vdim); break;
+    case SL_BETA: case SL_ALPHA: mat(d, L->heads); break;
+    case SL_RATE: case SL_DT_BIAS: v(L->heads); break;
+    case SL_Y: case SL_X: mat(d, (int64_t)L->heads * L->dim); break;
+    case SL_CONV: mat((int64_t)L->heads * L->dim, L->conv_taps); break;
+    case SL_RA: case SL_RI: mat((int64_t)L->heads * L->dim, L->dim); break;
     case SL_K_CONV: mat((int64_t)L->kv_heads * L->dim, L->conv_taps); break;
     case SL_S_SG: mat(d, 1); break;
   }
@@ -203,23 +250,27 @@ int upload_bias(rewb200_model* m, const rewb200_layer& L, GqaDev& G, const float
   return REWB200_OK;
 }
 
-// Convolution weights [taps][channels] from the stored [channels][taps] of queries or keys, whose first channel is c0.
-int upload_conv(rewb200_model* m, const GqaDev& G, int64_t c0, int64_t channels, const float* host) {
-  std::vector<float> t((size_t)G.m.taps * channels);
+// Convolution weights [taps][all] from the stored [channels][taps] of the channels from c0 on.
+int upload_conv(rewb200_model* m, float* w, int taps, int64_t all, int64_t c0, int64_t channels, const float* host) {
+  std::vector<float> t((size_t)taps * channels);
   for (int64_t ch = 0; ch < channels; ++ch)
-    for (int j = 0; j < G.m.taps; ++j) t[(size_t)j * channels + ch] = host[ch * G.m.taps + j];
-  RB_CUDA(cudaMemcpy2DAsync(G.conv + c0, gqa_channels(G.m) * sizeof(float), t.data(), channels * sizeof(float), channels * sizeof(float), G.m.taps,
-                            cudaMemcpyHostToDevice, m->c->stream));
+    for (int j = 0; j < taps; ++j) t[(size_t)j * channels + ch] = host[ch * taps + j];
+  RB_CUDA(cudaMemcpy2DAsync(w + c0, all * sizeof(float), t.data(), channels * sizeof(float), channels * sizeof(float), taps, cudaMemcpyHostToDevice,
+                            m->c->stream));
   RB_CUDA(cudaStreamSynchronize(m->c->stream));
   return REWB200_OK;
 }
 
 // The Linear weights of a layer's mixer that are no routed experts (all of them padded matrices of the model dtype).
+// The input projection of a layer's mixers; a second mixer's columns follow the first one's.
+LinW& in_of(LayerDev& D) {
+  return D.mixer == MIX_LATENT ? D.a.in : D.mixer == MIX_GQA ? D.g.in : D.mixer == MIX_GLA ? D.l.in : D.mixer == MIX_DELTA ? D.d.in : D.r.in;
+}
 std::vector<LinW*> mixer_linears(LayerDev& D) {
   if (D.mixer == MIX_LATENT) return {&D.a.in, &D.a.uq, &D.a.ukv, &D.o};
-  if (D.mixer == MIX_GQA) return {&D.g.in, &D.o};
-  return {&D.l.in, &D.o};
+  return {&in_of(D), &D.o};
 }
+bool has(const LayerDev& D, int mixer) { return D.mixer == mixer || D.beside == mixer; }
 bool has_dense(const LayerDev& D) { return D.ffn_local > 0; }
 
 }  // namespace
@@ -228,40 +279,71 @@ int layered_create(rewb200_model* m, const rewb200_layer* layers, const rewb200_
   const int n = m->cfg.n_layers;
   const size_t es = dtype_size(m->cfg.dtype);
   m->layered = true;
-  m->spec.assign(layers, layers + n);
+  RB_REQUIRE(stack->n_beside >= 0 && stack->n_beside <= n, "layered model: at most one second mixer a layer");
+  m->spec.assign(layers, layers + n + stack->n_beside);
   m->stack = *stack;
   const rewb200_stack& st = m->stack;
   RB_REQUIRE(st.loop_times >= 0 && (st.loop_times == 0 || (st.loop_start >= 0 && st.loop_start < st.loop_stop && st.loop_stop <= n)),
              "layered model: the loop must cover layers start .. stop - 1 of the stack");
-  RB_REQUIRE(st.block >= BLOCK_PARALLEL && st.block <= BLOCK_ONE_NORM, "layered model: unknown block");
+  RB_REQUIRE(st.block >= BLOCK_PARALLEL && st.block <= BLOCK_SANDWICH, "layered model: unknown block");
+  RB_REQUIRE(st.block == BLOCK_SANDWICH || ((st.embed_scale == 0.f || st.embed_scale == 1.f) && st.bigram_buckets == 0 && !st.loop_in),
+             "layered model: scaled embeddings, bigram tables and a Linear ahead of a pass belong to blocks normed on both sides");
+  RB_REQUIRE(st.block != BLOCK_SANDWICH || st.loop_times == 0 || st.loop_in, "layered model: a loop of blocks normed on both sides opens with a Linear");
+  RB_REQUIRE(st.bigram_buckets >= 0, "layered model: the bigram table must not have a negative size");
   RB_REQUIRE(st.block != BLOCK_OUTPUT_NORM || st.loop_times == 0, "layered model: blocks normed on the way back run without a loop");
   RB_REQUIRE(st.logit_softcap >= 0.f, "layered model: the cap of the logits must not be negative");
+  std::vector<char> taken(st.n_beside, 0);
+  for (int l = 0; l < n; ++l)
+    for (int k = 0; k < (m->spec[l].beside ? 2 : 1); ++k) {
+      const std::string who = "layer " + std::to_string(l) + ": ";
+      if (k == 1) {
+        const int b = m->spec[l].beside;
+        RB_REQUIRE(b > 0 && b <= st.n_beside && !taken[b - 1], who + "no such second mixer");
+        taken[b - 1] = 1;
+        const int first = m->spec[l].mixer, second = m->spec[n + b - 1].mixer;
+        RB_REQUIRE((second == MIX_DELTA || second == MIX_LRU) && first != second && first != MIX_LATENT, who + "these mixers do not stand beside one another");
+      }
+      const rewb200_layer& L = mixer_spec(m, l, k == 1);
+      RB_REQUIRE(L.mixer >= MIX_LATENT && L.mixer <= MIX_LRU, who + "unknown mixer");
+      RB_REQUIRE(L.heads > 0 && L.dim > 0 && L.vdim > 0, who + "mixer sizes must be positive");
+      RB_REQUIRE(L.sink >= SINK_NONE && L.sink <= SINK_ONE, who + "unknown sink");
+      RB_REQUIRE(L.out_gate >= 0 && L.out_gate <= (L.mixer == MIX_GQA ? 2 : L.mixer == MIX_LATENT ? 1 : 0), who + "unknown output gate");
+      RB_REQUIRE(L.mixer == MIX_GQA || (!L.values_from_keys && !L.qkv_bias && !L.rope_pairs && !L.v_norm && !L.keep_first && !L.head_mix),
+                 who + "biases, values from keys, neighbouring pairs, normed values, kept keys and mixed heads belong to grouped-query attention");
+      RB_REQUIRE(L.conv_taps >= 0 && (L.mixer == MIX_GQA || L.mixer >= MIX_DELTA || L.conv_taps == 0), who + "this mixer has no convolution");
+      RB_REQUIRE(L.mix_scale == 0.f || L.mix_scale == 1.f || L.mixer == MIX_GQA || L.mixer >= MIX_DELTA, who + "this mixer's output has no factor");
+      if (L.kv_from >= 0) {
+        RB_REQUIRE((L.mixer == MIX_LATENT || L.mixer == MIX_GQA) && L.kv_from < l, who + "kv_from must name an earlier layer");
+        const rewb200_layer& S = m->spec[L.kv_from];
+        const bool same = L.mixer == MIX_LATENT ? S.kv_rank == L.kv_rank && S.rot_dim == L.rot_dim : S.kv_heads == L.kv_heads && S.dim == L.dim && S.vdim == L.vdim;
+        RB_REQUIRE(S.mixer == L.mixer && S.kv_from < 0 && same, who + "kv_from must name a layer of the same mixer with latents, or keys and values, of its own and the same sizes");
+      }
+      if (L.mixer == MIX_LATENT) {
+        RB_REQUIRE(L.rot_dim >= 0 && L.q_rank > 0 && L.kv_rank > 0, who + "mixer sizes must be positive");
+        RB_REQUIRE(L.rope_dims >= 0 && L.rope_dims % 2 == 0 && L.rope_dims <= L.rot_dim, who + "rotated features must be pairs within rot_dim");
+        RB_REQUIRE(L.window >= 0, who + "the window must not be negative");
+      } else if (L.mixer == MIX_GQA) {
+        RB_REQUIRE(L.kv_heads > 0 && L.heads % L.kv_heads == 0, who + "heads must be divisible by kv_heads");
+        RB_REQUIRE(L.bias_rows >= 0 && (L.bias_rows == 0 || (L.bias_max > 0 && L.bias_max <= 1 << 20)), who + "the distance bias needs a positive bias_max");
+        RB_REQUIRE(L.temp_every >= 0, who + "temp_every must not be negative");
+        RB_REQUIRE(L.rope_dims >= 0 && L.rope_dims % 2 == 0 && L.rope_dims <= L.dim, who + "rotated features must be pairs within the head");
+        RB_REQUIRE(!L.values_from_keys || L.vdim == L.dim, who + "values that are the keys have their size");
+        RB_REQUIRE(!L.qkv_bias || (L.conv_taps == 0 && !L.values_from_keys), who + "biases and a convolution, or values that are keys, do not go together");
+        RB_REQUIRE(L.window >= 0 && L.keep_first >= 0 && (L.window > 0 || L.keep_first == 0), who + "kept first keys need a window");
+      } else if (L.mixer == MIX_GLA) {
+        RB_REQUIRE(L.decay_rank > 0 && L.tau > 0.f, who + "decay_rank and tau must be positive");
+      } else if (L.mixer == MIX_DELTA) {
+        RB_REQUIRE(L.kv_heads > 0 && L.heads % L.kv_heads == 0 && L.conv_taps > 0, who + "the delta rule needs a convolution and heads divisible by kv_heads");
+      } else {
+        RB_REQUIRE(L.vdim == L.dim && L.conv_taps > 0 && L.heads <= 256, who + "a linear recurrent unit needs a convolution and at most 256 blocks");
+      }
+    }
   for (int l = 0; l < n; ++l) {
     const rewb200_layer& L = m->spec[l];
     const std::string who = "layer " + std::to_string(l) + ": ";
-    RB_REQUIRE(L.mixer >= MIX_LATENT && L.mixer <= MIX_GLA, who + "unknown mixer");
-    RB_REQUIRE(L.heads > 0 && L.dim > 0 && L.vdim > 0, who + "mixer sizes must be positive");
-    RB_REQUIRE(L.sink >= SINK_NONE && L.sink <= SINK_ONE, who + "unknown sink");
-    RB_REQUIRE(L.conv_taps >= 0 && (L.mixer == MIX_GQA || (L.conv_taps == 0 && !L.values_from_keys)), who + "convolutions and values from keys belong to grouped-query attention");
-    if (L.kv_from >= 0) {
-      RB_REQUIRE(L.mixer != MIX_GLA && L.kv_from < l, who + "kv_from must name an earlier layer");
-      const rewb200_layer& S = m->spec[L.kv_from];
-      const bool same = L.mixer == MIX_LATENT ? S.kv_rank == L.kv_rank && S.rot_dim == L.rot_dim : S.kv_heads == L.kv_heads && S.dim == L.dim && S.vdim == L.vdim;
-      RB_REQUIRE(S.mixer == L.mixer && S.kv_from < 0 && same, who + "kv_from must name a layer of the same mixer with latents, or keys and values, of its own and the same sizes");
-    }
-    if (L.mixer == MIX_LATENT) {
-      RB_REQUIRE(L.rot_dim >= 0 && L.q_rank > 0 && L.kv_rank > 0, who + "mixer sizes must be positive");
-      RB_REQUIRE(L.rope_dims >= 0 && L.rope_dims % 2 == 0 && L.rope_dims <= L.rot_dim, who + "rotated features must be pairs within rot_dim");
-      RB_REQUIRE(L.window >= 0, who + "the window must not be negative");
-    } else if (L.mixer == MIX_GQA) {
-      RB_REQUIRE(L.kv_heads > 0 && L.heads % L.kv_heads == 0, who + "heads must be divisible by kv_heads");
-      RB_REQUIRE(L.bias_rows >= 0 && (L.bias_rows == 0 || (L.bias_max > 0 && L.bias_max <= 1 << 20)), who + "the distance bias needs a positive bias_max");
-      RB_REQUIRE(L.temp_every >= 0, who + "temp_every must not be negative");
-      RB_REQUIRE(L.rope_dims >= 0 && L.rope_dims % 2 == 0 && L.rope_dims <= L.dim, who + "rotated features must be pairs within the head");
-      RB_REQUIRE(!L.values_from_keys || L.vdim == L.dim, who + "values that are the keys have their size");
-    } else {
-      RB_REQUIRE(L.decay_rank > 0 && L.tau > 0.f, who + "decay_rank and tau must be positive");
-    }
+    RB_REQUIRE(L.ff_act >= 0 && L.ff_act <= 1 && (L.ff_act == 0 || L.ff == 1), who + "unknown activation");
+    RB_REQUIRE(!L.ff_bias || (L.ff_act == 1 && st.block == BLOCK_SANDWICH), who + "biases of the feed-forward belong to one without a gate in blocks normed on both sides");
+    RB_REQUIRE(st.block != BLOCK_SANDWICH || L.ff <= 1, who + "blocks normed on both sides have a dense feed-forward or none");
     RB_REQUIRE(L.ff >= 0 && L.ff <= 2 && (L.ff == 0 || L.ffn > 0), who + "unknown feed-forward");
     RB_REQUIRE(L.shared_ffn >= 0 && (L.ff == 2 || L.shared_ffn == 0), who + "a shared expert stands beside routed ones");
     RB_REQUIRE(!L.shared_gate || (L.shared_ffn > 0 && st.block != BLOCK_OUTPUT_NORM), who + "the gate of a shared expert needs one, in a parallel block");
@@ -271,7 +353,9 @@ int layered_create(rewb200_model* m, const rewb200_layer* layers, const rewb200_
   const int64_t d = m->cfg.d_model, dp = m->dp = pad8(d);
   m->vp = pad8(m->cfg.vocab);
   RB_TRY(zero_weights(m, &m->embed, (size_t)m->cfg.vocab * dp * es));
-  if (st.loop_times > 0) RB_TRY(zero_weights(m, (void**)&m->step_vec, (size_t)st.loop_times * dp * sizeof(float)));
+  if (st.bigram_buckets > 0) RB_TRY(zero_weights(m, &m->bigram, ((size_t)st.bigram_buckets + 1) * dp * es));
+  if (has_loop_in(m)) RB_TRY(zero_lin(m, &m->loop_in, 2 * dp, dp));
+  else if (st.loop_times > 0) RB_TRY(zero_weights(m, (void**)&m->step_vec, (size_t)st.loop_times * dp * sizeof(float)));
   std::map<std::pair<double, int>, float2*> tables;
   auto rope_of = [&](const rewb200_layer& L, const float2** out) -> int {
     if (L.rope_dims == 0) return REWB200_OK;
@@ -282,6 +366,32 @@ int layered_create(rewb200_model* m, const rewb200_layer* layers, const rewb200_
   };
   // a sink of one is a score of zero: the zeros the array starts with
   auto sink_of = [&](const rewb200_layer& L, float** out) { return L.sink ? zero_weights(m, (void**)out, L.heads * sizeof(float)) : REWB200_OK; };
+  auto f32 = [&](float** p, int64_t count) { return zero_weights(m, (void**)p, (size_t)count * sizeof(float)); };
+  auto scale_of = [](const rewb200_layer& L) { return L.mix_scale == 0.f ? 1.f : L.mix_scale; };
+  // The parts of a delta rule or recurrent unit but the input projection, whose columns it returns.
+  auto delta_of = [&](const rewb200_layer& L, DeltaDev& A, int64_t* cols) -> int {
+    const int64_t hv = (int64_t)L.heads * L.vdim;
+    RB_TRY(f32(&A.rate, L.heads));
+    RB_TRY(f32(&A.dt_bias, L.heads));
+    RB_TRY(f32(&A.norm, L.vdim));
+    A.m = DeltaDims{L.heads, L.kv_heads, L.dim, L.vdim, A.rate, A.dt_bias, A.norm, scale_of(L)};
+    const int64_t ch = delta_channels(A.m);
+    RB_TRY(f32(&A.w, L.conv_taps * ch));
+    A.conv = ConvDims{ch, L.conv_taps, A.w, nullptr, nullptr, 1};
+    *cols = ch + hv + 2 * L.heads;
+    return REWB200_OK;
+  };
+  auto lru_of = [&](const rewb200_layer& L, LruDev& A, int64_t* cols) -> int {
+    const int64_t w = (int64_t)L.heads * L.dim, ldn = pad8(L.dim);
+    for (float** p : {&A.x_bias, &A.conv_bias, &A.y_bias, &A.decay}) RB_TRY(f32(p, w));
+    RB_TRY(f32(&A.w, L.conv_taps * w));
+    RB_TRY(f32(&A.gate_bias, L.heads * 2 * ldn));
+    RB_TRY(zero_weights(m, &A.gates, (size_t)L.heads * ldn * 2 * ldn * es));
+    A.m = LruDims{L.heads, L.dim, (int)ldn, A.decay, A.y_bias, scale_of(L)};
+    A.conv = ConvDims{w, L.conv_taps, A.w, A.x_bias, A.conv_bias, 0};
+    *cols = 2 * w;
+    return REWB200_OK;
+  };
   m->layers.resize(n);
   int64_t widest = dp, q_cols = 0, attn_cols = 0;
   for (int l = 0; l < n; ++l) {
@@ -290,7 +400,22 @@ int layered_create(rewb200_model* m, const rewb200_layer* layers, const rewb200_
     D.mixer = L.mixer;
     RB_TRY(zero_weights(m, (void**)&D.ln1g, dp * sizeof(float)));
     if (L.ff && st.block != BLOCK_ONE_NORM) RB_TRY(zero_weights(m, (void**)&D.ln2g, dp * sizeof(float)));
+    if (st.block == BLOCK_SANDWICH) RB_TRY(f32(&D.back1, dp));
+    if (st.block == BLOCK_SANDWICH && L.ff) RB_TRY(f32(&D.back2, dp));
     const bool own = L.kv_from < 0;
+    int64_t beside_cols = 0;   // of the second mixer in the input projection
+    if (L.beside) {
+      const rewb200_layer& M = mixer_spec(m, l, true);
+      D.beside = M.mixer;
+      RB_TRY(M.mixer == MIX_DELTA ? delta_of(M, D.d, &beside_cols) : lru_of(M, D.r, &beside_cols));
+    }
+    // the projection for `cols` columns of the first mixer and those of the second
+    auto in_lin = [&](LinW* w, int64_t cols) -> int {
+      D.beside_in = pad8(cols);
+      RB_TRY(zero_lin(m, w, dp, D.beside_in + pad8(beside_cols)));
+      widest = std::max(widest, w->N);
+      return REWB200_OK;
+    };
     if (L.mixer == MIX_LATENT) {
       LatentDev& A = D.a;
       A.m = LatentDims{L.heads, L.dim, L.rot_dim, L.vdim, L.q_rank, L.kv_rank, L.rope_dims, L.window, L.out_gate, L.scale, nullptr, m->cfg.max_seq, own ? 1 : 0, nullptr};
@@ -309,37 +434,50 @@ int layered_create(rewb200_model* m, const rewb200_layer* layers, const rewb200_
       GqaDev& G = D.g;
       G.ldk = pad8(L.dim);
       G.ldv = pad8(L.vdim);
-      RB_TRY(zero_lin(m, &G.in, dp, pad8((int64_t)L.heads * L.dim + (own ? (int64_t)L.kv_heads * (L.dim + (L.values_from_keys ? 0 : L.vdim)) : 0) + (L.out_gate ? L.heads : 0))));
+      G.gate_col = (int64_t)L.heads * L.dim + (own ? (int64_t)L.kv_heads * (L.dim + (L.values_from_keys ? 0 : L.vdim)) : 0);
+      RB_TRY(in_lin(&G.in, G.gate_col + (L.out_gate == 2 ? (int64_t)L.heads * L.vdim : L.out_gate ? L.heads : 0)));
+      if (L.qkv_bias) RB_TRY(f32(&G.in_bias, G.gate_col));
+      if (L.head_mix) RB_TRY(f32(&G.talk, (int64_t)L.heads * L.heads));
       if (L.qk_norm) RB_TRY(zero_weights(m, (void**)&G.q_norm, L.dim * sizeof(float)));
       if (L.qk_norm && own) RB_TRY(zero_weights(m, (void**)&G.k_norm, L.dim * sizeof(float)));
       const int nb = L.bias_rows > 0 ? bias_distances(L.bias_rows, L.bias_max) : 0;
       if (nb > 0) RB_TRY(zero_weights(m, (void**)&G.bias, (size_t)L.heads * nb * sizeof(float)));
       RB_TRY(sink_of(L, &G.sink));
-      G.m = GqaDims{L.heads, L.kv_heads, L.dim, L.vdim, own ? 1 : 0, L.out_gate, L.scale, G.q_norm, G.k_norm, L.temp_every, L.temp_coef, G.bias, nb, G.sink,
-                    L.values_from_keys, L.conv_taps, nullptr, L.rope_dims, nullptr};
+      G.m = GqaDims{L.heads, L.kv_heads, L.dim, L.vdim, own ? 1 : 0, L.out_gate == 1, L.scale, G.q_norm, G.k_norm, L.temp_every, L.temp_coef, G.bias, nb, G.sink,
+                    L.values_from_keys, L.conv_taps, nullptr, L.rope_dims, nullptr, L.rope_pairs, L.v_norm, G.in_bias, L.window, L.keep_first, G.talk,
+                    L.out_gate == 2, scale_of(L)};
       RB_TRY(rope_of(L, &G.m.rope));
       if (L.conv_taps > 0) RB_TRY(zero_weights(m, (void**)&G.conv, (size_t)L.conv_taps * gqa_channels(G.m) * sizeof(float)));
       G.m.conv = G.conv;
-      widest = std::max(widest, G.in.N);
       q_cols = std::max(q_cols, pad8((int64_t)L.heads * L.dim));
+    } else if (L.mixer == MIX_DELTA) {
+      int64_t cols = 0;
+      RB_TRY(delta_of(L, D.d, &cols));
+      RB_TRY(in_lin(&D.d.in, cols));
+    } else if (L.mixer == MIX_LRU) {
+      int64_t cols = 0;
+      RB_TRY(lru_of(L, D.r, &cols));
+      RB_TRY(in_lin(&D.r.in, cols));
     } else {
       GlaDev& A = D.l;
       const int64_t hk = (int64_t)L.heads * L.dim, hv = (int64_t)L.heads * L.vdim;
-      RB_TRY(zero_lin(m, &A.in, dp, pad8(2 * hk + 2 * hv + L.decay_rank)));
+      RB_TRY(in_lin(&A.in, 2 * hk + 2 * hv + L.decay_rank));
       RB_TRY(zero_weights(m, (void**)&A.a2, hk * L.decay_rank * sizeof(float)));
       RB_TRY(zero_weights(m, (void**)&A.a2_b, hk * sizeof(float)));
       RB_TRY(zero_weights(m, (void**)&A.norm, L.vdim * sizeof(float)));
       A.m = GlaDims{L.heads, L.dim, L.vdim, L.decay_rank, L.tau, A.a2, A.a2_b, A.norm};
-      widest = std::max(widest, A.in.N);
     }
-    RB_TRY(zero_lin(m, &D.o, pad8((int64_t)L.heads * L.vdim), dp));
+    D.beside_out = pad8((int64_t)L.heads * L.vdim);
+    const rewb200_layer& M = mixer_spec(m, l, D.beside != 0);
+    RB_TRY(zero_lin(m, &D.o, D.beside_out + (D.beside ? pad8((int64_t)M.heads * M.vdim) : 0), dp));
     attn_cols = std::max(attn_cols, D.o.K);
     D.ff = L.ff;
     const int64_t fp = pad8(L.ffn);
     if (L.ff == 1) {
       D.ffn_local = fp;
+      D.gelu = L.ff_act == 1;
       m->max_ffn = std::max(m->max_ffn, fp);
-      RB_TRY(zero_lin(m, &D.gu, dp, 2 * fp));
+      RB_TRY(zero_lin(m, &D.gu, dp, D.gelu ? fp : 2 * fp));
       RB_TRY(zero_lin(m, &D.down, fp, dp));
     } else if (L.ff == 2) {
       MoeDev& X = D.x;
@@ -382,7 +520,7 @@ int layered_create(rewb200_model* m, const rewb200_layer* layers, const rewb200_
     if (m->layers[R.layer].moe) ++m->n_moe;
     R.cache = (int)r;
     const rewb200_layer& L = m->spec[R.layer];
-    if (L.mixer != MIX_GLA && L.kv_from >= 0)   // the latest run of that layer: in a loop, the one of the same pass
+    if (L.kv_from >= 0)   // the latest run of that layer: in a loop, the one of the same pass
       for (size_t q = 0; q < r; ++q)
         if (m->runs[q].layer == L.kv_from) R.cache = (int)q;
   }
@@ -440,12 +578,19 @@ int layered_set_tensor(rewb200_model* m, int64_t index, const float* host, int64
     RB_CUDA(cudaGetLastError());
     return REWB200_OK;
   }
+  if (t.slot == SL_BIGRAM) return cols(m->bigram, m->dp, 0);
+  if (t.slot == SL_LOOP_IN) {   // the rows of x, then those of the embeddings
+    const int64_t d = R / 2;
+    RB_TRY(scatter(m, C, 0, 0, d, C, m->loop_in.w, true, m->dp, C, C, 0));
+    return scatter(m, C, d, 0, d, C, (char*)m->loop_in.w + (size_t)m->dp * m->dp * es, true, m->dp, C, C, 0);
+  }
   if (t.slot == SL_STEP) return scatter(m, C, 0, 0, R, C, m->step_vec, false, m->dp, C, C, 0);
   if (t.slot == SL_FINAL) return norm(m->ng, zc);
   if (t.slot == SL_HEAD) return cols(m->lm.w, m->vp, 0);
   LayerDev& D = m->layers[t.layer];
-  const rewb200_layer& L = m->spec[t.layer];
+  const rewb200_layer& L = mixer_spec(m, t.layer, t.second);
   LatentDev& A = D.a;
+  const int64_t in0 = t.second ? D.beside_in : 0;
   const int64_t fp = pad8(L.ffn);
   // gate / up columns of `f` logical ones: bf16 interleaves groups of 8, f32 concatenates
   auto gate_up = [&](void* w, bool up, int64_t f) {
@@ -460,9 +605,13 @@ int layered_set_tensor(rewb200_model* m, int64_t index, const float* host, int64
       case SL_Q: return cols(G.in.w, G.in.N, 0);
       case SL_K: return cols(G.in.w, G.in.N, hk);
       case SL_V: return cols(G.in.w, G.in.N, hk + kv * L.dim);
-      case SL_G: return cols(G.in.w, G.in.N, hk + kv * (L.dim + (L.values_from_keys ? 0 : L.vdim)));
-      case SL_Q_CONV: return upload_conv(m, G, 0, hk, host);
-      case SL_K_CONV: return upload_conv(m, G, hk, kv * L.dim, host);
+      case SL_G: return cols(G.in.w, G.in.N, G.gate_col);
+      case SL_Q_CONV: return upload_conv(m, G.conv, G.m.taps, gqa_channels(G.m), 0, hk, host);
+      case SL_K_CONV: return upload_conv(m, G.conv, G.m.taps, gqa_channels(G.m), hk, kv * L.dim, host);
+      case SL_TALK: return vector(G.talk);
+      case SL_Q_B: return vector(G.in_bias);
+      case SL_K_B: return vector(G.in_bias + hk);
+      case SL_V_B: return vector(G.in_bias + hk + kv * L.dim);
       case SL_Q_NORM: return norm(G.q_norm, false);
       case SL_K_NORM: return norm(G.k_norm, false);
       case SL_SINK: return vector(G.sink);
@@ -484,9 +633,70 @@ int layered_set_tensor(rewb200_model* m, int64_t index, const float* host, int64
       default: break;
     }
   }
+  if (L.mixer == MIX_DELTA) {
+    DeltaDev& G = D.d;
+    LinW& in = in_of(D);
+    const int64_t gk = (int64_t)L.kv_heads * L.dim, ch = G.conv.channels;
+    auto conv = [&](int64_t c0, int64_t n) { return upload_conv(m, G.w, L.conv_taps, ch, c0, n, host); };
+    switch (t.slot) {
+      case SL_Q: return cols(in.w, in.N, in0);
+      case SL_K: return cols(in.w, in.N, in0 + gk);
+      case SL_V: return cols(in.w, in.N, in0 + 2 * gk);
+      case SL_V_GATE: return cols(in.w, in.N, in0 + ch);
+      case SL_BETA: return cols(in.w, in.N, in0 + ch + hv);
+      case SL_ALPHA: return cols(in.w, in.N, in0 + ch + hv + L.heads);
+      case SL_Q_CONV: return conv(0, gk);
+      case SL_K_CONV: return conv(gk, gk);
+      case SL_V_CONV: return conv(2 * gk, hv);
+      case SL_RATE:
+        RB_TRY(vector(G.rate));
+        return delta_rate_launch(m->c, G.rate, L.heads);
+      case SL_DT_BIAS: return vector(G.dt_bias);
+      case SL_V_NORM: return norm(G.norm, false);
+      default: break;
+    }
+  }
+  if (L.mixer == MIX_LRU) {
+    LruDev& G = D.r;
+    LinW& in = in_of(D);
+    const int64_t ldn = G.m.ldn;
+    // a gate's matrices [out, in] per block, transposed into [in][r | i]
+    auto gate = [&](int64_t off) -> int {
+      const int64_t n = L.dim;
+      std::vector<float> w((size_t)(L.heads * n * n));
+      for (int64_t b = 0; b < L.heads; ++b)
+        for (int64_t o = 0; o < n; ++o)
+          for (int64_t i = 0; i < n; ++i) w[(b * n + i) * n + o] = host[(b * n + o) * n + i];
+      RB_TRY(upload_stage(m, w.data(), numel));
+      for (int64_t b = 0; b < L.heads; ++b)
+        RB_TRY(scatter(m, n, b * n, 0, n, n, (char*)G.gates + (size_t)b * ldn * 2 * ldn * es, true, 2 * ldn, n, n, off));
+      return REWB200_OK;
+    };
+    auto gate_bias = [&](int64_t off) { return scatter(m, L.dim, 0, 0, L.heads, L.dim, G.gate_bias + off, false, 2 * ldn, L.dim, L.dim, 0); };
+    switch (t.slot) {
+      case SL_Y: return cols(in.w, in.N, in0);
+      case SL_X: return cols(in.w, in.N, in0 + hk);
+      case SL_Y_B: return vector(G.y_bias);
+      case SL_X_B: return vector(G.x_bias);
+      case SL_CONV: return upload_conv(m, G.w, L.conv_taps, hk, 0, hk, host);
+      case SL_CONV_B: return vector(G.conv_bias);
+      case SL_RA: return gate(0);
+      case SL_RI: return gate(ldn);
+      case SL_RA_B: return gate_bias(0);
+      case SL_RI_B: return gate_bias(ldn);
+      case SL_LAM:
+        RB_TRY(vector(G.decay));
+        return lru_decay_launch(m->c, G.decay, hk);
+      default: break;
+    }
+  }
   switch (t.slot) {
     case SL_NORM1: return norm(D.ln1g, zc);
     case SL_NORM2: return norm(D.ln2g, zc);
+    case SL_BACK1: return norm(D.back1, zc);
+    case SL_BACK2: return norm(D.back2, zc);
+    case SL_UP_B: return vector(D.gu.b);
+    case SL_DOWN_B: return vector(D.down.b);
     case SL_DQ_NORM: return norm(A.q_norm, false);
     case SL_DKV_NORM: return norm(A.kv_norm, false);
     case SL_DQ: return cols(A.in.w, A.in.N, 0);
@@ -496,9 +706,9 @@ int layered_set_tensor(rewb200_model* m, int64_t index, const float* host, int64
     case SL_UQ: return cols(A.uq.w, A.uq.N, 0);
     case SL_UK: return cols(A.ukv.w, A.ukv.N, 0);
     case SL_UV: return cols(A.ukv.w, A.ukv.N, (int64_t)L.heads * L.dim);
-    case SL_O: return cols(D.o.w, m->dp, 0);
+    case SL_O: return cols((char*)D.o.w + (size_t)(t.second ? D.beside_out : 0) * m->dp * es, m->dp, 0);
     case SL_GATE: return gate_up(D.gu.w, false, L.ffn);
-    case SL_UP: return gate_up(D.gu.w, true, L.ffn);
+    case SL_UP: return D.gelu ? cols(D.gu.w, D.gu.N, 0) : gate_up(D.gu.w, true, L.ffn);
     case SL_DOWN: return cols(D.down.w, m->dp, 0);
     case SL_ROUTER: return cols(D.x.router.w, D.x.router.N, 0);
     case SL_ROUTER_B: return vector(D.x.router.b);
@@ -523,11 +733,27 @@ int layered_init_random(rewb200_model* m, uint64_t seed, float std) {
   auto fill = [&](void* w, int64_t n) { return fill_normal_launch(c, w, dt, n, ++k, std); };
   RB_TRY(fill(m->embed, (int64_t)m->cfg.vocab * m->dp));
   RB_TRY(fill(m->lm.w, m->lm.K * m->lm.N));
+  if (m->bigram) RB_TRY(fill(m->bigram, ((int64_t)m->stack.bigram_buckets + 1) * m->dp));
+  if (m->loop_in.w) RB_TRY(fill(m->loop_in.w, m->loop_in.K * m->loop_in.N));
   if (m->step_vec) RB_TRY(fill_normal_launch(c, m->step_vec, REWB200_F32, m->stack.loop_times * m->dp, ++k, std));
   RB_TRY(fill_const_launch(c, m->ng, REWB200_F32, m->dp, 1.f));
   for (LayerDev& D : m->layers) {
     RB_TRY(fill_const_launch(c, D.ln1g, REWB200_F32, m->dp, 1.f));
     if (D.ln2g) RB_TRY(fill_const_launch(c, D.ln2g, REWB200_F32, m->dp, 1.f));
+    for (float* p : {D.back1, D.back2})
+      if (p) RB_TRY(fill_const_launch(c, p, REWB200_F32, m->dp, 1.f));
+    if (has(D, MIX_DELTA)) {
+      RB_TRY(fill_normal_launch(c, D.d.w, REWB200_F32, D.d.conv.taps * D.d.conv.channels, ++k, 0.5f));
+      RB_TRY(fill_const_launch(c, D.d.rate, REWB200_F32, D.d.m.heads, 0.05f));
+      RB_TRY(fill_const_launch(c, D.d.norm, REWB200_F32, D.d.m.vdim, 1.f));
+    }
+    if (has(D, MIX_LRU)) {
+      const int64_t w = (int64_t)D.r.m.blocks * D.r.m.n;
+      RB_REQUIRE(D.r.m.n == D.r.m.ldn, "random weights need blocks of a multiple of 8 channels");
+      RB_TRY(fill_normal_launch(c, D.r.w, REWB200_F32, D.r.conv.taps * w, ++k, 0.5f));
+      RB_TRY(fill_const_launch(c, D.r.decay, REWB200_F32, w, -0.1f));
+      RB_TRY(fill(D.r.gates, (int64_t)D.r.m.blocks * D.r.m.n * 2 * D.r.m.n));
+    }
     if (D.mixer == MIX_LATENT) {
       RB_TRY(fill_const_launch(c, D.a.q_norm, REWB200_F32, D.a.m.q_rank, 1.f));
       if (D.a.kv_norm) RB_TRY(fill_const_launch(c, D.a.kv_norm, REWB200_F32, D.a.m.kv_rank, 1.f));
@@ -536,7 +762,8 @@ int layered_init_random(rewb200_model* m, uint64_t seed, float std) {
       if (D.g.k_norm) RB_TRY(fill_const_launch(c, D.g.k_norm, REWB200_F32, D.g.m.dim, 1.f));
       if (D.g.conv) RB_TRY(fill_normal_launch(c, D.g.conv, REWB200_F32, D.g.m.taps * gqa_channels(D.g.m), ++k, 0.5f));
       if (D.g.bias) RB_TRY(fill_normal_launch(c, D.g.bias, REWB200_F32, (int64_t)D.g.m.heads * D.g.m.n_bias, ++k, 1.f));
-    } else {
+      if (D.g.talk) RB_TRY(fill_normal_launch(c, D.g.talk, REWB200_F32, (int64_t)D.g.m.heads * D.g.m.heads, ++k, 0.3f));
+    } else if (D.mixer == MIX_GLA) {
       RB_TRY(fill_const_launch(c, D.l.norm, REWB200_F32, D.l.m.vdim, 1.f));
       RB_TRY(fill_const_launch(c, D.l.a2_b, REWB200_F32, (int64_t)D.l.m.heads * D.l.m.dim, 2.f));
       RB_TRY(fill_normal_launch(c, D.l.a2, REWB200_F32, (int64_t)D.l.m.heads * D.l.m.dim * D.l.m.rank, ++k, std));
@@ -557,8 +784,10 @@ int layered_init_random(rewb200_model* m, uint64_t seed, float std) {
 int layered_plans(rewb200_model* m) {
   if (m->cfg.dtype != REWB200_BF16) return REWB200_OK;
   auto plan = [&](LinW& w) { return linear_bf16_plan(&w.plan, (const bf16*)w.w, w.K, w.N, 0); };
+  if (m->loop_in.w) RB_TRY(plan(m->loop_in));
   for (LayerDev& D : m->layers) {
     for (LinW* w : mixer_linears(D)) RB_TRY(plan(*w));
+    if (has(D, MIX_LRU)) RB_TRY(linear_bf16_plan(&D.r.plan_gates, (const bf16*)D.r.gates, D.r.m.ldn, 2 * D.r.m.ldn, D.r.m.blocks));
     if (has_dense(D))
       for (LinW* w : {&D.gu, &D.down}) RB_TRY(plan(*w));
     if (D.ff == 2) {
@@ -581,11 +810,29 @@ int layered_acts(rewb200_session* s, int64_t rows) {
     heads = std::max<int64_t>(heads, std::max(D.a.m.heads, D.g.m.heads));
   }
   heads = std::max<int64_t>(heads, 1);
+  int64_t conv = 0, gates = 0, blocks = 0;
+  for (const LayerDev& D : m->layers) {
+    if (has(D, MIX_DELTA)) conv = std::max(conv, pad8(D.d.conv.channels));
+    if (!has(D, MIX_LRU)) continue;
+    conv = std::max<int64_t>(conv, (int64_t)D.r.m.blocks * D.r.m.ldn);
+    gates = std::max<int64_t>(gates, (int64_t)D.r.m.blocks * 2 * D.r.m.ldn);
+    blocks = std::max<int64_t>(blocks, D.r.m.blocks);
+  }
+  auto zeroed = [&](void** p, size_t bytes) -> int {
+    RB_TRY(acts_alloc(c, p, bytes));
+    RB_CUDA(cudaMemsetAsync(*p, 0, bytes, c->stream));
+    return REWB200_OK;
+  };
+  if (conv) RB_TRY(zeroed(&s->conv, (size_t)rows * conv * es));
+  if (gates) RB_TRY(zeroed((void**)&s->gate_pre, (size_t)rows * gates * sizeof(float)));
+  if (gates) RB_TRY(zeroed((void**)&s->group_rows, (size_t)(blocks + 1) * sizeof(int)));
+  if (m->bigram) RB_TRY(zeroed((void**)&s->big_rows, (size_t)rows * sizeof(int)));
+  if (m->loop_in.w) RB_TRY(zeroed(&s->cat, (size_t)rows * 2 * m->dp * es));
   RB_TRY(acts_alloc(c, &s->xn2, (size_t)rows * m->dp * es));
   RB_TRY(acts_alloc(c, &s->cq, (size_t)rows * cq * es));
   RB_TRY(acts_alloc(c, (void**)&s->gate, (size_t)rows * heads * sizeof(float)));
   RB_TRY(acts_alloc(c, (void**)&s->part2, s->part_bytes));
-  if (m->stack.block != BLOCK_OUTPUT_NORM && std::any_of(m->spec.begin(), m->spec.end(), [](const rewb200_layer& L) { return L.shared_ffn > 0; })) {
+  if (m->stack.block != BLOCK_OUTPUT_NORM && m->stack.block != BLOCK_SANDWICH && std::any_of(m->spec.begin(), m->spec.end(), [](const rewb200_layer& L) { return L.shared_ffn > 0; })) {
     RB_TRY(acts_alloc(c, (void**)&s->part3, s->part_bytes));
     RB_TRY(acts_alloc(c, (void**)&s->shared_gate, (size_t)rows * sizeof(float)));
   }
@@ -608,6 +855,8 @@ int layered_session(rewb200_session* s, int64_t n_pages) {
   s->tmK.resize(n);
   s->tmV.resize(n);
   s->state.resize(n, nullptr);
+  s->conv_state.resize(n, nullptr);
+  s->state2.resize(n, nullptr);
   auto zeroed = [&](void** p, size_t bytes) -> int {
     RB_CUDA(cudaMalloc(p, bytes));
     RB_CUDA(cudaMemsetAsync(*p, 0, bytes, m->c->stream));
@@ -628,7 +877,15 @@ int layered_session(rewb200_session* s, int64_t n_pages) {
     // a state needs no clearing between sequences: a portion that starts at position 0 does not read it
     if (D.mixer == MIX_GLA)
       RB_TRY(zeroed((void**)&s->state[r], (size_t)s->B * D.l.m.heads * D.l.m.dim * gla_state_ld(D.l.m.vdim) * sizeof(float)));
+    if (has(D, MIX_DELTA) || has(D, MIX_LRU)) {
+      const bool delta = has(D, MIX_DELTA);
+      const int64_t elems = delta ? (int64_t)D.d.m.heads * D.d.m.dim * gla_state_ld(D.d.m.vdim) : (int64_t)D.r.m.blocks * D.r.m.n;
+      const int64_t conv = conv_state_elems(delta ? D.d.conv : D.r.conv);
+      RB_TRY(zeroed((void**)&s->state2[r], (size_t)s->B * elems * sizeof(float)));
+      if (conv > 0) RB_TRY(zeroed((void**)&s->conv_state[r], (size_t)s->B * conv * sizeof(float)));
+    }
   }
+  if (m->bigram) RB_TRY(zeroed((void**)&s->last_ids, (size_t)s->B * sizeof(int)));
   return REWB200_OK;
 }
 
@@ -675,6 +932,7 @@ int layered_prepare(rewb200_session* s, const FwdOpts& o, int64_t rows) {
   int64_t abs_rows = rows, n_keys = 0;
   s->plan_host.clear();
   s->plan_abs_tiles = s->plan_chunks = s->plan_exp_tiles = s->plan_keys = s->plan_gla_chunks = s->plan_tails = 0;
+  s->plan_gqa_small = s->plan_delta_small = s->plan_delta_large = s->plan_delta_chunks = s->plan_portions = s->plan_longest = 0;
   if (!uniform) {
     std::vector<int>& h = s->plan_host;
     h.assign(2 * rows, 0);
@@ -684,12 +942,18 @@ int layered_prepare(rewb200_session* s, const FwdOpts& o, int64_t rows) {
     int64_t reach = 0;  // the widest window of any layer, 0: everything
     const bool bf = m->cfg.dtype == REWB200_BF16;
     bool exp_ok = bf && c->latent_impl == 0, gqa_ok = bf && c->gqa_impl == 0, gla_ok = bf && c->gla_impl == 0;
-    bool has_latent = false, has_gqa = false, has_gla = false;
+    bool has_latent = false, has_gqa = false, has_gla = false, has_delta = false, delta_ok = bf && c->gla_impl == 0;
     int taps = 0;           // of the longest convolution
     for (const LayerDev& D : m->layers) {
+      if (has(D, MIX_DELTA)) {
+        has_delta = true;
+        delta_ok = delta_ok && delta_chunk_ok(D.d.m);
+        taps = std::max(taps, D.d.conv.taps);
+      }
+      if (has(D, MIX_LRU)) taps = std::max(taps, D.r.conv.taps);
       if (D.mixer == MIX_GQA) {
         has_gqa = true;
-        gqa_ok = gqa_ok && gqa_prefill_ok(D.g.m);
+        gqa_ok = gqa_ok && !gqa_is_mixed(D.g.m) && gqa_prefill_ok(D.g.m);
         taps = std::max(taps, D.g.m.taps);
       }
       if (D.mixer == MIX_GLA) {
@@ -704,8 +968,18 @@ int layered_prepare(rewb200_session* s, const FwdOpts& o, int64_t rows) {
     std::vector<int2> gqa_small;
     std::vector<GqaTile> gqa_large;
     std::vector<GlaPortion> gla_small, gla_large;
-    std::vector<int2> gla_chunk, tails;
+    std::vector<int2> gla_chunk, tails, delta_chunk;
+    std::vector<GlaPortion> delta_small, delta_large, portions;
     for (const StepEntry& e : *o.entries) {
+      portions.push_back({e.row0, e.n, e.pos0, e.lane, 0});
+      s->plan_longest = std::max(s->plan_longest, e.n);
+      if (has_delta) {
+        const bool large = delta_ok && e.n >= CHUNK_MIN_ROWS;
+        const GlaPortion p = {e.row0, e.n, e.pos0, e.lane, large ? (int)delta_chunk.size() : 0};
+        (large ? delta_large : delta_small).push_back(p);
+        if (large)
+          for (int i = 0; i < delta_chunks(e.n); ++i) delta_chunk.push_back(delta_chunk_rows(p, i));
+      }
       for (int i = 0; i < e.n; ++i) {
         h[e.row0 + i] = e.lane;
         h[rows + e.row0 + i] = e.pos0 + i;
@@ -752,6 +1026,10 @@ int layered_prepare(rewb200_session* s, const FwdOpts& o, int64_t rows) {
     s->plan_gla_large = (int)gla_large.size();
     s->plan_gla_chunks = (int)gla_chunk.size();
     s->plan_tails = (int)tails.size();
+    s->plan_delta_small = (int)delta_small.size();
+    s->plan_delta_large = (int)delta_large.size();
+    s->plan_delta_chunks = (int)delta_chunk.size();
+    s->plan_portions = (int)portions.size();
     s->plan_abs_tiles = (int)tiles.size();
     s->plan_chunks = (int)chunks.size();
     s->plan_exp_tiles = (int)exps.size();
@@ -772,6 +1050,11 @@ int layered_prepare(rewb200_session* s, const FwdOpts& o, int64_t rows) {
     append(gqa_large.data(), gqa_large.size() * sizeof(GqaTile));
     append(gla_small.data(), gla_small.size() * sizeof(GlaPortion));
     append(gla_large.data(), gla_large.size() * sizeof(GlaPortion));
+    append(portions.data(), portions.size() * sizeof(GlaPortion));
+    append(delta_small.data(), delta_small.size() * sizeof(GlaPortion));
+    append(delta_large.data(), delta_large.size() * sizeof(GlaPortion));
+    if (h.size() % 2) h.push_back(0);
+    append(delta_chunk.data(), delta_chunk.size() * sizeof(int2));
     if (h.size() > s->plan_cap) {
       s->plan_cap = 0;
       RB_TRY(regrow(s, &s->plan_dev, h.size() * 2 * sizeof(int)));
@@ -794,18 +1077,27 @@ int layered_prepare(rewb200_session* s, const FwdOpts& o, int64_t rows) {
     s->kvx_rows = n_keys;
   }
   // ---- scratch of the absorbed path
-  size_t chunk = 0;
-  for (const LayerDev& D : m->layers)
-    if (D.mixer == MIX_GLA) chunk = std::max(chunk, gla_chunk_bytes(D.l.m));
-  if (chunk * s->plan_gla_chunks > s->gla_work_bytes) {
+  size_t chunk = 0, mix = 0;
+  for (const LayerDev& D : m->layers) {
+    if (D.mixer == MIX_GLA) chunk = std::max(chunk, gla_chunk_bytes(D.l.m) * s->plan_gla_chunks);
+    if (has(D, MIX_DELTA)) chunk = std::max(chunk, delta_chunk_bytes(D.d.m) * s->plan_delta_chunks);
+    if (D.mixer == MIX_GQA && gqa_is_mixed(D.g.m))
+      mix = std::max(mix, gqa_mix_bytes(c, D.g.m, m->cfg.dtype, rows, uniform ? rows : s->plan_gqa_small, uniform ? 1 : GQA_TILE_ROWS, (int64_t)s->max_pages * PAGE));
+  }
+  if (chunk > s->gla_work_bytes) {
     s->gla_work_bytes = 0;
-    RB_TRY(regrow(s, &s->gla_work, chunk * s->plan_gla_chunks));
-    s->gla_work_bytes = chunk * s->plan_gla_chunks;
+    RB_TRY(regrow(s, &s->gla_work, chunk));
+    s->gla_work_bytes = chunk;
+  }
+  if (mix > s->mix_bytes) {
+    s->mix_bytes = 0;
+    RB_TRY(regrow(s, &s->mix_work, mix));
+    s->mix_bytes = mix;
   }
   int64_t units = 0, stats = 0, qe = 0;
   int64_t g_units = 0, g_stats = 0;
   for (const LayerDev& D : m->layers) {
-    if (D.mixer == MIX_GQA) {
+    if (D.mixer == MIX_GQA && !gqa_is_mixed(D.g.m)) {
       const int sp = gqa_kv_splits(c, D.g.m, uniform ? rows : s->plan_gqa_small, s->max_len);
       g_stats = std::max<int64_t>(g_stats, (int64_t)D.g.m.heads * sp);
       g_units = std::max<int64_t>(g_units, (int64_t)D.g.m.heads * sp * D.g.m.vdim);
@@ -857,7 +1149,8 @@ struct StepLists {
   const int2 *key_list = nullptr, *gla_chunks = nullptr, *tails = nullptr;
   RowTiles gqa_small = {};
   const GqaTile* gqa_large = nullptr;
-  const GlaPortion *gla_small = nullptr, *gla_large = nullptr;
+  const GlaPortion *gla_small = nullptr, *gla_large = nullptr, *portions = nullptr, *delta_small = nullptr, *delta_large = nullptr;
+  const int2* delta_chunks = nullptr;
 };
 
 StepLists step_lists(const rewb200_session* s, const FwdOpts& o, int64_t rows) {
@@ -882,12 +1175,18 @@ StepLists step_lists(const rewb200_session* s, const FwdOpts& o, int64_t rows) {
   t.gqa_large = reinterpret_cast<const GqaTile*>(t.gqa_small.list + t.gqa_small.count);
   t.gla_small = reinterpret_cast<const GlaPortion*>(t.gqa_large + s->plan_gqa_large);
   t.gla_large = t.gla_small + s->plan_gla_small;
+  t.portions = t.gla_large + s->plan_gla_large;
+  t.delta_small = t.portions + s->plan_portions;
+  t.delta_large = t.delta_small + s->plan_delta_small;
+  const int* end = reinterpret_cast<const int*>(t.delta_large + s->plan_delta_large);
+  t.delta_chunks = reinterpret_cast<const int2*>(end + (end - s->plan_dev) % 2);
   return t;
 }
 
 // The mixers read s->xn and leave their output (ahead of the output projection) in s->attn.
 
-int gqa_mixer(rewb200_session* s, const FwdOpts& o, const StepLists& t, size_t r, int64_t rows, bool in_graph) {
+// *slabs: slabs of the input projection, which a second mixer reads too.
+int gqa_mixer(rewb200_session* s, const FwdOpts& o, const StepLists& t, size_t r, int64_t rows, bool in_graph, int* slabs) {
   rewb200_model* m = s->m;
   Ctx* c = m->c;
   const int dt = m->cfg.dtype;
@@ -926,6 +1225,43 @@ int gqa_mixer(rewb200_session* s, const FwdOpts& o, const StepLists& t, size_t r
   RB_TRY(gqa_post_launch(c, pa, rows));
   if (!t.uniform) RB_TRY(gqa_conv_state_launch(c, pa));
   if (o.trace) RB_TRY(o.trace->mark(TC_QKV_POST));
+  *slabs = ks;
+  if (gqa_is_mixed(G.m)) {
+    GqaMixArgs ma;
+    memset(&ma, 0, sizeof(ma));
+    ma.m = G.m;
+    ma.map = t.map;
+    ma.tiles = t.gqa_small;
+    ma.max_tile_rows = t.uniform ? 1 : GQA_TILE_ROWS;
+    ma.rows = rows;
+    ma.q = s->q;
+    ma.ldq = ldq;
+    if (G.m.gate_elem) ma.gate = s->part + G.gate_col;
+    ma.nsplit = ks;
+    ma.split_stride = pa.split_stride;
+    ma.ld = pa.ld;
+    if (G.m.gate) ma.gate_head = s->gate;
+    ma.out = s->attn;
+    ma.ldo = D.o.K;
+    ma.kc = pa.kc;
+    ma.vc = pa.vc;
+    if (dt == REWB200_BF16) {
+      ma.tm_k = &s->tmK[R.cache];
+      ma.tm_v = &s->tmV[R.cache];
+    }
+    ma.ldk = G.ldk;
+    ma.ldv = G.ldv;
+    ma.block_table = s->block_table;
+    ma.max_pages = s->max_pages;
+    ma.dtype = dt;
+    ma.work = s->mix_work;
+    ma.work_bytes = s->mix_bytes;
+    ma.early_kv = in_graph ? 1 : 0;
+    ma.status = c->d_status;
+    RB_TRY(gqa_mix_launch(c, ma));
+    if (o.trace) RB_TRY(o.trace->mark(TC_ATTN));
+    return REWB200_OK;
+  }
   GqaAttnArgs aa;
   memset(&aa, 0, sizeof(aa));
   aa.m = G.m;
@@ -976,7 +1312,7 @@ int gqa_mixer(rewb200_session* s, const FwdOpts& o, const StepLists& t, size_t r
   return REWB200_OK;
 }
 
-int gla_mixer(rewb200_session* s, const FwdOpts& o, const StepLists& t, size_t r, int64_t rows, bool in_graph) {
+int gla_mixer(rewb200_session* s, const FwdOpts& o, const StepLists& t, size_t r, int64_t rows, bool in_graph, int* slabs) {
   rewb200_model* m = s->m;
   Ctx* c = m->c;
   LayerDev& D = m->layers[m->runs[r].layer];
@@ -984,6 +1320,7 @@ int gla_mixer(rewb200_session* s, const FwdOpts& o, const StepLists& t, size_t r
   int ks = 1;
   RB_TRY(run_linear(s, A.in, s->xn, m->dp, rows, true, 0, s->part, A.in.N, &ks));
   if (o.trace) RB_TRY(o.trace->mark(TC_QKV));
+  *slabs = ks;
   GlaArgs ga;
   memset(&ga, 0, sizeof(ga));
   ga.m = A.m;
@@ -1113,19 +1450,165 @@ int latent_mixer(rewb200_session* s, const FwdOpts& o, const StepLists& t, size_
   return REWB200_OK;
 }
 
-int mixer(rewb200_session* s, const FwdOpts& o, const StepLists& t, size_t r, int64_t rows, bool in_graph) {
-  switch (s->m->layers[s->m->runs[r].layer].mixer) {
-    case MIX_GQA: return gqa_mixer(s, o, t, r, rows, in_graph);
-    case MIX_GLA: return gla_mixer(s, o, t, r, rows, in_graph);
-    default: return latent_mixer(s, o, t, r, rows, in_graph);
+// What the two mixers below read of the input projection (columns from `col` on, `ks` slabs) and where their output goes.
+struct MixerAt {
+  const LinW* in;
+  int64_t col, out_col;
+  int ks;
+};
+
+int delta_mixer(rewb200_session* s, const FwdOpts& o, const StepLists& t, size_t r, int64_t rows, bool in_graph, const MixerAt& at) {
+  rewb200_model* m = s->m;
+  Ctx* c = m->c;
+  LayerDev& D = m->layers[m->runs[r].layer];
+  DeltaDev& A = D.d;
+  const size_t es = dtype_size(m->cfg.dtype);
+  const int64_t ch = A.conv.channels;
+  ConvArgs ca;
+  memset(&ca, 0, sizeof(ca));
+  ca.m = A.conv;
+  ca.partial = s->part + at.col;
+  ca.nsplit = at.ks;
+  ca.split_stride = rows * at.in->N;
+  ca.ld = at.in->N;
+  ca.map = t.map;
+  ca.capacity = s->max_len;
+  ca.out = s->conv;
+  ca.ldo = pad8(ch);
+  ca.dtype = m->cfg.dtype;
+  ca.state = s->conv_state[r];
+  ca.tails = t.tails;
+  ca.n_tails = s->plan_tails;
+  ca.early = in_graph ? 1 : 0;
+  ca.status = c->d_status;
+  RB_TRY(conv_launch(c, ca, rows));
+  if (o.trace) RB_TRY(o.trace->mark(TC_QKV_POST));
+  DeltaArgs da;
+  memset(&da, 0, sizeof(da));
+  da.m = A.m;
+  da.list = t.delta_small;
+  da.count = t.uniform ? (int)rows : s->plan_delta_small;
+  da.pos0 = s->d_pos;
+  da.b0 = o.b0;
+  da.x = s->conv;
+  da.ldx = ca.ldo;
+  da.partial = ca.partial + ch;
+  da.nsplit = at.ks;
+  da.split_stride = ca.split_stride;
+  da.ld = ca.ld;
+  da.eps = m->cfg.eps;
+  da.state = s->state2[r];
+  da.ldv = (int)gla_state_ld(A.m.vdim);
+  da.out = (char*)s->attn + at.out_col * es;
+  da.ldo = D.o.K;
+  da.dtype = m->cfg.dtype;
+  da.early = in_graph ? 1 : 0;
+  da.status = c->d_status;
+  RB_TRY(delta_recurrent_launch(c, da));
+  if (!t.uniform && s->plan_delta_large > 0) {
+    da.list = t.delta_large;
+    da.count = s->plan_delta_large;
+    da.chunks = t.delta_chunks;
+    da.n_chunks = s->plan_delta_chunks;
+    da.work = s->gla_work;
+    RB_TRY(delta_chunk_launch(c, da));
   }
+  if (o.trace) RB_TRY(o.trace->mark(TC_ATTN));
+  return REWB200_OK;
 }
 
-// A gated SiLU feed-forward (dense, or the shared expert beside routed ones): f32 slabs of the result in `out`.
+int lru_mixer(rewb200_session* s, const FwdOpts& o, const StepLists& t, size_t r, int64_t rows, bool in_graph, const MixerAt& at) {
+  rewb200_model* m = s->m;
+  Ctx* c = m->c;
+  LayerDev& D = m->layers[m->runs[r].layer];
+  LruDev& A = D.r;
+  const bool bf = m->cfg.dtype == REWB200_BF16;
+  const int64_t width = A.conv.channels, ldn = A.m.ldn;
+  ConvArgs ca;
+  memset(&ca, 0, sizeof(ca));
+  ca.m = A.conv;
+  ca.partial = s->part + at.col + width;
+  ca.nsplit = at.ks;
+  ca.split_stride = rows * at.in->N;
+  ca.ld = at.in->N;
+  ca.map = t.map;
+  ca.capacity = s->max_len;
+  ca.out = s->conv;
+  ca.ldo = ldn;
+  ca.group = A.m.n;
+  ca.offsets = s->group_rows;
+  ca.dtype = m->cfg.dtype;
+  ca.state = s->conv_state[r];
+  ca.tails = t.tails;
+  ca.n_tails = s->plan_tails;
+  ca.early = in_graph ? 1 : 0;
+  ca.status = c->d_status;
+  RB_TRY(conv_launch(c, ca, rows));
+  if (o.trace) RB_TRY(o.trace->mark(TC_QKV_POST));
+  // both gates of every block: a stacked matrix per block on the block's channels
+  if (bf) {
+    RB_TRY(linear_bf16_launch(c, A.plan_gates, (const bf16*)s->conv, ldn, rows * A.m.blocks, EPI_BIAS_F32, 1, s->gate_pre, 2 * ldn, A.gate_bias,
+                              s->group_rows, (int)rows));
+  } else {
+    for (int b = 0; b < A.m.blocks; ++b)
+      RB_TRY(gemm_f32_ld_launch(c, (const float*)s->conv + (int64_t)b * rows * ldn, ldn, (const float*)A.gates + (int64_t)b * ldn * 2 * ldn, 2 * ldn,
+                                A.gate_bias + (int64_t)b * 2 * ldn, s->gate_pre + (int64_t)b * rows * 2 * ldn, 2 * ldn, rows, ldn, 2 * ldn));
+  }
+  if (o.trace) RB_TRY(o.trace->mark(TC_GATE_UP));
+  LruArgs la;
+  memset(&la, 0, sizeof(la));
+  la.m = A.m;
+  la.list = t.portions;
+  la.count = t.uniform ? (int)rows : s->plan_portions;
+  la.longest = s->plan_longest;
+  la.pos0 = s->d_pos;
+  la.b0 = o.b0;
+  la.rows = rows;
+  la.gates = s->gate_pre;
+  la.u = s->conv;
+  la.partial = s->part + at.col;
+  la.nsplit = at.ks;
+  la.split_stride = ca.split_stride;
+  la.ld = ca.ld;
+  la.state = s->state2[r];
+  la.out = (char*)s->attn + at.out_col * dtype_size(m->cfg.dtype);
+  la.ldo = D.o.K;
+  la.dtype = m->cfg.dtype;
+  la.early = in_graph ? 1 : 0;
+  RB_TRY(lru_launch(c, la));
+  if (o.trace) RB_TRY(o.trace->mark(TC_ATTN));
+  return REWB200_OK;
+}
+
+int mixer(rewb200_session* s, const FwdOpts& o, const StepLists& t, size_t r, int64_t rows, bool in_graph) {
+  LayerDev& D = s->m->layers[s->m->runs[r].layer];
+  MixerAt at = {&in_of(D), 0, 0, 1};
+  auto recurrent = [&](int kind) { return kind == MIX_DELTA ? delta_mixer(s, o, t, r, rows, in_graph, at) : lru_mixer(s, o, t, r, rows, in_graph, at); };
+  switch (D.mixer) {
+    case MIX_GQA: RB_TRY(gqa_mixer(s, o, t, r, rows, in_graph, &at.ks)); break;
+    case MIX_GLA: RB_TRY(gla_mixer(s, o, t, r, rows, in_graph, &at.ks)); break;
+    case MIX_LATENT: return latent_mixer(s, o, t, r, rows, in_graph);
+    default:
+      RB_TRY(run_linear(s, *at.in, s->xn, s->m->dp, rows, true, 0, s->part, at.in->N, &at.ks));
+      if (o.trace) RB_TRY(o.trace->mark(TC_QKV));
+      RB_TRY(recurrent(D.mixer));
+  }
+  if (!D.beside) return REWB200_OK;
+  at.col = D.beside_in;
+  at.out_col = D.beside_out;
+  return recurrent(D.beside);
+}
+
+// A feed-forward, gated SiLU (dense, or the shared expert beside routed ones) or tanh GELU: f32 slabs of the result in `out`,
+// without the bias of the down projection.
 int dense_ff(rewb200_session* s, const FwdOpts& o, LayerDev& D, const void* x, int64_t rows, float* out, int* ks) {
   rewb200_model* m = s->m;
   const int64_t dp = m->dp;
-  if (m->cfg.dtype == REWB200_BF16) {
+  if (D.gelu) {
+    const bool bf = m->cfg.dtype == REWB200_BF16;
+    RB_TRY(run_linear(s, D.gu, x, dp, rows, false, bf ? EPI_GELU_BF16 : EPI_BIAS_F32, bf ? s->h : (void*)s->gu32, D.ffn_local, nullptr));
+    if (!bf) RB_TRY(gelu_f32_launch(m->c, s->gu32, (float*)s->h, rows * D.ffn_local));
+  } else if (m->cfg.dtype == REWB200_BF16) {
     RB_TRY(run_linear(s, D.gu, x, dp, rows, false, EPI_SWIGLU_BF16, s->h, D.ffn_local, nullptr));
   } else {
     RB_TRY(run_linear(s, D.gu, x, dp, rows, false, EPI_BIAS_F32, s->gu32, 2 * D.ffn_local, nullptr));
@@ -1238,6 +1721,96 @@ int output_norm_blocks(rewb200_session* s, const FwdOpts& o, const NormArgs& na,
   return REWB200_OK;
 }
 
+// Blocks normed on both sides: x += back1(mixer(norm1(x))), x += back2(ff(norm2(x))).
+int sandwich_blocks(rewb200_session* s, const FwdOpts& o, const NormArgs& na, int64_t rows, bool in_graph) {
+  rewb200_model* m = s->m;
+  Ctx* c = m->c;
+  const int64_t dp = m->dp;
+  const size_t es = dtype_size(m->cfg.dtype);
+  const StepLists t = step_lists(s, o, rows);
+  OutputNormArgs base;
+  memset(&base, 0, sizeof(base));
+  base.x_res = s->x_res;
+  base.split_stride = rows * dp;
+  base.eps = m->cfg.eps;
+  base.d = dp;
+  base.d_mean = na.d_mean;
+  base.out = s->xn;
+  base.dtype = m->cfg.dtype;
+  base.status = c->d_status;
+  auto enters = [&](size_t r) { return m->loop_in.w && r < m->runs.size() && m->runs[r].step >= 0; };
+  // what the launch that finishes x leaves for run r: its norm (the final one behind the last run), or x itself ahead of a pass
+  auto ahead_of = [&](size_t r, OutputNormArgs& a) {
+    if (enters(r)) {
+      a.out = s->cat;
+      a.ldo = 2 * dp;
+    } else {
+      a.final_gamma = r < m->runs.size() ? m->layers[m->runs[r].layer].ln1g : m->ng;
+    }
+  };
+  if (o.trace) RB_TRY(o.trace->begin(c->stream));
+  {
+    OutputNormArgs a = base;
+    a.embed = na.embed;
+    a.embed_scale = m->stack.embed_scale;
+    a.ids = na.ids;
+    a.vocab = na.vocab;
+    if (m->bigram) {
+      RB_TRY(bigram_rows_launch(c, na.ids, t.map.row_lane, t.map.row_pos, s->d_pos, o.b0, rows, m->stack.bigram_buckets, m->stack.bigram_mul_prev,
+                                m->stack.bigram_mul_cur, m->cfg.vocab, s->last_ids, s->big_rows, c->d_status));
+      a.embed2 = m->bigram;
+      a.ids2 = s->big_rows;
+    }
+    if (m->loop_in.w) {
+      a.out_x = (char*)s->cat + dp * es;
+      a.ldx = 2 * dp;
+    }
+    ahead_of(0, a);
+    RB_TRY(output_norm_launch(c, a, rows));
+    if (o.trace) RB_TRY(o.trace->mark(TC_EMBED));
+  }
+  for (size_t r = 0; r < m->runs.size(); ++r) {
+    LayerDev& D = m->layers[m->runs[r].layer];
+    if (enters(r)) {
+      OutputNormArgs a = base;
+      a.nsplit = 1;
+      RB_TRY(run_linear(s, m->loop_in, s->cat, 2 * dp, rows, true, 0, s->part, dp, &a.nsplit));
+      a.partial = s->part;
+      a.replace = 1;
+      a.final_gamma = D.ln1g;
+      RB_TRY(output_norm_launch(c, a, rows));
+      if (o.trace) RB_TRY(o.trace->mark(TC_EMBED));
+    }
+    RB_TRY(mixer(s, o, t, r, rows, in_graph));
+    OutputNormArgs a = base;
+    a.nsplit = 1;
+    RB_TRY(run_linear(s, D.o, s->attn, D.o.K, rows, true, 0, s->part, dp, &a.nsplit));
+    if (o.trace) RB_TRY(o.trace->mark(TC_O));
+    a.partial = s->part;
+    a.gamma = D.back1;
+    if (D.ff) a.final_gamma = D.ln2g;
+    else ahead_of(r + 1, a);
+    RB_TRY(output_norm_launch(c, a, rows));
+    if (o.trace) RB_TRY(o.trace->mark(TC_NORM_ATTN));
+    if (D.ff) {
+      OutputNormArgs b = base;
+      b.nsplit = 1;
+      RB_TRY(dense_ff(s, o, D, s->xn, rows, s->part, &b.nsplit));
+      b.partial = s->part;
+      b.bias = D.gelu ? D.down.b : nullptr;
+      b.gamma = D.back2;
+      ahead_of(r + 1, b);
+      RB_TRY(output_norm_launch(c, b, rows));
+      if (o.trace) RB_TRY(o.trace->mark(TC_NORM_FFN));
+    }
+    if (s->layer_rec && !t.uniform) {
+      RB_CUDA(cudaMemcpyAsync(s->layer_rec + r * s->rows_cap * dp, s->x_res, (size_t)rows * dp * sizeof(float), cudaMemcpyDeviceToDevice, c->stream));
+      s->layer_rows = rows;
+    }
+  }
+  return REWB200_OK;
+}
+
 }  // namespace
 
 // The layer runs of a layered model over `rows` rows; na carries the residual, the embedding and the ids.  Leaves the
@@ -1248,6 +1821,7 @@ int layered_blocks(rewb200_session* s, const FwdOpts& o, const NormArgs& na, int
   const int dt = m->cfg.dtype;
   const int64_t dp = m->dp;
   if (m->stack.block == BLOCK_OUTPUT_NORM) return output_norm_blocks(s, o, na, rows, in_graph);
+  if (m->stack.block == BLOCK_SANDWICH) return sandwich_blocks(s, o, na, rows, in_graph);
   void* const ff_in = m->stack.block == BLOCK_ONE_NORM ? s->xn : s->xn2;   // what the feed-forward reads
   const StepLists t = step_lists(s, o, rows);
   auto ahead_of = [&](size_t r, NormArgs& a) {  // what the norm launch in front of run r adds and writes

@@ -77,7 +77,8 @@ struct Ctx {
   bool record_layers = false;   // layered models keep the residual stream after every layer run (a test aid)
   int latent_impl = 0;          // latent attention: 0 by step size, 1 plain kernels, 2 always on the cached latents
   int gqa_impl = 0;             // layered grouped-query attention: 0 by step size, 1 plain kernels, 2 never the large-portion kernel
-  int gla_impl = 0;             // gated linear attention: 0 by step size, 1 plain kernels, 2 always token by token
+  int gla_impl = 0;             // gated linear attention and delta rule: 0 by step size, 1 plain kernels, 2 always token by token
+  int conv_impl = 0;            // short convolutions: 0 by size, 1 plain kernel
   int inject_alloc_fail = 0;  // test hook: the n-th activation allocation from now fails on the host
   int option_epoch = 0;      // bumped by rewb200_set_option; captured graphs from older epochs are rebuilt
   void* pinned = nullptr;    // pinned host staging for H2D/D2H of buffers
@@ -193,6 +194,7 @@ enum Epilogue : int {
   EPI_BIAS_BF16 = 2,    // out_bf16[row][col] = acc + bias[col]
   EPI_SWIGLU_BF16 = 3,  // columns interleaved gate/up in groups of 8: out[row][col/2..] = silu(g+bg)*(u+bu)
   EPI_RELU2_BF16 = 4,   // out_bf16[row][col] = max(acc + bias[col], 0)^2
+  EPI_GELU_BF16 = 5,    // out_bf16[row][col] = tanh GELU of acc + bias[col]
 };
 
 struct LinearBf16Plan {
@@ -285,12 +287,15 @@ int residual_norm_launch(Ctx* c, const NormArgs& a, int64_t rows);
 // dst = cap * tanh(src / cap), n columns of `rows` rows; src may be dst.
 int softcap_launch(Ctx* c, const float* src, int64_t lds, float* dst, int64_t ldd, int64_t rows, int64_t n, float cap);
 
-// Blocks whose sublayers read the residual itself and are normed on the way back: x += gamma * y / rms(y), y the sum of two
-// sets of f32 slabs.  Leaves x (or, with final_gamma, its RMS norm) in `out`.  Without slabs the row is only written out;
-// with an embedding table it starts from the row of its id.
+// Blocks whose sublayers are normed on the way back: x += gamma * y / rms(y), y the sum of two sets of f32 slabs and a bias.
+// Leaves x (or, with final_gamma, its RMS norm) in `out`.  Without slabs the row is only written out; with an embedding table
+// it starts from the scaled row of its id, and a row of a second table if there is one.
 struct OutputNormArgs {
   float* x_res;            // [rows][d]
   const void* embed;       // [vocab][d] act dtype or nullptr
+  float embed_scale;       // factor of the embedding row; 0 reads as 1
+  const void* embed2;      // second table [..][d] or nullptr
+  const int* ids2;         // its row for every row
   const int* ids;
   int vocab;
   const float* partial;    // [nsplit][rows][d]
@@ -298,15 +303,25 @@ struct OutputNormArgs {
   const float* partial2;
   int nsplit2;
   int64_t split_stride;
+  const float* bias;       // [d] added to the slabs' sum, or nullptr
+  int replace;             // 1: x becomes the sum itself, without norm
   const float* gamma;
   const float* final_gamma;
   float eps;
   int64_t d, d_mean;       // d_mean: width the statistics divide by when rows are padded with zeros (0: d)
   void* out;
+  int64_t ldo;             // row stride of out (0: d)
+  void* out_x;             // x itself, act dtype, row stride ldx, or nullptr
+  int64_t ldx;
   int dtype;
   int* status;
 };
 int output_norm_launch(Ctx* c, const OutputNormArgs& a, int64_t rows);
+// Rows of a bigram table: out[row] = (previous id * mul_prev + id * mul_cur) mod buckets, `buckets` for a sequence's first
+// token.  row_lane / row_pos nullptr: row r is the next token of lane b0 + r at position pos[b0 + r].  last: the last id of
+// every lane, read and brought up to date.
+int bigram_rows_launch(Ctx* c, const int* ids, const int* row_lane, const int* row_pos, const int* pos, int b0, int64_t rows, int64_t buckets,
+                       int64_t mul_prev, int64_t mul_cur, int vocab, int* last, int* out, int* status);
 
 struct KvLayout {
   void* k;                // [n_pages][kvh][page][hd]

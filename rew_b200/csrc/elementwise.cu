@@ -482,6 +482,8 @@ __global__ void __launch_bounds__(CL == 1 ? 512 : 256) output_norm_kernel(Output
     }
     erow = reinterpret_cast<const T*>(a.embed) + id * d + col0;
   }
+  const float es = a.embed_scale == 0.f ? 1.0f : a.embed_scale;
+  const T* erow2 = a.embed2 ? reinterpret_cast<const T*>(a.embed2) + (int64_t)a.ids2[row] * d + col0 : nullptr;
   // sum of squares over the row
   auto row_sum = [&](float v, int slot) -> float {
     v = block_sum(v, red);
@@ -503,15 +505,25 @@ __global__ void __launch_bounds__(CL == 1 ? 512 : 256) output_norm_kernel(Output
     const int64_t i = ((int64_t)c * THREADS + threadIdx.x) * 4;
     x[c] = y[c] = make_float4(0.f, 0.f, 0.f, 0.f);
     if (i >= dq) continue;
-    x[c] = erow ? Vec4<T>::load(erow + i) : *reinterpret_cast<const float4*>(xr + i);
+    if (erow) {
+      const float4 e = Vec4<T>::load(erow + i);
+      x[c] = make_float4(e.x * es, e.y * es, e.z * es, e.w * es);
+      if (erow2) add4(x[c], Vec4<T>::load(erow2 + i));
+    } else if (!a.replace) {
+      x[c] = *reinterpret_cast<const float4*>(xr + i);
+    }
     const int64_t at = row * d + col0 + i;
+    if (a.bias) y[c] = *reinterpret_cast<const float4*>(a.bias + col0 + i);
 #pragma unroll 8
     for (int s = 0; s < a.nsplit; ++s) add4(y[c], *reinterpret_cast<const float4*>(a.partial + s * a.split_stride + at));
 #pragma unroll 4
     for (int s = 0; s < a.nsplit2; ++s) add4(y[c], *reinterpret_cast<const float4*>(a.partial2 + s * a.split_stride + at));
     ss += y[c].x * y[c].x + y[c].y * y[c].y + y[c].z * y[c].z + y[c].w * y[c].w;
   }
-  if (a.nsplit + a.nsplit2 > 0) {
+  if (a.replace) {
+#pragma unroll
+    for (int c = 0; c < NCH; ++c) x[c] = y[c];
+  } else if (a.nsplit + a.nsplit2 > 0) {
     const float f = 1.0f / sqrtf(row_sum(ss, 0) / dm + a.eps);
 #pragma unroll
     for (int c = 0; c < NCH; ++c) {
@@ -528,12 +540,14 @@ __global__ void __launch_bounds__(CL == 1 ? 512 : 256) output_norm_kernel(Output
     for (int c = 0; c < NCH; ++c) ss += x[c].x * x[c].x + x[c].y * x[c].y + x[c].z * x[c].z + x[c].w * x[c].w;
     f2 = 1.0f / sqrtf(row_sum(ss, 1) / dm + a.eps);
   }
-  T* orow = reinterpret_cast<T*>(a.out) + row * d + col0;
+  T* orow = reinterpret_cast<T*>(a.out) + row * (a.ldo > 0 ? a.ldo : d) + col0;
+  T* oxrow = a.out_x ? reinterpret_cast<T*>(a.out_x) + row * a.ldx + col0 : nullptr;
 #pragma unroll
   for (int c = 0; c < NCH; ++c) {
     const int64_t i = ((int64_t)c * THREADS + threadIdx.x) * 4;
     if (i >= dq) continue;
     *reinterpret_cast<float4*>(xr + i) = x[c];
+    if (oxrow) Vec4<T>::store(oxrow + i, x[c]);
     float4 o = x[c];
     if (a.final_gamma) {
       const float4 g = *reinterpret_cast<const float4*>(a.final_gamma + col0 + i);
@@ -1145,6 +1159,42 @@ int output_norm_launch(Ctx* c, const OutputNormArgs& a, int64_t rows) {
   const int nch = (int)((a.d / 4 + 511) / 512);
   return bf ? RB_ONORM(bf16, 1) : RB_ONORM(float, 1);
 #undef RB_ONORM
+}
+
+// One CTA: all rows are looked up before any lane's last id changes.
+__global__ void __launch_bounds__(1024) bigram_rows_kernel(const int* ids, const int* row_lane, const int* row_pos, const int* pos, int b0, int64_t rows,
+                                                           int64_t buckets, int64_t mul_prev, int64_t mul_cur, int vocab, int* last, int* out, int* status) {
+  pdl_launch_dependents();
+  pdl_wait();
+  auto lane_of = [&](int64_t r) { return row_lane ? row_lane[r] : b0 + (int)r; };
+  auto pos_of = [&](int64_t r) { return row_pos ? row_pos[r] : pos[b0 + r]; };
+  for (int64_t r = threadIdx.x; r < rows; r += blockDim.x) {
+    const int p = pos_of(r), lane = lane_of(r);
+    int64_t h = buckets;
+    if (p > 0) {
+      const bool same = row_lane && r > 0 && row_lane[r - 1] == lane && row_pos[r - 1] == p - 1;
+      int a = same ? ids[r - 1] : last[lane], b = ids[r];
+      if (a < 0 || a >= vocab || b < 0 || b >= vocab) {
+        atomicExch(status, KS_BAD_INDEX);
+        a = b = 0;
+      }
+      h = (a * mul_prev + b * mul_cur) % buckets;
+      if (h < 0) h += buckets;
+    }
+    out[r] = (int)h;
+  }
+  __syncthreads();
+  for (int64_t r = threadIdx.x; r < rows; r += blockDim.x)
+    if (!row_lane || r + 1 == rows || row_lane[r + 1] != row_lane[r]) last[lane_of(r)] = ids[r];
+}
+
+int bigram_rows_launch(Ctx* c, const int* ids, const int* row_lane, const int* row_pos, const int* pos, int b0, int64_t rows, int64_t buckets,
+                       int64_t mul_prev, int64_t mul_cur, int vocab, int* last, int* out, int* status) {
+  if (rows == 0) return REWB200_OK;
+  RB_CUDA(launch_k(bigram_rows_kernel, dim3(1), dim3(1024), 0, c->stream, c->use_pdl, ids, row_lane, row_pos, pos, b0, rows, buckets, mul_prev, mul_cur,
+                   vocab, last, out, status));
+  ++g_launch_total;
+  return REWB200_OK;
 }
 
 // dst[r][i] = cap * tanh(src[r][i] / cap) for the first n columns of every row; src may be dst

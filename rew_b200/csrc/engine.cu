@@ -17,6 +17,7 @@
 //     captured once into a CUDA graph and replayed; token ids, positions and
 //     the step counter live on the device, so a run of n steps needs no host
 //     round trip until the ids are copied back.
+#include "act.cuh"
 #include "engine.cuh"
 
 using namespace rewb;
@@ -61,6 +62,26 @@ __global__ void swiglu_rows_f32_kernel(const float* gu, float* out, int64_t rows
 }
 
 // f32 path: out = max(x, 0)^2
+__global__ void gelu_f32_kernel(const float* x, float* out, int64_t n) {
+  const int64_t i = (int64_t)blockIdx.x * blockDim.x + threadIdx.x;
+  if (i < n) out[i] = gelu_tanh_act(x[i]);
+}
+
+// bf16 tanh GELU of four columns' slab sums and biases; N is a multiple of 8
+__global__ void __launch_bounds__(128) gelu_slabs_kernel(const float* part, int ksplit, int64_t rows, int64_t N, const float* bias, bf16* out) {
+  pdl_launch_dependents();
+  const int64_t i = ((int64_t)blockIdx.x * 128 + threadIdx.x) * 4;
+  if (i >= rows * N) return;
+  float4 v = *reinterpret_cast<const float4*>(bias + i % N);
+  pdl_wait();
+#pragma unroll 4
+  for (int s = 0; s < ksplit; ++s) {
+    const float4 p = *reinterpret_cast<const float4*>(part + s * rows * N + i);
+    v.x += p.x; v.y += p.y; v.z += p.z; v.w += p.w;
+  }
+  *reinterpret_cast<uint2*>(out + i) = make_uint2(pack_bf16(gelu_tanh_fast(v.x), gelu_tanh_fast(v.y)), pack_bf16(gelu_tanh_fast(v.z), gelu_tanh_fast(v.w)));
+}
+
 __global__ void relu2_f32_kernel(const float* x, float* out, int64_t n) {
   const int64_t i = (int64_t)blockIdx.x * blockDim.x + threadIdx.x;
   if (i >= n) return;
@@ -266,6 +287,13 @@ int swiglu_rows_f32_launch(Ctx* c, const float* gu, float* out, int64_t rows, in
   return REWB200_OK;
 }
 
+int gelu_f32_launch(Ctx* c, const float* x, float* out, int64_t n) {
+  gelu_f32_kernel<<<(unsigned)((n + 255) / 256), 256, 0, c->stream>>>(x, out, n);
+  RB_CUDA(cudaGetLastError());
+  ++g_launch_total;
+  return REWB200_OK;
+}
+
 int ensure_acts(rewb200_session* s, int64_t rows, int64_t logits_rows) {
   rewb200_model* m = s->m;
   const rewb200_config& c = m->cfg;
@@ -276,7 +304,8 @@ int ensure_acts(rewb200_session* s, int64_t rows, int64_t logits_rows) {
                      (void**)&s->moe_logits, (void**)&s->moe_topw, (void**)&s->moe_topi, (void**)&s->moe_ints, &s->moe_send,
                      &s->moe_recv, &s->moe_xs, &s->moe_hs, (void**)&s->moe_ys, (void**)&s->moe_ret, (void**)&s->moe_back,
                      (void**)&s->moe_tmp, (void**)&s->route_rec, &s->xn2, &s->cq, (void**)&s->gate, (void**)&s->part2,
-                     (void**)&s->part3, (void**)&s->shared_gate, (void**)&s->layer_rec};
+                     (void**)&s->part3, (void**)&s->shared_gate, (void**)&s->layer_rec, &s->cat, &s->conv, (void**)&s->gate_pre,
+                     (void**)&s->group_rows, (void**)&s->big_rows};
     // From here until every allocation below has succeeded the session holds no activation buffers: a failed
     // growth must leave it in a state where the next call allocates again instead of launching on NULL.
     s->rows_cap = 0;
@@ -391,12 +420,19 @@ int run_linear(rewb200_session* s, const LinW& w, const void* x, int64_t ldx, in
       }
     }
     if (ksplit_out) *ksplit_out = ks;
-    if (!partial && epi == EPI_SWIGLU_BF16 && rows <= 64 && w.N % 16 == 0 && c->gu_split) {
-      // a gate|up with too few feature tiles to fill the GPU: split K, then sum + SwiGLU in a second small launch
+    if (!partial && (epi == EPI_SWIGLU_BF16 || epi == EPI_GELU_BF16) && rows <= 64 && w.N % 16 == 0 && c->gu_split) {
+      // a gate|up with too few feature tiles to fill the GPU: split K, then sum + activation in a second small launch
       int kg = std::min(4, linear_bf16_pick_ksplit(c, rows, w.K, w.N));
       while (kg > 1 && (size_t)kg * rows * w.N * sizeof(float) > s->part_bytes) kg /= 2;
       if (kg > 1) {
         RB_TRY(linear_bf16_launch(c, w.plan, (const bf16*)x, ldx, rows, EPI_PARTIAL_F32, kg, s->part, w.N, nullptr, nullptr, 0));
+        if (epi == EPI_GELU_BF16) {
+          RB_REQUIRE(ldo == w.N, "GELU output rows must be dense");
+          RB_CUDA(launch_k(gelu_slabs_kernel, dim3((unsigned)((rows * w.N / 4 + 127) / 128)), dim3(128), 0, c->stream, c->use_pdl,
+                           (const float*)s->part, kg, rows, w.N, (const float*)w.b, (bf16*)out));
+          ++g_launch_total;
+          return REWB200_OK;
+        }
         const int64_t n = rows * (w.N / 16);
         RB_REQUIRE(ldo == w.N / 2, "SwiGLU output rows must be dense");
         RB_CUDA(launch_k(swiglu_slabs_il_kernel, dim3((unsigned)((n + 127) / 128)), dim3(128), 0, c->stream, c->use_pdl,
@@ -1638,12 +1674,13 @@ void rewb200_session_free(rewb200_session* s) {
   if (s->graph) cudaGraphExecDestroy(s->graph);
   for (void* p : s->kc) cudaFree(p);
   for (void* p : s->vc) cudaFree(p);
-  for (void* p : s->state) cudaFree(p);
+  for (const auto* list : {&s->state, &s->conv_state, &s->state2})
+    for (void* p : *list) cudaFree(p);
   void* ptrs[] = {s->d_active, s->d_ids_prefill, s->block_table, s->d_pos, s->d_ids, s->d_next, s->d_out, s->d_step, s->x_res, s->xn, s->q,
                   s->attn, s->h, s->part, s->gu32, s->logits, s->attn_scratch, s->argmax_scratch, s->gather_scratch,
                   s->samp_hist, s->samp_hist_len, s->samp_steps, s->samp_keys, s->samp_work, s->samp_logprob, s->moe_logits, s->moe_topw, s->moe_topi, s->moe_ints,
                   s->moe_send, s->moe_recv, s->moe_xs, s->moe_hs, s->moe_ys, s->moe_ret, s->moe_back, s->moe_tmp, s->route_rec,
-                  s->xn2, s->cq, s->gate, s->part2, s->part3, s->shared_gate, s->qeff, s->olat, s->ml, s->gqa_part, s->gqa_ml, s->gla_work, s->kvx, s->latx, s->layer_rec, s->xg, s->logits_pad, s->plan_dev, s->feed_dev};
+                  s->xn2, s->cq, s->gate, s->part2, s->part3, s->shared_gate, s->qeff, s->olat, s->ml, s->gqa_part, s->gqa_ml, s->gla_work, s->kvx, s->latx, s->layer_rec, s->xg, s->logits_pad, s->plan_dev, s->feed_dev, s->cat, s->conv, s->gate_pre, s->group_rows, s->big_rows, s->last_ids, s->mix_work};
   for (void* p : ptrs)
     if (p) cudaFree(p);
   if (s->h_ids) cudaFreeHost(s->h_ids);

@@ -5,9 +5,13 @@
 #include <cstring>
 
 #include "common.cuh"
+#include "conv.cuh"
+#include "delta.cuh"
 #include "gla.cuh"
 #include "gqa.cuh"
+#include "gqa_mix.cuh"
 #include "latent.cuh"
+#include "lru.cuh"
 #include "ptx.cuh"
 
 namespace rewb {
@@ -93,7 +97,8 @@ struct LatentDev {
 struct GqaDev {
   GqaDims m = {};
   LinW in;                     // [d, heads * dim | kv_heads * dim | kv_heads * vdim | heads]: queries, keys, values (unless v_from_k), gate
-  float *q_norm = nullptr, *k_norm = nullptr, *bias = nullptr, *sink = nullptr, *conv = nullptr;
+  float *q_norm = nullptr, *k_norm = nullptr, *bias = nullptr, *sink = nullptr, *conv = nullptr, *in_bias = nullptr, *talk = nullptr;
+  int64_t gate_col = 0;        // of the gate in `in`
   int64_t ldk = 0, ldv = 0;    // elements of a cached key / value row, padded
 };
 
@@ -102,6 +107,24 @@ struct GlaDev {
   GlaDims m = {};
   LinW in;                     // [d, heads * dim | heads * dim | heads * vdim | heads * vdim | rank]: q, k, v, gate, decay features
   float *a2 = nullptr, *a2_b = nullptr, *norm = nullptr;
+};
+
+// Gated delta rule of one layer (delta.cuh).
+struct DeltaDev {
+  DeltaDims m = {};
+  ConvDims conv = {};          // of queries, keys and values
+  LinW in;                     // [d, kv_heads * dim | kv_heads * dim | heads * vdim | heads * vdim | heads | heads]: q, k, v, gate, step, decay
+  float *w = nullptr, *rate = nullptr, *dt_bias = nullptr, *norm = nullptr;
+};
+
+// Linear recurrent unit of one layer (lru.cuh).
+struct LruDev {
+  LruDims m = {};
+  ConvDims conv = {};
+  LinW in;                     // [d, width | width]: output branch, recurrent branch
+  void* gates = nullptr;       // [blocks][ldn][2 ldn]: both gates of a block
+  LinearBf16Plan plan_gates;
+  float *w = nullptr, *x_bias = nullptr, *conv_bias = nullptr, *y_bias = nullptr, *gate_bias = nullptr, *decay = nullptr;
 };
 
 struct LayerDev {
@@ -114,7 +137,13 @@ struct LayerDev {
   LatentDev a;
   GqaDev g;
   GlaDev l;
+  DeltaDev d;
+  LruDev r;
+  int beside = 0;              // mixer of the second one on the same input, and the first of its columns in the first one's
+  int64_t beside_in = 0, beside_out = 0;   // input projection and of its rows in `o`
+  float *back1 = nullptr, *back2 = nullptr;   // norms of the sublayers' outputs
   int ff = 0;                  // layered models: rewb200_layer::ff
+  bool gelu = false;           // dense feed-forward W_down gelu(W_up x)
 };
 
 // One execution of a layer of a layered model; a layer inside the loop runs once per pass, each with its own cache.
@@ -150,6 +179,8 @@ struct rewb200_model {
   rewb200_stack stack = {};
   std::vector<LayerRun> runs;
   float* step_vec = nullptr;    // [loop_times][dp]
+  void* bigram = nullptr;       // [bigram_buckets + 1][dp]
+  LinW loop_in;                 // [2 dp, dp]
   int64_t dp = 0;               // row stride of the residual stream: d_model, padded to a multiple of 8 (layered)
   int64_t vp = 0;               // columns of the lm_head matrix: the vocabulary, padded
   int max_topk = 0, max_experts = 0, n_moe = 0;   // n_moe: MoE layer runs of a step
@@ -165,6 +196,8 @@ struct rewb200_session {
   std::vector<void*> kc, vc;           // per layer
   std::vector<CUtensorMap> tmK, tmV;   // per layer (bf16)
   std::vector<float*> state;           // layered models: recurrent or convolution state per layer run [B][..] f32, or nullptr
+  std::vector<float*> conv_state, state2;  // convolution state beside a recurrent one, and the recurrent state of a second mixer
+  int* last_ids = nullptr;             // the last id of every lane (bigram tables)
   int* block_table = nullptr;
   int *d_pos = nullptr, *d_ids = nullptr, *d_next = nullptr, *d_out = nullptr, *d_step = nullptr;
   int out_capacity = 0;
@@ -211,6 +244,13 @@ struct rewb200_session {
   int64_t gqa_units = 0, gqa_stats = 0;
   void *kvx = nullptr, *latx = nullptr;  // keys / values expanded per head, and the gathered cache rows they come from
   int64_t kvx_rows = 0;
+  void* cat = nullptr;                 // rows [x | embeddings] that open a pass of a loop
+  void* conv = nullptr;                // what leaves a convolution
+  float* gate_pre = nullptr;           // gates of a linear recurrent unit ahead of their sigmoids
+  int* group_rows = nullptr;           // first row of every block of them
+  int* big_rows = nullptr;             // rows of the bigram table
+  float* mix_work = nullptr;           // scores of attention with mixed heads
+  size_t mix_bytes = 0;
   float* layer_rec = nullptr;          // option record_layers: [runs][rows_cap][d]
   int64_t layer_rows = 0;
   void* xg = nullptr;                  // rows of xn gathered for the lm_head
@@ -221,7 +261,8 @@ struct rewb200_session {
   std::vector<int> plan_host;
   int plan_abs_tiles = 0, plan_chunks = 0, plan_exp_tiles = 0, plan_keys = 0, plan_tails = 0;
   int plan_gqa_small = 0, plan_gqa_large = 0, plan_gla_small = 0, plan_gla_large = 0, plan_gla_chunks = 0;
-  uint8_t* gla_work = nullptr;         // blocks of the chunks of gated linear attention
+  int plan_delta_small = 0, plan_delta_large = 0, plan_delta_chunks = 0, plan_portions = 0, plan_longest = 0;
+  uint8_t* gla_work = nullptr;         // blocks of the chunks of gated linear attention or of the delta rule
   size_t gla_work_bytes = 0;
   int* feed_dev = nullptr;             // ids and row lists of a rewb200_lanes_feed step
   size_t feed_cap = 0;
@@ -329,6 +370,7 @@ int acts_alloc(Ctx* c, void** p, size_t bytes);
 int run_linear(rewb200_session* s, const LinW& w, const void* x, int64_t ldx, int64_t rows, bool partial, int epi,
                void* out, int64_t ldo, int* ksplit_out, const QkvPostArgs* fuse_qkv = nullptr, bool* fused = nullptr);
 int swiglu_rows_f32_launch(Ctx* c, const float* gu, float* out, int64_t rows, int64_t f);
+int gelu_f32_launch(Ctx* c, const float* x, float* out, int64_t n);
 // Routed experts of one MoE layer for the normalised rows x [rows][d]: router, top-k, expert Linears, weighted sum
 // into `out` (nullptr: slab 0 of s->part).
 int moe_routed(rewb200_session* s, MoeDev& X, const void* x, int64_t d, int64_t rows, bool accumulate, float* out = nullptr,

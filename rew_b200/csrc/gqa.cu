@@ -129,7 +129,7 @@ __global__ void __launch_bounds__(256) gqa_post_kernel(GqaPostArgs a, int64_t ro
   auto ahead_of = [&](int r) { return min(__clz(~(cont << (31 - HIST - r))), HIST); };   // rows of its portion ahead of row r in this step, at most HIST
   auto state_at = [&](int lane, int pos) -> float* { return a.state + ((int64_t)lane * (a.m.taps - 1) + pos % (a.m.taps - 1)) * C + col; };
   float4 t0 = make_float4(0.f, 0.f, 0.f, 0.f), t1 = t0;   // (cos, sin) of this lane's four features
-  const bool rot_reg = PC == 1 && half > 0 && half % 4 == 0;
+  const bool rot_reg = PC == 1 && half > 0 && half % 4 == 0 && !a.m.pairs;
   auto rope_row = [&](int pos) { return a.m.rope + (int64_t)(ok_at(pos) ? pos : 0) * half; };
   auto rope_load = [&](int pos) {
     const int i = ln * 4;
@@ -198,6 +198,14 @@ __global__ void __launch_bounds__(256) gqa_post_kernel(GqaPostArgs a, int64_t ro
 #pragma unroll
       for (int c = 0; c < PC; ++c) x[r][c] = r < nr ? slab4(a, p + r * a.ld + col, (c * 32 + ln) * 4, n) : make_float4(0.f, 0.f, 0.f, 0.f);
   }
+  if (a.m.in_bias) {
+#pragma unroll
+    for (int c = 0; c < PC; ++c) {
+      const float4 b = slab4(a.m.in_bias + col, 1, 0, (c * 32 + ln) * 4, n);
+#pragma unroll
+      for (int r = 0; r < RW; ++r) add4(x[r][c], b);
+    }
+  }
   if constexpr (TIME) {
     if (conv_reg) {
       if (a.map.row_lane) {
@@ -258,11 +266,11 @@ __global__ void __launch_bounds__(256) gqa_post_kernel(GqaPostArgs a, int64_t ro
     if (r >= nr) break;
     const int pos = pos_of(r), page = __shfl_sync(ALL, my_page, r + HIST);
     float f = 1.f;
-    if (w) {
+    if (w || (is_v && a.m.v_norm)) {
       float ss = 0.f;
 #pragma unroll
       for (int c = 0; c < PC; ++c) ss += x[r][c].x * x[r][c].x + x[r][c].y * x[r][c].y + x[r][c].z * x[r][c].z + x[r][c].w * x[r][c].w;
-      f = 1.0f / sqrtf(warp_sum(ss) / (float)K + a.eps);
+      f = 1.0f / sqrtf(warp_sum(ss) / (float)n + a.eps);
     }
     if (is_q && a.m.temp_every > 0) f *= 1.0f + a.m.temp_coef * logf((float)((pos + 1) / a.m.temp_every + 1));
     T* dst;
@@ -288,6 +296,21 @@ __global__ void __launch_bounds__(256) gqa_post_kernel(GqaPostArgs a, int64_t ro
         const float4 o = make_float4(__shfl_sync(ALL, e.x, from), __shfl_sync(ALL, e.y, from), __shfl_sync(ALL, e.z, from), __shfl_sync(ALL, e.w, from));
         if (ln * 4 < 2 * half)
           x[r][0] = make_float4(e.x * t0.x + sg * (o.x * t0.y), e.y * t0.z + sg * (o.y * t0.w), e.z * t1.x + sg * (o.z * t1.y), e.w * t1.z + sg * (o.w * t1.w));
+      } else if (half > 0 && a.m.pairs) {
+        const float2* cs = rope_row(pos);
+#pragma unroll
+        for (int c = 0; c < PC; ++c) {
+          const int i = (c * 32 + ln) * 2;     // this lane's first pair
+          float4& e = x[r][c];
+          if (i < half) {
+            const float2 t = cs[i];
+            e = make_float4(e.x * t.x - e.y * t.y, e.y * t.x + e.x * t.y, e.z, e.w);
+          }
+          if (i + 1 < half) {
+            const float2 t = cs[i + 1];
+            e = make_float4(e.x, e.y, e.z * t.x - e.w * t.y, e.w * t.x + e.z * t.y);
+          }
+        }
       } else if (half > 0) {
         float* s = s_rot[threadIdx.x >> 5];
         const float2* cs = rope_row(pos);
@@ -339,6 +362,8 @@ __global__ void __launch_bounds__(256, 4) gqa_post_rows_kernel(GqaPostArgs a, in
     if (on && !is_v && b < a.m.taps) cw[b] = *reinterpret_cast<const float4*>(a.m.conv + (a.m.taps - 1 - b) * C + col);
   }
   const float* w = is_v ? nullptr : is_q ? a.m.q_norm : a.m.k_norm;
+  const bool normed = w || (is_v && a.m.v_norm);
+  const float4 bias = a.m.in_bias && on ? make_float4(a.m.in_bias[col], a.m.in_bias[col + 1], a.m.in_bias[col + 2], a.m.in_bias[col + 3]) : zero;
   const float4 g = NORM && w && on ? make_float4(w[i], w[i + 1], w[i + 2], w[i + 3]) : one;
   pdl_wait();
   if ((int)threadIdx.x < nr) {
@@ -368,6 +393,7 @@ __global__ void __launch_bounds__(256, 4) gqa_post_rows_kernel(GqaPostArgs a, in
   }
   auto value = [&](const float* p) {
     float4 v = on ? *reinterpret_cast<const float4*>(p) : zero;
+    add4(v, bias);
     for (int s = 1; s < a.nsplit; ++s)
       if (on) add4(v, *reinterpret_cast<const float4*>(p + s * a.split_stride));
     return v;
@@ -389,7 +415,7 @@ __global__ void __launch_bounds__(256, 4) gqa_post_rows_kernel(GqaPostArgs a, in
   const bool lo = i < half, turned = i < 2 * half;
   const int from = (lo ? ln + half / 4 : ln - half / 4) & 31;
   const float sg = lo ? -1.f : 1.f;
-  const float2* const rope = a.m.rope + (lo ? i : i - half);
+  const float2* const rope = a.m.rope + (a.m.pairs ? i / 2 : lo ? i : i - half);
   const int hk = is_v ? unit - H - G : unit - H;
   T* const q = reinterpret_cast<T*>(a.q) + row0 * a.ldq + (int64_t)unit * K + i;
   T* const kc = reinterpret_cast<T*>(a.kc) + (int64_t)hk * PAGE_TOKENS * a.ldk + i;
@@ -408,7 +434,7 @@ __global__ void __launch_bounds__(256, 4) gqa_post_rows_kernel(GqaPostArgs a, in
     if (turned) {
       const float2* cs = rope + (int64_t)max(in.x, 0) * half;
       t0 = *reinterpret_cast<const float4*>(cs);
-      t1 = *reinterpret_cast<const float4*>(cs + 2);
+      if (!a.m.pairs) t1 = *reinterpret_cast<const float4*>(cs + 2);
     }
     if (in.z == 0 && r > 0) from_state(in, 1);      // a portion starts here
     float4 y = make_float4(cw[0].x * x.x, cw[0].y * x.y, cw[0].z * x.z, cw[0].w * x.w);
@@ -422,11 +448,13 @@ __global__ void __launch_bounds__(256, 4) gqa_post_rows_kernel(GqaPostArgs a, in
     if (twice && on && in.x >= 0) put(vc + (int64_t)in.y * a.ldv, y);
     if constexpr (NORM) {
       float f = 1.f;
-      if (w) f = 1.0f / sqrtf(warp_sum(y.x * y.x + y.y * y.y + y.z * y.z + y.w * y.w) / (float)K + a.eps);
+      if (normed) f = 1.0f / sqrtf(warp_sum(y.x * y.x + y.y * y.y + y.z * y.z + y.w * y.w) / (float)n + a.eps);
       if (is_q && a.m.temp_every > 0) f *= 1.0f + a.m.temp_coef * logf((float)((in.x + 1) / a.m.temp_every + 1));
       y = make_float4(y.x * f * g.x, y.y * f * g.y, y.z * f * g.z, y.w * f * g.w);
     }
-    if (half > 0) {
+    if (half > 0 && a.m.pairs) {
+      if (turned) y = make_float4(y.x * t0.x - y.y * t0.y, y.y * t0.x + y.x * t0.y, y.z * t0.z - y.w * t0.w, y.w * t0.z + y.z * t0.w);
+    } else if (half > 0) {
       const float4 o = make_float4(__shfl_sync(ALL, y.x, from), __shfl_sync(ALL, y.y, from), __shfl_sync(ALL, y.z, from), __shfl_sync(ALL, y.w, from));
       if (turned) y = make_float4(y.x * t0.x + o.x * (sg * t0.y), y.y * t0.z + o.y * (sg * t0.w), y.z * t1.x + o.z * (sg * t1.y), y.w * t1.z + o.w * (sg * t1.w));
     }
@@ -862,7 +890,7 @@ int gqa_post_launch(Ctx* c, const GqaPostArgs& a, int64_t rows) {
     int tr = MAX_TR;         // long walks, but four CTAs for every SM
     while (tr > 4 && (rows + tr - 1) / tr * grid.y < 4 * c->sm_count) tr /= 2;
     const dim3 g((unsigned)((rows + tr - 1) / tr), grid.y);
-    const bool norm = a.m.q_norm || a.m.k_norm || a.m.temp_every > 0;
+    const bool norm = a.m.q_norm || a.m.k_norm || a.m.temp_every > 0 || a.m.v_norm;
     auto go_rows = [&](auto kernel) { return launch_k(kernel, g, dim3(256), 0, c->stream, c->use_pdl, a, rows, tr); };
     RB_CUDA(bf ? (norm ? go_rows(gqa_post_rows_kernel<bf16, true>) : go_rows(gqa_post_rows_kernel<bf16, false>))
                : (norm ? go_rows(gqa_post_rows_kernel<float, true>) : go_rows(gqa_post_rows_kernel<float, false>)));

@@ -1,7 +1,8 @@
 // Grouped-query attention of layered models: a short causal convolution over time on queries and keys, per-head RMS norms,
 // a query temperature that grows with the position, rotated features, a learned bias per head and distance bucket, a number
-// per head in the softmax denominator ("sink"), an output gate per head, each of them optional.  Argument structs and
-// launchers of gqa.cu and gqa_prefill.cu.
+// per head in the softmax denominator ("sink"), an output gate per head, each of them optional.  Layers with a window, kept first
+// keys, mixed heads or a gate per feature run the kernels of gqa_mix.cuh.  Argument structs and launchers of gqa.cu and
+// gqa_prefill.cu.
 //
 // Caches: keys [pages][kv_heads][64][ldk], values [pages][kv_heads][64][ldv].
 #pragma once
@@ -26,7 +27,16 @@ struct GqaDims {
   const float* conv;       // [taps][gqa_channels]: the weight of the value taps - 1 - j tokens ago is row j
   int rope_dims;           // rotated features at the start of a head, pairs (i, i + rope_dims / 2); 0: none
   const float2* rope;      // [max_pos][rope_dims / 2] (cos, sin)
+  int pairs;               // rotated features are pairs (2i, 2i + 1)
+  int v_norm;              // values are divided by their root mean square
+  const float* in_bias;    // by column of the projection's queries, keys and values, or nullptr (no convolution then)
+  int window, keep_first;  // keys a query sees, itself included (0: all), and the first keys of the sequence it sees besides
+  const float* talk;       // [heads][heads] mixes the heads' weights after the softmax, or nullptr
+  int gate_elem;           // the output gate is per feature
+  float out_scale;         // of the output
 };
+// What the kernels of gqa_mix.cuh are for.
+inline bool gqa_is_mixed(const GqaDims& m) { return m.window > 0 || m.talk || m.gate_elem || m.out_scale != 1.0f; }
 
 // Channels of the projection the convolution runs on: queries, then keys of its own.
 inline __host__ __device__ int64_t gqa_channels(const GqaDims& m) { return (int64_t)(m.heads + (m.own_kv ? m.kv_heads : 0)) * m.dim; }
@@ -35,8 +45,8 @@ inline __host__ __device__ int64_t gqa_channels(const GqaDims& m) { return (int6
 inline int64_t gqa_state_elems(const GqaDims& m) { return m.taps > 1 ? (m.taps - 1) * gqa_channels(m) : 0; }
 
 // Finishes the fused input projection [q | k | v | gate] (q | gate without keys of its own, no v where the values are the
-// keys): sums the split-K slabs, runs the convolution, norms queries and keys, applies the temperature, rotates, appends keys
-// and values to the cache.
+// keys): sums the split-K slabs, adds biases, runs the convolution, norms queries, keys and values, applies the temperature,
+// rotates, appends keys and values to the cache.  A gate per feature is left to the kernel that reads it.
 struct GqaPostArgs {
   GqaDims m;
   const float* partial;    // [nsplit][rows][ld]

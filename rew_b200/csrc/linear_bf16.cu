@@ -18,6 +18,7 @@
 // kernel serves the grouped launches of the MoE experts (blockIdx.z = expert,
 // 3-D tensor map, device-side row offsets) and stays selectable for everything
 // else with the option linear = "mma" (128-row tiles for more than 64 rows).
+#include "act.cuh"
 #include "common.cuh"
 #include "ptx.cuh"
 
@@ -237,6 +238,9 @@ __global__ void __launch_bounds__(160) linear_bf16_kernel(const __grid_constant_
               if (a.epi == EPI_RELU2_BF16) {
                 v0 = fmaxf(v0, 0.f) * fmaxf(v0, 0.f);
                 v1 = fmaxf(v1, 0.f) * fmaxf(v1, 0.f);
+              } else if (a.epi == EPI_GELU_BF16) {
+                v0 = gelu_tanh_fast(v0);
+                v1 = gelu_tanh_fast(v1);
               }
               bf16* o = reinterpret_cast<bf16*>(a.out) + grow * a.ldo + c;
               *reinterpret_cast<uint32_t*>(o) = pack_bf16(v0, v1);

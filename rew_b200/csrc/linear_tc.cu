@@ -22,6 +22,7 @@
 // exit, where TMEM is released.
 #include <string.h>
 
+#include "act.cuh"
 #include "common.cuh"
 #include "ptx.cuh"
 #include "tc.cuh"
@@ -81,9 +82,10 @@ __device__ __forceinline__ float ld_dsmem_f32(uint32_t cluster_addr) {
 }
 
 __device__ __forceinline__ float silu_f(float x) { return x * (1.0f / (1.0f + __expf(-x))); }
-// bf16 outputs: the square of relu (EPI_RELU2_BF16) or the value itself
-__device__ __forceinline__ float act_f(float v, bool relu2) {
-  if (!relu2) return v;
+// bf16 outputs: the square of relu (EPI_RELU2_BF16), tanh GELU (EPI_GELU_BF16) or the value itself
+__device__ __forceinline__ float act_f(float v, int epi) {
+  if (epi == EPI_GELU_BF16) return gelu_tanh_fast(v);
+  if (epi != EPI_RELU2_BF16) return v;
   v = fmaxf(v, 0.f);
   return v * v;
 }
@@ -365,14 +367,13 @@ __global__ void __launch_bounds__(192) linear_tc_kernel(const __grid_constant__ 
             else if (a.epi == EPI_BIAS_F32)
               reinterpret_cast<float*>(a.out)[grow * a.ldo + feat] = v;
             else
-              reinterpret_cast<bf16*>(a.out)[grow * a.ldo + feat] = __float2bfloat16_rn(act_f(v, a.epi == EPI_RELU2_BF16));
+              reinterpret_cast<bf16*>(a.out)[grow * a.ldo + feat] = __float2bfloat16_rn(act_f(v, a.epi));
           }
         }
       }
     } else {
       const bool swiglu = a.epi == EPI_SWIGLU_BF16;
       const bool out_f32 = a.epi == EPI_PARTIAL_F32 || a.epi == EPI_BIAS_F32;
-      const bool relu2 = a.epi == EPI_RELU2_BF16;
       const int tile_cols = swiglu ? 64 : 128;
       const int row_bytes = tile_cols * (out_f32 ? 4 : 2);
       uint8_t* stg = smem;
@@ -407,7 +408,7 @@ __global__ void __launch_bounds__(192) linear_tc_kernel(const __grid_constant__ 
           } else {
   #pragma unroll
             for (int j = 0; j < 32; ++j)
-              reinterpret_cast<bf16*>(stg + (c0 + j) * row_bytes)[q * 32 + lane] = __float2bfloat16_rn(act_f(__uint_as_float(r[j]) + bias_v, relu2));
+              reinterpret_cast<bf16*>(stg + (c0 + j) * row_bytes)[q * 32 + lane] = __float2bfloat16_rn(act_f(__uint_as_float(r[j]) + bias_v, a.epi));
           }
         }
       }
@@ -638,7 +639,6 @@ __global__ void __launch_bounds__(192) linear_tc_persist_kernel(const __grid_con
     const int et = threadIdx.x - 64;
     const bool swiglu = a.epi == EPI_SWIGLU_BF16;
     const bool out_f32 = a.epi == EPI_PARTIAL_F32 || a.epi == EPI_BIAS_F32;
-    const bool relu2 = a.epi == EPI_RELU2_BF16;
     const int tile_cols = swiglu ? 64 : 128;
     const int row_bytes = tile_cols * (out_f32 ? 4 : 2);
     const int chunks_per_row = row_bytes / 16;
@@ -675,7 +675,7 @@ __global__ void __launch_bounds__(192) linear_tc_persist_kernel(const __grid_con
           } else {
 #pragma unroll
             for (int jj = 0; jj < 32; ++jj)
-              reinterpret_cast<bf16*>(stg + jj * C::STG_LD)[q * 32 + lane] = __float2bfloat16_rn(act_f(__uint_as_float(r[jj]) + bias_v, relu2));
+              reinterpret_cast<bf16*>(stg + jj * C::STG_LD)[q * 32 + lane] = __float2bfloat16_rn(act_f(__uint_as_float(r[jj]) + bias_v, a.epi));
           }
         }
         asm volatile("bar.sync 1, 128;" ::: "memory");  // the four epilogue warps only
@@ -890,7 +890,6 @@ __global__ void __cluster_dims__(2, 1, 1) __launch_bounds__(192) linear_tc_pair_
     const int et = threadIdx.x - 64;
     const bool swiglu = a.epi == EPI_SWIGLU_BF16;
     const bool out_f32 = a.epi == EPI_PARTIAL_F32 || a.epi == EPI_BIAS_F32;
-    const bool relu2 = a.epi == EPI_RELU2_BF16;
     const int tile_cols = swiglu ? 64 : 128;
     const int row_bytes = tile_cols * (out_f32 ? 4 : 2);
     const int chunks_per_row = row_bytes / 16;
@@ -927,7 +926,7 @@ __global__ void __cluster_dims__(2, 1, 1) __launch_bounds__(192) linear_tc_pair_
           } else {
 #pragma unroll
             for (int jj = 0; jj < 32; ++jj)
-              reinterpret_cast<bf16*>(stg + jj * C::STG_LD)[q * 32 + lane] = __float2bfloat16_rn(act_f(__uint_as_float(r[jj]) + bias_v, relu2));
+              reinterpret_cast<bf16*>(stg + jj * C::STG_LD)[q * 32 + lane] = __float2bfloat16_rn(act_f(__uint_as_float(r[jj]) + bias_v, a.epi));
           }
         }
         asm volatile("bar.sync 1, 128;" ::: "memory");  // the four epilogue warps only

@@ -301,6 +301,9 @@ int rewb200_set_option(int slot, const char* key, const char* value) {
   } else if (k == "linear_attention") {
     RB_REQUIRE(v == "auto" || v == "plain" || v == "recurrent", "option linear_attention: expected auto, plain or recurrent");
     c->gla_impl = v == "plain" ? 1 : v == "recurrent" ? 2 : 0;
+  } else if (k == "short_conv") {
+    RB_REQUIRE(v == "auto" || v == "plain", "option short_conv: expected auto or plain");
+    c->conv_impl = v == "plain" ? 1 : 0;
   } else if (k == "inject_alloc_fail") {
     const int n = atoi(v.c_str());
     RB_REQUIRE(n >= 0, "option inject_alloc_fail: a non-negative count");

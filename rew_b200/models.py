@@ -37,6 +37,15 @@ def _load_kugirax(path, dtype, max_seq, slot):
     return kugirax.load(path, dtype, max_seq, slot)
 
 
+def _is_musavik(cfg):
+    return cfg.get("architecture") == "Musavik"
+
+
+def _load_musavik(path, dtype, max_seq, slot):
+    from . import musavik
+    return musavik.load(path, dtype, max_seq, slot)
+
+
 def _is_hf_llama(cfg):
     return cfg.get("model_type") == "llama" or "LlamaForCausalLM" in (cfg.get("architectures") or [])
 
@@ -52,6 +61,7 @@ FAMILIES = [
     ("rezupel", _is_rezupel, _load_rezupel),
     ("girulorn", _is_girulorn, _load_girulorn),
     ("kugirax", _is_kugirax, _load_kugirax),
+    ("musavik", _is_musavik, _load_musavik),
     ("llama", _is_hf_llama, _load_hf_llama),
 ]
 
