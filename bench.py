@@ -84,6 +84,9 @@ WORKLOADS = {
     "kugirax_b1": dict(model="kugirax.dense_8b", batch=1, prompt=512),
     "kugirax_b8_s2048": dict(model="kugirax.dense_8b", batch=8, prompt=2048),
     "kugirax_moe_b64": dict(model="kugirax.moe_lite", batch=64, prompt=256),
+    "musavik_b32": dict(model="musavik.dense_8b", batch=32, prompt=512),
+    "musavik_b1": dict(model="musavik.dense_8b", batch=1, prompt=512),
+    "musavik_b8_s2048": dict(model="musavik.dense_8b", batch=8, prompt=2048),
     "moe_b1": dict(model="deepseek_v2_lite", batch=1, prompt=512),
     "moe_b8_s2048": dict(model="deepseek_v2_lite", batch=8, prompt=2048),
     # the attention operator alone: batch 8, 32 query / 8 kv heads, head_dim 128, 4096 positions

@@ -72,14 +72,14 @@ def load(model_dir, dtype, max_seq=None, slot=0):
 
 # Benchmark configuration (shapes only; weights are synthetic).
 def dense_8b(**kw):
-    """Layers of the width and heads of the 8B Llama shape; the feed-forward without a gate has as many weights.  Recurrent
-    blocks and attention beside the delta rule take turns; no loop."""
+    """As many layers, the width and about the weights of the 8B Llama shape, mixers and feed-forwards alike; recurrent blocks
+    and attention beside the delta rule take turns, without a loop."""
     from . import _lib
     ff = dict(ff="dense", ffn=21504, ff_act="gelu_tanh", ff_bias=True)
-    delta = LayerSpec(mixer="delta", heads=16, kv_heads=16, dim=128, vdim=128, conv_taps=4, ff="none")
-    both = LayerSpec(mixer="attention", heads=32, kv_heads=8, dim=128, vdim=128, scale=128 ** -0.5, out_gate="element", qkv_bias=True, qk_norm=True,
+    delta = LayerSpec(mixer="delta", heads=8, kv_heads=8, dim=128, vdim=128, conv_taps=4, ff="none")
+    both = LayerSpec(mixer="attention", heads=16, kv_heads=4, dim=128, vdim=128, scale=128 ** -0.5, out_gate="element", qkv_bias=True, qk_norm=True,
                      v_norm=True, rope_pairs=True, rope_base=500000.0, rope_dims=128, window=1024, keep_first=64, head_mix=True, mix_scale=0.5,
                      beside=delta, beside_names=("left.", "right."), **ff)
-    lru = LayerSpec(mixer="lru", heads=16, dim=256, vdim=256, conv_taps=4, **ff)
+    lru = LayerSpec(mixer="lru", heads=12, dim=256, vdim=256, conv_taps=4, **ff)
     return LayeredConfig(**{**dict(vocab=128256, d_model=4096, layers=[both if i % 2 else lru for i in range(32)], eps=1e-5, block="sandwich",
                                    own_head=True, embed_scale=64.0, bigram=(16384, 31, 17), max_seq=2560, dtype=_lib.BF16), **kw})
