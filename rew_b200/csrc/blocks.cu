@@ -855,8 +855,7 @@ int layered_session(rewb200_session* s, int64_t n_pages) {
   s->tmK.resize(n);
   s->tmV.resize(n);
   s->state.resize(n, nullptr);
-  s->conv_state.resize(n, nullptr);
-  s->state2.resize(n, nullptr);
+  for (auto* list : {&s->delta_state, &s->delta_conv, &s->lru_state, &s->lru_conv}) list->resize(n, nullptr);
   auto zeroed = [&](void** p, size_t bytes) -> int {
     RB_CUDA(cudaMalloc(p, bytes));
     RB_CUDA(cudaMemsetAsync(*p, 0, bytes, m->c->stream));
@@ -877,13 +876,12 @@ int layered_session(rewb200_session* s, int64_t n_pages) {
     // a state needs no clearing between sequences: a portion that starts at position 0 does not read it
     if (D.mixer == MIX_GLA)
       RB_TRY(zeroed((void**)&s->state[r], (size_t)s->B * D.l.m.heads * D.l.m.dim * gla_state_ld(D.l.m.vdim) * sizeof(float)));
-    if (has(D, MIX_DELTA) || has(D, MIX_LRU)) {
-      const bool delta = has(D, MIX_DELTA);
-      const int64_t elems = delta ? (int64_t)D.d.m.heads * D.d.m.dim * gla_state_ld(D.d.m.vdim) : (int64_t)D.r.m.blocks * D.r.m.n;
-      const int64_t conv = conv_state_elems(delta ? D.d.conv : D.r.conv);
-      RB_TRY(zeroed((void**)&s->state2[r], (size_t)s->B * elems * sizeof(float)));
-      if (conv > 0) RB_TRY(zeroed((void**)&s->conv_state[r], (size_t)s->B * conv * sizeof(float)));
-    }
+    auto recurrent = [&](float** state, int64_t elems, float** conv, const ConvDims& cd) -> int {
+      RB_TRY(zeroed((void**)state, (size_t)s->B * elems * sizeof(float)));
+      return conv_state_elems(cd) > 0 ? zeroed((void**)conv, (size_t)s->B * conv_state_elems(cd) * sizeof(float)) : REWB200_OK;
+    };
+    if (has(D, MIX_DELTA)) RB_TRY(recurrent(&s->delta_state[r], (int64_t)D.d.m.heads * D.d.m.dim * gla_state_ld(D.d.m.vdim), &s->delta_conv[r], D.d.conv));
+    if (has(D, MIX_LRU)) RB_TRY(recurrent(&s->lru_state[r], (int64_t)D.r.m.blocks * D.r.m.n, &s->lru_conv[r], D.r.conv));
   }
   if (m->bigram) RB_TRY(zeroed((void**)&s->last_ids, (size_t)s->B * sizeof(int)));
   return REWB200_OK;
@@ -1476,7 +1474,7 @@ int delta_mixer(rewb200_session* s, const FwdOpts& o, const StepLists& t, size_t
   ca.out = s->conv;
   ca.ldo = pad8(ch);
   ca.dtype = m->cfg.dtype;
-  ca.state = s->conv_state[r];
+  ca.state = s->delta_conv[r];
   ca.tails = t.tails;
   ca.n_tails = s->plan_tails;
   ca.early = in_graph ? 1 : 0;
@@ -1497,7 +1495,7 @@ int delta_mixer(rewb200_session* s, const FwdOpts& o, const StepLists& t, size_t
   da.split_stride = ca.split_stride;
   da.ld = ca.ld;
   da.eps = m->cfg.eps;
-  da.state = s->state2[r];
+  da.state = s->delta_state[r];
   da.ldv = (int)gla_state_ld(A.m.vdim);
   da.out = (char*)s->attn + at.out_col * es;
   da.ldo = D.o.K;
@@ -1538,7 +1536,7 @@ int lru_mixer(rewb200_session* s, const FwdOpts& o, const StepLists& t, size_t r
   ca.group = A.m.n;
   ca.offsets = s->group_rows;
   ca.dtype = m->cfg.dtype;
-  ca.state = s->conv_state[r];
+  ca.state = s->lru_conv[r];
   ca.tails = t.tails;
   ca.n_tails = s->plan_tails;
   ca.early = in_graph ? 1 : 0;
@@ -1570,7 +1568,7 @@ int lru_mixer(rewb200_session* s, const FwdOpts& o, const StepLists& t, size_t r
   la.nsplit = at.ks;
   la.split_stride = ca.split_stride;
   la.ld = ca.ld;
-  la.state = s->state2[r];
+  la.state = s->lru_state[r];
   la.out = (char*)s->attn + at.out_col * dtype_size(m->cfg.dtype);
   la.ldo = D.o.K;
   la.dtype = m->cfg.dtype;

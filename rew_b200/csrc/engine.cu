@@ -1674,7 +1674,7 @@ void rewb200_session_free(rewb200_session* s) {
   if (s->graph) cudaGraphExecDestroy(s->graph);
   for (void* p : s->kc) cudaFree(p);
   for (void* p : s->vc) cudaFree(p);
-  for (const auto* list : {&s->state, &s->conv_state, &s->state2})
+  for (const auto* list : {&s->state, &s->delta_state, &s->delta_conv, &s->lru_state, &s->lru_conv})
     for (void* p : *list) cudaFree(p);
   void* ptrs[] = {s->d_active, s->d_ids_prefill, s->block_table, s->d_pos, s->d_ids, s->d_next, s->d_out, s->d_step, s->x_res, s->xn, s->q,
                   s->attn, s->h, s->part, s->gu32, s->logits, s->attn_scratch, s->argmax_scratch, s->gather_scratch,

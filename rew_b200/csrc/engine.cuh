@@ -196,7 +196,7 @@ struct rewb200_session {
   std::vector<void*> kc, vc;           // per layer
   std::vector<CUtensorMap> tmK, tmV;   // per layer (bf16)
   std::vector<float*> state;           // layered models: recurrent or convolution state per layer run [B][..] f32, or nullptr
-  std::vector<float*> conv_state, state2;  // convolution state beside a recurrent one, and the recurrent state of a second mixer
+  std::vector<float*> delta_state, delta_conv, lru_state, lru_conv;  // recurrent and convolution states of the mixers that have both
   int* last_ids = nullptr;             // the last id of every lane (bigram tables)
   int* block_table = nullptr;
   int *d_pos = nullptr, *d_ids = nullptr, *d_next = nullptr, *d_out = nullptr, *d_step = nullptr;

@@ -599,9 +599,10 @@ int gqa_mix_launch(Ctx* c, const GqaMixArgs& a) {
   for (int64_t t0 = 0; t0 < a.tiles.count; t0 += piece) {
     const int64_t n = std::min<int64_t>(piece, a.tiles.count - t0);
     cf.tile0 = (int)t0;
-    cf.s = a.work;
+    // in this order every part starts on 16 bytes: vdim is a multiple of 8, slots one of 64
+    cf.o_part = a.work;
+    cf.s = a.work + (cf.splits > 1 ? (size_t)room * a.m.heads * cf.splits * a.m.vdim : 0);
     cf.ml = reinterpret_cast<float2*>(cf.s + (size_t)room * a.m.heads * cf.slots);
-    cf.o_part = reinterpret_cast<float*>(cf.ml + (size_t)room * a.m.heads * cf.splits);
     const dim3 grid((unsigned)cf.splits, (unsigned)(n * cf.subtiles), (unsigned)(a.m.kv_heads * cf.hgroups));
     cf.nb = (a.m.dim + 63) / 64;
     cf.stages = cf.nb <= 2 ? 3 : 2;
