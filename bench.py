@@ -27,6 +27,9 @@ data-path collective): weak scaling.
     kugirax_b32, kugirax_b1, kugirax_b8_s2048, kugirax_moe_b64
              Kugirax (attention with a short convolution and latent attention with sinks in turn, one-norm
              blocks) at the sizes of l8_b32, l8_b1, l8_b8_s2048 and moe_b64
+    musavik_b32, musavik_b1, musavik_b8_s2048
+             Musavik (linear recurrent units, and windowed attention with mixed heads beside a gated delta
+             rule, in turn; blocks normed on both sides) at the sizes of l8_b32, l8_b1 and l8_b8_s2048
 
 `value` is decode tokens/s of the whole job with ids, weights and cache resident
 in HBM (CUDA events around K graph replays); `e2e` is tokens/s of one generate()

@@ -87,7 +87,7 @@ def test_clock_record_counts_only_samples_inside_the_timed_region():
     assert short["samples"] == 3 and short["window"].startswith("warm-up + timed region") and short["reasons"] == ["sw_power_cap"]
 
 
-@pytest.mark.parametrize("workload", ["rezupel_b32", "girulorn_b64", "kugirax_b32"])
+@pytest.mark.parametrize("workload", ["rezupel_b32", "girulorn_b64", "kugirax_b32", "musavik_b32"])
 def test_reference_arm_says_why_a_layered_workload_is_unavailable(workload):
     r = _run("--impl", "reference", "--workload", workload, "--steps", "1", "--warmup", "1")
     assert r.returncode == 0, r.stderr[-2000:]
