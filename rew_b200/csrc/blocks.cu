@@ -782,6 +782,12 @@ int layered_init_random(rewb200_model* m, uint64_t seed, float std) {
 }
 
 int layered_plans(rewb200_model* m) {
+  for (LayerDev& D : m->layers)
+    if (D.g.talk) {
+      D.g.talk_host.resize((size_t)D.g.m.heads * D.g.m.heads);
+      RB_CUDA(cudaMemcpyAsync(D.g.talk_host.data(), D.g.talk, D.g.talk_host.size() * sizeof(float), cudaMemcpyDeviceToHost, m->c->stream));
+      RB_CUDA(cudaStreamSynchronize(m->c->stream));
+    }
   if (m->cfg.dtype != REWB200_BF16) return REWB200_OK;
   auto plan = [&](LinW& w) { return linear_bf16_plan(&w.plan, (const bf16*)w.w, w.K, w.N, 0); };
   if (m->loop_in.w) RB_TRY(plan(m->loop_in));
@@ -930,7 +936,7 @@ int layered_prepare(rewb200_session* s, const FwdOpts& o, int64_t rows) {
   int64_t abs_rows = rows, n_keys = 0;
   s->plan_host.clear();
   s->plan_abs_tiles = s->plan_chunks = s->plan_exp_tiles = s->plan_keys = s->plan_gla_chunks = s->plan_tails = 0;
-  s->plan_gqa_small = s->plan_delta_small = s->plan_delta_large = s->plan_delta_chunks = s->plan_portions = s->plan_longest = 0;
+  s->plan_gqa_small = s->plan_gqa_large = s->plan_delta_small = s->plan_delta_large = s->plan_delta_chunks = s->plan_portions = s->plan_longest = 0;
   if (!uniform) {
     std::vector<int>& h = s->plan_host;
     h.assign(2 * rows, 0);
@@ -951,7 +957,7 @@ int layered_prepare(rewb200_session* s, const FwdOpts& o, int64_t rows) {
       if (has(D, MIX_LRU)) taps = std::max(taps, D.r.conv.taps);
       if (D.mixer == MIX_GQA) {
         has_gqa = true;
-        gqa_ok = gqa_ok && !gqa_is_mixed(D.g.m) && gqa_prefill_ok(D.g.m);
+        gqa_ok = gqa_ok && (gqa_is_mixed(D.g.m) ? gqa_mix_prefill_ok(D.g.m) : gqa_prefill_ok(D.g.m));
         taps = std::max(taps, D.g.m.taps);
       }
       if (D.mixer == MIX_GLA) {
@@ -1075,17 +1081,24 @@ int layered_prepare(rewb200_session* s, const FwdOpts& o, int64_t rows) {
     s->kvx_rows = n_keys;
   }
   // ---- scratch of the absorbed path
-  size_t chunk = 0, mix = 0;
+  size_t chunk = 0, mix = 0, lse = 0;
   for (const LayerDev& D : m->layers) {
     if (D.mixer == MIX_GLA) chunk = std::max(chunk, gla_chunk_bytes(D.l.m) * s->plan_gla_chunks);
     if (has(D, MIX_DELTA)) chunk = std::max(chunk, delta_chunk_bytes(D.d.m) * s->plan_delta_chunks);
-    if (D.mixer == MIX_GQA && gqa_is_mixed(D.g.m))
+    if (D.mixer != MIX_GQA || !gqa_is_mixed(D.g.m)) continue;
+    if (s->plan_gqa_large > 0) lse = std::max(lse, (size_t)rows * D.g.m.heads * sizeof(float));
+    if (uniform || s->plan_gqa_small > 0)
       mix = std::max(mix, gqa_mix_bytes(c, D.g.m, m->cfg.dtype, rows, uniform ? rows : s->plan_gqa_small, uniform ? 1 : GQA_TILE_ROWS, (int64_t)s->max_pages * PAGE));
   }
   if (chunk > s->gla_work_bytes) {
     s->gla_work_bytes = 0;
     RB_TRY(regrow(s, &s->gla_work, chunk));
     s->gla_work_bytes = chunk;
+  }
+  if (lse > s->mix_lse_bytes) {
+    s->mix_lse_bytes = 0;
+    RB_TRY(regrow(s, &s->mix_lse, lse));
+    s->mix_lse_bytes = lse;
   }
   if (mix > s->mix_bytes) {
     s->mix_bytes = 0;
@@ -1257,6 +1270,8 @@ int gqa_mixer(rewb200_session* s, const FwdOpts& o, const StepLists& t, size_t r
     ma.early_kv = in_graph ? 1 : 0;
     ma.status = c->d_status;
     RB_TRY(gqa_mix_launch(c, ma));
+    if (!t.uniform && s->plan_gqa_large > 0)
+      RB_TRY(gqa_mix_prefill_launch(c, ma, t.gqa_large, s->plan_gqa_large, G.talk ? G.talk_host.data() : nullptr, s->mix_lse));
     if (o.trace) RB_TRY(o.trace->mark(TC_ATTN));
     return REWB200_OK;
   }

@@ -95,10 +95,10 @@ size_t dtype_size(int dtype);
 // box_inner x box_outer elements, 128-byte swizzle (box_inner must be 64).
 int make_tmap_2d_bf16(CUtensorMap* out, const void* base, uint64_t inner, uint64_t outer,
                       uint64_t row_stride_bytes, uint32_t box_inner, uint32_t box_outer);
-// 3D variant (dim 2 = groups, e.g. experts) with box depth 1.
+// 3D variant (dim 2 = groups, e.g. experts).
 int make_tmap_3d_bf16(CUtensorMap* out, const void* base, uint64_t inner, uint64_t outer, uint64_t groups,
                       uint64_t row_stride_bytes, uint64_t group_stride_bytes, uint32_t box_inner,
-                      uint32_t box_outer);
+                      uint32_t box_outer, uint32_t box_groups = 1);
 
 // NF4 weight-only Linear (nf4.cu).  Column map: logical column n of the quantised matrix lives at
 // device column (w / gran) * gstride + w % gran + (n / seg_len) * seg_off with w = n % seg_len

@@ -1680,7 +1680,7 @@ void rewb200_session_free(rewb200_session* s) {
                   s->attn, s->h, s->part, s->gu32, s->logits, s->attn_scratch, s->argmax_scratch, s->gather_scratch,
                   s->samp_hist, s->samp_hist_len, s->samp_steps, s->samp_keys, s->samp_work, s->samp_logprob, s->moe_logits, s->moe_topw, s->moe_topi, s->moe_ints,
                   s->moe_send, s->moe_recv, s->moe_xs, s->moe_hs, s->moe_ys, s->moe_ret, s->moe_back, s->moe_tmp, s->route_rec,
-                  s->xn2, s->cq, s->gate, s->part2, s->part3, s->shared_gate, s->qeff, s->olat, s->ml, s->gqa_part, s->gqa_ml, s->gla_work, s->kvx, s->latx, s->layer_rec, s->xg, s->logits_pad, s->plan_dev, s->feed_dev, s->cat, s->conv, s->gate_pre, s->group_rows, s->big_rows, s->last_ids, s->mix_work};
+                  s->xn2, s->cq, s->gate, s->part2, s->part3, s->shared_gate, s->qeff, s->olat, s->ml, s->gqa_part, s->gqa_ml, s->gla_work, s->kvx, s->latx, s->layer_rec, s->xg, s->logits_pad, s->plan_dev, s->feed_dev, s->cat, s->conv, s->gate_pre, s->group_rows, s->big_rows, s->last_ids, s->mix_work, s->mix_lse};
   for (void* p : ptrs)
     if (p) cudaFree(p);
   if (s->h_ids) cudaFreeHost(s->h_ids);

@@ -99,6 +99,7 @@ struct GqaDev {
   LinW in;                     // [d, heads * dim | kv_heads * dim | kv_heads * vdim | heads]: queries, keys, values (unless v_from_k), gate
   float *q_norm = nullptr, *k_norm = nullptr, *bias = nullptr, *sink = nullptr, *conv = nullptr, *in_bias = nullptr, *talk = nullptr;
   int64_t gate_col = 0;        // of the gate in `in`
+  std::vector<float> talk_host;   // the matrix that mixes the heads, read back when the model is finished
   int64_t ldk = 0, ldv = 0;    // elements of a cached key / value row, padded
 };
 
@@ -251,6 +252,8 @@ struct rewb200_session {
   int* big_rows = nullptr;             // rows of the bigram table
   float* mix_work = nullptr;           // scores of attention with mixed heads
   size_t mix_bytes = 0;
+  float* mix_lse = nullptr;            // its softmax denominators in large portions
+  size_t mix_lse_bytes = 0;
   float* layer_rec = nullptr;          // option record_layers: [runs][rows_cap][d]
   int64_t layer_rows = 0;
   void* xg = nullptr;                  // rows of xn gathered for the lm_head

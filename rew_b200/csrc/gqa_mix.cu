@@ -579,8 +579,8 @@ int plain_launch(Ctx* c, const GqaMixArgs& a) {
 }  // namespace
 
 int gqa_mix_launch(Ctx* c, const GqaMixArgs& a) {
-  if (a.dtype != REWB200_BF16 || c->gqa_impl == 1 || !mma_ok(a.m)) return plain_launch(c, a);
   if (a.tiles.count == 0) return REWB200_OK;
+  if (a.dtype != REWB200_BF16 || c->gqa_impl == 1 || !mma_ok(a.m)) return plain_launch(c, a);
   MixCfg cf = config(a.m, a.max_tile_rows);
   const int64_t pages = most_pages(a.m, a.max_tile_rows, a.max_pages);
   cf.slots = pages * PAGE_TOKENS;

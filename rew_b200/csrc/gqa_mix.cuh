@@ -36,4 +36,9 @@ struct GqaMixArgs {
 size_t gqa_mix_bytes(Ctx* c, const GqaDims& m, int dtype, int64_t rows, int64_t tiles, int64_t max_tile_rows, int64_t max_ctx);
 int gqa_mix_launch(Ctx* c, const GqaMixArgs& a);
 
+// Large prompt portions on tcgen05; tiles as in GqaPrefillArgs, talk_host: the mixing matrix on the host (nullptr: none), lse:
+// scratch [rows][heads].  Of `a`, the tiles and the scratch are not read.
+bool gqa_mix_prefill_ok(const GqaDims& m);
+int gqa_mix_prefill_launch(Ctx* c, const GqaMixArgs& a, const GqaTile* tiles, int count, const float* talk_host, float* lse);
+
 }  // namespace rewb

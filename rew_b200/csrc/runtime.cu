@@ -98,13 +98,13 @@ int make_tmap_2d_bf16(CUtensorMap* out, const void* base, uint64_t inner, uint64
 
 int make_tmap_3d_bf16(CUtensorMap* out, const void* base, uint64_t inner, uint64_t outer, uint64_t groups,
                       uint64_t row_stride_bytes, uint64_t group_stride_bytes, uint32_t box_inner,
-                      uint32_t box_outer) {
+                      uint32_t box_outer, uint32_t box_groups) {
   RB_TRY(load_encode());
   RB_REQUIRE((reinterpret_cast<uintptr_t>(base) & 15) == 0, "tensor map base must be 16-byte aligned");
   RB_REQUIRE(row_stride_bytes % 16 == 0 && group_stride_bytes % 16 == 0, "tensor map strides must be multiples of 16 bytes");
   cuuint64_t dims[3] = {inner, outer, groups};
   cuuint64_t strides[2] = {row_stride_bytes, group_stride_bytes};
-  cuuint32_t box[3] = {box_inner, box_outer, 1};
+  cuuint32_t box[3] = {box_inner, box_outer, box_groups};
   cuuint32_t estr[3] = {1, 1, 1};
   CUresult r = g_encode(out, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<void*>(base), dims, strides, box, estr,
                         CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
