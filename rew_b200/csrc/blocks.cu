@@ -445,7 +445,7 @@ int layered_create(rewb200_model* m, const rewb200_layer* layers, const rewb200_
       RB_TRY(sink_of(L, &G.sink));
       G.m = GqaDims{L.heads, L.kv_heads, L.dim, L.vdim, own ? 1 : 0, L.out_gate == 1, L.scale, G.q_norm, G.k_norm, L.temp_every, L.temp_coef, G.bias, nb, G.sink,
                     L.values_from_keys, L.conv_taps, nullptr, L.rope_dims, nullptr, L.rope_pairs, L.v_norm, G.in_bias, L.window, L.keep_first, G.talk,
-                    L.out_gate == 2, scale_of(L)};
+                    0, L.out_gate == 2, scale_of(L)};
       RB_TRY(rope_of(L, &G.m.rope));
       if (L.conv_taps > 0) RB_TRY(zero_weights(m, (void**)&G.conv, (size_t)L.conv_taps * gqa_channels(G.m) * sizeof(float)));
       G.m.conv = G.conv;
@@ -787,6 +787,7 @@ int layered_plans(rewb200_model* m) {
       D.g.talk_host.resize((size_t)D.g.m.heads * D.g.m.heads);
       RB_CUDA(cudaMemcpyAsync(D.g.talk_host.data(), D.g.talk, D.g.talk_host.size() * sizeof(float), cudaMemcpyDeviceToHost, m->c->stream));
       RB_CUDA(cudaStreamSynchronize(m->c->stream));
+      D.g.m.talk_wide = std::any_of(D.g.talk_host.begin(), D.g.talk_host.end(), [](float t) { return !(std::fabs(t) < 65504.f); });
     }
   if (m->cfg.dtype != REWB200_BF16) return REWB200_OK;
   auto plan = [&](LinW& w) { return linear_bf16_plan(&w.plan, (const bf16*)w.w, w.K, w.N, 0); };
@@ -1194,10 +1195,11 @@ StepLists step_lists(const rewb200_session* s, const FwdOpts& o, int64_t rows) {
   return t;
 }
 
-// The mixers read s->xn and leave their output (ahead of the output projection) in s->attn.
+// The mixers read the input projection in s->part (latent attention: s->xn) and leave their output (ahead of the output
+// projection) in s->attn.
 
-// *slabs: slabs of the input projection, which a second mixer reads too.
-int gqa_mixer(rewb200_session* s, const FwdOpts& o, const StepLists& t, size_t r, int64_t rows, bool in_graph, int* slabs) {
+// ks: slabs of the input projection.
+int gqa_mixer(rewb200_session* s, const FwdOpts& o, const StepLists& t, size_t r, int64_t rows, bool in_graph, int ks) {
   rewb200_model* m = s->m;
   Ctx* c = m->c;
   const int dt = m->cfg.dtype;
@@ -1205,9 +1207,6 @@ int gqa_mixer(rewb200_session* s, const FwdOpts& o, const StepLists& t, size_t r
   LayerDev& D = m->layers[R.layer];
   GqaDev& G = D.g;
   const int64_t ldq = pad8((int64_t)G.m.heads * G.m.dim);
-  int ks = 1;
-  RB_TRY(run_linear(s, G.in, s->xn, m->dp, rows, true, 0, s->part, G.in.N, &ks));
-  if (o.trace) RB_TRY(o.trace->mark(TC_QKV));
   GqaPostArgs pa;
   memset(&pa, 0, sizeof(pa));
   pa.m = G.m;
@@ -1236,7 +1235,6 @@ int gqa_mixer(rewb200_session* s, const FwdOpts& o, const StepLists& t, size_t r
   RB_TRY(gqa_post_launch(c, pa, rows));
   if (!t.uniform) RB_TRY(gqa_conv_state_launch(c, pa));
   if (o.trace) RB_TRY(o.trace->mark(TC_QKV_POST));
-  *slabs = ks;
   if (gqa_is_mixed(G.m)) {
     GqaMixArgs ma;
     memset(&ma, 0, sizeof(ma));
@@ -1325,15 +1323,11 @@ int gqa_mixer(rewb200_session* s, const FwdOpts& o, const StepLists& t, size_t r
   return REWB200_OK;
 }
 
-int gla_mixer(rewb200_session* s, const FwdOpts& o, const StepLists& t, size_t r, int64_t rows, bool in_graph, int* slabs) {
+int gla_mixer(rewb200_session* s, const FwdOpts& o, const StepLists& t, size_t r, int64_t rows, bool in_graph, int ks) {
   rewb200_model* m = s->m;
   Ctx* c = m->c;
   LayerDev& D = m->layers[m->runs[r].layer];
   GlaDev& A = D.l;
-  int ks = 1;
-  RB_TRY(run_linear(s, A.in, s->xn, m->dp, rows, true, 0, s->part, A.in.N, &ks));
-  if (o.trace) RB_TRY(o.trace->mark(TC_QKV));
-  *slabs = ks;
   GlaArgs ga;
   memset(&ga, 0, sizeof(ga));
   ga.m = A.m;
@@ -1593,25 +1587,6 @@ int lru_mixer(rewb200_session* s, const FwdOpts& o, const StepLists& t, size_t r
   return REWB200_OK;
 }
 
-int mixer(rewb200_session* s, const FwdOpts& o, const StepLists& t, size_t r, int64_t rows, bool in_graph) {
-  LayerDev& D = s->m->layers[s->m->runs[r].layer];
-  MixerAt at = {&in_of(D), 0, 0, 1};
-  auto recurrent = [&](int kind) { return kind == MIX_DELTA ? delta_mixer(s, o, t, r, rows, in_graph, at) : lru_mixer(s, o, t, r, rows, in_graph, at); };
-  switch (D.mixer) {
-    case MIX_GQA: RB_TRY(gqa_mixer(s, o, t, r, rows, in_graph, &at.ks)); break;
-    case MIX_GLA: RB_TRY(gla_mixer(s, o, t, r, rows, in_graph, &at.ks)); break;
-    case MIX_LATENT: return latent_mixer(s, o, t, r, rows, in_graph);
-    default:
-      RB_TRY(run_linear(s, *at.in, s->xn, s->m->dp, rows, true, 0, s->part, at.in->N, &at.ks));
-      if (o.trace) RB_TRY(o.trace->mark(TC_QKV));
-      RB_TRY(recurrent(D.mixer));
-  }
-  if (!D.beside) return REWB200_OK;
-  at.col = D.beside_in;
-  at.out_col = D.beside_out;
-  return recurrent(D.beside);
-}
-
 // A feed-forward, gated SiLU (dense, or the shared expert beside routed ones) or tanh GELU: f32 slabs of the result in `out`,
 // without the bias of the down projection.
 int dense_ff(rewb200_session* s, const FwdOpts& o, LayerDev& D, const void* x, int64_t rows, float* out, int* ks) {
@@ -1644,6 +1619,38 @@ int on_side_stream(Ctx* c, F&& body) {
   c->stream = main_stream;
   RB_TRY(st);
   RB_CUDA(cudaEventRecord(c->ev_join, c->side));
+  return REWB200_OK;
+}
+
+// The mixers of run r.  *joined: a second one ran beside the first on the side stream, so what follows has two predecessors.
+int mixer(rewb200_session* s, const FwdOpts& o, const StepLists& t, size_t r, int64_t rows, bool in_graph, bool* joined = nullptr) {
+  rewb200_model* m = s->m;
+  Ctx* c = m->c;
+  LayerDev& D = m->layers[m->runs[r].layer];
+  if (D.mixer == MIX_LATENT) return latent_mixer(s, o, t, r, rows, in_graph);
+  MixerAt at = {&in_of(D), 0, 0, 1};
+  RB_TRY(run_linear(s, *at.in, s->xn, m->dp, rows, true, 0, s->part, at.in->N, &at.ks));
+  if (o.trace) RB_TRY(o.trace->mark(TC_QKV));
+  auto recurrent = [&](int kind, const MixerAt& p) { return kind == MIX_DELTA ? delta_mixer(s, o, t, r, rows, in_graph, p) : lru_mixer(s, o, t, r, rows, in_graph, p); };
+  MixerAt second = at;
+  second.col = D.beside_in;
+  second.out_col = D.beside_out;
+  // small steps are chains of short launches: two chains at a time
+  const bool fork = joined && D.beside && D.mixer == MIX_GQA && m->cfg.dtype == REWB200_BF16 && rows <= 64 && c->moe_overlap && !o.trace;
+  if (fork)
+    RB_TRY(on_side_stream(c, [&]() -> int {
+      const bool pdl = c->use_pdl;
+      c->use_pdl = false;   // follows an event wait: plain launches
+      const int st = recurrent(D.beside, second);
+      c->use_pdl = pdl;
+      return st;
+    }));
+  if (D.mixer == MIX_GQA) RB_TRY(gqa_mixer(s, o, t, r, rows, in_graph, at.ks));
+  else if (D.mixer == MIX_GLA) RB_TRY(gla_mixer(s, o, t, r, rows, in_graph, at.ks));
+  else RB_TRY(recurrent(D.mixer, at));
+  if (fork) RB_CUDA(cudaStreamWaitEvent(c->stream, c->ev_join, 0));
+  else if (D.beside) RB_TRY(recurrent(D.beside, second));
+  if (joined) *joined = fork;
   return REWB200_OK;
 }
 
@@ -1794,10 +1801,15 @@ int sandwich_blocks(rewb200_session* s, const FwdOpts& o, const NormArgs& na, in
       RB_TRY(output_norm_launch(c, a, rows));
       if (o.trace) RB_TRY(o.trace->mark(TC_EMBED));
     }
-    RB_TRY(mixer(s, o, t, r, rows, in_graph));
+    bool joined = false;
+    RB_TRY(mixer(s, o, t, r, rows, in_graph, &joined));
     OutputNormArgs a = base;
     a.nsplit = 1;
-    RB_TRY(run_linear(s, D.o, s->attn, D.o.K, rows, true, 0, s->part, dp, &a.nsplit));
+    const bool pdl = c->use_pdl;
+    if (joined) c->use_pdl = false;   // two predecessors: a plain dependency
+    const int st = run_linear(s, D.o, s->attn, D.o.K, rows, true, 0, s->part, dp, &a.nsplit);
+    c->use_pdl = pdl;
+    RB_TRY(st);
     if (o.trace) RB_TRY(o.trace->mark(TC_O));
     a.partial = s->part;
     a.gamma = D.back1;

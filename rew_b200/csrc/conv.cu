@@ -79,7 +79,7 @@ __global__ void __launch_bounds__(NT) conv_kernel(ConvArgs a, int64_t rows, int 
   const int64_t g = a.group > 0 ? ch / a.group : 0;
   T* out = reinterpret_cast<T*>(a.out) + (a.group > 0 ? (g * rows + row0) * a.ldo + ch - g * a.group : row0 * a.ldo + ch);
   const bool keep = !a.tails && a.m.taps > 1 && on;
-  constexpr int AHEAD = 4;    // rows requested together
+  constexpr int AHEAD = TAPS <= 4 ? 8 : 4;    // rows requested together
   for (int r0 = 0; r0 < nr; r0 += AHEAD) {
     float4 xs[AHEAD];
 #pragma unroll
@@ -97,7 +97,9 @@ __global__ void __launch_bounds__(NT) conv_kernel(ConvArgs a, int64_t rows, int 
       if (keep && in.x >= 0) *state_at(in.y, in.x) = h[0];
 #pragma unroll
       for (int b = TAPS - 1; b > 0; --b) h[b] = h[b - 1];
-      if (a.m.silu) y = make_float4(silu_act(y.x), silu_act(y.y), silu_act(y.z), silu_act(y.w));
+      if (a.m.silu)
+        y = sizeof(T) == 2 ? make_float4(silu_fast(y.x), silu_fast(y.y), silu_fast(y.z), silu_fast(y.w))
+                           : make_float4(silu_act(y.x), silu_act(y.y), silu_act(y.z), silu_act(y.w));
       if (!on) continue;
       if constexpr (sizeof(T) == 2) *reinterpret_cast<uint2*>(out + r * a.ldo) = make_uint2(pack_bf16(y.x, y.y), pack_bf16(y.z, y.w));
       else *reinterpret_cast<float4*>(out + r * a.ldo) = y;

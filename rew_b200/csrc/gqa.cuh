@@ -32,6 +32,7 @@ struct GqaDims {
   const float* in_bias;    // by column of the projection's queries, keys and values, or nullptr (no convolution then)
   int window, keep_first;  // keys a query sees, itself included (0: all), and the first keys of the sequence it sees besides
   const float* talk;       // [heads][heads] mixes the heads' weights after the softmax, or nullptr
+  int talk_wide;           // it has numbers that f16 has not
   int gate_elem;           // the output gate is per feature
   float out_scale;         // of the output
 };

@@ -661,7 +661,7 @@ size_t attn_smem(const GqaDims& m, const Shape& s, int nbk, int nbv, int stages)
 
 bool gqa_mix_prefill_ok(const GqaDims& m) {
   Shape s;
-  return m.dim % 8 == 0 && m.vdim % 8 == 0 && m.dim <= 128 && m.vdim <= 128 && m.scale > 0.f && !m.bias && !m.sink && shape_of(m, &s);
+  return m.dim % 8 == 0 && m.vdim % 8 == 0 && m.dim <= 128 && m.vdim <= 128 && m.scale > 0.f && !m.bias && !m.sink && !m.talk_wide && shape_of(m, &s);
 }
 
 int gqa_mix_prefill_launch(Ctx* c, const GqaMixArgs& g, const GqaTile* tiles, int count, const float* talk_host, float* lse) {

@@ -65,9 +65,15 @@ __global__ void __launch_bounds__(NW == 1 ? 128 : 32 * NW) lru_kernel(LruArgs a)
         i[k] = 0.f;
         continue;
       }
-      const float la = decay * sigmoid_act(r[k]);
-      i[k] = sqrtf(-expm1f(2.0f * la)) * sigmoid_act(i[k]) * u[k];
-      r[k] = expf(la);
+      if constexpr (sizeof(T) == 2) {
+        const float la = decay * sigmoid_fast(r[k]);
+        r[k] = __expf(la);
+        i[k] = sqrt_fast(one_minus_exp(2.0f * la, r[k] * r[k])) * sigmoid_fast(i[k]) * u[k];
+      } else {
+        const float la = decay * sigmoid_act(r[k]);
+        i[k] = sqrtf(-expm1f(2.0f * la)) * sigmoid_act(i[k]) * u[k];
+        r[k] = expf(la);
+      }
     }
     float c = S;
     if constexpr (NW > 1) {
