@@ -98,9 +98,11 @@ int rewb200_sync(int slot, int timeout_ms);
  *   "gqa_attention" = "auto" | "plain" | "paged"   grouped-query attention of layered models: the tcgen05 kernel for large prompt
  *                                            portions and the paged kernel otherwise (default); always the plain kernel;
  *                                            always the paged kernel
- *   "linear_attention" = "auto" | "plain" | "recurrent"   gated linear attention: in chunks for large prompt portions and token
- *                                            by token otherwise (default); token by token with the state in global
- *                                            memory; always token by token
+ *   "linear_attention" = "auto" | "plain" | "recurrent"   gated linear attention and gated delta rule: in chunks for large prompt
+ *                                            portions and token by token otherwise (default); token by token with the
+ *                                            state in global memory; always token by token
+ *   "short_conv" = "auto" | "plain"          short convolutions with a state of their own: channels in groups of four (default);
+ *                                            always the plain kernel
  *   "inject_alloc_fail" = "n"                test hook: the n-th activation-buffer allocation from now fails on the host
  *   "moe_overlap" = "on" | "off"             MoE layers on one rank, steps of at most 64 rows: the shared experts run on a
  *                                            second stream beside the routed experts (default on)

@@ -83,7 +83,13 @@ __global__ void __launch_bounds__(NT) conv_kernel(ConvArgs a, int64_t rows, int 
   for (int r0 = 0; r0 < nr; r0 += AHEAD) {
     float4 xs[AHEAD];
 #pragma unroll
-    for (int u = 0; u < AHEAD; ++u) xs[u] = r0 + u < nr ? value(p + (r0 + u) * a.ld) : zero;
+    for (int u = 0; u < AHEAD; ++u) xs[u] = on && r0 + u < nr ? *reinterpret_cast<const float4*>(p + (r0 + u) * a.ld) : zero;
+    for (int s = 1; s < a.nsplit; ++s)
+#pragma unroll
+      for (int u = 0; u < AHEAD; ++u)
+        if (on && r0 + u < nr) add4(xs[u], *reinterpret_cast<const float4*>(p + s * a.split_stride + (r0 + u) * a.ld));
+#pragma unroll
+    for (int u = 0; u < AHEAD; ++u) add4(xs[u], bi);
 #pragma unroll
     for (int u = 0; u < AHEAD; ++u) {
       const int r = r0 + u;

@@ -11,17 +11,16 @@ extern int64_t g_launch_total;
 
 namespace {
 
-constexpr int TT = 8;     // tokens a warp holds in registers
 
 __device__ __forceinline__ GlaPortion portion_of(const LruArgs& a, int i) {
   if (a.list) return a.list[i];
   return GlaPortion{i, 1, a.pos0[a.b0 + i], a.b0 + i, 0};
 }
 
-// A lane owns one channel.  NW == 1: grid (channels / 128, portions), a warp walks its portion.  NW > 1: grid (channels / 32,
+// A lane owns one channel, TT tokens at a time.  NW == 1: grid (channels / 128, portions), a warp walks its portion.  NW > 1: grid (channels / 32,
 // portions), the warps of a CTA take consecutive runs of TT tokens; each reduces its run to (decay, contribution), the runs'
 // effects meet in shared memory, and every warp replays its run from the state it then knows.
-template <typename T, int NW>
+template <typename T, int NW, int TT>
 __global__ void __launch_bounds__(NW == 1 ? 128 : 32 * NW) lru_kernel(LruArgs a) {
   __shared__ float2 runs[2][NW][32];
   pdl_launch_dependents();
@@ -112,10 +111,12 @@ __global__ void lru_decay_kernel(float* lam, int64_t n) {
 int lru_launch(Ctx* c, const LruArgs& a) {
   if (a.count == 0) return REWB200_OK;
   const int width = a.m.blocks * a.m.n;
-  const bool bf = a.dtype == REWB200_BF16, wide = a.list && a.longest > 2 * TT;
-  const dim3 grid((unsigned)(wide ? (width + 31) / 32 : (width + 127) / 128), (unsigned)a.count);
-  if (wide) RB_CUDA(bf ? launch_k(lru_kernel<bf16, 8>, grid, dim3(256), 0, c->stream, c->use_pdl, a) : launch_k(lru_kernel<float, 8>, grid, dim3(256), 0, c->stream, c->use_pdl, a));
-  else RB_CUDA(bf ? launch_k(lru_kernel<bf16, 1>, grid, dim3(128), 0, c->stream, c->use_pdl, a) : launch_k(lru_kernel<float, 1>, grid, dim3(128), 0, c->stream, c->use_pdl, a));
+  const bool bf = a.dtype == REWB200_BF16, wide = a.list && a.longest > 16, single = !a.list || a.longest == 1;
+  const dim3 grid((unsigned)(wide ? (width + 31) / 32 : (width + 127) / 128), (unsigned)a.count), block(wide ? 256 : 128);
+  auto go = [&](auto kernel) { return launch_k(kernel, grid, block, 0, c->stream, c->use_pdl, a); };
+  RB_CUDA(wide ? (bf ? go(lru_kernel<bf16, 8, 8>) : go(lru_kernel<float, 8, 8>))
+          : single ? (bf ? go(lru_kernel<bf16, 1, 1>) : go(lru_kernel<float, 1, 1>))
+                   : (bf ? go(lru_kernel<bf16, 1, 8>) : go(lru_kernel<float, 1, 8>)));
   ++g_launch_total;
   return REWB200_OK;
 }
