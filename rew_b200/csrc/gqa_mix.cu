@@ -1,5 +1,4 @@
 // Kernels of gqa_mix.cuh for any dtype and size.  Scores, softmax, mixing and gates are f32.
-#include <cooperative_groups.h>
 #include <math.h>
 
 #include <algorithm>
@@ -8,8 +7,6 @@
 #include "act.cuh"
 #include "gqa_mix.cuh"
 #include "ptx.cuh"
-
-namespace cg = cooperative_groups;
 
 namespace rewb {
 
@@ -128,7 +125,7 @@ __global__ void __launch_bounds__(128) mix_plain_values_kernel(GqaMixArgs a, int
 }
 
 // ------------------------------------------------------------------ bf16 on the tensor cores
-// Portions, and single tokens outside the limits of mix_cluster_kernel: two launches over the pages a tile of rows sees (kept pages, then the window's), grid (splits, tiles * subtiles, kv heads *
+// Two launches over the pages a tile of rows sees (kept pages, then the window's), grid (splits, tiles * subtiles, kv heads *
 // head groups), four consumer warps and a TMA warp; a CTA's 16 rows are `heads_per` query heads of one kv head times
 // `tokens_per` tokens.
 //   mix_scores_kernel   scores in base 2 (-inf where a query does not see the key) to scratch [row][head][slots], and the
@@ -526,304 +523,6 @@ __global__ void __launch_bounds__(256) mix_merge_kernel(GqaMixArgs a, MixCfg cf,
   }
 }
 
-// Single tokens (a decode step) in one launch: a cluster of kv heads * splits CTAs has all heads of a token, so that scores and
-// softmax sums meet over distributed shared memory instead of scratch.  grid (cluster, tiles), cluster rank = split * kv heads +
-// kv head; four consumer warps and a TMA warp, whose ring takes the CTA's key pages and then its value pages.
-//   scores of the group's heads -> shared memory, maximum and sum per head | cluster barrier | weights of all heads for the
-//   CTA's keys, mixed (f32) -> bf16 | times values | sums of the splits meet (cluster barrier), gate, output
-struct MixCluster {
-  int splits, stages, stage_bytes, keys;   // keys: of a CTA at most (whole pages)
-};
-struct MixClusterSmem {
-  size_t q, s, p, ml, n, t, g, o, part, bars, end;
-};
-__host__ __device__ inline MixClusterSmem mix_cluster_smem(const GqaDims& m, const MixCluster& cl) {
-  MixClusterSmem o;
-  const size_t group = m.heads / m.kv_heads;
-  auto up = [](size_t x) { return (x + 15) / 16 * 16; };
-  o.q = (size_t)cl.stages * cl.stage_bytes;
-  o.s = o.q + (size_t)((m.dim + 63) / 64) * 2048;
-  o.p = o.s + up(group * (cl.keys + 8) * 4);
-  o.ml = o.p + up(group * (cl.keys + 8) * 2);
-  o.n = o.ml + up(group * 8);
-  o.t = o.n + up((size_t)m.heads * 8);
-  o.g = o.t + up((size_t)m.heads * group * 4);
-  o.o = o.g + up(group * m.vdim * 4);
-  o.part = o.o + up(group * m.vdim * 4);
-  o.bars = o.part + 512;
-  o.end = o.bars + 16 * 16;
-  return o;
-}
-
-template <int KS, int VW>
-__global__ void __launch_bounds__(160) mix_cluster_kernel(const __grid_constant__ CUtensorMap tm_k, const __grid_constant__ CUtensorMap tm_v, GqaMixArgs a,
-                                                          MixCluster cl) {
-  extern __shared__ uint8_t smem_raw[];
-  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
-  const GqaDims& m = a.m;
-  const MixClusterSmem of = mix_cluster_smem(m, cl);
-  uint8_t* sQ = smem + of.q;                                      // [box][16 rows][128 bytes]
-  float* sS = reinterpret_cast<float*>(smem + of.s);              // [group][keys + 8] scores, base 2
-  bf16* sP = reinterpret_cast<bf16*>(smem + of.p);                // [group][keys + 8] mixed weights
-  float2* sML = reinterpret_cast<float2*>(smem + of.ml);          // [group] maximum and sum of this CTA's keys
-  float2* sN = reinterpret_cast<float2*>(smem + of.n);            // [heads] maximum, 1 / sum, of all keys
-  float* sT = reinterpret_cast<float*>(smem + of.t);              // [heads][group] mixing matrix
-  float* sG = reinterpret_cast<float*>(smem + of.g);              // [group][vdim] gates
-  float* sO = reinterpret_cast<float*>(smem + of.o);              // [group][vdim] sums of this CTA's keys
-  float* sM = reinterpret_cast<float*>(smem + of.part);           // [4 warps][16] maxima, [4][16] sums
-  uint64_t *full = reinterpret_cast<uint64_t*>(smem + of.bars), *empty = full + 16;
-  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, l8 = lane & 7, lq = lane >> 3, g = lane >> 2, t = lane & 3;
-  const int H = m.heads, V = m.vdim, group = H / m.kv_heads, ldk = cl.keys + 8;
-  const int hk = (int)blockIdx.x % m.kv_heads, split = (int)blockIdx.x / m.kv_heads, head0 = hk * group;
-  auto cluster = cg::this_cluster();
-  if (tid == 128) {
-    for (int i = 0; i < cl.stages; ++i) {
-      mbar_init(&full[i], 1);
-      mbar_init(&empty[i], 4);
-    }
-    fence_barrier_init();
-    tma_prefetch_desc(&tm_k);
-    tma_prefetch_desc(&tm_v);
-  }
-  pdl_launch_dependents();
-  __syncthreads();
-  if (!a.early_kv) pdl_wait();
-  const int2 tr = tile_rows(a.tiles, (int)blockIdx.y);
-  if (tr.y <= 0) return;   // the whole cluster
-  const int64_t row = tr.x;
-  const int seq = row_lane(a.map, row), pos = min(max(row_pos(a.map, row), 0), a.max_pages * PAGE_TOKENS - 1);
-  const Pages pg = pages_of(m, pos, pos);
-  const int per = (pg.n + cl.splits - 1) / cl.splits, first = split * per, nt = max(0, min(per, pg.n - first));
-  bool ok = true;
-  int loaded = 0;
-  auto load_until = [&](int end) {   // the TMA thread: pages of keys, then of values
-    for (; ok && loaded < end; ++loaded) {
-      const int st = loaded % cl.stages, page = pg.at(first + (loaded < nt ? loaded : loaded - nt));
-      const int n = ((loaded < nt ? m.dim : V) + 63) / 64;
-      if (loaded >= cl.stages) ok = mbar_wait(&empty[st], ((loaded / cl.stages) - 1) & 1, a.status);
-      if (!ok) return;
-      const int y = (a.block_table[(int64_t)seq * a.max_pages + page] * m.kv_heads + hk) * PAGE_TOKENS;
-      mbar_expect_tx(&full[st], n * 8192);
-      for (int b = 0; b < n; ++b) tma_load_2d(smem + st * cl.stage_bytes + b * 8192, loaded < nt ? &tm_k : &tm_v, &full[st], b * 64, y);
-    }
-  };
-  if (warp == 4) {
-    if (lane == 0) {
-      if (a.early_kv) {
-        int early = 0;   // not the page the step writes
-        while (early < min(cl.stages, 2 * nt) && pg.at(first + (early < nt ? early : early - nt)) < pos / PAGE_TOKENS) ++early;
-        load_until(early);
-        pdl_wait();
-      }
-      load_until(min(2 * nt, nt + cl.stages));   // no further: values are read behind the cluster barrier, which this warp joins
-    }
-    __syncwarp();
-  } else {
-    for (int i = tid; i < H * group; i += 128) {   // depends on no earlier kernel
-      const int j = i / group, h = head0 + i % group;
-      sT[i] = m.talk ? m.talk[(int64_t)h * H + j] : j == h ? 1.f : 0.f;
-    }
-    if (a.early_kv) pdl_wait();
-    for (int i = tid; i < 16 * ((m.dim + 63) / 64) * 8; i += 128) {
-      const int hh = i & 15, c = i >> 4;
-      uint4 v = make_uint4(0, 0, 0, 0);
-      if (hh < group && c * 8 < m.dim)   // dim is a multiple of 8
-        v = *reinterpret_cast<const uint4*>(reinterpret_cast<const bf16*>(a.q) + row * a.ldq + (int64_t)(head0 + hh) * m.dim + c * 8);
-      *reinterpret_cast<uint4*>(sQ + (c >> 3) * 2048 + swz128((uint32_t)hh, (uint32_t)(c & 7))) = v;
-    }
-    for (int i = tid; i < group * V; i += 128) {
-      float z = (a.gate_head ? a.gate_head[row * H + head0 + i / V] : 1.0f) * m.out_scale;
-      if (a.gate) {
-        const float* gp = a.gate + row * a.ld + (int64_t)head0 * V + i;
-        float e = 0.f;
-#pragma unroll 4
-        for (int k = 0; k < a.nsplit; ++k) e += gp[k * a.split_stride];
-        z *= sigmoid_act(e);
-      }
-      sG[i] = z;
-    }
-    consumers_sync();
-    const int ks = (m.dim + 15) / 16;
-    uint32_t qf[KS][4];
-    const uint32_t q_base = smem_u32(sQ);
-#pragma unroll
-    for (int k = 0; k < KS; ++k)
-      if (k < ks)
-        ldmatrix_x4(qf[k][0], qf[k][1], qf[k][2], qf[k][3], q_base + (k >> 2) * 2048 + swz128((lq & 1) * 8 + l8, (k & 3) * 2 + (lq >> 1)));
-    const float sl2 = m.scale * LOG2E;
-    const int low = m.window > 0 ? pos - m.window : -1;
-    float mrun[2] = {-INFINITY, -INFINITY}, lrun[2] = {0.f, 0.f};
-    uint32_t k_off[4];
-#pragma unroll
-    for (int u = 0; u < 4; ++u) k_off[u] = swz128(warp * 16 + (lq >> 1) * 8 + l8, u * 2 + (lq & 1));
-    const uint32_t ring = smem_u32(smem);
-    for (int it = 0; it < nt; ++it) {
-      const int st = it % cl.stages;
-      if (ok) ok = mbar_wait(&full[st], (it / cl.stages) & 1, a.status);
-      const uint32_t kp = ring + st * cl.stage_bytes;
-      float sc[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
-#pragma unroll
-      for (int k = 0; k < KS; ++k) {
-        if (k >= ks) break;
-        uint32_t b0, b1, b2, b3;
-        ldmatrix_x4(b0, b1, b2, b3, kp + (k >> 2) * 8192 + k_off[k & 3]);
-        mma_bf16_16816(sc[0], qf[k], b0, b1);
-        mma_bf16_16816(sc[1], qf[k], b2, b3);
-      }
-      __syncwarp();
-      if (lane == 0) mbar_arrive(&empty[st]);
-      const int in_page = warp * 16 + 2 * t, key0 = pg.at(first + it) * PAGE_TOKENS + in_page;
-      float mx[2] = {-INFINITY, -INFINITY};
-#pragma unroll
-      for (int n = 0; n < 2; ++n)
-#pragma unroll
-        for (int e = 0; e < 4; ++e) {
-          const int x = e >> 1, key = key0 + n * 8 + (e & 1);
-          sc[n][e] = key <= pos && (key > low || key < m.keep_first) ? sc[n][e] * sl2 : -INFINITY;
-          mx[x] = fmaxf(mx[x], sc[n][e]);
-        }
-#pragma unroll
-      for (int x = 0; x < 2; ++x) {
-        if (g + 8 * x < group) {
-          float* p = sS + (g + 8 * x) * ldk + it * PAGE_TOKENS + in_page;
-          *reinterpret_cast<float2*>(p) = make_float2(sc[0][2 * x], sc[0][2 * x + 1]);
-          *reinterpret_cast<float2*>(p + 8) = make_float2(sc[1][2 * x], sc[1][2 * x + 1]);
-        }
-        const float mn = fmaxf(mrun[x], mx[x]), use = mn == -INFINITY ? 0.f : mn;
-        lrun[x] = lrun[x] * ex2(mrun[x] - use) + (ex2(sc[0][2 * x] - use) + ex2(sc[0][2 * x + 1] - use)) + (ex2(sc[1][2 * x] - use) + ex2(sc[1][2 * x + 1] - use));
-        mrun[x] = mn;
-      }
-    }
-#pragma unroll
-    for (int x = 0; x < 2; ++x) {
-      float mn = mrun[x];
-      mn = fmaxf(mn, __shfl_xor_sync(0xffffffffu, mn, 1));
-      mn = fmaxf(mn, __shfl_xor_sync(0xffffffffu, mn, 2));
-      lrun[x] *= ex2(mrun[x] - (mn == -INFINITY ? 0.f : mn));
-      lrun[x] += __shfl_xor_sync(0xffffffffu, lrun[x], 1);
-      lrun[x] += __shfl_xor_sync(0xffffffffu, lrun[x], 2);
-      if (t == 0) {
-        sM[warp * 16 + g + 8 * x] = mn;
-        sM[64 + warp * 16 + g + 8 * x] = lrun[x];
-      }
-    }
-    consumers_sync();
-    if (tid < group) {
-      float M = -INFINITY, l = 0.f;
-#pragma unroll
-      for (int w = 0; w < 4; ++w) M = fmaxf(M, sM[w * 16 + tid]);
-      const float use = M == -INFINITY ? 0.f : M;
-#pragma unroll
-      for (int w = 0; w < 4; ++w) l += ex2(sM[w * 16 + tid] - use) * sM[64 + w * 16 + tid];
-      sML[tid] = make_float2(M, l);
-    }
-  }
-  cluster.sync();   // scores and sums of all heads
-  if (warp == 4) {
-    if (lane == 0) load_until(2 * nt);
-    __syncwarp();
-  } else {
-    for (int j = tid; j < H; j += 128) {
-      float M = -INFINITY, l = 0.f;
-      for (int s = 0; s < cl.splits; ++s) M = fmaxf(M, cluster.map_shared_rank(sML, s * m.kv_heads + j / group)[j % group].x);
-      const float use = M == -INFINITY ? 0.f : M;
-      for (int s = 0; s < cl.splits; ++s) {
-        const float2 e = cluster.map_shared_rank(sML, s * m.kv_heads + j / group)[j % group];
-        l += ex2(e.x - use) * e.y;
-      }
-      sN[j] = make_float2(use, l > 0.f ? 1.0f / l : 0.f);
-    }
-    consumers_sync();
-    auto mix = [&](auto n) {   // n: group rounded up
-      constexpr int N = decltype(n)::value;
-      for (int key = tid; key < nt * PAGE_TOKENS; key += 128) {
-        float w[N];
-#pragma unroll
-        for (int hh = 0; hh < N; ++hh) w[hh] = 0.f;
-        for (int c = 0; c < m.kv_heads; ++c) {
-          const float* s = cluster.map_shared_rank(sS, split * m.kv_heads + c) + key;
-          float e[N];
-#pragma unroll
-          for (int u = 0; u < N; ++u) e[u] = u < group ? s[u * ldk] : -INFINITY;
-#pragma unroll
-          for (int u = 0; u < N; ++u) {
-            if (u >= group) break;
-            const int j = c * group + u;
-            const float2 nj = sN[j];
-            const float p = ex2(e[u] - nj.x) * nj.y;
-#pragma unroll
-            for (int hh = 0; hh < N; ++hh)
-              if (hh < group) w[hh] = fmaf(sT[j * group + hh], p, w[hh]);
-          }
-        }
-#pragma unroll
-        for (int hh = 0; hh < N; ++hh)
-          if (hh < group) sP[hh * ldk + key] = __float2bfloat16_rn(w[hh]);
-      }
-    };
-    if (group <= 4) mix(std::integral_constant<int, 4>{});
-    else if (group <= 8) mix(std::integral_constant<int, 8>{});
-    else mix(std::integral_constant<int, 16>{});
-    consumers_sync();
-    // ---- times values: a warp has its columns of all keys; rows past the group repeat its last one and are dropped
-    float acc[VW][2][4];
-#pragma unroll
-    for (int j = 0; j < VW; ++j)
-#pragma unroll
-      for (int e = 0; e < 8; ++e) acc[j][e >> 2][e & 3] = 0.f;
-    const int vg = (V + 15) / 16;
-    const uint32_t ring = smem_u32(smem), pa = smem_u32(sP) + (min((lq & 1) * 8 + l8, group - 1) * ldk + (lq >> 1) * 8) * 2;
-    for (int it = 0; it < nt; ++it) {
-      const int i = nt + it, st = i % cl.stages;
-      if (ok) ok = mbar_wait(&full[st], (i / cl.stages) & 1, a.status);
-      const uint32_t vp = ring + st * cl.stage_bytes;
-#pragma unroll
-      for (int k = 0; k < 4; ++k) {
-        uint32_t pf[4];
-        ldmatrix_x4(pf[0], pf[1], pf[2], pf[3], pa + it * PAGE_TOKENS * 2 + k * 32);
-#pragma unroll
-        for (int j = 0; j < VW; ++j) {
-          const int c = warp * VW + j;
-          if (c >= vg) break;
-          uint32_t v0, v1, v2, v3;
-          ldmatrix_x4_trans(v0, v1, v2, v3, vp + (c >> 2) * 8192 + swz128(k * 16 + (lq & 1) * 8 + l8, (c & 3) * 2 + (lq >> 1)));
-          mma_bf16_16816(acc[j][0], pf, v0, v1);
-          mma_bf16_16816(acc[j][1], pf, v2, v3);
-        }
-      }
-      __syncwarp();
-      if (lane == 0) mbar_arrive(&empty[st]);
-    }
-#pragma unroll
-    for (int x = 0; x < 2; ++x) {
-      const int hh = g + 8 * x;
-      if (hh >= group) continue;
-#pragma unroll
-      for (int j = 0; j < VW; ++j)
-#pragma unroll
-        for (int n = 0; n < 2; ++n) {
-          const int col = (warp * VW + j) * 16 + n * 8 + 2 * t;
-          if (col < V) *reinterpret_cast<float2*>(sO + hh * V + col) = make_float2(acc[j][n][2 * x], acc[j][n][2 * x + 1]);   // vdim is a multiple of 8
-        }
-    }
-  }
-  cluster.sync();   // the sums of all splits; nobody reads scores any more
-  if (warp < 4) {
-    const int units = group * V / 4, share = (units + cl.splits - 1) / cl.splits;
-    for (int u = split * share + tid; u < min((split + 1) * share, units); u += 128) {
-      float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
-      for (int s = 0; s < cl.splits; ++s) {
-        const float4 x = reinterpret_cast<const float4*>(cluster.map_shared_rank(sO, s * m.kv_heads + hk))[u];
-        o.x += x.x; o.y += x.y; o.z += x.z; o.w += x.w;
-      }
-      const float4 ge = reinterpret_cast<const float4*>(sG)[u];
-      *reinterpret_cast<uint2*>(reinterpret_cast<bf16*>(a.out) + row * a.ldo + (int64_t)head0 * V + u * 4) =
-          make_uint2(pack_bf16(o.x * ge.x, o.y * ge.y), pack_bf16(o.z * ge.z, o.w * ge.w));
-    }
-  }
-  if (cl.splits > 1) cluster.sync();   // a peer may still read this CTA's sums
-}
-
 bool mma_ok(const GqaDims& m) {
   return m.dim % 8 == 0 && m.vdim % 8 == 0 && m.dim <= 256 && m.vdim <= 256 && !m.bias && !m.sink && m.heads <= 256;
 }
@@ -860,41 +559,6 @@ size_t gqa_mix_bytes(Ctx* c, const GqaDims& m, int dtype, int64_t rows, int64_t 
 
 namespace {
 
-// Whether a step of single tokens goes to mix_cluster_kernel, and its cluster.
-bool cluster_plan(Ctx* c, const GqaDims& m, int64_t tiles, int64_t pages, MixCluster& cl) {
-  if (m.kv_heads > 8 || (m.kv_heads & (m.kv_heads - 1)) || m.heads / m.kv_heads > 16) return false;
-  cl.stage_bytes = (std::max(m.dim, m.vdim) + 63) / 64 * 8192;
-  cl.splits = 8 / m.kv_heads;
-  while (cl.splits > pages) cl.splits /= 2;
-  cl.keys = (int)((pages + cl.splits - 1) / cl.splits * PAGE_TOKENS);
-  cl.stages = 0;
-  const size_t rest = mix_cluster_smem(m, cl).end + 1024;
-  const bool two = tiles * m.kv_heads * cl.splits > c->sm_count;   // two CTAs per SM
-  for (const size_t room : {(size_t)(two ? 110 : 220) * 1024, (size_t)220 * 1024}) {
-    if (rest >= room) continue;
-    cl.stages = (int)std::min<size_t>({(room - rest) / cl.stage_bytes, (size_t)(2 * cl.keys / PAGE_TOKENS), (size_t)16});
-    if (cl.stages >= 3 || cl.stages == 2 * cl.keys / PAGE_TOKENS) return true;
-  }
-  return false;
-}
-
-int cluster_launch(Ctx* c, const GqaMixArgs& a, const MixCluster& cl) {
-  const int ks = (a.m.dim + 15) / 16, vg = (a.m.vdim + 15) / 16;
-  const size_t smem = mix_cluster_smem(a.m, cl).end + 1024;
-  const int n = a.m.kv_heads * cl.splits;
-  auto go = [&](auto kernel) -> int {
-    if (smem > 48 * 1024) RB_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
-    RB_CUDA(launch_k_cluster(kernel, dim3((unsigned)n, (unsigned)a.tiles.count), dim3(160), smem, c->stream, c->use_pdl, dim3((unsigned)n), *a.tm_k, *a.tm_v, a, cl));
-    ++g_launch_total;
-    return REWB200_OK;
-  };
-  auto by_v = [&](auto k) -> int {
-    constexpr int KS = decltype(k)::value;
-    return vg <= 4 ? go(mix_cluster_kernel<KS, 1>) : vg <= 8 ? go(mix_cluster_kernel<KS, 2>) : go(mix_cluster_kernel<KS, 4>);
-  };
-  return ks <= 4 ? by_v(std::integral_constant<int, 4>{}) : ks <= 8 ? by_v(std::integral_constant<int, 8>{}) : by_v(std::integral_constant<int, 16>{});
-}
-
 int plain_launch(Ctx* c, const GqaMixArgs& a) {
   const int64_t slots = most_seen(a.m, (int64_t)a.max_pages * PAGE_TOKENS);
   const int64_t piece = std::min<int64_t>(a.rows, (int64_t)(a.work_bytes / ((size_t)a.m.heads * slots * sizeof(float))));
@@ -917,10 +581,8 @@ int plain_launch(Ctx* c, const GqaMixArgs& a) {
 int gqa_mix_launch(Ctx* c, const GqaMixArgs& a) {
   if (a.tiles.count == 0) return REWB200_OK;
   if (a.dtype != REWB200_BF16 || c->gqa_impl == 1 || !mma_ok(a.m)) return plain_launch(c, a);
-  const int64_t pages = most_pages(a.m, a.max_tile_rows, a.max_pages);
-  MixCluster cl = {};
-  if (a.max_tile_rows == 1 && c->gqa_impl == 0 && cluster_plan(c, a.m, a.tiles.count, pages, cl)) return cluster_launch(c, a, cl);
   MixCfg cf = config(a.m, a.max_tile_rows);
+  const int64_t pages = most_pages(a.m, a.max_tile_rows, a.max_pages);
   cf.slots = pages * PAGE_TOKENS;
   cf.splits = splits_of(c, a.m, cf, a.tiles.count, pages);
   const size_t per = row_bytes(a.m, cf.slots, cf.splits);
