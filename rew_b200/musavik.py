@@ -82,4 +82,4 @@ def dense_8b(**kw):
                      beside=delta, beside_names=("left.", "right."), **ff)
     lru = LayerSpec(mixer="lru", heads=12, dim=256, vdim=256, conv_taps=4, **ff)
     return LayeredConfig(**{**dict(vocab=128256, d_model=4096, layers=[both if i % 2 else lru for i in range(32)], eps=1e-5, block="sandwich",
-                                   own_head=True, embed_scale=64.0, bigram=(16384, 31, 17), max_seq=2560, dtype=_lib.BF16), **kw})
+                                   own_head=True, embed_scale=64.0, bigram=(16384, 1009, 7), max_seq=2560, dtype=_lib.BF16), **kw})
