@@ -266,7 +266,7 @@ def test_freed_pages_and_states_hold_nothing_over(rb):
 
 def test_the_last_token_belongs_to_its_lane(rb, dtype):
     """Bigram rows across steps that interleave lanes, and after a lane was given to another request."""
-    cfg = K.config([K.rglru(None, width=16, blocks=1, conv=1)], bigram=(1009, 31, 17))
+    cfg = K.config([K.rglru(None, width=16, blocks=1, conv=1)], bigram=(1009, 29, 13))
     t = {k: v.copy() for k, v in K.weights(cfg, seed=16).items()}
     t["bigram"] *= 4.0
     t["l0.mix.o"][:] = 0.0
